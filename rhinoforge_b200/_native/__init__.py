@@ -184,6 +184,56 @@ class RfGdn(C.Structure):
                 ("fresh", C.c_void_p)] + [(n, C.c_int32) for n in ("num_seqs", "Hk", "Hv", "Dk", "Dv", "dtype")]
 
 
+class RfRows(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("seq_of_row", "q_start", "q_len", "slot", "pos", "page_table")] + \
+               [("pt_stride", C.c_int32), ("num_seqs", C.c_int32)]
+
+
+class RfStreamNorm(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("x", "table", "ids", "row_idx", "y", "y_norm_w", "x_out", "x_cast", "norm_w", "out",
+                                          "shift", "shift_state")] + [("rows", RfRows)] + \
+               [("n_rows", C.c_int32), ("H", C.c_int32), ("dim", C.c_int32), ("eps", C.c_float), ("dtype", C.c_int32)]
+
+
+class RfHeadLinear(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64), ("xs", C.c_int32), ("y", C.c_void_p), ("ldy", C.c_int64),
+                ("ys", C.c_int32), ("w", C.c_void_p)] + [(n, C.c_int32) for n in ("rows", "heads", "n", "k", "dtype")]
+
+
+class RfLatentAttn(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("o", C.c_void_p), ("pool", C.c_void_p), ("rows", RfRows)] + \
+               [(n, C.c_int32) for n in ("n_rows", "heads", "rank", "window", "max_kv")] + \
+               [("scale", C.c_float), ("dtype", C.c_int32), ("ws", C.c_void_p), ("ws_bytes", C.c_uint64)]
+
+
+class RfHgrn2(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64), ("f_off", C.c_int32), ("v_off", C.c_int32), ("f_bias", C.c_void_p),
+                ("lower", C.c_void_p), ("norm_w", C.c_void_p), ("state", C.c_void_p), ("out", C.c_void_p), ("ldo", C.c_int64),
+                ("rows", RfRows)] + [(n, C.c_int32) for n in ("heads", "dim", "vdim", "vdim_true")] + \
+               [("eps", C.c_float), ("dtype", C.c_int32)]
+
+
+class RfMixedConfig(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("layers", "hidden", "hidden_true", "vocab", "vocab_ld", "dtype", "max_tokens", "max_seqs",
+                                         "max_seq_len", "side_dim")] + \
+               [("side_ld", C.c_int64), ("eps", C.c_float), ("weights_packed", C.c_int32), ("long_min", C.c_int32)] + \
+               [(n, C.c_void_p) for n in ("embed", "side_table", "final_norm", "w_lm")]
+
+
+class RfMixedLayer(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "vdim", "vdim_true", "rank", "rank_true", "window", "expand_hd",
+                                         "inter", "act")] + [("scale", C.c_float), ("in_dim", C.c_int32)] + \
+               [(n, C.c_void_p) for n in ("norm1", "norm2", "shift", "shift_state", "w_in", "w_o", "w_up", "w_down", "latent_norm",
+                                          "w_absorb", "w_unabsorb", "w_expand", "latent_pool", "f_bias", "lower", "head_norm",
+                                          "rec_state", "side_gate", "side_proj", "side_norm")]
+
+
+class RfMixedForward(C.Structure):
+    _fields_ = [("ids", C.c_void_p), ("rows", RfRows)] + \
+               [(n, C.c_int32) for n in ("tokens", "short_seqs", "short_rows", "decode", "max_kv")] + \
+               [(n, C.c_void_p) for n in ("h_q_len", "h_pos0", "taps")]
+
+
 def available() -> bool:
     return LIB_PATH.exists()
 
@@ -212,6 +262,10 @@ def lib() -> C.CDLL:
         l.rf_stack_arena_bytes.restype = C.c_uint64
         l.rf_stack_status_ptr.restype = C.c_void_p
         l.rf_kvpool_create.restype = C.c_int64
+        l.rf_mixed_create.restype = C.c_int64
+        l.rf_mixed_arena_bytes.restype = C.c_uint64
+        l.rf_mixed_status_ptr.restype = C.c_void_p
+        l.rf_latent_attn_scratch_bytes.restype = C.c_uint64
         l.rf_pack_weight_bytes.restype = C.c_uint64
         l.rf_pack_w4_bytes.restype = C.c_uint64
         l.rf_pack_w4_bytes.argtypes = [C.c_int64, C.c_int64, C.c_int32, C.c_int32]

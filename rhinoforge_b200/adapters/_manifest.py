@@ -10,6 +10,7 @@ BUILTIN_ADAPTERS = (
     ("SiglipVisionModel", "rhinoforge_b200.adapters.siglip", "SiglipAdapter"),
     ("Qwen3_5ForConditionalGeneration", "rhinoforge_b200.adapters.qwen3_5", "Qwen3_5Adapter"),
     ("Qwen3VLForConditionalGeneration", "rhinoforge_b200.adapters.qwen3_vl", "Qwen3VLAdapter"),
+    ("Vabarax", "rhinoforge_b200.adapters.vabarax", "VabaraxAdapter"),
 )
 
 __all__ = ["BUILTIN_ADAPTERS"]

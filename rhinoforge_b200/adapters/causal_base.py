@@ -125,23 +125,19 @@ class CausalLMAdapter:
         """Pack the weights once, create the native runtime and return the runtime handle."""
         if self._handle is not None:
             return self._handle
-        if self._dtype not in (torch.float16, torch.bfloat16):
-            raise RPUUnsupportedDtypeError(f"kernels take float16 or bfloat16, got {self._dtype}")
+        self._check_dtype()
         if not _PACK_LOCK.acquire(blocking=False):
             raise RPUBackendError("another model is being packed for the accelerator in this process")
         try:
             owner = self.model if self.model is not None else self
             live_handle.claim(owner)
             from ..runtime.causal_lm import RPUCausalLM
-            from ..runtime.engine import DecoderEngine
             cfg = self.decoder_config()
             get = self._weights()
             self._validate_shapes(cfg, get)
-            chunk = prefill_chunk_rows(self._rpu_execution)
             quant = "w8a16" if config_is_w8a16(self.config) else None
             try:
-                engine = DecoderEngine(cfg, get, dtype=self._dtype, max_batch=max_batch, max_seq_len=16,
-                                       max_prefill_tokens=chunk, tp=tp, quant=quant)
+                engine = self._build_engine(cfg, get, max_batch=max_batch, tp=tp, quant=quant)
             except Exception as e:
                 live_handle.poison(owner, f"{type(self).__name__}.to_rpu failed after weight packing began: {e}")
                 raise
@@ -150,6 +146,15 @@ class CausalLMAdapter:
             return self._handle
         finally:
             _PACK_LOCK.release()
+
+    def _check_dtype(self) -> None:
+        if self._dtype not in (torch.float16, torch.bfloat16):
+            raise RPUUnsupportedDtypeError(f"kernels take float16 or bfloat16, got {self._dtype}")
+
+    def _build_engine(self, cfg: DecoderConfig, get, *, max_batch: int, tp=None, quant: Optional[str] = None):
+        from ..runtime.engine import DecoderEngine
+        return DecoderEngine(cfg, get, dtype=self._dtype, max_batch=max_batch, max_seq_len=16,
+                             max_prefill_tokens=prefill_chunk_rows(self._rpu_execution), tp=tp, quant=quant)
 
     def _validate_shapes(self, cfg: DecoderConfig, get) -> None:
         names = getattr(get, "names", None)

@@ -19,7 +19,21 @@ _ROUTES = {
     "Qwen3VLForConditionalGeneration": "use RPUModelForConditionalGeneration.from_pretrained(...)",
     "LlamaForCausalLM": "use RPUModelForCausalLM.from_pretrained(...) and .to('rpu')",
     "Qwen3ForCausalLM": "use RPUModelForCausalLM.from_pretrained(...) and .to('rpu')",
+    "Vabarax": "use RPUModelForCausalLM.from_pretrained(..., device='rpu')",
 }
+
+
+def local_native_config(path):
+    """The raw ``config.json`` mapping of a local checkpoint folder that names its design under ``architecture`` (configurations
+    Hugging Face does not know), else None."""
+    f = Path(path) / "config.json"
+    if not f.is_file():
+        return None
+    try:
+        raw = json.loads(f.read_text(encoding="utf-8"))
+    except ValueError as e:
+        raise UnsupportedModelError(f"{str(f)!r} is not valid JSON: {e}") from e
+    return raw if isinstance(raw, dict) and isinstance(raw.get("architecture"), str) and "architectures" not in raw else None
 
 
 def resolve_loader_device(device, *, entry_point: str) -> bool:
@@ -73,8 +87,15 @@ def checkpoint_tensor_getter(path: str) -> Callable[[str], torch.Tensor]:
             handles[shard] = safe_open(str(root / shard), framework="pt")
         return handles[shard].get_tensor(name)
 
+    def shape(name: str):
+        shard = weight_map[name]
+        if shard not in handles:
+            handles[shard] = safe_open(str(root / shard), framework="pt")
+        return handles[shard].get_slice(name).get_shape()
+
     get.names = frozenset(weight_map)  # type: ignore[attr-defined]
+    get.shape = shape  # type: ignore[attr-defined]
     return get
 
 
-__all__ = ["resolve_loader_device", "resolve_config_architecture", "checkpoint_tensor_getter"]
+__all__ = ["resolve_loader_device", "resolve_config_architecture", "local_native_config", "checkpoint_tensor_getter"]

@@ -18,6 +18,7 @@ import torch
 from ..runtime.control import rpu_env_int
 from ..runtime.device import resolve_device
 from ..runtime.kv_cache import PagedKV
+from ..runtime.mixed_cache import MixedCache
 
 try:  # the HF base class is optional
     from transformers.cache_utils import Cache as _HFCache
@@ -40,27 +41,9 @@ def _padding_room(model) -> int:
     return rpu_env_int("RPU_CAUSAL_PREFILL_PADDING_BUDGET", 64)
 
 
-class RPUCache(PagedKV, _HFCache):
+class _CacheProtocol:
+    """Position bookkeeping and the Hugging Face ``Cache`` protocol over a paged sequence store."""
     is_sliding_window = False
-
-    def __init__(self, num_layers: int, batch_size: int, max_seq_len: int, num_kv_heads: int, head_dim: int,
-                 device="rpu", dtype: torch.dtype = torch.float16, attn_tp: int = 1):
-        if dtype not in (torch.float16, torch.bfloat16):
-            raise ValueError(f"RPUCache dtype must be torch.float16 or torch.bfloat16, got {dtype}")
-        if isinstance(attn_tp, bool) or not isinstance(attn_tp, int) or attn_tp <= 0:
-            raise ValueError(f"RPUCache attn_tp must be a positive integer, got {attn_tp!r}")
-        try:
-            dev = resolve_device(device) if not str(device).startswith("cpu") else torch.device("cpu")
-        except (TypeError, ValueError) as exc:
-            raise ValueError(f"RPUCache invalid device {device!r}") from exc
-        if dev.type not in ("cpu", "cuda"):
-            raise ValueError(f"RPUCache device must be cpu, rpu or cuda; got {device!r}")
-        local_heads = max(1, num_kv_heads // attn_tp) if num_kv_heads >= attn_tp else 1
-        PagedKV.__init__(self, num_layers, batch_size, max_seq_len, local_heads, head_dim, device=dev, dtype=dtype)
-        self.total_kv_heads = num_kv_heads
-        self.attn_tp = attn_tp
-        self._seen_tokens = 0
-        self.layers = []
 
     # -- the single length source ------------------------------------------------------------
     @property
@@ -122,6 +105,28 @@ class RPUCache(PagedKV, _HFCache):
     def seen_tokens(self) -> int:
         return self._seen_tokens
 
+
+class RPUCache(_CacheProtocol, PagedKV, _HFCache):
+
+    def __init__(self, num_layers: int, batch_size: int, max_seq_len: int, num_kv_heads: int, head_dim: int,
+                 device="rpu", dtype: torch.dtype = torch.float16, attn_tp: int = 1):
+        if dtype not in (torch.float16, torch.bfloat16):
+            raise ValueError(f"RPUCache dtype must be torch.float16 or torch.bfloat16, got {dtype}")
+        if isinstance(attn_tp, bool) or not isinstance(attn_tp, int) or attn_tp <= 0:
+            raise ValueError(f"RPUCache attn_tp must be a positive integer, got {attn_tp!r}")
+        try:
+            dev = resolve_device(device) if not str(device).startswith("cpu") else torch.device("cpu")
+        except (TypeError, ValueError) as exc:
+            raise ValueError(f"RPUCache invalid device {device!r}") from exc
+        if dev.type not in ("cpu", "cuda"):
+            raise ValueError(f"RPUCache device must be cpu, rpu or cuda; got {device!r}")
+        local_heads = max(1, num_kv_heads // attn_tp) if num_kv_heads >= attn_tp else 1
+        PagedKV.__init__(self, num_layers, batch_size, max_seq_len, local_heads, head_dim, device=dev, dtype=dtype)
+        self.total_kv_heads = num_kv_heads
+        self.attn_tp = attn_tp
+        self._seen_tokens = 0
+        self.layers = []
+
     def get_cache(self, layer_idx: int):
         return self.kv[layer_idx, 0], self.kv[layer_idx, 1]
 
@@ -168,6 +173,9 @@ class RPUCache(PagedKV, _HFCache):
             need = prompt + int(max_new_tokens) + _padding_room(model) + 1
         else:
             need = int(max_seq_len)
+        make = getattr(getattr(model, "engine", None), "make_cache", None)
+        if make is not None:            # decoders whose per-sequence state is more than K/V pages bring their own cache
+            return make(batch_size, (need + 15) // 16 * 16)
         cfg = getattr(model, "config", None)
         text = getattr(cfg, "text_config", cfg)
         if text is None:
@@ -196,4 +204,34 @@ class RPUCache(PagedKV, _HFCache):
         return out
 
 
-__all__ = ["RPUCache"]
+class RPUMixedCache(_CacheProtocol, MixedCache, _HFCache):
+    """Cache of a decoder with per-layer mixers (latent pages, recurrent states, token-shift rows).  Recurrent state summarises
+    the whole prefix: it can be reset, not rewound."""
+
+    def __init__(self, cfg, batch_size: int, max_seq_len: int, *, device="rpu", dtype: torch.dtype = torch.bfloat16,
+                 pool_tokens: Optional[int] = None):
+        dev = resolve_device(device) if not str(device).startswith("cpu") else torch.device("cpu")
+        MixedCache.__init__(self, cfg, batch_size, max_seq_len, device=dev, dtype=dtype, pool_tokens=pool_tokens)
+        self._seen_tokens = 0
+        self.layers = []
+
+    def reset(self) -> None:
+        self.position = 0
+        self._seen_tokens = 0
+
+    def reset_to_position(self, pos: int) -> None:
+        if pos not in (0, self.position):
+            raise ValueError("RPUMixedCache cannot rewind to a non-zero position: recurrent states summarise the whole prefix. "
+                             "Call reset() and prefill again.")
+        if pos == 0:
+            self.reset()
+
+    def __len__(self) -> int:
+        return self.num_layers
+
+    def __repr__(self) -> str:
+        return (f"RPUMixedCache(num_layers={self.num_layers}, batch_size={self.batch_size}, max_seq_len={self.max_seq_len}, "
+                f"position={self.position})")
+
+
+__all__ = ["RPUCache", "RPUMixedCache"]

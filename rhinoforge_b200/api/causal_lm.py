@@ -17,7 +17,7 @@ import torch
 from ..runtime import live_handle
 from ..runtime.registry import get_adapter
 from ._execution import normalize_rpu_execution
-from ._loading import checkpoint_tensor_getter, resolve_config_architecture, resolve_loader_device
+from ._loading import checkpoint_tensor_getter, local_native_config, resolve_config_architecture, resolve_loader_device
 from .errors import RPUUnsupportedDtypeError, UnsupportedModelError
 
 _claim_live_instance = live_handle.claim
@@ -29,7 +29,7 @@ class RPUModelForCausalLM:
 
     _RESERVED_HF_KWARGS = frozenset({"torch_dtype", "dtype", "device_map", "device", "low_cpu_mem_usage", "tp_plan",
                                      "load_in_8bit", "load_in_4bit", "quantization_config"})
-    _SUPPORTED_BUILTIN_ARCHITECTURES = frozenset({"LlamaForCausalLM", "Qwen3ForCausalLM"})
+    _SUPPORTED_BUILTIN_ARCHITECTURES = frozenset({"LlamaForCausalLM", "Qwen3ForCausalLM", "Vabarax"})
     _CONFIG_KWARGS = frozenset({"cache_dir", "revision", "subfolder", "local_files_only", "token", "force_download",
                                 "proxies"})
     SUPPORTED_DTYPES = (torch.float16, torch.bfloat16)
@@ -40,7 +40,9 @@ class RPUModelForCausalLM:
         ep = "RPUModelForCausalLM.from_pretrained"
         execution = normalize_rpu_execution(rpu_execution, entry_point=ep,
                                             supported={"prefill": ("chunk_size", "padding_rows", "padding_budget")})
-        if dtype not in cls.SUPPORTED_DTYPES:
+        native = local_native_config(hf_repo_or_path) if os.path.isdir(hf_repo_or_path) else None
+        native_cls = get_adapter(native["architecture"]) if native is not None else None
+        if dtype not in getattr(native_cls, "SUPPORTED_DTYPES", cls.SUPPORTED_DTYPES):
             raise RPUUnsupportedDtypeError(f"the kernels take torch.float16 or torch.bfloat16, got {dtype}. Load the "
                                            "CPU reference separately if you need an fp32 baseline for comparison.")
         clash = cls._RESERVED_HF_KWARGS & set(hf_kwargs)
@@ -50,12 +52,17 @@ class RPUModelForCausalLM:
         if hf_kwargs.pop("trust_remote_code", False) is not False:
             raise ValueError(f"{ep} requires trust_remote_code=False; custom model code is not supported.")
         to_rpu = resolve_loader_device(device, entry_point=ep)
-        from transformers import AutoConfig
         cfg_kwargs = {k: v for k, v in hf_kwargs.items() if k in cls._CONFIG_KWARGS}
-        try:
-            config = AutoConfig.from_pretrained(hf_repo_or_path, trust_remote_code=False, **cfg_kwargs)
-        except (OSError, ValueError) as e:
-            raise UnsupportedModelError(f"Could not load HF config for {hf_repo_or_path!r}: {type(e).__name__}: {e}.") from e
+        if native_cls is not None:
+            if not to_rpu:
+                raise UnsupportedModelError(f"{ep}: {native['architecture']} has no host-side model; pass device='rpu'")
+            config = native_cls.config_from_dict(native)
+        else:
+            from transformers import AutoConfig
+            try:
+                config = AutoConfig.from_pretrained(hf_repo_or_path, trust_remote_code=False, **cfg_kwargs)
+            except (OSError, ValueError) as e:
+                raise UnsupportedModelError(f"Could not load HF config for {hf_repo_or_path!r}: {type(e).__name__}: {e}.") from e
         arch = resolve_config_architecture(config, source=hf_repo_or_path, entry_point=ep,
                                            supported_builtins=cls._SUPPORTED_BUILTIN_ARCHITECTURES)
         adapter_cls = get_adapter(arch)

@@ -34,7 +34,17 @@ template <> struct Num<__nv_bfloat16> {
   }
 };
 
-// 8 x 16-bit values in one 16-byte register quad.
+// 32-bit storage: the same helpers, no rounding.
+template <> struct Num<float> {
+  static constexpr int kFmt = 2;
+  using T2 = float2;
+  static __device__ __forceinline__ float to_f(float v) { return v; }
+  static __device__ __forceinline__ float from_f(float v) { return v; }
+  static __device__ __forceinline__ float2 to_f2(float2 v) { return v; }
+  static __device__ __forceinline__ float2 from_f2(float a, float b) { return make_float2(a, b); }
+};
+
+// 8 values: one 16-byte register quad of 16-bit values, or two of 32-bit ones.
 template <typename T> struct alignas(16) Vec8 {
   typename Num<T>::T2 v[4];
 };
@@ -76,6 +86,11 @@ __device__ __forceinline__ float gelu_erf_f(float x) {
   return 0.5f * x * (1.0f + erff(x * 0.7071067811865476f));
 }
 
+__device__ __forceinline__ float relu2_f(float x) {
+  const float r = fmaxf(x, 0.f);
+  return r * r;
+}
+
 enum Act : int32_t {
   kActNone = 0,
   kActSiluMul = 1,      // dual accumulator: silu(g) * u
@@ -83,6 +98,7 @@ enum Act : int32_t {
   kActGeluTanh = 3,
   kActGeluErf = 4,
   kActSilu = 5,
+  kActRelu2 = 6,        // relu(g)^2
 };
 
 __device__ __forceinline__ float apply_act(int act, float g, float u) {
@@ -92,6 +108,7 @@ __device__ __forceinline__ float apply_act(int act, float g, float u) {
     case kActGeluTanh: return gelu_tanh_f(g);
     case kActGeluErf: return gelu_erf_f(g);
     case kActSilu: return silu_f(g);
+    case kActRelu2: return relu2_f(g);
     default: return g;
   }
 }
@@ -222,6 +239,10 @@ __device__ __forceinline__ void apply_act_n(int act, const float (&g)[N], const 
     case kActSilu:
 #pragma unroll
       for (int j = 0; j < N; ++j) v[j] = silu_f(g[j]);
+      break;
+    case kActRelu2:
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[j] = relu2_f(g[j]);
       break;
     default:
 #pragma unroll

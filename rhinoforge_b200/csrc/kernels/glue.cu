@@ -265,7 +265,8 @@ extern "C" int rf_argmax(const void* logits, int rows, int V, int64_t ld, int32_
   const int chunks = (V + kArgmaxChunk - 1) / kArgmaxChunk;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   dim3 g1(chunks, rows);
-  RF_DISPATCH_T(dtype, RF_CUDA_CHECK(::rf::launch_k(argmax_stage1<T>, dim3(g1), dim3(256), 0, s, 1, (const T*)logits, V, ld, (ArgPair*)scratch, chunks)));
+  if (dtype == kF32) RF_CUDA_CHECK(::rf::launch_k(argmax_stage1<float>, dim3(g1), dim3(256), 0, s, 1, (const float*)logits, V, ld, (ArgPair*)scratch, chunks));
+  else RF_DISPATCH_T(dtype, RF_CUDA_CHECK(::rf::launch_k(argmax_stage1<T>, dim3(g1), dim3(256), 0, s, 1, (const T*)logits, V, ld, (ArgPair*)scratch, chunks)));
   RF_CUDA_CHECK(::rf::launch_k(argmax_stage2, dim3(rows), dim3(128), 0, s, 1, (const ArgPair*)scratch, chunks, out_ids, out_vals, offset));
   RF_CUDA_CHECK(cudaGetLastError());
   ::rf::count_launch();

@@ -1,0 +1,250 @@
+// The fp32 residual stream between sublayers (pending sublayer output added, optionally normalised; RMSNorm; token shift),
+// the per-token gate of a side input, and the fp32 GEMM of models served in 32 bits.
+#include "../common/dtype.cuh"
+#include "../common/host_util.h"
+#include "../common/ptx.cuh"
+#include "../rf_api.h"
+
+namespace rf {
+
+__device__ __forceinline__ float stream_block_sum(float v, float* red) {
+  v = warp_sum(v);
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = (blockDim.x + 31) >> 5;
+  __syncthreads();
+  if (l == 0) red[w] = v;
+  __syncthreads();
+  float t = 0.f;
+  for (int i = 0; i < nw; ++i) t += red[i];       // every thread adds the same values in the same order
+  return t;
+}
+
+template <typename T> struct alignas(sizeof(T) * 4) Quad { T v[4]; };
+template <typename T>
+__device__ __forceinline__ float4 load4(const T* p) {
+  const Quad<T> q = *reinterpret_cast<const Quad<T>*>(p);
+  return make_float4(Num<T>::to_f(q.v[0]), Num<T>::to_f(q.v[1]), Num<T>::to_f(q.v[2]), Num<T>::to_f(q.v[3]));
+}
+template <typename T>
+__device__ __forceinline__ void store4(T* p, float4 f) {
+  Quad<T> q;
+  q.v[0] = Num<T>::from_f(f.x); q.v[1] = Num<T>::from_f(f.y); q.v[2] = Num<T>::from_f(f.z); q.v[3] = Num<T>::from_f(f.w);
+  *reinterpret_cast<Quad<T>*>(p) = q;
+}
+__device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+
+// A CTA walks rows_per_cta neighbouring rows.  A thread always touches the same columns, so the shared copies of the
+// current row (xs) and of the previous token's normalised row (hp) need no barriers of their own.
+template <typename T>
+__global__ void stream_norm_kernel(const RfStreamNorm p, int rows_per_cta) {
+  pdl_prologue();
+  extern __shared__ __align__(16) float sm[];
+  float* xs = sm;
+  float* hp = sm + p.H;
+  float* red = hp + (p.shift ? p.H : 0);
+  const int H = p.H, step = blockDim.x * 4, c0 = threadIdx.x * 4;
+  const float inv_dim = 1.f / (float)p.dim;
+  const T* table = reinterpret_cast<const T*>(p.table);
+  const T* y = reinterpret_cast<const T*>(p.y);
+
+  // loads row r into xs with the pending output added, returns 1 / rms of it (when the row is normalised)
+  auto load_row = [&](int r, bool write) -> float {
+    const int src = p.row_idx ? p.row_idx[r] : r;
+    float yr = 1.f;
+    if (y && p.y_norm_w) {
+      float s = 0.f;
+      for (int i = c0; i < H; i += step) s += sq4(load4(y + (size_t)src * H + i));
+      yr = rsqrtf(stream_block_sum(s, red) * inv_dim + p.eps);
+    }
+    const float* xr = p.x ? p.x + (size_t)src * H : nullptr;
+    const T* er = p.x ? nullptr : table + (size_t)p.ids[src] * H;
+    float s = 0.f;
+    for (int i = c0; i < H; i += step) {
+      float4 v = xr ? *reinterpret_cast<const float4*>(xr + i) : load4(er + i);
+      if (y) {
+        float4 a = load4(y + (size_t)src * H + i);
+        if (p.y_norm_w) {
+          const float4 w = *reinterpret_cast<const float4*>(p.y_norm_w + i);
+          a.x *= yr * w.x; a.y *= yr * w.y; a.z *= yr * w.z; a.w *= yr * w.w;
+        }
+        v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+      }
+      *reinterpret_cast<float4*>(xs + i) = v;
+      s += sq4(v);
+      if (write) {
+        if (p.x_out) *reinterpret_cast<float4*>(p.x_out + (size_t)r * H + i) = v;
+        if (p.x_cast) store4(reinterpret_cast<T*>(p.x_cast) + (size_t)r * H + i, v);
+      }
+    }
+    return p.norm_w ? rsqrtf(stream_block_sum(s, red) * inv_dim + p.eps) : 1.f;
+  };
+  auto normed = [&](int i, float rstd) -> float4 {
+    const float4 v = *reinterpret_cast<const float4*>(xs + i), w = *reinterpret_cast<const float4*>(p.norm_w + i);
+    return make_float4(v.x * rstd * w.x, v.y * rstd * w.y, v.z * rstd * w.z, v.w * rstd * w.w);
+  };
+
+  const int r0 = blockIdx.x * rows_per_cta, r1 = min(p.n_rows, r0 + rows_per_cta);
+  for (int r = r0; r < r1; ++r) {
+    float* state = nullptr;
+    bool state_here = false;
+    if (p.shift) {
+      const int seq = p.rows.seq_of_row ? p.rows.seq_of_row[r] : r;
+      const int q0 = p.rows.q_start ? p.rows.q_start[seq] : r;
+      if (r == q0) {
+        // first row of its sequence in this launch: the carried row is read here and replaced here, by the CTA that
+        // read it (the sequence's last row is normalised a second time for that)
+        const int n = p.rows.q_len ? p.rows.q_len[seq] : 1;
+        state = p.shift_state + (size_t)(p.rows.slot ? p.rows.slot[seq] : seq) * H;
+        const bool fresh = p.rows.pos[r] == 0;
+        for (int i = c0; i < H; i += step)
+          *reinterpret_cast<float4*>(hp + i) = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(state + i);
+        if (n > 1) {
+          const float rl = load_row(r + n - 1, false);
+          for (int i = c0; i < H; i += step) *reinterpret_cast<float4*>(state + i) = normed(i, rl);
+        } else {
+          state_here = true;
+        }
+      } else if (r == r0) {
+        const float rl = load_row(r - 1, false);
+        for (int i = c0; i < H; i += step) *reinterpret_cast<float4*>(hp + i) = normed(i, rl);
+      }
+    }
+    const float rstd = load_row(r, true);
+    if (!p.norm_w) continue;
+    T* out = reinterpret_cast<T*>(p.out) + (size_t)r * H;
+    for (int i = c0; i < H; i += step) {
+      float4 h = normed(i, rstd);
+      if (p.shift) {
+        const float4 b = *reinterpret_cast<const float4*>(hp + i), mu = *reinterpret_cast<const float4*>(p.shift + i);
+        *reinterpret_cast<float4*>(hp + i) = h;
+        if (state_here) *reinterpret_cast<float4*>(state + i) = h;
+        h.x += (b.x - h.x) * mu.x; h.y += (b.y - h.y) * mu.y; h.z += (b.z - h.z) * mu.z; h.w += (b.w - h.w) * mu.w;
+      }
+      store4(out + i, h);
+    }
+  }
+}
+
+template <typename T>
+__global__ void token_gate_kernel(T* __restrict__ g, int64_t ldg, const T* __restrict__ table, int64_t ldt,
+                                  const int32_t* __restrict__ ids, int col0, int rows, int cols) {
+  pdl_prologue();
+  const int per = cols / 8;
+  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= (int64_t)rows * per) return;
+  const int r = (int)(i / per), c = (int)(i % per) * 8;
+  float a[8], b[8];
+  load8(g + (size_t)r * ldg + c, a);
+  load8(table + (size_t)ids[r] * ldt + col0 + c, b);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) a[j] *= b[j];
+  store8(g + (size_t)r * ldg + c, a);
+}
+
+// ------------------------------------------------------------------ fp32 GEMM ----
+constexpr int kFBM = 64, kFBN = 64, kFBK = 16;
+
+__device__ __forceinline__ float act_f32(int act, float v) {
+  switch (act) {
+    case kActRelu2: return relu2_f(v);
+    case kActSilu: return v / (1.f + expf(-v));
+    case kActGeluTanh: return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
+    case kActGeluErf: return 0.5f * v * (1.f + erff(v * 0.7071067811865476f));
+    default: return v;
+  }
+}
+
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ x, int64_t ldx, const float* __restrict__ w,
+                                                       int64_t ldw, float* __restrict__ out, int64_t ldo, int M, int N,
+                                                       int K, int act) {
+  pdl_prologue();
+  __shared__ __align__(16) float sx[kFBK][kFBM + 4], sw[kFBK][kFBN + 4];
+  const int n0 = blockIdx.x * kFBN, m0 = blockIdx.y * kFBM, tid = threadIdx.x;
+  const int tx = tid % 16, ty = tid / 16, lr = tid / 4, lk = (tid % 4) * 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += kFBK) {
+    const bool kin = k0 + lk < K;            // K is a multiple of 4
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
+    if (kin && m0 + lr < M) a = *reinterpret_cast<const float4*>(x + (size_t)(m0 + lr) * ldx + k0 + lk);
+    if (kin && n0 + lr < N) b = *reinterpret_cast<const float4*>(w + (size_t)(n0 + lr) * ldw + k0 + lk);
+    sx[lk][lr] = a.x; sx[lk + 1][lr] = a.y; sx[lk + 2][lr] = a.z; sx[lk + 3][lr] = a.w;
+    sw[lk][lr] = b.x; sw[lk + 1][lr] = b.y; sw[lk + 2][lr] = b.z; sw[lk + 3][lr] = b.w;
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kFBK; ++k) {
+      const float4 av = *reinterpret_cast<const float4*>(&sx[k][ty * 4]), bv = *reinterpret_cast<const float4*>(&sw[k][tx * 4]);
+      const float am[4] = {av.x, av.y, av.z, av.w}, bn[4] = {bv.x, bv.y, bv.z, bv.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(am[i], bn[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
+      if (m < M && n < N) out[(size_t)m * ldo + n] = act_f32(act, acc[i][j]);
+    }
+}
+
+}  // namespace rf
+
+using namespace rf;
+
+#define RF_DISPATCH3(dtype, ...)                                        \
+  if ((dtype) == kF16) { using T = __half; __VA_ARGS__; }               \
+  else if ((dtype) == kBF16) { using T = __nv_bfloat16; __VA_ARGS__; }  \
+  else { using T = float; __VA_ARGS__; }
+
+extern "C" int rf_stream_norm(const RfStreamNorm* a, rf_stream_t stream) {
+  RF_SKIP_IF_REPLAYING();
+  RF_REQUIRE(a && a->H > 0 && a->H % 8 == 0 && a->dim > 0 && a->dim <= a->H, "stream_norm: row length");
+  RF_REQUIRE(a->x || (a->table && a->ids), "stream_norm: no input");
+  RF_REQUIRE(!a->norm_w || a->out, "stream_norm: no output");
+  RF_REQUIRE(a->dtype >= 0 && a->dtype <= 2, "stream_norm: dtype %d", a->dtype);
+  if (a->shift) RF_REQUIRE(a->norm_w && a->shift_state && a->rows.pos && !a->row_idx && a->x_out != a->x,
+                           "stream_norm: the token shift needs a norm, its state, positions, all rows and separate streams");
+  if (a->n_rows == 0) return RF_OK;
+  // halo of one row per CTA with the shift: walk several rows per CTA once that still fills the GPU
+  const int rpc = (a->shift && a->rows.q_start) ? std::max(1, std::min(8, a->n_rows / (2 * sm_count()))) : 1;
+  const int threads = std::min(512, std::max(64, round_up(ceil_div(a->H / 4, a->H >= 4096 ? 2 : 1), 32)));
+  const size_t smem = ((size_t)a->H * (a->shift ? 2 : 1) + 32) * sizeof(float);
+  RF_REQUIRE(smem <= 200 * 1024, "stream_norm: rows of %d values do not fit in shared memory", a->H);
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  RF_DISPATCH3(a->dtype, {
+    RF_ALLOW_SMEM_PER_DEVICE(stream_norm_kernel<T>, 200 * 1024);
+    RF_CUDA_CHECK(::rf::launch_k(stream_norm_kernel<T>, dim3(ceil_div(a->n_rows, rpc)), dim3(threads), smem, s, 1, *a, rpc));
+  });
+  ::rf::count_launch();
+  return RF_OK;
+}
+
+extern "C" int rf_token_gate(void* g, int64_t ldg, const void* table, int64_t ld_table, const int32_t* ids, int32_t col0,
+                             int32_t rows, int32_t cols, int32_t dtype, rf_stream_t stream) {
+  RF_SKIP_IF_REPLAYING();
+  RF_REQUIRE(g && table && ids && cols % 8 == 0 && ldg % 8 == 0 && ld_table % 8 == 0 && col0 % 8 == 0, "token_gate arguments");
+  if (rows == 0) return RF_OK;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const int64_t n = (int64_t)rows * (cols / 8);
+  RF_DISPATCH3(dtype, RF_CUDA_CHECK(::rf::launch_k(token_gate_kernel<T>, dim3((unsigned)((n + 127) / 128)), dim3(128), 0, s, 1,
+                                                   (T*)g, ldg, (const T*)table, ld_table, ids, col0, rows, cols)));
+  ::rf::count_launch();
+  return RF_OK;
+}
+
+extern "C" int rf_gemm_f32(const RfGemm* g, rf_stream_t stream) {
+  RF_SKIP_IF_REPLAYING();
+  RF_REQUIRE(g && g->x && g->w && g->out && g->M >= 0 && g->N > 0 && g->K > 0, "gemm_f32 arguments");
+  RF_REQUIRE(g->K % 4 == 0 && g->ldx % 4 == 0 && g->ldw % 4 == 0, "gemm_f32: K and the pitches must be multiples of 4");
+  RF_REQUIRE(!g->residual && !g->bias && !g->scale && !g->row_scale && g->dual_offset == 0 && !g->w_packed && g->ar_world <= 1,
+             "gemm_f32 has an activation epilogue only");
+  if (g->M == 0) return RF_OK;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  RF_CUDA_CHECK(::rf::launch_k(gemm_f32_kernel, dim3(ceil_div(g->N, kFBN), ceil_div(g->M, kFBM)), dim3(256), 0, s, 1,
+                               (const float*)g->x, g->ldx, (const float*)g->w, g->ldw, (float*)g->out, g->ldo, g->M, g->N,
+                               g->K, g->act));
+  ::rf::count_launch();
+  return RF_OK;
+}

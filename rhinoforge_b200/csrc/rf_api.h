@@ -295,6 +295,92 @@ int rf_cumsum_f32(const float* x, float* y, int rows, int n, rf_stream_t stream)
 int rf_unit_tril_inv_f32(const float* m, float* out, int batch, int n, rf_stream_t stream);
 
 
+// ----------------------------------- decoders with per-layer mixers ----
+// Where the rows of a launch belong: row r is one token of sequence seq_of_row[r] (null: row = sequence, one token each),
+// sequence s occupies rows [q_start[s], q_start[s] + q_len[s]) (null: one row), keeps its recurrent state and its page-table
+// row in slot[s] (null: s), and pos[r] is the row's position in its sequence.  A sequence whose first row has position 0
+// starts from an empty state.
+typedef struct RfRows {
+  const int32_t* seq_of_row; const int32_t* q_start; const int32_t* q_len; const int32_t* slot; const int32_t* pos;
+  const int32_t* page_table; int32_t pt_stride; int32_t num_seqs;
+} RfRows;
+
+// The fp32 residual stream between two sublayers, one launch:
+//   v = x[row]  (or the embedding row table[ids[row]] when x is null)
+//   v += y[row]  or, with y_norm_w,  v += y / rms(y) * y_norm_w          (the sublayer output that is still outstanding)
+//   x_out = v (fp32), x_cast = v (activation dtype)
+//   h = v / rms(v) * norm_w;  with `shift`: out = h + (h_prev - h) * shift, h_prev the h of the sequence's previous token
+//   (carried over launches in shift_state[slot], zeros before the first token); without: out = h.
+// H is the (padded, multiple of 8) row length, dim the true one that the means run over.  x_out must not alias x when
+// `shift` is set.  row_idx (optional) selects the rows that are processed (not together with shift).
+typedef struct RfStreamNorm {
+  const float* x; const void* table; const int32_t* ids; const int32_t* row_idx;
+  const void* y; const float* y_norm_w;
+  float* x_out; void* x_cast;
+  const float* norm_w; void* out;
+  const float* shift; float* shift_state;
+  RfRows rows;
+  int32_t n_rows, H, dim; float eps; int32_t dtype;    // dtype 2: fp32 activations
+} RfStreamNorm;
+int rf_stream_norm(const RfStreamNorm* a, rf_stream_t stream);
+
+// out[M, N] = act(x[M, K] . w[N, K]^T) in true fp32 (row-major operands, no tensor cores): the linear layers of a model that
+// is served in 32 bits.  Uses x, w, out, their pitches, M, N, K and act of RfGemm.
+int rf_gemm_f32(const RfGemm* g, rf_stream_t stream);
+
+// g[r, c] *= table[ids[r] * ld_table + col0 + c] for c < cols (a gate multiplied by a per-token embedding slice)
+int rf_token_gate(void* g, int64_t ldg, const void* table, int64_t ld_table, const int32_t* ids, int32_t col0, int32_t rows,
+                  int32_t cols, int32_t dtype, rf_stream_t stream);
+
+// Per-head linear map y[r, h, n] = sum_k x[r, h, k] w[h, n, k]; head h of row r starts at x + r * ldx + h * xs
+// (y + r * ldy + h * ys).  Sizes n, k, xs, ys and pitches are multiples of 8.
+typedef struct RfHeadLinear {
+  const void* x; int64_t ldx; int32_t xs;
+  void* y; int64_t ldy; int32_t ys;
+  const void* w;
+  int32_t rows, heads, n, k, dtype;
+} RfHeadLinear;
+int rf_head_linear(const RfHeadLinear* a, rf_stream_t stream);
+
+// Latent-attention cache: one row of `rank` (padded to a multiple of 16) values per token, pool [pages, 16, rank].
+// rf_latent_insert: c = x / rms(x) * norm_w (mean over the true rank), stored at the row's position.
+int rf_latent_insert(const void* x, int64_t ldx, const float* norm_w, void* pool, const RfRows* rows, int32_t n_rows,
+                     int32_t rank, int32_t rank_true, float eps, int32_t dtype, rf_stream_t stream);
+// Dense copies of the latents that the rows of num_seqs sequences can see under a window (the last min(first position,
+// window - 1) cached tokens and the sequence's own rows), packed back to back; kv_start / kv_len (device, [num_seqs])
+// receive each sequence's first row and row count.  window <= 0: everything.  max_len: host bound of kv_len.
+int rf_latent_gather(const void* pool, void* out, const RfRows* rows, int32_t window, int32_t rank, int32_t max_len,
+                     int32_t* kv_start, int32_t* kv_len, int32_t dtype, rf_stream_t stream);
+
+// Attention in the latent space (keys and values folded into the queries and the output): every row attends from its own
+// position to the window before it, score = (q[r, h] . c[j]) * scale, o[r, h] = sum_j softmax(score)_j c[j].
+// q, o: [rows, heads, rank] dense.  window <= 0: no lower bound.  max_kv: host bound of the keys one row sees.
+typedef struct RfLatentAttn {
+  const void* q; void* o; const void* pool;
+  RfRows rows;
+  int32_t n_rows, heads, rank, window, max_kv; float scale; int32_t dtype;
+  float* ws; uint64_t ws_bytes;      // split partials, optional
+} RfLatentAttn;
+int rf_latent_attn(const RfLatentAttn* a, rf_stream_t stream);
+uint64_t rf_latent_attn_scratch_bytes(int rows, int heads, int rank, int max_kv);
+
+// Linear attention whose forget gate also decides what is written (HGRN2), over packed input rows [q | f | v]:
+//   q = silu(q), f = lower + (1 - lower) * sigmoid(f + f_bias), S = diag(f) S + (1 - f) v^T, o = S^T q,
+//   out = o / rms(o) * norm_w per head (mean over the true value size; null norm_w: plain o)
+// state: fp32 [slots, heads, dim, vdim].  Padding channels of dim have lower = 1, padding value columns are zero.
+typedef struct RfHgrn2 {
+  const void* x; int64_t ldx; int32_t f_off, v_off;
+  const float* f_bias; const float* lower; const float* norm_w;
+  float* state; void* out; int64_t ldo;
+  RfRows rows;
+  int32_t heads, dim, vdim, vdim_true; float eps; int32_t dtype;
+} RfHgrn2;
+int rf_hgrn2_recurrent(const RfHgrn2* a, rf_stream_t stream);
+// Same contract, evaluated block by block (prefill-sized portions; 16-bit activations).
+int rf_hgrn2_chunked(const RfHgrn2* a, rf_stream_t stream);
+int rf_hgrn2_chunked_supported(int dim, int vdim, int dtype);
+
+
 // ------------------------------------------------- mixture of experts ----
 // Router: scores = sigmoid(logits) (score_fn 0) or softmax(logits) (1); the k experts with the largest
 // (score + bias) are selected, ties to the lower index; weights are the UNBIASED scores, divided by their

@@ -13,7 +13,7 @@ import torch
 
 from .. import _native as N
 
-ACT = {None: 0, "none": 0, "silu_mul": 1, "gelu_tanh_mul": 2, "gelu_tanh": 3, "gelu_erf": 4, "silu": 5}
+ACT = {None: 0, "none": 0, "silu_mul": 1, "gelu_tanh_mul": 2, "gelu_tanh": 3, "gelu_erf": 4, "silu": 5, "relu2": 6}
 ELT = {"add": 0, "mul": 1, "silu_mul": 2, "gelu_tanh_mul": 3, "axpy": 4, "gelu_tanh": 5, "gelu_erf": 6,
        "silu": 7, "scale": 8, "sigmoid_mul": 9, "mul_row": 10, "tanh": 11}
 

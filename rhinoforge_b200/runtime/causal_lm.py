@@ -204,5 +204,32 @@ class RPUCausalLM:
         out = torch.cat([ids.to(self.engine.device, torch.int64), torch.cat(new, 1).to(torch.int64)], 1)
         return out.to(input_ids.device)
 
+    def bind_cache(self, *, batch_size: int, max_seq_len: int, pool_tokens: Optional[int] = None):
+        """Make and bind a cache of ``batch_size`` request slots over a pool of ``pool_tokens`` tokens; returns it."""
+        make = getattr(self.engine, "make_cache", None)
+        if make is not None:
+            cache = make(batch_size, max_seq_len, pool_tokens=pool_tokens)
+        else:
+            from .kv_cache import PagedKV
+            old = self.engine.cache
+            cache = PagedKV(old.num_layers, batch_size, max_seq_len, old.num_kv_heads, old.head_dim, device=old.device,
+                            dtype=old.dtype, pool_tokens=pool_tokens)
+        self.engine.bind_cache(cache)
+        return cache
+
+    @torch.no_grad()
+    def generate_batch(self, prompts, max_new_tokens: int, *, eos_token_id: Optional[int] = None, slots: Optional[int] = None,
+                       token_budget: Optional[int] = None, pool_tokens: Optional[int] = None):
+        """Greedy continuations of any number of prompts of any lengths through the request scheduler (continuous batching:
+        prompt portions run beside decoded tokens).  Returns one list of new token ids per prompt."""
+        from .scheduler import RequestScheduler
+        prompts = [torch.as_tensor(p).reshape(-1) for p in prompts]
+        if not prompts:
+            return []
+        n = min(slots or len(prompts), len(prompts), self.engine.max_batch)
+        longest = max(int(p.numel()) for p in prompts) + max_new_tokens
+        self.bind_cache(batch_size=n, max_seq_len=(longest + 15) // 16 * 16, pool_tokens=pool_tokens)
+        return RequestScheduler(self.engine, token_budget=token_budget).generate(prompts, max_new_tokens, eos_token_id=eos_token_id)
+
     def close(self) -> None:
         self.engine.close()

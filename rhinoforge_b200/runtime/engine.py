@@ -539,7 +539,8 @@ class DecoderEngine:
     def extend(self, tokens: Sequence[torch.Tensor], *, return_logits: bool = False, logits_rows: int = 1,
                inputs_embeds: Optional[Sequence[torch.Tensor]] = None,
                positions3: Optional[Sequence[torch.Tensor]] = None,
-               deepstack: Optional[Sequence[Optional[tuple]]] = None):
+               deepstack: Optional[Sequence[Optional[tuple]]] = None, slots: Optional[Sequence[int]] = None,
+               want: Optional[Sequence[Sequence[int]]] = None, decode_room: int = 1):
         """Append ``tokens[s]`` (1-D int tensors, host or device) to sequence ``s`` at its current
         length and return the greedy next token of every sequence ([B] int32 on the device; with
         ``return_logits`` also the last-row logits of this rank's vocab shard).  Long inputs run as
@@ -551,20 +552,29 @@ class DecoderEngine:
         ``feats[l][i]`` to the hidden row ``rows[i]`` of sequence ``s`` after layer ``l`` (DeepStack).
 
         ``logits_rows`` (with ``return_logits``): 1 returns ``[B, vocab]`` of the last rows; ``k > 1`` or ``0`` (all) returns a
-        list with one ``[rows_s, vocab]`` tensor per sequence holding its last ``k`` (or all) new rows."""
+        list with one ``[rows_s, vocab]`` tensor per sequence holding its last ``k`` (or all) new rows.
+
+        ``slots`` maps the sequences of this call to cache slots (default ``0 .. B-1``): a scheduler appends to any subset of the
+        live requests.  ``want[s]`` (with ``return_logits``) names the new rows of sequence ``s`` whose logits are returned, as a
+        list of ``[len(want[s]), vocab]`` tensors.  ``decode_room`` tokens of page room are kept behind the new ones for the
+        decode step that follows."""
         B = len(tokens)
         cache = self.cache
+        dense = slots is None
+        slots = list(range(B)) if dense else [int(s) for s in slots]
+        if len(slots) != B or len(set(slots)) != B or any(not 0 <= s < cache.batch_size for s in slots):
+            raise RPUBackendError(f"slots {slots} are not {B} different slots of a cache with {cache.batch_size}")
         if B > cache.batch_size:
             raise RPUBackendError(f"batch {B} exceeds the cache's batch_size {cache.batch_size}")
         self._liveness()
-        starts = [int(cache.lengths[s]) for s in range(B)]
+        starts = [int(cache.lengths[s]) for s in slots]
         lens = [int(p.numel()) for p in tokens]
         for s, L in enumerate(lens):
             if L < 1:
                 raise RPUBackendError("every sequence needs at least one new token")
-            cache.check_fits(s, L + 1)
+            cache.check_fits(slots[s], L + decode_room)
         for s, L in enumerate(lens):              # pages for the new tokens and the first decode step
-            cache.ensure(s, starts[s] + L + 1)
+            cache.ensure(slots[s], starts[s] + L + decode_room)
         cache.sync_table()
         logits_all = torch.empty((B, self.vocab_local), dtype=self.dtype, device=self.device) if return_logits else None
         first = torch.zeros(B, dtype=torch.int32, device=self.device)
@@ -585,13 +595,17 @@ class DecoderEngine:
         if chunk:
             items.append(chunk)
         row_logits = None
-        if return_logits and logits_rows != 1:
-            row_logits = {"keep": int(logits_rows), "out": [[] for _ in range(B)]}
+        if return_logits and (logits_rows != 1 or want is not None):
+            row_logits = {"keep": int(logits_rows), "want": want, "out": [[] for _ in range(B)]}
         for ch in items:
-            self._prefill_chunk(ch, tokens, lens, starts, first, logits_all, inputs_embeds, positions3, deepstack, row_logits)
-        self.batch = B
+            self._prefill_chunk(ch, tokens, lens, starts, first, logits_all, inputs_embeds, positions3, deepstack, row_logits,
+                                slots=slots)
         for s, L in enumerate(lens):
-            cache.lengths[s] = starts[s] + L
+            cache.lengths[slots[s]] = starts[s] + L
+        if not dense:                             # the decode state below describes slots 0 .. B-1
+            self.batch = 0
+            return self._extend_result(first, logits_all, row_logits, return_logits)
+        self.batch = B
         # decode state: the token to feed next is `first`, at position = new length
         self.ids[:B].copy_(first)
         new_len = torch.from_numpy(cache.lengths[:B].astype("int32"))
@@ -605,12 +619,31 @@ class DecoderEngine:
         else:
             self.pos[:B].copy_(new_len[:, None].expand(B, self.pos_stride))
         self.kv_len[:B].copy_(new_len + 1)
+        return self._extend_result(first, logits_all, row_logits, return_logits)
+
+    def _extend_result(self, first, logits_all, row_logits, return_logits):
         if row_logits is not None:
             return first, [torch.cat(parts) if parts else logits_all.new_empty((0, self.vocab_local)) for parts in row_logits["out"]]
         return (first, logits_all) if return_logits else first
 
+    @staticmethod
+    def _wanted_rows(row_logits, s: int, off: int, cnt: int, length: int) -> List[int]:
+        """Rows of sequence ``s`` inside ``[off, off + cnt)`` whose logits were asked for, relative to ``off``."""
+        if row_logits["want"] is not None:
+            return [int(w) - off for w in row_logits["want"][s] if off <= int(w) < off + cnt]
+        lo = 0 if row_logits["keep"] == 0 else max(length - row_logits["keep"], 0)
+        return list(range(max(off, lo) - off, cnt))
+
+    @torch.no_grad()
+    def run_step(self, tokens: Sequence[torch.Tensor], slots: Sequence[int], want: Sequence[Sequence[int]]):
+        """One scheduler step: append ``tokens[i]`` to the request in cache slot ``slots[i]``, portions of prompts beside single
+        decoded tokens, and return ``(next, logits)``: the greedy token behind every entry's last row (``[n]`` int32, device)
+        and, per entry, the logits ``[len(want[i]), vocab]`` of the rows it names.  Only the pages the new tokens need are
+        taken."""
+        return self.extend(tokens, slots=slots, want=want, return_logits=True, decode_room=0)
+
     def _prefill_chunk(self, ch, prompts, lens, starts, first, logits_all, inputs_embeds, positions3,
-                       deepstack=None, row_logits=None) -> None:
+                       deepstack=None, row_logits=None, slots=None) -> None:
         T = sum(c[2] for c in ch)
         n = len(ch)
         meta = torch.empty((6, max(n, 1)), dtype=torch.int32)
@@ -623,7 +656,7 @@ class DecoderEngine:
         for j, (s, off, cnt) in enumerate(ch):
             base = starts[s]
             meta[0, j], meta[1, j], meta[2, j] = o, cnt, base + off + cnt   # q_start, q_len, kv_len
-            meta[3, j] = s
+            meta[3, j] = slots[s]
             meta[4, j] = o + cnt - 1
             meta[5, j] = 1 if (base + off) == 0 else 0        # starts from an empty recurrent state
             tokmeta[0, o:o + cnt] = s
@@ -682,15 +715,14 @@ class DecoderEngine:
             f.deepstack, f.deepstack_rows = ds_ptrs.data_ptr(), ds_rows_d.data_ptr()
             f.n_deepstack, f.n_deepstack_rows = len(ds_layers), ds_rows_d.numel()
         N.check(N.lib().rf_stack_forward(self.handle, C.byref(f), self._stream()), "rf_stack_forward")
-        if row_logits is not None:                 # logits of the requested trailing rows of every sequence in this chunk
-            keep = row_logits["keep"]
+        if row_logits is not None:                 # logits of the requested rows of every sequence in this chunk
             o2 = 0
             for (s, off, cnt) in ch:
-                lo = 0 if keep == 0 else max(lens[s] - keep, 0)
-                a, b = max(off, lo), off + cnt
-                for r0 in range(a, b, self.max_batch):
-                    nr = min(self.max_batch, b - r0)
-                    idx = torch.arange(o2 + r0 - off, o2 + r0 - off + nr, dtype=torch.int32, device=self.device)
+                rows_w = self._wanted_rows(row_logits, s, off, cnt, lens[s])
+                for r0 in range(0, len(rows_w), self.max_batch):
+                    part = rows_w[r0:r0 + self.max_batch]
+                    nr = len(part)
+                    idx = torch.tensor([o2 + r for r in part], dtype=torch.int32).to(self.device)
                     lg = torch.empty((nr, self.vocab_local), dtype=self.dtype, device=self.device)
                     self._head(nr, idx, lg)
                     row_logits["out"][s].append(lg)
@@ -729,13 +761,17 @@ class DecoderEngine:
                                           C.c_void_p(self.step.data_ptr()), self.hist_steps, self._stream()),
                 "rf_decode_advance")
 
+    def _decode_state(self) -> List[torch.Tensor]:
+        """Device tensors a decode step advances: the counters, and the states of recurrent layers (which, unlike K/V pages,
+        a repeated step would change twice)."""
+        return [self.pos, self.kv_len, self.ids, self.step] + [t for l in self.gdn_layers
+                                                               for t in (self.gdn_conv_state[l], self.gdn_rec_state[l])]
+
     def capture(self, B: int) -> None:
         """BUILD: run one eager step (loads kernels, sets attributes), rewind, then capture."""
         if B in self.graphs:
             return
-        snap = (self.pos.clone(), self.kv_len.clone(), self.ids.clone(), self.step.clone())
-        # recurrent layers are not idempotent: the eager build step must not advance their state
-        gdn_snap = {l: (self.gdn_conv_state[l].clone(), self.gdn_rec_state[l].clone()) for l in self.gdn_layers}
+        snap = [(t, t.clone()) for t in self._decode_state()]
         s = torch.cuda.Stream()
         s.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(s):
@@ -745,10 +781,8 @@ class DecoderEngine:
         with torch.cuda.graph(g, stream=s):
             self._decode_step(B)
         torch.cuda.synchronize()
-        self.pos.copy_(snap[0]); self.kv_len.copy_(snap[1]); self.ids.copy_(snap[2]); self.step.copy_(snap[3])
-        for l, (cv, rc) in gdn_snap.items():
-            self.gdn_conv_state[l].copy_(cv)
-            self.gdn_rec_state[l].copy_(rc)
+        for t, saved in snap:
+            t.copy_(saved)
         self.graphs[B] = g
 
     def decode(self, n_steps: int, *, use_graph: bool = True) -> torch.Tensor:

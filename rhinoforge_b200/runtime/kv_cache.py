@@ -27,18 +27,13 @@ from .errors import RPUBackendError
 PAGE_TOKENS = 16
 
 
-class PagedKV:
-    def __init__(self, num_layers: int, batch_size: int, max_seq_len: int, num_kv_heads: int, head_dim: int, *,
-                 device="cuda", dtype=torch.float16, pool_tokens: Optional[int] = None):
-        for name, v in (("num_layers", num_layers), ("batch_size", batch_size), ("max_seq_len", max_seq_len),
-                        ("num_kv_heads", num_kv_heads), ("head_dim", head_dim)):
-            if isinstance(v, bool) or not isinstance(v, int) or v <= 0:
-                raise ValueError(f"RPUCache {name} must be a positive integer, got {v!r}")
-        if head_dim % 16:
-            raise ValueError(f"RPUCache head_dim must be divisible by 16, got {head_dim}")
+class PagedSequences:
+    """Page ownership of ``batch_size`` sequence slots over a pool of 16-token pages: the part every cache shares,
+    whatever it stores per page.  Subclasses allocate ``num_pages`` pages of device memory."""
+
+    def _init_pages(self, batch_size: int, max_seq_len: int, device, pool_tokens: Optional[int] = None) -> None:
         self._pool = None
-        self.num_layers, self.batch_size, self.max_seq_len = num_layers, batch_size, max_seq_len
-        self.num_kv_heads, self.head_dim, self.dtype = num_kv_heads, head_dim, dtype
+        self.batch_size, self.max_seq_len = batch_size, max_seq_len
         self.device = torch.device(device)
         self.pages_per_seq = (max_seq_len + PAGE_TOKENS - 1) // PAGE_TOKENS
         self.num_pages = batch_size * self.pages_per_seq
@@ -46,18 +41,13 @@ class PagedKV:
             if isinstance(pool_tokens, bool) or not isinstance(pool_tokens, int) or pool_tokens <= 0:
                 raise ValueError(f"RPUCache pool_tokens must be a positive integer, got {pool_tokens!r}")
             self.num_pages = min(self.num_pages, (pool_tokens + PAGE_TOKENS - 1) // PAGE_TOKENS)
-        self.kv = torch.zeros((num_layers, 2, self.num_pages, num_kv_heads, PAGE_TOKENS, head_dim), dtype=dtype,
-                              device=self.device)
         self.page_table = torch.zeros((batch_size, self.pages_per_seq), dtype=torch.int32, device=self.device)
         self._pt_host = torch.zeros((batch_size, self.pages_per_seq), dtype=torch.int32)
-        if self.device.type == "cuda":
-            self._pt_host = self._pt_host.pin_memory()
         # cached length and page capacity (in tokens) of every sequence slot: numpy so that a decode step
         # advances / checks the whole batch with one vector operation
         self.lengths = np.zeros(batch_size, dtype=np.int64)
         self._capacity = np.zeros(batch_size, dtype=np.int64)
         self._dirty = False
-        self._pool = None
         if N.available() or self.device.type == "cuda":
             self._pool = C.c_int64(N.lib().rf_kvpool_create(self.num_pages, batch_size, self.pages_per_seq))
         else:  # host-only sizing without the native library: identity mapping
@@ -106,7 +96,9 @@ class PagedKV:
         self.sync_table()
 
     def sync_table(self) -> None:
-        self.page_table.copy_(self._pt_host, non_blocking=True)
+        # a private copy travels: the host table may change again before the stream reaches this upload
+        src = self._pt_host.clone()
+        self.page_table.copy_(src.pin_memory() if self.device.type == "cuda" else src, non_blocking=True)
         self._dirty = False
 
     def release(self, seq: int) -> None:
@@ -122,6 +114,37 @@ class PagedKV:
 
     def free_pages(self) -> int:
         return N.lib().rf_kvpool_free_pages(self._pool) if self._pool is not None else 0
+
+    def close(self) -> None:
+        if getattr(self, "_pool", None) is not None:
+            try:
+                N.lib().rf_kvpool_destroy(self._pool)
+            except Exception:  # noqa: BLE001
+                pass
+            self._pool = None
+
+    def __del__(self):
+        self.close()
+
+    def check_fits(self, seq: int, extra: int) -> None:
+        if self.lengths[seq] + extra > self.max_seq_len:
+            raise RPUBackendError(f"RPUCache position overflow: position={self.lengths[seq]}, seq_len={extra}, "
+                                  f"max_seq_len={self.max_seq_len}")
+
+
+class PagedKV(PagedSequences):
+    def __init__(self, num_layers: int, batch_size: int, max_seq_len: int, num_kv_heads: int, head_dim: int, *,
+                 device="cuda", dtype=torch.float16, pool_tokens: Optional[int] = None):
+        for name, v in (("num_layers", num_layers), ("batch_size", batch_size), ("max_seq_len", max_seq_len),
+                        ("num_kv_heads", num_kv_heads), ("head_dim", head_dim)):
+            if isinstance(v, bool) or not isinstance(v, int) or v <= 0:
+                raise ValueError(f"RPUCache {name} must be a positive integer, got {v!r}")
+        if head_dim % 16:
+            raise ValueError(f"RPUCache head_dim must be divisible by 16, got {head_dim}")
+        self.num_layers, self.num_kv_heads, self.head_dim, self.dtype = num_layers, num_kv_heads, head_dim, dtype
+        self._init_pages(batch_size, max_seq_len, device, pool_tokens)
+        self.kv = torch.zeros((num_layers, 2, self.num_pages, num_kv_heads, PAGE_TOKENS, head_dim), dtype=dtype,
+                              device=self.device)
 
     def layer_ptrs(self, layer: int):
         return self.kv[layer, 0].data_ptr(), self.kv[layer, 1].data_ptr()
@@ -157,21 +180,5 @@ class PagedKV:
     def zero_(self) -> None:
         self.kv.zero_()
 
-    def close(self) -> None:
-        if getattr(self, "_pool", None) is not None:
-            try:
-                N.lib().rf_kvpool_destroy(self._pool)
-            except Exception:  # noqa: BLE001
-                pass
-            self._pool = None
-
-    def __del__(self):
-        self.close()
-
     def nbytes(self) -> int:
         return self.kv.numel() * self.kv.element_size()
-
-    def check_fits(self, seq: int, extra: int) -> None:
-        if self.lengths[seq] + extra > self.max_seq_len:
-            raise RPUBackendError(f"RPUCache position overflow: position={self.lengths[seq]}, seq_len={extra}, "
-                                  f"max_seq_len={self.max_seq_len}")

@@ -1,0 +1,367 @@
+"""Serving engine of decoders with per-layer mixers (:mod:`rhinoforge_b200.models.mixed`).
+
+The engine interface is :class:`DecoderEngine`'s: ``prefill`` / ``extend`` / ``run_step`` pack portions of any sequences into one
+launch, ``decode`` replays a captured graph, ``generate`` strings them together.  What differs is behind it: the native
+executor is the mixed stack (fp32 residual stream, one mixer per layer), the cache a :class:`MixedCache`, and the decode graph
+addresses sequences through a slot array, so a scheduler step of single tokens replays it for any subset of the live requests.
+
+Weights are padded once at load to the granularity of the kernels (rows of 8 / 16 values, attention heads to 64 / 128 / 256
+for the tcgen05 prefill attention); padding rows and columns are zero.
+"""
+from __future__ import annotations
+
+import ctypes as C
+import os
+from typing import Dict, List, Optional, Sequence
+
+import torch
+
+from .. import _native as N
+from ..models.mixed import HGRN2, LatentAttention, MixedConfig
+from ..ops import kernels as K
+from ..parallel.tp import TPContext
+from .engine import DecoderEngine, WeightGetter
+from .errors import RPUBackendError
+from .mixed_cache import MixedCache, pad_to
+
+
+def _pad2(w: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
+    if tuple(w.shape) == (rows, cols):
+        return w
+    out = w.new_zeros((rows, cols))
+    out[:w.shape[0], :w.shape[1]] = w
+    return out
+
+
+def _pad_heads(w: torch.Tensor, heads: int, true: int, padded: int) -> torch.Tensor:
+    """``[heads * true, K]`` -> ``[heads * padded, K]`` with zero rows behind every head."""
+    if true == padded:
+        return w
+    out = w.new_zeros((heads, padded, w.shape[1]))
+    out[:, :true] = w.view(heads, true, w.shape[1])
+    return out.view(heads * padded, w.shape[1])
+
+
+class MixedDecoderEngine(DecoderEngine):
+    LONG_MIN = 16          # portions of at least this many tokens take the prefill forms of the mixers
+    HEAD_ROWS = 64         # rows one logits launch takes
+
+    def __init__(self, cfg: MixedConfig, get_weight: WeightGetter, *, device="cuda", dtype=torch.bfloat16, max_batch: int = 1,
+                 max_seq_len: int = 2048, max_prefill_tokens: int = 8192, tp: Optional[TPContext] = None, hist_steps: int = 4096,
+                 kv_cache: Optional[MixedCache] = None, kv_pool_tokens: Optional[int] = None):
+        if not torch.cuda.is_available():
+            raise RPUBackendError("MixedDecoderEngine needs a CUDA device")
+        if tp is not None and tp.enabled:
+            raise RPUBackendError(f"{cfg.name}: tensor parallelism is not built for decoders with per-layer mixers")
+        if dtype not in (torch.float16, torch.bfloat16, torch.float32):
+            raise RPUBackendError(f"{cfg.name}: activations are float16, bfloat16 or float32, got {dtype}")
+        self.cfg, self.dtype = cfg, dtype
+        self.tp = tp or TPContext.single(device)
+        self.device = torch.device(self.tp.device if self.tp.device is not None else device)
+        self.comm, self.quant = None, None
+        self.max_batch = max_batch
+        self.max_tokens = max(max_prefill_tokens, max_batch)
+        self.fp32 = dtype == torch.float32
+        self.packed = not self.fp32 and os.environ.get("RF_PACKED_WEIGHTS", "1") != "0"
+        self.long_min = (1 << 30) if self.fp32 else self.LONG_MIN
+        self.H = pad_to(cfg.hidden_size, 8)
+        self.vocab_local = cfg.vocab_size
+        self.vocab_ld = pad_to(cfg.vocab_size, 8)
+        self.head_rows = max(max_batch, self.HEAD_ROWS)
+        self._keep: List[torch.Tensor] = []
+        self.cache = kv_cache if kv_cache is not None else MixedCache(cfg, max_batch, max_seq_len, device=self.device, dtype=dtype,
+                                                                      pool_tokens=kv_pool_tokens)
+        self._check_cache(self.cache)
+        lib = N.lib()
+        self.handle = None
+        self._load(get_weight, max(max_seq_len, self.cache.max_seq_len))
+        nbytes = lib.rf_mixed_arena_bytes(self.handle)
+        self.arena = torch.zeros(nbytes + 1024, dtype=torch.uint8, device=self.device)
+        base = (self.arena.data_ptr() + 1023) // 1024 * 1024
+        N.check(lib.rf_mixed_bind_arena(self.handle, C.c_void_p(base), C.c_uint64(nbytes)), "rf_mixed_bind_arena")
+        off = lib.rf_mixed_status_ptr(self.handle) - self.arena.data_ptr()
+        self.status = self.arena[off:off + 32].view(torch.int32)
+        # ---- decode state, advanced on the device
+        i32 = dict(dtype=torch.int32, device=self.device)
+        self.ids, self.out_ids = torch.zeros(max_batch, **i32), torch.zeros(self.head_rows, **i32)
+        self.out_vals = torch.zeros(self.head_rows, dtype=torch.float32, device=self.device)
+        self.pos_stride = 1
+        self.pos, self.kv_len = torch.zeros((max_batch, 1), **i32), torch.zeros(max_batch, **i32)
+        self.slot = torch.arange(max_batch, **i32)
+        self.logits = torch.zeros((max_batch, self.vocab_ld), dtype=dtype, device=self.device)
+        self.step = torch.zeros(1, **i32)
+        self.hist_steps = hist_steps
+        self.hist = torch.zeros((hist_steps, max_batch), **i32)
+        self.graphs: Dict[int, torch.cuda.CUDAGraph] = {}
+        self.batch = 0
+        self._hb = self._host_steps = 0
+        self.heartbeat_every = 0
+
+    # ------------------------------------------------------------------ weights
+    def _f32(self, t: torch.Tensor, n: int, fill: float = 0.0) -> torch.Tensor:
+        out = torch.full((n,), fill, dtype=torch.float32, device=self.device)
+        out[:t.numel()] = t.reshape(-1).to(self.device, torch.float32)
+        self._keep.append(out)
+        return out
+
+    def _linear(self, w: torch.Tensor) -> torch.Tensor:
+        t = w.to(self.device, self.dtype).contiguous()
+        if self.packed:
+            t = K.pack_weight(t)
+        self._keep.append(t)
+        return t
+
+    def _plain(self, w: torch.Tensor) -> torch.Tensor:
+        t = w.to(self.device, self.dtype).contiguous()
+        self._keep.append(t)
+        return t
+
+    def _load(self, get: WeightGetter, max_context: int) -> None:
+        cfg, lib, H = self.cfg, N.lib(), self.H
+        g = lambda name: get(name).to(self.device)
+        P = pad_to(cfg.side_dim, 8)
+        V, L = cfg.vocab_size, cfg.num_layers
+        self.embed = self._plain(_pad2(g("embed"), V, H))
+        side = g("side.embed").view(V, L, cfg.side_dim)
+        if P != cfg.side_dim:
+            wide = side.new_zeros((V, L, P))
+            wide[:, :, :cfg.side_dim] = side
+            side = wide
+        self.side_table = self._plain(side.reshape(V, L * P))
+        self.final_norm = self._f32(g("final.norm"), H)
+        lm = self._linear(_pad2(self.embed, self.vocab_ld, H))
+        sc = N.RfMixedConfig()
+        sc.layers, sc.hidden, sc.hidden_true, sc.vocab, sc.vocab_ld = L, H, cfg.hidden_size, V, self.vocab_ld
+        sc.dtype = 2 if self.fp32 else K.dtype_code(self.dtype)
+        sc.max_tokens, sc.max_seqs, sc.max_seq_len = self.max_tokens, self.max_batch, max_context
+        sc.side_dim, sc.side_ld, sc.eps = P, L * P, cfg.rms_eps
+        sc.weights_packed, sc.long_min = int(self.packed), self.long_min
+        sc.embed, sc.side_table, sc.final_norm, sc.w_lm = (t.data_ptr() for t in (self.embed, self.side_table, self.final_norm, lm))
+        h = lib.rf_mixed_create(C.byref(sc))
+        if h < 0:
+            N.check(-1, "rf_mixed_create")
+        self.handle = C.c_int64(h)
+        for i, layer in enumerate(cfg.layers):
+            m, p = layer.mixer, f"l{i}."
+            lw = N.RfMixedLayer()
+            lw.heads = m.heads
+            lw.norm1, lw.shift = self._f32(g(p + "norm1"), H).data_ptr(), self._f32(g(p + "shift"), H).data_ptr()
+            latent, recurrent, shift_rows = self.cache.layer_ptrs(i)
+            lw.shift_state = shift_rows
+            (self._load_latent if isinstance(m, LatentAttention) else self._load_hgrn2)(lw, m, g, p + "mix.")
+            lw.latent_pool, lw.rec_state = latent, recurrent
+            if layer.mlp is not None:
+                lw.inter, lw.act = pad_to(layer.mlp.ff, 8), 0
+                lw.norm2 = self._f32(g(p + "norm2"), H).data_ptr()
+                lw.w_up = self._linear(_pad2(g(p + "mlp.up"), lw.inter, H)).data_ptr()
+                lw.w_down = self._linear(_pad2(g(p + "mlp.down"), H, lw.inter)).data_ptr()
+            lw.side_gate = self._linear(_pad2(g(p + "side.gate"), P, H)).data_ptr()
+            lw.side_proj = self._linear(_pad2(g(p + "side.proj"), H, P)).data_ptr()
+            lw.side_norm = self._f32(g(p + "side.norm"), H).data_ptr()
+            N.check(lib.rf_mixed_set_layer(self.handle, i, C.byref(lw)), "rf_mixed_set_layer")
+        torch.cuda.empty_cache()
+
+    def _load_latent(self, lw, m: LatentAttention, g, p: str) -> None:
+        H, R = self.H, pad_to(m.kv_rank, 16)
+        big = max(m.dim, m.vdim)
+        hd = next((x for x in (64, 128, 256) if big <= x), 0) if not self.fp32 else 0
+        D, VD = hd or pad_to(m.dim, 8), hd or pad_to(m.vdim, 8)
+        lw.mixer, lw.dim, lw.vdim, lw.vdim_true = 0, D, VD, m.vdim
+        lw.rank, lw.rank_true, lw.window, lw.scale, lw.expand_hd = R, m.kv_rank, m.window or 0, m.scale, hd
+        q = _pad_heads(_pad2(g(p + "q"), m.heads * m.dim, H), m.heads, m.dim, D)
+        dkv = _pad2(g(p + "dkv"), R, H)
+        w_in = torch.cat((q, dkv), 0)
+        lw.in_dim = w_in.shape[0]
+        lw.w_in = self._linear(w_in).data_ptr()
+        lw.latent_norm = self._f32(g(p + "dkv.norm"), R).data_ptr()
+        uk = _pad_heads(_pad2(g(p + "uk"), m.heads * m.dim, R), m.heads, m.dim, D)
+        uv = _pad_heads(_pad2(g(p + "uv"), m.heads * m.vdim, R), m.heads, m.vdim, VD)
+        lw.w_absorb = self._plain(uk.view(m.heads, D, R).transpose(1, 2)).data_ptr()
+        lw.w_unabsorb = self._plain(uv).data_ptr()
+        if hd:
+            lw.w_expand = self._linear(torch.cat((uk, uv), 0)).data_ptr()
+        o = g(p + "o")
+        o = _pad_heads(o.t().contiguous(), m.heads, m.vdim, VD).t()
+        lw.w_o = self._linear(_pad2(o, H, m.heads * VD)).data_ptr()
+
+    def _load_hgrn2(self, lw, m: HGRN2, g, p: str) -> None:
+        H, D, VD = self.H, pad_to(m.dim, 8), pad_to(m.vdim, 8)
+        lw.mixer, lw.dim, lw.vdim, lw.vdim_true = 1, D, VD, m.vdim
+        head_rows = lambda name, true, padded: _pad_heads(_pad2(g(p + name), m.heads * true, H), m.heads, true, padded)
+        w_in = torch.cat((head_rows("q", m.dim, D), head_rows("f", m.dim, D), head_rows("v", m.vdim, VD)), 0)
+        lw.in_dim = w_in.shape[0]
+        lw.w_in = self._linear(w_in).data_ptr()
+        per_head = lambda t, fill: _fill_heads(t.float(), m.heads, m.dim, D, fill)
+        lw.f_bias = self._f32(per_head(g(p + "f.b"), 0.0), m.heads * D).data_ptr()
+        lw.lower = self._f32(per_head(g(p + "lower"), 1.0), m.heads * D).data_ptr()    # padding channels keep their (zero) state
+        lw.head_norm = self._f32(g(p + "norm"), VD).data_ptr()
+        o = _pad_heads(g(p + "o").t().contiguous(), m.heads, m.vdim, VD).t()
+        lw.w_o = self._linear(_pad2(o, H, m.heads * VD)).data_ptr()
+
+    # ------------------------------------------------------------------ cache
+    def _check_cache(self, cache) -> None:
+        if not isinstance(cache, MixedCache) or cache.cfg != self.cfg or cache.dtype != self.dtype or cache.batch_size > self.max_batch:
+            raise RPUBackendError(f"{self.cfg.name}: the cache was not made for this model (dtype {getattr(cache, 'dtype', None)}, batch "
+                                  f"{getattr(cache, 'batch_size', None)}; engine {self.dtype}, max_batch {self.max_batch})")
+
+    def make_cache(self, batch_size: int, max_seq_len: int, *, pool_tokens: Optional[int] = None):
+        """A cache object for this model (``RPUCache.from_model`` ends here)."""
+        from ..api.cache import RPUMixedCache
+        return RPUMixedCache(self.cfg, batch_size, max_seq_len, device=self.device, dtype=self.dtype, pool_tokens=pool_tokens)
+
+    def bind_cache(self, cache) -> None:
+        if cache is self.cache:
+            return
+        self._check_cache(cache)
+        for i in range(self.cfg.num_layers):
+            N.check(N.lib().rf_mixed_set_state(self.handle, i, *(C.c_void_p(x) for x in cache.layer_ptrs(i))), "rf_mixed_set_state")
+        self.cache = cache
+        self.graphs.clear()
+        self.batch = 0
+
+    def reset(self) -> None:
+        for s in range(self.cache.batch_size):
+            self.cache.release(s)
+        self.step.zero_()
+        self.batch = 0
+
+    # ------------------------------------------------------------------ launches
+    def _rows(self, r: "N.RfRows", num_seqs: int) -> None:
+        r.page_table, r.pt_stride, r.num_seqs = self.cache.page_table.data_ptr(), self.cache.page_table.stride(0), num_seqs
+
+    def _logits_of(self, row_idx: Optional[torch.Tensor], rows: int, out: torch.Tensor) -> None:
+        N.check(N.lib().rf_mixed_head(self.handle, C.c_void_p(None if row_idx is None else row_idx.data_ptr()), rows,
+                                      C.c_void_p(self.out_ids.data_ptr()), C.c_void_p(self.out_vals.data_ptr()),
+                                      C.c_void_p(out.data_ptr()), self._stream()), "rf_mixed_head")
+
+    def _prefill_chunk(self, ch, prompts, lens, starts, first, logits_all, inputs_embeds, positions3, deepstack=None,
+                       row_logits=None, slots=None, taps: Optional[torch.Tensor] = None) -> None:
+        if inputs_embeds is not None or positions3 is not None or deepstack is not None:
+            raise RPUBackendError(f"{self.cfg.name} takes token ids only")
+        ch = sorted(ch, key=lambda c: c[2] >= self.long_min)          # short portions first (stable)
+        T, n = sum(c[2] for c in ch), len(ch)
+        seq_meta = torch.empty((4, n), dtype=torch.int32)             # q_start, q_len, first position, slot
+        tok_meta = torch.empty((3, T), dtype=torch.int32)             # sequence, position, token id
+        o = 0
+        for j, (s, off, cnt) in enumerate(ch):
+            pos0 = starts[s] + off
+            seq_meta[0, j], seq_meta[1, j], seq_meta[2, j], seq_meta[3, j] = o, cnt, pos0, slots[s]
+            tok_meta[0, o:o + cnt] = j
+            tok_meta[1, o:o + cnt] = torch.arange(pos0, pos0 + cnt, dtype=torch.int32)
+            tok_meta[2, o:o + cnt] = prompts[s][off:off + cnt].to("cpu", torch.int32)
+            o += cnt
+        sm, tm = seq_meta.pin_memory().to(self.device, non_blocking=True), tok_meta.pin_memory().to(self.device, non_blocking=True)
+        short = [c for c in ch if c[2] < self.long_min]
+        f = N.RfMixedForward()
+        f.rows.q_start, f.rows.q_len, f.rows.slot = sm[0].data_ptr(), sm[1].data_ptr(), sm[3].data_ptr()
+        f.rows.seq_of_row, f.rows.pos, f.ids = tm[0].data_ptr(), tm[1].data_ptr(), tm[2].data_ptr()
+        self._rows(f.rows, n)
+        f.tokens, f.short_seqs, f.short_rows, f.decode = T, len(short), sum(c[2] for c in short), 0
+        f.max_kv = max(starts[s] + off + cnt for s, off, cnt in (short or ch))
+        f.h_q_len, f.h_pos0 = seq_meta[1].data_ptr(), seq_meta[2].data_ptr()
+        f.taps = None if taps is None else taps.data_ptr()
+        N.check(N.lib().rf_mixed_forward(self.handle, C.byref(f), self._stream()), "rf_mixed_forward")
+        # rows whose logits are wanted, then the last rows of the prompts that end in this chunk (for the next token)
+        jobs, row0 = [], {}
+        o = 0
+        for (s, off, cnt) in ch:
+            row0[s] = o
+            if row_logits is not None:
+                jobs += [(o + r, s, True) for r in self._wanted_rows(row_logits, s, off, cnt, lens[s])]
+            if off + cnt == lens[s]:
+                jobs.append((o + cnt - 1, s, False))
+            o += cnt
+        for b0 in range(0, len(jobs), self.head_rows):
+            sub = jobs[b0:b0 + self.head_rows]
+            idx = torch.tensor([r for r, _, _ in sub], dtype=torch.int32).pin_memory().to(self.device, non_blocking=True)
+            lg = torch.empty((len(sub), self.vocab_ld), dtype=self.dtype, device=self.device)
+            self._logits_of(idx, len(sub), lg)
+            for k, (_, s, wanted) in enumerate(sub):
+                if wanted:
+                    row_logits["out"][s].append(lg[k:k + 1, :self.vocab_local])
+                else:
+                    first[s:s + 1].copy_(self.out_ids[k:k + 1])
+                    if logits_all is not None:
+                        logits_all[s].copy_(lg[k, :self.vocab_local])
+
+    @torch.no_grad()
+    def residual_taps(self, tokens: torch.Tensor) -> torch.Tensor:
+        """The fp32 residual stream after every layer ``[layers, tokens, hidden]`` of one prompt run from position 0 in slot 0
+        (diagnostics and tests)."""
+        n = int(tokens.numel())
+        self.reset()
+        self.cache.ensure(0, n)
+        self.cache.sync_table()
+        taps = torch.zeros((self.cfg.num_layers, n, self.H), dtype=torch.float32, device=self.device)
+        first = torch.zeros(1, dtype=torch.int32, device=self.device)
+        self._prefill_chunk([(0, 0, n)], [tokens], [n], [0], first, None, None, None, slots=[0], taps=taps)
+        self.cache.release(0)
+        return taps[:, :, :self.cfg.hidden_size]
+
+    def _decode_step(self, B: int, logits_out: Optional[torch.Tensor] = None) -> None:
+        f = N.RfMixedForward()
+        f.ids, f.rows.pos, f.rows.slot = self.ids.data_ptr(), self.pos.data_ptr(), self.slot.data_ptr()
+        self._rows(f.rows, B)
+        f.tokens = f.short_seqs = f.short_rows = B
+        f.decode, f.max_kv = 1, self.cache.max_seq_len
+        N.check(N.lib().rf_mixed_forward(self.handle, C.byref(f), self._stream()), "rf_mixed_forward")
+        self._logits_of(None, B, self.logits)
+        N.check(N.lib().rf_decode_advance(C.c_void_p(self.pos.data_ptr()), 1, C.c_void_p(self.kv_len.data_ptr()), B,
+                                          C.c_void_p(self.out_ids.data_ptr()), C.c_void_p(self.ids.data_ptr()),
+                                          C.c_void_p(self.hist.data_ptr()), C.c_void_p(self.step.data_ptr()),
+                                          self.hist_steps, self._stream()), "rf_decode_advance")
+
+    def _decode_state(self) -> List[torch.Tensor]:
+        return [self.pos, self.kv_len, self.ids, self.step] + self.cache.state_tensors()
+
+    # ------------------------------------------------------------------ scheduler step
+    @torch.no_grad()
+    def run_step(self, tokens: Sequence[torch.Tensor], slots: Sequence[int], want: Sequence[Sequence[int]]):
+        """See :meth:`DecoderEngine.run_step`.  A step of single tokens replays the decode graph of its batch size."""
+        if any(int(t.numel()) != 1 for t in tokens) or len(tokens) > self.max_batch:
+            return super().run_step(tokens, slots, want)
+        cache, B = self.cache, len(tokens)
+        slots = [int(s) for s in slots]
+        if len(set(slots)) != B or any(not 0 <= s < cache.batch_size for s in slots):
+            raise RPUBackendError(f"slots {slots} are not {B} different slots of a cache with {cache.batch_size}")
+        for s in slots:
+            cache.check_fits(s, 1)
+        for s in slots:
+            cache.ensure(s, int(cache.lengths[s]) + 1)
+        cache.sync_table()
+        host = torch.tensor([[int(t) for t in tokens], [int(cache.lengths[s]) for s in slots], slots], dtype=torch.int32).pin_memory()
+        dev = host.to(self.device, non_blocking=True)
+        self.ids[:B].copy_(dev[0])
+        self.pos[:B, 0].copy_(dev[1])
+        self.slot[:B].copy_(dev[2])
+        self.batch = 0
+        self.capture(B)
+        self.graphs[B].replay()
+        for s in slots:
+            cache.lengths[s] += 1
+        lg = self.logits[:B, :self.vocab_local].clone()
+        return self.out_ids[:B].clone(), [lg[i:i + 1].expand(len(w), -1) for i, w in enumerate(want)]
+
+    def extend(self, tokens, **kw):
+        out = super().extend(tokens, **kw)
+        if self.batch:
+            self.slot.copy_(torch.arange(self.max_batch, dtype=torch.int32, device=self.device))
+        return out
+
+    def close(self) -> None:
+        torch.cuda.synchronize()
+        self.graphs.clear()
+        if getattr(self, "handle", None) is not None:
+            N.lib().rf_mixed_destroy(self.handle)
+            self.handle = None
+        if getattr(self, "cache", None) is not None:
+            self.cache.close()
+
+
+def _fill_heads(t: torch.Tensor, heads: int, true: int, padded: int, fill: float) -> torch.Tensor:
+    out = torch.full((heads, padded), fill, dtype=t.dtype, device=t.device)
+    out[:, :true] = t.view(heads, true)
+    return out.reshape(-1)
+
+
+__all__ = ["MixedDecoderEngine"]
