@@ -34,31 +34,17 @@ __global__ void latent_insert_kernel(const T* __restrict__ x, int64_t ldx, const
   for (int i = lane; i < rank; i += 32) dst[i] = Num<T>::from_f(Num<T>::to_f(xr[i]) * rstd * w[i]);
 }
 
-// cached tokens in front of a sequence's own rows that the window of its first row reaches
-__device__ __forceinline__ int window_past(int pos0, int window) { return window > 0 ? min(pos0, window - 1) : pos0; }
-
 template <typename T>
-__global__ void latent_gather_kernel(const T* __restrict__ pool, T* __restrict__ out, const RfRows rows, int window, int rank,
-                                     int32_t* __restrict__ kv_start, int32_t* __restrict__ kv_len) {
+__global__ void latent_gather_kernel(const T* __restrict__ pool, T* __restrict__ out, const RfRows rows,
+                                     const int32_t* __restrict__ kv_start, const int32_t* __restrict__ kv_len, int rank) {
   pdl_prologue();
-  const int seq = blockIdx.y;
-  __shared__ int s_base;
-  if (threadIdx.x == 0) {
-    int b = 0;
-    for (int s = 0; s < seq; ++s) b += window_past(rows.pos[rows.q_start[s]], window) + rows.q_len[s];
-    s_base = b;
-  }
-  __syncthreads();
-  const int pos0 = rows.pos[rows.q_start[seq]], past = window_past(pos0, window), n = past + rows.q_len[seq];
-  if (blockIdx.x == 0 && threadIdx.x == 0) {
-    kv_start[seq] = s_base;
-    kv_len[seq] = n;
-  }
+  const int seq = blockIdx.y, n = kv_len[seq], base = kv_start[seq];
+  const int first = rows.pos[rows.q_start[seq]] + rows.q_len[seq] - n;       // position of the first copied row
   const int32_t* pt = rows.page_table + (size_t)seq_slot(rows, seq) * rows.pt_stride;
   const int per = rank / 8;
   for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < (int64_t)n * per; i += (int64_t)gridDim.x * blockDim.x) {
-    const int j = (int)(i / per), c = (int)(i % per) * 8, pos = pos0 - past + j;
-    *reinterpret_cast<Vec8<T>*>(out + (size_t)(s_base + j) * rank + c) =
+    const int j = (int)(i / per), c = (int)(i % per) * 8, pos = first + j;
+    *reinterpret_cast<Vec8<T>*>(out + (size_t)(base + j) * rank + c) =
         *reinterpret_cast<const Vec8<T>*>(pool + ((size_t)pt[pos >> 4] * 16 + (pos & 15)) * rank + c);
   }
 }
@@ -184,8 +170,8 @@ extern "C" int rf_latent_insert(const void* x, int64_t ldx, const float* norm_w,
   return RF_OK;
 }
 
-extern "C" int rf_latent_gather(const void* pool, void* out, const RfRows* rows, int32_t window, int32_t rank, int32_t max_len,
-                                int32_t* kv_start, int32_t* kv_len, int32_t dtype, rf_stream_t stream) {
+extern "C" int rf_latent_gather(const void* pool, void* out, const RfRows* rows, const int32_t* kv_start, const int32_t* kv_len,
+                                int32_t rank, int32_t max_len, int32_t dtype, rf_stream_t stream) {
   RF_SKIP_IF_REPLAYING();
   RF_REQUIRE(pool && out && kv_start && kv_len && rank > 0 && rank % 16 == 0 && max_len > 0, "latent_gather arguments");
   int rc = check_rows(rows);
@@ -194,7 +180,7 @@ extern "C" int rf_latent_gather(const void* pool, void* out, const RfRows* rows,
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int blocks = (int)std::min<int64_t>(ceil_div(max_len, 1) * (int64_t)(rank / 8) / 1024 + 1, 512);
   RF_DISPATCH3(dtype, RF_CUDA_CHECK(::rf::launch_k(latent_gather_kernel<T>, dim3(blocks, rows->num_seqs), dim3(256), 0, s, 1,
-                                                   (const T*)pool, (T*)out, *rows, window, rank, kv_start, kv_len)));
+                                                   (const T*)pool, (T*)out, *rows, kv_start, kv_len, rank)));
   ::rf::count_launch();
   return RF_OK;
 }

@@ -13,9 +13,21 @@
 
 namespace rf {
 
+// Prefill-sized portions under one window: how many keys each sequence sees and how the sequences are grouped so that the
+// expanded keys and values of a group fit the buffers.  kv_start / kv_len are uploaded once per forward, ahead of the layer
+// loop: the attention kernels read them before their dependency wait, so no kernel of the loop may write them.
+struct PortionGroup { int seq0, seqs, total, max_len, max_q; };
+struct WindowPlan {
+  int window = 0;
+  const int32_t* kv_start = nullptr;      // device, one per prefill-sized sequence
+  const int32_t* kv_len = nullptr;
+  std::vector<PortionGroup> groups;
+};
+
 struct MixedStack {
   RfMixedConfig cfg;
   std::vector<RfMixedLayer> layers;
+  std::vector<WindowPlan> windows;        // one per distinct window of the expanded layers
   uint8_t* base = nullptr;
   uint64_t off_x[2] = {}, off_h = 0, off_cast = 0, off_wide = 0, off_mix = 0, off_y = 0, off_side = 0, off_qlat = 0, off_olat = 0,
            off_ctx = 0, off_kv = 0, off_kvmeta = 0, off_attn_ws = 0, off_head = 0, off_argmax = 0, off_sk_ws = 0, off_sk_flags = 0,
@@ -49,6 +61,13 @@ struct MixedStack {
         past = std::max<uint64_t>(past, l.window > 0 ? std::min(l.window - 1, cfg.max_seq_len) : cfg.max_seq_len);
       }
     }
+    windows.clear();
+    for (const RfMixedLayer& l : layers) {
+      if (l.mixer != RF_MIXER_LATENT_ATTENTION || l.expand_hd <= 0) continue;
+      bool known = false;
+      for (const WindowPlan& w : windows) known |= w.window == l.window;
+      if (!known) { windows.emplace_back(); windows.back().window = l.window; }
+    }
     lat_rows = std::min<int>(cfg.max_tokens, std::max(cfg.max_seqs, 512));
     ctx_rows = (int)(T + past);
     uint64_t o = 0;
@@ -65,7 +84,7 @@ struct MixedStack {
     off_attn_ws = o; o += al(attn_ws_bytes);
     off_ctx = o; o += al(kvw ? (uint64_t)ctx_rows * rank * e : 0);
     off_kv = o; o += al((uint64_t)ctx_rows * kvw * e);
-    off_kvmeta = o; o += al((uint64_t)cfg.max_seqs * 2 * sizeof(int32_t));
+    off_kvmeta = o; o += al((uint64_t)cfg.max_seqs * 2 * windows.size() * sizeof(int32_t));
     off_head = o; o += al((uint64_t)std::max(cfg.max_seqs, 64) * H * e);
     argmax_bytes = rf_argmax_scratch_bytes(std::max(cfg.max_seqs, 64), cfg.vocab);
     off_argmax = o; o += al(argmax_bytes);
@@ -149,39 +168,60 @@ static int latent_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedF
   }
   if (!expand) return RF_OK;
   // ---- prefill-sized portions: keys and values of the visible rows, group by group so that the buffers stay bounded
-  int row = f.short_rows;
-  int32_t* kv_start = s.at<int32_t>(s.off_kvmeta);
-  int32_t* kv_len = kv_start + c.max_seqs;
-  for (int s0 = f.short_seqs; s0 < f.rows.num_seqs;) {
-    int s1 = s0, total = 0, max_len = 0, max_q = 0, q_rows = 0;
-    for (; s1 < f.rows.num_seqs; ++s1) {
-      const int past = w.window > 0 ? std::min(f.h_pos0[s1], w.window - 1) : f.h_pos0[s1], len = past + f.h_q_len[s1];
-      if (s1 > s0 && total + len > s.ctx_rows) break;
-      RF_REQUIRE(len <= s.ctx_rows, "mixed stack: %d visible rows exceed the plan (%d)", len, s.ctx_rows);
-      total += len; q_rows += f.h_q_len[s1];
-      max_len = std::max(max_len, len); max_q = std::max(max_q, f.h_q_len[s1]);
-    }
-    const RfRows g = sub_rows(f.rows, s0, s1 - s0);
+  const WindowPlan* plan = nullptr;
+  for (const WindowPlan& p : s.windows)
+    if (p.window == w.window) plan = &p;
+  RF_REQUIRE(plan != nullptr, "mixed stack: no plan for window %d", w.window);
+  for (const PortionGroup& grp : plan->groups) {
+    const RfRows g = sub_rows(f.rows, f.short_seqs + grp.seq0, grp.seqs);
+    const int32_t* kv_start = plan->kv_start + grp.seq0;
+    const int32_t* kv_len = plan->kv_len + grp.seq0;
     void* ctx = s.at(s.off_ctx);
     uint8_t* kv = s.at<uint8_t>(s.off_kv);
     const int KD = w.heads * w.expand_hd, KV = 2 * KD;
-    rc = rf_latent_gather(w.latent_pool, ctx, &g, w.window, w.rank, max_len, kv_start, kv_len, c.dtype, st);
+    rc = rf_latent_gather(w.latent_pool, ctx, &g, kv_start, kv_len, w.rank, grp.max_len, c.dtype, st);
     if (rc) return rc;
-    rc = linear(s, ctx, w.rank, w.w_expand, kv, KV, total, KV, w.rank, kActNone, st);
+    rc = linear(s, ctx, w.rank, w.w_expand, kv, KV, grp.total, KV, w.rank, kActNone, st);
     if (rc) return rc;
     RfAttn a = {};
     a.q = wide; a.ldq = w.in_dim; a.out = mix; a.ldo = VD; a.q_rows_total = T;     // q_start holds rows of the whole batch
-    a.k = kv; a.v = kv + (size_t)KD * e; a.ldk = KV; a.ldv = KV; a.kv_rows_total = total;
-    a.num_seqs = s1 - s0; a.Hq = w.heads; a.Hkv = w.heads; a.hd = w.expand_hd;
+    a.k = kv; a.v = kv + (size_t)KD * e; a.ldk = KV; a.ldv = KV; a.kv_rows_total = grp.total;
+    a.num_seqs = grp.seqs; a.Hq = w.heads; a.Hkv = w.heads; a.hd = w.expand_hd;
     a.q_start = g.q_start; a.q_len = g.q_len; a.kv_start = kv_start; a.kv_len = kv_len;
-    a.max_q_len = max_q; a.max_kv_len = max_len; a.causal = 1; a.window = w.window > 0 ? w.window : 0;
+    a.max_q_len = grp.max_q; a.max_kv_len = grp.max_len; a.causal = 1; a.window = w.window > 0 ? w.window : 0;
     a.scale = w.scale; a.status = s.status(); a.dtype = c.dtype;
     rc = rf_attn_prefill(&a, st);
     if (rc) return rc;
-    row += q_rows;
-    s0 = s1;
   }
-  (void)row;
+  return RF_OK;
+}
+
+// Group the prefill-sized sequences of this forward per window and upload their key ranges.
+static int plan_windows(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
+  const int n = f.rows.num_seqs - f.short_seqs;
+  if (n <= 0 || s.windows.empty()) return RF_OK;
+  int32_t* dev = s.at<int32_t>(s.off_kvmeta);
+  std::vector<int32_t> host((size_t)s.windows.size() * 2 * n);
+  for (size_t i = 0; i < s.windows.size(); ++i) {
+    WindowPlan& p = s.windows[i];
+    int32_t* start = host.data() + i * 2 * n;
+    int32_t* len = start + n;
+    p.kv_start = dev + i * 2 * n; p.kv_len = p.kv_start + n;
+    p.groups.clear();
+    for (int j = 0; j < n; ++j) {
+      const int q = f.h_q_len[f.short_seqs + j], pos0 = f.h_pos0[f.short_seqs + j];
+      len[j] = (p.window > 0 ? std::min(pos0, p.window - 1) : pos0) + q;
+      RF_REQUIRE(q > 0 && len[j] <= s.ctx_rows, "mixed stack: %d visible rows exceed the plan (%d)", len[j], s.ctx_rows);
+      if (p.groups.empty() || p.groups.back().total + len[j] > s.ctx_rows) p.groups.push_back(PortionGroup{j, 0, 0, 0, 0});
+      PortionGroup& g = p.groups.back();
+      start[j] = g.total;
+      ++g.seqs;
+      g.total += len[j];
+      g.max_len = std::max(g.max_len, (int)len[j]);
+      g.max_q = std::max(g.max_q, q);
+    }
+  }
+  RF_CUDA_CHECK(cudaMemcpyAsync(dev, host.data(), host.size() * sizeof(int32_t), cudaMemcpyHostToDevice, st));
   return RF_OK;
 }
 
@@ -220,6 +260,8 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
   else RF_REQUIRE(f.rows.seq_of_row && f.rows.q_start && f.rows.q_len, "mixed stack: portions need seq_of_row, q_start and q_len");
   if (f.short_seqs < f.rows.num_seqs) RF_REQUIRE(f.h_q_len && f.h_pos0, "mixed stack: portions need the host arrays");
   if (f.tokens == 0) return RF_OK;
+  int rc = plan_windows(s, f, st);
+  if (rc) return rc;
   const int T = f.tokens, H = c.hidden;
   void* h = s.at(s.off_h);
   void* cast = s.at(s.off_cast);
@@ -229,7 +271,6 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
   int cur = -1;                       // stream buffer in use; -1: still the embedding
   const void* pend = nullptr;         // sublayer output that the next stream_norm adds
   const float* pend_norm = nullptr;
-  int rc = RF_OK;
   // stream step: adds the pending output, optionally writes the 16-bit copy and / or the normalised rows
   auto step = [&](const float* norm_w, const float* shift, float* shift_state, bool want_cast) -> int {
     RfStreamNorm a = {};

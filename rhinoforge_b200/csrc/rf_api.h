@@ -346,11 +346,10 @@ int rf_head_linear(const RfHeadLinear* a, rf_stream_t stream);
 // rf_latent_insert: c = x / rms(x) * norm_w (mean over the true rank), stored at the row's position.
 int rf_latent_insert(const void* x, int64_t ldx, const float* norm_w, void* pool, const RfRows* rows, int32_t n_rows,
                      int32_t rank, int32_t rank_true, float eps, int32_t dtype, rf_stream_t stream);
-// Dense copies of the latents that the rows of num_seqs sequences can see under a window (the last min(first position,
-// window - 1) cached tokens and the sequence's own rows), packed back to back; kv_start / kv_len (device, [num_seqs])
-// receive each sequence's first row and row count.  window <= 0: everything.  max_len: host bound of kv_len.
-int rf_latent_gather(const void* pool, void* out, const RfRows* rows, int32_t window, int32_t rank, int32_t max_len,
-                     int32_t* kv_start, int32_t* kv_len, int32_t dtype, rf_stream_t stream);
+// Dense copies of the latents that sequences can see: the last kv_len[s] cached rows of sequence s, its own new rows (already
+// inserted) included, to rows [kv_start[s], kv_start[s] + kv_len[s]) of out.  max_len: host bound of kv_len.
+int rf_latent_gather(const void* pool, void* out, const RfRows* rows, const int32_t* kv_start, const int32_t* kv_len, int32_t rank,
+                     int32_t max_len, int32_t dtype, rf_stream_t stream);
 
 // Attention in the latent space (keys and values folded into the queries and the output): every row attends from its own
 // position to the window before it, score = (q[r, h] . c[j]) * scale, o[r, h] = sum_j softmax(score)_j c[j].
