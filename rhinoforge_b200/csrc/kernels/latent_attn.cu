@@ -213,9 +213,9 @@ static int launch_latent_attn(const RfLatentAttn* a, cudaStream_t s) {
     ::rf::count_launch();                                                                                         \
     return RF_OK;                                                                                                 \
   }
-  RF_LA(2) RF_LA(4) RF_LA(8) RF_LA(16) RF_LA(32)
+  RF_LA(2) RF_LA(4) RF_LA(8) RF_LA(16) RF_LA(32) RF_LA(64)
 #undef RF_LA
-  return fail(RF_ERR_UNSUPPORTED, "latent attention: rank %d is larger than 1024", a->rank);
+  return fail(RF_ERR_UNSUPPORTED, "latent attention: rank %d is larger than 2048", a->rank);
 }
 
 extern "C" int rf_latent_attn(const RfLatentAttn* a, rf_stream_t stream) {

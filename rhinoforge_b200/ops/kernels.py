@@ -554,6 +554,124 @@ def unit_tril_inv(m: torch.Tensor) -> torch.Tensor:
     return out
 
 
+# ----------------------------------------------------------------------------- decoders with per-layer mixers
+def dtype_code_any(t: torch.dtype) -> int:
+    """Like :func:`dtype_code`, for the kernels that also run in fp32."""
+    return 2 if t == torch.float32 else dtype_code(t)
+
+
+def rows(pos: torch.Tensor, *, seq_of_row: Optional[torch.Tensor] = None, q_start: Optional[torch.Tensor] = None,
+         q_len: Optional[torch.Tensor] = None, slot: Optional[torch.Tensor] = None, page_table: Optional[torch.Tensor] = None):
+    """Launch description of packed rows (``RfRows``): int32 device tensors; without ``q_start`` every row is a sequence."""
+    r = N.RfRows()
+    r.pos, r.seq_of_row, r.q_start, r.q_len, r.slot = _i32(pos), _i32(seq_of_row), _i32(q_start), _i32(q_len), _i32(slot)
+    if page_table is not None:
+        r.page_table, r.pt_stride = _i32(page_table), page_table.stride(0)
+    r.num_seqs = int(q_len.numel() if q_len is not None else pos.numel())
+    r._keep = (pos, seq_of_row, q_start, q_len, slot, page_table)
+    return r
+
+
+def stream_norm(x: Optional[torch.Tensor], r, *, dtype: torch.dtype, eps: float, norm_w: Optional[torch.Tensor] = None,
+                table: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None,
+                y_norm_w: Optional[torch.Tensor] = None, shift: Optional[torch.Tensor] = None,
+                shift_state: Optional[torch.Tensor] = None, dim: Optional[int] = None, cast: bool = False):
+    """One step of an fp32 residual stream: add the outstanding sublayer output ``y`` (RMS-normed with ``y_norm_w``), RMSNorm
+    with ``norm_w``, mix with the previous token's normalised row (``shift``, state per slot).  Without ``x`` the stream starts
+    from ``table[ids]``.  Returns ``(x_out fp32, h or None, x in dtype or None)``."""
+    H = (x if x is not None else table).shape[1]
+    n = x.shape[0] if x is not None else ids.numel()
+    dev = (x if x is not None else table).device
+    a = N.RfStreamNorm()
+    x_out = torch.empty((n, H), dtype=torch.float32, device=dev)
+    h = torch.empty((n, H), dtype=dtype, device=dev) if norm_w is not None else None
+    xc = torch.empty((n, H), dtype=dtype, device=dev) if cast else None
+    a.x, a.table, a.ids, a.y, a.y_norm_w = _ptr(x), _ptr(table), _ptr(ids), _ptr(y), _ptr(y_norm_w)
+    a.x_out, a.x_cast, a.norm_w, a.out, a.shift, a.shift_state = _ptr(x_out), _ptr(xc), _ptr(norm_w), _ptr(h), _ptr(shift), _ptr(shift_state)
+    a.rows, a.n_rows, a.H, a.dim, a.eps, a.dtype = r, n, H, dim or H, eps, dtype_code_any(dtype)
+    N.check(N.lib().rf_stream_norm(C.byref(a), _stream()), "rf_stream_norm")
+    return x_out, h, xc
+
+
+def gemm_f32(x: torch.Tensor, w: torch.Tensor, act: Optional[str] = None) -> torch.Tensor:
+    """``act(x @ w.T)`` in true fp32."""
+    assert x.dtype == torch.float32 and w.dtype == torch.float32 and x.stride(1) == 1 and w.stride(1) == 1
+    out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32, device=x.device)
+    g = N.RfGemm()
+    g.x, g.ldx, g.w, g.ldw, g.out, g.ldo = x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0)
+    g.M, g.N, g.K, g.dtype, g.act = x.shape[0], w.shape[0], x.shape[1], 2, ACT[act]
+    N.check(N.lib().rf_gemm_f32(C.byref(g), _stream()), "rf_gemm_f32")
+    return out
+
+
+def token_gate(g: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, col0: int) -> torch.Tensor:
+    """In place ``g[r] *= table[ids[r], col0 : col0 + cols]``."""
+    N.check(N.lib().rf_token_gate(C.c_void_p(g.data_ptr()), C.c_int64(g.stride(0)), C.c_void_p(table.data_ptr()),
+                                  C.c_int64(table.stride(0)), C.c_void_p(_i32(ids)), col0, g.shape[0], g.shape[1],
+                                  dtype_code_any(g.dtype), _stream()), "rf_token_gate")
+    return g
+
+
+def head_linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """Per-head linear map ``[rows, heads, k] x [heads, n, k] -> [rows, heads, n]`` (``x`` contiguous in its last dim)."""
+    R, Hh, Kd = x.shape
+    n = w.shape[1]
+    assert w.shape == (Hh, n, Kd) and w.is_contiguous() and x.stride(2) == 1
+    out = torch.empty((R, Hh, n), dtype=x.dtype, device=x.device)
+    a = N.RfHeadLinear()
+    a.x, a.ldx, a.xs, a.y, a.ldy, a.ys, a.w = x.data_ptr(), x.stride(0), x.stride(1), out.data_ptr(), Hh * n, n, w.data_ptr()
+    a.rows, a.heads, a.n, a.k, a.dtype = R, Hh, n, Kd, dtype_code_any(x.dtype)
+    N.check(N.lib().rf_head_linear(C.byref(a), _stream()), "rf_head_linear")
+    return out
+
+
+def latent_insert(x: torch.Tensor, norm_w: torch.Tensor, pool: torch.Tensor, r, eps: float, rank: Optional[int] = None) -> None:
+    """RMS-normed latent rows into the paged pool ``[pages, 16, rank_padded]``."""
+    N.check(N.lib().rf_latent_insert(C.c_void_p(x.data_ptr()), C.c_int64(x.stride(0)), C.c_void_p(norm_w.data_ptr()),
+                                     C.c_void_p(pool.data_ptr()), C.byref(r), x.shape[0], pool.shape[2], rank or pool.shape[2],
+                                     C.c_float(eps), dtype_code_any(x.dtype), _stream()), "rf_latent_insert")
+
+
+def latent_gather(pool: torch.Tensor, r, kv_start: torch.Tensor, kv_len: torch.Tensor, total: int, max_len: int) -> torch.Tensor:
+    """Dense copies of the last ``kv_len[s]`` cached latent rows of every sequence."""
+    out = torch.zeros((total, pool.shape[2]), dtype=pool.dtype, device=pool.device)
+    N.check(N.lib().rf_latent_gather(C.c_void_p(pool.data_ptr()), C.c_void_p(out.data_ptr()), C.byref(r), C.c_void_p(_i32(kv_start)),
+                                     C.c_void_p(_i32(kv_len)), pool.shape[2], max_len, dtype_code_any(pool.dtype), _stream()),
+            "rf_latent_gather")
+    return out
+
+
+def latent_attention(q: torch.Tensor, pool: torch.Tensor, r, *, window: int, scale: float, max_kv: int) -> torch.Tensor:
+    """Attention of ``q [rows, heads, rank]`` over the cached latent rows (keys and values both) -> ``[rows, heads, rank]``."""
+    R, Hh, rank = q.shape
+    assert q.is_contiguous() and pool.shape[2] == rank
+    o = torch.empty_like(q)
+    a = N.RfLatentAttn()
+    a.q, a.o, a.pool, a.rows = q.data_ptr(), o.data_ptr(), pool.data_ptr(), r
+    a.n_rows, a.heads, a.rank, a.window, a.max_kv, a.scale, a.dtype = R, Hh, rank, window, max_kv, scale, dtype_code_any(q.dtype)
+    need = N.lib().rf_latent_attn_scratch_bytes(R, Hh, rank, max_kv)
+    if need:
+        ws = torch.empty(need, dtype=torch.uint8, device=q.device)
+        a.ws, a.ws_bytes = ws.data_ptr(), need
+    N.check(N.lib().rf_latent_attn(C.byref(a), _stream()), "rf_latent_attn")
+    return o
+
+
+def hgrn2(x: torch.Tensor, f_bias: torch.Tensor, lower: torch.Tensor, norm_w: Optional[torch.Tensor], state: torch.Tensor, r, *,
+          eps: float, vdim: Optional[int] = None, chunked: bool = False) -> torch.Tensor:
+    """HGRN2 linear attention over packed rows ``x = [q | f | v]`` with the fp32 ``state [slots, heads, dim, vdim]`` updated in
+    place; returns the head-normed outputs ``[rows, heads * vdim]``."""
+    _, Hh, D, VD = state.shape
+    out = torch.empty((x.shape[0], Hh * VD), dtype=x.dtype, device=x.device)
+    a = N.RfHgrn2()
+    a.x, a.ldx, a.f_off, a.v_off = x.data_ptr(), x.stride(0), Hh * D, 2 * Hh * D
+    a.f_bias, a.lower, a.norm_w, a.state, a.out, a.ldo = f_bias.data_ptr(), lower.data_ptr(), _ptr(norm_w), state.data_ptr(), out.data_ptr(), Hh * VD
+    a.rows, a.heads, a.dim, a.vdim, a.vdim_true, a.eps, a.dtype = r, Hh, D, VD, vdim or VD, eps, dtype_code_any(x.dtype)
+    fn = "rf_hgrn2_chunked" if chunked else "rf_hgrn2_recurrent"
+    N.check(getattr(N.lib(), fn)(C.byref(a), _stream()), fn)
+    return out
+
+
 # ----------------------------------------------------------------------------- mixture of experts
 def moe_select(logits: torch.Tensor, k: int, *, bias: Optional[torch.Tensor] = None, score_fn: str = "sigmoid",
                norm_topk: bool = True, scale: float = 1.0, dense: bool = False):
