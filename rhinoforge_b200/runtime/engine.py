@@ -808,7 +808,7 @@ class DecoderEngine:
             for _ in range(n_steps):
                 self._decode_step(B)
         self.cache.lengths[:B] += n_steps
-        return self.hist[start:start + n_steps, :B].t()
+        return self.hist.view(-1)[start * B:(start + n_steps) * B].view(n_steps, B).t()      # rows of B: one per step of this batch
 
     def step_from_host(self, host_ids: torch.Tensor, host_out: torch.Tensor) -> None:
         """One decode step driven from the host: copy this step's input ids from pinned host

@@ -1,0 +1,256 @@
+"""Kernels of decoders with per-layer mixers, each against a plain formulation of the same operation."""
+import pytest
+import torch
+
+import _vabarax_oracle as oracle
+
+pytestmark = pytest.mark.gpu
+DTYPES = [torch.float32, torch.bfloat16]
+
+
+def K():
+    from rhinoforge_b200.ops import kernels
+    return kernels
+
+
+def i32(*v):
+    return torch.tensor(v, dtype=torch.int32, device="cuda")
+
+
+def pack(lens, pos0, slots=None):
+    """Row description of packed portions: (rows, positions, slots as a list)."""
+    q_start = [sum(lens[:i]) for i in range(len(lens))]
+    seq = [s for s, n in enumerate(lens) for _ in range(n)]
+    pos = [pos0[s] + i for s, n in enumerate(lens) for i in range(n)]
+    slots = list(range(len(lens))) if slots is None else slots
+    return dict(pos=i32(*pos), seq_of_row=i32(*seq), q_start=i32(*q_start), q_len=i32(*lens), slot=i32(*slots)), pos, seq
+
+
+def page_tables(n_slots, pages_per_seq, seed=0):
+    """A scattered page table and the number of pages it needs."""
+    g = torch.Generator().manual_seed(seed)
+    perm = torch.randperm(n_slots * pages_per_seq, generator=g).to(torch.int32)
+    return perm.view(n_slots, pages_per_seq).cuda(), n_slots * pages_per_seq
+
+
+def close(got, want, dtype, scale=1.0):
+    tol = 2e-5 if dtype == torch.float32 else 1.5e-2
+    torch.testing.assert_close(got.double().cpu(), want.double().cpu(), rtol=tol, atol=tol * scale)
+
+
+# ------------------------------------------------------------------------------------------------ residual stream
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,dim", [(40, 37), (512, 512), (4104, 4099)])
+def test_stream_norm_adds_the_pending_output_normalises_and_shifts(dtype, H, dim):
+    lens, pos0, slots = [1, 7, 2, 30], [5, 0, 9, 0], [3, 1, 0, 4]
+    d, pos, seq = pack(lens, pos0, slots)
+    n = sum(lens)
+    g = torch.Generator().manual_seed(1)
+    rnd = lambda *s: torch.nn.functional.pad(torch.randn(*s, dim, generator=g, dtype=torch.float64), (0, H - dim))
+    x, y, w, yw, mu, state = rnd(n), rnd(n).to(dtype).double(), rnd(), rnd(), torch.rand(H, generator=g, dtype=torch.float64), rnd(5)
+    f32 = lambda t: t.to("cuda", torch.float32)
+    st = f32(state)
+    x, mu, w, yw = f32(x), f32(mu), f32(w), f32(yw)
+    xo, h, xc = K().stream_norm(x, K().rows(**d), dtype=dtype, eps=1e-3, norm_w=w, y=y.to("cuda", dtype), y_norm_w=yw, shift=mu,
+                                shift_state=st, dim=dim, cast=True)
+    D = lambda t: t.double().cpu()[..., :dim]
+    X = D(x) + oracle.rms(y[:, :dim], 1e-3, D(yw))
+    N_ = oracle.rms(X, 1e-3, D(w))
+    want, want_state = torch.empty_like(N_), D(state).clone()
+    for s, L in enumerate(lens):
+        o = sum(lens[:s])
+        prev = None if pos0[s] == 0 else D(f32(state))[slots[s]]
+        want[o:o + L] = oracle.token_shift(N_[o:o + L], D(mu), prev)
+        want_state[slots[s]] = N_[o + L - 1]
+    close(xo[:, :dim], X, torch.float32, 4)
+    close(xc[:, :dim], X, dtype, 4)
+    close(h[:, :dim], want, dtype, 4)
+    close(st[:, :dim], want_state, torch.float32, 4)            # slot 2 belongs to nobody: untouched
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_stream_starts_from_the_embedding_row_and_gates_by_token(dtype):
+    g = torch.Generator().manual_seed(2)
+    table = torch.randn(11, 48, generator=g).to("cuda", dtype)
+    ids = i32(3, 10, 0, 3)
+    xo, h, _ = K().stream_norm(None, K().rows(i32(0, 0, 0, 0)), dtype=dtype, eps=1e-6, norm_w=torch.ones(48, device="cuda"), table=table, ids=ids)
+    want = table[ids.long()].double()
+    close(xo, want, torch.float32)
+    close(h, oracle.rms(want, 1e-6), dtype)
+    gate = torch.randn(4, 16, generator=g).to("cuda", dtype)
+    want = gate.double() * table[ids.long(), 24:40].double()
+    close(K().token_gate(gate, table, ids, 24), want, dtype)
+
+
+def test_fp32_gemm_and_squared_relu():
+    g = torch.Generator().manual_seed(3)
+    for M, N, Kd in ((1, 5, 8), (67, 130, 52), (200, 64, 1000)):
+        x, w = torch.randn(M, Kd, generator=g).cuda(), torch.randn(N, Kd, generator=g).cuda()
+        p = x.double() @ w.double().T
+        torch.testing.assert_close(K().gemm_f32(x, w).double(), p, rtol=1e-5, atol=1e-4)
+        torch.testing.assert_close(K().gemm_f32(x, w, "relu2").double(), torch.relu(p) ** 2, rtol=1e-4, atol=1e-3)
+        torch.testing.assert_close(K().gemm_f32(x, w, "gelu_tanh").double(), oracle.gelu_tanh(p), rtol=1e-5, atol=1e-4)
+
+
+@pytest.mark.parametrize("M", [3, 200, 700])
+def test_tensor_core_gemm_with_squared_relu(M):
+    g = torch.Generator().manual_seed(4)
+    x, w = (torch.randn(M, 256, generator=g) / 16).cuda().bfloat16(), torch.randn(384, 256, generator=g).cuda().bfloat16()
+    want = torch.relu(x.double() @ w.double().T) ** 2
+    close(K().gemm(x, K().pack_weight(w), packed_shape=(384, 256), act="relu2"), want, torch.bfloat16, 1)
+
+
+# ------------------------------------------------------------------------------------------------ latent attention
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("rows,heads,n,k", [(1, 1, 8, 16), (5, 3, 72, 40), (70, 5, 128, 96), (33, 2, 528, 64), (9, 17, 64, 528)])
+def test_head_linear(dtype, rows, heads, n, k):
+    g = torch.Generator().manual_seed(5)
+    buf = torch.randn(rows, heads * k + 24, generator=g).to("cuda", dtype)
+    x = buf[:, 8:8 + heads * k].unflatten(1, (heads, k))
+    w = (torch.randn(heads, n, k, generator=g) / k ** 0.5).to("cuda", dtype)
+    close(K().head_linear(x, w), torch.einsum("rhk,hnk->rhn", x.double(), w.double()), dtype)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_latent_insert_and_gather_through_a_scattered_page_table(dtype):
+    lens, pos0, slots = [3, 18, 1], [14, 0, 31], [2, 0, 1]
+    d, pos, seq = pack(lens, pos0, slots)
+    pt, pages = page_tables(3, 3)
+    rank, true = 48, 41
+    pool = torch.full((pages, 16, rank), 7.0, device="cuda", dtype=dtype)
+    g = torch.Generator().manual_seed(6)
+    x = torch.nn.functional.pad(torch.randn(sum(lens), true, generator=g), (0, rank - true)).to("cuda", dtype)
+    w = torch.randn(rank, generator=g).cuda()
+    r = K().rows(page_table=pt, **d)
+    K().latent_insert(x, w, pool, r, 1e-5, rank=true)
+    want = oracle.rms(x[:, :true].double().cpu(), 1e-5, w[:true].double().cpu())
+    flat = pool.view(-1, rank)
+    where = [int(pt[slots[s], p // 16]) * 16 + p % 16 for s, p in zip(seq, pos)]
+    close(flat[where][:, :true], want, dtype)
+    untouched = torch.ones(flat.shape[0], dtype=torch.bool)
+    untouched[where] = False
+    assert (flat[untouched.cuda()] == 7.0).all()
+    pool.copy_(torch.randn(pool.shape, generator=g))
+    kv_len, kv_start = [17, 10, 20], [0, 17, 27]
+    out = K().latent_gather(pool, r, i32(*kv_start), i32(*kv_len), 47, 20)
+    for s in range(3):
+        end = pos0[s] + lens[s]
+        rows = [int(pt[slots[s], p // 16]) * 16 + p % 16 for p in range(end - kv_len[s], end)]
+        assert torch.equal(out[kv_start[s]:kv_start[s] + kv_len[s]], pool.view(-1, rank)[rows])
+
+
+def latent_reference(q, pool, pt, slot_of_row, pos, window, scale):
+    out = torch.empty(q.shape, dtype=torch.float64)
+    flat = pool.view(-1, pool.shape[2]).double().cpu()
+    for r, p in enumerate(pos):
+        lo = max(0, p - window + 1) if window else 0
+        c = flat[[int(pt[slot_of_row[r], j // 16]) * 16 + j % 16 for j in range(lo, p + 1)]]
+        out[r] = torch.softmax(q[r].double().cpu() @ c.T * scale, -1) @ c
+    return out
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("heads,rank,window", [(1, 16, 1), (3, 48, 5), (16, 64, 33), (20, 208, 64), (5, 512, 0), (2, 528, 70), (33, 96, 200)])
+def test_latent_attention_windows_and_ranks(dtype, heads, rank, window):
+    pos = [0, 1, 15, 16, 40, 63, 64, 65, 127, 300, 303]
+    n = len(pos)
+    pt, pages = page_tables(n, 19, seed=heads)
+    g = torch.Generator().manual_seed(rank)
+    pool = torch.randn(pages, 16, rank, generator=g).to("cuda", dtype)
+    q = torch.randn(n, heads, rank, generator=g).to("cuda", dtype)
+    slots = [(5 * i + 3) % n for i in range(n)]
+    scale = 2.0 / rank ** 0.5
+    r = K().rows(i32(*pos), slot=i32(*slots), page_table=pt)
+    got = K().latent_attention(q, pool, r, window=window, scale=scale, max_kv=304)
+    close(got, latent_reference(q, pool, pt, slots, pos, window, scale), dtype)
+    # the same rows one launch at a time (another split of the keys)
+    for i in (0, 4, 9):
+        one = K().latent_attention(q[i:i + 1].contiguous(), pool, K().rows(i32(pos[i]), slot=i32(slots[i]), page_table=pt), window=window,
+                                   scale=scale, max_kv=304)
+        close(one[0], got[i], dtype)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("window,distance,seen", [(72, 71, True), (72, 72, False), (64, 63, True), (64, 64, False), (1, 0, True), (1, 1, False),
+                                                  (17, 16, True), (17, 17, False), (0, 299, True), (200, 199, True), (200, 200, False)])
+def test_one_key_that_stands_out_at_the_edge_of_the_window(dtype, window, distance, seen):
+    """All keys are equal but one, which wins the softmax outright when it is visible."""
+    rank, p = 32, 299
+    pt, pages = page_tables(1, 20, seed=3)
+    pool = torch.zeros(pages, 16, rank, device="cuda", dtype=dtype)
+    pool[..., 0] = 1.0
+    j = p - distance
+    pool[int(pt[0, j // 16]), j % 16] = torch.nn.functional.one_hot(torch.tensor(1), rank).to("cuda", dtype)
+    q = torch.zeros(1, 4, rank, device="cuda", dtype=dtype)
+    q[..., 1] = 30.0
+    o = K().latent_attention(q, pool, K().rows(i32(p), page_table=pt), window=window, scale=1.0, max_kv=300)
+    assert abs(float(o[0, 3, 1]) - (1.0 if seen else 0.0)) < 1e-3 and abs(float(o[0, 3, 0]) - (0.0 if seen else 1.0)) < 1e-3
+
+
+# ------------------------------------------------------------------------------------------------ HGRN2
+def hgrn2_reference(x, fb, lower, nw, state, lens, pos0, slots, heads, D, VD, eps, vdim):
+    out = torch.zeros(x.shape[0], heads, VD, dtype=torch.float64)
+    x, fb, lower, state = x.double().cpu(), fb.double().cpu(), lower.double().cpu(), state.double().cpu().clone()
+    o = 0
+    for s, L in enumerate(lens):
+        xs = x[o:o + L]
+        z = xs[:, :heads * D]
+        q = (z * torch.sigmoid(z)).view(L, heads, D)
+        f = (lower + (1 - lower) * torch.sigmoid(xs[:, heads * D:2 * heads * D] + fb)).view(L, heads, D)
+        v = xs[:, 2 * heads * D:2 * heads * D + heads * VD].view(L, heads, VD)
+        for h in range(heads):
+            start = torch.zeros(D, VD, dtype=torch.float64) if pos0[s] == 0 else state[slots[s], h]
+            y, state[slots[s], h] = oracle.gated_recurrence(q[:, h], f[:, h], v[:, h], start)
+            out[o:o + L, h, :vdim] = oracle.rms(y[:, :vdim], eps, nw.double().cpu()[:vdim])
+        o += L
+    return out.reshape(x.shape[0], heads * VD), state
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("chunked", [False, True])
+@pytest.mark.parametrize("heads,D,VD,vdim", [(1, 8, 8, 8), (2, 48, 64, 64), (3, 40, 24, 21), (2, 128, 128, 128), (1, 136, 160, 155), (1, 64, 320, 320),
+                                             (1, 272, 64, 64)])
+def test_hgrn2_against_the_recurrence(dtype, chunked, heads, D, VD, vdim):
+    lens, pos0, slots = [1, 70, 2, 16, 17, 131], [4, 0, 33, 64, 0, 9], [5, 2, 0, 1, 4, 6]
+    d, _, _ = pack(lens, pos0, slots)
+    n = sum(lens)
+    g = torch.Generator().manual_seed(D + VD)
+    width = heads * (2 * D + VD)
+    x = torch.randn(n, (width + 15) // 8 * 8, generator=g)
+    x[:, heads * D:2 * heads * D] *= 4.0                       # gates from nearly closed to nearly open
+    v = x[:, 2 * heads * D:width].view(n, heads, VD)
+    v[..., vdim:] = 0.0
+    x = x.to("cuda", dtype)
+    fb, lower = torch.randn(heads * D, generator=g).cuda(), torch.rand(heads * D, generator=g).cuda() ** 3
+    lower[0] = 0.0
+    fb[0] = -12.0                                              # one channel forgets almost everything at every token
+    lower[1] = 0.9999
+    nw = torch.nn.functional.pad(torch.randn(vdim, generator=g), (0, VD - vdim)).cuda()
+    state = torch.randn(7, heads, D, VD, generator=g)
+    state[..., vdim:] = 0.0
+    state = state.cuda()
+    want, want_state = hgrn2_reference(x, fb, lower, nw, state, lens, pos0, slots, heads, D, VD, 1e-5, vdim)
+    got = K().hgrn2(x, fb, lower, nw, state, K().rows(**d), eps=1e-5, vdim=vdim, chunked=chunked)
+    close(got, want, dtype, 4)
+    torch.testing.assert_close(state.double().cpu(), want_state, rtol=1e-4, atol=1e-4)
+
+
+def test_hgrn2_keeps_a_value_written_long_ago():
+    """A channel whose gate stays open carries one token's value over hundreds of others."""
+    D = VD = 64
+    n = 700
+    x = torch.zeros(n, 2 * D + VD, device="cuda", dtype=torch.bfloat16)
+    x[:, D:2 * D] = 20.0                                       # f = 1: nothing written, nothing forgotten
+    x[3, D + 5], x[3, 2 * D + 9] = -20.0, 3.0                  # token 3 writes value channel 9 into key channel 5
+    x[n - 1, 5] = 8.0                                          # the last token asks for key channel 5
+    fb, lower = torch.zeros(D, device="cuda"), torch.zeros(D, device="cuda")
+    for chunked in (False, True):
+        for cut in (n, 400, 100):
+            state = torch.zeros(1, 1, D, VD, device="cuda")
+            outs = []
+            for a in range(0, n, cut):
+                L = min(cut, n - a)
+                d, _, _ = pack([L], [a], [0])
+                outs.append(K().hgrn2(x[a:a + L].contiguous(), fb, lower, None, state, K().rows(**d), eps=1e-6, chunked=chunked))
+            o = torch.cat(outs)[n - 1].float()
+            assert abs(float(o[9]) - 3.0 * 8.0) < 0.2 and float(o.abs().sum() - o[9].abs()) < 0.05, (chunked, cut)
