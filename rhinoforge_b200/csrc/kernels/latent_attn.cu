@@ -87,6 +87,111 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const RfHeadLinear p) 
   }
 }
 
+__device__ __forceinline__ void la_cp16(uint32_t dst, const void* src, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void la_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void la_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// 16-bit form on the tensor cores: 64 rows x (NT * 32) outputs of one head per CTA, warps side by side along the outputs, a
+// ring of 64-wide k blocks.  The weights of the first blocks are fetched ahead of the dependency wait.
+constexpr int kHmRows = 64, kHmK = 64, kHmLd = kHmK + 8, kHmStages = 4;
+
+template <typename T, int NT>
+__global__ void __launch_bounds__(128) head_linear_mma_kernel(const RfHeadLinear p) {
+  pdl_launch_dependents();
+  constexpr int BN = NT * 32;
+  extern __shared__ __align__(16) uint8_t hsm[];
+  constexpr uint32_t kXBytes = kHmRows * kHmLd * 2, kStage = kXBytes + BN * kHmLd * 2;
+  const uint32_t ring = smem_u32(hsm);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.y, n0 = blockIdx.x * BN, r0 = blockIdx.z * kHmRows;
+  const T* x = reinterpret_cast<const T*>(p.x) + (size_t)h * p.xs;
+  const T* w = reinterpret_cast<const T*>(p.w) + (size_t)h * p.n * p.k;
+  const int nblk = (p.k + kHmK - 1) / kHmK, mt = min(4, (p.rows - r0 + 15) / 16);
+  auto load_w = [&](int b) {
+    const uint32_t dst = ring + (uint32_t)(b % kHmStages) * kStage + kXBytes;
+    for (int i = tid; i < BN * 8; i += 128) {
+      const int r = i >> 3, c = (i & 7) * 8, k = b * kHmK + c;
+      const bool ok = n0 + r < p.n && k < p.k;
+      la_cp16(dst + (uint32_t)(r * kHmLd + c) * 2, ok ? w + (size_t)(n0 + r) * p.k + k : w, ok);
+    }
+  };
+  auto load_x = [&](int b) {
+    const uint32_t dst = ring + (uint32_t)(b % kHmStages) * kStage;
+    for (int i = tid; i < mt * 16 * 8; i += 128) {
+      const int r = i >> 3, c = (i & 7) * 8, k = b * kHmK + c;
+      const bool ok = r0 + r < p.rows && k < p.k;
+      la_cp16(dst + (uint32_t)(r * kHmLd + c) * 2, ok ? x + (size_t)(r0 + r) * p.ldx + k : x, ok);
+    }
+  };
+  for (int b = 0; b < kHmStages - 1; ++b)
+    if (b < nblk) load_w(b);
+  pdl_wait();
+  for (int b = 0; b < kHmStages - 1; ++b) {
+    if (b < nblk) load_x(b);
+    la_commit();
+  }
+  float acc[4][NT][4] = {};
+  for (int b = 0; b < nblk; ++b) {
+    la_wait<kHmStages - 2>();
+    __syncthreads();
+    if (b + kHmStages - 1 < nblk) {
+      load_w(b + kHmStages - 1);
+      load_x(b + kHmStages - 1);
+    }
+    la_commit();
+    const uint32_t sx = ring + (uint32_t)(b % kHmStages) * kStage, sw = sx + kXBytes;
+#pragma unroll
+    for (int ks = 0; ks < kHmK / 32; ++ks) {
+      uint32_t bf[NT][4];
+#pragma unroll
+      for (int t = 0; t < NT; ++t)       // eight outputs, two k16 steps
+        ldsm_x4(sw + (uint32_t)((warp * NT * 8 + t * 8 + (lane & 7)) * kHmLd + ks * 32 + (lane >> 3) * 8) * 2, bf[t][0], bf[t][1], bf[t][2], bf[t][3]);
+#pragma unroll
+      for (int m = 0; m < 4; ++m) {
+        if (m < mt) {
+#pragma unroll
+          for (int hk = 0; hk < 2; ++hk) {
+            uint32_t a[4];
+            ldsm_x4(sx + (uint32_t)((m * 16 + (lane & 15)) * kHmLd + ks * 32 + hk * 16 + (lane >> 4) * 8) * 2, a[0], a[1], a[2], a[3]);
+#pragma unroll
+            for (int t = 0; t < NT; ++t) MmaOp<T>::mma(acc[m][t], a, bf[t][hk * 2], bf[t][hk * 2 + 1]);
+          }
+        }
+      }
+    }
+  }
+  T* y = reinterpret_cast<T*>(p.y) + (size_t)h * p.ys;
+  const int g = lane >> 2, q = lane & 3;
+#pragma unroll
+  for (int m = 0; m < 4; ++m)
+#pragma unroll
+    for (int t = 0; t < NT; ++t)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int r = r0 + m * 16 + g + half * 8, n = n0 + warp * NT * 8 + t * 8 + q * 2;
+        if (m < mt && r < p.rows && n < p.n)
+          *reinterpret_cast<uint32_t*>(y + (size_t)r * p.ldy + n) = MmaOp<T>::pack(acc[m][t][half * 2], acc[m][t][half * 2 + 1]);
+      }
+}
+
+template <typename T>
+static int launch_head_linear_mma(const RfHeadLinear* a, cudaStream_t s) {
+  const int rt = ceil_div(a->rows, kHmRows);
+#define RF_HM(NT)                                                                                                            \
+  do {                                                                                                                       \
+    constexpr size_t smem = (size_t)kHmStages * (kHmRows + NT * 32) * kHmLd * 2;                                              \
+    RF_ALLOW_SMEM_PER_DEVICE((head_linear_mma_kernel<T, NT>), smem);                                                         \
+    RF_CUDA_CHECK(::rf::launch_k(head_linear_mma_kernel<T, NT>, dim3(ceil_div(a->n, NT * 32), a->heads, rt), dim3(128), smem, s, 1, *a)); \
+  } while (0)
+  if ((long)ceil_div(a->n, 64) * a->heads * rt < sm_count()) RF_HM(1);
+  else RF_HM(2);
+#undef RF_HM
+  ::rf::count_launch();
+  return RF_OK;
+}
+
 // --------------------------------------------- attention in the latent space ----
 // One CTA per (row, head), four warps striding over the keys with an online softmax each, merged at the end.  A lane keeps
 // elements lane, lane + 32, .. of the query, the key row and the accumulator.  All products in fp32.
@@ -142,6 +247,203 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const RfLatentAttn p) 
   }
 }
 
+// 16-bit form on the tensor cores.  One CTA (eight warps) takes MT * 16 heads of one row and a range of its keys, 64 keys per
+// step: every warp scores 8 keys against all heads, the softmax runs row-wise over shared memory, and every warp accumulates
+// NT * 8 columns of the latent output.  The cached rows are keys and values both, so a key block is read once.  The
+// probabilities enter the second product as a 16-bit pair (value + remainder), so they keep about 16 mantissa bits.
+constexpr int kLaKeys = 64, kLaThreads = 256;
+
+struct LatentSplit {
+  float* o;      // [rows, heads, splits, rank] partial outputs, unnormalised
+  float* ml;     // [rows, heads, splits, 2] running maximum (log2 domain) and sum
+  int splits;
+};
+
+__host__ __device__ constexpr int la_ld(int rank) { return (rank + 31) / 32 * 32 + 8; }
+static size_t la_smem(int rank, int mt) {
+  return (size_t)(16 * mt + 2 * kLaKeys) * la_ld(rank) * 2 + (size_t)16 * mt * (kLaKeys + 4) * 4 + (size_t)2 * 16 * mt * (kLaKeys + 8) * 2 +
+         (size_t)16 * mt * 3 * 4;
+}
+
+template <typename T, int NT, int MT>
+__global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const RfLatentAttn p, const LatentSplit sp) {
+  pdl_prologue();
+  constexpr int M = 16 * MT, LDS = kLaKeys + 4, LDP = kLaKeys + 8;
+  extern __shared__ __align__(16) uint8_t lsm[];
+  const int rank = p.rank, ld = la_ld(rank), rp = ld - 8;
+  T* sQ = reinterpret_cast<T*>(lsm);                       // [M][ld]
+  T* sC = sQ + M * ld;                                     // [2][64][ld]
+  float* sS = reinterpret_cast<float*>(sC + 2 * kLaKeys * ld);   // [M][LDS]
+  T* sP = reinterpret_cast<T*>(sS + M * LDS);              // [2][M][LDP]: value, remainder
+  float* sM = reinterpret_cast<float*>(sP + 2 * M * LDP);  // running maximum, sum, rescale of this step
+  float* sL = sM + M;
+  float* sA = sL + M;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
+  const int split = blockIdx.x, h0 = blockIdx.y * M, row = blockIdx.z;
+  const int pos = p.rows.pos[row];
+  const int32_t* pt = p.rows.page_table + (size_t)seq_slot(p.rows, row_seq(p.rows, row)) * p.rows.pt_stride;
+  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const int blocks = (pos - lo) / kLaKeys + 1, per = (blocks + sp.splits - 1) / sp.splits;
+  const int b0 = split * per, b1 = min(blocks, b0 + per);
+  const T* pool = reinterpret_cast<const T*>(p.pool);
+  const T* q = reinterpret_cast<const T*>(p.q) + ((size_t)row * p.heads + h0) * rank;
+  const int heads_here = min(M, p.heads - h0), chunks = rp / 8;
+
+  for (int i = tid; i < M * chunks; i += kLaThreads) {
+    const int r = i / chunks, c = (i % chunks) * 8;
+    const bool ok = r < heads_here && c < rank;
+    la_cp16(smem_u32(sQ + r * ld + c), ok ? q + (size_t)r * rank + c : q, ok);
+  }
+  auto load_keys = [&](int b) {                            // four threads per key row
+    const int r = tid >> 2, j = lo + b * kLaKeys + r;
+    const bool in = j <= pos;
+    const T* src = in ? pool + ((size_t)pt[j >> 4] * 16 + (j & 15)) * rank : pool;
+    T* dst = sC + ((b & 1) * kLaKeys + r) * ld;
+    for (int c = (tid & 3) * 8; c < rp; c += 32) la_cp16(smem_u32(dst + c), in && c < rank ? src + c : pool, in && c < rank);
+  };
+  if (tid < M) { sM[tid] = -INFINITY; sL[tid] = 0.f; }
+  if (b0 < b1) load_keys(b0);
+  la_commit();
+  float acc[MT][NT][4] = {};
+  const float scale_log2 = p.scale * 1.4426950408889634f;
+
+  for (int b = b0; b < b1; ++b) {
+    if (b + 1 < b1) load_keys(b + 1);
+    la_commit();
+    la_wait<1>();
+    __syncthreads();
+    const T* kc = sC + (b & 1) * kLaKeys * ld;
+    {  // scores of this warp's eight keys
+      float s[MT][4] = {};
+      for (int k = 0; k < rp; k += 32) {
+        uint32_t bf[4];
+        ldsm_x4(smem_u32(kc + (warp * 8 + (lane & 7)) * ld + k + (lane >> 3) * 8), bf[0], bf[1], bf[2], bf[3]);
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int hk = 0; hk < 2; ++hk) {
+            uint32_t a[4];
+            ldsm_x4(smem_u32(sQ + (m * 16 + (lane & 15)) * ld + k + hk * 16 + (lane >> 4) * 8), a[0], a[1], a[2], a[3]);
+            MmaOp<T>::mma(s[m], a, bf[hk * 2], bf[hk * 2 + 1]);
+          }
+      }
+      const int key = warp * 8 + q4 * 2, j = lo + b * kLaKeys + key;
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          float2 v;
+          v.x = j <= pos ? s[m][half * 2] * scale_log2 : -INFINITY;
+          v.y = j + 1 <= pos ? s[m][half * 2 + 1] * scale_log2 : -INFINITY;
+          *reinterpret_cast<float2*>(sS + (m * 16 + g + half * 8) * LDS + key) = v;
+        }
+    }
+    __syncthreads();
+    // softmax step of 2 * MT rows per warp (every block holds at least one visible key)
+#pragma unroll
+    for (int i = 0; i < 2 * MT; ++i) {
+      const int r = warp * 2 * MT + i;
+      const float2 v = *reinterpret_cast<const float2*>(sS + r * LDS + lane * 2);
+      const float old = sM[r], mx = fmaxf(old, warp_max(fmaxf(v.x, v.y)));
+      const float p0 = exp2f(v.x - mx), p1 = exp2f(v.y - mx);
+      const float sum = warp_sum(p0 + p1);
+      const T a0 = Num<T>::from_f(p0), a1 = Num<T>::from_f(p1);
+      *reinterpret_cast<uint32_t*>(sP + r * LDP + lane * 2) = MmaOp<T>::pack(p0, p1);
+      *reinterpret_cast<uint32_t*>(sP + (M + r) * LDP + lane * 2) = MmaOp<T>::pack(p0 - Num<T>::to_f(a0), p1 - Num<T>::to_f(a1));
+      __syncwarp();
+      if (lane == 0) {
+        const float corr = exp2f(old - mx);
+        sA[r] = corr;
+        sL[r] = sL[r] * corr + sum;
+        sM[r] = mx;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const float c0 = sA[m * 16 + g], c1 = sA[m * 16 + g + 8];
+#pragma unroll
+      for (int t = 0; t < NT; ++t) {
+        acc[m][t][0] *= c0; acc[m][t][1] *= c0; acc[m][t][2] *= c1; acc[m][t][3] *= c1;
+      }
+    }
+#pragma unroll
+    for (int kk = 0; kk < kLaKeys; kk += 32) {
+      uint32_t a[MT][2][2][4];                             // [m][value / remainder][k16 step]
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int hl = 0; hl < 2; ++hl)
+#pragma unroll
+          for (int hk = 0; hk < 2; ++hk)
+            ldsm_x4(smem_u32(sP + (hl * M + m * 16 + (lane & 15)) * LDP + kk + hk * 16 + (lane >> 4) * 8), a[m][hl][hk][0], a[m][hl][hk][1],
+                    a[m][hl][hk][2], a[m][hl][hk][3]);
+#pragma unroll
+      for (int t = 0; t < NT; ++t) {
+        const int c = (warp * NT + t) * 8;
+        if (c < rp) {
+          uint32_t bf[4];                                  // eight columns, 32 keys
+          ldsm_x4_t(smem_u32(kc + (kk + lane) * ld + c), bf[0], bf[1], bf[2], bf[3]);
+#pragma unroll
+          for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int hl = 0; hl < 2; ++hl) {
+              MmaOp<T>::mma(acc[m][t], a[m][hl][0], bf[0], bf[1]);
+              MmaOp<T>::mma(acc[m][t], a[m][hl][1], bf[2], bf[3]);
+            }
+        }
+      }
+    }
+    __syncthreads();                                       // the key buffer and the score tile are free again
+  }
+  __syncthreads();                                         // also for a range without blocks
+  // ---- results
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int r = m * 16 + g + half * 8;
+      if (r >= heads_here) continue;
+      const size_t hr = (size_t)row * p.heads + h0 + r;
+      const float inv = sp.splits == 1 ? 1.f / sL[r] : 1.f;
+#pragma unroll
+      for (int t = 0; t < NT; ++t) {
+        const int c = (warp * NT + t) * 8 + q4 * 2;
+        if (c >= rank) continue;
+        const float v0 = acc[m][t][half * 2] * inv, v1 = acc[m][t][half * 2 + 1] * inv;
+        if (sp.splits == 1) *reinterpret_cast<uint32_t*>(reinterpret_cast<T*>(p.o) + hr * rank + c) = MmaOp<T>::pack(v0, v1);
+        else *reinterpret_cast<float2*>(sp.o + (hr * sp.splits + split) * rank + c) = make_float2(v0, v1);
+      }
+      if (sp.splits > 1 && warp == 0 && q4 == 0) {
+        sp.ml[(hr * sp.splits + split) * 2] = sM[r];
+        sp.ml[(hr * sp.splits + split) * 2 + 1] = sL[r];
+      }
+    }
+}
+
+template <typename T>
+__global__ void latent_combine_kernel(const LatentSplit sp, T* __restrict__ o, int rank) {
+  pdl_prologue();
+  const size_t hr = blockIdx.x;
+  const float* ml = sp.ml + hr * sp.splits * 2;
+  float m = -INFINITY, l = 0.f;
+  for (int s = 0; s < sp.splits; ++s) m = fmaxf(m, ml[s * 2]);
+  for (int s = 0; s < sp.splits; ++s) l += ml[s * 2] == -INFINITY ? 0.f : exp2f(ml[s * 2] - m) * ml[s * 2 + 1];
+  const float inv = 1.f / l;
+  for (int c = threadIdx.x; c < rank; c += blockDim.x) {
+    float v = 0.f;
+    for (int s = 0; s < sp.splits; ++s)
+      if (ml[s * 2] != -INFINITY) v += exp2f(ml[s * 2] - m) * sp.o[(hr * sp.splits + s) * rank + c];
+    o[hr * rank + c] = Num<T>::from_f(v * inv);
+  }
+}
+
+// Split the keys of a row until about one CTA per SM exists; at least two key blocks per split.
+static int la_splits(int rows, int heads, int max_kv) {
+  const int mt = heads <= 16 ? 1 : 2, ctas = rows * ceil_div(heads, 16 * mt), blocks = ceil_div(std::max(max_kv, 1), kLaKeys);
+  return std::max(1, std::min(std::min(sm_count() / std::max(ctas, 1), blocks / 2), 64));
+}
+
 }  // namespace rf
 
 using namespace rf;
@@ -192,15 +494,59 @@ extern "C" int rf_head_linear(const RfHeadLinear* a, rf_stream_t stream) {
              "head_linear: sizes and pitches must be multiples of 8");
   if (a->rows == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (a->dtype == kF16) return launch_head_linear_mma<__half>(a, s);
+  if (a->dtype == kBF16) return launch_head_linear_mma<__nv_bfloat16>(a, s);
   RF_DISPATCH3(a->dtype, RF_CUDA_CHECK(::rf::launch_k(head_linear_kernel<T>, dim3(ceil_div(a->n, kHlN), a->heads, ceil_div(a->rows, kHlRows)),
                                                       dim3(128), 0, s, 1, *a)));
   ::rf::count_launch();
   return RF_OK;
 }
 
+// Room for the largest split of any launch of at most `rows` rows.
 extern "C" uint64_t rf_latent_attn_scratch_bytes(int rows, int heads, int rank, int max_kv) {
-  (void)rows; (void)heads; (void)rank; (void)max_kv;
-  return 0;
+  uint64_t most = 0;
+  const int ht = ceil_div(std::max(heads, 1), heads <= 16 ? 16 : 32);
+  for (int r = 1; r <= rows && r * ht <= sm_count(); ++r) {
+    const int sp = la_splits(r, heads, max_kv);
+    if (sp > 1) most = std::max<uint64_t>(most, (uint64_t)r * heads * sp * (rank + 2) * sizeof(float));
+  }
+  return most;
+}
+
+template <typename T>
+static int launch_latent_attn_mma(const RfLatentAttn* a, cudaStream_t s) {
+  LatentSplit sp = {};
+  sp.splits = la_splits(a->n_rows, a->heads, a->max_kv);
+  const uint64_t slots = (uint64_t)a->n_rows * a->heads * sp.splits;
+  if (sp.splits > 1 && (!a->ws || a->ws_bytes < slots * (a->rank + 2) * sizeof(float))) sp.splits = 1;
+  sp.o = a->ws;
+  sp.ml = a->ws ? a->ws + slots * a->rank : nullptr;
+  const int mt = a->heads <= 16 ? 1 : 2;
+  const size_t smem = la_smem(a->rank, mt);
+  const dim3 grid(sp.splits, ceil_div(a->heads, 16 * mt), a->n_rows);
+#define RF_LM(NT, MT)                                                                                             \
+  do {                                                                                                            \
+    RF_ALLOW_SMEM_PER_DEVICE((latent_attn_mma_kernel<T, NT, MT>), la_smem(NT * 64, MT));                          \
+    RF_CUDA_CHECK(::rf::launch_k(latent_attn_mma_kernel<T, NT, MT>, grid, dim3(kLaThreads), smem, s, 1, *a, sp)); \
+  } while (0)
+#define RF_LN(NT)             \
+  do {                        \
+    if (mt == 1) RF_LM(NT, 1); \
+    else RF_LM(NT, 2);         \
+  } while (0)
+  if (a->rank <= 64) RF_LN(1);
+  else if (a->rank <= 128) RF_LN(2);
+  else if (a->rank <= 256) RF_LN(4);
+  else RF_LN(8);
+#undef RF_LN
+#undef RF_LM
+  ::rf::count_launch();
+  if (sp.splits > 1) {
+    RF_CUDA_CHECK(::rf::launch_k(latent_combine_kernel<T>, dim3(a->n_rows * a->heads), dim3(std::min(512, round_up(a->rank, 32))), 0, s, 1,
+                                 sp, (T*)a->o, a->rank));
+    ::rf::count_launch();
+  }
+  return RF_OK;
 }
 
 template <typename T>
@@ -225,5 +571,7 @@ extern "C" int rf_latent_attn(const RfLatentAttn* a, rf_stream_t stream) {
   if (rc) return rc;
   if (a->n_rows == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (a->rank <= 512 && a->dtype == kF16) return launch_latent_attn_mma<__half>(a, s);
+  if (a->rank <= 512 && a->dtype == kBF16) return launch_latent_attn_mma<__nv_bfloat16>(a, s);
   RF_DISPATCH3(a->dtype, return launch_latent_attn<T>(a, s));
 }
