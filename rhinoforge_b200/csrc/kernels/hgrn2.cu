@@ -139,6 +139,330 @@ static int launch_recurrent(const RfHgrn2* a, cudaStream_t s) {
   return RF_OK;
 }
 
+// ------------------------------------------------------- block form (prefill) ----
+// Sixteen tokens per step.  With G_t the product of the gates from the block's start to t (inclusive), E_t the product of the
+// gates behind t to the block's end and S the state ahead of the block:
+//     O = (q * G) S + tril(P) V,   P[t, s] = sum_c q_t[c] (1 - f_s[c]) prod_{s < r <= t} f_r[c]
+//     S' = G_last * S + ((1 - f) * E)^T V
+// Every factor is a product of gates in [0, 1], built by running products: no logarithms, no exponentials of differences, and
+// nothing can overflow however fast a channel forgets.  P is evaluated in fp32 on the CUDA cores (its cost does not grow with
+// the sequence), the three matrix products run on the tensor cores with their fp32 operands as bf16 pairs (value + remainder,
+// about 16 mantissa bits; the values V are bf16 already).  The transposed state lives in the accumulator registers of the
+// warps - 16 value channels x a share of the key channels each - where the product with it reads it as an operand.
+// A CTA owns VG * 16 value channels of one head of one sequence; the CTAs of a head form a cluster that exchanges the sums of
+// squares of the head norm one step behind the computation.
+constexpr int kHcTok = 16, kHcThreads = 256, kHcWarps = 8;
+
+struct Hgrn2Smem {
+  int dp, raw_ld, q_ld, b_ld, o_ld;
+  uint32_t raw, sq, sf, qh, ql, kh, kl, gt, ph, pl, so, csum, total;
+};
+__host__ __device__ inline Hgrn2Smem hgrn2_smem(int dim, int vt, int dg) {
+  Hgrn2Smem m;
+  m.dp = (dim + 15) / 16 * 16;
+  m.raw_ld = 2 * m.dp + vt + 8;
+  m.q_ld = m.dp + 4;
+  m.b_ld = m.dp + 8;
+  m.o_ld = vt + 4;
+  uint32_t o = 0;
+  m.raw = o; o += 2 * kHcTok * m.raw_ld * 2;
+  m.sq = o; o += kHcTok * m.q_ld * 4;
+  m.sf = o; o += kHcTok * m.q_ld * 4;
+  m.qh = o; o += kHcTok * m.b_ld * 2;
+  m.ql = o; o += kHcTok * m.b_ld * 2;
+  m.kh = o; o += kHcTok * m.b_ld * 2;
+  m.kl = o; o += kHcTok * m.b_ld * 2;
+  m.gt = o; o += m.dp * 4;
+  m.ph = o; o += kHcTok * 24 * 2;
+  m.pl = o; o += kHcTok * 24 * 2;
+  m.so = o; o += dg * kHcTok * m.o_ld * 4;
+  m.csum = o; o += 2 * kHcTok * 4;
+  m.total = o;
+  return m;
+}
+
+__device__ __forceinline__ void hc_cp16(uint32_t dst, const void* src, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void hc_split(float v, __nv_bfloat16& hi, __nv_bfloat16& lo) {
+  hi = __float2bfloat16_rn(v);
+  lo = __float2bfloat16_rn(v - __bfloat162float(hi));
+}
+// value and remainder of two floats, packed
+__device__ __forceinline__ void hc_split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+  __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  const float2 f = __bfloat1622float2(h);
+  __nv_bfloat162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
+  hi = *reinterpret_cast<uint32_t*>(&h);
+  lo = *reinterpret_cast<uint32_t*>(&l);
+}
+
+// VG: groups of 16 value channels per CTA; the 8 / VG warps of a group share its key channels, DT 16-channel tiles each.
+template <int VG, int DT>
+__global__ void __launch_bounds__(kHcThreads, 1) hgrn2_chunked_kernel(const RfHgrn2 p, int col_tiles) {
+  pdl_prologue();
+  using T = __nv_bfloat16;
+  constexpr int VT = VG * 16, DG = kHcWarps / VG, NV = VT / 16;
+  extern __shared__ __align__(16) uint8_t csm[];
+  const Hgrn2Smem L = hgrn2_smem(p.dim, VT, DG);
+  const int DP = L.dp;
+  T* raw = reinterpret_cast<T*>(csm + L.raw);
+  float* sq = reinterpret_cast<float*>(csm + L.sq);
+  float* sf = reinterpret_cast<float*>(csm + L.sf);
+  T* qh = reinterpret_cast<T*>(csm + L.qh);
+  T* ql = reinterpret_cast<T*>(csm + L.ql);
+  T* kh = reinterpret_cast<T*>(csm + L.kh);
+  T* kl = reinterpret_cast<T*>(csm + L.kl);
+  float* gt = reinterpret_cast<float*>(csm + L.gt);
+  T* ph = reinterpret_cast<T*>(csm + L.ph);
+  T* pl = reinterpret_cast<T*>(csm + L.pl);
+  float* so = reinterpret_cast<float*>(csm + L.so);
+  float* csum = reinterpret_cast<float*>(csm + L.csum);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
+  const int vg = warp % VG, dg = warp / VG, head = blockIdx.y, seq = blockIdx.x, v0 = blockIdx.z * VT;
+  const int q0 = p.rows.q_start[seq], n = p.rows.q_len[seq], slot = p.rows.slot ? p.rows.slot[seq] : seq;
+  const bool fresh = p.rows.pos[q0] == 0;
+  float* S = p.state + ((size_t)slot * p.heads + head) * p.dim * p.vdim;
+  const T* x = reinterpret_cast<const T*>(p.x);
+  T* out = reinterpret_cast<T*>(p.out);
+
+  // transposed state: tile j covers key channels (j * DG + dg) * 16 .. + 15 as two accumulator tiles of eight
+  float st[DT][8];
+#pragma unroll
+  for (int j = 0; j < DT; ++j)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const int d = (j * DG + dg) * 16 + (e >> 2) * 8 + q4 * 2 + (e & 1), v = v0 + vg * 16 + g + ((e >> 1) & 1) * 8;
+      st[j][e] = (!fresh && d < p.dim && v < p.vdim) ? S[(size_t)d * p.vdim + v] : 0.f;
+    }
+
+  const int raw_chunks = (2 * DP + VT) / 8;
+  auto prefetch = [&](int b) {
+    for (int i = tid; i < kHcTok * raw_chunks; i += kHcThreads) {
+      const int t = i / raw_chunks, c = (i % raw_chunks) * 8, tok = b * kHcTok + t;
+      int src;
+      bool ok = tok < n;
+      if (c < DP) { src = head * p.dim + c; ok = ok && c < p.dim; }
+      else if (c < 2 * DP) { src = p.f_off + head * p.dim + c - DP; ok = ok && c - DP < p.dim; }
+      else { src = p.v_off + head * p.vdim + v0 + c - 2 * DP; ok = ok && v0 + c - 2 * DP < p.vdim; }
+      hc_cp16(smem_u32(raw + ((b & 1) * kHcTok + t) * L.raw_ld + c), ok ? x + (size_t)(q0 + tok) * p.ldx + src : x, ok);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  const int steps = (n + kHcTok - 1) / kHcTok;
+  // output of the step before, still to be normalised: token row `orow`, values ov of channels ocol ..
+  float ov[NV];
+  int orow = -1;
+  const int otok = tid >> 4, ocol = (tid & 15) * NV;
+  auto finish = [&](int buf, float own) {
+    float tot = own;
+    if (col_tiles > 1) {
+      tot = 0.f;
+      for (int c = 0; c < col_tiles; ++c) tot += ld_dsmem_f32(dsmem_addr(smem_u32(csum + buf * kHcTok + otok), (uint32_t)c));
+    }
+    const int v = v0 + ocol;
+    if (orow < 0 || v >= p.vdim) return;
+    const float r = p.norm_w ? rsqrtf(tot / (float)p.vdim_true + p.eps) : 1.f;
+    T* dst = out + (size_t)orow * p.ldo + head * p.vdim + v;
+#pragma unroll
+    for (int i = 0; i < NV; i += 2) {
+      const float w0 = p.norm_w ? p.norm_w[v + i] : 1.f, w1 = p.norm_w ? p.norm_w[v + i + 1] : 1.f;
+      *reinterpret_cast<uint32_t*>(dst + i) = MmaOp<T>::pack(ov[i] * r * w0, ov[i + 1] * r * w1);
+    }
+  };
+  prefetch(0);
+
+  for (int b = 0; b < steps; ++b) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    if (b + 1 < steps) prefetch(b + 1);
+    const T* rw = raw + (b & 1) * kHcTok * L.raw_ld;
+    const int valid = n - b * kHcTok;
+    // ---- gates
+    for (int i = tid; i < kHcTok * DP; i += kHcThreads) {
+      const int t = i / DP, c = i % DP, ch = head * p.dim + c;
+      float qv = 0.f, f = 1.f;
+      if (t < valid && c < p.dim) {
+        const float z = __bfloat162float(rw[t * L.raw_ld + c]), lo = __ldg(p.lower + ch);
+        qv = z * sigmoid_f32(z);
+        f = lo + (1.f - lo) * sigmoid_f32(__bfloat162float(rw[t * L.raw_ld + DP + c]) + __ldg(p.f_bias + ch));
+      }
+      sq[t * L.q_ld + c] = qv;
+      sf[t * L.q_ld + c] = f;
+    }
+    __syncthreads();
+    // ---- P: two source tokens per warp, sixteen lanes over the key channels
+    {
+      const int s = warp * 2 + (lane >> 4), cg = lane & 15;
+      float acc[kHcTok];
+#pragma unroll
+      for (int t = 0; t < kHcTok; ++t) acc[t] = 0.f;
+      for (int c = cg * 4; c < DP; c += 64) {
+        const float4 f0 = *reinterpret_cast<const float4*>(sf + s * L.q_ld + c);
+        float4 w = make_float4(1.f - f0.x, 1.f - f0.y, 1.f - f0.z, 1.f - f0.w);
+#pragma unroll
+        for (int t = 0; t < kHcTok; ++t) {
+          if (t >= warp * 2) {                   // the warp's first source token
+            if (t > s) {
+              const float4 f = *reinterpret_cast<const float4*>(sf + t * L.q_ld + c);
+              w.x *= f.x; w.y *= f.y; w.z *= f.z; w.w *= f.w;
+            }
+            const float4 q = *reinterpret_cast<const float4*>(sq + t * L.q_ld + c);
+            const float d = fmaf(q.x, w.x, fmaf(q.y, w.y, fmaf(q.z, w.z, q.w * w.w)));
+            acc[t] += t >= s ? d : 0.f;
+          }
+        }
+      }
+      // sum over the sixteen lanes; lane cg keeps t = cg
+#pragma unroll
+      for (int o = 8; o > 0; o >>= 1) {
+        const bool up = (cg & o) != 0;
+#pragma unroll
+        for (int i = 0; i < kHcTok / 2; ++i) {
+          if (i < o) {
+            const float send = up ? acc[i] : acc[i + o], keep = up ? acc[i + o] : acc[i];
+            acc[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+          }
+        }
+      }
+      hc_split(acc[0], ph[cg * 24 + s], pl[cg * 24 + s]);
+    }
+    // ---- running products per key channel (the last warps have the least to do above)
+    for (int i = kHcThreads - 1 - tid; i < 2 * DP; i += kHcThreads) {
+      if (i < DP) {
+        float G = 1.f;
+#pragma unroll
+        for (int t = 0; t < kHcTok; ++t) {
+          G *= sf[t * L.q_ld + i];
+          hc_split(sq[t * L.q_ld + i] * G, qh[t * L.b_ld + i], ql[t * L.b_ld + i]);
+        }
+        gt[i] = G;
+      } else {
+        const int c = i - DP;
+        float E = 1.f;
+#pragma unroll
+        for (int t = kHcTok - 1; t >= 0; --t) {
+          const float f = sf[t * L.q_ld + c];
+          hc_split((1.f - f) * E, kh[t * L.b_ld + c], kl[t * L.b_ld + c]);
+          E *= f;
+        }
+      }
+    }
+    if (b > 0 && col_tiles > 1) {
+      __syncwarp();
+      asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+      finish((b - 1) & 1, 0.f);
+    }
+    __syncthreads();
+    // ---- tensor cores
+    {
+      uint32_t va[4];                            // V^T of this warp's value channels (rows) over the sixteen tokens
+      ldsm_x4_t(smem_u32(rw + ((lane >> 4) * 8 + (lane & 7)) * L.raw_ld + 2 * DP + vg * 16 + ((lane >> 3) & 1) * 8), va[0], va[1], va[2], va[3]);
+      float o[2][4] = {};
+      if (dg == 0) {
+        uint32_t bh[4], bl[4];
+        const int off = ((lane >> 4) * 8 + (lane & 7)) * 24 + ((lane >> 3) & 1) * 8;
+        ldsm_x4(smem_u32(ph + off), bh[0], bh[1], bh[2], bh[3]);
+        ldsm_x4(smem_u32(pl + off), bl[0], bl[1], bl[2], bl[3]);
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          MmaOp<T>::mma(o[nt], va, bh[nt * 2], bh[nt * 2 + 1]);
+          MmaOp<T>::mma(o[nt], va, bl[nt * 2], bl[nt * 2 + 1]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < DT; ++j) {
+        const int d = (j * DG + dg) * 16;
+        if (d < DP) {
+          uint32_t ah[4], al[4], bh[4], bl[4];
+          hc_split2(st[j][0], st[j][1], ah[0], al[0]);
+          hc_split2(st[j][2], st[j][3], ah[1], al[1]);
+          hc_split2(st[j][4], st[j][5], ah[2], al[2]);
+          hc_split2(st[j][6], st[j][7], ah[3], al[3]);
+          const int qoff = ((lane >> 4) * 8 + (lane & 7)) * L.b_ld + d + ((lane >> 3) & 1) * 8;      // [token][channel], no transpose
+          ldsm_x4(smem_u32(qh + qoff), bh[0], bh[1], bh[2], bh[3]);
+          ldsm_x4(smem_u32(ql + qoff), bl[0], bl[1], bl[2], bl[3]);
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt) {
+            MmaOp<T>::mma(o[nt], ah, bh[nt * 2], bh[nt * 2 + 1]);
+            MmaOp<T>::mma(o[nt], al, bh[nt * 2], bh[nt * 2 + 1]);
+            MmaOp<T>::mma(o[nt], ah, bl[nt * 2], bl[nt * 2 + 1]);
+          }
+          const int koff = (lane & 15) * L.b_ld + d + (lane >> 4) * 8;                              // transposed: tokens are the k axis
+          ldsm_x4_t(smem_u32(kh + koff), bh[0], bh[1], bh[2], bh[3]);
+          ldsm_x4_t(smem_u32(kl + koff), bl[0], bl[1], bl[2], bl[3]);
+#pragma unroll
+          for (int h8 = 0; h8 < 2; ++h8) {
+            const float2 G = *reinterpret_cast<const float2*>(gt + d + h8 * 8 + q4 * 2);
+            float (&c)[4] = *reinterpret_cast<float (*)[4]>(&st[j][h8 * 4]);
+            c[0] *= G.x; c[1] *= G.y; c[2] *= G.x; c[3] *= G.y;
+            MmaOp<T>::mma(c, va, bh[h8 * 2], bh[h8 * 2 + 1]);
+            MmaOp<T>::mma(c, va, bl[h8 * 2], bl[h8 * 2 + 1]);
+          }
+        }
+      }
+      float* dst = so + dg * kHcTok * L.o_ld + vg * 16 + g;
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) dst[(nt * 8 + q4 * 2 + (e & 1)) * L.o_ld + (e >> 1) * 8] = o[nt][e];
+    }
+    __syncthreads();
+    // ---- this step's outputs: sixteen threads per token
+    {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        float v = 0.f;
+#pragma unroll
+        for (int k = 0; k < DG; ++k) v += so[(k * kHcTok + otok) * L.o_ld + ocol + i];
+        ov[i] = v;
+        ss += v * v;
+      }
+#pragma unroll
+      for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      orow = otok < valid ? q0 + b * kHcTok + otok : -1;
+      if (col_tiles > 1) {
+        if ((tid & 15) == 0) csum[(b & 1) * kHcTok + otok] = ss;
+        __syncwarp();
+        asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+      } else {
+        finish(0, ss);
+      }
+    }
+  }
+  if (col_tiles > 1) {
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+    finish((steps - 1) & 1, 0.f);
+    cluster_sync_all();                          // no CTA leaves while its sums may still be read
+  }
+#pragma unroll
+  for (int j = 0; j < DT; ++j)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const int d = (j * DG + dg) * 16 + (e >> 2) * 8 + q4 * 2 + (e & 1), v = v0 + vg * 16 + g + ((e >> 1) & 1) * 8;
+      if (d < p.dim && v < p.vdim) S[(size_t)d * p.vdim + v] = st[j][e];
+    }
+}
+
+template <int VG, int DT>
+static int launch_chunked_t(const RfHgrn2* a, int tiles, cudaStream_t s) {
+  const size_t smem = hgrn2_smem(a->dim, VG * 16, kHcWarps / VG).total;
+  RF_ALLOW_SMEM_PER_DEVICE((hgrn2_chunked_kernel<VG, DT>), 200 * 1024);
+  RF_CUDA_CHECK(::rf::launch_k(hgrn2_chunked_kernel<VG, DT>, dim3(a->rows.num_seqs, a->heads, tiles), dim3(kHcThreads), smem, s, tiles, *a, tiles));
+  ::rf::count_launch();
+  return RF_OK;
+}
+
+template <int VG>
+static int launch_chunked(const RfHgrn2* a, int tiles, cudaStream_t s) {
+  const int per = ceil_div(ceil_div(a->dim, 16), kHcWarps / VG);      // 16-channel tiles per warp
+  if (per <= 2) return launch_chunked_t<VG, 2>(a, tiles, s);
+  if (per <= 4) return launch_chunked_t<VG, 4>(a, tiles, s);
+  if (per <= 8) return launch_chunked_t<VG, 8>(a, tiles, s);
+  return launch_chunked_t<VG, 16>(a, tiles, s);
+}
+
 }  // namespace rf
 
 using namespace rf;
@@ -162,8 +486,25 @@ extern "C" int rf_hgrn2_recurrent(const RfHgrn2* a, rf_stream_t stream) {
 }
 
 extern "C" int rf_hgrn2_chunked_supported(int dim, int vdim, int dtype) {
-  (void)dim; (void)vdim; (void)dtype;
-  return 0;
+  return dtype == kBF16 && dim > 0 && dim <= 256 && vdim > 0 && vdim <= 1024;
 }
 
-extern "C" int rf_hgrn2_chunked(const RfHgrn2* a, rf_stream_t stream) { return rf_hgrn2_recurrent(a, stream); }
+extern "C" int rf_hgrn2_chunked(const RfHgrn2* a, rf_stream_t stream) {
+  RF_SKIP_IF_REPLAYING();
+  int rc = check_hgrn2(a);
+  if (rc) return rc;
+  if (!rf_hgrn2_chunked_supported(a->dim, a->vdim, a->dtype)) return rf_hgrn2_recurrent(a, stream);
+  RF_REQUIRE(a->rows.q_start && a->rows.q_len, "hgrn2: the block form works on portions");
+  if (a->rows.num_seqs == 0) return RF_OK;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  // value channels per CTA: as few as still share a head between at most eight CTAs, more once the GPU is full
+  int vt = a->vdim <= 32 ? 32 : a->vdim <= 64 ? 64 : 128;
+  for (int t : {32, 64}) {
+    const int tiles = ceil_div(a->vdim, t);
+    if (tiles <= 8 && (long)a->rows.num_seqs * a->heads * tiles <= 2 * sm_count()) { vt = t; break; }
+  }
+  const int tiles = ceil_div(a->vdim, vt);
+  if (vt == 32) return launch_chunked<2>(a, tiles, s);
+  if (vt == 64) return launch_chunked<4>(a, tiles, s);
+  return launch_chunked<8>(a, tiles, s);
+}
