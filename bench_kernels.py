@@ -5,6 +5,7 @@
     python bench_kernels.py attn_prefill --seqs 4 --len 2048 --heads 32 --kv-heads 8 --hd 128
     python bench_kernels.py attn_decode --seqs 64 --len 1024 --heads 32 --kv-heads 8 --hd 128
     python bench_kernels.py gdn --seqs 1 --len 1024 --hk 16 --hv 32
+    python bench_kernels.py mixed            # latent attention / HGRN2 / fp32 stream beside the like kernels at equal size
     python bench_kernels.py suite            # the shapes of one Qwen3-8B decode step and prefill chunk
 
 Every line is JSON: the achieved throughput and its fraction of the measured peaks in
@@ -85,6 +86,28 @@ def time_us(fn, iters: int = 20, warmup: int = 3) -> float:
     return statistics.median(ts)
 
 
+def time_cold_us(fn, iters: int = 15) -> float:
+    """One launch from a cold L2, replayed from a CUDA graph so that the host's launch path is not part of the time."""
+    fn()
+    torch.cuda.synchronize()
+    s = torch.cuda.Stream()
+    s.wait_stream(torch.cuda.current_stream())
+    g = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(g, stream=s):
+        fn()
+    ts = []
+    for _ in range(iters):
+        flush_l2()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        g.replay()
+        e1.record()
+        torch.cuda.synchronize()
+        ts.append(e0.elapsed_time(e1) * 1e3)
+    return statistics.median(ts)
+
+
 def report(name: str, us: float, *, flops: float = 0.0, bytes_: float = 0.0, **extra) -> dict:
     pk = peaks()
     out = {"kernel": name, "us": round(us, 2), **extra}
@@ -140,7 +163,7 @@ def _plan(m, n, k, dual, packed, int8, dtype, splits):
         return None
 
 
-def bench_attn_prefill(seqs, length, heads, kv_heads, hd, *, causal=True, dtype=torch.float16, profile=False):
+def bench_attn_prefill(seqs, length, heads, kv_heads, hd, *, causal=True, dtype=torch.float16, profile=False, timer=None):
     from rhinoforge_b200.ops import kernels as K
     T = seqs * length
     qkv = (torch.randn(T, (heads + 2 * kv_heads) * hd, device="cuda") * 0.5).to(dtype)
@@ -154,12 +177,12 @@ def bench_attn_prefill(seqs, length, heads, kv_heads, hd, *, causal=True, dtype=
         fn(); torch.cuda.synchronize()
         torch.cuda.profiler.start(); fn(); torch.cuda.synchronize(); torch.cuda.profiler.stop()
         return None
-    us = time_us(fn)
+    us = (timer or time_us)(fn)
     flops = 4.0 * seqs * heads * length * length * hd * (0.5 if causal else 1.0)
     return report("attn_prefill", us, flops=flops, seqs=seqs, len=length, heads=heads, kv_heads=kv_heads, hd=hd, causal=causal)
 
 
-def bench_attn_decode(seqs, length, heads, kv_heads, hd, *, dtype=torch.float16):
+def bench_attn_decode(seqs, length, heads, kv_heads, hd, *, dtype=torch.float16, timer=None):
     from rhinoforge_b200.ops import kernels as K
     from rhinoforge_b200.runtime.kv_cache import PagedKV
     cache = PagedKV(1, seqs, length + 16, kv_heads, hd, dtype=dtype)
@@ -171,14 +194,14 @@ def bench_attn_decode(seqs, length, heads, kv_heads, hd, *, dtype=torch.float16)
     ws = K.attn_decode_scratch(seqs, heads, hd, q.device)
     fn = lambda: K.attention_decode(q, out, Hq=heads, Hkv=kv_heads, hd=hd, kv_len=kl, max_kv_len=length, k_pool=cache.kv[0, 0],
                                     v_pool=cache.kv[0, 1], page_table=cache.page_table, ws=ws)
-    us = time_us(fn)
+    us = (timer or time_us)(fn)
     r = report("attn_decode", us, bytes_=2.0 * seqs * length * kv_heads * hd * 2, seqs=seqs, len=length, heads=heads,
                kv_heads=kv_heads, hd=hd)
     cache.close()
     return r
 
 
-def bench_gdn(seqs, length, hk, hv, *, dk=128, dv=128, dtype=torch.float16):
+def bench_gdn(seqs, length, hk, hv, *, dk=128, dv=128, dtype=torch.float16, timer=None, chunked=False):
     from rhinoforge_b200.ops import kernels as K
     T = seqs * length
     qkv = torch.randn(T, 2 * hk * dk + hv * dv, device="cuda").to(dtype)
@@ -191,9 +214,9 @@ def bench_gdn(seqs, length, hk, hv, *, dk=128, dv=128, dtype=torch.float16):
     if length == 1:
         fn = lambda: K.gdn_recurrent(qkv, ba[:, :half], ba[:, half:], state, A, dtb, Hk=hk, Hv=hv, Dk=dk, Dv=dv)
     else:
-        fn = lambda: K.gdn_recurrent(qkv, ba[:, :half], ba[:, half:], state, A, dtb, Hk=hk, Hv=hv, Dk=dk, Dv=dv, q_start=qs, q_len=ql)
-    us = time_us(fn, iters=10)
-    return report("gdn_recurrent", us, flops=6.0 * T * hv * dk * dv, bytes_=2.0 * seqs * hv * dk * dv * 4, seqs=seqs, len=length,
+        fn = lambda: K.gdn_recurrent(qkv, ba[:, :half], ba[:, half:], state, A, dtb, Hk=hk, Hv=hv, Dk=dk, Dv=dv, q_start=qs, q_len=ql, chunked=chunked)
+    us = timer(fn) if timer else time_us(fn, iters=10)
+    return report("gdn_chunked" if chunked else "gdn_recurrent", us, flops=6.0 * T * hv * dk * dv, bytes_=2.0 * seqs * hv * dk * dv * 4, seqs=seqs, len=length,
                   hk=hk, hv=hv, us_per_token=round(us / length, 3))
 
 
@@ -285,9 +308,87 @@ def suite() -> None:
     bench_gdn(1, 1024, 16, 32)
 
 
+def bench_mixed(hidden, heads, *, dim=128, vdim=128, rank=512, window=1024, batch=64, prefill=(4, 2048), dtype=torch.bfloat16) -> None:
+    """Kernels of a decoder with per-layer mixers (latent attention, HGRN2, fp32 residual stream), each beside the like kernel of
+    the K/V and Gated-DeltaNet decoders at equal size."""
+    from rhinoforge_b200.ops import kernels as K
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
+    tag = dict(hidden=hidden, heads=heads)
+    rnd = lambda *sh: torch.randn(*sh, device="cuda", dtype=dtype)
+    f32 = lambda *sh: torch.randn(*sh, device="cuda")
+    S, Lp = prefill
+    T = S * Lp
+    seq = i32([j for j in range(S) for _ in range(Lp)])
+    pos_p, starts, lens = i32(list(range(Lp)) * S), i32([j * Lp for j in range(S)]), i32([Lp] * S)
+    rows_p = lambda **kw: K.rows(pos_p, seq_of_row=seq, q_start=starts, q_len=lens, slot=i32(list(range(S))), **kw)
+    # ---- residual stream, decode and prefill rows
+    nw, mu, st = f32(hidden), torch.rand(hidden, device="cuda"), f32(max(batch, S), hidden)
+    for n, r in ((batch, K.rows(i32([7] * batch))), (T, rows_p())):
+        x, y, w16 = f32(n, hidden), rnd(n, hidden), rnd(hidden)
+        us = time_cold_us(lambda: K.stream_norm(x, r, dtype=dtype, eps=1e-6, norm_w=nw, y=y, shift=mu, shift_state=st))
+        report("stream_norm (add + norm + token shift)", us, bytes_=n * hidden * 12, rows=n, **tag)
+        xx, out = rnd(n, hidden), rnd(n, hidden)
+        us = time_cold_us(lambda: K.rmsnorm(xx, w16, 1e-6, residual=y, residual_out=xx, out=out))
+        report("like: rmsnorm with residual", us, bytes_=n * hidden * 8, rows=n, **tag)
+    # ---- latent attention, decode
+    wa, wu = rnd(heads, rank, dim) / dim ** 0.5, rnd(heads, vdim, rank) / rank ** 0.5
+    q = rnd(batch, heads, dim)
+    us = time_cold_us(lambda: K.head_linear(q, wa))
+    report("head_linear (query -> latent)", us, bytes_=2 * (wa.numel() + batch * heads * (dim + rank)), flops=2.0 * batch * wa.numel(), rows=batch, **tag)
+    ol = rnd(batch, heads, rank)
+    us = time_cold_us(lambda: K.head_linear(ol, wu))
+    report("head_linear (latent -> value)", us, bytes_=2 * (wu.numel() + batch * heads * (vdim + rank)), flops=2.0 * batch * wu.numel(), rows=batch, **tag)
+    del wa, wu
+    bench_gemm(batch, rank * heads // 4, dim * 4, packed=True, dtype=dtype)
+    for b in (1, batch):
+        pages = (window + 15) // 16 + 1
+        pool, ql = rnd(b * pages, 16, rank), rnd(b, heads, rank)
+        pt = torch.randperm(b * pages, device="cuda").to(torch.int32).view(b, pages)
+        r = K.rows(i32([window] * b), page_table=pt)
+        us = time_cold_us(lambda: K.latent_attention(ql, pool, r, window=window, scale=0.05, max_kv=window))
+        report("latent_attn decode", us, bytes_=2.0 * b * (window * rank + 2 * heads * rank), flops=4.0 * b * heads * window * rank, rows=b, window=window, **tag)
+        bench_attn_decode(b, window, heads, max(1, heads // 4), 128, dtype=dtype, timer=time_cold_us)
+    # ---- latent attention, prefill: gather + expansion + attention
+    pages = (Lp + 15) // 16
+    pool = rnd(S * pages, 16, rank)
+    pt = torch.randperm(S * pages, device="cuda").to(torch.int32).view(S, pages)
+    r = rows_p(page_table=pt)
+    us = time_cold_us(lambda: K.latent_gather(pool, r, starts, lens, T, Lp))
+    report("latent_gather", us, bytes_=4.0 * T * rank, rows=T, **tag)
+    bench_gemm(T, 2 * heads * dim, rank, packed=True, dtype=dtype)
+    qq, kv, oo = rnd(T, heads * dim), rnd(T, 2 * heads * dim), rnd(T, heads * dim)
+    vis = sum(min(i + 1, window) for i in range(Lp)) * S
+    us = time_cold_us(lambda: K.attention_prefill(qq, oo, Hq=heads, Hkv=heads, hd=dim, q_start=starts, q_len=lens, kv_len=lens, max_q_len=Lp,
+                                             k=kv[:, :heads * dim], v=kv[:, heads * dim:], kv_start=starts, causal=True, window=window, scale=0.05))
+    report("attention over expanded keys (windowed)", us, flops=4.0 * vis * heads * dim, rows=T, window=window, **tag)
+    bench_attn_prefill(S, Lp, heads, max(1, heads // 4), 128, dtype=dtype, timer=time_cold_us)
+    del qq, kv, oo, pool
+    # ---- linear attention
+    width = heads * (2 * dim + vdim)
+    fb, lo, hw = f32(heads * dim), torch.rand(heads * dim, device="cuda"), f32(vdim)
+    for b in (1, batch):
+        x, state = rnd(b, width), f32(b, heads, dim, vdim)
+        rr = K.rows(i32([5] * b))
+        us = time_cold_us(lambda: K.hgrn2(x, fb, lo, hw, state, rr, eps=1e-6))
+        report("hgrn2 decode step", us, bytes_=8.0 * state.numel() + 2.0 * b * (width + heads * vdim), rows=b, **tag)
+        bench_gdn(b, 1, heads, heads, dtype=dtype, timer=time_cold_us)
+    for s_, l_ in ((1, 4096), (S, Lp)):
+        x, state = rnd(s_ * l_, width), f32(s_, heads, dim, vdim)
+        rr = K.rows(i32(list(range(l_)) * s_), q_start=i32([j * l_ for j in range(s_)]), q_len=i32([l_] * s_))
+        us = time_cold_us(lambda: K.hgrn2(x, fb, lo, hw, state, rr, eps=1e-6, chunked=True))
+        report("hgrn2 prefill (16-token blocks)", us, flops=s_ * l_ * heads * (4.0 * dim * vdim + 32.0 * dim + 32.0 * vdim),
+               bytes_=2.0 * s_ * l_ * (width + heads * vdim), seqs=s_, length=l_, **tag)
+        bench_gdn(s_, l_, heads, heads, dtype=dtype, timer=time_cold_us, chunked=True)
+
+
+def mixed() -> None:
+    bench_mixed(2048, 16)
+    bench_mixed(4096, 32)
+
+
 def main() -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("what", choices=["gemm", "attn_prefill", "attn_decode", "gdn", "suite", "sweep", "heads"])
+    ap.add_argument("what", choices=["gemm", "attn_prefill", "attn_decode", "gdn", "suite", "sweep", "heads", "mixed"])
     for name, d in (("m", 64), ("n", 4096), ("k", 4096), ("seqs", 4), ("len", 2048), ("heads", 32), ("kv-heads", 8),
                     ("hd", 128), ("hk", 16), ("hv", 32)):
         ap.add_argument(f"--{name}", type=int, default=d)
@@ -313,6 +414,8 @@ def main() -> int:
         sweep()
     elif a.what == "heads":
         heads()
+    elif a.what == "mixed":
+        mixed()
     else:
         suite()
     return 0

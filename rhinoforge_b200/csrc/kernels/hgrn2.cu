@@ -151,35 +151,26 @@ static int launch_recurrent(const RfHgrn2* a, cudaStream_t s) {
 // warps - 16 value channels x a share of the key channels each - where the product with it reads it as an operand.
 // A CTA owns VG * 16 value channels of one head of one sequence; the CTAs of a head form a cluster that exchanges the sums of
 // squares of the head norm one step behind the computation.
-constexpr int kHcTok = 16, kHcThreads = 256, kHcWarps = 8;
+constexpr int kHcTok = 16, kHcThreads = 256, kHcWarps = 8, kHcRing = 4;
 
-struct Hgrn2Smem {
-  int dp, raw_ld, q_ld, b_ld, o_ld;
-  uint32_t raw, sq, sf, qh, ql, kh, kl, gt, ph, pl, so, csum, total;
+// Shared memory of a CTA with DP (padded) key channels and VT value channels, in bytes from the base.
+template <int DP, int VT> struct Hgrn2Geom {
+  static constexpr int kRawLd = 2 * DP + VT + 8, kQLd = DP + 4, kBLd = DP + 8, kPLd = 24, kOLd = VT + 4;
+  static constexpr int kDG = kHcWarps / (VT / 16);
+  static constexpr int raw = 0;                                   // [ring][16] rows q | f | v as they come
+  static constexpr int sq = raw + kHcRing * kHcTok * kRawLd * 2;  // [16][DP] silu(q), gates
+  static constexpr int sf = sq + kHcTok * kQLd * 4;
+  static constexpr int qh = sf + kHcTok * kQLd * 4;               // bf16 pairs of q * G and (1 - f) * E
+  static constexpr int ql = qh + kHcTok * kBLd * 2;
+  static constexpr int kh = ql + kHcTok * kBLd * 2;
+  static constexpr int kl = kh + kHcTok * kBLd * 2;
+  static constexpr int gt = kl + kHcTok * kBLd * 2;               // gate product of the whole block
+  static constexpr int ph = gt + DP * 4;
+  static constexpr int pl = ph + kHcTok * kPLd * 2;
+  static constexpr int so = pl + kHcTok * kPLd * 2;               // [warps of a value group][16][VT] partial outputs
+  static constexpr int csum = so + kDG * kHcTok * kOLd * 4;
+  static constexpr int total = csum + 2 * kHcTok * 4;
 };
-__host__ __device__ inline Hgrn2Smem hgrn2_smem(int dim, int vt, int dg) {
-  Hgrn2Smem m;
-  m.dp = (dim + 15) / 16 * 16;
-  m.raw_ld = 2 * m.dp + vt + 8;
-  m.q_ld = m.dp + 4;
-  m.b_ld = m.dp + 8;
-  m.o_ld = vt + 4;
-  uint32_t o = 0;
-  m.raw = o; o += 2 * kHcTok * m.raw_ld * 2;
-  m.sq = o; o += kHcTok * m.q_ld * 4;
-  m.sf = o; o += kHcTok * m.q_ld * 4;
-  m.qh = o; o += kHcTok * m.b_ld * 2;
-  m.ql = o; o += kHcTok * m.b_ld * 2;
-  m.kh = o; o += kHcTok * m.b_ld * 2;
-  m.kl = o; o += kHcTok * m.b_ld * 2;
-  m.gt = o; o += m.dp * 4;
-  m.ph = o; o += kHcTok * 24 * 2;
-  m.pl = o; o += kHcTok * 24 * 2;
-  m.so = o; o += dg * kHcTok * m.o_ld * 4;
-  m.csum = o; o += 2 * kHcTok * 4;
-  m.total = o;
-  return m;
-}
 
 __device__ __forceinline__ void hc_cp16(uint32_t dst, const void* src, bool valid) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
@@ -198,26 +189,25 @@ __device__ __forceinline__ void hc_split2(float a, float b, uint32_t& hi, uint32
 }
 
 // VG: groups of 16 value channels per CTA; the 8 / VG warps of a group share its key channels, DT 16-channel tiles each.
-template <int VG, int DT>
-__global__ void __launch_bounds__(kHcThreads, 1) hgrn2_chunked_kernel(const RfHgrn2 p, int col_tiles) {
+template <int VG, int DP>
+__global__ void __launch_bounds__(kHcThreads, DP == 256 ? 1 : 2) hgrn2_chunked_kernel(const RfHgrn2 p, int col_tiles) {
   pdl_prologue();
   using T = __nv_bfloat16;
-  constexpr int VT = VG * 16, DG = kHcWarps / VG, NV = VT / 16;
+  constexpr int VT = VG * 16, DG = kHcWarps / VG, NV = VT / 16, DT = DP / 16 / DG;
+  using L = Hgrn2Geom<DP, VT>;
   extern __shared__ __align__(16) uint8_t csm[];
-  const Hgrn2Smem L = hgrn2_smem(p.dim, VT, DG);
-  const int DP = L.dp;
-  T* raw = reinterpret_cast<T*>(csm + L.raw);
-  float* sq = reinterpret_cast<float*>(csm + L.sq);
-  float* sf = reinterpret_cast<float*>(csm + L.sf);
-  T* qh = reinterpret_cast<T*>(csm + L.qh);
-  T* ql = reinterpret_cast<T*>(csm + L.ql);
-  T* kh = reinterpret_cast<T*>(csm + L.kh);
-  T* kl = reinterpret_cast<T*>(csm + L.kl);
-  float* gt = reinterpret_cast<float*>(csm + L.gt);
-  T* ph = reinterpret_cast<T*>(csm + L.ph);
-  T* pl = reinterpret_cast<T*>(csm + L.pl);
-  float* so = reinterpret_cast<float*>(csm + L.so);
-  float* csum = reinterpret_cast<float*>(csm + L.csum);
+  T* raw = reinterpret_cast<T*>(csm + L::raw);
+  float* sq = reinterpret_cast<float*>(csm + L::sq);
+  float* sf = reinterpret_cast<float*>(csm + L::sf);
+  T* qh = reinterpret_cast<T*>(csm + L::qh);
+  T* ql = reinterpret_cast<T*>(csm + L::ql);
+  T* kh = reinterpret_cast<T*>(csm + L::kh);
+  T* kl = reinterpret_cast<T*>(csm + L::kl);
+  float* gt = reinterpret_cast<float*>(csm + L::gt);
+  T* ph = reinterpret_cast<T*>(csm + L::ph);
+  T* pl = reinterpret_cast<T*>(csm + L::pl);
+  float* so = reinterpret_cast<float*>(csm + L::so);
+  float* csum = reinterpret_cast<float*>(csm + L::csum);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
   const int vg = warp % VG, dg = warp / VG, head = blockIdx.y, seq = blockIdx.x, v0 = blockIdx.z * VT;
   const int q0 = p.rows.q_start[seq], n = p.rows.q_len[seq], slot = p.rows.slot ? p.rows.slot[seq] : seq;
@@ -236,24 +226,40 @@ __global__ void __launch_bounds__(kHcThreads, 1) hgrn2_chunked_kernel(const RfHg
       st[j][e] = (!fresh && d < p.dim && v < p.vdim) ? S[(size_t)d * p.vdim + v] : 0.f;
     }
 
-  const int raw_chunks = (2 * DP + VT) / 8;
   auto prefetch = [&](int b) {
-    for (int i = tid; i < kHcTok * raw_chunks; i += kHcThreads) {
-      const int t = i / raw_chunks, c = (i % raw_chunks) * 8, tok = b * kHcTok + t;
-      int src;
-      bool ok = tok < n;
-      if (c < DP) { src = head * p.dim + c; ok = ok && c < p.dim; }
-      else if (c < 2 * DP) { src = p.f_off + head * p.dim + c - DP; ok = ok && c - DP < p.dim; }
-      else { src = p.v_off + head * p.vdim + v0 + c - 2 * DP; ok = ok && v0 + c - 2 * DP < p.vdim; }
-      hc_cp16(smem_u32(raw + ((b & 1) * kHcTok + t) * L.raw_ld + c), ok ? x + (size_t)(q0 + tok) * p.ldx + src : x, ok);
+    constexpr int kChunks = (2 * DP + VT) / 8, kAll = kHcTok * kChunks;
+    if (b * kHcTok < n) {
+#pragma unroll
+      for (int k = 0; k < (kAll + kHcThreads - 1) / kHcThreads; ++k) {
+        const int i = tid + k * kHcThreads, t = i / kChunks, c = (i % kChunks) * 8, tok = b * kHcTok + t;
+        if (i < kAll) {
+          int src;
+          bool ok = tok < n;
+          if (c < DP) { src = head * p.dim + c; ok = ok && c < p.dim; }
+          else if (c < 2 * DP) { src = p.f_off + head * p.dim + c - DP; ok = ok && c - DP < p.dim; }
+          else { src = p.v_off + head * p.vdim + v0 + c - 2 * DP; ok = ok && v0 + c - 2 * DP < p.vdim; }
+          hc_cp16(smem_u32(raw + ((b % kHcRing) * kHcTok + t) * L::kRawLd + c), ok ? x + (size_t)(q0 + tok) * p.ldx + src : x, ok);
+        }
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
+  // this thread's share of the gates: two neighbouring key channels of every (512 / DP)-th token
+  constexpr int kGateStep = 2 * kHcThreads / DP;
+  const int gc = (tid % (DP / 2)) * 2, gtok = tid / (DP / 2);
+  float g_lo[2] = {1.f, 1.f}, g_b[2] = {0.f, 0.f};
+  if (gc < p.dim) {
+    g_lo[0] = p.lower[head * p.dim + gc]; g_lo[1] = p.lower[head * p.dim + gc + 1];
+    g_b[0] = p.f_bias[head * p.dim + gc]; g_b[1] = p.f_bias[head * p.dim + gc + 1];
+  }
   const int steps = (n + kHcTok - 1) / kHcTok;
   // output of the step before, still to be normalised: token row `orow`, values ov of channels ocol ..
   float ov[NV];
   int orow = -1;
   const int otok = tid >> 4, ocol = (tid & 15) * NV;
+  float nw[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) nw[i] = (p.norm_w && v0 + ocol + i < p.vdim) ? p.norm_w[v0 + ocol + i] : 1.f;
   auto finish = [&](int buf, float own) {
     float tot = own;
     if (col_tiles > 1) {
@@ -265,87 +271,88 @@ __global__ void __launch_bounds__(kHcThreads, 1) hgrn2_chunked_kernel(const RfHg
     const float r = p.norm_w ? rsqrtf(tot / (float)p.vdim_true + p.eps) : 1.f;
     T* dst = out + (size_t)orow * p.ldo + head * p.vdim + v;
 #pragma unroll
-    for (int i = 0; i < NV; i += 2) {
-      const float w0 = p.norm_w ? p.norm_w[v + i] : 1.f, w1 = p.norm_w ? p.norm_w[v + i + 1] : 1.f;
-      *reinterpret_cast<uint32_t*>(dst + i) = MmaOp<T>::pack(ov[i] * r * w0, ov[i + 1] * r * w1);
-    }
+    for (int i = 0; i < NV; i += 2) *reinterpret_cast<uint32_t*>(dst + i) = MmaOp<T>::pack(ov[i] * r * nw[i], ov[i + 1] * r * nw[i + 1]);
   };
-  prefetch(0);
+  for (int b = 0; b < kHcRing - 1; ++b) prefetch(b);
 
   for (int b = 0; b < steps; ++b) {
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    asm volatile("cp.async.wait_group %0;" ::"n"(kHcRing - 2) : "memory");
     __syncthreads();
-    if (b + 1 < steps) prefetch(b + 1);
-    const T* rw = raw + (b & 1) * kHcTok * L.raw_ld;
+    prefetch(b + kHcRing - 1);
+    const T* rw = raw + (b % kHcRing) * kHcTok * L::kRawLd;
     const int valid = n - b * kHcTok;
     // ---- gates
-    for (int i = tid; i < kHcTok * DP; i += kHcThreads) {
-      const int t = i / DP, c = i % DP, ch = head * p.dim + c;
-      float qv = 0.f, f = 1.f;
-      if (t < valid && c < p.dim) {
-        const float z = __bfloat162float(rw[t * L.raw_ld + c]), lo = __ldg(p.lower + ch);
-        qv = z * sigmoid_f32(z);
-        f = lo + (1.f - lo) * sigmoid_f32(__bfloat162float(rw[t * L.raw_ld + DP + c]) + __ldg(p.f_bias + ch));
-      }
-      sq[t * L.q_ld + c] = qv;
-      sf[t * L.q_ld + c] = f;
+#pragma unroll
+    for (int k = 0; k < kHcTok / kGateStep; ++k) {
+      const int t = gtok + k * kGateStep;
+      const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(rw + t * L::kRawLd + gc));
+      const float2 y = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(rw + t * L::kRawLd + DP + gc));
+      const bool in = t < valid && gc < p.dim;
+      float2 q, f;
+      q.x = in ? z.x * sigmoid_f32(z.x) : 0.f;
+      q.y = in ? z.y * sigmoid_f32(z.y) : 0.f;
+      f.x = in ? g_lo[0] + (1.f - g_lo[0]) * sigmoid_f32(y.x + g_b[0]) : 1.f;
+      f.y = in ? g_lo[1] + (1.f - g_lo[1]) * sigmoid_f32(y.y + g_b[1]) : 1.f;
+      *reinterpret_cast<float2*>(sq + t * L::kQLd + gc) = q;
+      *reinterpret_cast<float2*>(sf + t * L::kQLd + gc) = f;
     }
     __syncthreads();
-    // ---- P: two source tokens per warp, sixteen lanes over the key channels
-    {
-      const int s = warp * 2 + (lane >> 4), cg = lane & 15;
-      float acc[kHcTok];
+    if (warp < 4) {
+      // ---- P: source tokens warp, warp + 4, .. of this warp, the lanes over the key channels
+      float acc[4 * kHcTok];
 #pragma unroll
-      for (int t = 0; t < kHcTok; ++t) acc[t] = 0.f;
-      for (int c = cg * 4; c < DP; c += 64) {
-        const float4 f0 = *reinterpret_cast<const float4*>(sf + s * L.q_ld + c);
-        float4 w = make_float4(1.f - f0.x, 1.f - f0.y, 1.f - f0.z, 1.f - f0.w);
+      for (int i = 0; i < 4 * kHcTok; ++i) acc[i] = 0.f;
+      for (int c = lane * 4; c < DP; c += 128) {
+        float4 w[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float4 f0 = *reinterpret_cast<const float4*>(sf + (warp + 4 * i) * L::kQLd + c);
+          w[i] = make_float4(1.f - f0.x, 1.f - f0.y, 1.f - f0.z, 1.f - f0.w);
+        }
 #pragma unroll
         for (int t = 0; t < kHcTok; ++t) {
-          if (t >= warp * 2) {                   // the warp's first source token
-            if (t > s) {
-              const float4 f = *reinterpret_cast<const float4*>(sf + t * L.q_ld + c);
-              w.x *= f.x; w.y *= f.y; w.z *= f.z; w.w *= f.w;
+          const float4 f = *reinterpret_cast<const float4*>(sf + t * L::kQLd + c), q = *reinterpret_cast<const float4*>(sq + t * L::kQLd + c);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            if (t >= 4 * i) {                    // source token s = warp + 4 i cannot be later than t otherwise
+              const int s = warp + 4 * i;
+              if (t > s) { w[i].x *= f.x; w[i].y *= f.y; w[i].z *= f.z; w[i].w *= f.w; }
+              if (t >= s) acc[i * kHcTok + t] += fmaf(q.x, w[i].x, fmaf(q.y, w[i].y, fmaf(q.z, w[i].z, q.w * w[i].w)));
             }
-            const float4 q = *reinterpret_cast<const float4*>(sq + t * L.q_ld + c);
-            const float d = fmaf(q.x, w.x, fmaf(q.y, w.y, fmaf(q.z, w.z, q.w * w.w)));
-            acc[t] += t >= s ? d : 0.f;
           }
         }
       }
-      // sum over the sixteen lanes; lane cg keeps t = cg
+      // sum over the lanes: halves of the 64 sums change sides until a lane holds two of them, index lane * 2 (+ 1)
 #pragma unroll
-      for (int o = 8; o > 0; o >>= 1) {
-        const bool up = (cg & o) != 0;
+      for (int o = 16; o > 0; o >>= 1) {
+        const bool up = (lane & o) != 0;
 #pragma unroll
-        for (int i = 0; i < kHcTok / 2; ++i) {
-          if (i < o) {
-            const float send = up ? acc[i] : acc[i + o], keep = up ? acc[i + o] : acc[i];
+        for (int i = 0; i < 2 * kHcTok; ++i) {
+          if (i < 2 * o) {
+            const float send = up ? acc[i] : acc[i + 2 * o], keep = up ? acc[i + 2 * o] : acc[i];
             acc[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
           }
         }
       }
-      hc_split(acc[0], ph[cg * 24 + s], pl[cg * 24 + s]);
-    }
-    // ---- running products per key channel (the last warps have the least to do above)
-    for (int i = kHcThreads - 1 - tid; i < 2 * DP; i += kHcThreads) {
-      if (i < DP) {
-        float G = 1.f;
+      const int s = warp + 4 * (lane >> 3), t = (lane & 7) * 2;
+      hc_split(acc[0], ph[t * L::kPLd + s], pl[t * L::kPLd + s]);
+      hc_split(acc[1], ph[(t + 1) * L::kPLd + s], pl[(t + 1) * L::kPLd + s]);
+    } else {
+      // ---- running products per key channel
+      for (int c = tid - 128; c < DP; c += 128) {
+        float f[kHcTok], q[kHcTok];
+#pragma unroll
+        for (int t = 0; t < kHcTok; ++t) { f[t] = sf[t * L::kQLd + c]; q[t] = sq[t * L::kQLd + c]; }
+        float G = 1.f, E = 1.f;
 #pragma unroll
         for (int t = 0; t < kHcTok; ++t) {
-          G *= sf[t * L.q_ld + i];
-          hc_split(sq[t * L.q_ld + i] * G, qh[t * L.b_ld + i], ql[t * L.b_ld + i]);
+          G *= f[t];
+          hc_split(q[t] * G, qh[t * L::kBLd + c], ql[t * L::kBLd + c]);
+          const int r = kHcTok - 1 - t;
+          hc_split((1.f - f[r]) * E, kh[r * L::kBLd + c], kl[r * L::kBLd + c]);
+          E *= f[r];
         }
-        gt[i] = G;
-      } else {
-        const int c = i - DP;
-        float E = 1.f;
-#pragma unroll
-        for (int t = kHcTok - 1; t >= 0; --t) {
-          const float f = sf[t * L.q_ld + c];
-          hc_split((1.f - f) * E, kh[t * L.b_ld + c], kl[t * L.b_ld + c]);
-          E *= f;
-        }
+        gt[c] = G;
       }
     }
     if (b > 0 && col_tiles > 1) {
@@ -357,11 +364,11 @@ __global__ void __launch_bounds__(kHcThreads, 1) hgrn2_chunked_kernel(const RfHg
     // ---- tensor cores
     {
       uint32_t va[4];                            // V^T of this warp's value channels (rows) over the sixteen tokens
-      ldsm_x4_t(smem_u32(rw + ((lane >> 4) * 8 + (lane & 7)) * L.raw_ld + 2 * DP + vg * 16 + ((lane >> 3) & 1) * 8), va[0], va[1], va[2], va[3]);
+      ldsm_x4_t(smem_u32(rw + ((lane >> 4) * 8 + (lane & 7)) * L::kRawLd + 2 * DP + vg * 16 + ((lane >> 3) & 1) * 8), va[0], va[1], va[2], va[3]);
       float o[2][4] = {};
       if (dg == 0) {
         uint32_t bh[4], bl[4];
-        const int off = ((lane >> 4) * 8 + (lane & 7)) * 24 + ((lane >> 3) & 1) * 8;
+        const int off = ((lane >> 4) * 8 + (lane & 7)) * L::kPLd + ((lane >> 3) & 1) * 8;
         ldsm_x4(smem_u32(ph + off), bh[0], bh[1], bh[2], bh[3]);
         ldsm_x4(smem_u32(pl + off), bl[0], bl[1], bl[2], bl[3]);
 #pragma unroll
@@ -373,13 +380,13 @@ __global__ void __launch_bounds__(kHcThreads, 1) hgrn2_chunked_kernel(const RfHg
 #pragma unroll
       for (int j = 0; j < DT; ++j) {
         const int d = (j * DG + dg) * 16;
-        if (d < DP) {
+        {
           uint32_t ah[4], al[4], bh[4], bl[4];
           hc_split2(st[j][0], st[j][1], ah[0], al[0]);
           hc_split2(st[j][2], st[j][3], ah[1], al[1]);
           hc_split2(st[j][4], st[j][5], ah[2], al[2]);
           hc_split2(st[j][6], st[j][7], ah[3], al[3]);
-          const int qoff = ((lane >> 4) * 8 + (lane & 7)) * L.b_ld + d + ((lane >> 3) & 1) * 8;      // [token][channel], no transpose
+          const int qoff = ((lane >> 4) * 8 + (lane & 7)) * L::kBLd + d + ((lane >> 3) & 1) * 8;      // [token][channel], no transpose
           ldsm_x4(smem_u32(qh + qoff), bh[0], bh[1], bh[2], bh[3]);
           ldsm_x4(smem_u32(ql + qoff), bl[0], bl[1], bl[2], bl[3]);
 #pragma unroll
@@ -388,7 +395,7 @@ __global__ void __launch_bounds__(kHcThreads, 1) hgrn2_chunked_kernel(const RfHg
             MmaOp<T>::mma(o[nt], al, bh[nt * 2], bh[nt * 2 + 1]);
             MmaOp<T>::mma(o[nt], ah, bl[nt * 2], bl[nt * 2 + 1]);
           }
-          const int koff = (lane & 15) * L.b_ld + d + (lane >> 4) * 8;                              // transposed: tokens are the k axis
+          const int koff = (lane & 15) * L::kBLd + d + (lane >> 4) * 8;                              // transposed: tokens are the k axis
           ldsm_x4_t(smem_u32(kh + koff), bh[0], bh[1], bh[2], bh[3]);
           ldsm_x4_t(smem_u32(kl + koff), bl[0], bl[1], bl[2], bl[3]);
 #pragma unroll
@@ -401,11 +408,11 @@ __global__ void __launch_bounds__(kHcThreads, 1) hgrn2_chunked_kernel(const RfHg
           }
         }
       }
-      float* dst = so + dg * kHcTok * L.o_ld + vg * 16 + g;
+      float* dst = so + dg * kHcTok * L::kOLd + vg * 16 + g;
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) dst[(nt * 8 + q4 * 2 + (e & 1)) * L.o_ld + (e >> 1) * 8] = o[nt][e];
+        for (int e = 0; e < 4; ++e) dst[(nt * 8 + q4 * 2 + (e & 1)) * L::kOLd + (e >> 1) * 8] = o[nt][e];
     }
     __syncthreads();
     // ---- this step's outputs: sixteen threads per token
@@ -415,7 +422,7 @@ __global__ void __launch_bounds__(kHcThreads, 1) hgrn2_chunked_kernel(const RfHg
       for (int i = 0; i < NV; ++i) {
         float v = 0.f;
 #pragma unroll
-        for (int k = 0; k < DG; ++k) v += so[(k * kHcTok + otok) * L.o_ld + ocol + i];
+        for (int k = 0; k < DG; ++k) v += so[(k * kHcTok + otok) * L::kOLd + ocol + i];
         ov[i] = v;
         ss += v * v;
       }
@@ -445,22 +452,20 @@ __global__ void __launch_bounds__(kHcThreads, 1) hgrn2_chunked_kernel(const RfHg
     }
 }
 
-template <int VG, int DT>
+template <int VG, int DP>
 static int launch_chunked_t(const RfHgrn2* a, int tiles, cudaStream_t s) {
-  const size_t smem = hgrn2_smem(a->dim, VG * 16, kHcWarps / VG).total;
-  RF_ALLOW_SMEM_PER_DEVICE((hgrn2_chunked_kernel<VG, DT>), 200 * 1024);
-  RF_CUDA_CHECK(::rf::launch_k(hgrn2_chunked_kernel<VG, DT>, dim3(a->rows.num_seqs, a->heads, tiles), dim3(kHcThreads), smem, s, tiles, *a, tiles));
+  constexpr int smem = Hgrn2Geom<DP, VG * 16>::total;
+  RF_ALLOW_SMEM_PER_DEVICE((hgrn2_chunked_kernel<VG, DP>), smem);
+  RF_CUDA_CHECK(::rf::launch_k(hgrn2_chunked_kernel<VG, DP>, dim3(a->rows.num_seqs, a->heads, tiles), dim3(kHcThreads), smem, s, tiles, *a, tiles));
   ::rf::count_launch();
   return RF_OK;
 }
 
 template <int VG>
 static int launch_chunked(const RfHgrn2* a, int tiles, cudaStream_t s) {
-  const int per = ceil_div(ceil_div(a->dim, 16), kHcWarps / VG);      // 16-channel tiles per warp
-  if (per <= 2) return launch_chunked_t<VG, 2>(a, tiles, s);
-  if (per <= 4) return launch_chunked_t<VG, 4>(a, tiles, s);
-  if (per <= 8) return launch_chunked_t<VG, 8>(a, tiles, s);
-  return launch_chunked_t<VG, 16>(a, tiles, s);
+  if (a->dim <= 64) return launch_chunked_t<VG, 64>(a, tiles, s);
+  if (a->dim <= 128) return launch_chunked_t<VG, 128>(a, tiles, s);
+  return launch_chunked_t<VG, 256>(a, tiles, s);
 }
 
 }  // namespace rf
