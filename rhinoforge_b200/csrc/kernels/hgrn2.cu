@@ -12,6 +12,12 @@
 namespace rf {
 
 __device__ __forceinline__ float sigmoid_f32(float x) { return 1.f / (1.f + expf(-x)); }
+// for inputs that were rounded to 16 bits: a few ulp, on the special-function unit
+__device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+template <typename T> __device__ __forceinline__ float sigmoid_t(float x) {
+  if constexpr (sizeof(T) == 4) return sigmoid_f32(x);
+  else return sigmoid_fast(x);
+}
 
 // One CTA owns `cols` state columns (value channels) of one head of one sequence; thread = (column, row group), RPT state rows
 // per thread in registers (RPT = 0: the state stays in global memory, any head size).  When the value channels of a head are
@@ -48,9 +54,9 @@ __global__ void __launch_bounds__(RPT == 64 ? 512 : 1024) hgrn2_recurrent_kernel
     for (int i = threadIdx.x; i < p.dim; i += blockDim.x) {
       const int ch = head * p.dim + i;
       const float qv = Num<T>::to_f(xr[ch]);
-      sq[buf * p.dim + i] = qv * sigmoid_f32(qv);
+      sq[buf * p.dim + i] = qv * sigmoid_t<T>(qv);
       const float lo = p.lower[ch];
-      sf[buf * p.dim + i] = lo + (1.f - lo) * sigmoid_f32(Num<T>::to_f(xr[p.f_off + ch]) + p.f_bias[ch]);
+      sf[buf * p.dim + i] = lo + (1.f - lo) * sigmoid_t<T>(Num<T>::to_f(xr[p.f_off + ch]) + p.f_bias[ch]);
     }
     const float v = on ? Num<T>::to_f(xr[p.v_off + head * p.vdim + j]) : 0.f;
     __syncthreads();
@@ -169,7 +175,7 @@ template <int DP, int VT> struct Hgrn2Geom {
   static constexpr int pl = ph + kHcTok * kPLd * 2;
   static constexpr int so = pl + kHcTok * kPLd * 2;               // [warps of a value group][16][VT] partial outputs
   static constexpr int csum = so + kDG * kHcTok * kOLd * 4;
-  static constexpr int total = csum + 2 * kHcTok * 4;
+  static constexpr int total = csum + 2 * 8 * kHcTok * 4;         // [2][cluster rank][16]
 };
 
 __device__ __forceinline__ void hc_cp16(uint32_t dst, const void* src, bool valid) {
@@ -264,7 +270,7 @@ __global__ void __launch_bounds__(kHcThreads, DP == 256 ? 1 : 2) hgrn2_chunked_k
     float tot = own;
     if (col_tiles > 1) {
       tot = 0.f;
-      for (int c = 0; c < col_tiles; ++c) tot += ld_dsmem_f32(dsmem_addr(smem_u32(csum + buf * kHcTok + otok), (uint32_t)c));
+      for (int c = 0; c < col_tiles; ++c) tot += csum[(buf * 8 + c) * kHcTok + otok];
     }
     const int v = v0 + ocol;
     if (orow < 0 || v >= p.vdim) return;
@@ -289,10 +295,10 @@ __global__ void __launch_bounds__(kHcThreads, DP == 256 ? 1 : 2) hgrn2_chunked_k
       const float2 y = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(rw + t * L::kRawLd + DP + gc));
       const bool in = t < valid && gc < p.dim;
       float2 q, f;
-      q.x = in ? z.x * sigmoid_f32(z.x) : 0.f;
-      q.y = in ? z.y * sigmoid_f32(z.y) : 0.f;
-      f.x = in ? g_lo[0] + (1.f - g_lo[0]) * sigmoid_f32(y.x + g_b[0]) : 1.f;
-      f.y = in ? g_lo[1] + (1.f - g_lo[1]) * sigmoid_f32(y.y + g_b[1]) : 1.f;
+      q.x = in ? z.x * sigmoid_fast(z.x) : 0.f;
+      q.y = in ? z.y * sigmoid_fast(z.y) : 0.f;
+      f.x = in ? g_lo[0] + (1.f - g_lo[0]) * sigmoid_fast(y.x + g_b[0]) : 1.f;
+      f.y = in ? g_lo[1] + (1.f - g_lo[1]) * sigmoid_fast(y.y + g_b[1]) : 1.f;
       *reinterpret_cast<float2*>(sq + t * L::kQLd + gc) = q;
       *reinterpret_cast<float2*>(sf + t * L::kQLd + gc) = f;
     }
@@ -365,7 +371,7 @@ __global__ void __launch_bounds__(kHcThreads, DP == 256 ? 1 : 2) hgrn2_chunked_k
     {
       uint32_t va[4];                            // V^T of this warp's value channels (rows) over the sixteen tokens
       ldsm_x4_t(smem_u32(rw + ((lane >> 4) * 8 + (lane & 7)) * L::kRawLd + 2 * DP + vg * 16 + ((lane >> 3) & 1) * 8), va[0], va[1], va[2], va[3]);
-      float o[2][4] = {};
+      float o[2][4] = {}, o1[2][4] = {}, o2[2][4] = {};      // separate sums: no chain of dependent products
       if (dg == 0) {
         uint32_t bh[4], bl[4];
         const int off = ((lane >> 4) * 8 + (lane & 7)) * L::kPLd + ((lane >> 3) & 1) * 8;
@@ -392,8 +398,8 @@ __global__ void __launch_bounds__(kHcThreads, DP == 256 ? 1 : 2) hgrn2_chunked_k
 #pragma unroll
           for (int nt = 0; nt < 2; ++nt) {
             MmaOp<T>::mma(o[nt], ah, bh[nt * 2], bh[nt * 2 + 1]);
-            MmaOp<T>::mma(o[nt], al, bh[nt * 2], bh[nt * 2 + 1]);
-            MmaOp<T>::mma(o[nt], ah, bl[nt * 2], bl[nt * 2 + 1]);
+            MmaOp<T>::mma(o1[nt], al, bh[nt * 2], bh[nt * 2 + 1]);
+            MmaOp<T>::mma(o2[nt], ah, bl[nt * 2], bl[nt * 2 + 1]);
           }
           const int koff = (lane & 15) * L::kBLd + d + (lane >> 4) * 8;                              // transposed: tokens are the k axis
           ldsm_x4_t(smem_u32(kh + koff), bh[0], bh[1], bh[2], bh[3]);
@@ -412,7 +418,7 @@ __global__ void __launch_bounds__(kHcThreads, DP == 256 ? 1 : 2) hgrn2_chunked_k
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) dst[(nt * 8 + q4 * 2 + (e & 1)) * L::kOLd + (e >> 1) * 8] = o[nt][e];
+        for (int e = 0; e < 4; ++e) dst[(nt * 8 + q4 * 2 + (e & 1)) * L::kOLd + (e >> 1) * 8] = o[nt][e] + (o1[nt][e] + o2[nt][e]);
     }
     __syncthreads();
     // ---- this step's outputs: sixteen threads per token
@@ -430,7 +436,9 @@ __global__ void __launch_bounds__(kHcThreads, DP == 256 ? 1 : 2) hgrn2_chunked_k
       for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
       orow = otok < valid ? q0 + b * kHcTok + otok : -1;
       if (col_tiles > 1) {
-        if ((tid & 15) == 0) csum[(b & 1) * kHcTok + otok] = ss;
+        // lane c of a token's sixteen threads stores the sum into CTA c of the cluster
+        if ((tid & 15) < col_tiles)
+          st_dsmem_u32(dsmem_addr(smem_u32(csum + ((b & 1) * 8 + (int)cluster_ctarank()) * kHcTok + otok), (uint32_t)(tid & 15)), __float_as_uint(ss));
         __syncwarp();
         asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
       } else {
@@ -441,7 +449,6 @@ __global__ void __launch_bounds__(kHcThreads, DP == 256 ? 1 : 2) hgrn2_chunked_k
   if (col_tiles > 1) {
     asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
     finish((steps - 1) & 1, 0.f);
-    cluster_sync_all();                          // no CTA leaves while its sums may still be read
   }
 #pragma unroll
   for (int j = 0; j < DT; ++j)
@@ -506,7 +513,7 @@ extern "C" int rf_hgrn2_chunked(const RfHgrn2* a, rf_stream_t stream) {
   int vt = a->vdim <= 32 ? 32 : a->vdim <= 64 ? 64 : 128;
   for (int t : {32, 64}) {
     const int tiles = ceil_div(a->vdim, t);
-    if (tiles <= 8 && (long)a->rows.num_seqs * a->heads * tiles <= 2 * sm_count()) { vt = t; break; }
+    if (tiles <= 8 && (long)a->rows.num_seqs * a->heads * tiles <= sm_count()) { vt = std::min(vt, t); break; }
   }
   const int tiles = ceil_div(a->vdim, vt);
   if (vt == 32) return launch_chunked<2>(a, tiles, s);

@@ -248,8 +248,9 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const RfLatentAttn p) 
 }
 
 // 16-bit form on the tensor cores.  One CTA (eight warps) takes MT * 16 heads of one row and a range of its keys, 64 keys per
-// step: every warp scores 8 keys against all heads, the softmax runs row-wise over shared memory, and every warp accumulates
-// NT * 8 columns of the latent output.  The cached rows are keys and values both, so a key block is read once.  The
+// step.  Scores: a warp holds a quarter of the latent columns of all its queries in registers for the whole launch and scores
+// half of the keys; the quarters are summed by the softmax, which runs row-wise over shared memory.  Output: every warp
+// accumulates NT * 8 latent columns.  The cached rows are keys and values both, so a key block is read once.  The
 // probabilities enter the second product as a 16-bit pair (value + remainder), so they keep about 16 mantissa bits.
 constexpr int kLaKeys = 64, kLaThreads = 256;
 
@@ -259,23 +260,26 @@ struct LatentSplit {
   int splits;
 };
 
-__host__ __device__ constexpr int la_ld(int rank) { return (rank + 31) / 32 * 32 + 8; }
-static size_t la_smem(int rank, int mt) {
-  return (size_t)(16 * mt + 2 * kLaKeys) * la_ld(rank) * 2 + (size_t)16 * mt * (kLaKeys + 4) * 4 + (size_t)2 * 16 * mt * (kLaKeys + 8) * 2 +
-         (size_t)16 * mt * 3 * 4;
-}
+template <int NT, int MT> struct LaGeom {
+  static constexpr int M = 16 * MT, LD = NT * 64 + 8, LDS = kLaKeys + 4, LDP = kLaKeys + 8;
+  static constexpr int c = 0;                                       // [2][64][LD] key blocks (the queries pass through here first)
+  static constexpr int s = c + 2 * kLaKeys * LD * 2;                // [4][M][LDS] score quarters
+  static constexpr int p = s + 4 * M * LDS * 4;                     // [2][M][LDP] probabilities: value, remainder
+  static constexpr int m = p + 2 * M * LDP * 2;                     // running maximum, sum, rescale of this step
+  static constexpr int total = m + 3 * M * 4;
+};
 
 template <typename T, int NT, int MT>
 __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const RfLatentAttn p, const LatentSplit sp) {
   pdl_prologue();
-  constexpr int M = 16 * MT, LDS = kLaKeys + 4, LDP = kLaKeys + 8;
+  using L = LaGeom<NT, MT>;
+  constexpr int M = L::M, ld = L::LD, LDS = L::LDS, LDP = L::LDP, RP = NT * 64;
   extern __shared__ __align__(16) uint8_t lsm[];
-  const int rank = p.rank, ld = la_ld(rank), rp = ld - 8;
-  T* sQ = reinterpret_cast<T*>(lsm);                       // [M][ld]
-  T* sC = sQ + M * ld;                                     // [2][64][ld]
-  float* sS = reinterpret_cast<float*>(sC + 2 * kLaKeys * ld);   // [M][LDS]
-  T* sP = reinterpret_cast<T*>(sS + M * LDS);              // [2][M][LDP]: value, remainder
-  float* sM = reinterpret_cast<float*>(sP + 2 * M * LDP);  // running maximum, sum, rescale of this step
+  const int rank = p.rank;
+  T* sC = reinterpret_cast<T*>(lsm + L::c);
+  float* sS = reinterpret_cast<float*>(lsm + L::s);
+  T* sP = reinterpret_cast<T*>(lsm + L::p);
+  float* sM = reinterpret_cast<float*>(lsm + L::m);
   float* sL = sM + M;
   float* sA = sL + M;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
@@ -287,21 +291,36 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
   const int b0 = split * per, b1 = min(blocks, b0 + per);
   const T* pool = reinterpret_cast<const T*>(p.pool);
   const T* q = reinterpret_cast<const T*>(p.q) + ((size_t)row * p.heads + h0) * rank;
-  const int heads_here = min(M, p.heads - h0), chunks = rp / 8;
+  const int heads_here = min(M, p.heads - h0);
+  const int kq = warp >> 1, key0 = (warp & 1) * 32;        // this warp's column quarter and key half for the scores
 
-  for (int i = tid; i < M * chunks; i += kLaThreads) {
-    const int r = i / chunks, c = (i % chunks) * 8;
+  for (int i = tid; i < M * (RP / 8); i += kLaThreads) {
+    const int r = i / (RP / 8), c = (i % (RP / 8)) * 8;
     const bool ok = r < heads_here && c < rank;
-    la_cp16(smem_u32(sQ + r * ld + c), ok ? q + (size_t)r * rank + c : q, ok);
+    la_cp16(smem_u32(sC + r * ld + c), ok ? q + (size_t)r * rank + c : q, ok);
   }
+  la_commit();
+  if (tid < M) { sM[tid] = -INFINITY; sL[tid] = 0.f; }
+  la_wait<0>();
+  __syncthreads();
+  uint32_t qf[MT][NT][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int k = 0; k < NT; ++k)
+      ldsm_x4(smem_u32(sC + (m * 16 + (lane & 15)) * ld + kq * NT * 16 + k * 16 + (lane >> 4) * 8), qf[m][k][0], qf[m][k][1], qf[m][k][2], qf[m][k][3]);
+  __syncthreads();
   auto load_keys = [&](int b) {                            // four threads per key row
     const int r = tid >> 2, j = lo + b * kLaKeys + r;
     const bool in = j <= pos;
     const T* src = in ? pool + ((size_t)pt[j >> 4] * 16 + (j & 15)) * rank : pool;
     T* dst = sC + ((b & 1) * kLaKeys + r) * ld;
-    for (int c = (tid & 3) * 8; c < rp; c += 32) la_cp16(smem_u32(dst + c), in && c < rank ? src + c : pool, in && c < rank);
+#pragma unroll
+    for (int i = 0; i < RP / 32; ++i) {
+      const int c = (tid & 3) * 8 + i * 32;
+      la_cp16(smem_u32(dst + c), in && c < rank ? src + c : pool, in && c < rank);
+    }
   };
-  if (tid < M) { sM[tid] = -INFINITY; sL[tid] = 0.f; }
   if (b0 < b1) load_keys(b0);
   la_commit();
   float acc[MT][NT][4] = {};
@@ -313,37 +332,43 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
     la_wait<1>();
     __syncthreads();
     const T* kc = sC + (b & 1) * kLaKeys * ld;
-    {  // scores of this warp's eight keys
-      float s[MT][4] = {};
-      for (int k = 0; k < rp; k += 32) {
-        uint32_t bf[4];
-        ldsm_x4(smem_u32(kc + (warp * 8 + (lane & 7)) * ld + k + (lane >> 3) * 8), bf[0], bf[1], bf[2], bf[3]);
+    {
+      float s[MT][4][4] = {};
 #pragma unroll
-        for (int m = 0; m < MT; ++m)
+      for (int k = 0; k < NT; ++k)
 #pragma unroll
-          for (int hk = 0; hk < 2; ++hk) {
-            uint32_t a[4];
-            ldsm_x4(smem_u32(sQ + (m * 16 + (lane & 15)) * ld + k + hk * 16 + (lane >> 4) * 8), a[0], a[1], a[2], a[3]);
-            MmaOp<T>::mma(s[m], a, bf[hk * 2], bf[hk * 2 + 1]);
+        for (int np = 0; np < 2; ++np) {                   // sixteen keys, one k16 step
+          uint32_t bf[4];
+          ldsm_x4(smem_u32(kc + (key0 + np * 16 + (lane >> 4) * 8 + (lane & 7)) * ld + kq * NT * 16 + k * 16 + ((lane >> 3) & 1) * 8), bf[0], bf[1], bf[2], bf[3]);
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            MmaOp<T>::mma(s[m][np * 2], qf[m][k], bf[0], bf[1]);
+            MmaOp<T>::mma(s[m][np * 2 + 1], qf[m][k], bf[2], bf[3]);
           }
-      }
-      const int key = warp * 8 + q4 * 2, j = lo + b * kLaKeys + key;
+        }
+      float* dst = sS + kq * M * LDS;
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          float2 v;
-          v.x = j <= pos ? s[m][half * 2] * scale_log2 : -INFINITY;
-          v.y = j + 1 <= pos ? s[m][half * 2 + 1] * scale_log2 : -INFINITY;
-          *reinterpret_cast<float2*>(sS + (m * 16 + g + half * 8) * LDS + key) = v;
-        }
+        for (int n = 0; n < 4; ++n)
+#pragma unroll
+          for (int half = 0; half < 2; ++half)
+            *reinterpret_cast<float2*>(dst + (m * 16 + g + half * 8) * LDS + key0 + n * 8 + q4 * 2) = make_float2(s[m][n][half * 2], s[m][n][half * 2 + 1]);
     }
     __syncthreads();
     // softmax step of 2 * MT rows per warp (every block holds at least one visible key)
 #pragma unroll
     for (int i = 0; i < 2 * MT; ++i) {
       const int r = warp * 2 * MT + i;
-      const float2 v = *reinterpret_cast<const float2*>(sS + r * LDS + lane * 2);
+      float2 v = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 t = *reinterpret_cast<const float2*>(sS + (k * M + r) * LDS + lane * 2);
+        v.x += t.x; v.y += t.y;
+      }
+      const int j = lo + b * kLaKeys + lane * 2;
+      v.x = j <= pos ? v.x * scale_log2 : -INFINITY;
+      v.y = j + 1 <= pos ? v.y * scale_log2 : -INFINITY;
       const float old = sM[r], mx = fmaxf(old, warp_max(fmaxf(v.x, v.y)));
       const float p0 = exp2f(v.x - mx), p1 = exp2f(v.y - mx);
       const float sum = warp_sum(p0 + p1);
@@ -381,7 +406,7 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
 #pragma unroll
       for (int t = 0; t < NT; ++t) {
         const int c = (warp * NT + t) * 8;
-        if (c < rp) {
+        {
           uint32_t bf[4];                                  // eight columns, 32 keys
           ldsm_x4_t(smem_u32(kc + (kk + lane) * ld + c), bf[0], bf[1], bf[2], bf[3]);
 #pragma unroll
@@ -522,11 +547,11 @@ static int launch_latent_attn_mma(const RfLatentAttn* a, cudaStream_t s) {
   sp.o = a->ws;
   sp.ml = a->ws ? a->ws + slots * a->rank : nullptr;
   const int mt = a->heads <= 16 ? 1 : 2;
-  const size_t smem = la_smem(a->rank, mt);
   const dim3 grid(sp.splits, ceil_div(a->heads, 16 * mt), a->n_rows);
 #define RF_LM(NT, MT)                                                                                             \
   do {                                                                                                            \
-    RF_ALLOW_SMEM_PER_DEVICE((latent_attn_mma_kernel<T, NT, MT>), la_smem(NT * 64, MT));                          \
+    constexpr int smem = LaGeom<NT, MT>::total;                                                                   \
+    RF_ALLOW_SMEM_PER_DEVICE((latent_attn_mma_kernel<T, NT, MT>), smem);                                          \
     RF_CUDA_CHECK(::rf::launch_k(latent_attn_mma_kernel<T, NT, MT>, grid, dim3(kLaThreads), smem, s, 1, *a, sp)); \
   } while (0)
 #define RF_LN(NT)             \
