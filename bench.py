@@ -29,9 +29,10 @@ def parse_args(argv=None):
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="decode", choices=["decode", "pi05", "qwen3vl"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "pi05", "qwen3vl", "vabarax"],
                     help="decode: causal-LM decode throughput (headline); pi05: action-chunk latency; "
-                         "qwen3vl: multimodal prefill + decode")
+                         "qwen3vl: multimodal prefill + decode; vabarax: latent-attention / HGRN2 decoder beside the "
+                         "hybrid K/V + Gated-DeltaNet decoder at equal size")
     ap.add_argument("--model", default="qwen3-8b")
     ap.add_argument("--batch", type=int, default=64)
     ap.add_argument("--prompt-len", type=int, default=1024)
@@ -536,13 +537,143 @@ def run_qwen3vl(args) -> dict:
     }
 
 
+VABARAX_SIZES = {          # width, heads (of 128), latent rank, window, feed-forward, side width, layers (half attention)
+    "1b": (2048, 16, 256, 1024, 8192, 128, 16),
+    "4b": (3072, 24, 512, 1024, 12288, 256, 16),
+    "8b": (4096, 32, 512, 1024, 16384, 256, 16),
+}
+
+
+def _serve(eng, vocab: int, batches, prompt_len: int, steps: int, warmup: int, total_prompts: int):
+    """Device-timed prefill of ``total_prompts`` prompts and decode steps at every batch size of one engine."""
+    import torch
+    from rhinoforge_b200 import _native as N
+    lib = N.lib()
+    lib.rf_launch_count.restype = __import__("ctypes").c_uint64
+    gen = torch.Generator().manual_seed(0)
+    prompts = [torch.randint(0, vocab, (prompt_len,), generator=gen) for _ in range(max(max(batches), total_prompts))]
+    pre_ms, clocks = _timed(lambda: eng.prefill(prompts[:total_prompts]), 5, 3)
+    out = {"prefill_tok_s": total_prompts * prompt_len * 1000.0 / statistics.median(pre_ms), "prefill_ms": statistics.median(pre_ms), "decode": {}}
+    for B in batches:
+        eng.prefill(prompts[:B])
+        c0 = lib.rf_launch_count()
+        eng.capture(B)
+        per_step = int(lib.rf_launch_count() - c0) // 2
+        eng.decode(max(warmup, 3))
+        eng.reserve_steps(steps)
+        sampler = ClockSampler(torch.cuda.current_device())
+        sampler.start()
+        sampler.wait_first()
+        torch.cuda.synchronize()
+        sampler.mark()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(steps):
+            eng.graphs[B].replay()
+        e1.record()
+        torch.cuda.synchronize()
+        ms = e0.elapsed_time(e1) / steps
+        eng.advance_lengths(steps)
+        eng.check_status()
+        clocks = sampler.stop()
+        out["decode"][str(B)] = {"tok_s": B * 1000.0 / ms, "ms_per_step": ms, "launches_per_step": per_step, "clocks": clocks}
+    # end to end: the scheduler's step with this step's ids copied from the host and the next ids read back
+    from rhinoforge_b200.runtime.scheduler import RequestScheduler
+    B = max(batches)
+    sched = RequestScheduler(eng)
+    nxt = sched.step([(b, prompts[b][:64], ()) for b in range(B)])[0].cpu()
+    n = min(steps, 32)
+    t1 = None
+    for i in range(n + 3):
+        if i == 3:
+            torch.cuda.synchronize()
+            t1 = time.perf_counter()
+        nxt = sched.step([(b, nxt[b:b + 1], ()) for b in range(B)])[0].cpu()
+    out["e2e_tok_s"] = B * n / (time.perf_counter() - t1)
+    eng.check_status()
+    return out
+
+
+def run_vabarax(args) -> dict:
+    """Prefill and decode throughput of the Vabarax design at a few sizes, beside the closest decoder of this framework - the
+    hybrid of softmax attention (grouped K/V heads, SwiGLU) and Gated-DeltaNet layers - with the same width, heads, feed-forward
+    parameters, layer count, prompts and batch sizes.  Random weights, synthetic ids; a "step" is one decode step."""
+    import torch
+    from rhinoforge_b200.models.decoder import DecoderConfig
+    from rhinoforge_b200.models.mixed import DenseMLP, HGRN2, LatentAttention, MixedConfig, MixedLayer, random_weights, weight_shapes
+    from rhinoforge_b200.runtime.engine import DecoderEngine, random_weight_getter
+    from rhinoforge_b200.runtime.mixed_engine import MixedDecoderEngine
+    if args.gpus != 1:
+        raise SystemExit("the vabarax workload runs on one GPU")
+    torch.cuda.set_device(0)
+    batches = sorted({1, 8, args.batch})
+    vocab, prompt, npre = 32768, args.prompt_len, 8
+    max_seq = prompt + 2 * args.steps + args.warmup + 128
+    res = {}
+    for name, (H, heads, rank, window, ff, side, layers) in VABARAX_SIZES.items():
+        att = MixedLayer(LatentAttention(heads, 128, 128, rank, 128 ** -0.5, window), DenseMLP(ff))
+        lin = MixedLayer(HGRN2(heads, 128, 128), DenseMLP(ff))
+        cfg = MixedConfig("vabarax-" + name, vocab, H, 1e-6, (att, lin) * (layers // 2), side)
+        eng = MixedDecoderEngine(cfg, random_weights(cfg, device="cuda"), dtype=torch.bfloat16, max_batch=max(batches), max_seq_len=max_seq)
+        r = {"params_m": round(sum(int(torch.Size(s).numel()) for _, s, _ in weight_shapes(cfg)) / 1e6), "ours": _serve(
+            eng, vocab, batches, prompt, args.steps, args.warmup, npre), "cache_mb": round(eng.cache.nbytes() / 1e6)}
+        eng.close()
+        del eng
+        torch.cuda.empty_cache()
+        # the closest existing decoder: a GLU of 2/3 of the width has the same feed-forward parameters
+        inter = (2 * ff // 3 + 127) // 128 * 128
+        like = DecoderConfig("hybrid-" + name, vocab, H, inter, layers, heads, heads // 4, 128, tie_embeddings=True, norm="rms_gemma",
+                             attn_gate=True, model_type="qwen3_5", layer_types=("full_attention", "linear_attention") * (layers // 2),
+                             gdn_heads_k=heads, gdn_heads_v=heads, gdn_dk=128, gdn_dv=128)
+        try:
+            eng = DecoderEngine(like, _hybrid_weights(like, random_weight_getter), dtype=torch.bfloat16, max_batch=max(batches), max_seq_len=max_seq)
+            r["closest"] = _serve(eng, vocab, batches, prompt, args.steps, args.warmup, npre)
+            eng.close()
+            del eng
+        finally:
+            torch.cuda.empty_cache()
+        r["ratio"] = {"prefill": r["ours"]["prefill_tok_s"] / r["closest"]["prefill_tok_s"],
+                      **{f"decode_{b}": r["ours"]["decode"][str(b)]["tok_s"] / r["closest"]["decode"][str(b)]["tok_s"] for b in batches}}
+        res[name] = r
+    big = list(res.values())[-1]["ours"]
+    d = big["decode"][str(args.batch)]
+    return {"metric": "vabarax_decode_tokens_per_s", "value": d["tok_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
+            "warmup": max(args.warmup, 3), "ms_per_step": d["ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None,
+            "dtype": "bf16", "data": "synthetic", "impl": "ours",
+            "config": {"model": "Vabarax-8b-sized random-init", "global_batch": args.batch, "seq_len": prompt, "parallelism": "tp1",
+                       "sizes": {k: dict(zip(("width", "heads", "rank", "window", "ff", "side", "layers"), v)) for k, v in VABARAX_SIZES.items()},
+                       "l2": "weights exceed L2"},
+            "clocks": d["clocks"], "e2e": {"value": big["e2e_tok_s"], "unit": "tokens/s", "h2d_bytes_per_step": 12 * args.batch,
+                                           "d2h_bytes_per_step": 4 * args.batch},
+            "gpu_launches": d["launches_per_step"] * args.steps, "by_size": res}
+
+
+def _hybrid_weights(cfg, base):
+    """Random weights of a hybrid decoder: the dense tensors from ``base``, the doubled query projection and the
+    linear-attention tensors made here."""
+    import torch
+    dense = base(cfg, seed=0, std=0.02, dtype=torch.bfloat16)
+    H, hd = cfg.hidden_size, cfg.head_dim
+    key, val = cfg.gdn_heads_k * cfg.gdn_dk, cfg.gdn_heads_v * cfg.gdn_dv
+    shapes = {"in_proj_qkv.weight": (2 * key + val, H), "in_proj_z.weight": (val, H), "in_proj_b.weight": (cfg.gdn_heads_v, H),
+              "in_proj_a.weight": (cfg.gdn_heads_v, H), "out_proj.weight": (H, val), "conv1d.weight": (2 * key + val, 1, cfg.gdn_conv),
+              "A_log": (cfg.gdn_heads_v,), "dt_bias": (cfg.gdn_heads_v,), "norm.weight": (cfg.gdn_dv,), "q_proj.weight": (2 * cfg.num_heads * hd, H)}
+
+    def get(name: str):
+        tail = next((t for t in shapes if name.endswith("linear_attn." + t) or (t == "q_proj.weight" and name.endswith("self_attn." + t))), None)
+        if tail is None:
+            return dense(name)
+        return torch.randn(shapes[tail], device="cuda", dtype=torch.bfloat16).mul_(0.02)
+    return get
+
+
 def main(argv=None) -> int:
     args = parse_args(argv)
     if args.impl == "reference":
         if int(os.environ.get("RANK", "0")) == 0:          # one line per job, also under torch.distributed.run
             print(json.dumps({"impl": "reference", "unavailable": REFERENCE_UNAVAILABLE}))
         return 0
-    out = {"decode": run, "pi05": run_pi05, "qwen3vl": run_qwen3vl}[args.workload](args)
+    out = {"decode": run, "pi05": run_pi05, "qwen3vl": run_qwen3vl, "vabarax": run_vabarax}[args.workload](args)
     if out is not None:
         print(json.dumps(out))
     try:

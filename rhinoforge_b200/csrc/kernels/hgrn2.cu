@@ -45,7 +45,11 @@ __global__ void __launch_bounds__(RPT == 64 ? 512 : 1024) hgrn2_recurrent_kernel
   float st[NR];
   if constexpr (RPT > 0) {
 #pragma unroll
-    for (int r = 0; r < RPT; ++r) st[r] = (on && !fresh && row0 + r < p.dim) ? S[(size_t)(row0 + r) * p.vdim + j] : 0.f;
+    for (int r = 0; r < RPT; ++r) st[r] = (on && row0 + r < p.dim) ? __ldcs(S + (size_t)(row0 + r) * p.vdim + j) : 0.f;
+    if (fresh) {                               // checked after the loads are in flight
+#pragma unroll
+      for (int r = 0; r < RPT; ++r) st[r] = 0.f;
+    }
   }
   const float nw = (p.norm_w && on) ? p.norm_w[j] : 1.f;
   for (int t = 0; t < n; ++t) {
@@ -90,7 +94,7 @@ __global__ void __launch_bounds__(RPT == 64 ? 512 : 1024) hgrn2_recurrent_kernel
       if ((threadIdx.x & 31) == 0) ws[threadIdx.x >> 5] = s;
       __syncthreads();
       float tot = 0.f;
-      for (int w = 0; w < (int)((blockDim.x + 31) / 32); ++w) tot += ws[w];
+      for (int w = 0; w < cols / 32; ++w) tot += ws[w];        // row group 0's warps
       if (col_tiles > 1) {
         if (threadIdx.x == 0) csum[buf] = tot;
         cluster_sync_all();
@@ -105,7 +109,7 @@ __global__ void __launch_bounds__(RPT == 64 ? 512 : 1024) hgrn2_recurrent_kernel
     if (on) {
 #pragma unroll
       for (int r = 0; r < RPT; ++r)
-        if (row0 + r < p.dim) S[(size_t)(row0 + r) * p.vdim + j] = st[r];
+        if (row0 + r < p.dim) __stcs(S + (size_t)(row0 + r) * p.vdim + j, st[r]);
     }
   }
   if (col_tiles > 1) cluster_sync_all();       // no CTA leaves while its sum may still be read
