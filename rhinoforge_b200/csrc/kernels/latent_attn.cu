@@ -356,32 +356,52 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
             *reinterpret_cast<float2*>(dst + (m * 16 + g + half * 8) * LDS + key0 + n * 8 + q4 * 2) = make_float2(s[m][n][half * 2], s[m][n][half * 2 + 1]);
     }
     __syncthreads();
-    // softmax step of 2 * MT rows per warp (every block holds at least one visible key)
+    // softmax step of 2 * MT rows per warp, all of them in flight (every block holds at least one visible key)
+    {
+      constexpr int NR = 2 * MT;
+      const int r0 = warp * NR, j = lo + b * kLaKeys + lane * 2;
+      float2 v[NR];
+      float old[NR], mx[NR], sum[NR];
 #pragma unroll
-    for (int i = 0; i < 2 * MT; ++i) {
-      const int r = warp * 2 * MT + i;
-      float2 v = make_float2(0.f, 0.f);
+      for (int i = 0; i < NR; ++i) {
+        v[i] = make_float2(0.f, 0.f);
+        old[i] = sM[r0 + i];
 #pragma unroll
-      for (int k = 0; k < 4; ++k) {
-        const float2 t = *reinterpret_cast<const float2*>(sS + (k * M + r) * LDS + lane * 2);
-        v.x += t.x; v.y += t.y;
+        for (int k = 0; k < 4; ++k) {
+          const float2 t = *reinterpret_cast<const float2*>(sS + (k * M + r0 + i) * LDS + lane * 2);
+          v[i].x += t.x; v[i].y += t.y;
+        }
+        v[i].x = j <= pos ? v[i].x * scale_log2 : -INFINITY;
+        v[i].y = j + 1 <= pos ? v[i].y * scale_log2 : -INFINITY;
+        mx[i] = fmaxf(v[i].x, v[i].y);
       }
-      const int j = lo + b * kLaKeys + lane * 2;
-      v.x = j <= pos ? v.x * scale_log2 : -INFINITY;
-      v.y = j + 1 <= pos ? v.y * scale_log2 : -INFINITY;
-      const float old = sM[r], mx = fmaxf(old, warp_max(fmaxf(v.x, v.y)));
-      const float p0 = exp2f(v.x - mx), p1 = exp2f(v.y - mx);
-      const float sum = warp_sum(p0 + p1);
-      const T a0 = Num<T>::from_f(p0), a1 = Num<T>::from_f(p1);
-      *reinterpret_cast<uint32_t*>(sP + r * LDP + lane * 2) = MmaOp<T>::pack(p0, p1);
-      *reinterpret_cast<uint32_t*>(sP + (M + r) * LDP + lane * 2) = MmaOp<T>::pack(p0 - Num<T>::to_f(a0), p1 - Num<T>::to_f(a1));
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int i = 0; i < NR; ++i) mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], o));
+#pragma unroll
+      for (int i = 0; i < NR; ++i) {
+        mx[i] = fmaxf(mx[i], old[i]);
+        v[i].x = exp2f(v[i].x - mx[i]);
+        v[i].y = exp2f(v[i].y - mx[i]);
+        sum[i] = v[i].x + v[i].y;
+        const T a0 = Num<T>::from_f(v[i].x), a1 = Num<T>::from_f(v[i].y);
+        *reinterpret_cast<uint32_t*>(sP + (r0 + i) * LDP + lane * 2) = MmaOp<T>::pack(v[i].x, v[i].y);
+        *reinterpret_cast<uint32_t*>(sP + (M + r0 + i) * LDP + lane * 2) = MmaOp<T>::pack(v[i].x - Num<T>::to_f(a0), v[i].y - Num<T>::to_f(a1));
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int i = 0; i < NR; ++i) sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], o);
       __syncwarp();
-      if (lane == 0) {
-        const float corr = exp2f(old - mx);
-        sA[r] = corr;
-        sL[r] = sL[r] * corr + sum;
-        sM[r] = mx;
-      }
+#pragma unroll
+      for (int i = 0; i < NR; ++i)
+        if (lane == i) {
+          const float corr = exp2f(old[i] - mx[i]);
+          sA[r0 + i] = corr;
+          sL[r0 + i] = sL[r0 + i] * corr + sum[i];
+          sM[r0 + i] = mx[i];
+        }
     }
     __syncthreads();
 #pragma unroll
@@ -447,19 +467,36 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
 }
 
 template <typename T>
-__global__ void latent_combine_kernel(const LatentSplit sp, T* __restrict__ o, int rank) {
+__global__ void __launch_bounds__(128) latent_combine_kernel(const LatentSplit sp, T* __restrict__ o, int rank) {
   pdl_prologue();
   const size_t hr = blockIdx.x;
-  const float* ml = sp.ml + hr * sp.splits * 2;
-  float m = -INFINITY, l = 0.f;
-  for (int s = 0; s < sp.splits; ++s) m = fmaxf(m, ml[s * 2]);
-  for (int s = 0; s < sp.splits; ++s) l += ml[s * 2] == -INFINITY ? 0.f : exp2f(ml[s * 2] - m) * ml[s * 2 + 1];
-  const float inv = 1.f / l;
-  for (int c = threadIdx.x; c < rank; c += blockDim.x) {
-    float v = 0.f;
-    for (int s = 0; s < sp.splits; ++s)
-      if (ml[s * 2] != -INFINITY) v += exp2f(ml[s * 2] - m) * sp.o[(hr * sp.splits + s) * rank + c];
-    o[hr * rank + c] = Num<T>::from_f(v * inv);
+  __shared__ float sw[64];                                 // weight of every split
+  if (threadIdx.x < 32) {
+    const float* ml = sp.ml + hr * sp.splits * 2;
+    float m = -INFINITY, l = 0.f;
+    for (int s = threadIdx.x; s < sp.splits; s += 32) m = fmaxf(m, ml[s * 2]);
+    m = warp_max(m);
+    for (int s = threadIdx.x; s < sp.splits; s += 32) {
+      const float w = exp2f(ml[s * 2] - m);                // a split without keys: maximum -inf, weight 0
+      sw[s] = w;
+      l += w * ml[s * 2 + 1];
+    }
+    l = warp_sum(l);
+    for (int s = threadIdx.x; s < sp.splits; s += 32) sw[s] /= l;
+  }
+  __syncthreads();
+  for (int c = threadIdx.x * 4; c < rank; c += blockDim.x * 4) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int s = 0; s < sp.splits; ++s) {
+      const float4 t = *reinterpret_cast<const float4*>(sp.o + (hr * sp.splits + s) * rank + c);
+      const float w = sw[s];
+      v.x += w * t.x; v.y += w * t.y; v.z += w * t.z; v.w += w * t.w;
+    }
+    uint2 u;
+    u.x = MmaOp<T>::pack(v.x, v.y);
+    u.y = MmaOp<T>::pack(v.z, v.w);
+    *reinterpret_cast<uint2*>(o + hr * rank + c) = u;
   }
 }
 
@@ -567,7 +604,7 @@ static int launch_latent_attn_mma(const RfLatentAttn* a, cudaStream_t s) {
 #undef RF_LM
   ::rf::count_launch();
   if (sp.splits > 1) {
-    RF_CUDA_CHECK(::rf::launch_k(latent_combine_kernel<T>, dim3(a->n_rows * a->heads), dim3(std::min(512, round_up(a->rank, 32))), 0, s, 1,
+    RF_CUDA_CHECK(::rf::launch_k(latent_combine_kernel<T>, dim3(a->n_rows * a->heads), dim3(std::min(128, round_up(a->rank / 4, 32))), 0, s, 1,
                                  sp, (T*)a->o, a->rank));
     ::rf::count_launch();
   }

@@ -124,6 +124,121 @@ __global__ void stream_norm_kernel(const RfStreamNorm p, int rows_per_cta) {
   }
 }
 
+// The same for rows that fit the registers of a CTA (VPT quads per thread): every operand of a row is requested before the
+// first reduction, so a decode step pays one memory round trip, and the next row's operands are requested while the current
+// one is reduced.
+template <typename T, int VPT>
+__global__ void __launch_bounds__(VPT == 4 ? 512 : 1024) stream_norm_reg_kernel(const RfStreamNorm p, int rows_per_cta) {
+  pdl_launch_dependents();
+  __shared__ float red[2][32];
+  const int H = p.H, nthr = blockDim.x, nw = nthr >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float inv_dim = 1.f / (float)p.dim;
+  const T* table = reinterpret_cast<const T*>(p.table);
+  const T* y = reinterpret_cast<const T*>(p.y);
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  auto col = [&](int k) { return (threadIdx.x + k * nthr) * 4; };
+  // weights do not depend on the previous kernel
+  float4 nwt[VPT], mu[VPT], yw[VPT];
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const bool in = col(k) < H;
+    nwt[k] = p.norm_w && in ? *reinterpret_cast<const float4*>(p.norm_w + col(k)) : zero;
+    mu[k] = p.shift && in ? *reinterpret_cast<const float4*>(p.shift + col(k)) : zero;
+    yw[k] = p.y_norm_w && in ? *reinterpret_cast<const float4*>(p.y_norm_w + col(k)) : zero;
+  }
+  pdl_wait();
+  int flip = 0;
+  auto block_sum = [&](float v) -> float {       // one barrier: consecutive sums use different rows of `red`
+    v = warp_sum(v);
+    if (lane == 0) red[flip][warp] = v;
+    __syncthreads();
+    const float t = warp_sum(lane < nw ? red[flip][lane] : 0.f);
+    flip ^= 1;
+    return t;
+  };
+  float4 v[VPT], a[VPT];
+  auto load = [&](int r) {
+    const int src = p.row_idx ? p.row_idx[r] : r;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const bool in = col(k) < H;
+      v[k] = !in ? zero : p.x ? *reinterpret_cast<const float4*>(p.x + (size_t)src * H + col(k)) : load4(table + (size_t)p.ids[src] * H + col(k));
+      a[k] = y && in ? load4(y + (size_t)src * H + col(k)) : zero;
+    }
+  };
+  // v <- v + pending output; returns 1 / rms when the row is normalised
+  auto finish_row = [&]() -> float {
+    float yr = 1.f;
+    if (p.y_norm_w) {
+      float s = 0.f;
+#pragma unroll
+      for (int k = 0; k < VPT; ++k) s += sq4(a[k]);
+      yr = rsqrtf(block_sum(s) * inv_dim + p.eps);
+    }
+    float s = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      if (p.y_norm_w) {
+        a[k].x *= yr * yw[k].x; a[k].y *= yr * yw[k].y; a[k].z *= yr * yw[k].z; a[k].w *= yr * yw[k].w;
+      }
+      v[k].x += a[k].x; v[k].y += a[k].y; v[k].z += a[k].z; v[k].w += a[k].w;
+      s += sq4(v[k]);
+    }
+    return p.norm_w ? rsqrtf(block_sum(s) * inv_dim + p.eps) : 1.f;
+  };
+  auto normed = [&](int k, float r) { return make_float4(v[k].x * r * nwt[k].x, v[k].y * r * nwt[k].y, v[k].z * r * nwt[k].z, v[k].w * r * nwt[k].w); };
+
+  float4 hp[VPT];
+  const int r0 = blockIdx.x * rows_per_cta, r1 = min(p.n_rows, r0 + rows_per_cta);
+  for (int r = r0; r < r1; ++r) {
+    float* state = nullptr;
+    bool state_here = false, fresh = false;
+    if (p.shift) {
+      const int seq = p.rows.seq_of_row ? p.rows.seq_of_row[r] : r;
+      const int q0 = p.rows.q_start ? p.rows.q_start[seq] : r;
+      if (r == q0) {
+        const int n = p.rows.q_len ? p.rows.q_len[seq] : 1;
+        state = p.shift_state + (size_t)(p.rows.slot ? p.rows.slot[seq] : seq) * H;
+        fresh = p.rows.pos[r] == 0;
+#pragma unroll
+        for (int k = 0; k < VPT; ++k) hp[k] = col(k) < H ? *reinterpret_cast<const float4*>(state + col(k)) : zero;
+        if (n > 1) {                             // the carried row is replaced by the last row's, normalised here a second time
+          load(r + n - 1);
+          const float rl = finish_row();
+#pragma unroll
+          for (int k = 0; k < VPT; ++k)
+            if (col(k) < H) *reinterpret_cast<float4*>(state + col(k)) = normed(k, rl);
+        } else {
+          state_here = true;
+        }
+      } else if (r == r0) {
+        load(r - 1);
+        const float rl = finish_row();
+#pragma unroll
+        for (int k = 0; k < VPT; ++k) hp[k] = normed(k, rl);
+      }
+    }
+    load(r);
+    const float rstd = finish_row();
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int c = col(k);
+      if (c >= H) continue;
+      if (p.x_out) *reinterpret_cast<float4*>(p.x_out + (size_t)r * H + c) = v[k];
+      if (p.x_cast) store4(reinterpret_cast<T*>(p.x_cast) + (size_t)r * H + c, v[k]);
+      if (!p.norm_w) continue;
+      float4 h = normed(k, rstd);
+      if (p.shift) {
+        const float4 b = fresh ? zero : hp[k], m = mu[k];
+        hp[k] = h;
+        if (state_here) *reinterpret_cast<float4*>(state + c) = h;
+        h.x += (b.x - h.x) * m.x; h.y += (b.y - h.y) * m.y; h.z += (b.z - h.z) * m.z; h.w += (b.w - h.w) * m.w;
+      }
+      store4(reinterpret_cast<T*>(p.out) + (size_t)r * H + c, h);
+    }
+  }
+}
+
 template <typename T>
 __global__ void token_gate_kernel(T* __restrict__ g, int64_t ldg, const T* __restrict__ table, int64_t ldt,
                                   const int32_t* __restrict__ ids, int col0, int rows, int cols) {
@@ -209,10 +324,22 @@ extern "C" int rf_stream_norm(const RfStreamNorm* a, rf_stream_t stream) {
   if (a->n_rows == 0) return RF_OK;
   // halo of one row per CTA with the shift: walk several rows per CTA once that still fills the GPU
   const int rpc = (a->shift && a->rows.q_start) ? std::max(1, std::min(8, a->n_rows / (2 * sm_count()))) : 1;
-  const int threads = std::min(512, std::max(64, round_up(ceil_div(a->H / 4, a->H >= 4096 ? 2 : 1), 32)));
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const int quads = a->H / 4;
+  if (quads <= 2048) {
+    // decode rows: as many threads as there are quads (one round trip); many rows: smaller CTAs, several per SM
+    const int vpt = a->n_rows > 4 * sm_count() ? (quads > 512 ? 4 : quads > 256 ? 2 : 1) : (quads > 1024 ? 2 : 1);
+    const int threads = std::max(32, round_up(ceil_div(quads, vpt), 32));
+    const dim3 grid(ceil_div(a->n_rows, rpc));
+#define RF_SN(V) RF_DISPATCH3(a->dtype, RF_CUDA_CHECK(::rf::launch_k(stream_norm_reg_kernel<T, V>, grid, dim3(threads), 0, s, 1, *a, rpc)))
+    if (vpt == 1) { RF_SN(1); } else if (vpt == 2) { RF_SN(2); } else { RF_SN(4); }
+#undef RF_SN
+    ::rf::count_launch();
+    return RF_OK;
+  }
+  const int threads = 512;
   const size_t smem = ((size_t)a->H * (a->shift ? 2 : 1) + 32) * sizeof(float);
   RF_REQUIRE(smem <= 200 * 1024, "stream_norm: rows of %d values do not fit in shared memory", a->H);
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
   RF_DISPATCH3(a->dtype, {
     RF_ALLOW_SMEM_PER_DEVICE(stream_norm_kernel<T>, 200 * 1024);
     RF_CUDA_CHECK(::rf::launch_k(stream_norm_kernel<T>, dim3(ceil_div(a->n_rows, rpc)), dim3(threads), smem, s, 1, *a, rpc));

@@ -113,6 +113,8 @@ static int linear(const MixedStack& s, const void* x, int64_t ldx, const void* w
   g.w_packed = s.cfg.weights_packed;
   g.status = s.status();
   g.force_swap = -1;
+  // large weights stream through the tcgen05 kernel; the latency-bound kernel keeps the small ones (side input, latents)
+  g.streaming_only = (int64_t)N * K > (2 << 20);
   g.ws = s.at<float>(s.off_sk_ws); g.ws_bytes = s.sk_ws_bytes;
   g.sem = s.at<uint32_t>(s.off_sk_flags); g.sem_count = MixedStack::kSkFlags;
   return rf_gemm(&g, st);

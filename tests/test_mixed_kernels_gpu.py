@@ -40,7 +40,7 @@ def close(got, want, dtype, scale=1.0):
 
 # ------------------------------------------------------------------------------------------------ residual stream
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,dim", [(40, 37), (512, 512), (4104, 4099)])
+@pytest.mark.parametrize("H,dim", [(40, 37), (512, 512), (4104, 4099), (8200, 8200), (16400, 16391)])
 def test_stream_norm_adds_the_pending_output_normalises_and_shifts(dtype, H, dim):
     lens, pos0, slots = [1, 7, 2, 30], [5, 0, 9, 0], [3, 1, 0, 4]
     d, pos, seq = pack(lens, pos0, slots)
