@@ -210,7 +210,7 @@ class RfHgrn2(C.Structure):
     _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64), ("f_off", C.c_int32), ("v_off", C.c_int32), ("f_bias", C.c_void_p),
                 ("lower", C.c_void_p), ("norm_w", C.c_void_p), ("state", C.c_void_p), ("out", C.c_void_p), ("ldo", C.c_int64),
                 ("rows", RfRows)] + [(n, C.c_int32) for n in ("heads", "dim", "vdim", "vdim_true")] + \
-               [("eps", C.c_float), ("dtype", C.c_int32)]
+               [("eps", C.c_float), ("dtype", C.c_int32), ("status", C.c_void_p)]
 
 
 class RfMixedConfig(C.Structure):

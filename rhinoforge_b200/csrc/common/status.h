@@ -34,6 +34,7 @@ enum KernelTag : int32_t {
   kTagBarrier = 5,
   kTagMoe = 6,
   kTagW8A16 = 7,
+  kTagHgrn2 = 8,
 };
 
 }  // namespace rf

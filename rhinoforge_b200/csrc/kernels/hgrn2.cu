@@ -7,6 +7,7 @@
 #include "../common/host_util.h"
 #include "../common/mma.cuh"
 #include "../common/ptx.cuh"
+#include "../common/status.h"
 #include "../rf_api.h"
 
 namespace rf {
@@ -145,6 +146,168 @@ static int launch_recurrent(const RfHgrn2* a, cudaStream_t s) {
     default: RF_HG(0); break;
   }
 #undef RF_HG
+  ::rf::count_launch();
+  return RF_OK;
+}
+
+// ------------------------------------------------------- one token per sequence ----
+// A decode step reads and writes every state once, so it is a copy with a little arithmetic.  Persistent CTAs walk over the
+// (sequence, head) states: a ring of three shared-memory buffers keeps bulk loads of the next states and the bulk store of the
+// last one in flight while one is updated in place; the row of a state's token is fetched one state ahead.
+constexpr int kHdThreads = 512, kHdRing = 3;
+
+struct Hgrn2DecodeGeom {
+  int quads, groups;                     // 4-column groups per state row, rows updated side by side
+  uint32_t bytes, sq, sf, red, wsum, bar, total;
+};
+__host__ __device__ inline Hgrn2DecodeGeom hgrn2_decode_geom(int dim, int vdim) {
+  Hgrn2DecodeGeom g;
+  g.quads = vdim / 4;
+  g.groups = kHdThreads / g.quads;
+  g.bytes = (uint32_t)dim * vdim * 4;
+  uint32_t o = kHdRing * g.bytes;
+  g.sq = o; o += dim * 4;
+  g.sf = o; o += dim * 4;
+  g.red = o; o += g.groups * vdim * 4;
+  g.wsum = o; o += 32 * 4;
+  o = (o + 15) & ~15u;
+  g.bar = o; o += kHdRing * 8;
+  g.total = o;
+  return g;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kHdThreads) hgrn2_decode_kernel(const RfHgrn2 p) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(128) uint8_t dsm[];
+  const Hgrn2DecodeGeom G = hgrn2_decode_geom(p.dim, p.vdim);
+  float* sq = reinterpret_cast<float*>(dsm + G.sq);
+  float* sf = reinterpret_cast<float*>(dsm + G.sf);
+  float* red = reinterpret_cast<float*>(dsm + G.red);
+  float* wsum = reinterpret_cast<float*>(dsm + G.wsum);
+  uint64_t* full = reinterpret_cast<uint64_t*>(dsm + G.bar);
+  const int tid = threadIdx.x, items = p.rows.num_seqs * p.heads, step = gridDim.x;
+  const int quad = tid % G.quads, rg = tid / G.quads;      // rg >= groups: no state rows
+  const T* x = reinterpret_cast<const T*>(p.x);
+  T* out = reinterpret_cast<T*>(p.out);
+  const size_t per_head = (size_t)p.dim * p.vdim;
+  auto state_of = [&](int item) {
+    const int seq = item / p.heads, slot = p.rows.slot ? p.rows.slot[seq] : seq;
+    return p.state + ((size_t)slot * p.heads + item % p.heads) * per_head;
+  };
+  if (tid == 0) {
+    for (int s = 0; s < kHdRing; ++s) mbar_init(&full[s], 1);
+    fence_barrier_init();
+  }
+  __syncthreads();
+  pdl_wait();
+  int loaded = 0;                        // thread 0: states whose load was issued
+  auto load_state = [&](int item, int stage) {
+    mbar_arrive_expect_tx(&full[stage], G.bytes);
+    bulk_load_1d(dsm + stage * G.bytes, state_of(item), G.bytes, &full[stage]);
+    ++loaded;
+  };
+  if (tid == 0) {
+    if (blockIdx.x < items) load_state(blockIdx.x, 0);
+    if (blockIdx.x + step < items) load_state(blockIdx.x + step, 1);
+  }
+  // the token row of one state: this thread's channel of q and f, its four values, and whether the sequence starts here
+  float rq = 0.f, rf = 0.f, lo = 1.f, fb = 0.f;
+  float4 rv = make_float4(0.f, 0.f, 0.f, 0.f);
+  bool fresh = false;
+  auto fetch = [&](int item) {
+    const int seq = item / p.heads, head = item % p.heads;
+    const T* xr = x + (size_t)seq * p.ldx;
+    if (tid < p.dim) {
+      const int ch = head * p.dim + tid;
+      rq = Num<T>::to_f(xr[ch]);
+      rf = Num<T>::to_f(xr[p.f_off + ch]);
+      lo = p.lower[ch];
+      fb = p.f_bias[ch];
+    }
+    const T* vr = xr + p.v_off + head * p.vdim + quad * 4;
+    rv = make_float4(Num<T>::to_f(vr[0]), Num<T>::to_f(vr[1]), Num<T>::to_f(vr[2]), Num<T>::to_f(vr[3]));
+    fresh = p.rows.pos[seq] == 0;
+  };
+  if (blockIdx.x < items) fetch(blockIdx.x);
+
+  bool ok = true;
+  for (int item = blockIdx.x, it = 0; item < items; item += step, ++it) {
+    const int stage = it % kHdRing;
+    if (tid < p.dim) {
+      sq[tid] = rq * sigmoid_t<T>(rq);
+      sf[tid] = lo + (1.f - lo) * sigmoid_t<T>(rf + fb);
+    }
+    const float4 v = rv;
+    const bool start = fresh;
+    if (item + step < items) fetch(item + step);
+    const bool have = mbar_wait(&full[stage], (uint32_t)(it / kHdRing) & 1u);
+    if (__syncthreads_or(!have)) {
+      ok = false;
+      if (tid == 0) report_status(p.status, kStatusTmaTimeout, kTagHgrn2, item);
+      break;
+    }
+    float4 part = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (rg < G.groups) {
+      float4* S = reinterpret_cast<float4*>(dsm + stage * G.bytes) + quad;
+#pragma unroll 4
+      for (int r = rg; r < p.dim; r += G.groups) {
+        const float f = sf[r], w = 1.f - f, q = sq[r];
+        float4 s = S[(size_t)r * G.quads];
+        if (start) s = make_float4(0.f, 0.f, 0.f, 0.f);
+        s.x = f * s.x + w * v.x; s.y = f * s.y + w * v.y; s.z = f * s.z + w * v.z; s.w = f * s.w + w * v.w;
+        S[(size_t)r * G.quads] = s;
+        part.x = fmaf(s.x, q, part.x); part.y = fmaf(s.y, q, part.y); part.z = fmaf(s.z, q, part.z); part.w = fmaf(s.w, q, part.w);
+      }
+      *reinterpret_cast<float4*>(red + rg * p.vdim + quad * 4) = part;
+    }
+    fence_proxy_async();
+    __syncthreads();
+    if (tid == 0) {
+      bulk_store_1d(state_of(item), dsm + stage * G.bytes, G.bytes);
+      bulk_commit_group();
+      if (item + 2 * step < items) {
+        bulk_wait_read_1();              // the store before this one has left its buffer
+        load_state(item + 2 * step, (it + 2) % kHdRing);
+      }
+    }
+    const int seq = item / p.heads, head = item % p.heads;
+    float o = 0.f;
+    if (tid < p.vdim)
+      for (int g = 0; g < G.groups; ++g) o += red[g * p.vdim + tid];
+    const float ss = warp_sum(o * o);
+    if ((tid & 31) == 0) wsum[tid >> 5] = ss;
+    __syncthreads();
+    if (tid < p.vdim) {
+      float r = 1.f;
+      if (p.norm_w) {
+        float tot = 0.f;
+        for (int w = 0; w < (p.vdim + 31) / 32; ++w) tot += wsum[w];
+        r = rsqrtf(tot / (float)p.vdim_true + p.eps) * p.norm_w[tid];
+      }
+      out[(size_t)seq * p.ldo + head * p.vdim + tid] = Num<T>::from_f(o * r);
+    }
+  }
+  if (tid == 0) {
+    if (!ok) {                           // let every load that was issued land before the CTA exits
+      for (int s = max(0, loaded - kHdRing); s < loaded; ++s) mbar_wait(&full[s % kHdRing], (uint32_t)(s / kHdRing) & 1u, 20ull * 1000 * 1000);
+    }
+    bulk_wait_all();
+  }
+}
+
+static bool hgrn2_decode_eligible(const RfHgrn2* a) {
+  return !a->rows.q_start && a->dim <= kHdThreads && a->vdim <= kHdThreads && a->vdim % 4 == 0 &&
+         hgrn2_decode_geom(a->dim, a->vdim).total <= 220 * 1024;
+}
+
+template <typename T>
+static int launch_decode(const RfHgrn2* a, cudaStream_t s) {
+  const Hgrn2DecodeGeom g = hgrn2_decode_geom(a->dim, a->vdim);
+  RF_ALLOW_SMEM_PER_DEVICE(hgrn2_decode_kernel<T>, 220 * 1024);
+  const int per_sm = std::max(1, std::min(4, (int)(227 * 1024 / (g.total + 1024))));
+  const int grid = std::min(a->rows.num_seqs * a->heads, per_sm * sm_count());
+  RF_CUDA_CHECK(::rf::launch_k(hgrn2_decode_kernel<T>, dim3(grid), dim3(kHdThreads), g.total, s, 1, *a));
   ::rf::count_launch();
   return RF_OK;
 }
@@ -496,6 +659,11 @@ extern "C" int rf_hgrn2_recurrent(const RfHgrn2* a, rf_stream_t stream) {
   if (rc) return rc;
   if (a->rows.num_seqs == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (hgrn2_decode_eligible(a)) {
+    if (a->dtype == kF32) return launch_decode<float>(a, s);
+    if (a->dtype == kF16) return launch_decode<__half>(a, s);
+    return launch_decode<__nv_bfloat16>(a, s);
+  }
   if (a->dtype == kF32) return launch_recurrent<float>(a, s);
   if (a->dtype == kF16) return launch_recurrent<__half>(a, s);
   return launch_recurrent<__nv_bfloat16>(a, s);

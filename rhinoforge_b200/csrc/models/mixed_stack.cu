@@ -238,6 +238,7 @@ static int hgrn2(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f, 
   a.f_bias = w.f_bias; a.lower = w.lower; a.norm_w = w.head_norm;
   a.state = w.rec_state; a.out = mix; a.ldo = (int64_t)w.heads * w.vdim;
   a.heads = w.heads; a.dim = w.dim; a.vdim = w.vdim; a.vdim_true = w.vdim_true; a.eps = c.eps; a.dtype = c.dtype;
+  a.status = s.status();
   const bool chunked = rf_hgrn2_chunked_supported(w.dim, w.vdim, c.dtype) != 0;
   const int n_rec = chunked ? f.short_seqs : f.rows.num_seqs;
   if (n_rec > 0) {

@@ -373,6 +373,7 @@ typedef struct RfHgrn2 {
   float* state; void* out; int64_t ldo;
   RfRows rows;
   int32_t heads, dim, vdim, vdim_true; float eps; int32_t dtype;
+  int32_t* status;                     // device status block, optional
 } RfHgrn2;
 int rf_hgrn2_recurrent(const RfHgrn2* a, rf_stream_t stream);
 // Same contract, evaluated block by block (prefill-sized portions; 16-bit activations).

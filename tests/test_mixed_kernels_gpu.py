@@ -254,3 +254,32 @@ def test_hgrn2_keeps_a_value_written_long_ago():
                 outs.append(K().hgrn2(x[a:a + L].contiguous(), fb, lower, None, state, K().rows(**d), eps=1e-6, chunked=chunked))
             o = torch.cat(outs)[n - 1].float()
             assert abs(float(o[9]) - 3.0 * 8.0) < 0.2 and float(o.abs().sum() - o[9].abs()) < 0.05, (chunked, cut)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("batch,heads,D,VD,vdim", [(1, 1, 8, 8, 8), (3, 2, 48, 64, 61), (70, 8, 128, 128, 128), (5, 3, 40, 24, 24), (2, 2, 264, 160, 160),
+                                                   (300, 3, 16, 32, 32)])
+def test_hgrn2_decode_step_of_many_sequences(dtype, batch, heads, D, VD, vdim):
+    """One token per sequence, several steps in a row: more states than resident CTAs, scattered slots, fresh sequences."""
+    g = torch.Generator().manual_seed(batch)
+    width = heads * (2 * D + VD)
+    fb, lower = torch.randn(heads * D, generator=g).cuda(), torch.rand(heads * D, generator=g).cuda()
+    nw = torch.nn.functional.pad(torch.randn(vdim, generator=g), (0, VD - vdim)).cuda()
+    state = torch.randn(batch + 2, heads, D, VD, generator=g)
+    state[..., vdim:] = 0.0
+    state[1] = float("nan")                                     # left behind by someone; the sequence in it starts afresh
+    state = state.cuda()
+    slots = [(i + 1) % (batch + 2) for i in range(batch)]
+    pos = [0 if i % 3 == 0 else 7 + i for i in range(batch)]
+    untouched = state[0].clone()
+    for step in range(2):
+        x = torch.randn(batch, width, generator=g)
+        x[:, 2 * heads * D:].view(batch, heads, VD)[..., vdim:] = 0.0
+        x = x.to("cuda", dtype)
+        start = torch.nan_to_num(state)
+        want, want_state = hgrn2_reference(x, fb, lower, nw, start, [1] * batch, pos, slots, heads, D, VD, 1e-5, vdim)
+        got = K().hgrn2(x, fb, lower, nw, state, K().rows(i32(*pos), slot=i32(*slots)), eps=1e-5, vdim=vdim)
+        close(got, want, dtype, 4)
+        torch.testing.assert_close(state.double().cpu()[1:], want_state[1:], rtol=1e-4, atol=1e-4)
+        pos = [p + 1 for p in pos]
+    assert torch.equal(state[0], untouched)
