@@ -46,6 +46,7 @@ class RfGemm(C.Structure):
         ("w_bits", C.c_int32), ("w_group", C.c_int32), ("w_fp4", C.c_int32), ("ss_tiles", C.c_int32),
         ("ss_out", C.c_void_p), ("ss_in", C.c_void_p), ("ss_ld", C.c_int32), ("ss_dim", C.c_int32),
         ("ss_eps", C.c_float), ("streaming_only", C.c_int32),
+        ("mul", C.c_void_p), ("mul_row", C.c_void_p), ("mul_ld", C.c_int64),
     ]
 
 

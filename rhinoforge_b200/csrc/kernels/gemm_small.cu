@@ -36,6 +36,7 @@ struct SmallParams {
   const void* residual; int64_t ldr;
   const void* bias;
   const void* scale;          // optional per-output-column factor, applied before the bias (16-bit weights only)
+  const void* mul; const int32_t* mul_row; int64_t mul_ld;   // optional gate: result *= mul[mul_row[m] * mul_ld + n]
   int M, N, K, act, dual_offset, packed, kb_total, dual_tiles, splits;
 };
 
@@ -224,6 +225,11 @@ gemm_small_kernel(const SmallParams p) {
       }
     }
     float v0 = apply_act(p.act, g0, u0), v1 = apply_act(p.act, g1, u1);
+    if (p.mul) {
+      const T* e = reinterpret_cast<const T*>(p.mul) + (size_t)p.mul_row[m] * p.mul_ld + n;
+      v0 *= Num<T>::to_f(e[0]);
+      v1 *= Num<T>::to_f(e[1]);
+    }
     if (res) {
       v0 += Num<T>::to_f(res[(size_t)m * p.ldr + n]);
       v1 += Num<T>::to_f(res[(size_t)m * p.ldr + n + 1]);
@@ -361,6 +367,7 @@ int gemm_small_run(const RfGemm* g, cudaStream_t s) {
   SmallParams p;
   p.x = g->x; p.ldx = g->ldx; p.w = g->w; p.ldw = g->ldw; p.out = g->out; p.ldo = g->ldo;
   p.residual = g->residual; p.ldr = g->ldr; p.bias = g->bias; p.scale = g->scale;
+  p.mul = g->mul; p.mul_row = g->mul_row; p.mul_ld = g->mul_ld;
   p.M = g->M; p.N = g->N; p.K = g->K; p.act = g->act; p.dual_offset = g->dual_offset; p.packed = g->w_packed ? 1 : 0;
   p.kb_total = (g->K + 63) / 64;
   p.dual_tiles = dual ? (g->dual_offset + 127) / 128 : 0;    // the up section starts this many 128-row tiles after the gate section

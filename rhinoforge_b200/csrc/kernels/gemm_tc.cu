@@ -1353,6 +1353,7 @@ int widen_packed(const void* src, void* dst, int64_t blocks, int dtype, cudaStre
 static int run_gemm(const RfGemm* g, cudaStream_t stream, bool w8) {
   int rc = check_gemm(g);
   if (rc) return rc;
+  if (g->mul) RF_REQUIRE(!w8 && g->mul_row && rf::gemm_small_eligible(g), "GEMM %dx%dx%d has no gate-by-token epilogue (see rf_gemm_takes_mul)", g->M, g->N, g->K);
   if (!w8 && rf::gemm_small_eligible(g)) return rf::gemm_small_run(g, stream);      // latency-bound shapes: gemm_small.cu
   if (!w8 && rf::gemm_sk_eligible(g, nullptr)) return rf::launch_gemm_sk(g, stream);
   GemmPlan pl;
@@ -1394,6 +1395,8 @@ static int run_gemm(const RfGemm* g, cudaStream_t stream, bool w8) {
   RF_GEMM_DISPATCH(__nv_bfloat16, false)
 #undef RF_GEMM_DISPATCH
 }
+
+extern "C" int rf_gemm_takes_mul(const RfGemm* g) { return g && check_gemm(g) == RF_OK && !g->w_int8 && rf::gemm_small_eligible(g); }
 
 extern "C" int rf_gemm_plan_info(const RfGemm* g, int32_t* out) {
   RF_REQUIRE(g && out, "rf_gemm_plan_info: null argument");

@@ -15,23 +15,30 @@ __device__ __forceinline__ int row_seq(const RfRows& r, int row) { return r.seq_
 __device__ __forceinline__ int seq_slot(const RfRows& r, int seq) { return r.slot ? r.slot[seq] : seq; }
 
 // --------------------------------------------------------------- cache rows ----
+// One warp normalises one row and stores it at its position.
 template <typename T>
-__global__ void latent_insert_kernel(const T* __restrict__ x, int64_t ldx, const float* __restrict__ w, T* __restrict__ pool,
-                                     const RfRows rows, int n_rows, int rank, int rank_true, float eps) {
-  pdl_prologue();
-  const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;   // one warp per row
-  if (row >= n_rows) return;
-  const T* xr = x + (size_t)row * ldx;
+__device__ __forceinline__ void latent_insert_row(const RfLatentInsert& p, int row, int lane) {
+  const T* xr = reinterpret_cast<const T*>(p.x) + (size_t)row * p.ldx;
   float s = 0.f;
-  for (int i = lane; i < rank; i += 32) {
-    const float v = Num<T>::to_f(xr[i]);
-    s += v * v;
+  for (int i = lane * 2; i < p.rank; i += 64) {
+    const float a = Num<T>::to_f(xr[i]), b = Num<T>::to_f(xr[i + 1]);
+    s += a * a + b * b;
   }
-  const float rstd = rsqrtf(warp_sum(s) / (float)rank_true + eps);
-  const int pos = rows.pos[row];
-  const int page = rows.page_table[(size_t)seq_slot(rows, row_seq(rows, row)) * rows.pt_stride + (pos >> 4)];
-  T* dst = pool + ((size_t)page * 16 + (pos & 15)) * rank;
-  for (int i = lane; i < rank; i += 32) dst[i] = Num<T>::from_f(Num<T>::to_f(xr[i]) * rstd * w[i]);
+  const int pos = p.rows.pos[row];
+  const int page = p.rows.page_table[(size_t)seq_slot(p.rows, row_seq(p.rows, row)) * p.rows.pt_stride + (pos >> 4)];
+  const float rstd = rsqrtf(warp_sum(s) / (float)p.rank_true + p.eps);
+  T* dst = reinterpret_cast<T*>(p.pool) + ((size_t)page * 16 + (pos & 15)) * p.rank;
+  for (int i = lane * 2; i < p.rank; i += 64) {
+    dst[i] = Num<T>::from_f(Num<T>::to_f(xr[i]) * rstd * p.norm_w[i]);
+    dst[i + 1] = Num<T>::from_f(Num<T>::to_f(xr[i + 1]) * rstd * p.norm_w[i + 1]);
+  }
+}
+
+template <typename T>
+__global__ void latent_insert_kernel(const RfLatentInsert p) {
+  pdl_prologue();
+  const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (row < p.n_rows) latent_insert_row<T>(p, row, threadIdx.x & 31);
 }
 
 template <typename T>
@@ -98,8 +105,14 @@ template <int N> __device__ __forceinline__ void la_wait() { asm volatile("cp.as
 constexpr int kHmRows = 64, kHmK = 64, kHmLd = kHmK + 8, kHmStages = 4;
 
 template <typename T, int NT>
-__global__ void __launch_bounds__(128) head_linear_mma_kernel(const RfHeadLinear p) {
+__global__ void __launch_bounds__(128) head_linear_mma_kernel(const RfHeadLinear p, const RfLatentInsert ins, int row_tiles) {
   pdl_launch_dependents();
+  if ((int)blockIdx.z >= row_tiles) {    // the grid's last planes insert latent rows, one per warp
+    pdl_wait();
+    const int row = ((((int)blockIdx.z - row_tiles) * gridDim.y + blockIdx.y) * gridDim.x + blockIdx.x) * 4 + (threadIdx.x >> 5);
+    if (row < ins.n_rows) latent_insert_row<T>(ins, row, threadIdx.x & 31);
+    return;
+  }
   constexpr int BN = NT * 32;
   extern __shared__ __align__(16) uint8_t hsm[];
   constexpr uint32_t kXBytes = kHmRows * kHmLd * 2, kStage = kXBytes + BN * kHmLd * 2;
@@ -177,13 +190,16 @@ __global__ void __launch_bounds__(128) head_linear_mma_kernel(const RfHeadLinear
 }
 
 template <typename T>
-static int launch_head_linear_mma(const RfHeadLinear* a, cudaStream_t s) {
+static int launch_head_linear_mma(const RfHeadLinear* a, const RfLatentInsert* c, cudaStream_t s) {
   const int rt = ceil_div(a->rows, kHmRows);
+  const RfLatentInsert ins = c ? *c : RfLatentInsert{};
 #define RF_HM(NT)                                                                                                            \
   do {                                                                                                                       \
     constexpr size_t smem = (size_t)kHmStages * (kHmRows + NT * 32) * kHmLd * 2;                                              \
+    const int gx = ceil_div(a->n, NT * 32);                                                                                  \
+    const dim3 grid(gx, a->heads, rt + ceil_div(ceil_div(ins.n_rows, 4), gx * a->heads));                                    \
     RF_ALLOW_SMEM_PER_DEVICE((head_linear_mma_kernel<T, NT>), smem);                                                         \
-    RF_CUDA_CHECK(::rf::launch_k(head_linear_mma_kernel<T, NT>, dim3(ceil_div(a->n, NT * 32), a->heads, rt), dim3(128), smem, s, 1, *a)); \
+    RF_CUDA_CHECK(::rf::launch_k(head_linear_mma_kernel<T, NT>, grid, dim3(128), smem, s, 1, *a, ins, rt)); \
   } while (0)
   if ((long)ceil_div(a->n, 64) * a->heads * rt < sm_count()) RF_HM(1);
   else RF_HM(2);
@@ -500,10 +516,10 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentSplit s
   }
 }
 
-// Split the keys of a row until about one CTA per SM exists; at least two key blocks per split.
+// Split the keys of a row until about one CTA per SM exists.
 static int la_splits(int rows, int heads, int max_kv) {
   const int mt = heads <= 16 ? 1 : 2, ctas = rows * ceil_div(heads, 16 * mt), blocks = ceil_div(std::max(max_kv, 1), kLaKeys);
-  return std::max(1, std::min(std::min(sm_count() / std::max(ctas, 1), blocks / 2), 64));
+  return std::max(1, std::min(std::min(sm_count() / std::max(ctas, 1), blocks), 64));
 }
 
 }  // namespace rf
@@ -520,16 +536,22 @@ static int check_rows(const RfRows* r) {
   return RF_OK;
 }
 
+static int check_insert(const RfLatentInsert* c) {
+  RF_REQUIRE(c && c->x && c->norm_w && c->pool && c->rank > 0 && c->rank % 16 == 0 && c->rank_true > 0 && c->rank_true <= c->rank,
+             "latent_insert arguments");
+  return check_rows(&c->rows);
+}
+
 extern "C" int rf_latent_insert(const void* x, int64_t ldx, const float* norm_w, void* pool, const RfRows* rows, int32_t n_rows,
                                 int32_t rank, int32_t rank_true, float eps, int32_t dtype, rf_stream_t stream) {
   RF_SKIP_IF_REPLAYING();
-  RF_REQUIRE(x && norm_w && pool && rank > 0 && rank % 16 == 0 && rank_true > 0 && rank_true <= rank, "latent_insert arguments");
-  int rc = check_rows(rows);
+  RF_REQUIRE(rows, "latent_insert: no rows");
+  const RfLatentInsert c = {x, ldx, norm_w, pool, *rows, n_rows, rank, rank_true, eps};
+  int rc = check_insert(&c);
   if (rc) return rc;
   if (n_rows == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  RF_DISPATCH3(dtype, RF_CUDA_CHECK(::rf::launch_k(latent_insert_kernel<T>, dim3(ceil_div(n_rows, 4)), dim3(128), 0, s, 1,
-                                                   (const T*)x, ldx, norm_w, (T*)pool, *rows, n_rows, rank, rank_true, eps)));
+  RF_DISPATCH3(dtype, RF_CUDA_CHECK(::rf::launch_k(latent_insert_kernel<T>, dim3(ceil_div(n_rows, 4)), dim3(128), 0, s, 1, c)));
   ::rf::count_launch();
   return RF_OK;
 }
@@ -549,19 +571,40 @@ extern "C" int rf_latent_gather(const void* pool, void* out, const RfRows* rows,
   return RF_OK;
 }
 
-extern "C" int rf_head_linear(const RfHeadLinear* a, rf_stream_t stream) {
-  RF_SKIP_IF_REPLAYING();
+static int check_head_linear(const RfHeadLinear* a) {
   RF_REQUIRE(a && a->x && a->y && a->w && a->heads > 0 && a->n > 0 && a->k > 0, "head_linear arguments");
   RF_REQUIRE(a->n % 8 == 0 && a->k % 8 == 0 && a->xs % 8 == 0 && a->ys % 8 == 0 && a->ldx % 8 == 0 && a->ldy % 8 == 0,
              "head_linear: sizes and pitches must be multiples of 8");
+  return RF_OK;
+}
+
+extern "C" int rf_head_linear(const RfHeadLinear* a, rf_stream_t stream) {
+  RF_SKIP_IF_REPLAYING();
+  int rc = check_head_linear(a);
+  if (rc) return rc;
   if (a->rows == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (a->dtype == kF16) return launch_head_linear_mma<__half>(a, s);
-  if (a->dtype == kBF16) return launch_head_linear_mma<__nv_bfloat16>(a, s);
+  if (a->dtype == kF16) return launch_head_linear_mma<__half>(a, nullptr, s);
+  if (a->dtype == kBF16) return launch_head_linear_mma<__nv_bfloat16>(a, nullptr, s);
   RF_DISPATCH3(a->dtype, RF_CUDA_CHECK(::rf::launch_k(head_linear_kernel<T>, dim3(ceil_div(a->n, kHlN), a->heads, ceil_div(a->rows, kHlRows)),
                                                       dim3(128), 0, s, 1, *a)));
   ::rf::count_launch();
   return RF_OK;
+}
+
+extern "C" int rf_latent_absorb(const RfHeadLinear* q, const RfLatentInsert* c, rf_stream_t stream) {
+  RF_SKIP_IF_REPLAYING();
+  int rc = check_insert(c);
+  if (rc) return rc;
+  RF_REQUIRE(q != nullptr, "latent_absorb: no queries");
+  if (q->dtype == kF32 || q->rows == 0) {
+    rc = rf_latent_insert(c->x, c->ldx, c->norm_w, c->pool, &c->rows, c->n_rows, c->rank, c->rank_true, c->eps, q->dtype, stream);
+    return rc ? rc : rf_head_linear(q, stream);
+  }
+  rc = check_head_linear(q);
+  if (rc) return rc;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return q->dtype == kF16 ? launch_head_linear_mma<__half>(q, c, s) : launch_head_linear_mma<__nv_bfloat16>(q, c, s);
 }
 
 // Room for the largest split of any launch of at most `rows` rows.

@@ -104,12 +104,11 @@ static HandleRegistry<MixedStack>& registry() {
 }
 
 // out[M, N] = act(x[M, K] . w[N, K]^T): the tcgen05 GEMMs for 16-bit stacks, the fp32 GEMM for 32-bit ones.
-static int linear(const MixedStack& s, const void* x, int64_t ldx, const void* w, void* out, int64_t ldo, int M, int N, int K,
-                  int act, cudaStream_t st) {
+static RfGemm gemm_args(const MixedStack& s, const void* x, int64_t ldx, const void* w, void* out, int64_t ldo, int M, int N, int K, int act) {
   RfGemm g = {};
   g.x = x; g.ldx = ldx; g.w = w; g.ldw = K; g.out = out; g.ldo = ldo;
   g.M = M; g.N = N; g.K = K; g.dtype = s.cfg.dtype; g.act = act;
-  if (s.fp32()) return rf_gemm_f32(&g, st);
+  if (s.fp32()) return g;
   g.w_packed = s.cfg.weights_packed;
   g.status = s.status();
   g.force_swap = -1;
@@ -117,7 +116,27 @@ static int linear(const MixedStack& s, const void* x, int64_t ldx, const void* w
   g.streaming_only = (int64_t)N * K > (2 << 20);
   g.ws = s.at<float>(s.off_sk_ws); g.ws_bytes = s.sk_ws_bytes;
   g.sem = s.at<uint32_t>(s.off_sk_flags); g.sem_count = MixedStack::kSkFlags;
-  return rf_gemm(&g, st);
+  return g;
+}
+
+static int linear(const MixedStack& s, const void* x, int64_t ldx, const void* w, void* out, int64_t ldo, int M, int N, int K,
+                  int act, cudaStream_t st) {
+  const RfGemm g = gemm_args(s, x, ldx, w, out, ldo, M, N, K, act);
+  return s.fp32() ? rf_gemm_f32(&g, st) : rf_gemm(&g, st);
+}
+
+// gelu(W_gate x) times this layer's slice of the tokens' side rows: in the GEMM's epilogue where it has one for that
+static int side_gate(const MixedStack& s, const void* x, const RfMixedLayer& w, const int32_t* ids, int layer, void* out, int T, cudaStream_t st) {
+  const RfMixedConfig& c = s.cfg;
+  const int P = c.side_dim;
+  RfGemm g = gemm_args(s, x, c.hidden, w.side_gate, out, P, T, P, c.hidden, kActGeluTanh);
+  if (!s.fp32() && rf_gemm_takes_mul(&g)) {
+    g.mul = (const uint8_t*)c.side_table + (size_t)layer * P * s.esz(); g.mul_row = ids; g.mul_ld = c.side_ld;
+    return rf_gemm(&g, st);
+  }
+  int rc = s.fp32() ? rf_gemm_f32(&g, st) : rf_gemm(&g, st);
+  if (rc) return rc;
+  return rf_token_gate(out, P, c.side_table, c.side_ld, ids, layer * P, T, P, c.dtype, st);
 }
 
 // Rows and sequences from `seq0` / `row0` on: the same launch description for a part of the batch.
@@ -137,18 +156,21 @@ static int latent_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedF
   uint8_t* wide = s.at<uint8_t>(s.off_wide);
   int rc = linear(s, h, H, w.w_in, wide, w.in_dim, T, w.in_dim, H, kActNone, st);
   if (rc) return rc;
-  rc = rf_latent_insert(wide + (size_t)QD * e, w.in_dim, w.latent_norm, w.latent_pool, &f.rows, T, w.rank, w.rank_true, c.eps, c.dtype, st);
-  if (rc) return rc;
+  RfLatentInsert ins = {wide + (size_t)QD * e, w.in_dim, w.latent_norm, w.latent_pool, f.rows, T, w.rank, w.rank_true, c.eps};
   // ---- decode rows and short portions (and everything without an expanded form): in the latent space
   const bool expand = w.expand_hd > 0 && f.short_seqs < f.rows.num_seqs;
   const int lat_total = expand ? f.short_rows : T;
+  if (lat_total == 0) {
+    rc = rf_latent_insert(ins.x, ins.ldx, ins.norm_w, ins.pool, &ins.rows, T, w.rank, w.rank_true, c.eps, c.dtype, st);
+    if (rc) return rc;
+  }
   for (int r0 = 0; r0 < lat_total; r0 += s.lat_rows) {
     const int n = std::min(s.lat_rows, lat_total - r0);
     RfHeadLinear q = {};
     q.x = wide + (size_t)r0 * w.in_dim * e; q.ldx = w.in_dim; q.xs = w.dim;
     q.y = s.at(s.off_qlat); q.ldy = (int64_t)w.heads * w.rank; q.ys = w.rank;
     q.w = w.w_absorb; q.rows = n; q.heads = w.heads; q.n = w.rank; q.k = w.dim; q.dtype = c.dtype;
-    rc = rf_head_linear(&q, st);
+    rc = r0 == 0 ? rf_latent_absorb(&q, &ins, st) : rf_head_linear(&q, st);      // every row is cached before the first attends
     if (rc) return rc;
     RfLatentAttn a = {};
     a.q = s.at(s.off_qlat); a.o = s.at(s.off_olat); a.pool = w.latent_pool;
@@ -313,9 +335,7 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
       rc = step(nullptr, nullptr, nullptr, true);
       if (rc) return rc;
       const int P = c.side_dim;
-      rc = linear(s, cast, H, w.side_gate, side, P, T, P, H, kActGeluTanh, st);
-      if (rc) return rc;
-      rc = rf_token_gate(side, P, c.side_table, c.side_ld, f.ids, l * P, T, P, c.dtype, st);
+      rc = side_gate(s, cast, w, f.ids, l, side, T, st);
       if (rc) return rc;
       rc = linear(s, side, P, w.side_proj, y, H, T, H, P, kActNone, st);
       if (rc) return rc;

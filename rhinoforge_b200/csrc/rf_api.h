@@ -96,6 +96,9 @@ typedef struct RfGemm {
   int32_t ss_ld, ss_dim;
   float ss_eps;
   int32_t streaming_only;      // 1: never the latency-bound mma.sync kernel (gemm_small.cu), whatever the shape
+  // Gate by token (shapes for which rf_gemm_takes_mul returns 1): the activated result of row m, column n is multiplied by
+  // mul[mul_row[m] * mul_ld + n] (same dtype), a slice of an embedding table.
+  const void* mul; const int32_t* mul_row; int64_t mul_ld;
 } RfGemm;
 // bytes of the tile-major image of a [rows, K] weight with `sections` equal row sections
 uint64_t rf_pack_weight_bytes(int64_t rows, int64_t K, int32_t sections, int32_t elem_bytes);
@@ -104,6 +107,7 @@ uint64_t rf_pack_w4_bytes(int64_t rows, int64_t K, int32_t sections, int32_t gro
 int32_t rf_w4_block_bytes(int32_t group);
 
 int rf_gemm(const RfGemm* g, rf_stream_t stream);
+int rf_gemm_takes_mul(const RfGemm* g);   // host-only: can this GEMM apply RfGemm.mul in its epilogue?
 // Launch plan of a shape without launching: out[10] = {swap, bn, splits, stages, grid_x, grid_y, smem bytes, k_blocks,
 // persistent kernel, two-shot all-reduce}.  Host-only.
 int rf_gemm_plan_info(const RfGemm* g, int32_t* out);
@@ -346,6 +350,13 @@ int rf_head_linear(const RfHeadLinear* a, rf_stream_t stream);
 // rf_latent_insert: c = x / rms(x) * norm_w (mean over the true rank), stored at the row's position.
 int rf_latent_insert(const void* x, int64_t ldx, const float* norm_w, void* pool, const RfRows* rows, int32_t n_rows,
                      int32_t rank, int32_t rank_true, float eps, int32_t dtype, rf_stream_t stream);
+// The insertion above together with the per-head map of the queries into the latent space (one launch in 16 bits): what a
+// decode step does between the input projection and the attention.
+typedef struct RfLatentInsert {
+  const void* x; int64_t ldx; const float* norm_w; void* pool; RfRows rows;
+  int32_t n_rows, rank, rank_true; float eps;
+} RfLatentInsert;
+int rf_latent_absorb(const RfHeadLinear* q, const RfLatentInsert* c, rf_stream_t stream);
 // Dense copies of the latents that sequences can see: the last kv_len[s] cached rows of sequence s, its own new rows (already
 // inserted) included, to rows [kv_start[s], kv_start[s] + kv_len[s]) of out.  max_len: host bound of kv_len.
 int rf_latent_gather(const void* pool, void* out, const RfRows* rows, const int32_t* kv_start, const int32_t* kv_len, int32_t rank,

@@ -84,7 +84,8 @@ def gemm(x: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
          publish: bool = False, norm_w: Optional[torch.Tensor] = None, norm_out: Optional[torch.Tensor] = None,
          norm_eps: float = 1e-6, norm_gemma: bool = False, w_bits: int = 0, w_group: int = 0,
          w_fp4: bool = False, ss_out: Optional[torch.Tensor] = None, ss_in: Optional[torch.Tensor] = None,
-         ss_dim: int = 0, ss_eps: float = 1e-6) -> torch.Tensor:
+         ss_dim: int = 0, ss_eps: float = 1e-6, mul: Optional[torch.Tensor] = None,
+         mul_row: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``out = epilogue(x @ w.T)`` on the tcgen05 kernel (or the CUDA-core GEMV).
 
     ``dual=True``: ``w`` stacks ``[gate; up]`` (2N rows) and ``act`` is a ``*_mul``
@@ -103,6 +104,7 @@ def gemm(x: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
     output values per 128-column tile and token.  ``ss_in`` (the ``ss_out`` of the GEMM that produced ``x``): the result
     is scaled per token by ``rsqrt(sum(ss_in[:, token]) / ss_dim + ss_eps)``: an RMSNorm of ``x`` whose weights were
     multiplied into the columns of ``w`` beforehand.
+    ``mul`` / ``mul_row`` (few rows, small weights): row ``m`` of the activated result is multiplied by ``mul[mul_row[m], :N]``.
     """
     M, K = x.shape
     if packed_shape is not None:          # ``w`` is the tile-major image made by pack_weight(); (rows, K) is its logical shape
@@ -143,6 +145,8 @@ def gemm(x: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
     if ss_in is not None:
         g.ss_in, g.ss_tiles, g.ss_dim, g.ss_eps = ss_in.data_ptr(), ss_in.shape[0], ss_dim or K, ss_eps
     g.force_splits, g.force_swap, g.force_bn = force_splits, force_swap, force_bn
+    if mul is not None:
+        g.mul, g.mul_row, g.mul_ld = mul.data_ptr(), _i32(mul_row), mul.stride(0)
     if w_scratch is not None:
         g.w_scratch, g.w_scratch_bytes = w_scratch.data_ptr(), w_scratch.numel() * w_scratch.element_size()
     lib = N.lib()

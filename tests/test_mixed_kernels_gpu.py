@@ -283,3 +283,13 @@ def test_hgrn2_decode_step_of_many_sequences(dtype, batch, heads, D, VD, vdim):
         torch.testing.assert_close(state.double().cpu()[1:], want_state[1:], rtol=1e-4, atol=1e-4)
         pos = [p + 1 for p in pos]
     assert torch.equal(state[0], untouched)
+
+
+@pytest.mark.parametrize("M,N,Kd", [(1, 16, 64), (5, 128, 2048), (64, 256, 1024), (200, 64, 320)])
+def test_gemm_epilogue_gates_by_token(M, N, Kd):
+    g = torch.Generator().manual_seed(M)
+    x, w = torch.randn(M, Kd, generator=g).cuda().bfloat16(), (torch.randn(N, Kd, generator=g) / Kd ** 0.5).cuda().bfloat16()
+    table = torch.randn(9, N + 24, generator=g).cuda().bfloat16()
+    ids = torch.randint(0, 9, (M,), generator=g).to("cuda", torch.int32)
+    got = K().gemm(x, K().pack_weight(w), packed_shape=(N, Kd), act="gelu_tanh", mul=table[:, 8:], mul_row=ids)
+    close(got, oracle.gelu_tanh(x.double() @ w.double().T) * table.double()[ids.long(), 8:8 + N], torch.bfloat16)

@@ -73,11 +73,13 @@ def check(got, want, dtype, what="", loose=False):
     so in 16 bits single positions may differ more."""
     got, want = got.double().cpu(), want.double()
     err = (got - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
-    limit = 5e-5 if dtype == F32 else 4e-2
     if loose and dtype != F32:
-        assert float(err.quantile(0.95)) < limit and float(err.max()) < 1.0, what
+        assert float(err.quantile(0.95)) < 4e-2 and float(err.max()) < 1.0, what
         return
-    assert float(err.max()) < limit, f"{what}: relative error {float(err.max()):.2e} at row {int(err.argmax())}"
+    most, rest = (5e-5, 5e-5) if dtype == F32 else (6e-2, 2.5e-2)      # single positions are more sensitive to rounding than most
+    assert float(err.max()) < most, f"{what}: relative error {float(err.max()):.2e} at row {int(err.argmax())}"
+    if err.numel() >= 32:
+        assert float(err.quantile(0.97)) < rest, f"{what}: 97 % of the rows within {float(err.quantile(0.97)):.2e}"
 
 
 def run(eng, toks, cuts, slot=0, decode_tail=0):
