@@ -58,7 +58,7 @@ struct MixedStack {
       heads = std::max<uint64_t>(heads, l.heads);
       if (l.expand_hd > 0) {
         kvw = std::max<uint64_t>(kvw, 2ull * l.heads * l.expand_hd);
-        past = std::max<uint64_t>(past, l.window > 0 ? std::min(l.window - 1, cfg.max_seq_len) : cfg.max_seq_len);
+        past = std::max<uint64_t>(past, l.window > 0 ? l.window - 1 : cfg.max_seq_len);
       }
     }
     windows.clear();
@@ -411,6 +411,15 @@ extern "C" int rf_mixed_set_state(int64_t h, int32_t layer, void* latent_pool, f
   if (latent_pool) s.layers[layer].latent_pool = latent_pool;
   if (rec_state) s.layers[layer].rec_state = rec_state;
   if (shift_state) s.layers[layer].shift_state = shift_state;
+  return RF_OK;
+}
+
+extern "C" int rf_mixed_set_context(int64_t h, int32_t max_seq_len) {
+  RF_GET_MIXED(h);
+  RF_REQUIRE(max_seq_len > 0, "mixed stack: context of %d tokens", max_seq_len);
+  s.cfg.max_seq_len = std::max(s.cfg.max_seq_len, max_seq_len);
+  s.planned = false;
+  s.base = nullptr;
   return RF_OK;
 }
 

@@ -71,6 +71,8 @@ int rf_mixed_destroy(int64_t h);
 int rf_mixed_set_layer(int64_t h, int32_t layer, const RfMixedLayer* w);
 // Re-point the per-layer state of a layer (binding another cache object); null keeps the pointer.
 int rf_mixed_set_state(int64_t h, int32_t layer, void* latent_pool, float* rec_state, float* shift_state);
+// Raise max_seq_len (a larger cache is bound); the arena has to be planned and bound again.
+int rf_mixed_set_context(int64_t h, int32_t max_seq_len);
 uint64_t rf_mixed_arena_bytes(int64_t h);
 int rf_mixed_bind_arena(int64_t h, void* base, uint64_t bytes);
 int32_t* rf_mixed_status_ptr(int64_t h);

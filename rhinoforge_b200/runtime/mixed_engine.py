@@ -72,15 +72,10 @@ class MixedDecoderEngine(DecoderEngine):
         self.cache = kv_cache if kv_cache is not None else MixedCache(cfg, max_batch, max_seq_len, device=self.device, dtype=dtype,
                                                                       pool_tokens=kv_pool_tokens)
         self._check_cache(self.cache)
-        lib = N.lib()
         self.handle = None
-        self._load(get_weight, max(max_seq_len, self.cache.max_seq_len))
-        nbytes = lib.rf_mixed_arena_bytes(self.handle)
-        self.arena = torch.zeros(nbytes + 1024, dtype=torch.uint8, device=self.device)
-        base = (self.arena.data_ptr() + 1023) // 1024 * 1024
-        N.check(lib.rf_mixed_bind_arena(self.handle, C.c_void_p(base), C.c_uint64(nbytes)), "rf_mixed_bind_arena")
-        off = lib.rf_mixed_status_ptr(self.handle) - self.arena.data_ptr()
-        self.status = self.arena[off:off + 32].view(torch.int32)
+        self._max_context = max(max_seq_len, self.cache.max_seq_len)
+        self._load(get_weight, self._max_context)
+        self._bind_arena()
         # ---- decode state, advanced on the device
         i32 = dict(dtype=torch.int32, device=self.device)
         self.ids, self.out_ids = torch.zeros(max_batch, **i32), torch.zeros(self.head_rows, **i32)
@@ -96,6 +91,15 @@ class MixedDecoderEngine(DecoderEngine):
         self.batch = 0
         self._hb = self._host_steps = 0
         self.heartbeat_every = 0
+
+    def _bind_arena(self) -> None:
+        lib = N.lib()
+        nbytes = lib.rf_mixed_arena_bytes(self.handle)
+        self.arena = torch.zeros(nbytes + 1024, dtype=torch.uint8, device=self.device)
+        base = (self.arena.data_ptr() + 1023) // 1024 * 1024
+        N.check(lib.rf_mixed_bind_arena(self.handle, C.c_void_p(base), C.c_uint64(nbytes)), "rf_mixed_bind_arena")
+        off = lib.rf_mixed_status_ptr(self.handle) - self.arena.data_ptr()
+        self.status = self.arena[off:off + 32].view(torch.int32)
 
     # ------------------------------------------------------------------ weights
     def _f32(self, t: torch.Tensor, n: int, fill: float = 0.0) -> torch.Tensor:
@@ -164,7 +168,8 @@ class MixedDecoderEngine(DecoderEngine):
     def _load_latent(self, lw, m: LatentAttention, g, p: str) -> None:
         H, R = self.H, pad_to(m.kv_rank, 16)
         big = max(m.dim, m.vdim)
-        hd = next((x for x in (64, 128, 256) if big <= x), 0) if not self.fp32 else 0
+        # heads of the tcgen05 prefill attention; without one (fp32, very wide heads) every row attends in the latent space
+        hd = next((x for x in (64, 128, 256) if big <= x), 0) if not self.fp32 and m.scale > 0 else 0
         D, VD = hd or pad_to(m.dim, 8), hd or pad_to(m.vdim, 8)
         lw.mixer, lw.dim, lw.vdim, lw.vdim_true = 0, D, VD, m.vdim
         lw.rank, lw.rank_true, lw.window, lw.scale, lw.expand_hd = R, m.kv_rank, m.window or 0, m.scale, hd
@@ -218,6 +223,13 @@ class MixedDecoderEngine(DecoderEngine):
         self.cache = cache
         self.graphs.clear()
         self.batch = 0
+        if cache.max_seq_len > self._max_context:
+            # attention without a window may have to expand every cached row of a portion's sequence
+            self._max_context = cache.max_seq_len
+            if any(isinstance(layer.mixer, LatentAttention) and layer.mixer.window is None for layer in self.cfg.layers):
+                torch.cuda.synchronize()
+                N.check(N.lib().rf_mixed_set_context(self.handle, self._max_context), "rf_mixed_set_context")
+                self._bind_arena()
 
     def reset(self) -> None:
         for s in range(self.cache.batch_size):

@@ -26,7 +26,7 @@ def token_shift(h, mu, previous=None):
 
 def latent_attention(h, w, p, m, eps):
     """Softmax attention whose keys and values are linear maps of one small latent row per token."""
-    n, heads, d, dv, window = h.shape[0], m["heads"], m["dim"], m["vdim"], m["mask"]["size"]
+    n, heads, d, dv, window = h.shape[0], m["heads"], m["dim"], m["vdim"], m.get("mask", {}).get("size", h.shape[0])
     q = (h @ w[p + "q"].T).view(n, heads, d)
     c = rms(h @ w[p + "dkv"].T, eps, w[p + "dkv.norm"])
     k = (c @ w[p + "uk"].T).view(n, heads, d)

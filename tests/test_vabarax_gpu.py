@@ -29,6 +29,10 @@ CONFIGS = {
     "big-heads": MixedConfig("big-heads", 120, 64, 1e-6, (
         MixedLayer(LatentAttention(2, 264, 40, 48, 0.3, 9), DenseMLP(64)),
         MixedLayer(HGRN2(2, 264, 16))), 8),
+    "linear-only": MixedConfig("linear-only", 64, 48, 1e-6, (MixedLayer(HGRN2(2, 24, 24), DenseMLP(40)), MixedLayer(HGRN2(1, 8, 96))), 8),
+    "no-window": MixedConfig("no-window", 90, 64, 1e-6, (
+        MixedLayer(LatentAttention(3, 32, 32, 48, 0.5), DenseMLP(64)),
+        MixedLayer(LatentAttention(2, 64, 16, 32, 0.4, 700))), 8),
 }
 _engines, _weights = {}, {}
 
@@ -208,6 +212,16 @@ def test_window_edges_show_in_the_logits(window, path):
             diff = float((last(other) - ref).abs().max())
             assert (diff > 1e-3) == visible, (dtype, back, diff)
         eng.close()
+
+
+def test_a_larger_cache_can_be_bound_later():
+    """Engines are built small and get their cache at the first request: attention without a window then needs more room."""
+    from rhinoforge_b200.runtime.mixed_engine import MixedDecoderEngine
+    w = weights("no-window")
+    eng = MixedDecoderEngine(CONFIGS["no-window"], lambda n: w[n], dtype=BF16, max_batch=2, max_seq_len=16, max_prefill_tokens=64)
+    eng.bind_cache(eng.make_cache(2, 320))
+    check(run(eng, tokens("no-window", 300), [64, 40, 3], slot=1), reference("no-window", 300), BF16)
+    eng.close()
 
 
 def test_checkpoint_folder_generates_through_the_public_entry_points(tmp_path):

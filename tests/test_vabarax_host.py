@@ -197,3 +197,41 @@ def test_trace_replay_writes_logits_in_entry_order(tmp_path, monkeypatch, capsys
     read = lambda n: np.fromfile(tmp_path / f"{n}.f32", dtype="<f4").reshape(-1, 3)[:, 0].tolist()
     assert read(0) == [5.0, 7.0] and not (tmp_path / "1.f32").exists() and read(2) == [8.0, 3.0]
     assert model.kw == {"batch_size": 4, "max_seq_len": 112, "pool_tokens": 112}
+
+
+def test_native_argument_blocks_have_the_same_size_on_both_sides():
+    import ctypes as C
+
+    from rhinoforge_b200 import _native as N
+    if not N.available():
+        pytest.skip("native library is not built")
+    sizes = (C.c_int32 * 8)()
+    N.lib().rf_mixed_struct_sizes(sizes)
+    ours = (N.RfMixedConfig, N.RfMixedLayer, N.RfMixedForward, N.RfRows, N.RfStreamNorm, N.RfLatentAttn, N.RfHgrn2, N.RfHeadLinear)
+    assert list(sizes) == [C.sizeof(x) for x in ours]
+
+
+def test_example_configuration_is_checked(tmp_path):
+    import importlib.util
+    from pathlib import Path
+    root = Path(__file__).resolve().parents[1]
+    spec = importlib.util.spec_from_file_location("vabarax_example", root / "examples" / "vabarax.py")
+    mod = importlib.util.module_from_spec(spec)
+    spec.loader.exec_module(mod)
+    good = (root / "examples" / "configs" / "vabarax.toml").read_text()
+    assert mod.load_config(root / "examples" / "configs" / "vabarax.toml")["generation"]["max_new_tokens"] == 16
+    for old, new in (("prompt_tokens = [[5", "prompt_tokens = [[], [5"), ("slots = 2", "slots = 0"), ('"bfloat16"', '"int8"'),
+                     ("max_new_tokens = 16", "max_new_tokens = true")):
+        assert old in good
+        f = tmp_path / "c.toml"
+        f.write_text(good.replace(old, new, 1))
+        with pytest.raises(ValueError):
+            mod.load_config(f)
+
+
+def test_weight_table_names_every_tensor_once():
+    cfg = small_config()
+    names = [n for n, _, _ in weight_shapes(cfg)]
+    assert len(names) == len(set(names))
+    assert {"embed", "side.embed", "final.norm", "l0.mix.lower", "l0.mlp.up", "l1.mix.dkv.norm", "l1.side.norm"} <= set(names)
+    assert not any(n.startswith("l1.mlp") or n == "l1.norm2" for n in names)
