@@ -263,12 +263,12 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const RfLatentAttn p) 
   }
 }
 
-// 16-bit form on the tensor cores.  One CTA (eight warps) takes MT * 16 heads of one row and a range of its keys, 64 keys per
-// step.  Scores: a warp holds a quarter of the latent columns of all its queries in registers for the whole launch and scores
-// half of the keys; the quarters are summed by the softmax, which runs row-wise over shared memory.  Output: every warp
-// accumulates NT * 8 latent columns.  The cached rows are keys and values both, so a key block is read once.  The
+// 16-bit form on the tensor cores.  One CTA (W warps) takes MT * 16 heads of one row and a range of its keys, 64 keys per
+// step.  Scores: a warp holds its share (2 / W) of the latent columns of all queries in registers for the whole launch and scores
+// half of the keys; the shares are summed by the softmax, which runs row-wise over shared memory.  Output: every warp
+// accumulates NT * 64 / W latent columns.  The cached rows are keys and values both, so a key block is read once.  The
 // probabilities enter the second product as a 16-bit pair (value + remainder), so they keep about 16 mantissa bits.
-constexpr int kLaKeys = 64, kLaThreads = 256;
+constexpr int kLaKeys = 64;
 
 struct LatentSplit {
   float* o;      // [rows, heads, splits, rank] partial outputs, unnormalised
@@ -277,19 +277,21 @@ struct LatentSplit {
 };
 
 template <int NT, int MT> struct LaGeom {
+  static constexpr int W = NT >= 2 ? 16 : 8, KG = W / 2;            // warps; shares of the latent columns
   static constexpr int M = 16 * MT, LD = NT * 64 + 8, LDS = kLaKeys + 4, LDP = kLaKeys + 8;
   static constexpr int c = 0;                                       // [2][64][LD] key blocks (the queries pass through here first)
-  static constexpr int s = c + 2 * kLaKeys * LD * 2;                // [4][M][LDS] score quarters
-  static constexpr int p = s + 4 * M * LDS * 4;                     // [2][M][LDP] probabilities: value, remainder
+  static constexpr int s = c + 2 * kLaKeys * LD * 2;                // [KG][M][LDS] partial scores
+  static constexpr int p = s + KG * M * LDS * 4;                     // [2][M][LDP] probabilities: value, remainder
   static constexpr int m = p + 2 * M * LDP * 2;                     // running maximum, sum, rescale of this step
   static constexpr int total = m + 3 * M * 4;
 };
 
 template <typename T, int NT, int MT>
-__global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const RfLatentAttn p, const LatentSplit sp) {
+__global__ void __launch_bounds__(32 * LaGeom<NT, MT>::W, 1) latent_attn_mma_kernel(const RfLatentAttn p, const LatentSplit sp) {
   pdl_prologue();
   using L = LaGeom<NT, MT>;
   constexpr int M = L::M, ld = L::LD, LDS = L::LDS, LDP = L::LDP, RP = NT * 64;
+  constexpr int W = L::W, KG = L::KG, kThreads = 32 * W, KS = RP / KG / 16, NTW = RP / W / 8;   // k16 steps of a share, output tiles per warp
   extern __shared__ __align__(16) uint8_t lsm[];
   const int rank = p.rank;
   T* sC = reinterpret_cast<T*>(lsm + L::c);
@@ -308,9 +310,9 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
   const T* pool = reinterpret_cast<const T*>(p.pool);
   const T* q = reinterpret_cast<const T*>(p.q) + ((size_t)row * p.heads + h0) * rank;
   const int heads_here = min(M, p.heads - h0);
-  const int kq = warp >> 1, key0 = (warp & 1) * 32;        // this warp's column quarter and key half for the scores
+  const int kq = warp >> 1, key0 = (warp & 1) * 32;        // this warp's column share and key half for the scores
 
-  for (int i = tid; i < M * (RP / 8); i += kLaThreads) {
+  for (int i = tid; i < M * (RP / 8); i += kThreads) {
     const int r = i / (RP / 8), c = (i % (RP / 8)) * 8;
     const bool ok = r < heads_here && c < rank;
     la_cp16(smem_u32(sC + r * ld + c), ok ? q + (size_t)r * rank + c : q, ok);
@@ -319,27 +321,28 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
   if (tid < M) { sM[tid] = -INFINITY; sL[tid] = 0.f; }
   la_wait<0>();
   __syncthreads();
-  uint32_t qf[MT][NT][4];
+  uint32_t qf[MT][KS][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int k = 0; k < NT; ++k)
-      ldsm_x4(smem_u32(sC + (m * 16 + (lane & 15)) * ld + kq * NT * 16 + k * 16 + (lane >> 4) * 8), qf[m][k][0], qf[m][k][1], qf[m][k][2], qf[m][k][3]);
+    for (int k = 0; k < KS; ++k)
+      ldsm_x4(smem_u32(sC + (m * 16 + (lane & 15)) * ld + kq * KS * 16 + k * 16 + (lane >> 4) * 8), qf[m][k][0], qf[m][k][1], qf[m][k][2], qf[m][k][3]);
   __syncthreads();
-  auto load_keys = [&](int b) {                            // four threads per key row
-    const int r = tid >> 2, j = lo + b * kLaKeys + r;
+  auto load_keys = [&](int b) {
+    constexpr int TPR = kThreads / kLaKeys;                // threads per key row
+    const int r = tid / TPR, j = lo + b * kLaKeys + r;
     const bool in = j <= pos;
     const T* src = in ? pool + ((size_t)pt[j >> 4] * 16 + (j & 15)) * rank : pool;
     T* dst = sC + ((b & 1) * kLaKeys + r) * ld;
 #pragma unroll
-    for (int i = 0; i < RP / 32; ++i) {
-      const int c = (tid & 3) * 8 + i * 32;
+    for (int i = 0; i < RP / (8 * TPR); ++i) {
+      const int c = (tid % TPR + i * TPR) * 8;
       la_cp16(smem_u32(dst + c), in && c < rank ? src + c : pool, in && c < rank);
     }
   };
   if (b0 < b1) load_keys(b0);
   la_commit();
-  float acc[MT][NT][4] = {};
+  float acc[MT][NTW][4] = {};
   const float scale_log2 = p.scale * 1.4426950408889634f;
 
   for (int b = b0; b < b1; ++b) {
@@ -351,11 +354,11 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
     {
       float s[MT][4][4] = {};
 #pragma unroll
-      for (int k = 0; k < NT; ++k)
+      for (int k = 0; k < KS; ++k)
 #pragma unroll
         for (int np = 0; np < 2; ++np) {                   // sixteen keys, one k16 step
           uint32_t bf[4];
-          ldsm_x4(smem_u32(kc + (key0 + np * 16 + (lane >> 4) * 8 + (lane & 7)) * ld + kq * NT * 16 + k * 16 + ((lane >> 3) & 1) * 8), bf[0], bf[1], bf[2], bf[3]);
+          ldsm_x4(smem_u32(kc + (key0 + np * 16 + (lane >> 4) * 8 + (lane & 7)) * ld + kq * KS * 16 + k * 16 + ((lane >> 3) & 1) * 8), bf[0], bf[1], bf[2], bf[3]);
 #pragma unroll
           for (int m = 0; m < MT; ++m) {
             MmaOp<T>::mma(s[m][np * 2], qf[m][k], bf[0], bf[1]);
@@ -372,9 +375,9 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
             *reinterpret_cast<float2*>(dst + (m * 16 + g + half * 8) * LDS + key0 + n * 8 + q4 * 2) = make_float2(s[m][n][half * 2], s[m][n][half * 2 + 1]);
     }
     __syncthreads();
-    // softmax step of 2 * MT rows per warp, all of them in flight (every block holds at least one visible key)
+    // softmax step of M / W rows per warp, all of them in flight (every block holds at least one visible key)
     {
-      constexpr int NR = 2 * MT;
+      constexpr int NR = M / W;
       const int r0 = warp * NR, j = lo + b * kLaKeys + lane * 2;
       float2 v[NR];
       float old[NR], mx[NR], sum[NR];
@@ -383,7 +386,7 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
         v[i] = make_float2(0.f, 0.f);
         old[i] = sM[r0 + i];
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
+        for (int k = 0; k < KG; ++k) {
           const float2 t = *reinterpret_cast<const float2*>(sS + (k * M + r0 + i) * LDS + lane * 2);
           v[i].x += t.x; v[i].y += t.y;
         }
@@ -424,7 +427,7 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
     for (int m = 0; m < MT; ++m) {
       const float c0 = sA[m * 16 + g], c1 = sA[m * 16 + g + 8];
 #pragma unroll
-      for (int t = 0; t < NT; ++t) {
+      for (int t = 0; t < NTW; ++t) {
         acc[m][t][0] *= c0; acc[m][t][1] *= c0; acc[m][t][2] *= c1; acc[m][t][3] *= c1;
       }
     }
@@ -440,8 +443,8 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
             ldsm_x4(smem_u32(sP + (hl * M + m * 16 + (lane & 15)) * LDP + kk + hk * 16 + (lane >> 4) * 8), a[m][hl][hk][0], a[m][hl][hk][1],
                     a[m][hl][hk][2], a[m][hl][hk][3]);
 #pragma unroll
-      for (int t = 0; t < NT; ++t) {
-        const int c = (warp * NT + t) * 8;
+      for (int t = 0; t < NTW; ++t) {
+        const int c = (warp * NTW + t) * 8;
         {
           uint32_t bf[4];                                  // eight columns, 32 keys
           ldsm_x4_t(smem_u32(kc + (kk + lane) * ld + c), bf[0], bf[1], bf[2], bf[3]);
@@ -468,8 +471,8 @@ __global__ void __launch_bounds__(kLaThreads, 1) latent_attn_mma_kernel(const Rf
       const size_t hr = (size_t)row * p.heads + h0 + r;
       const float inv = sp.splits == 1 ? 1.f / sL[r] : 1.f;
 #pragma unroll
-      for (int t = 0; t < NT; ++t) {
-        const int c = (warp * NT + t) * 8 + q4 * 2;
+      for (int t = 0; t < NTW; ++t) {
+        const int c = (warp * NTW + t) * 8 + q4 * 2;
         if (c >= rank) continue;
         const float v0 = acc[m][t][half * 2] * inv, v1 = acc[m][t][half * 2 + 1] * inv;
         if (sp.splits == 1) *reinterpret_cast<uint32_t*>(reinterpret_cast<T*>(p.o) + hr * rank + c) = MmaOp<T>::pack(v0, v1);
@@ -632,7 +635,7 @@ static int launch_latent_attn_mma(const RfLatentAttn* a, cudaStream_t s) {
   do {                                                                                                            \
     constexpr int smem = LaGeom<NT, MT>::total;                                                                   \
     RF_ALLOW_SMEM_PER_DEVICE((latent_attn_mma_kernel<T, NT, MT>), smem);                                          \
-    RF_CUDA_CHECK(::rf::launch_k(latent_attn_mma_kernel<T, NT, MT>, grid, dim3(kLaThreads), smem, s, 1, *a, sp)); \
+    RF_CUDA_CHECK(::rf::launch_k(latent_attn_mma_kernel<T, NT, MT>, grid, dim3(32 * LaGeom<NT, MT>::W), smem, s, 1, *a, sp)); \
   } while (0)
 #define RF_LN(NT)             \
   do {                        \
