@@ -1,4 +1,4 @@
-// HGRN2 linear attention: the forget gate of a channel also decides how much of the value is written,
+// HGRN2 linear attention: one gate per key channel sets how much of the state is kept and, as its complement, how much is added,
 //   S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T,   o_t = S_t^T q_t,
 // with an fp32 state per (slot, head), q = silu(.), f = lower + (1 - lower) sigmoid(. + bias), and an RMSNorm per head on o.
 //   * rf_hgrn2_recurrent: token by token (decode steps, short portions, everything in fp32),

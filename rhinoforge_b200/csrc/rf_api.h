@@ -374,7 +374,7 @@ typedef struct RfLatentAttn {
 int rf_latent_attn(const RfLatentAttn* a, rf_stream_t stream);
 uint64_t rf_latent_attn_scratch_bytes(int rows, int heads, int rank, int max_kv);
 
-// Linear attention whose forget gate also decides what is written (HGRN2), over packed input rows [q | f | v]:
+// HGRN2 linear attention (what a gate takes from the state it gives to the new value), over packed input rows [q | f | v]:
 //   q = silu(q), f = lower + (1 - lower) * sigmoid(f + f_bias), S = diag(f) S + (1 - f) v^T, o = S^T q,
 //   out = o / rms(o) * norm_w per head (mean over the true value size; null norm_w: plain o)
 // state: fp32 [slots, heads, dim, vdim].  Padding channels of dim have lower = 1, padding value columns are zero.

@@ -19,8 +19,8 @@ from ..runtime.errors import UnsupportedModelError
 
 @dataclass(frozen=True)
 class LatentAttention:
-    """Attention over one cached latent row per token; keys and values of a head are linear maps of it.  ``window``: a query
-    sees itself and the ``window - 1`` tokens before it (None: every earlier token)."""
+    """Attention over one cached latent row per token; keys and values of a head are linear maps of it.  ``window``: how many
+    positions a query sees, its own included (None: all of them)."""
     heads: int
     dim: int
     vdim: int
@@ -31,7 +31,7 @@ class LatentAttention:
 
 @dataclass(frozen=True)
 class HGRN2:
-    """Linear attention whose forget gate also decides what is written (state ``[heads, dim, vdim]``)."""
+    """Linear attention with one gate per key channel for keeping and adding (state ``[heads, dim, vdim]``)."""
     heads: int
     dim: int
     vdim: int

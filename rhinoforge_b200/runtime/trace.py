@@ -4,7 +4,7 @@
 
 Steps are read from standard input, one JSON object per line::
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": ["b"]}
+    {"step": 4, "entries": [{"id": "r1", "tokens": [11, 48], "want": [1]}, {"id": "r2", "tokens": [7], "want": []}], "end": ["r1"]}
 
 All entries of a step run as one batch through the request scheduler and the engine's step; nothing is sampled.  The logits at
 the wanted places go to ``OUT/<step>.f32`` (little-endian fp32, ``[wanted, vocab]``, in the order of the entries), then

@@ -171,7 +171,7 @@ def test_latent_attention_windows_and_ranks(dtype, heads, rank, window):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("window,distance,seen", [(72, 71, True), (72, 72, False), (64, 63, True), (64, 64, False), (1, 0, True), (1, 1, False),
+@pytest.mark.parametrize("window,distance,seen", [(90, 89, True), (90, 90, False), (64, 63, True), (64, 64, False), (1, 0, True), (1, 1, False),
                                                   (17, 16, True), (17, 17, False), (0, 299, True), (200, 199, True), (200, 200, False)])
 def test_one_key_that_stands_out_at_the_edge_of_the_window(dtype, window, distance, seen):
     """All keys are equal but one, which wins the softmax outright when it is visible."""
@@ -208,7 +208,7 @@ def hgrn2_reference(x, fb, lower, nw, state, lens, pos0, slots, heads, D, VD, ep
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("chunked", [False, True])
-@pytest.mark.parametrize("heads,D,VD,vdim", [(1, 8, 8, 8), (2, 48, 64, 64), (3, 40, 24, 21), (2, 128, 128, 128), (1, 136, 160, 155), (1, 64, 320, 320),
+@pytest.mark.parametrize("heads,D,VD,vdim", [(1, 8, 8, 8), (2, 56, 72, 72), (3, 40, 24, 21), (2, 128, 128, 128), (1, 136, 160, 155), (1, 64, 320, 320),
                                              (1, 272, 64, 64)])
 def test_hgrn2_against_the_recurrence(dtype, chunked, heads, D, VD, vdim):
     lens, pos0, slots = [1, 70, 2, 16, 17, 131], [4, 0, 33, 64, 0, 9], [5, 2, 0, 1, 4, 6]
@@ -257,7 +257,7 @@ def test_hgrn2_keeps_a_value_written_long_ago():
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("batch,heads,D,VD,vdim", [(1, 1, 8, 8, 8), (3, 2, 48, 64, 61), (70, 8, 128, 128, 128), (5, 3, 40, 24, 24), (2, 2, 264, 160, 160),
+@pytest.mark.parametrize("batch,heads,D,VD,vdim", [(1, 1, 8, 8, 8), (3, 2, 56, 72, 61), (70, 8, 128, 128, 128), (5, 3, 40, 24, 24), (2, 2, 264, 160, 160),
                                                    (300, 3, 16, 32, 32)])
 def test_hgrn2_decode_step_of_many_sequences(dtype, batch, heads, D, VD, vdim):
     """One token per sequence, several steps in a row: more states than resident CTAs, scattered slots, fresh sequences."""

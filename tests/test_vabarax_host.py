@@ -220,7 +220,7 @@ def test_example_configuration_is_checked(tmp_path):
     spec.loader.exec_module(mod)
     good = (root / "examples" / "configs" / "vabarax.toml").read_text()
     assert mod.load_config(root / "examples" / "configs" / "vabarax.toml")["generation"]["max_new_tokens"] == 16
-    for old, new in (("prompt_tokens = [[5", "prompt_tokens = [[], [5"), ("slots = 2", "slots = 0"), ('"bfloat16"', '"int8"'),
+    for old, new in (("prompt_tokens = [[9", "prompt_tokens = [[], [9"), ("slots = 2", "slots = 0"), ('"bfloat16"', '"int8"'),
                      ("max_new_tokens = 16", "max_new_tokens = true")):
         assert old in good
         f = tmp_path / "c.toml"
