@@ -106,6 +106,8 @@ class RfAttn(C.Structure):
         ("scale", C.c_float),
         ("ws", C.c_void_p), ("ws_bytes", C.c_uint64),
         ("status", C.c_void_p), ("dtype", C.c_int32),
+        ("slot", C.c_void_p), ("chunk", C.c_int32), ("sink", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_int64),
+        ("seq_of_row", C.c_void_p), ("pos", C.c_void_p),
     ]
 
 
@@ -193,7 +195,8 @@ class RfRows(C.Structure):
 class RfStreamNorm(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("x", "table", "ids", "row_idx", "y", "y_norm_w", "x_out", "x_cast", "norm_w", "out",
                                           "shift", "shift_state")] + [("rows", RfRows)] + \
-               [("n_rows", C.c_int32), ("H", C.c_int32), ("dim", C.c_int32), ("eps", C.c_float), ("dtype", C.c_int32)]
+               [("n_rows", C.c_int32), ("H", C.c_int32), ("dim", C.c_int32), ("eps", C.c_float), ("dtype", C.c_int32),
+                ("embed_scale", C.c_float), ("y_slots", C.c_void_p), ("y_picks", C.c_int32)]
 
 
 class RfHeadLinear(C.Structure):
@@ -218,15 +221,63 @@ class RfMixedConfig(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("layers", "hidden", "hidden_true", "vocab", "vocab_ld", "dtype", "max_tokens", "max_seqs",
                                          "max_seq_len", "side_dim")] + \
                [("side_ld", C.c_int64), ("eps", C.c_float), ("weights_packed", C.c_int32), ("long_min", C.c_int32)] + \
-               [(n, C.c_void_p) for n in ("embed", "side_table", "final_norm", "w_lm")]
+               [(n, C.c_void_p) for n in ("embed", "side_table", "final_norm", "w_lm")] + \
+               [("embed_scale", C.c_float), ("norm_after", C.c_int32)]
+
+
+class RfMixedState(C.Structure):
+    _fields_ = [("latent_pool", C.c_void_p), ("k_pool", C.c_void_p), ("v_pool", C.c_void_p), ("pool_pages", C.c_int64),
+                ("rec_state", C.c_void_p), ("conv_state", C.c_void_p), ("shift_state", C.c_void_p)]
 
 
 class RfMixedLayer(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "vdim", "vdim_true", "rank", "rank_true", "window", "expand_hd",
-                                         "inter", "act")] + [("scale", C.c_float), ("in_dim", C.c_int32)] + \
-               [(n, C.c_void_p) for n in ("norm1", "norm2", "shift", "shift_state", "w_in", "w_o", "w_up", "w_down", "latent_norm",
-                                          "w_absorb", "w_unabsorb", "w_expand", "latent_pool", "f_bias", "lower", "head_norm",
-                                          "rec_state", "side_gate", "side_proj", "side_norm")]
+                                         "inter", "act")] + [("scale", C.c_float), ("in_dim", C.c_int32), ("out_dim", C.c_int32)] + \
+               [(n, C.c_void_p) for n in ("norm1", "norm2", "shift", "w_in", "w_o", "w_up", "w_down", "latent_norm", "w_absorb",
+                                          "w_unabsorb", "w_expand", "f_bias", "lower", "head_norm", "side_gate", "side_proj",
+                                          "side_norm")] + \
+               [(n, C.c_int32) for n in ("kv_heads", "dim_true", "tensor_core", "chunk", "gated", "rot_dims", "v_role")] + \
+               [("v_lambda", C.c_float)] + [(n, C.c_void_p) for n in ("cos", "sin", "q_norm", "k_norm", "sink")] + \
+               [(n, C.c_int32) for n in ("inner", "states", "dt_rank", "taps")] + \
+               [(n, C.c_void_p) for n in ("conv_w", "conv_b", "a2", "d_skip", "dt_bias", "w_x", "w_dt", "w_dt_rows")] + \
+               [(n, C.c_int32) for n in ("experts", "top", "groups", "keep", "score_fn", "norm_topk", "shared_inter", "bank_inter")] + \
+               [("route_scale", C.c_float)] + [(n, C.c_void_p) for n in ("router", "correction", "shared_up", "shared_down")] + \
+               [("st", RfMixedState)]
+
+
+class RfQkvInsert(C.Structure):
+    _fields_ = [("qkv", C.c_void_p), ("ld", C.c_int64), ("k_off", C.c_int32), ("v_off", C.c_int32)] + \
+               [(n, C.c_void_p) for n in ("q_norm", "k_norm", "cos", "sin", "v_first", "k_pool", "v_pool")] + [("rows", RfRows)] + \
+               [(n, C.c_int32) for n in ("n_rows", "heads", "kv_heads", "hd", "dim", "vdim", "rot_dims", "v_role")] + \
+               [("v_lambda", C.c_float), ("eps", C.c_float), ("dtype", C.c_int32)]
+
+
+class RfConvSilu(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64), ("y", C.c_void_p), ("ldy", C.c_int64), ("w", C.c_void_p), ("bias", C.c_void_p),
+                ("state", C.c_void_p), ("rows", RfRows)] + [(n, C.c_int32) for n in ("max_q_len", "channels", "taps", "dtype")]
+
+
+class RfMamba1(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64), ("z", C.c_void_p), ("ldz", C.c_int64), ("bc", C.c_void_p), ("ld_bc", C.c_int64),
+                ("dt", C.c_void_p), ("ld_dt", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("w_dt", "dt_bias", "a2", "d", "state", "out")] + [("ldo", C.c_int64), ("rows", RfRows)] + \
+               [(n, C.c_int32) for n in ("inner", "states", "rank", "dtype")]
+
+
+class RfMoeRouter(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("w", "correction", "ids", "weights", "rank", "counters", "start", "tiles", "slot_of",
+                                          "token_of_slot", "slot_w")] + \
+               [(n, C.c_int32) for n in ("rows", "experts", "width", "k", "groups", "keep", "score_fn", "norm_topk")] + \
+               [("scale", C.c_float)] + [(n, C.c_int32) for n in ("tile_rows", "slot_ld", "has_shared", "shared_tiles", "scatter", "dtype")]
+
+
+class RfMoeExperts(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64), ("w", C.c_void_p), ("w_shared", C.c_void_p), ("out", C.c_void_p), ("ldo", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("tiles", "token_of_slot", "slot_w")] + \
+               [(n, C.c_int32) for n in ("max_tiles", "experts", "n", "k", "shared_n", "shared_k", "dual", "tile_rows",
+                                         "bank_section_row_tiles", "bank_kb_total", "rt_per_expert", "kb_per_expert",
+                                         "shared_section_row_tiles", "shared_kb_total", "dtype")]
 
 
 class RfMixedForward(C.Structure):
@@ -267,6 +318,7 @@ def lib() -> C.CDLL:
         l.rf_mixed_arena_bytes.restype = C.c_uint64
         l.rf_mixed_status_ptr.restype = C.c_void_p
         l.rf_latent_attn_scratch_bytes.restype = C.c_uint64
+        l.rf_attn_decode_scratch_bound.restype = C.c_uint64
         l.rf_pack_weight_bytes.restype = C.c_uint64
         l.rf_pack_w4_bytes.restype = C.c_uint64
         l.rf_pack_w4_bytes.argtypes = [C.c_int64, C.c_int64, C.c_int32, C.c_int32]

@@ -11,6 +11,7 @@ BUILTIN_ADAPTERS = (
     ("Qwen3_5ForConditionalGeneration", "rhinoforge_b200.adapters.qwen3_5", "Qwen3_5Adapter"),
     ("Qwen3VLForConditionalGeneration", "rhinoforge_b200.adapters.qwen3_vl", "Qwen3VLAdapter"),
     ("Vabarax", "rhinoforge_b200.adapters.vabarax", "VabaraxAdapter"),
+    ("Zulopel", "rhinoforge_b200.adapters.zulopel", "ZulopelAdapter"),
 )
 
 __all__ = ["BUILTIN_ADAPTERS"]

@@ -20,6 +20,7 @@ _ROUTES = {
     "LlamaForCausalLM": "use RPUModelForCausalLM.from_pretrained(...) and .to('rpu')",
     "Qwen3ForCausalLM": "use RPUModelForCausalLM.from_pretrained(...) and .to('rpu')",
     "Vabarax": "use RPUModelForCausalLM.from_pretrained(..., device='rpu')",
+    "Zulopel": "use RPUModelForCausalLM.from_pretrained(..., device='rpu')",
 }
 
 

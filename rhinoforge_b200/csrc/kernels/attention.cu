@@ -99,15 +99,20 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   constexpr int kStageBytes = 4 * kPageBytes;
   AttnCtl* ctl = reinterpret_cast<AttnCtl*>(smem + (size_t)p.stages * kStageBytes);
 
-  const int split = blockIdx.x, kvh = blockIdx.y, seq = blockIdx.z;
+  const int split = blockIdx.x, kvh = (int)blockIdx.y / p.g_tiles, g_first = ((int)blockIdx.y % p.g_tiles) * 16, seq = blockIdx.z;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int kvlen = p.kv_len[seq];
+  // by row: the row's own position bounds its keys and its sequence's slot owns the pages
+  const int owner = p.pos && p.seq_of_row ? p.seq_of_row[seq] : seq;
+  const int pt_row = p.slot ? p.slot[owner] : owner;
+  const int kvlen = p.pos ? p.pos[seq] + 1 : p.kv_len[seq];
+  const int kvlo = p.chunk > 0 && kvlen > 0 ? (kvlen - 1) / p.chunk * p.chunk : 0;
   const int total_pages = (kvlen + 15) >> 4;
-  const int pg_begin = split * p.pages_per_split;
+  const int pg_begin = (kvlo >> 4) + split * p.pages_per_split;
   const int pg_end = min(total_pages, pg_begin + p.pages_per_split);
   const int npg = max(0, pg_end - pg_begin);
   const int iters = (npg + 3) >> 2;
-  const int G = p.G;
+  const int G = min(p.G - g_first, 16);          // query heads of this CTA
+  const int head0 = kvh * p.G + g_first;
 
   if (tid == 0) {
     for (int s = 0; s < p.stages; ++s) {
@@ -142,7 +147,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
           const int pg = pg_begin + it * 4 + w;
           int row, col0;
           if (p.paged) {
-            const int page_id = p.page_table[(size_t)seq * p.pt_stride + pg];
+            const int page_id = p.page_table[(size_t)pt_row * p.pt_stride + pg];
             row = (page_id * p.Hkv + kvh) * 16;
             col0 = 0;
           } else {
@@ -161,7 +166,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     uint32_t qf[HD / 16][4];
     {
       const int g0 = lane >> 2, g1 = g0 + 8;
-      const T* qbase = reinterpret_cast<const T*>(p.q) + (size_t)seq * p.ldq + (size_t)kvh * G * HD;
+      const T* qbase = reinterpret_cast<const T*>(p.q) + (size_t)seq * p.ldq + (size_t)head0 * HD;
 #pragma unroll
       for (int ks = 0; ks < HD / 16; ++ks) {
         const int col = ks * 16 + (lane & 3) * 2;
@@ -191,8 +196,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int t0 = tok0 + (e & 1), t1 = tok0 + 8 + (e & 1);
-          x[0][e] = t0 < kvlen ? s0[e] * p.scale_log2 : -INFINITY;
-          x[1][e] = t1 < kvlen ? s1[e] * p.scale_log2 : -INFINITY;
+          x[0][e] = t0 < kvlen && t0 >= kvlo ? s0[e] * p.scale_log2 : -INFINITY;
+          x[1][e] = t1 < kvlen && t1 >= kvlo ? s1[e] * p.scale_log2 : -INFINITY;
         }
         const float mx0 = quad_max(fmaxf(fmaxf(x[0][0], x[0][1]), fmaxf(x[1][0], x[1][1])));
         const float mx1 = quad_max(fmaxf(fmaxf(x[0][2], x[0][3]), fmaxf(x[1][2], x[1][3])));
@@ -250,7 +255,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     if (p.splits > 1) {
       for (int idx = tid; idx < G * HD; idx += blockDim.x) {
         const int g = idx / HD, col = idx % HD;
-        const size_t base = ((size_t)seq * p.Hq + (size_t)kvh * G + g) * p.splits + split;
+        const size_t base = ((size_t)seq * p.Hq + head0 + g) * p.splits + split;
         p.ws_o[base * HD + col] = 0.f;
         if (col == 0) p.ws_lse[base] = -INFINITY;
       }
@@ -271,10 +276,13 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
         den += f * ml[w * 16 + g];
       }
     }
-    const float val = den > 0.f ? num / den : 0.f;
-    const int head = kvh * G + g;
+    const int head = head0 + g;
+    if (p.splits == 1 && p.sink && M != -INFINITY) den += exp2f(p.sink[head] * kLog2e - M);
+    float val = den > 0.f ? num / den : 0.f;
     if (p.splits == 1) {
-      reinterpret_cast<T*>(p.out)[(size_t)seq * p.ldo + (size_t)head * HD + col] = Num<T>::from_f(val);
+      const size_t col_of_row = (size_t)head * HD + col;
+      if (p.gate) val *= sigmoid_fast(Num<T>::to_f(reinterpret_cast<const T*>(p.gate)[(size_t)seq * p.ld_gate + col_of_row]));
+      reinterpret_cast<T*>(p.out)[(size_t)seq * p.ldo + col_of_row] = Num<T>::from_f(val);
     } else {
       const size_t base = ((size_t)seq * p.Hq + head) * p.splits + split;
       p.ws_o[base * HD + col] = val;
@@ -286,7 +294,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 template <typename T>
 __global__ void attn_decode_combine_kernel(const float* __restrict__ ws_o,
                                            const float* __restrict__ ws_lse, T* __restrict__ out,
-                                           int64_t ldo, int Hq, int hd, int splits) {
+                                           int64_t ldo, int Hq, int hd, int splits, const float* __restrict__ sink,
+                                           const T* __restrict__ gate, int64_t ldg) {
   pdl_prologue();
   const int head = blockIdx.x, seq = blockIdx.y;
   const size_t base = ((size_t)seq * Hq + head) * splits;
@@ -300,8 +309,11 @@ __global__ void attn_decode_combine_kernel(const float* __restrict__ ws_o,
         num += f * ws_o[(base + s) * hd + col];
         den += f;
       }
+      if (sink) den += exp2f(sink[head] * kLog2e - M);
     }
-    out[(size_t)seq * ldo + (size_t)head * hd + col] = Num<T>::from_f(den > 0.f ? num / den : 0.f);
+    float val = den > 0.f ? num / den : 0.f;
+    if (gate) val *= sigmoid_fast(Num<T>::to_f(gate[(size_t)seq * ldg + (size_t)head * hd + col]));
+    out[(size_t)seq * ldo + (size_t)head * hd + col] = Num<T>::from_f(val);
   }
 }
 
@@ -507,7 +519,7 @@ static int fill_params(const RfAttn* a, AttnParams* p) {
   RF_REQUIRE(a && a->q && a->out, "attention needs q and out");
   RF_REQUIRE(a->hd == 64 || a->hd == 128 || a->hd == 256, "attention head_dim %d (64/128/256; pad others)", a->hd);
   RF_REQUIRE(a->Hkv > 0 && a->Hq % a->Hkv == 0, "attention heads %d / kv heads %d", a->Hq, a->Hkv);
-  RF_REQUIRE(a->kv_len && a->num_seqs > 0, "attention needs kv_len and sequences");
+  RF_REQUIRE((a->kv_len || a->pos) && a->num_seqs > 0, "attention needs kv_len and sequences");
   RF_REQUIRE(a->dtype == 0 || a->dtype == 1, "attention dtype");
   const bool paged = a->k_pool != nullptr;
   if (paged) RF_REQUIRE(a->v_pool && a->page_table && a->pool_pages > 0, "paged attention needs v_pool, page_table, pool_pages");
@@ -522,6 +534,9 @@ static int fill_params(const RfAttn* a, AttnParams* p) {
   p->seg_q = a->seg_q; p->seg_k = a->seg_k;
   const float scale = a->scale > 0.f ? a->scale : 1.0f / sqrtf((float)a->hd);
   p->scale_log2 = scale * 1.4426950408889634f;
+  if (a->slot || a->chunk > 0 || a->pos) RF_REQUIRE(paged, "slots, chunks and attention by row need the paged pool");
+  p->slot = a->slot; p->chunk = a->chunk; p->sink = a->sink; p->gate = a->gate; p->ld_gate = a->ld_gate;
+  p->seq_of_row = a->seq_of_row; p->pos = a->pos; p->g_tiles = ceil_div(p->G, 16);
   p->ws_o = nullptr; p->ws_lse = nullptr; p->splits = 1; p->pages_per_split = 1 << 28; p->stages = 2;
   p->status = a->status;
   return RF_OK;
@@ -549,7 +564,7 @@ struct DecodeSplitPlan {
 };
 static DecodeSplitPlan plan_decode_split(int num_seqs, int Hq, int Hkv, int hd, int max_kv_len, bool allow_split) {
   const int max_pages = std::max(1, (max_kv_len + 15) / 16);
-  const int ctas = num_seqs * Hkv;
+  const int ctas = num_seqs * Hkv * ceil_div(Hq / Hkv, 16);
   int splits = 1;
   // RF_ATTN_DECODE_CTAS_PER_SM (default 2; 1 for heads of 256): CTAs per SM the split aims at; RF_ATTN_DECODE_MIN_PAGES (default 8): fewest
   // pages a split may cover
@@ -583,7 +598,9 @@ static int launch_decode(const RfAttn* a, AttnParams& p, cudaStream_t s) {
   auto kfn = attn_decode_kernel<T, HD>;
   RF_ALLOW_SMEM_PER_DEVICE(kfn, 200 * 1024);
   // split the KV range so that small batches still fill the machine
-  const DecodeSplitPlan pl = plan_decode_split(a->num_seqs, a->Hq, a->Hkv, HD, a->max_kv_len, a->ws != nullptr);
+  // a chunk may begin anywhere in a page: one page more than its own size
+  const int max_kv = a->chunk > 0 ? std::min(a->max_kv_len, a->chunk) + 15 : a->max_kv_len;
+  const DecodeSplitPlan pl = plan_decode_split(a->num_seqs, a->Hq, a->Hkv, HD, max_kv, a->ws != nullptr);
   const int splits = pl.splits;
   if (splits > 1) {
     RF_REQUIRE(pl.scratch_bytes <= a->ws_bytes, "decode attention scratch too small: need %llu B",
@@ -597,13 +614,13 @@ static int launch_decode(const RfAttn* a, AttnParams& p, cudaStream_t s) {
     static const int ef = [] { const char* e = getenv("RF_ATTN_KV_EVICT_FIRST"); return e ? atoi(e) : 1; }();
     p.kv_stream = ef;
   }
-  dim3 grid(splits, a->Hkv, a->num_seqs);
+  dim3 grid(splits, a->Hkv * p.g_tiles, a->num_seqs);
   RF_CUDA_CHECK(::rf::launch_k(kfn, dim3(grid), dim3(160), smem, s, 1, tmK, tmV, p));
   RF_CUDA_CHECK(cudaGetLastError());
   ::rf::count_launch();
   if (splits > 1) {
     dim3 g2(a->Hq, a->num_seqs);
-    RF_CUDA_CHECK(::rf::launch_k(attn_decode_combine_kernel<T>, dim3(g2), dim3(HD < 128 ? HD : 128), 0, s, 1, p.ws_o, p.ws_lse, (T*)a->out, a->ldo, a->Hq, HD, splits));
+    RF_CUDA_CHECK(::rf::launch_k(attn_decode_combine_kernel<T>, dim3(g2), dim3(HD < 128 ? HD : 128), 0, s, 1, p.ws_o, p.ws_lse, (T*)a->out, a->ldo, a->Hq, HD, splits, a->sink, (const T*)a->gate, a->ld_gate));
     RF_CUDA_CHECK(cudaGetLastError());
   ::rf::count_launch();
   }
@@ -651,12 +668,19 @@ extern "C" uint64_t rf_attn_decode_scratch_bytes(int num_seqs, int Hq, int hd) {
   return (uint64_t)num_seqs * Hq * 64 * (hd + 1) * sizeof(float);
 }
 
+extern "C" uint64_t rf_attn_decode_scratch_bound(int Hq, int Hkv, int hd) {
+  // plan_decode_split splits only below `limit` CTAs, into at most limit / CTAs parts: rows x K/V heads x splits <= limit
+  const char* e = getenv("RF_ATTN_DECODE_CTAS_PER_SM");
+  const uint64_t limit = (uint64_t)std::max(2, e ? atoi(e) : 0) * sm_count();
+  return limit * (Hq / std::max(Hkv, 1)) * (hd + 1) * sizeof(float);
+}
+
 extern "C" int rf_attn_decode(const RfAttn* a, rf_stream_t stream) {
   RF_SKIP_IF_REPLAYING();
   AttnParams p;
   int rc = fill_params(a, &p);
   if (rc) return rc;
-  RF_REQUIRE(a->Hq / a->Hkv <= 16, "decode attention handles GQA groups up to 16, got %d", a->Hq / a->Hkv);
+  RF_REQUIRE(a->num_seqs <= 65535, "decode attention: %d rows in one launch", a->num_seqs);
   RF_REQUIRE(a->max_kv_len > 0, "decode attention needs max_kv_len");
   RF_REQUIRE(a->window <= 0, "decode attention has no sliding-window form (window=%d): every query would see the whole "
              "context", a->window);
@@ -681,6 +705,7 @@ extern "C" int rf_attn_prefill(const RfAttn* a, rf_stream_t stream) {
   // tcgen05 kernel by default; RF_ATTN_TC=0 selects the mma.sync kernel (A/B timing)
   static const bool use_tc = [] { const char* e = getenv("RF_ATTN_TC"); return !(e && e[0] == '0'); }();
   if (use_tc) return rf::launch_prefill_tc(a, p, s);
+  RF_REQUIRE(!a->slot && a->chunk <= 0 && !a->sink && !a->gate, "slots, chunks, sinks and gates need the tcgen05 prefill kernel");
   RF_ATTN_DISPATCH(launch_prefill)
 }
 

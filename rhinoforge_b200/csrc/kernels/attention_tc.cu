@@ -74,13 +74,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   if (qt * kFaRows >= qlen) return;                       // before any barrier or allocation
   const int kvlen = p.kv_len[seq];
   const int kvh = h / p.G;
+  const int pt_row = p.slot ? p.slot[seq] : seq;
   const int qpos0 = kvlen - qlen;                         // position of query row 0 on the kv axis
   const int q_row0 = p.q_start[seq] + qt * kFaRows;
   const int rows_here = min(kFaRows, qlen - qt * kFaRows);
   int kv_hi = kvlen;
   if (p.causal) kv_hi = min(kvlen, qpos0 + qt * kFaRows + rows_here);
   int kv_lo = 0;
-  if (p.window > 0) kv_lo = max(0, qpos0 + qt * kFaRows - p.window + 1) & ~(KVB - 1);
+  if (p.window > 0) kv_lo = max(0, qpos0 + qt * kFaRows - p.window + 1);
+  if (p.chunk > 0) kv_lo = max(kv_lo, (qpos0 + qt * kFaRows) / p.chunk * p.chunk);   // the first row's chunk
+  kv_lo &= ~(KVB - 1);
   const int nblk = kv_hi > kv_lo ? (kv_hi - kv_lo + KVB - 1) / KVB : 0;
 
   if (tid == 0) {
@@ -141,7 +144,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           int row, col0;
           if (p.paged) {
             const int pi = min((t0 >> 4) + w, p.pt_stride - 1);
-            const int page_id = p.page_table[(size_t)seq * p.pt_stride + pi];
+            const int page_id = p.page_table[(size_t)pt_row * p.pt_stride + pi];
             row = (page_id * p.Hkv + kvh) * 16;
             col0 = 0;
           } else {
@@ -219,7 +222,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     uint8_t* prow = psm + r * 128;
     // bounds of the valid kv positions of this row that do not depend on data: [lo, hi]
     const int hi_row = min(kvlen - 1, p.causal ? qpos0 + qi : 0x7fffffff);
-    const int lo_row = p.window > 0 ? qpos0 + qi - p.window + 1 : 0;
+    int lo_row = p.window > 0 ? qpos0 + qi - p.window + 1 : 0;
+    if (p.chunk > 0) lo_row = max(lo_row, (qpos0 + qi) / p.chunk * p.chunk);
     const bool data_mask = mrow != nullptr || p.seg_q != nullptr;
     for (int j = 0; j < nblk; ++j) {
       const int b = j & 1;
@@ -332,7 +336,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     }
     tc_fence_after_sync();
     if (ok) {
+      if (p.sink && l > 0.f) l += exp2f(p.sink[h] * kLog2e - m_ref);
       const float inv = l > 0.f ? 1.f / l : 0.f;
+      const T* grow = p.gate ? reinterpret_cast<const T*>(p.gate) + (size_t)(p.q_start[seq] + qi) * p.ld_gate + (size_t)h * HD : nullptr;
       T* orow = reinterpret_cast<T*>(p.out) + (size_t)(p.q_start[seq] + qi) * p.ldo + (size_t)h * HD;
 #pragma unroll 1
       for (int c0 = 0; c0 < HD; c0 += 32) {
@@ -350,6 +356,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             float f8[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) f8[i] = __uint_as_float(ov[u * 8 + i]) * inv;
+            if (grow) {
+              float g8[8];
+              load8(grow + c0 + u * 8, g8);
+#pragma unroll
+              for (int i = 0; i < 8; ++i) f8[i] *= sigmoid_fast(g8[i]);
+            }
             store8(orow + c0 + u * 8, f8);
           }
         }

@@ -243,7 +243,7 @@ using namespace rf;
 // 32-key tile, which is less fixed cost than the tensor-memory kernel's set-up.  RF_ATTN_TINY=0 turns that routing off.
 bool rf_attn_tiny_eligible(const RfAttn* a) {
   static const bool on = [] { const char* e = getenv("RF_ATTN_TINY"); return !(e && e[0] == '0'); }();
-  if (!on || !a || a->k_pool || !a->k || !a->v || a->mask || a->seg_q || a->seg_k) return false;
+  if (!on || !a || a->k_pool || !a->k || !a->v || a->mask || a->seg_q || a->seg_k || a->chunk > 0 || a->sink || a->gate) return false;
   if (a->hd != 64 && a->hd != 128) return false;
   if (a->ldq % 8 || a->ldk % 8 || a->ldv % 8 || a->ldo % 2) return false;
   const int max_q = a->q_len ? a->max_q_len : 1;
@@ -266,7 +266,7 @@ int rf_attn_wide(const RfAttn* a, rf_stream_t stream) {
   RF_REQUIRE(a->hd == 512 || a->hd == 128 || a->hd == 64, "register-accumulator attention takes head_dim 64 / 128 / 512, got %d", a->hd);
   RF_REQUIRE(a->Hkv > 0 && a->Hq % a->Hkv == 0, "attention heads %d / kv heads %d", a->Hq, a->Hkv);
   RF_REQUIRE(a->k && a->v && a->kv_start && a->kv_len && !a->k_pool, "this attention path takes contiguous K / V rows (k, v, kv_start, kv_len)");
-  RF_REQUIRE(!a->mask && !a->seg_q && !a->seg_k, "this attention path takes causal / window masks only");
+  RF_REQUIRE(!a->mask && !a->seg_q && !a->seg_k && a->chunk <= 0 && !a->sink && !a->gate, "this attention path takes causal / window masks only");
   RF_REQUIRE(a->ldq % 8 == 0 && a->ldk % 8 == 0 && a->ldv % 8 == 0 && a->ldo % 2 == 0, "attention row pitches must be multiples of 16 bytes");
   RF_REQUIRE(a->num_seqs > 0 && (a->dtype == 0 || a->dtype == 1), "attention needs sequences and a 16-bit dtype");
   WideParams p;

@@ -21,7 +21,16 @@ struct AttnParams {
   int32_t splits, pages_per_split, stages;
   int32_t kv_stream;      // decode: K/V pages are read with the L2 evict-first policy
   int32_t* status;
+  const int32_t* slot;    // page-table row of a sequence
+  int32_t chunk;
+  const float* sink;      // natural-log units
+  const void* gate; int64_t ld_gate;
+  const int32_t* seq_of_row; const int32_t* pos;
+  int32_t g_tiles;        // decode: CTAs that share one K/V head (16 query heads each)
 };
+
+constexpr float kLog2e = 1.4426950408889634f;
+__device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 
 
 }  // namespace rf

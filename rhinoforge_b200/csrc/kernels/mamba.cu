@@ -1,0 +1,453 @@
+// Selective scan (Mamba) layers: causal convolution with carried inputs, the token-by-token recurrence with its step-size
+// projection (decode rows and short portions), and the tiled scan of prefill-sized portions.
+//
+// The state of a channel is a short fp32 vector.  Four neighbouring lanes hold one channel, each lane every fourth quad of its
+// states, so that a warp reads and writes the states of eight channels as whole lines.
+#include "../common/dtype.cuh"
+#include "../common/host_util.h"
+#include "../common/ptx.cuh"
+#include "../rf_api.h"
+
+namespace rf {
+
+template <typename T> __device__ __forceinline__ float exp2_t(float x);
+template <> __device__ __forceinline__ float exp2_t<float>(float x) { return exp2f(x); }
+template <> __device__ __forceinline__ float exp2_t<__half>(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+template <> __device__ __forceinline__ float exp2_t<__nv_bfloat16>(float x) { return exp2_t<__half>(x); }
+
+// log(1 + exp(v)) = max(v, 0) + log1p(exp(-|v|)); in 16-bit models the second term comes from the special-function units, and
+// from the first terms of the series where 1 + e would drop the digits of e.
+template <typename T> __device__ __forceinline__ float softplus_t(float v) {
+  const float e = __expf(-fabsf(v));
+  const float series = e * (1.f - e * (0.5f - e * (1.f / 3.f - e * (0.25f - e * 0.2f))));
+  return fmaxf(v, 0.f) + (e < 0.0625f ? series : __logf(1.f + e));
+}
+template <> __device__ __forceinline__ float softplus_t<float>(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+template <typename T> __device__ __forceinline__ float silu_t(float v) { return silu_f(v); }
+template <> __device__ __forceinline__ float silu_t<float>(float v) { return v / (1.f + expf(-v)); }
+
+__device__ __forceinline__ void zero8(float (&f)[8]) {
+#pragma unroll
+  for (int j = 0; j < 8; ++j) f[j] = 0.f;
+}
+
+// --------------------------------------------------------------------------------------- causal convolution ----
+// A thread owns eight channels over `tile` consecutive rows of one sequence; the thread of the first rows also replaces the
+// carried inputs.  TAPS = 0: any number of taps, every input read again for each of them.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) conv_silu_kernel(const RfConvSilu p, int tile) {
+  pdl_prologue();
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 8, seq = blockIdx.z;
+  const int q0 = p.rows.q_start ? p.rows.q_start[seq] : seq, n = p.rows.q_len ? p.rows.q_len[seq] : 1;
+  const int t0 = blockIdx.y * tile, t1 = min(n, t0 + tile), taps = TAPS > 0 ? TAPS : p.taps, past = taps - 1;
+  if (c >= p.channels || t0 >= n) return;
+  const bool fresh = p.rows.pos[q0] == 0;
+  T* state = reinterpret_cast<T*>(p.state) + (size_t)(p.rows.slot ? p.rows.slot[seq] : seq) * past * p.channels + c;
+  const T* x = reinterpret_cast<const T*>(p.x) + (size_t)q0 * p.ldx + c;
+  T* y = reinterpret_cast<T*>(p.y) + (size_t)q0 * p.ldy + c;
+  // input at place i of this launch's rows; negative places are carried ones
+  auto input = [&](int i, float (&f)[8]) {
+    if (i >= 0) load8(x + (size_t)i * p.ldx, f);
+    else if (!fresh) load8(state + (size_t)(past + i) * p.channels, f);
+    else zero8(f);
+  };
+  float bias[8];
+  zero8(bias);
+  if (p.bias) load8(p.bias + c, bias);
+  if constexpr (TAPS > 0) {
+    float w[TAPS][8], win[TAPS][8];
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) load8(p.w + (size_t)k * p.channels + c, w[k]);
+#pragma unroll
+    for (int k = 0; k < TAPS - 1; ++k) input(t0 - (TAPS - 1) + k, win[k]);
+#pragma unroll 4
+    for (int t = t0; t < t1; ++t) {
+      load8(x + (size_t)t * p.ldx, win[TAPS - 1]);
+      float a[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        a[j] = bias[j];
+#pragma unroll
+        for (int k = 0; k < TAPS; ++k) a[j] += w[k][j] * win[k][j];
+        a[j] = silu_t<T>(a[j]);
+      }
+      store8(y + (size_t)t * p.ldy, a);
+#pragma unroll
+      for (int k = 0; k < TAPS - 1; ++k)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) win[k][j] = win[k + 1][j];
+    }
+  } else {
+    for (int t = t0; t < t1; ++t) {
+      float a[8], w[8], v[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a[j] = bias[j];
+      for (int k = 0; k < taps; ++k) {
+        load8(p.w + (size_t)k * p.channels + c, w);
+        input(t - past + k, v);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) a[j] += w[j] * v[j];
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a[j] = silu_t<T>(a[j]);
+      store8(y + (size_t)t * p.ldy, a);
+    }
+  }
+  if (blockIdx.y == 0)
+    for (int i = 0; i < past; ++i) {             // ascending: row i comes from a later row of the old state, or from this launch
+      float v[8];
+      input(n - past + i, v);
+      store8(state + (size_t)i * p.channels, v);
+    }
+}
+
+// ------------------------------------------------------------------------------------------- recurrence ----
+constexpr int kMbChannels = 64;       // channels per CTA (256 threads)
+constexpr int kMbRows = 8;            // rows staged in shared memory at a time
+
+// A CTA owns 64 channels of `seqs_per_cta` neighbouring sequences, whose rows are contiguous.  The step size of a row comes
+// from the step-size weights of these channels, kept in shared memory.
+template <typename T, int QPL>
+__global__ void __launch_bounds__(256) mamba_recurrent_kernel(const RfMamba1 p, int seqs_per_cta) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) uint8_t mb_raw[];
+  constexpr int CH = kMbChannels, SP = 16 * QPL;                    // SP: states per channel in shared memory, zero padded
+  const int rank_p = (p.rank + 31) & ~31, wp = rank_p + 8;
+  float* s_dt = reinterpret_cast<float*>(mb_raw);                   // [rows][rank_p]
+  float* s_b = s_dt + kMbRows * rank_p;                             // [rows][SP]
+  float* s_c = s_b + kMbRows * SP;
+  float* s_x = s_c + kMbRows * SP;                                  // [rows][CH]
+  float* s_z = s_x + kMbRows * CH;
+  T* s_w = reinterpret_cast<T*>(s_z + kMbRows * CH);                // [CH][wp]
+  const int tid = threadIdx.x, l = tid & 3, ci = tid >> 2, c0 = blockIdx.x * CH, c = c0 + ci;
+  const bool live = c < p.inner;
+  // the weights do not depend on the previous kernel
+  for (int i = tid; i < CH * (wp / 8); i += 256) {
+    const int r = i / (wp / 8), k = (i % (wp / 8)) * 8;
+    float f[8];
+    zero8(f);
+    if (c0 + r < p.inner && k < p.rank) load8(reinterpret_cast<const T*>(p.w_dt) + (size_t)(c0 + r) * p.rank + k, f);
+    store8(s_w + (size_t)r * wp + k, f);
+  }
+  for (int i = tid; i < kMbRows * (rank_p + 2 * SP); i += 256) s_dt[i] = 0.f;
+  const int nq = p.states / 4;
+  float4 A[QPL];
+#pragma unroll
+  for (int q = 0; q < QPL; ++q)
+    A[q] = live && l + 4 * q < nq ? reinterpret_cast<const float4*>(p.a2 + (size_t)c * p.states)[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
+  const float bias = live ? p.dt_bias[c] : 0.f, D = live ? p.d[c] : 0.f;
+  pdl_wait();
+  const int s0 = blockIdx.y * seqs_per_cta, s1 = min(p.rows.num_seqs, s0 + seqs_per_cta);
+  const int row_begin = p.rows.q_start ? p.rows.q_start[s0] : s0;
+  const int row_end = p.rows.q_start ? p.rows.q_start[s1 - 1] + p.rows.q_len[s1 - 1] : s1;
+  auto state_of = [&](int seq) { return p.state + ((size_t)(p.rows.slot ? p.rows.slot[seq] : seq) * p.inner + c) * p.states; };
+  auto load_state = [&](int seq, float4 (&S)[QPL]) {
+    const bool fresh = p.rows.pos[p.rows.q_start ? p.rows.q_start[seq] : seq] == 0;
+    const float4* st = reinterpret_cast<const float4*>(state_of(seq));
+#pragma unroll
+    for (int q = 0; q < QPL; ++q) S[q] = live && !fresh && l + 4 * q < nq ? st[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
+  };
+  float4 S[QPL], next[QPL];
+  int seq = s0, left = p.rows.q_len ? p.rows.q_len[s0] : 1;
+  load_state(s0, next);
+  bool start = true;
+  for (int r0 = row_begin; r0 < row_end; r0 += kMbRows) {
+    const int nr = min(kMbRows, row_end - r0);
+    __syncthreads();
+    for (int i = tid; i < nr * (p.rank / 8); i += 256) {
+      const int r = i / (p.rank / 8), k = (i % (p.rank / 8)) * 8;
+      float f[8];
+      load8(reinterpret_cast<const T*>(p.bc) + (size_t)(r0 + r) * p.ld_bc + k, f);
+      store8(s_dt + r * rank_p + k, f);
+    }
+    for (int i = tid; i < nr * (p.states / 4); i += 256) {          // B and C: states / 8 pieces each
+      const int r = i / (p.states / 4), k = (i % (p.states / 4)) * 8;
+      const bool is_c = k >= p.states;
+      float f[8];
+      load8(reinterpret_cast<const T*>(p.bc) + (size_t)(r0 + r) * p.ld_bc + p.rank + k, f);
+      store8((is_c ? s_c : s_b) + r * SP + (is_c ? k - p.states : k), f);
+    }
+    for (int i = tid; i < nr * (CH / 8) * 2; i += 256) {
+      const int zi = i & 1, r = (i >> 1) / (CH / 8), k = ((i >> 1) % (CH / 8)) * 8;
+      float f[8];
+      zero8(f);
+      if (c0 + k < p.inner) load8((zi ? reinterpret_cast<const T*>(p.z) + (size_t)(r0 + r) * p.ldz : reinterpret_cast<const T*>(p.x) + (size_t)(r0 + r) * p.ldx) + c0 + k, f);
+      store8((zi ? s_z : s_x) + r * CH + k, f);
+    }
+    __syncthreads();
+    for (int r = 0; r < nr; ++r) {
+      if (start) {
+#pragma unroll
+        for (int q = 0; q < QPL; ++q) S[q] = next[q];
+        if (seq + 1 < s1) load_state(seq + 1, next);
+        start = false;
+      }
+      float dot = 0.f;
+      const T* wr = s_w + (size_t)ci * wp + l * 8;
+      const float* dr = s_dt + r * rank_p + l * 8;
+      for (int k = 0; k < rank_p; k += 32) {
+        float w8[8], d8[8];
+        load8(wr + k, w8);
+        load8(dr + k, d8);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) dot += w8[j] * d8[j];
+      }
+      dot += __shfl_xor_sync(0xffffffffu, dot, 1);
+      dot += __shfl_xor_sync(0xffffffffu, dot, 2);
+      const float dt = softplus_t<T>(dot + bias), x = s_x[r * CH + ci], dx = dt * x;
+      float y = 0.f;
+#pragma unroll
+      for (int q = 0; q < QPL; ++q) {
+        const float4 B = *reinterpret_cast<const float4*>(s_b + r * SP + (l + 4 * q) * 4), C = *reinterpret_cast<const float4*>(s_c + r * SP + (l + 4 * q) * 4);
+        S[q].x = S[q].x * exp2_t<T>(dt * A[q].x) + dx * B.x; y += S[q].x * C.x;
+        S[q].y = S[q].y * exp2_t<T>(dt * A[q].y) + dx * B.y; y += S[q].y * C.y;
+        S[q].z = S[q].z * exp2_t<T>(dt * A[q].z) + dx * B.z; y += S[q].z * C.z;
+        S[q].w = S[q].w * exp2_t<T>(dt * A[q].w) + dx * B.w; y += S[q].w * C.w;
+      }
+      y += __shfl_xor_sync(0xffffffffu, y, 1);
+      y += __shfl_xor_sync(0xffffffffu, y, 2);
+      if (l == 0) s_x[r * CH + ci] = (y + D * x) * silu_t<T>(s_z[r * CH + ci]);     // read by these four lanes only, all of them done
+      if (--left == 0) {
+        float4* st = reinterpret_cast<float4*>(state_of(seq));
+        if (live) {
+#pragma unroll
+          for (int q = 0; q < QPL; ++q)
+            if (l + 4 * q < nq) st[l + 4 * q] = S[q];
+        }
+        if (++seq < s1) left = p.rows.q_len ? p.rows.q_len[seq] : 1;
+        start = true;
+      }
+    }
+    __syncthreads();
+    for (int i = tid; i < nr * (CH / 8); i += 256) {
+      const int r = i / (CH / 8), k = (i % (CH / 8)) * 8;
+      if (c0 + k >= p.inner) continue;
+      float f[8];
+      load8(s_x + r * CH + k, f);
+      store8(reinterpret_cast<T*>(p.out) + (size_t)(r0 + r) * p.ldo + c0 + k, f);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------- scan ----
+constexpr int kScanRows = 32;
+
+// A CTA owns CH channels of one sequence and walks it in tiles of 32 rows: one thread fetches eight channels of one row (the
+// next tile's while the current one is scanned), turns the step sizes and gates once per (row, channel), and the four lanes of a
+// channel run the recurrence, four rows at a time so that the sums over lanes cost three shuffles per four rows.
+template <typename T, int CH, int QPL>
+__global__ void __launch_bounds__(CH * 4) mamba_scan_kernel(const RfMamba1 p) {
+  pdl_prologue();
+  extern __shared__ __align__(16) float sc_sm[];
+  constexpr int SP = 16 * QPL, NT = CH * 4, TR = kScanRows;
+  float* s_dt = sc_sm;                     // [TR][CH] step sizes
+  float* s_dx = s_dt + TR * CH;            // step size times input; then the result
+  float* s_d = s_dx + TR * CH;             // D times input
+  float* s_g = s_d + TR * CH;              // silu(z)
+  float* s_b = s_g + TR * CH;              // [TR][SP]
+  float* s_c = s_b + TR * SP;
+  const int tid = threadIdx.x, l = tid & 3, ci = tid >> 2, c0 = blockIdx.x * CH, c = c0 + ci, seq = blockIdx.y;
+  const int q0 = p.rows.q_start ? p.rows.q_start[seq] : seq, n = p.rows.q_len ? p.rows.q_len[seq] : 1;
+  const int nq = p.states / 4;
+  const bool live = c < p.inner, fresh = p.rows.pos[q0] == 0;
+  for (int i = tid; i < TR * SP * 2; i += NT) s_b[i] = 0.f;
+  float4 A[QPL], S[QPL];
+  float* st = p.state + ((size_t)(p.rows.slot ? p.rows.slot[seq] : seq) * p.inner + (live ? c : 0)) * p.states;
+#pragma unroll
+  for (int q = 0; q < QPL; ++q) {
+    const bool in = live && l + 4 * q < nq;
+    A[q] = in ? reinterpret_cast<const float4*>(p.a2 + (size_t)c * p.states)[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
+    S[q] = in && !fresh ? reinterpret_cast<const float4*>(st)[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  // the thread's piece of a tile
+  const int lr = tid / (CH / 8), lc = (tid % (CH / 8)) * 8;
+  const bool in_c = c0 + lc < p.inner;
+  float bias[8], D[8];
+  zero8(bias); zero8(D);
+  if (in_c) { load8(p.dt_bias + c0 + lc, bias); load8(p.d + c0 + lc, D); }
+  const T* xp = reinterpret_cast<const T*>(p.x) + (size_t)q0 * p.ldx + c0 + lc;
+  const T* zp = reinterpret_cast<const T*>(p.z) + (size_t)q0 * p.ldz + c0 + lc;
+  const T* dp = reinterpret_cast<const T*>(p.dt) + (size_t)q0 * p.ld_dt + c0 + lc;
+  const T* bp = reinterpret_cast<const T*>(p.bc) + (size_t)q0 * p.ld_bc + p.rank;
+  Vec8<T> vx, vz, vd;
+  auto fetch = [&](int t0) {
+    if (t0 + lr < n && in_c) {
+      vx = *reinterpret_cast<const Vec8<T>*>(xp + (size_t)(t0 + lr) * p.ldx);
+      vz = *reinterpret_cast<const Vec8<T>*>(zp + (size_t)(t0 + lr) * p.ldz);
+      vd = *reinterpret_cast<const Vec8<T>*>(dp + (size_t)(t0 + lr) * p.ld_dt);
+    }
+  };
+  fetch(0);
+  for (int t0 = 0; t0 < n; t0 += TR) {
+    const int nr = min(TR, n - t0);
+    __syncthreads();                       // the previous tile's results have left
+    {
+      float dt[8], dx[8], dd[8], g[8];
+      zero8(dt); zero8(dx); zero8(dd); zero8(g);
+      if (lr < nr && in_c) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float2 x2 = Num<T>::to_f2(vx.v[j]), z2 = Num<T>::to_f2(vz.v[j]), d2 = Num<T>::to_f2(vd.v[j]);
+          dt[2 * j] = softplus_t<T>(d2.x + bias[2 * j]); dt[2 * j + 1] = softplus_t<T>(d2.y + bias[2 * j + 1]);
+          dx[2 * j] = dt[2 * j] * x2.x; dx[2 * j + 1] = dt[2 * j + 1] * x2.y;
+          dd[2 * j] = D[2 * j] * x2.x; dd[2 * j + 1] = D[2 * j + 1] * x2.y;
+          g[2 * j] = silu_t<T>(z2.x); g[2 * j + 1] = silu_t<T>(z2.y);
+        }
+      }
+      store8(s_dt + lr * CH + lc, dt);     // rows behind the end: step size 0 leaves the state as it is
+      store8(s_dx + lr * CH + lc, dx);
+      store8(s_d + lr * CH + lc, dd);
+      store8(s_g + lr * CH + lc, g);
+    }
+    for (int i = tid; i < TR * (p.states / 4); i += NT) {
+      const int r = i / (p.states / 4), k = (i % (p.states / 4)) * 8;
+      const bool is_c = k >= p.states;
+      float f[8];
+      zero8(f);
+      if (r < nr) load8(bp + (size_t)(t0 + r) * p.ld_bc + k, f);
+      store8((is_c ? s_c : s_b) + r * SP + (is_c ? k - p.states : k), f);
+    }
+    __syncthreads();
+    if (t0 + TR < n) fetch(t0 + TR);
+    for (int t = 0; t < nr; t += 4) {
+      float v[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const float dt = s_dt[(t + u) * CH + ci], dx = s_dx[(t + u) * CH + ci];
+        v[u] = 0.f;
+#pragma unroll
+        for (int q = 0; q < QPL; ++q) {
+          const float4 B = *reinterpret_cast<const float4*>(s_b + (t + u) * SP + (l + 4 * q) * 4), C = *reinterpret_cast<const float4*>(s_c + (t + u) * SP + (l + 4 * q) * 4);
+          S[q].x = S[q].x * exp2_t<T>(dt * A[q].x) + dx * B.x; v[u] += S[q].x * C.x;
+          S[q].y = S[q].y * exp2_t<T>(dt * A[q].y) + dx * B.y; v[u] += S[q].y * C.y;
+          S[q].z = S[q].z * exp2_t<T>(dt * A[q].z) + dx * B.z; v[u] += S[q].z * C.z;
+          S[q].w = S[q].w * exp2_t<T>(dt * A[q].w) + dx * B.w; v[u] += S[q].w * C.w;
+        }
+      }
+      // lane l ends with the sum of row t + l: swap halves with the lane two away, then with the neighbour
+      const bool hi = l & 2, odd = l & 1;
+      const float a0 = __shfl_xor_sync(0xffffffffu, hi ? v[0] : v[2], 2), a1 = __shfl_xor_sync(0xffffffffu, hi ? v[1] : v[3], 2);
+      const float w0 = (hi ? v[2] : v[0]) + a0, w1 = (hi ? v[3] : v[1]) + a1;
+      const float y = (odd ? w1 : w0) + __shfl_xor_sync(0xffffffffu, odd ? w0 : w1, 1);
+      const int at = (t + l) * CH + ci;
+      s_dx[at] = (y + s_d[at]) * s_g[at];
+    }
+    __syncthreads();
+    if (lr < nr && in_c) {
+      float f[8];
+      load8(s_dx + lr * CH + lc, f);
+      store8(reinterpret_cast<T*>(p.out) + (size_t)(q0 + t0 + lr) * p.ldo + c0 + lc, f);
+    }
+  }
+  if (live) {
+#pragma unroll
+    for (int q = 0; q < QPL; ++q)
+      if (l + 4 * q < nq) reinterpret_cast<float4*>(st)[l + 4 * q] = S[q];
+  }
+}
+
+// ------------------------------------------------------------------------------------------------- host ----
+static int check_mamba(const RfMamba1* a) {
+  RF_REQUIRE(a && a->x && a->z && a->bc && a->dt_bias && a->a2 && a->d && a->state && a->out && a->rows.pos, "mamba: missing buffers");
+  RF_REQUIRE(a->inner > 0 && a->inner % 8 == 0 && a->states > 0 && a->states % 8 == 0 && a->states <= 256 && a->rank > 0 && a->rank % 8 == 0,
+             "mamba: %d channels, %d states, step rank %d", a->inner, a->states, a->rank);
+  RF_REQUIRE(a->ldx % 8 == 0 && a->ldz % 8 == 0 && a->ld_bc % 8 == 0 && a->ldo % 8 == 0, "mamba: pitches must be multiples of 8");
+  RF_REQUIRE(a->dtype >= 0 && a->dtype <= 2, "mamba: dtype %d", a->dtype);
+  return RF_OK;
+}
+
+template <typename T, int QPL>
+static int launch_recurrent(const RfMamba1* a, cudaStream_t s) {
+  const int tiles = ceil_div(a->inner, kMbChannels), seqs = a->rows.num_seqs;
+  // share the step-size weights of a channel tile between sequences once there are enough CTAs without it
+  const int spc = std::max(1, std::min(8, seqs * tiles / (6 * sm_count())));
+  const int rank_p = (a->rank + 31) & ~31;
+  const size_t smem = (size_t)kMbRows * (rank_p + 32 * QPL + 2 * kMbChannels) * sizeof(float) + (size_t)kMbChannels * (rank_p + 8) * sizeof(T);
+  RF_REQUIRE(smem <= 200 * 1024, "mamba: a step rank of %d does not fit in shared memory", a->rank);
+  RF_ALLOW_SMEM_PER_DEVICE((mamba_recurrent_kernel<T, QPL>), 200 * 1024);
+  RF_CUDA_CHECK(::rf::launch_k(mamba_recurrent_kernel<T, QPL>, dim3(tiles, ceil_div(seqs, spc)), dim3(256), smem, s, 1, *a, spc));
+  ::rf::count_launch();
+  return RF_OK;
+}
+
+template <typename T, int QPL>
+static int launch_scan(const RfMamba1* a, cudaStream_t s) {
+  const int seqs = a->rows.num_seqs;
+  const size_t per = (size_t)kScanRows * 32 * QPL * sizeof(float);
+  if (ceil_div(a->inner, 64) * seqs >= sm_count()) {
+    const size_t smem = (size_t)kScanRows * 64 * 4 * sizeof(float) + per;
+    RF_ALLOW_SMEM_PER_DEVICE((mamba_scan_kernel<T, 64, QPL>), 128 * 1024);
+    RF_CUDA_CHECK(::rf::launch_k(mamba_scan_kernel<T, 64, QPL>, dim3(ceil_div(a->inner, 64), seqs), dim3(256), smem, s, 1, *a));
+  } else {
+    const size_t smem = (size_t)kScanRows * 32 * 4 * sizeof(float) + per;
+    RF_ALLOW_SMEM_PER_DEVICE((mamba_scan_kernel<T, 32, QPL>), 128 * 1024);
+    RF_CUDA_CHECK(::rf::launch_k(mamba_scan_kernel<T, 32, QPL>, dim3(ceil_div(a->inner, 32), seqs), dim3(128), smem, s, 1, *a));
+  }
+  ::rf::count_launch();
+  return RF_OK;
+}
+
+}  // namespace rf
+
+using namespace rf;
+
+#define RF_MAMBA_STATES(T, FN)                  \
+  {                                             \
+    const int q = (a->states + 15) / 16;        \
+    if (q <= 1) return FN<T, 1>(a, s);          \
+    if (q <= 2) return FN<T, 2>(a, s);          \
+    if (q <= 4) return FN<T, 4>(a, s);          \
+    if (q <= 8) return FN<T, 8>(a, s);          \
+    return FN<T, 16>(a, s);                     \
+  }
+#define RF_MAMBA_DISPATCH(FN)                                   \
+  cudaStream_t s = static_cast<cudaStream_t>(stream);           \
+  if (a->dtype == kF16) RF_MAMBA_STATES(__half, FN)             \
+  if (a->dtype == kBF16) RF_MAMBA_STATES(__nv_bfloat16, FN)     \
+  RF_MAMBA_STATES(float, FN)
+
+extern "C" int rf_mamba1_recurrent(const RfMamba1* a, rf_stream_t stream) {
+  RF_SKIP_IF_REPLAYING();
+  int rc = check_mamba(a);
+  if (rc) return rc;
+  RF_REQUIRE(a->w_dt, "mamba recurrence: step-size weights");
+  if (a->rows.num_seqs == 0) return RF_OK;
+  RF_MAMBA_DISPATCH(launch_recurrent)
+}
+
+extern "C" int rf_mamba1_scan(const RfMamba1* a, rf_stream_t stream) {
+  RF_SKIP_IF_REPLAYING();
+  int rc = check_mamba(a);
+  if (rc) return rc;
+  RF_REQUIRE(a->dt && a->ld_dt % 8 == 0, "mamba scan: step-size rows");
+  RF_REQUIRE(a->rows.num_seqs <= 65535, "mamba scan: %d sequences", a->rows.num_seqs);
+  if (a->rows.num_seqs == 0) return RF_OK;
+  RF_MAMBA_DISPATCH(launch_scan)
+}
+
+extern "C" int rf_conv_silu(const RfConvSilu* a, rf_stream_t stream) {
+  RF_SKIP_IF_REPLAYING();
+  RF_REQUIRE(a && a->x && a->y && a->w && a->rows.pos && (a->taps == 1 || a->state), "conv_silu: missing buffers");
+  RF_REQUIRE(a->channels > 0 && a->channels % 8 == 0 && a->ldx % 8 == 0 && a->ldy % 8 == 0 && a->taps >= 1, "conv_silu: %d channels, %d taps",
+             a->channels, a->taps);
+  RF_REQUIRE(a->dtype >= 0 && a->dtype <= 2 && a->x != a->y && a->max_q_len >= 1 && a->rows.num_seqs <= 65535, "conv_silu: options");
+  if (a->rows.num_seqs == 0) return RF_OK;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const int tile = std::max(16, a->taps - 1);      // later tiles find their past in the rows of this launch
+  const dim3 grid(ceil_div(a->channels, 1024), ceil_div(a->max_q_len, tile), a->rows.num_seqs);
+#define RF_CONV(T)                                                                                                       \
+  switch (a->taps) {                                                                                                     \
+    case 2: RF_CUDA_CHECK(::rf::launch_k(conv_silu_kernel<T, 2>, grid, dim3(128), 0, s, 1, *a, tile)); break;            \
+    case 3: RF_CUDA_CHECK(::rf::launch_k(conv_silu_kernel<T, 3>, grid, dim3(128), 0, s, 1, *a, tile)); break;            \
+    case 4: RF_CUDA_CHECK(::rf::launch_k(conv_silu_kernel<T, 4>, grid, dim3(128), 0, s, 1, *a, tile)); break;            \
+    default: RF_CUDA_CHECK(::rf::launch_k(conv_silu_kernel<T, 0>, grid, dim3(128), 0, s, 1, *a, tile)); break;           \
+  }
+  if (a->dtype == kF16) { RF_CONV(__half) } else if (a->dtype == kBF16) { RF_CONV(__nv_bfloat16) } else { RF_CONV(float) }
+#undef RF_CONV
+  ::rf::count_launch();
+  return RF_OK;
+}

@@ -30,6 +30,22 @@ __device__ __forceinline__ void store4(T* p, float4 f) {
   q.v[0] = Num<T>::from_f(f.x); q.v[1] = Num<T>::from_f(f.y); q.v[2] = Num<T>::from_f(f.z); q.v[3] = Num<T>::from_f(f.w);
   *reinterpret_cast<Quad<T>*>(p) = q;
 }
+// four columns of the outstanding output of row `src`: one row, or the sum of the picked ones
+template <typename T>
+__device__ __forceinline__ float4 pending4(const RfStreamNorm& p, const T* y, int src, int col) {
+  if (p.y_picks <= 0) return load4(y + (size_t)src * p.H + col);
+  float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+  const int32_t* slots = p.y_slots + (size_t)src * p.y_picks;
+#pragma unroll 4
+  for (int j = 0; j < p.y_picks; ++j) {
+    const int r = slots[j];
+    if (r < 0) continue;
+    const float4 v = load4(y + (size_t)r * p.H + col);
+    s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
+  }
+  return s;
+}
+__device__ __forceinline__ float4 mul4(float4 v, float f) { return make_float4(v.x * f, v.y * f, v.z * f, v.w * f); }
 __device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
 
 // A CTA walks rows_per_cta neighbouring rows.  A thread always touches the same columns, so the shared copies of the
@@ -52,16 +68,16 @@ __global__ void stream_norm_kernel(const RfStreamNorm p, int rows_per_cta) {
     float yr = 1.f;
     if (y && p.y_norm_w) {
       float s = 0.f;
-      for (int i = c0; i < H; i += step) s += sq4(load4(y + (size_t)src * H + i));
+      for (int i = c0; i < H; i += step) s += sq4(pending4(p, y, src, i));
       yr = rsqrtf(stream_block_sum(s, red) * inv_dim + p.eps);
     }
     const float* xr = p.x ? p.x + (size_t)src * H : nullptr;
     const T* er = p.x ? nullptr : table + (size_t)p.ids[src] * H;
     float s = 0.f;
     for (int i = c0; i < H; i += step) {
-      float4 v = xr ? *reinterpret_cast<const float4*>(xr + i) : load4(er + i);
+      float4 v = xr ? *reinterpret_cast<const float4*>(xr + i) : mul4(load4(er + i), p.embed_scale);
       if (y) {
-        float4 a = load4(y + (size_t)src * H + i);
+        float4 a = pending4(p, y, src, i);
         if (p.y_norm_w) {
           const float4 w = *reinterpret_cast<const float4*>(p.y_norm_w + i);
           a.x *= yr * w.x; a.y *= yr * w.y; a.z *= yr * w.z; a.w *= yr * w.w;
@@ -162,8 +178,8 @@ __global__ void __launch_bounds__(VPT == 4 ? 512 : 1024) stream_norm_reg_kernel(
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
       const bool in = col(k) < H;
-      v[k] = !in ? zero : p.x ? *reinterpret_cast<const float4*>(p.x + (size_t)src * H + col(k)) : load4(table + (size_t)p.ids[src] * H + col(k));
-      a[k] = y && in ? load4(y + (size_t)src * H + col(k)) : zero;
+      v[k] = !in ? zero : p.x ? *reinterpret_cast<const float4*>(p.x + (size_t)src * H + col(k)) : mul4(load4(table + (size_t)p.ids[src] * H + col(k)), p.embed_scale);
+      a[k] = y && in ? pending4(p, y, src, col(k)) : zero;
     }
   };
   // v <- v + pending output; returns 1 / rms when the row is normalised
@@ -313,8 +329,13 @@ using namespace rf;
   else if ((dtype) == kBF16) { using T = __nv_bfloat16; __VA_ARGS__; }  \
   else { using T = float; __VA_ARGS__; }
 
-extern "C" int rf_stream_norm(const RfStreamNorm* a, rf_stream_t stream) {
+extern "C" int rf_stream_norm(const RfStreamNorm* args, rf_stream_t stream) {
   RF_SKIP_IF_REPLAYING();
+  RF_REQUIRE(args != nullptr, "stream_norm: null arguments");
+  RfStreamNorm filled = *args;
+  if (filled.embed_scale == 0.f) filled.embed_scale = 1.f;
+  const RfStreamNorm* a = &filled;
+  RF_REQUIRE(a->y_picks <= 0 || (a->y && a->y_slots), "stream_norm: picked rows need y and y_slots");
   RF_REQUIRE(a && a->H > 0 && a->H % 8 == 0 && a->dim > 0 && a->dim <= a->H, "stream_norm: row length");
   RF_REQUIRE(a->x || (a->table && a->ids), "stream_norm: no input");
   RF_REQUIRE(!a->norm_w || a->out, "stream_norm: no output");

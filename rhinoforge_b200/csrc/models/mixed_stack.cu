@@ -31,27 +31,49 @@ struct MixedStack {
   uint8_t* base = nullptr;
   uint64_t off_x[2] = {}, off_h = 0, off_cast = 0, off_wide = 0, off_mix = 0, off_y = 0, off_side = 0, off_qlat = 0, off_olat = 0,
            off_ctx = 0, off_kv = 0, off_kvmeta = 0, off_attn_ws = 0, off_head = 0, off_argmax = 0, off_sk_ws = 0, off_sk_flags = 0,
-           off_status = 0, total = 0;
-  uint64_t attn_ws_bytes = 0, argmax_bytes = 0, sk_ws_bytes = 0;
+           off_status = 0, off_vfirst = 0, off_conv = 0, off_bc = 0, off_dt = 0, off_moe = 0, off_xg = 0, off_hg = 0, off_yg = 0, total = 0;
+  uint64_t attn_ws_bytes = 0, argmax_bytes = 0, sk_ws_bytes = 0, rows_ws_bytes = 0;
+  int moe_tiles = 0;      // tile-list entries of any mixture-of-experts layer
   int lat_rows = 0;       // rows one latent-space attention launch takes
   int ctx_rows = 0;       // rows of expanded keys / values one group of portions takes
   int cur = 0;            // which stream buffer holds the last forward's rows
-  bool side_pending = false;
+  // the sublayer output that is still to be added behind the last layer
+  struct Pending { const void* y = nullptr; const float* norm = nullptr; const int32_t* slots = nullptr; int picks = 0; } tail;
+  const int32_t* full_len = nullptr;      // device: cached tokens, new ones included, of every prefill-sized sequence
+  int max_full = 0, max_long_q = 0;
   bool planned = false;
   static constexpr int kSkFlags = 1024;
+  static constexpr int kMoeSmallRows = 256;   // up to here the experts' weights are streamed past the rows
 
   size_t esz() const { return cfg.dtype == kF32 ? 4 : 2; }
   bool fp32() const { return cfg.dtype == kF32; }
   template <typename P = void> P* at(uint64_t off) const { return reinterpret_cast<P*>(base + off); }
+  static int moe_ld(const RfMixedLayer& l) { return std::max(l.bank_inter, l.shared_inter); }
   int32_t* status() const { return base ? at<int32_t>(off_status) : nullptr; }
 
   void plan() {
     auto al = [](uint64_t v) { return (v + 1023) & ~uint64_t(1023); };
     const uint64_t T = (uint64_t)cfg.max_tokens, H = (uint64_t)cfg.hidden, e = esz();
     uint64_t wide = 8, mix = 8, lat = 0, rank = 0, kvw = 0, past = 0, heads = 0;
+    uint64_t vfirst = 0, inner = 0, bc = 0, picks = 0, experts = 0, hg = 0;
+    rows_ws_bytes = 0; moe_tiles = 0;
     for (const RfMixedLayer& l : layers) {
       wide = std::max<uint64_t>(wide, std::max(l.in_dim, l.inter));
-      mix = std::max<uint64_t>(mix, (uint64_t)l.heads * l.vdim);
+      mix = std::max<uint64_t>(mix, (uint64_t)l.out_dim);
+      if (l.mixer == RF_MIXER_ATTENTION) {
+        vfirst = std::max<uint64_t>(vfirst, (uint64_t)l.kv_heads * l.vdim);
+        if (l.tensor_core) rows_ws_bytes = std::max<uint64_t>(rows_ws_bytes, rf_attn_decode_scratch_bound(l.heads, l.kv_heads, l.dim));
+      }
+      if (l.mixer == RF_MIXER_MAMBA1) {
+        inner = std::max<uint64_t>(inner, l.inner);
+        bc = std::max<uint64_t>(bc, l.dt_rank + 2 * l.states);
+      }
+      if (l.experts > 0) {
+        picks = std::max<uint64_t>(picks, l.top + 1);
+        experts = std::max<uint64_t>(experts, l.experts);
+        hg = std::max<uint64_t>(hg, moe_ld(l));
+        moe_tiles = std::max(moe_tiles, l.experts + (int)(T * (l.top + 1) / 16) + 2);
+      }
       if (l.mixer != RF_MIXER_LATENT_ATTENTION) continue;
       lat = std::max<uint64_t>(lat, (uint64_t)l.heads * l.rank);
       rank = std::max<uint64_t>(rank, l.rank);
@@ -81,10 +103,20 @@ struct MixedStack {
     off_qlat = o; o += al((uint64_t)lat_rows * lat * e);
     off_olat = o; o += al((uint64_t)lat_rows * lat * e);
     attn_ws_bytes = lat ? rf_latent_attn_scratch_bytes(lat_rows, (int)heads, (int)rank, cfg.max_seq_len) : 0;
+    attn_ws_bytes = std::max(attn_ws_bytes, rows_ws_bytes);
     off_attn_ws = o; o += al(attn_ws_bytes);
     off_ctx = o; o += al(kvw ? (uint64_t)ctx_rows * rank * e : 0);
     off_kv = o; o += al((uint64_t)ctx_rows * kvw * e);
-    off_kvmeta = o; o += al((uint64_t)cfg.max_seqs * 2 * windows.size() * sizeof(int32_t));
+    off_kvmeta = o; o += al((uint64_t)cfg.max_seqs * (2 * windows.size() + 1) * sizeof(int32_t));
+    off_vfirst = o; o += al(T * vfirst * e);
+    off_conv = o; o += al(T * inner * e);
+    off_bc = o; o += al(T * bc * e);
+    off_dt = o; o += al(fp32() ? 0 : T * inner * e);
+    // ids, weights, rank | slot_of, token_of_slot, slot_w (one column more) | counters, start | tile list
+    off_moe = o; o += al(picks ? (6 * T * picks + 2 * (experts + 4) + 8 + 4ull * moe_tiles) * 4 : 0);
+    off_xg = o; o += al(fp32() || !picks ? 0 : T * (picks - 1) * H * e);
+    off_hg = o; o += al(T * picks * hg * e);
+    off_yg = o; o += al(T * picks * H * e);
     off_head = o; o += al((uint64_t)std::max(cfg.max_seqs, 64) * H * e);
     argmax_bytes = rf_argmax_scratch_bytes(std::max(cfg.max_seqs, 64), cfg.vocab);
     off_argmax = o; o += al(argmax_bytes);
@@ -156,7 +188,7 @@ static int latent_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedF
   uint8_t* wide = s.at<uint8_t>(s.off_wide);
   int rc = linear(s, h, H, w.w_in, wide, w.in_dim, T, w.in_dim, H, kActNone, st);
   if (rc) return rc;
-  RfLatentInsert ins = {wide + (size_t)QD * e, w.in_dim, w.latent_norm, w.latent_pool, f.rows, T, w.rank, w.rank_true, c.eps};
+  RfLatentInsert ins = {wide + (size_t)QD * e, w.in_dim, w.latent_norm, w.st.latent_pool, f.rows, T, w.rank, w.rank_true, c.eps};
   // ---- decode rows and short portions (and everything without an expanded form): in the latent space
   const bool expand = w.expand_hd > 0 && f.short_seqs < f.rows.num_seqs;
   const int lat_total = expand ? f.short_rows : T;
@@ -173,7 +205,7 @@ static int latent_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedF
     rc = r0 == 0 ? rf_latent_absorb(&q, &ins, st) : rf_head_linear(&q, st);      // every row is cached before the first attends
     if (rc) return rc;
     RfLatentAttn a = {};
-    a.q = s.at(s.off_qlat); a.o = s.at(s.off_olat); a.pool = w.latent_pool;
+    a.q = s.at(s.off_qlat); a.o = s.at(s.off_olat); a.pool = w.st.latent_pool;
     a.rows = f.rows; a.rows.pos += r0;
     if (a.rows.seq_of_row) a.rows.seq_of_row += r0;
     else if (a.rows.slot) a.rows.slot += r0;
@@ -203,7 +235,7 @@ static int latent_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedF
     void* ctx = s.at(s.off_ctx);
     uint8_t* kv = s.at<uint8_t>(s.off_kv);
     const int KD = w.heads * w.expand_hd, KV = 2 * KD;
-    rc = rf_latent_gather(w.latent_pool, ctx, &g, kv_start, kv_len, w.rank, grp.max_len, c.dtype, st);
+    rc = rf_latent_gather(w.st.latent_pool, ctx, &g, kv_start, kv_len, w.rank, grp.max_len, c.dtype, st);
     if (rc) return rc;
     rc = linear(s, ctx, w.rank, w.w_expand, kv, KV, grp.total, KV, w.rank, kActNone, st);
     if (rc) return rc;
@@ -223,9 +255,17 @@ static int latent_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedF
 // Group the prefill-sized sequences of this forward per window and upload their key ranges.
 static int plan_windows(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
   const int n = f.rows.num_seqs - f.short_seqs;
-  if (n <= 0 || s.windows.empty()) return RF_OK;
+  if (n <= 0) return RF_OK;
   int32_t* dev = s.at<int32_t>(s.off_kvmeta);
-  std::vector<int32_t> host((size_t)s.windows.size() * 2 * n);
+  std::vector<int32_t> host((s.windows.size() * 2 + 1) * n);
+  s.full_len = dev + s.windows.size() * 2 * n;
+  s.max_full = s.max_long_q = 0;
+  for (int j = 0; j < n; ++j) {
+    const int q = f.h_q_len[f.short_seqs + j], len = f.h_pos0[f.short_seqs + j] + q;
+    host[s.windows.size() * 2 * n + j] = len;
+    s.max_full = std::max(s.max_full, len);
+    s.max_long_q = std::max(s.max_long_q, q);
+  }
   for (size_t i = 0; i < s.windows.size(); ++i) {
     WindowPlan& p = s.windows[i];
     int32_t* start = host.data() + i * 2 * n;
@@ -258,7 +298,7 @@ static int hgrn2(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f, 
   RfHgrn2 a = {};
   a.x = wide; a.ldx = w.in_dim; a.f_off = w.heads * w.dim; a.v_off = 2 * w.heads * w.dim;
   a.f_bias = w.f_bias; a.lower = w.lower; a.norm_w = w.head_norm;
-  a.state = w.rec_state; a.out = mix; a.ldo = (int64_t)w.heads * w.vdim;
+  a.state = w.st.rec_state; a.out = mix; a.ldo = (int64_t)w.heads * w.vdim;
   a.heads = w.heads; a.dim = w.dim; a.vdim = w.vdim; a.vdim_true = w.vdim_true; a.eps = c.eps; a.dtype = c.dtype;
   a.status = s.status();
   const bool chunked = rf_hgrn2_chunked_supported(w.dim, w.vdim, c.dtype) != 0;
@@ -275,6 +315,158 @@ static int hgrn2(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f, 
   return rc;
 }
 
+static int grouped_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f, const void* h, void* mix, cudaStream_t st) {
+  const RfMixedConfig& c = s.cfg;
+  const int T = f.tokens, H = c.hidden, hd = w.dim, QD = w.heads * hd, KD = w.kv_heads * hd;
+  const size_t e = s.esz();
+  uint8_t* wide = s.at<uint8_t>(s.off_wide);
+  int rc = linear(s, h, H, w.w_in, wide, w.in_dim, T, w.in_dim, H, kActNone, st);
+  if (rc) return rc;
+  RfQkvInsert q = {};
+  q.qkv = wide; q.ld = w.in_dim; q.k_off = QD; q.v_off = QD + KD;
+  q.q_norm = w.q_norm; q.k_norm = w.k_norm; q.cos = w.cos; q.sin = w.sin;
+  q.v_first = s.at(s.off_vfirst); q.k_pool = w.st.k_pool; q.v_pool = w.st.v_pool; q.rows = f.rows;
+  q.n_rows = T; q.heads = w.heads; q.kv_heads = w.kv_heads; q.hd = hd; q.dim = w.dim_true; q.vdim = w.vdim_true;
+  q.rot_dims = w.rot_dims; q.v_role = w.v_role; q.v_lambda = w.v_lambda; q.eps = c.eps; q.dtype = c.dtype;
+  rc = rf_qkv_insert(&q, st);
+  if (rc) return rc;
+  RfAttn a = {};
+  a.q = wide; a.ldq = w.in_dim; a.out = mix; a.ldo = QD; a.q_rows_total = T;
+  a.k_pool = w.st.k_pool; a.v_pool = w.st.v_pool; a.pool_pages = w.st.pool_pages;
+  a.page_table = f.rows.page_table; a.pt_stride = f.rows.pt_stride;
+  a.Hq = w.heads; a.Hkv = w.kv_heads; a.hd = hd; a.scale = w.scale; a.chunk = w.chunk; a.sink = w.sink;
+  if (w.gated) { a.gate = wide + (size_t)(QD + 2 * KD) * e; a.ld_gate = w.in_dim; }
+  a.status = s.status(); a.dtype = c.dtype;
+  // ---- decoded rows and short portions, by row (without a tensor-core form: every row)
+  const int by_row = w.tensor_core ? f.short_rows : T;
+  for (int r0 = 0; r0 < by_row; r0 += 32768) {
+    RfAttn b = a;
+    b.num_seqs = std::min(32768, by_row - r0);
+    b.q = wide + (size_t)r0 * w.in_dim * e; b.out = (uint8_t*)mix + (size_t)r0 * QD * e;
+    if (a.gate) b.gate = (const uint8_t*)a.gate + (size_t)r0 * w.in_dim * e;
+    b.pos = f.rows.pos + r0; b.seq_of_row = f.rows.seq_of_row ? f.rows.seq_of_row + r0 : nullptr;
+    b.slot = f.rows.slot ? f.rows.slot + (b.seq_of_row ? 0 : r0) : nullptr;
+    RF_REQUIRE(r0 == 0 || b.slot, "mixed stack: %d decode rows need slots", by_row);
+    b.max_kv_len = f.max_kv; b.ws = s.at<float>(s.off_attn_ws); b.ws_bytes = s.attn_ws_bytes;
+    rc = w.tensor_core ? rf_attn_decode(&b, st) : rf_attn_rows(&b, st);
+    if (rc) return rc;
+  }
+  const int n_long = f.rows.num_seqs - f.short_seqs;
+  if (!w.tensor_core || n_long <= 0) return RF_OK;
+  const RfRows g = sub_rows(f.rows, f.short_seqs, n_long);
+  a.num_seqs = n_long; a.q_start = g.q_start; a.q_len = g.q_len; a.slot = g.slot; a.kv_len = s.full_len;
+  a.max_q_len = s.max_long_q; a.max_kv_len = s.max_full; a.causal = 1;
+  return rf_attn_prefill(&a, st);
+}
+
+static int mamba1(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f, const void* h, void* mix, cudaStream_t st) {
+  const RfMixedConfig& c = s.cfg;
+  const int T = f.tokens, H = c.hidden, BC = w.dt_rank + 2 * w.states;
+  const size_t e = s.esz();
+  uint8_t* wide = s.at<uint8_t>(s.off_wide);
+  void* conv = s.at(s.off_conv);
+  uint8_t* bc = s.at<uint8_t>(s.off_bc);
+  uint8_t* dt = s.at<uint8_t>(s.off_dt);
+  int rc = linear(s, h, H, w.w_in, wide, w.in_dim, T, w.in_dim, H, kActNone, st);
+  if (rc) return rc;
+  RfConvSilu cv = {};
+  cv.x = wide; cv.ldx = w.in_dim; cv.y = conv; cv.ldy = w.inner; cv.w = w.conv_w; cv.bias = w.conv_b; cv.state = w.st.conv_state;
+  cv.rows = f.rows; cv.channels = w.inner; cv.taps = w.taps; cv.dtype = c.dtype; cv.max_q_len = 1;
+  if (!f.decode)
+    for (int i = 0; i < f.rows.num_seqs; ++i) cv.max_q_len = std::max(cv.max_q_len, (int)f.h_q_len[i]);
+  rc = rf_conv_silu(&cv, st);
+  if (rc) return rc;
+  rc = linear(s, conv, w.inner, w.w_x, bc, BC, T, BC, w.inner, kActNone, st);
+  if (rc) return rc;
+  RfMamba1 a = {};
+  a.x = conv; a.ldx = w.inner; a.z = wide + (size_t)w.inner * e; a.ldz = w.in_dim; a.bc = bc; a.ld_bc = BC;
+  a.dt = dt; a.ld_dt = w.inner; a.w_dt = w.w_dt_rows; a.dt_bias = w.dt_bias; a.a2 = w.a2; a.d = w.d_skip;
+  a.state = w.st.rec_state; a.out = mix; a.ldo = w.inner;
+  a.inner = w.inner; a.states = w.states; a.rank = w.dt_rank; a.dtype = c.dtype;
+  const int n_rec = s.fp32() ? f.rows.num_seqs : f.short_seqs;
+  if (n_rec > 0) {
+    a.rows = sub_rows(f.rows, 0, n_rec);
+    rc = rf_mamba1_recurrent(&a, st);
+    if (rc) return rc;
+  }
+  if (n_rec < f.rows.num_seqs) {
+    const int r0 = f.short_rows;
+    rc = linear(s, bc + (size_t)r0 * BC * e, BC, w.w_dt, dt + (size_t)r0 * w.inner * e, w.inner, T - r0, w.inner, w.dt_rank, kActNone, st);
+    if (rc) return rc;
+    a.rows = sub_rows(f.rows, n_rec, f.rows.num_seqs - n_rec);
+    rc = rf_mamba1_scan(&a, st);
+  }
+  return rc;
+}
+
+// The experts' results stay where they are, one row per pick; the next stream step adds them up (see RfStreamNorm.y_slots).
+static int experts(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f, const void* h, MixedStack::Pending* out, cudaStream_t st) {
+  const RfMixedConfig& c = s.cfg;
+  const int T = f.tokens, H = c.hidden, E = w.experts, k = w.top, pairs = T * k, has_shared = w.shared_inter > 0, cols = k + has_shared;
+  const size_t e = s.esz();
+  const int ldh = MixedStack::moe_ld(w), bank_rt = ceil_div(w.bank_inter, 128), kbH = ceil_div(H, 64);
+  int32_t* m = s.at<int32_t>(s.off_moe);
+  RfMoeRouter r = {};
+  r.x = h; r.ldx = H; r.w = w.router; r.correction = w.correction;
+  r.counters = m; m += E + 4;
+  r.start = m; m += E + 4;
+  m = s.at<int32_t>(s.off_moe) + ((m - s.at<int32_t>(s.off_moe) + 3) & ~3);
+  r.tiles = m; m += 4 + 4 * s.moe_tiles;
+  r.ids = m; m += pairs;
+  r.weights = (float*)m; m += pairs;
+  r.rank = m; m += pairs;
+  r.slot_of = m; m += T * cols;
+  r.token_of_slot = m; m += T * cols;
+  r.slot_w = (float*)m;
+  r.rows = T; r.experts = E; r.width = H; r.k = k; r.groups = w.groups; r.keep = w.keep; r.score_fn = w.score_fn;
+  r.norm_topk = w.norm_topk; r.scale = w.route_scale; r.slot_ld = cols; r.has_shared = has_shared; r.dtype = c.dtype;
+  uint8_t* hg = s.at<uint8_t>(s.off_hg);
+  uint8_t* yg = s.at<uint8_t>(s.off_yg);
+  out->y = yg; out->slots = r.slot_of; out->picks = cols;
+  if (s.fp32() || T <= MixedStack::kMoeSmallRows) {
+    r.tile_rows = s.fp32() ? 64 : (pairs <= 16 * E ? 16 : 32);
+    r.shared_tiles = has_shared; r.scatter = 1;
+    int rc = rf_moe_router(&r, st);
+    if (rc) return rc;
+    RfMoeExperts x = {};
+    x.tiles = r.tiles; x.experts = E; x.tile_rows = r.tile_rows; x.dtype = c.dtype;
+    x.max_tiles = std::min(E, pairs) + pairs / r.tile_rows + (has_shared ? ceil_div(T, r.tile_rows) : 0);
+    x.x = h; x.ldx = H; x.token_of_slot = r.token_of_slot; x.w = w.w_up; x.w_shared = w.shared_up; x.out = hg; x.ldo = ldh;
+    x.n = w.inter; x.k = H; x.dual = 1;
+    x.bank_section_row_tiles = E * bank_rt; x.bank_kb_total = kbH; x.rt_per_expert = bank_rt;
+    if (has_shared) { x.shared_n = w.shared_inter; x.shared_k = H; x.shared_section_row_tiles = ceil_div(w.shared_inter, 128); x.shared_kb_total = kbH; }
+    rc = rf_moe_experts(&x, st);
+    if (rc) return rc;
+    x.x = hg; x.ldx = ldh; x.token_of_slot = nullptr; x.slot_w = r.slot_w; x.w = w.w_down; x.w_shared = w.shared_down; x.out = yg; x.ldo = H;
+    x.n = H; x.k = w.inter; x.dual = 0;
+    x.bank_section_row_tiles = 0; x.bank_kb_total = E * w.bank_inter / 64; x.rt_per_expert = 0; x.kb_per_expert = w.bank_inter / 64;
+    if (has_shared) { x.shared_n = H; x.shared_k = w.shared_inter; x.shared_section_row_tiles = 0; x.shared_kb_total = ceil_div(w.shared_inter, 64); }
+    return rf_moe_experts(&x, st);
+  }
+  r.tile_rows = 128;
+  int rc = rf_moe_router(&r, st);
+  if (rc) return rc;
+  void* xg = s.at(s.off_xg);
+  rc = rf_moe_gather(&r, xg, H, st);
+  if (rc) return rc;
+  RfMoeGroupedGemm g = {};
+  g.x = xg; g.ldx = H; g.w = w.w_up; g.out = hg; g.ldo = ldh; g.tiles = r.tiles + 3; g.max_rows = pairs; g.N = w.bank_inter; g.K = H;
+  g.dual = 1; g.act = kActSiluMul; g.bank_section_row_tiles = E * bank_rt; g.bank_kb_total = kbH; g.rt_per_expert = bank_rt;
+  g.dtype = c.dtype; g.status = s.status();
+  rc = rf_moe_grouped_gemm(&g, st);
+  if (rc) return rc;
+  g.x = hg; g.ldx = ldh; g.w = w.w_down; g.out = yg; g.ldo = H; g.row_scale = r.slot_w; g.N = H; g.K = w.bank_inter; g.dual = 0;
+  g.act = kActNone; g.bank_section_row_tiles = 0; g.bank_kb_total = E * w.bank_inter / 64; g.rt_per_expert = 0; g.kb_per_expert = w.bank_inter / 64;
+  rc = rf_moe_grouped_gemm(&g, st);
+  if (rc || !has_shared) return rc;
+  uint8_t* hs = hg + (size_t)pairs * ldh * e;
+  RfGemm u = gemm_args(s, h, H, w.shared_up, hs, ldh, T, w.shared_inter, H, kActSiluMul);
+  u.dual_offset = w.shared_inter;
+  rc = rf_gemm(&u, st);
+  if (rc) return rc;
+  return linear(s, hs, ldh, w.shared_down, yg + (size_t)pairs * H * e, H, T, H, w.shared_inter, kActNone, st);
+}
+
 static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
   const RfMixedConfig& c = s.cfg;
   RF_REQUIRE(s.base != nullptr, "mixed stack: arena is not bound");
@@ -283,7 +475,7 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
   RF_REQUIRE(f.rows.num_seqs > 0 && f.rows.num_seqs <= c.max_seqs, "mixed stack: %d sequences (max %d)", f.rows.num_seqs, c.max_seqs);
   if (f.decode) RF_REQUIRE(f.tokens == f.rows.num_seqs && f.short_seqs == f.tokens, "mixed stack: a decode step has one row per sequence");
   else RF_REQUIRE(f.rows.seq_of_row && f.rows.q_start && f.rows.q_len, "mixed stack: portions need seq_of_row, q_start and q_len");
-  if (f.short_seqs < f.rows.num_seqs) RF_REQUIRE(f.h_q_len && f.h_pos0, "mixed stack: portions need the host arrays");
+  if (!f.decode) RF_REQUIRE(f.h_q_len && f.h_pos0, "mixed stack: portions need the host arrays");
   if (f.tokens == 0) return RF_OK;
   int rc = plan_windows(s, f, st);
   if (rc) return rc;
@@ -294,42 +486,51 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
   void* y = s.at(s.off_y);
   void* side = s.at(s.off_side);
   int cur = -1;                       // stream buffer in use; -1: still the embedding
-  const void* pend = nullptr;         // sublayer output that the next stream_norm adds
-  const float* pend_norm = nullptr;
+  MixedStack::Pending pend;           // sublayer output that the next stream_norm adds
   // stream step: adds the pending output, optionally writes the 16-bit copy and / or the normalised rows
   auto step = [&](const float* norm_w, const float* shift, float* shift_state, bool want_cast) -> int {
     RfStreamNorm a = {};
     a.x = cur < 0 ? nullptr : s.at<float>(s.off_x[cur]);
-    a.table = c.embed; a.ids = f.ids;
-    a.y = pend; a.y_norm_w = pend_norm;
+    a.table = c.embed; a.ids = f.ids; a.embed_scale = c.embed_scale;
+    a.y = pend.y; a.y_norm_w = pend.norm; a.y_slots = pend.slots; a.y_picks = pend.picks;
     const int nxt = cur < 0 ? 0 : cur ^ 1;
     a.x_out = s.at<float>(s.off_x[nxt]);
     a.x_cast = want_cast ? cast : nullptr;
     a.norm_w = norm_w; a.out = norm_w ? h : nullptr; a.shift = shift; a.shift_state = shift_state;
     a.rows = f.rows; a.n_rows = T; a.H = H; a.dim = c.hidden_true; a.eps = c.eps; a.dtype = c.dtype;
     cur = nxt;
-    pend = nullptr; pend_norm = nullptr;
+    pend = {};
     return rf_stream_norm(&a, st);
   };
   for (int l = 0; l < c.layers; ++l) {
     const RfMixedLayer& w = s.layers[l];
-    rc = step(w.norm1, w.shift, w.shift_state, false);
+    rc = c.norm_after ? step(nullptr, nullptr, nullptr, true) : step(w.norm1, w.shift, w.st.shift_state, false);
     if (rc) return rc;
-    rc = w.mixer == RF_MIXER_LATENT_ATTENTION ? latent_attention(s, w, f, h, mix, st) : hgrn2(s, w, f, h, mix, st);
+    const void* in = c.norm_after ? cast : h;
+    switch (w.mixer) {
+      case RF_MIXER_LATENT_ATTENTION: rc = latent_attention(s, w, f, in, mix, st); break;
+      case RF_MIXER_HGRN2: rc = hgrn2(s, w, f, in, mix, st); break;
+      case RF_MIXER_ATTENTION: rc = grouped_attention(s, w, f, in, mix, st); break;
+      default: rc = mamba1(s, w, f, in, mix, st);
+    }
     if (rc) return rc;
-    const int MD = w.heads * w.vdim;
-    rc = linear(s, mix, MD, w.w_o, y, H, T, H, MD, kActNone, st);
+    rc = linear(s, mix, w.out_dim, w.w_o, y, H, T, H, w.out_dim, kActNone, st);
     if (rc) return rc;
-    pend = y;
+    pend.y = y; pend.norm = c.norm_after ? w.norm1 : nullptr;
     if (w.inter > 0) {
-      rc = step(w.norm2, nullptr, nullptr, false);
+      rc = c.norm_after ? step(nullptr, nullptr, nullptr, true) : step(w.norm2, nullptr, nullptr, false);
       if (rc) return rc;
-      void* wide = s.at(s.off_wide);
-      rc = linear(s, h, H, w.w_up, wide, w.inter, T, w.inter, H, kActRelu2, st);
+      if (w.experts > 0) {
+        rc = experts(s, w, f, in, &pend, st);
+      } else {
+        void* wide = s.at(s.off_wide);
+        rc = linear(s, in, H, w.w_up, wide, w.inter, T, w.inter, H, kActRelu2, st);
+        if (rc) return rc;
+        rc = linear(s, wide, w.inter, w.w_down, y, H, T, H, w.inter, kActNone, st);
+        pend.y = y;
+      }
       if (rc) return rc;
-      rc = linear(s, wide, w.inter, w.w_down, y, H, T, H, w.inter, kActNone, st);
-      if (rc) return rc;
-      pend = y;
+      pend.norm = c.norm_after ? w.norm2 : nullptr;
     }
     if (c.side_dim > 0) {
       rc = step(nullptr, nullptr, nullptr, true);
@@ -339,11 +540,11 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
       if (rc) return rc;
       rc = linear(s, side, P, w.side_proj, y, H, T, H, P, kActNone, st);
       if (rc) return rc;
-      pend = y; pend_norm = w.side_norm;
+      pend.y = y; pend.norm = w.side_norm;
     }
     if (f.taps) {
       RfStreamNorm a = {};
-      a.x = s.at<float>(s.off_x[cur]); a.y = pend; a.y_norm_w = pend_norm;
+      a.x = s.at<float>(s.off_x[cur]); a.y = pend.y; a.y_norm_w = pend.norm; a.y_slots = pend.slots; a.y_picks = pend.picks;
       a.x_out = f.taps + (size_t)l * T * H;
       a.rows = f.rows; a.n_rows = T; a.H = H; a.dim = c.hidden_true; a.eps = c.eps; a.dtype = c.dtype;
       rc = rf_stream_norm(&a, st);
@@ -351,7 +552,7 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
     }
   }
   s.cur = cur;
-  s.side_pending = c.side_dim > 0;
+  s.tail = pend;
   return RF_OK;
 }
 
@@ -385,18 +586,40 @@ extern "C" int rf_mixed_destroy(int64_t h) {
 extern "C" int rf_mixed_set_layer(int64_t h, int32_t layer, const RfMixedLayer* w) {
   RF_GET_MIXED(h);
   RF_REQUIRE(w && layer >= 0 && layer < s.cfg.layers, "layer index %d out of range", layer);
-  RF_REQUIRE(w->heads > 0 && w->dim > 0 && w->dim % 8 == 0 && w->vdim > 0 && w->vdim % 8 == 0 && w->in_dim % 8 == 0 &&
-                 w->inter >= 0 && w->inter % 8 == 0, "layer %d: head and feed-forward sizes", layer);
-  RF_REQUIRE(w->norm1 && w->w_in && w->w_o && (!w->shift || w->shift_state), "layer %d: missing weights", layer);
+  RF_REQUIRE(w->in_dim % 8 == 0 && w->out_dim > 0 && w->out_dim % 8 == 0 && w->inter >= 0 && w->inter % 8 == 0, "layer %d: projection and feed-forward sizes", layer);
+  if (w->mixer != RF_MIXER_MAMBA1) {
+    RF_REQUIRE(w->heads > 0 && w->dim > 0 && w->dim % 8 == 0 && w->vdim > 0 && w->vdim % 8 == 0, "layer %d: head sizes", layer);
+    RF_REQUIRE(w->out_dim == w->heads * w->vdim, "layer %d: output projection columns", layer);
+  }
+  RF_REQUIRE(w->norm1 && w->w_in && w->w_o && (!w->shift || w->st.shift_state), "layer %d: missing weights", layer);
   if (w->inter > 0) RF_REQUIRE(w->norm2 && w->w_up && w->w_down && w->act == RF_MIXED_ACT_RELU2, "layer %d: feed-forward weights", layer);
+  if (w->experts > 0) {
+    RF_REQUIRE(w->inter > 0 && w->router && w->experts <= 256 && w->top > 0 && w->top <= 32 && w->groups > 0 && w->experts % w->groups == 0 &&
+                   w->keep > 0 && w->keep <= w->groups && w->top <= w->experts / w->groups * w->keep,
+               "layer %d: %d experts in %d groups, %d kept, %d chosen", layer, w->experts, w->groups, w->keep, w->top);
+    RF_REQUIRE(w->bank_inter >= w->inter && w->bank_inter % (s.cfg.dtype == kF32 ? 8 : 128) == 0 && w->shared_inter >= 0 && w->shared_inter % 8 == 0 &&
+                   (w->shared_inter == 0 || (w->shared_up && w->shared_down)), "layer %d: expert widths", layer);
+    RF_REQUIRE(s.cfg.dtype == kF32 || s.cfg.weights_packed, "layer %d: experts need tile-major weights", layer);
+  }
   if (w->mixer == RF_MIXER_LATENT_ATTENTION) {
-    RF_REQUIRE(w->rank > 0 && w->rank % 16 == 0 && w->rank_true > 0 && w->latent_norm && w->w_absorb && w->w_unabsorb && w->latent_pool,
+    RF_REQUIRE(w->rank > 0 && w->rank % 16 == 0 && w->rank_true > 0 && w->latent_norm && w->w_absorb && w->w_unabsorb && w->st.latent_pool,
                "layer %d: latent-attention weights", layer);
     RF_REQUIRE(w->in_dim >= w->heads * w->dim + w->rank, "layer %d: input projection rows", layer);
     RF_REQUIRE(w->expand_hd == 0 || (w->w_expand && w->dim == w->expand_hd && w->vdim == w->expand_hd && s.cfg.dtype != kF32),
                "layer %d: expanded heads", layer);
+  } else if (w->mixer == RF_MIXER_ATTENTION) {
+    RF_REQUIRE(w->dim == w->vdim && w->kv_heads > 0 && w->heads % w->kv_heads == 0 && w->dim_true > 0 && w->dim_true <= w->dim &&
+                   w->vdim_true > 0 && w->vdim_true <= w->vdim && w->st.k_pool && w->st.v_pool && w->st.pool_pages > 0, "layer %d: attention", layer);
+    RF_REQUIRE(w->in_dim >= ((w->gated ? 2 : 1) * w->heads + 2 * w->kv_heads) * w->dim, "layer %d: input projection rows", layer);
+    RF_REQUIRE(!w->tensor_core || (s.cfg.dtype != kF32 && (w->dim == 64 || w->dim == 128 || w->dim == 256) && w->scale > 0.f), "layer %d: heads", layer);
+    RF_REQUIRE(w->rot_dims % 2 == 0 && w->rot_dims >= 0 && w->rot_dims <= w->dim_true && (w->rot_dims == 0 || (w->cos && w->sin)), "layer %d: rotation", layer);
+  } else if (w->mixer == RF_MIXER_MAMBA1) {
+    RF_REQUIRE(w->inner > 0 && w->inner % 8 == 0 && w->states > 0 && w->states % 8 == 0 && w->states <= 256 && w->dt_rank > 0 && w->dt_rank % 8 == 0 &&
+                   w->taps > 0 && w->in_dim == 2 * w->inner && w->out_dim == w->inner, "layer %d: scan sizes", layer);
+    RF_REQUIRE(w->conv_w && w->a2 && w->d_skip && w->dt_bias && w->w_x && w->w_dt && w->w_dt_rows && w->st.rec_state && (w->taps == 1 || w->st.conv_state),
+               "layer %d: scan weights", layer);
   } else {
-    RF_REQUIRE(w->mixer == RF_MIXER_HGRN2 && w->f_bias && w->lower && w->head_norm && w->rec_state, "layer %d: HGRN2 weights", layer);
+    RF_REQUIRE(w->mixer == RF_MIXER_HGRN2 && w->f_bias && w->lower && w->head_norm && w->st.rec_state, "layer %d: HGRN2 weights", layer);
     RF_REQUIRE(w->in_dim >= w->heads * (2 * w->dim + w->vdim), "layer %d: input projection rows", layer);
   }
   if (s.cfg.side_dim > 0) RF_REQUIRE(s.cfg.side_table && w->side_gate && w->side_proj && w->side_norm, "layer %d: side-input weights", layer);
@@ -405,12 +628,18 @@ extern "C" int rf_mixed_set_layer(int64_t h, int32_t layer, const RfMixedLayer* 
   return RF_OK;
 }
 
-extern "C" int rf_mixed_set_state(int64_t h, int32_t layer, void* latent_pool, float* rec_state, float* shift_state) {
+extern "C" int rf_mixed_set_state(int64_t h, int32_t layer, const RfMixedState* st) {
   RF_GET_MIXED(h);
-  RF_REQUIRE(layer >= 0 && layer < s.cfg.layers, "layer index %d out of range", layer);
-  if (latent_pool) s.layers[layer].latent_pool = latent_pool;
-  if (rec_state) s.layers[layer].rec_state = rec_state;
-  if (shift_state) s.layers[layer].shift_state = shift_state;
+  RF_REQUIRE(st && layer >= 0 && layer < s.cfg.layers, "layer index %d out of range", layer);
+  s.layers[layer].st = *st;
+  return RF_OK;
+}
+
+extern "C" int rf_mixed_set_rotation(int64_t h, int32_t layer, const float* cos, const float* sin) {
+  RF_GET_MIXED(h);
+  RF_REQUIRE(cos && sin && layer >= 0 && layer < s.cfg.layers, "rotation tables of layer %d", layer);
+  s.layers[layer].cos = cos;
+  s.layers[layer].sin = sin;
   return RF_OK;
 }
 
@@ -461,8 +690,7 @@ extern "C" int rf_mixed_head(int64_t h, const int32_t* row_idx, int32_t rows, in
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   RfStreamNorm a = {};
   a.x = s.at<float>(s.off_x[s.cur]); a.row_idx = row_idx;
-  if (s.side_pending) { a.y = s.at(s.off_y); a.y_norm_w = s.layers[c.layers - 1].side_norm; }
-  else a.y = s.at(s.off_y);
+  a.y = s.tail.y; a.y_norm_w = s.tail.norm; a.y_slots = s.tail.slots; a.y_picks = s.tail.picks;
   a.norm_w = c.final_norm; a.out = s.at(s.off_head);
   a.n_rows = rows; a.H = c.hidden; a.dim = c.hidden_true; a.eps = c.eps; a.dtype = c.dtype;
   int rc = rf_stream_norm(&a, st);
@@ -477,5 +705,7 @@ extern "C" int rf_mixed_head(int64_t h, const int32_t* row_idx, int32_t rows, in
 extern "C" void rf_mixed_struct_sizes(int32_t* out) {
   out[0] = (int32_t)sizeof(RfMixedConfig); out[1] = (int32_t)sizeof(RfMixedLayer); out[2] = (int32_t)sizeof(RfMixedForward);
   out[3] = (int32_t)sizeof(RfRows); out[4] = (int32_t)sizeof(RfStreamNorm); out[5] = (int32_t)sizeof(RfLatentAttn);
-  out[6] = (int32_t)sizeof(RfHgrn2); out[7] = (int32_t)sizeof(RfHeadLinear);
+  out[6] = (int32_t)sizeof(RfHgrn2); out[7] = (int32_t)sizeof(RfHeadLinear); out[8] = (int32_t)sizeof(RfMixedState);
+  out[9] = (int32_t)sizeof(RfAttn); out[10] = (int32_t)sizeof(RfQkvInsert); out[11] = (int32_t)sizeof(RfConvSilu);
+  out[12] = (int32_t)sizeof(RfMamba1); out[13] = (int32_t)sizeof(RfMoeRouter); out[14] = (int32_t)sizeof(RfMoeExperts);
 }

@@ -1,6 +1,7 @@
 // Decoder stack whose layers differ: every layer names its own mixer (latent attention with a sliding window, HGRN2 linear
-// attention), head sizes and feed-forward, and the stack adds what such designs share: an fp32 residual stream, a token
-// shift in front of every mixer and a gated per-token side input behind every layer.  Activations are fp16 / bf16, or fp32
+// attention, grouped-head attention with chunks and sinks, a selective scan), sizes and feed-forward (dense or a mixture of
+// experts), and the stack adds what such designs share: an fp32 residual stream, norms in front of the sublayers or on their
+// outputs, a token shift in front of every mixer and a gated per-token side input behind every layer (both optional).  Activations are fp16 / bf16, or fp32
 // throughout (dtype 2).  Like rf_stack_* one handle owns the weight pointers and a static arena and enqueues the whole layer
 // loop on a stream, so a decode step can be captured into a CUDA graph.
 #pragma once
@@ -12,7 +13,7 @@
 extern "C" {
 #endif
 
-enum RfMixerKind { RF_MIXER_LATENT_ATTENTION = 0, RF_MIXER_HGRN2 = 1 };
+enum RfMixerKind { RF_MIXER_LATENT_ATTENTION = 0, RF_MIXER_HGRN2 = 1, RF_MIXER_ATTENTION = 2, RF_MIXER_MAMBA1 = 3 };
 enum RfMixedAct { RF_MIXED_ACT_RELU2 = 0 };
 
 typedef struct RfMixedConfig {
@@ -30,7 +31,19 @@ typedef struct RfMixedConfig {
   const void* side_table;        // [vocab, layers * side_dim]
   const float* final_norm;
   const void* w_lm;              // [vocab_ld, hidden]
+  float embed_scale;
+  int32_t norm_after;            // 0: sublayers read the normalised stream; 1: they read the stream, norms act on their outputs
 } RfMixedConfig;
+
+// Per-sequence memory of a layer; what a layer does not use is null.
+typedef struct RfMixedState {
+  void* latent_pool;                    // [pages, 16, rank]
+  void* k_pool; void* v_pool;           // [pages, kv_heads, 16, head size]
+  int64_t pool_pages;
+  float* rec_state;                     // HGRN2: [slots, heads, dim, vdim]; scan: [slots, inner, states]
+  void* conv_state;                     // [slots, taps - 1, inner]
+  float* shift_state;                   // [slots, hidden]
+} RfMixedState;
 
 // Padded sizes: per-head sizes and ranks are multiples of 8 / 16 with zero rows behind the true ones.
 typedef struct RfMixedLayer {
@@ -40,23 +53,41 @@ typedef struct RfMixedLayer {
   int32_t inter;                        // 0: the layer has no feed-forward
   int32_t act;                          // RfMixedAct
   float scale;
-  int32_t in_dim;                       // rows of w_in: [q | latent] or [q | f | v]
+  int32_t in_dim;                       // rows of w_in: [q | latent], [q | f | v], [q | k | v | gate] or [x | z]
+  int32_t out_dim;                      // columns of w_o
   const float* norm1; const float* norm2; const float* shift;
-  float* shift_state;                   // [slots, hidden]
   const void* w_in; const void* w_o; const void* w_up; const void* w_down;
   const float* latent_norm;
   const void* w_absorb;                 // [heads, rank, dim]: query -> latent space
   const void* w_unabsorb;               // [heads, vdim, rank]: latent space -> value
   const void* w_expand;                 // [2 * heads * expand_hd, rank]: keys of all heads, then values
-  void* latent_pool;                    // [pages, 16, rank]
   const float* f_bias; const float* lower; const float* head_norm;
-  float* rec_state;                     // [slots, heads, dim, vdim]
   const void* side_gate; const void* side_proj; const float* side_norm;
+  // grouped-head attention: heads of dim == vdim values (true sizes dim_true, vdim_true)
+  int32_t kv_heads, dim_true;
+  int32_t tensor_core;                  // 1: heads of 64 / 128 / 256 on the tensor-core kernels; 0: attention by row in fp32
+  int32_t chunk;                        // > 0: positions see their own chunk of this many positions
+  int32_t gated;                        // the input projection holds an output gate behind the values
+  int32_t rot_dims, v_role;             // RfVMix
+  float v_lambda;
+  const float* cos; const float* sin;   // [positions, rot_dims / 2]
+  const float* q_norm; const float* k_norm; const float* sink;
+  // selective scan
+  int32_t inner, states, dt_rank, taps;
+  const float* conv_w; const float* conv_b; const float* a2; const float* d_skip; const float* dt_bias;
+  const void* w_x;                      // [dt_rank + 2 * states, inner]
+  const void* w_dt; const void* w_dt_rows;   // [inner, dt_rank]: as the linear layers take it, and row-major
+  // mixture of experts (experts > 0; inter is an expert's width, w_up and w_down the banks)
+  int32_t experts, top, groups, keep, score_fn, norm_topk, shared_inter;
+  int32_t bank_inter;                   // inter padded to the bank's granularity (128 in 16 bits)
+  float route_scale;
+  const void* router; const float* correction; const void* shared_up; const void* shared_down;
+  RfMixedState st;
 } RfMixedLayer;
 
 // One step: portions of several sequences packed into rows.  The first `short_seqs` sequences (`short_rows` rows) have fewer
 // than long_min tokens each, the rest are prefill-sized.  decode = 1: one row per sequence, seq_of_row / q_start / q_len null.
-// h_q_len / h_pos0 are HOST arrays [num_seqs] (new tokens and first position), read only for prefill-sized sequences.
+// h_q_len / h_pos0 are HOST arrays [num_seqs] (new tokens and first position); decode steps do not read them.
 typedef struct RfMixedForward {
   const int32_t* ids;
   RfRows rows;
@@ -69,8 +100,10 @@ typedef struct RfMixedForward {
 int64_t rf_mixed_create(const RfMixedConfig* cfg);
 int rf_mixed_destroy(int64_t h);
 int rf_mixed_set_layer(int64_t h, int32_t layer, const RfMixedLayer* w);
-// Re-point the per-layer state of a layer (binding another cache object); null keeps the pointer.
-int rf_mixed_set_state(int64_t h, int32_t layer, void* latent_pool, float* rec_state, float* shift_state);
+// Re-point the per-sequence memory of a layer (binding another cache object).
+int rf_mixed_set_state(int64_t h, int32_t layer, const RfMixedState* st);
+// Re-point the rotation tables of a layer (a longer context).
+int rf_mixed_set_rotation(int64_t h, int32_t layer, const float* cos, const float* sin);
 // Raise max_seq_len (a larger cache is bound); the arena has to be planned and bound again.
 int rf_mixed_set_context(int64_t h, int32_t max_seq_len);
 uint64_t rf_mixed_arena_bytes(int64_t h);
@@ -81,7 +114,8 @@ int rf_mixed_forward(int64_t h, const RfMixedForward* f, rf_stream_t stream);
 // [rows, vocab_ld] in the activation dtype; out_ids (optional) receives the arg-max.
 int rf_mixed_head(int64_t h, const int32_t* row_idx, int32_t rows, int32_t* out_ids, float* out_vals, void* logits,
                   rf_stream_t stream);
-void rf_mixed_struct_sizes(int32_t* out);   // sizeof: config, layer, forward, RfRows, RfStreamNorm, RfLatentAttn, RfHgrn2, RfHeadLinear
+void rf_mixed_struct_sizes(int32_t* out);   // sizeof: config, layer, forward, RfRows, RfStreamNorm, RfLatentAttn, RfHgrn2, RfHeadLinear, state, RfAttn, RfQkvInsert,
+                                            // RfConvSilu, RfMamba1, RfMoeRouter, RfMoeExperts
 
 #ifdef __cplusplus
 }

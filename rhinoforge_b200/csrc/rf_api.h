@@ -251,10 +251,20 @@ typedef struct RfAttn {
   float scale;              // <= 0: 1/sqrt(hd)
   float* ws; uint64_t ws_bytes;  // decode split-KV scratch, optional
   int32_t* status; int32_t dtype;
+  // Options of the paged forms:
+  const int32_t* slot;      // page-table row of every sequence (null: the sequence's own index)
+  int32_t chunk;            // > 0: position i sees j only if i / chunk == j / chunk (positions count from the sequence's start)
+  const float* sink;        // [Hq]: the softmax denominator also holds exp(sink[h])
+  const void* gate; int64_t ld_gate;   // [rows, Hq * hd]: the result is multiplied by sigmoid(gate) before it is rounded
+  // rf_attn_decode by row: with `pos`, query row r is position pos[r] of sequence seq_of_row[r] (null: r) and sees everything
+  // up to itself; kv_len is not used and num_seqs counts rows.
+  const int32_t* seq_of_row; const int32_t* pos;
 } RfAttn;
 int rf_attn_prefill(const RfAttn* a, rf_stream_t stream);
 int rf_attn_decode(const RfAttn* a, rf_stream_t stream);
 uint64_t rf_attn_decode_scratch_bytes(int num_seqs, int Hq, int hd);
+// The most scratch rf_attn_decode asks for at any number of sequences and keys.
+uint64_t rf_attn_decode_scratch_bound(int Hq, int Hkv, int hd);
 
 
 // --------------------------------------------- linear attention (GDN) ----
@@ -315,6 +325,8 @@ typedef struct RfRows {
 //   x_out = v (fp32), x_cast = v (activation dtype)
 //   h = v / rms(v) * norm_w;  with `shift`: out = h + (h_prev - h) * shift, h_prev the h of the sequence's previous token
 //   (carried over launches in shift_state[slot], zeros before the first token); without: out = h.
+// Embedding rows are multiplied by embed_scale (0 counts as 1).  With y_picks > 0 the outstanding output is the sum of y_picks rows of y, those
+// that y_slots[row * y_picks ...] names (negative: none): the experts' results of a mixture of experts.
 // H is the (padded, multiple of 8) row length, dim the true one that the means run over.  x_out must not alias x when
 // `shift` is set.  row_idx (optional) selects the rows that are processed (not together with shift).
 typedef struct RfStreamNorm {
@@ -325,6 +337,8 @@ typedef struct RfStreamNorm {
   const float* shift; float* shift_state;
   RfRows rows;
   int32_t n_rows, H, dim; float eps; int32_t dtype;    // dtype 2: fp32 activations
+  float embed_scale;
+  const int32_t* y_slots; int32_t y_picks;
 } RfStreamNorm;
 int rf_stream_norm(const RfStreamNorm* a, rf_stream_t stream);
 
@@ -373,6 +387,51 @@ typedef struct RfLatentAttn {
 } RfLatentAttn;
 int rf_latent_attn(const RfLatentAttn* a, rf_stream_t stream);
 uint64_t rf_latent_attn_scratch_bytes(int rows, int heads, int rank, int max_kv);
+
+// Grouped-head attention over paged K/V pools [pages, kv_heads, 16, hd]: what lies between the input projection and the
+// attention, in one launch and in fp32 - RMSNorm of every query and key head over its true size `dim` (optional), rotation of the
+// first rot_dims dimensions (rotate-half pairs, cos / sin [positions, rot_dims / 2]), value mixing, insertion of keys and values
+// at the row's position.  A row holds heads * hd query values, then kv_heads * hd keys at k_off and values at v_off, every head
+// padded with zeros to hd; queries are replaced in place.
+// Value mixing: the first mixing layer stores its values in v_first [rows, kv_heads, vdim], later ones take
+// v = (1 - v_lambda) v + v_lambda v_first.
+enum RfVMix { RF_VMIX_NONE = 0, RF_VMIX_FIRST = 1, RF_VMIX_MIX = 2 };
+typedef struct RfQkvInsert {
+  void* qkv; int64_t ld; int32_t k_off, v_off;
+  const float* q_norm; const float* k_norm; const float* cos; const float* sin;
+  void* v_first; void* k_pool; void* v_pool;
+  RfRows rows;
+  int32_t n_rows, heads, kv_heads, hd, dim, vdim, rot_dims, v_role; float v_lambda, eps; int32_t dtype;
+} RfQkvInsert;
+int rf_qkv_insert(const RfQkvInsert* a, rf_stream_t stream);
+// Attention by row on the CUDA cores in fp32, any head size up to 2048 and any scale: the by-row form of rf_attn_decode (pos,
+// seq_of_row, slot, chunk, sink, gate) for 32-bit models and heads the tensor-core kernels do not take.
+int rf_attn_rows(const RfAttn* a, rf_stream_t stream);
+
+// Causal convolution per channel over packed rows, silu applied: y[t] = silu(bias + sum_k w[k] x[t - (taps - 1) + k]).  The last
+// taps - 1 inputs of every sequence are carried in state [slots, taps - 1, channels], oldest first.  w: [taps, channels] fp32.
+typedef struct RfConvSilu {
+  const void* x; int64_t ldx; void* y; int64_t ldy;
+  const float* w; const float* bias; void* state;
+  RfRows rows;
+  int32_t max_q_len, channels, taps, dtype;
+} RfConvSilu;
+int rf_conv_silu(const RfConvSilu* a, rf_stream_t stream);
+
+// Selective scan (Mamba): with dt = softplus(step size + dt_bias),  S = 2^(dt a2) S + dt x B,  y = (S C + d x) silu(z).
+// a2 [inner, states] is -exp(A_log) / ln 2; rows of bc hold [step-size input: rank | B: states | C: states]; state: fp32
+// [slots, inner, states].  Padding states have a2 = 0 and zero B and C.
+// The recurrent form computes the step sizes itself from w_dt [inner, rank] (row-major, activation dtype) and takes any portions;
+// the scan form takes them projected (dt [rows, inner], before the bias) and is for prefill-sized portions.
+typedef struct RfMamba1 {
+  const void* x; int64_t ldx; const void* z; int64_t ldz; const void* bc; int64_t ld_bc; const void* dt; int64_t ld_dt;
+  const void* w_dt; const float* dt_bias; const float* a2; const float* d;
+  float* state; void* out; int64_t ldo;
+  RfRows rows;
+  int32_t inner, states, rank, dtype;
+} RfMamba1;
+int rf_mamba1_recurrent(const RfMamba1* a, rf_stream_t stream);
+int rf_mamba1_scan(const RfMamba1* a, rf_stream_t stream);
 
 // HGRN2 linear attention (what a gate takes from the state it gives to the new value), over packed input rows [q | f | v]:
 //   q = silu(q), f = lower + (1 - lower) * sigmoid(f + f_bias), S = diag(f) S + (1 - f) v^T, o = S^T q,
@@ -433,6 +492,40 @@ int rf_moe_group(const int32_t* ids, const float* w, int rows, int k, int E, int
 // out[t, :] += sum_j y[slot_of[t, j], :]  (fp32, picks in order j = 0..k-1, one rounding)
 int rf_moe_combine(void* out, int64_t ldo, const void* y, int64_t ldy, const int32_t* slot_of, int rows, int k, int H,
                    int dtype, rf_stream_t stream);
+
+
+// Router and expert plan in one launch.  logits = x w^T in fp32, scores = softmax (or sigmoid) over all experts, choice scores =
+// scores + correction; only experts of the `keep` best of `groups` equal groups (a group counts as much as its best expert) can be
+// chosen, the k largest choice scores are; weights are the chosen experts' scores, divided by their sum with norm_topk, times
+// scale.  Outputs: ids / weights [rows, k]; rank [rows, k] = the pick's place among its expert's picks; start [experts];
+// the tile list (the count in words 0 and 3, entries of four words from word 4 on: tiles + 3 is a list for rf_moe_grouped_gemm;
+// blocks of tile_rows rows, with shared_tiles followed by blocks of the shared expert, number `experts`, over sorted rows
+// [rows * k, rows * k + rows)).  With `scatter` (few rows) also
+// what rf_moe_gather otherwise writes: slot_of [rows, slot_ld] (sorted row of every pick, then of the shared expert),
+// token_of_slot and slot_w.  counters: experts + 1 words, zero before the first launch and left zero.
+enum RfMoeScore { RF_MOE_SIGMOID = 0, RF_MOE_SOFTMAX = 1 };
+typedef struct RfMoeRouter {
+  const void* x; int64_t ldx; const void* w; const float* correction;
+  int32_t* ids; float* weights; int32_t* rank; int32_t* counters; int32_t* start; int32_t* tiles;
+  int32_t* slot_of; int32_t* token_of_slot; float* slot_w;
+  int32_t rows, experts, width, k, groups, keep, score_fn, norm_topk; float scale;
+  int32_t tile_rows, slot_ld, has_shared, shared_tiles, scatter, dtype;
+} RfMoeRouter;
+int rf_moe_router(const RfMoeRouter* a, rf_stream_t stream);
+// Copies every row of x to the sorted rows of its picks (and writes slot_of, token_of_slot, slot_w).
+int rf_moe_gather(const RfMoeRouter* a, void* out, int64_t ldo, rf_stream_t stream);
+
+// Expert GEMMs of few rows over the tile list of rf_moe_router: out[s] = act(x[row of s] W_e^T) (* slot_w[s]); the row is
+// token_of_slot[s], or s itself where that is null.  16-bit: banks are tile-major images as in rf_moe_grouped_gemm, the shared
+// expert has its own; tiles of 16 or 32 rows.  32-bit: banks are plain [experts][n][k] matrices (dual: all gates, then all ups);
+// tiles of 64 rows.
+typedef struct RfMoeExperts {
+  const void* x; int64_t ldx; const void* w; const void* w_shared; void* out; int64_t ldo;
+  const int32_t* tiles; const int32_t* token_of_slot; const float* slot_w;
+  int32_t max_tiles, experts, n, k, shared_n, shared_k, dual, tile_rows;
+  int32_t bank_section_row_tiles, bank_kb_total, rt_per_expert, kb_per_expert, shared_section_row_tiles, shared_kb_total, dtype;
+} RfMoeExperts;
+int rf_moe_experts(const RfMoeExperts* a, rf_stream_t stream);
 
 
 // ------------------------------------------------------------- KV pool ----

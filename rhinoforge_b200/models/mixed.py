@@ -1,14 +1,16 @@
 """Decoders whose layers name their own mixer: configuration records and weight tables.
 
-A :class:`MixedConfig` is a list of layers, each with one mixer (:class:`LatentAttention`, :class:`HGRN2`) and an optional
-feed-forward (:class:`DenseMLP`), over what the layers share: the width of an fp32 residual stream, RMSNorm epsilon, tied
-embedding, a token shift in front of every mixer and a gated per-token side input behind every layer.  The native executor
-is ``csrc/models/mixed_stack.cu``, the engine :mod:`rhinoforge_b200.runtime.mixed_engine`.
+A :class:`MixedConfig` is a list of layers, each with one mixer (:class:`LatentAttention`, :class:`HGRN2`,
+:class:`GroupedAttention`, :class:`Mamba1`) and an optional feed-forward (:class:`DenseMLP`, :class:`MoE`), over what the layers
+share: the width of an fp32 residual stream, RMSNorm epsilon, where the norms sit, and optionally a token shift in front of every
+mixer and a gated per-token side input behind every layer.  The native executor is ``csrc/models/mixed_stack.cu``, the engine
+:mod:`rhinoforge_b200.runtime.mixed_engine`.
 
-Reader of Vabarax's ``config.json``: :meth:`MixedConfig.from_vabarax`.
+Readers of ``config.json``: :meth:`MixedConfig.from_vabarax`, :meth:`MixedConfig.from_zulopel`.
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 from typing import Any, Dict, Iterator, Mapping, Optional, Tuple, Union
 
@@ -38,21 +40,109 @@ class HGRN2:
 
 
 @dataclass(frozen=True)
+class YarnScaling:
+    """Stretch of a rotation made for ``original`` positions by ``factor``: pairs of dimensions that turn more than ``fast`` times
+    over the original length keep their frequency, those that turn less than ``slow`` times are divided by the factor."""
+    factor: float
+    original: int
+    fast: float
+    slow: float
+
+
+@dataclass(frozen=True)
+class Rotary:
+    """Rotation of the first ``dims`` dimensions of a head, dimension i paired with i + dims / 2."""
+    dims: int
+    base: float
+    scaling: Optional[YarnScaling] = None
+
+    def frequencies(self) -> torch.Tensor:
+        """float64 ``[dims / 2]``, stretch applied."""
+        f = torch.tensor([self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)], dtype=torch.float64)
+        y = self.scaling
+        if y is None:
+            return f
+        pair = lambda turns: self.dims * math.log(y.original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
+        lo, hi = max(math.floor(pair(y.fast)), 0), min(math.ceil(pair(y.slow)), self.dims - 1)
+        ramp = ((torch.arange(self.dims // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return f / y.factor * ramp + f * (1.0 - ramp)
+
+    def tables(self, positions: int, device) -> Tuple[torch.Tensor, torch.Tensor]:
+        """fp32 cos and sin ``[positions, dims / 2]`` of positions 0, 1, ..., the stretch's magnitude factor included."""
+        amp = 1.0 if self.scaling is None else 0.1 * math.log(self.scaling.factor) + 1.0
+        angle = torch.arange(positions, dtype=torch.float64, device=device)[:, None] * self.frequencies().to(device)[None]
+        return (angle.cos() * amp).float().contiguous(), (angle.sin() * amp).float().contiguous()
+
+
+@dataclass(frozen=True)
+class GroupedAttention:
+    """Softmax attention with ``heads // kv_heads`` query heads per key / value head.  ``chunk``: positions see their own chunk of
+    this many positions only (None: everything before them).  ``sink``: one more learned term in every head's softmax denominator.
+    ``v_mix``: values are mixed with those of the first layer that says so.  ``gate``: sigmoid gate on the heads' outputs."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    chunk: Optional[int] = None
+    rot: Optional[Rotary] = None
+    v_mix: bool = False
+    qk_norm: bool = True
+    sink: bool = True
+    gate: bool = True
+
+
+@dataclass(frozen=True)
+class Mamba1:
+    """Selective scan over ``inner`` channels with ``state`` states each, behind a causal convolution of ``conv`` taps."""
+    inner: int
+    state: int
+    dt_rank: int
+    conv: int
+
+
+@dataclass(frozen=True)
 class DenseMLP:
     """``down(relu(up h)^2)``."""
     ff: int
 
 
 @dataclass(frozen=True)
+class MoE:
+    """``top`` of ``experts`` SwiGLU experts of width ``ff`` per token, chosen among the ``keep`` best of ``groups`` groups by
+    softmax score plus correction and weighted by normalised score; ``shared_ff`` > 0: one more expert that every token uses."""
+    experts: int
+    top: int
+    ff: int
+    groups: int = 1
+    keep: int = 1
+    shared_ff: int = 0
+
+
+@dataclass(frozen=True)
 class MixedLayer:
-    mixer: Union[LatentAttention, HGRN2]
-    mlp: Optional[DenseMLP] = None
+    mixer: Union[LatentAttention, HGRN2, GroupedAttention, Mamba1]
+    mlp: Optional[Union[DenseMLP, MoE]] = None
 
 
 def _int(d: Mapping[str, Any], key: str, where: str) -> int:
     v = d.get(key)
     if isinstance(v, bool) or not isinstance(v, int) or v <= 0:
         raise UnsupportedModelError(f"{where}: {key!r} must be a positive integer, got {v!r}")
+    return v
+
+
+def _float(d: Mapping[str, Any], key: str, where: str, positive: bool = False) -> float:
+    v = d.get(key)
+    if isinstance(v, bool) or not isinstance(v, (int, float)) or not math.isfinite(v) or (positive and v <= 0):
+        raise UnsupportedModelError(f"{where}: {key!r} must be a {'positive ' if positive else ''}number, got {v!r}")
+    return float(v)
+
+
+def _map(d: Mapping[str, Any], key: str, where: str) -> Mapping[str, Any]:
+    v = d.get(key)
+    if not isinstance(v, Mapping):
+        raise UnsupportedModelError(f"{where}: {key!r} must be a mapping, got {v!r}")
     return v
 
 
@@ -69,7 +159,12 @@ class MixedConfig:
     hidden_size: int
     rms_eps: float
     layers: Tuple[MixedLayer, ...]
-    side_dim: int
+    side_dim: int = 0              # width of the per-token side input behind every layer (0: none)
+    token_shift: bool = True       # mix every token's normalised row with the one before, in front of every mixer
+    norm_after: bool = False       # norms on the sublayers' outputs instead of their inputs
+    layer_scale: bool = False      # element-wise factors on the sublayers' outputs
+    tied_head: bool = True
+    embed_scale: float = 1.0
     model_type: str = "vabarax"
     raw: Optional[Mapping[str, Any]] = field(default=None, compare=False, repr=False)
 
@@ -112,6 +207,71 @@ class MixedConfig:
                    rms_eps=float(c["norm"]["eps"]), layers=tuple(layers), side_dim=_int(c["token_side"], "dim", "Vabarax token_side"),
                    raw=c)
 
+    @classmethod
+    def zulopel(cls, name: str, vocab: int, width: int, eps: float, layers, embed_scale: float = 1.0, **kw) -> "MixedConfig":
+        """A decoder of the Zulopel design: grouped attention and selective-scan layers in any order, mixture-of-experts
+        feed-forwards, norms and layer scales on the sublayers' outputs, an untied head."""
+        cfg = cls(name, vocab, width, eps, tuple(layers), 0, token_shift=False, norm_after=True, layer_scale=True, tied_head=False,
+                  embed_scale=embed_scale, model_type="zulopel", **kw)
+        widths = {(i, m.kv_heads * m.vdim) for i, m in enumerate(x.mixer for x in cfg.layers) if isinstance(m, GroupedAttention) and m.v_mix}
+        if len({w for _, w in widths}) > 1:
+            raise UnsupportedModelError(f"{name}: layers that mix values need values of one size, got (layer, size) {sorted(widths)}")
+        return cfg
+
+    @classmethod
+    def from_zulopel(cls, c: Mapping[str, Any]) -> "MixedConfig":
+        """The mapping of a Zulopel ``config.json``.  Keys that the reader does not know are refused rather than ignored."""
+        _known(c, ("architecture", "embedding", "layers", "norm", "vocab", "width"), "Zulopel")
+        if not isinstance(c.get("layers"), list) or not c["layers"]:
+            raise UnsupportedModelError("Zulopel: 'layers' must be a non-empty list")
+        layers = []
+        for i, entry in enumerate(c["layers"]):
+            where = f"Zulopel layer {i}"
+            if not isinstance(entry, Mapping):
+                raise UnsupportedModelError(f"{where}: must be a mapping")
+            _known(entry, ("type", "mixer", "mlp"), where)
+            kind, m = entry.get("type"), _map(entry, "mixer", where)
+            if kind == "attention":
+                mixer: Union[GroupedAttention, Mamba1] = _zulopel_attention(m, where)
+            elif kind == "mamba1":
+                _known(m, ("inner", "state", "dt_rank", "conv"), where)
+                mixer = Mamba1(*(_int(m, k, where) for k in ("inner", "state", "dt_rank", "conv")))
+            else:
+                raise UnsupportedModelError(f"{where}: mixer type {kind!r} is not built")
+            layers.append(MixedLayer(mixer, None if entry.get("mlp") is None else _zulopel_experts(_map(entry, "mlp", where), where + " mlp")))
+        norm = _map(c, "norm", "Zulopel")
+        _known(norm, ("eps",), "Zulopel norm")
+        emb = c.get("embedding") or {}
+        _known(emb, ("scale",), "Zulopel embedding")
+        return cls.zulopel("zulopel", _int(c, "vocab", "Zulopel"), _int(c, "width", "Zulopel"), _float(norm, "eps", "Zulopel norm"), layers,
+                           _float(emb, "scale", "Zulopel embedding") if "scale" in emb else 1.0, raw=c)
+
+    def to_zulopel(self) -> Dict[str, Any]:
+        """The inverse of :meth:`from_zulopel`."""
+        out = []
+        for layer in self.layers:
+            m, f = layer.mixer, layer.mlp
+            if isinstance(m, Mamba1):
+                d: Dict[str, Any] = {"inner": m.inner, "state": m.state, "dt_rank": m.dt_rank, "conv": m.conv}
+            else:
+                d = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale, "v_mix": m.v_mix}
+                if m.chunk is not None:
+                    d["mask"] = {"size": m.chunk}
+                if m.rot is not None:
+                    d["rot"] = {"dims": m.rot.dims, "base": m.rot.base}
+                    if m.rot.scaling is not None:
+                        y = m.rot.scaling
+                        d["rot"]["scaling"] = {"factor": y.factor, "original": y.original, "fast": y.fast, "slow": y.slow}
+            mlp = None
+            if f is not None:
+                mlp = {"kind": "moe", "expert": {"ff": f.ff},
+                       "router": {"experts": f.experts, "top": f.top, "groups": {"count": f.groups, "keep": f.keep}}}
+                if f.shared_ff:
+                    mlp["shared"] = {"ff": f.shared_ff}
+            out.append({"type": "mamba1" if isinstance(m, Mamba1) else "attention", "mixer": d, "mlp": mlp})
+        return {"architecture": "Zulopel", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.rms_eps},
+                "embedding": {"scale": self.embed_scale}, "layers": out}
+
     def to_vabarax(self) -> Dict[str, Any]:
         """The inverse of :meth:`from_vabarax`."""
         out = []
@@ -128,23 +288,92 @@ class MixedConfig:
                 "token_side": {"dim": self.side_dim}, "layers": out}
 
 
+def _zulopel_attention(m: Mapping[str, Any], where: str) -> GroupedAttention:
+    _known(m, ("heads", "kv_heads", "dim", "vdim", "scale", "mask", "rot", "v_mix"), where)
+    mask, rot = m.get("mask") or {}, None
+    _known(mask, ("size",), where + " mask")
+    if m.get("rot"):
+        r, w = _map(m, "rot", where), where + " rot"
+        _known(r, ("dims", "base", "scaling"), w)
+        yarn = None
+        if r.get("scaling"):
+            sc, ws = _map(r, "scaling", w), w + " scaling"
+            _known(sc, ("factor", "original", "fast", "slow"), ws)
+            yarn = YarnScaling(_float(sc, "factor", ws, True), _float(sc, "original", ws, True), _float(sc, "fast", ws, True),
+                               _float(sc, "slow", ws, True))
+        rot = Rotary(_int(r, "dims", w), _float(r, "base", w, True), yarn)
+    a = GroupedAttention(_int(m, "heads", where), _int(m, "kv_heads", where), _int(m, "dim", where), _int(m, "vdim", where),
+                         _float(m, "scale", where), _int(mask, "size", where + " mask") if mask else None, rot, bool(m.get("v_mix", False)))
+    if a.heads % a.kv_heads:
+        raise UnsupportedModelError(f"{where}: {a.heads} heads do not share {a.kv_heads} key / value heads evenly")
+    if rot is not None and (rot.dims % 2 or rot.dims > a.dim):
+        raise UnsupportedModelError(f"{where}: rotation of {rot.dims} of {a.dim} dimensions")
+    return a
+
+
+def _zulopel_experts(f: Mapping[str, Any], where: str) -> MoE:
+    _known(f, ("kind", "expert", "router", "shared"), where)
+    if f.get("kind") != "moe":
+        raise UnsupportedModelError(f"{where}: feed-forward kind {f.get('kind')!r} is not built")
+    expert, r = _map(f, "expert", where), _map(f, "router", where)
+    _known(expert, ("ff",), where + " expert")
+    _known(r, ("experts", "top", "groups"), where + " router")
+    groups = r.get("groups") or {"count": 1, "keep": 1}
+    _known(groups, ("count", "keep"), where + " groups")
+    shared = f.get("shared") or {}
+    _known(shared, ("ff",), where + " shared")
+    e = MoE(_int(r, "experts", where), _int(r, "top", where), _int(expert, "ff", where), _int(groups, "count", where), _int(groups, "keep", where),
+            _int(shared, "ff", where + " shared") if shared else 0)
+    if e.experts % e.groups or e.keep > e.groups or e.top > e.experts // e.groups * e.keep:
+        raise UnsupportedModelError(f"{where}: {e.top} of {e.experts} experts in {e.keep} of {e.groups} groups")
+    if e.experts > 256 or e.top > 32:
+        raise UnsupportedModelError(f"{where}: the router takes up to 256 experts and 32 choices")
+    return e
+
+
 def weight_shapes(cfg: MixedConfig) -> Iterator[Tuple[str, Tuple[int, ...], str]]:
-    """(tensor name, shape, kind) of a checkpoint; kind is 'linear', 'embed', 'norm', 'unit' (values in [0, 1)) or 'bias'."""
+    """(tensor name, shape, kind) of a checkpoint; kind is 'linear', 'embed', 'norm', 'unit' (values in [0, 1)), 'bias', 'scale'
+    (positive factors), 'log_a' (logarithms of decay rates), 'dt_bias' (step sizes before softplus) or 'correction'."""
     H, P = cfg.hidden_size, cfg.side_dim
     yield "embed", (cfg.vocab_size, H), "embed"
-    yield "side.embed", (cfg.vocab_size, cfg.num_layers * P), "embed"
+    if P:
+        yield "side.embed", (cfg.vocab_size, cfg.num_layers * P), "embed"
     for i, layer in enumerate(cfg.layers):
         p, m = f"l{i}.", layer.mixer
-        qd, vd = m.heads * m.dim, m.heads * m.vdim
         yield p + "norm1", (H,), "norm"
-        yield p + "shift", (H,), "unit"
-        yield p + "mix.q", (qd, H), "linear"
-        if isinstance(m, LatentAttention):
+        if cfg.token_shift:
+            yield p + "shift", (H,), "unit"
+        if isinstance(m, Mamba1):
+            yield p + "mix.in", (2 * m.inner, H), "linear"
+            yield p + "mix.conv", (m.inner, m.conv), "linear"
+            yield p + "mix.conv.b", (m.inner,), "bias"
+            yield p + "mix.x", (m.dt_rank + 2 * m.state, m.inner), "linear"
+            yield p + "mix.dt", (m.inner, m.dt_rank), "linear"
+            yield p + "mix.dt.b", (m.inner,), "dt_bias"
+            yield p + "mix.A_log", (m.inner, m.state), "log_a"
+            yield p + "mix.D", (m.inner,), "norm"
+            vd = m.inner
+        else:
+            qd, vd = m.heads * m.dim, m.heads * m.vdim
+            yield p + "mix.q", (qd, H), "linear"
+        if isinstance(m, GroupedAttention):
+            yield p + "mix.k", (m.kv_heads * m.dim, H), "linear"
+            yield p + "mix.v", (m.kv_heads * m.vdim, H), "linear"
+            if m.qk_norm:
+                yield p + "mix.q.norm", (m.dim,), "norm"
+                yield p + "mix.k.norm", (m.dim,), "norm"
+            if m.v_mix:
+                yield p + "mix.vmix", (), "unit"
+            if m.sink:
+                yield p + "mix.sink", (m.heads,), "bias"
+            if m.gate:
+                yield p + "mix.g", (vd, H), "linear"
+        elif isinstance(m, LatentAttention):
             yield p + "mix.dkv", (m.kv_rank, H), "linear"
             yield p + "mix.dkv.norm", (m.kv_rank,), "norm"
             yield p + "mix.uk", (qd, m.kv_rank), "linear"
             yield p + "mix.uv", (vd, m.kv_rank), "linear"
-        else:
+        elif isinstance(m, HGRN2):
             yield p + "mix.f", (qd, H), "linear"
             yield p + "mix.f.b", (qd,), "bias"
             yield p + "mix.lower", (qd,), "unit"
@@ -153,17 +382,34 @@ def weight_shapes(cfg: MixedConfig) -> Iterator[Tuple[str, Tuple[int, ...], str]
         yield p + "mix.o", (H, vd), "linear"
         if layer.mlp is not None:
             yield p + "norm2", (H,), "norm"
+        if isinstance(layer.mlp, MoE):
+            f = layer.mlp
+            for e, ff in [(f"e{j}", f.ff) for j in range(f.experts)] + ([("shared", f.shared_ff)] if f.shared_ff else []):
+                yield f"{p}mlp.{e}.gate", (ff, H), "linear"
+                yield f"{p}mlp.{e}.up", (ff, H), "linear"
+                yield f"{p}mlp.{e}.down", (H, ff), "linear"
+            yield p + "mlp.router", (f.experts, H), "linear"
+            yield p + "mlp.correction", (f.experts,), "correction"
+        elif layer.mlp is not None:
             yield p + "mlp.up", (layer.mlp.ff, H), "linear"
             yield p + "mlp.down", (H, layer.mlp.ff), "linear"
-        yield p + "side.gate", (P, H), "linear"
-        yield p + "side.proj", (H, P), "linear"
-        yield p + "side.norm", (H,), "norm"
+        if cfg.layer_scale:
+            yield p + "ls1", (H,), "scale"
+            if layer.mlp is not None:
+                yield p + "ls2", (H,), "scale"
+        if P:
+            yield p + "side.gate", (P, H), "linear"
+            yield p + "side.proj", (H, P), "linear"
+            yield p + "side.norm", (H,), "norm"
     yield "final.norm", (H,), "norm"
+    if not cfg.tied_head:
+        yield "head", (cfg.vocab_size, H), "linear"
 
 
 def random_weights(cfg: MixedConfig, *, seed: int = 0, dtype=torch.bfloat16, device="cpu", gain: float = 1.0):
     """Weight getter with random values generated on demand (one seeded generator per tensor): linears and embeddings scaled by
-    ``gain / sqrt(columns)`` so that activations stay of order one, norms around one, units uniform in [0, 1)."""
+    ``gain / sqrt(columns)`` so that activations stay of order one, norms around one, units uniform in [0, 1), layer scales around
+    one half, decay rates from 1 to 16 and step sizes from 0.001 to 0.1 (both spread evenly in their logarithms)."""
     table = {name: (idx, shape, kind) for idx, (name, shape, kind) in enumerate(weight_shapes(cfg))}
     dev = torch.device(device)
 
@@ -174,7 +420,16 @@ def random_weights(cfg: MixedConfig, *, seed: int = 0, dtype=torch.bfloat16, dev
         t = torch.empty(shape, dtype=torch.float32, device=dev)
         if kind == "unit":
             return t.uniform_(0, 1, generator=g).to(dtype)
+        if kind == "scale":
+            return t.uniform_(0.25, 0.75, generator=g).to(dtype)
+        if kind == "log_a":
+            return t.uniform_(0.0, math.log(16.0), generator=g).to(dtype)
+        if kind == "dt_bias":
+            step = t.uniform_(math.log(1e-3), math.log(1e-1), generator=g).exp_()
+            return (step + torch.log(-torch.expm1(-step))).to(dtype)
         t.normal_(0.0, 1.0, generator=g)
+        if kind == "correction":
+            return (0.1 * t).to(dtype)
         if kind == "norm":
             return (1.0 + 0.1 * t).to(dtype)
         if kind == "linear":
@@ -185,4 +440,5 @@ def random_weights(cfg: MixedConfig, *, seed: int = 0, dtype=torch.bfloat16, dev
     return get
 
 
-__all__ = ["MixedConfig", "MixedLayer", "LatentAttention", "HGRN2", "DenseMLP", "weight_shapes", "random_weights"]
+__all__ = ["MixedConfig", "MixedLayer", "LatentAttention", "HGRN2", "GroupedAttention", "Mamba1", "Rotary", "YarnScaling", "DenseMLP", "MoE",
+           "weight_shapes", "random_weights"]

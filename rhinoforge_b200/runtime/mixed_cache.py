@@ -1,10 +1,10 @@
-"""Per-sequence state of decoders with per-layer mixers: paged latent rows of the attention layers, fp32 recurrent states of
-the linear-attention layers and the token-shift rows of every layer.
+"""Per-sequence state of decoders with per-layer mixers: paged latent rows or keys and values of the attention layers, fp32
+recurrent states and convolution inputs of the recurrent layers, and the token-shift rows of designs that have them.
 
-Latent rows live in 16-token pages addressed through the page table of :class:`PagedSequences`; a layer's pool is
-``[pages, 16, rank]`` and all layers share the page numbers.  Recurrent and shift state belong to the sequence SLOT: nothing
-has to be cleared when a slot is given to another request, because a row at position 0 starts from an empty state in every
-kernel.
+Latent rows, keys and values live in 16-token pages addressed through the page table of :class:`PagedSequences`; a layer's pool
+is ``[pages, 16, rank]`` (latent) or ``[pages, kv_heads, 16, head size]`` and all layers share the page numbers.  Recurrent,
+convolution and shift state belong to the sequence SLOT: nothing has to be cleared when a slot is given to another request,
+because a row at position 0 starts from an empty state in every kernel.
 """
 from __future__ import annotations
 
@@ -12,12 +12,21 @@ from typing import List, Optional
 
 import torch
 
-from ..models.mixed import HGRN2, LatentAttention, MixedConfig
+from .. import _native as N
+from ..models.mixed import HGRN2, GroupedAttention, LatentAttention, Mamba1, MixedConfig
 from .kv_cache import PAGE_TOKENS, PagedSequences
 
 
 def pad_to(n: int, m: int) -> int:
     return (n + m - 1) // m * m
+
+
+def head_layout(m: GroupedAttention, dtype: torch.dtype):
+    """``(stored head size, runs on the tensor cores)`` of a grouped-attention layer: heads of keys and values are padded to one of
+    the tensor-core kernels' sizes where those take the layer, else to eight values."""
+    big = max(m.dim, m.vdim)
+    hd = next((x for x in (64, 128, 256) if big <= x), 0) if dtype != torch.float32 and m.scale > 0 else 0
+    return (hd, True) if hd else (pad_to(big, 8), False)
 
 
 class MixedCache(PagedSequences):
@@ -29,31 +38,51 @@ class MixedCache(PagedSequences):
         self.cfg, self.dtype, self.num_layers = cfg, dtype, cfg.num_layers
         self._init_pages(batch_size, max_seq_len, device, pool_tokens)
         self.latent: List[Optional[torch.Tensor]] = []
+        self.kv: List[Optional[torch.Tensor]] = []                # [2, pages, kv_heads, 16, head size]
         self.recurrent: List[Optional[torch.Tensor]] = []
+        self.conv: List[Optional[torch.Tensor]] = []
+        zeros = lambda *shape, dt=dtype: torch.zeros(shape, dtype=dt, device=self.device)
         for layer in cfg.layers:
             m = layer.mixer
-            self.latent.append(torch.zeros((self.num_pages, PAGE_TOKENS, pad_to(m.kv_rank, 16)), dtype=dtype, device=self.device)
-                               if isinstance(m, LatentAttention) else None)
-            self.recurrent.append(torch.zeros((batch_size, m.heads, pad_to(m.dim, 8), pad_to(m.vdim, 8)), dtype=torch.float32,
-                                              device=self.device) if isinstance(m, HGRN2) else None)
-        self.shift = torch.zeros((cfg.num_layers, batch_size, pad_to(cfg.hidden_size, 8)), dtype=torch.float32, device=self.device)
+            latent = kv = rec = conv = None
+            if isinstance(m, LatentAttention):
+                latent = zeros(self.num_pages, PAGE_TOKENS, pad_to(m.kv_rank, 16))
+            elif isinstance(m, GroupedAttention):
+                kv = zeros(2, self.num_pages, m.kv_heads, PAGE_TOKENS, head_layout(m, dtype)[0])
+            elif isinstance(m, HGRN2):
+                rec = zeros(batch_size, m.heads, pad_to(m.dim, 8), pad_to(m.vdim, 8), dt=torch.float32)
+            elif isinstance(m, Mamba1):
+                rec = zeros(batch_size, pad_to(m.inner, 8), pad_to(m.state, 8), dt=torch.float32)
+                conv = zeros(batch_size, m.conv - 1, pad_to(m.inner, 8)) if m.conv > 1 else None
+            self.latent.append(latent)
+            self.kv.append(kv)
+            self.recurrent.append(rec)
+            self.conv.append(conv)
+        self.shift = zeros(cfg.num_layers, batch_size, pad_to(cfg.hidden_size, 8), dt=torch.float32) if cfg.token_shift else None
 
-    def layer_ptrs(self, layer: int):
-        """Device addresses ``(latent pool, recurrent state, shift rows)`` of one layer; None where it has none."""
+    def layer_state(self, layer: int) -> N.RfMixedState:
+        """Device addresses of one layer's memory; null where it has none."""
         ptr = lambda t: None if t is None else t.data_ptr()
-        return ptr(self.latent[layer]), ptr(self.recurrent[layer]), self.shift[layer].data_ptr()
+        st = N.RfMixedState()
+        st.latent_pool, st.rec_state, st.conv_state = (ptr(x[layer]) for x in (self.latent, self.recurrent, self.conv))
+        if self.kv[layer] is not None:
+            st.k_pool, st.v_pool, st.pool_pages = self.kv[layer][0].data_ptr(), self.kv[layer][1].data_ptr(), self.num_pages
+        st.shift_state = None if self.shift is None else self.shift[layer].data_ptr()
+        return st
 
     def state_tensors(self) -> List[torch.Tensor]:
-        """Everything a step advances in place (latent pages are only ever written at new positions)."""
-        return [t for t in self.recurrent if t is not None] + [self.shift]
+        """Everything a step advances in place (pages are only ever written at new positions)."""
+        return [t for t in self.recurrent + self.conv + [self.shift] if t is not None]
+
+    def _tensors(self) -> List[torch.Tensor]:
+        return [t for t in self.latent + self.kv if t is not None] + self.state_tensors()
 
     def zero_(self) -> None:
-        for t in self.latent + self.recurrent + [self.shift]:
-            if t is not None:
-                t.zero_()
+        for t in self._tensors():
+            t.zero_()
 
     def nbytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in self.latent + self.recurrent + [self.shift] if t is not None)
+        return sum(t.numel() * t.element_size() for t in self._tensors())
 
 
-__all__ = ["MixedCache", "pad_to"]
+__all__ = ["MixedCache", "head_layout", "pad_to"]

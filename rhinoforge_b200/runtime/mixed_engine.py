@@ -6,23 +6,24 @@ executor is the mixed stack (fp32 residual stream, one mixer per layer), the cac
 addresses sequences through a slot array, so a scheduler step of single tokens replays it for any subset of the live requests.
 
 Weights are padded once at load to the granularity of the kernels (rows of 8 / 16 values, attention heads to 64 / 128 / 256
-for the tcgen05 prefill attention); padding rows and columns are zero.
+for the tcgen05 prefill attention, expert widths to 128 inside the expert banks); padding rows and columns are zero.
 """
 from __future__ import annotations
 
 import ctypes as C
+import math
 import os
 from typing import Dict, List, Optional, Sequence
 
 import torch
 
 from .. import _native as N
-from ..models.mixed import HGRN2, LatentAttention, MixedConfig
+from ..models.mixed import HGRN2, GroupedAttention, LatentAttention, Mamba1, MixedConfig, MoE
 from ..ops import kernels as K
 from ..parallel.tp import TPContext
 from .engine import DecoderEngine, WeightGetter
 from .errors import RPUBackendError
-from .mixed_cache import MixedCache, pad_to
+from .mixed_cache import MixedCache, head_layout, pad_to
 
 
 def _pad2(w: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
@@ -62,7 +63,8 @@ class MixedDecoderEngine(DecoderEngine):
         self.max_batch = max_batch
         self.max_tokens = max(max_prefill_tokens, max_batch)
         self.fp32 = dtype == torch.float32
-        self.packed = not self.fp32 and os.environ.get("RF_PACKED_WEIGHTS", "1") != "0"
+        experts = any(isinstance(layer.mlp, MoE) for layer in cfg.layers)      # expert banks exist in the tile-major form only
+        self.packed = not self.fp32 and (experts or os.environ.get("RF_PACKED_WEIGHTS", "1") != "0")
         self.long_min = (1 << 30) if self.fp32 else self.LONG_MIN
         self.H = pad_to(cfg.hidden_size, 8)
         self.vocab_local = cfg.vocab_size
@@ -108,10 +110,10 @@ class MixedDecoderEngine(DecoderEngine):
         self._keep.append(out)
         return out
 
-    def _linear(self, w: torch.Tensor) -> torch.Tensor:
+    def _linear(self, w: torch.Tensor, sections: int = 1) -> torch.Tensor:
         t = w.to(self.device, self.dtype).contiguous()
         if self.packed:
-            t = K.pack_weight(t)
+            t = K.pack_weight(t, sections)
         self._keep.append(t)
         return t
 
@@ -126,21 +128,27 @@ class MixedDecoderEngine(DecoderEngine):
         P = pad_to(cfg.side_dim, 8)
         V, L = cfg.vocab_size, cfg.num_layers
         self.embed = self._plain(_pad2(g("embed"), V, H))
-        side = g("side.embed").view(V, L, cfg.side_dim)
-        if P != cfg.side_dim:
-            wide = side.new_zeros((V, L, P))
-            wide[:, :, :cfg.side_dim] = side
-            side = wide
-        self.side_table = self._plain(side.reshape(V, L * P))
+        self.side_table = None
+        if P:
+            side = g("side.embed").view(V, L, cfg.side_dim)
+            if P != cfg.side_dim:
+                wide = side.new_zeros((V, L, P))
+                wide[:, :, :cfg.side_dim] = side
+                side = wide
+            self.side_table = self._plain(side.reshape(V, L * P))
         self.final_norm = self._f32(g("final.norm"), H)
-        lm = self._linear(_pad2(self.embed, self.vocab_ld, H))
+        lm = self._linear(_pad2(self.embed if cfg.tied_head else g("head"), self.vocab_ld, H))
+        self._rotations: Dict[object, tuple] = {}
+        self._v_mixing = False                  # has a value-mixing layer been loaded already?
         sc = N.RfMixedConfig()
         sc.layers, sc.hidden, sc.hidden_true, sc.vocab, sc.vocab_ld = L, H, cfg.hidden_size, V, self.vocab_ld
         sc.dtype = 2 if self.fp32 else K.dtype_code(self.dtype)
         sc.max_tokens, sc.max_seqs, sc.max_seq_len = self.max_tokens, self.max_batch, max_context
         sc.side_dim, sc.side_ld, sc.eps = P, L * P, cfg.rms_eps
         sc.weights_packed, sc.long_min = int(self.packed), self.long_min
-        sc.embed, sc.side_table, sc.final_norm, sc.w_lm = (t.data_ptr() for t in (self.embed, self.side_table, self.final_norm, lm))
+        sc.embed, sc.final_norm, sc.w_lm = (t.data_ptr() for t in (self.embed, self.final_norm, lm))
+        sc.side_table = None if self.side_table is None else self.side_table.data_ptr()
+        sc.embed_scale, sc.norm_after = cfg.embed_scale, int(cfg.norm_after)
         h = lib.rf_mixed_create(C.byref(sc))
         if h < 0:
             N.check(-1, "rf_mixed_create")
@@ -148,20 +156,27 @@ class MixedDecoderEngine(DecoderEngine):
         for i, layer in enumerate(cfg.layers):
             m, p = layer.mixer, f"l{i}."
             lw = N.RfMixedLayer()
-            lw.heads = m.heads
-            lw.norm1, lw.shift = self._f32(g(p + "norm1"), H).data_ptr(), self._f32(g(p + "shift"), H).data_ptr()
-            latent, recurrent, shift_rows = self.cache.layer_ptrs(i)
-            lw.shift_state = shift_rows
-            (self._load_latent if isinstance(m, LatentAttention) else self._load_hgrn2)(lw, m, g, p + "mix.")
-            lw.latent_pool, lw.rec_state = latent, recurrent
+            lw.heads = getattr(m, "heads", 0)
+            # layer scales act on the normalised outputs: one factor with the norm's weight
+            norm = lambda name, scale: g(p + name).float() * g(p + scale).float() if cfg.layer_scale else g(p + name)
+            lw.norm1 = self._f32(norm("norm1", "ls1"), H).data_ptr()
+            if cfg.token_shift:
+                lw.shift = self._f32(g(p + "shift"), H).data_ptr()
+            load = {LatentAttention: self._load_latent, HGRN2: self._load_hgrn2, GroupedAttention: self._load_grouped, Mamba1: self._load_mamba1}
+            load[type(m)](lw, m, g, p + "mix.")
+            lw.st = self.cache.layer_state(i)
             if layer.mlp is not None:
+                lw.norm2 = self._f32(norm("norm2", "ls2"), H).data_ptr()
+            if isinstance(layer.mlp, MoE):
+                self._load_moe(lw, layer.mlp, g, p + "mlp.")
+            elif layer.mlp is not None:
                 lw.inter, lw.act = pad_to(layer.mlp.ff, 8), 0
-                lw.norm2 = self._f32(g(p + "norm2"), H).data_ptr()
                 lw.w_up = self._linear(_pad2(g(p + "mlp.up"), lw.inter, H)).data_ptr()
                 lw.w_down = self._linear(_pad2(g(p + "mlp.down"), H, lw.inter)).data_ptr()
-            lw.side_gate = self._linear(_pad2(g(p + "side.gate"), P, H)).data_ptr()
-            lw.side_proj = self._linear(_pad2(g(p + "side.proj"), H, P)).data_ptr()
-            lw.side_norm = self._f32(g(p + "side.norm"), H).data_ptr()
+            if P:
+                lw.side_gate = self._linear(_pad2(g(p + "side.gate"), P, H)).data_ptr()
+                lw.side_proj = self._linear(_pad2(g(p + "side.proj"), H, P)).data_ptr()
+                lw.side_norm = self._f32(g(p + "side.norm"), H).data_ptr()
             N.check(lib.rf_mixed_set_layer(self.handle, i, C.byref(lw)), "rf_mixed_set_layer")
         torch.cuda.empty_cache()
 
@@ -187,7 +202,84 @@ class MixedDecoderEngine(DecoderEngine):
             lw.w_expand = self._linear(torch.cat((uk, uv), 0)).data_ptr()
         o = g(p + "o")
         o = _pad_heads(o.t().contiguous(), m.heads, m.vdim, VD).t()
-        lw.w_o = self._linear(_pad2(o, H, m.heads * VD)).data_ptr()
+        lw.w_o, lw.out_dim = self._linear(_pad2(o, H, m.heads * VD)).data_ptr(), m.heads * VD
+
+    def _rotation(self, rot):
+        """cos and sin tables over the longest context, one pair per distinct rotation."""
+        if rot not in self._rotations:
+            self._rotations[rot] = rot.tables(self._max_context, self.device)
+        return self._rotations[rot]
+
+    def _load_grouped(self, lw, m: GroupedAttention, g, p: str) -> None:
+        H = self.H
+        hd, tensor_core = head_layout(m, self.dtype)
+        lw.mixer, lw.dim, lw.vdim, lw.dim_true, lw.vdim_true = 2, hd, hd, m.dim, m.vdim
+        lw.kv_heads, lw.tensor_core, lw.chunk, lw.scale = m.kv_heads, int(tensor_core), m.chunk or 0, m.scale
+        rows = lambda name, heads, true: _pad_heads(_pad2(g(p + name), heads * true, H), heads, true, hd)
+        parts = [rows("q", m.heads, m.dim), rows("k", m.kv_heads, m.dim), rows("v", m.kv_heads, m.vdim)]
+        if m.gate:
+            parts.append(rows("g", m.heads, m.vdim))
+            lw.gated = 1
+        w_in = torch.cat(parts, 0)
+        lw.in_dim = w_in.shape[0]
+        lw.w_in = self._linear(w_in).data_ptr()
+        if m.qk_norm:
+            lw.q_norm, lw.k_norm = self._f32(g(p + "q.norm"), hd).data_ptr(), self._f32(g(p + "k.norm"), hd).data_ptr()
+        if m.sink:
+            lw.sink = self._f32(g(p + "sink"), m.heads).data_ptr()
+        if m.rot is not None:
+            cos, sin = self._rotation(m.rot)
+            lw.rot_dims, lw.cos, lw.sin = m.rot.dims, cos.data_ptr(), sin.data_ptr()
+        if m.v_mix:
+            lw.v_role = 2 if self._v_mixing else 1
+            lw.v_lambda = float(g(p + "vmix")) if self._v_mixing else 0.0
+            self._v_mixing = True
+        o = _pad_heads(g(p + "o").t().contiguous(), m.heads, m.vdim, hd).t()
+        lw.w_o, lw.out_dim = self._linear(_pad2(o, H, m.heads * hd)).data_ptr(), m.heads * hd
+
+    def _load_mamba1(self, lw, m: Mamba1, g, p: str) -> None:
+        H, I, S, R = self.H, pad_to(m.inner, 8), pad_to(m.state, 8), pad_to(m.dt_rank, 8)
+        lw.mixer, lw.inner, lw.states, lw.dt_rank, lw.taps = 3, I, S, R, m.conv
+        w_in = g(p + "in")
+        w_in = torch.cat([_pad2(w_in[:m.inner], I, H), _pad2(w_in[m.inner:], I, H)], 0)
+        lw.w_in, lw.in_dim = self._linear(w_in).data_ptr(), 2 * I
+        lw.conv_w = self._f32(_pad2(g(p + "conv").t().float(), m.conv, I), m.conv * I).data_ptr()
+        lw.conv_b = self._f32(g(p + "conv.b"), I).data_ptr()
+        dt, b, c = g(p + "x").split((m.dt_rank, m.state, m.state), 0)
+        lw.w_x = self._linear(torch.cat((_pad2(dt, R, I), _pad2(b, S, I), _pad2(c, S, I)), 0)).data_ptr()
+        w_dt = _pad2(g(p + "dt"), I, R)
+        lw.w_dt, lw.w_dt_rows = self._linear(w_dt).data_ptr(), self._plain(w_dt).data_ptr()
+        lw.dt_bias = self._f32(g(p + "dt.b"), I).data_ptr()
+        a2 = g(p + "A_log").double().exp() * (-1.0 / math.log(2.0))       # the kernels raise two to these
+        lw.a2 = self._f32(_pad2(a2.float(), I, S), I * S).data_ptr()
+        lw.d_skip = self._f32(g(p + "D"), I).data_ptr()
+        lw.w_o, lw.out_dim = self._linear(_pad2(g(p + "o"), H, I)).data_ptr(), I
+
+    def _load_moe(self, lw, f: MoE, g, p: str) -> None:
+        """Expert banks: gates then ups of all experts stacked along the rows; downs one behind the other along the columns in
+        16 bits (tile-major image), along the rows in 32."""
+        H, I = self.H, pad_to(f.ff, 8)
+        B = I if self.fp32 else pad_to(f.ff, 128)
+        lw.inter, lw.bank_inter, lw.act = I, B, 0
+        lw.experts, lw.top, lw.groups, lw.keep = f.experts, f.top, f.groups, f.keep
+        lw.score_fn, lw.norm_topk, lw.route_scale = 1, 1, 1.0
+        up = torch.zeros((2, f.experts, B, H), dtype=self.dtype, device=self.device)
+        down = torch.zeros((f.experts, H, B), dtype=self.dtype, device=self.device)
+        for e in range(f.experts):
+            for i, name in enumerate(("gate", "up")):
+                w = g(f"{p}e{e}.{name}")
+                up[i, e, :f.ff, :w.shape[1]] = w
+            w = g(f"{p}e{e}.down")
+            down[e, :w.shape[0], :f.ff] = w
+        lw.w_up = self._linear(up.view(2 * f.experts * B, H), 2).data_ptr()
+        lw.w_down = self._linear(down.view(f.experts * H, B) if self.fp32 else down.transpose(0, 1).reshape(H, f.experts * B)).data_ptr()
+        lw.router = self._plain(_pad2(g(p + "router"), f.experts, H)).data_ptr()
+        lw.correction = self._f32(g(p + "correction"), f.experts).data_ptr()
+        if f.shared_ff:
+            S = lw.shared_inter = pad_to(f.shared_ff, 8)
+            gate_up = torch.cat((_pad2(g(p + "shared.gate"), S, H), _pad2(g(p + "shared.up"), S, H)), 0)
+            lw.shared_up = self._linear(gate_up, 2).data_ptr()
+            lw.shared_down = self._linear(_pad2(g(p + "shared.down"), H, S)).data_ptr()
 
     def _load_hgrn2(self, lw, m: HGRN2, g, p: str) -> None:
         H, D, VD = self.H, pad_to(m.dim, 8), pad_to(m.vdim, 8)
@@ -201,7 +293,7 @@ class MixedDecoderEngine(DecoderEngine):
         lw.lower = self._f32(per_head(g(p + "lower"), 1.0), m.heads * D).data_ptr()    # padding channels keep their (zero) state
         lw.head_norm = self._f32(g(p + "norm"), VD).data_ptr()
         o = _pad_heads(g(p + "o").t().contiguous(), m.heads, m.vdim, VD).t()
-        lw.w_o = self._linear(_pad2(o, H, m.heads * VD)).data_ptr()
+        lw.w_o, lw.out_dim = self._linear(_pad2(o, H, m.heads * VD)).data_ptr(), m.heads * VD
 
     # ------------------------------------------------------------------ cache
     def _check_cache(self, cache) -> None:
@@ -219,13 +311,20 @@ class MixedDecoderEngine(DecoderEngine):
             return
         self._check_cache(cache)
         for i in range(self.cfg.num_layers):
-            N.check(N.lib().rf_mixed_set_state(self.handle, i, *(C.c_void_p(x) for x in cache.layer_ptrs(i))), "rf_mixed_set_state")
+            N.check(N.lib().rf_mixed_set_state(self.handle, i, C.byref(cache.layer_state(i))), "rf_mixed_set_state")
         self.cache = cache
         self.graphs.clear()
         self.batch = 0
         if cache.max_seq_len > self._max_context:
             # attention without a window may have to expand every cached row of a portion's sequence
             self._max_context = cache.max_seq_len
+            if self._rotations:
+                torch.cuda.synchronize()
+                self._rotations.clear()
+                for i, layer in enumerate(self.cfg.layers):
+                    if getattr(layer.mixer, "rot", None) is not None:
+                        N.check(N.lib().rf_mixed_set_rotation(self.handle, i, *(C.c_void_p(t.data_ptr()) for t in self._rotation(layer.mixer.rot))),
+                                "rf_mixed_set_rotation")
             if any(isinstance(layer.mixer, LatentAttention) and layer.mixer.window is None for layer in self.cfg.layers):
                 torch.cuda.synchronize()
                 N.check(N.lib().rf_mixed_set_context(self.handle, self._max_context), "rf_mixed_set_context")
