@@ -43,6 +43,7 @@ struct MixedStack {
   int max_full = 0, max_long_q = 0;
   bool planned = false;
   static constexpr int kSkFlags = 1024;
+  static constexpr int kMoeExperts = 260;     // 256 experts and a ticket, in whole int4
   static constexpr int kMoeSmallRows = 256;   // up to here the experts' weights are streamed past the rows
 
   size_t esz() const { return cfg.dtype == kF32 ? 4 : 2; }
@@ -55,7 +56,7 @@ struct MixedStack {
     auto al = [](uint64_t v) { return (v + 1023) & ~uint64_t(1023); };
     const uint64_t T = (uint64_t)cfg.max_tokens, H = (uint64_t)cfg.hidden, e = esz();
     uint64_t wide = 8, mix = 8, lat = 0, rank = 0, kvw = 0, past = 0, heads = 0;
-    uint64_t vfirst = 0, inner = 0, bc = 0, picks = 0, experts = 0, hg = 0;
+    uint64_t vfirst = 0, inner = 0, bc = 0, picks = 0, hg = 0;
     rows_ws_bytes = 0; moe_tiles = 0;
     for (const RfMixedLayer& l : layers) {
       wide = std::max<uint64_t>(wide, std::max(l.in_dim, l.inter));
@@ -70,7 +71,6 @@ struct MixedStack {
       }
       if (l.experts > 0) {
         picks = std::max<uint64_t>(picks, l.top + 1);
-        experts = std::max<uint64_t>(experts, l.experts);
         hg = std::max<uint64_t>(hg, moe_ld(l));
         moe_tiles = std::max(moe_tiles, l.experts + (int)(T * (l.top + 1) / 16) + 2);
       }
@@ -112,8 +112,8 @@ struct MixedStack {
     off_conv = o; o += al(T * inner * e);
     off_bc = o; o += al(T * bc * e);
     off_dt = o; o += al(fp32() ? 0 : T * inner * e);
-    // ids, weights, rank | slot_of, token_of_slot, slot_w (one column more) | counters, start | tile list
-    off_moe = o; o += al(picks ? (6 * T * picks + 2 * (experts + 4) + 8 + 4ull * moe_tiles) * 4 : 0);
+    // counters, start | tile list | ids, weights, rank | slot_of, token_of_slot, slot_w (one column more)
+    off_moe = o; o += al(picks ? (6 * T * picks + 2 * kMoeExperts + 4 + 4ull * moe_tiles) * 4 : 0);
     off_xg = o; o += al(fp32() || !picks ? 0 : T * (picks - 1) * H * e);
     off_hg = o; o += al(T * picks * hg * e);
     off_yg = o; o += al(T * picks * H * e);
@@ -408,9 +408,8 @@ static int experts(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f
   int32_t* m = s.at<int32_t>(s.off_moe);
   RfMoeRouter r = {};
   r.x = h; r.ldx = H; r.w = w.router; r.correction = w.correction;
-  r.counters = m; m += E + 4;
-  r.start = m; m += E + 4;
-  m = s.at<int32_t>(s.off_moe) + ((m - s.at<int32_t>(s.off_moe) + 3) & ~3);
+  r.counters = m; m += MixedStack::kMoeExperts;      // the same place whatever a layer's expert count: they are zero between launches
+  r.start = m; m += MixedStack::kMoeExperts;
   r.tiles = m; m += 4 + 4 * s.moe_tiles;
   r.ids = m; m += pairs;
   r.weights = (float*)m; m += pairs;

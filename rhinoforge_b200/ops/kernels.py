@@ -413,11 +413,14 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, *, Hq: int, Hkv: int, 
                       kv_start: Optional[torch.Tensor] = None, causal: bool = True, window: int = 0,
                       mask: Optional[torch.Tensor] = None, seg_q: Optional[torch.Tensor] = None,
                       seg_k: Optional[torch.Tensor] = None, scale: float = 0.0,
-                      status: Optional[torch.Tensor] = None, max_kv_len: int = 0) -> torch.Tensor:
+                      status: Optional[torch.Tensor] = None, max_kv_len: int = 0, slot: Optional[torch.Tensor] = None, chunk: int = 0,
+                      sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Flash-style attention over ``q`` rows [tokens, Hq*hd]; KV from the paged pool or from
     contiguous ``k``/``v`` [rows, Hkv*hd] (may be column slices of a packed qkv buffer).
     ``max_kv_len``: a host-side bound on ``kv_len`` (0: unknown); short contiguous problems (at most 64 query rows per
-    sequence over at most 512 keys, heads of 64 / 128, causal / window masks only) then take the low-latency kernel."""
+    sequence over at most 512 keys, heads of 64 / 128, causal / window masks only) then take the low-latency kernel.
+    Paged form: ``slot`` names every sequence's page-table row, ``chunk`` limits every position to its own chunk, ``sink`` ``[Hq]``
+    adds ``exp(sink)`` to the softmax denominators, the result is multiplied by ``sigmoid(gate)``."""
     a = N.RfAttn()
     a.q, a.ldq, a.out, a.ldo = q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0)
     a.q_rows_total = q.shape[0]
@@ -438,6 +441,8 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, *, Hq: int, Hkv: int, 
         a.mask_seq_stride = mask.stride(0) if mask.dim() == 3 else 0
     a.seg_q, a.seg_k = _i32(seg_q), _i32(seg_k)
     a.scale = scale
+    a.slot, a.chunk, a.sink = _i32(slot), chunk, _ptr(sink)
+    a.gate, a.ld_gate = _ptr(gate), 0 if gate is None else gate.stride(0)
     a.status = _ptr(status)
     a.dtype = dtype_code(q.dtype)
     N.check(N.lib().rf_attn_prefill(C.byref(a), _stream()), "rf_attn_prefill")
@@ -463,6 +468,27 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, *, Hq: int, Hkv: int, h
     a.status = _ptr(status)
     a.dtype = dtype_code(q.dtype)
     N.check(N.lib().rf_attn_decode(C.byref(a), _stream()), "rf_attn_decode")
+    return out
+
+
+def attention_rows(q: torch.Tensor, r, k_pool: torch.Tensor, v_pool: torch.Tensor, *, Hq: int, Hkv: int, hd: int, scale: float, max_kv: int,
+                   chunk: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, split: bool = True,
+                   tensor_core: bool = True) -> torch.Tensor:
+    """Every row of ``q [rows, Hq * hd]`` over the cached keys of its sequence up to its own position (``r``: :func:`rows`), with the
+    options of :func:`attention_prefill`.  ``tensor_core=False``: the fp32 kernel for any head size and dtype."""
+    out = torch.empty((q.shape[0], Hq * hd), dtype=q.dtype, device=q.device)
+    a = N.RfAttn()
+    a.q, a.ldq, a.out, a.ldo, a.q_rows_total, a.num_seqs = q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), q.shape[0], q.shape[0]
+    a.Hq, a.Hkv, a.hd, a.scale, a.max_kv_len, a.chunk, a.sink = Hq, Hkv, hd, scale, max_kv, chunk, _ptr(sink)
+    a.k_pool, a.v_pool, a.pool_pages = k_pool.data_ptr(), v_pool.data_ptr(), k_pool.shape[0]
+    a.page_table, a.pt_stride, a.slot, a.seq_of_row, a.pos = r.page_table, r.pt_stride, r.slot, r.seq_of_row, r.pos
+    a.gate, a.ld_gate = _ptr(gate), 0 if gate is None else gate.stride(0)
+    if split and tensor_core:
+        ws = torch.empty(N.lib().rf_attn_decode_scratch_bound(Hq, Hkv, hd), dtype=torch.uint8, device=q.device)
+        a.ws, a.ws_bytes = ws.data_ptr(), ws.numel()
+    a.dtype = dtype_code_any(q.dtype)
+    fn = "rf_attn_decode" if tensor_core else "rf_attn_rows"
+    N.check(getattr(N.lib(), fn)(C.byref(a), _stream()), fn)
     return out
 
 
@@ -579,10 +605,12 @@ def rows(pos: torch.Tensor, *, seq_of_row: Optional[torch.Tensor] = None, q_star
 def stream_norm(x: Optional[torch.Tensor], r, *, dtype: torch.dtype, eps: float, norm_w: Optional[torch.Tensor] = None,
                 table: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None,
                 y_norm_w: Optional[torch.Tensor] = None, shift: Optional[torch.Tensor] = None,
-                shift_state: Optional[torch.Tensor] = None, dim: Optional[int] = None, cast: bool = False):
+                shift_state: Optional[torch.Tensor] = None, dim: Optional[int] = None, cast: bool = False, embed_scale: float = 1.0,
+                y_slots: Optional[torch.Tensor] = None):
     """One step of an fp32 residual stream: add the outstanding sublayer output ``y`` (RMS-normed with ``y_norm_w``), RMSNorm
     with ``norm_w``, mix with the previous token's normalised row (``shift``, state per slot).  Without ``x`` the stream starts
-    from ``table[ids]``.  Returns ``(x_out fp32, h or None, x in dtype or None)``."""
+    from ``table[ids] * embed_scale``.  ``y_slots [rows, picks]``: the outstanding output is the sum of these rows of ``y`` (negative:
+    none).  Returns ``(x_out fp32, h or None, x in dtype or None)``."""
     H = (x if x is not None else table).shape[1]
     n = x.shape[0] if x is not None else ids.numel()
     dev = (x if x is not None else table).device
@@ -593,6 +621,7 @@ def stream_norm(x: Optional[torch.Tensor], r, *, dtype: torch.dtype, eps: float,
     a.x, a.table, a.ids, a.y, a.y_norm_w = _ptr(x), _ptr(table), _ptr(ids), _ptr(y), _ptr(y_norm_w)
     a.x_out, a.x_cast, a.norm_w, a.out, a.shift, a.shift_state = _ptr(x_out), _ptr(xc), _ptr(norm_w), _ptr(h), _ptr(shift), _ptr(shift_state)
     a.rows, a.n_rows, a.H, a.dim, a.eps, a.dtype = r, n, H, dim or H, eps, dtype_code_any(dtype)
+    a.embed_scale, a.y_slots, a.y_picks = embed_scale, _i32(y_slots), 0 if y_slots is None else y_slots.shape[1]
     N.check(N.lib().rf_stream_norm(C.byref(a), _stream()), "rf_stream_norm")
     return x_out, h, xc
 
@@ -676,7 +705,112 @@ def hgrn2(x: torch.Tensor, f_bias: torch.Tensor, lower: torch.Tensor, norm_w: Op
     return out
 
 
+def qkv_insert(qkv: torch.Tensor, r, k_pool: torch.Tensor, v_pool: torch.Tensor, *, heads: int, kv_heads: int, hd: int, eps: float,
+               dim: Optional[int] = None, vdim: Optional[int] = None, q_norm: Optional[torch.Tensor] = None,
+               k_norm: Optional[torch.Tensor] = None, cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None,
+               v_first: Optional[torch.Tensor] = None, v_role: str = "none", v_lambda: float = 0.0) -> None:
+    """Per-head norms, rotation, value mixing and page insertion of packed rows ``[q | k | v]`` (heads of ``hd`` values, ``dim`` /
+    ``vdim`` of them used); queries are replaced in place, keys and values go to the pools ``[pages, kv_heads, 16, hd]``."""
+    a = N.RfQkvInsert()
+    a.qkv, a.ld, a.k_off, a.v_off = qkv.data_ptr(), qkv.stride(0), heads * hd, (heads + kv_heads) * hd
+    a.q_norm, a.k_norm, a.cos, a.sin, a.v_first = _ptr(q_norm), _ptr(k_norm), _ptr(cos), _ptr(sin), _ptr(v_first)
+    a.k_pool, a.v_pool, a.rows, a.n_rows = k_pool.data_ptr(), v_pool.data_ptr(), r, qkv.shape[0]
+    a.heads, a.kv_heads, a.hd, a.dim, a.vdim = heads, kv_heads, hd, dim or hd, vdim or hd
+    a.rot_dims = 0 if cos is None else 2 * cos.shape[1]
+    a.v_role, a.v_lambda, a.eps, a.dtype = {"none": 0, "first": 1, "mix": 2}[v_role], v_lambda, eps, dtype_code_any(qkv.dtype)
+    N.check(N.lib().rf_qkv_insert(C.byref(a), _stream()), "rf_qkv_insert")
+
+
+def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor], r, *, max_q_len: int = 1) -> torch.Tensor:
+    """Causal convolution per channel and silu over packed rows; ``w`` fp32 ``[taps, channels]``, ``state [slots, taps - 1, channels]``
+    holds the last inputs and is replaced."""
+    y = torch.empty((x.shape[0], w.shape[1]), dtype=x.dtype, device=x.device)
+    a = N.RfConvSilu()
+    a.x, a.ldx, a.y, a.ldy, a.w, a.bias, a.state = x.data_ptr(), x.stride(0), y.data_ptr(), y.stride(0), w.data_ptr(), _ptr(bias), _ptr(state)
+    a.rows, a.max_q_len, a.channels, a.taps, a.dtype = r, max_q_len, w.shape[1], w.shape[0], dtype_code_any(x.dtype)
+    N.check(N.lib().rf_conv_silu(C.byref(a), _stream()), "rf_conv_silu")
+    return y
+
+
+def mamba1(x: torch.Tensor, z: torch.Tensor, bc: torch.Tensor, a2: torch.Tensor, d: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, r, *,
+           w_dt: Optional[torch.Tensor] = None, dt: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Selective scan over packed rows with the fp32 ``state [slots, inner, states]`` updated in place.  With ``dt`` (projected step
+    sizes) the tiled scan, else the recurrence, which projects the step-size columns of ``bc`` with ``w_dt [inner, rank]`` itself."""
+    I, S = a2.shape
+    out = torch.empty((x.shape[0], I), dtype=x.dtype, device=x.device)
+    a = N.RfMamba1()
+    a.x, a.ldx, a.z, a.ldz, a.bc, a.ld_bc = x.data_ptr(), x.stride(0), z.data_ptr(), z.stride(0), bc.data_ptr(), bc.stride(0)
+    a.dt, a.ld_dt, a.w_dt = _ptr(dt), 0 if dt is None else dt.stride(0), _ptr(w_dt)
+    a.dt_bias, a.a2, a.d, a.state, a.out, a.ldo = dt_bias.data_ptr(), a2.data_ptr(), d.data_ptr(), state.data_ptr(), out.data_ptr(), I
+    a.rows, a.inner, a.states, a.rank, a.dtype = r, I, S, bc.shape[1] - 2 * S, dtype_code_any(x.dtype)
+    fn = "rf_mamba1_recurrent" if dt is None else "rf_mamba1_scan"
+    N.check(getattr(N.lib(), fn)(C.byref(a), _stream()), fn)
+    return out
+
+
 # ----------------------------------------------------------------------------- mixture of experts
+class RoutedBatch:
+    """Router of one batch and everything its expert GEMMs need (:func:`moe_router`)."""
+
+    def __init__(self, x: torch.Tensor, w: torch.Tensor, k: int, *, correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1,
+                 score_fn: str = "softmax", norm_topk: bool = True, scale: float = 1.0, tile_rows: int = 16, shared: bool = False,
+                 scatter: bool = True):
+        T, E = x.shape[0], w.shape[0]
+        i32 = lambda *sh: torch.zeros(sh, dtype=torch.int32, device=x.device)
+        self.x, self.w, self.correction, self.tile_rows, self.k = x, w, correction, tile_rows, k
+        self.ids, self.weights, self.rank = i32(T, k), torch.zeros((T, k), dtype=torch.float32, device=x.device), i32(T, k)
+        self.counters, self.start = i32(E + 1), i32(E)
+        self.max_tiles = min(E, T * k) + T * k // tile_rows + ((T + tile_rows - 1) // tile_rows if shared else 0)
+        self.tiles = i32(4 * (self.max_tiles + 1))
+        self.slot_of, self.token_of_slot = i32(T, k + shared), i32(T * (k + shared))
+        self.slot_w = torch.zeros(T * (k + shared), dtype=torch.float32, device=x.device)
+        a = self.args = N.RfMoeRouter()
+        a.x, a.ldx, a.w, a.correction = x.data_ptr(), x.stride(0), w.data_ptr(), _ptr(correction)
+        a.ids, a.weights, a.rank, a.counters, a.start, a.tiles, a.slot_of, a.token_of_slot, a.slot_w = (t.data_ptr() for t in (
+            self.ids, self.weights, self.rank, self.counters, self.start, self.tiles, self.slot_of, self.token_of_slot, self.slot_w))
+        a.rows, a.experts, a.width, a.k, a.groups, a.keep = T, E, w.shape[1], k, groups, keep
+        a.score_fn, a.norm_topk, a.scale = {"sigmoid": 0, "softmax": 1}[score_fn], int(norm_topk), scale
+        a.tile_rows, a.slot_ld, a.has_shared, a.shared_tiles, a.scatter = tile_rows, k + shared, int(shared), int(shared and scatter), int(scatter)
+        a.dtype = dtype_code_any(x.dtype)
+
+    def route(self) -> "RoutedBatch":
+        N.check(N.lib().rf_moe_router(C.byref(self.args), _stream()), "rf_moe_router")
+        return self
+
+    def gather(self) -> torch.Tensor:
+        """Rows of ``x`` in sorted order (also fills ``slot_of``, ``token_of_slot`` and ``slot_w``)."""
+        out = torch.zeros((self.x.shape[0] * self.k, self.x.shape[1]), dtype=self.x.dtype, device=self.x.device)
+        N.check(N.lib().rf_moe_gather(C.byref(self.args), C.c_void_p(out.data_ptr()), C.c_int64(out.stride(0)), _stream()), "rf_moe_gather")
+        return out
+
+
+def moe_router(x: torch.Tensor, w: torch.Tensor, k: int, **kw) -> RoutedBatch:
+    """Logits (fp32), scores, group-limited choice, weights and the tile list of the expert GEMMs, in one launch."""
+    return RoutedBatch(x, w, k, **kw).route()
+
+
+def moe_experts(b: RoutedBatch, x: torch.Tensor, bank: torch.Tensor, *, n: int, k: int, experts: int, expert_pad: int = 0, dual: bool = False,
+                gathered: bool = True, weighted: bool = False, shared: Optional[torch.Tensor] = None, shared_n: int = 0, shared_k: int = 0,
+                out_cols: int = 0) -> torch.Tensor:
+    """Expert GEMMs of few rows over the tile list of a routed batch; ``bank`` (and ``shared``) as the mixed engine packs them,
+    ``expert_pad`` the padded expert width inside 16-bit banks."""
+    cols = max(out_cols, n, shared_n)
+    out = torch.zeros((b.slot_w.numel(), cols), dtype=x.dtype, device=x.device)
+    a = N.RfMoeExperts()
+    a.x, a.ldx, a.w, a.w_shared, a.out, a.ldo = x.data_ptr(), x.stride(0), bank.data_ptr(), _ptr(shared), out.data_ptr(), cols
+    a.tiles, a.token_of_slot, a.slot_w = b.tiles.data_ptr(), b.token_of_slot.data_ptr() if gathered else None, b.slot_w.data_ptr() if weighted else None
+    a.max_tiles, a.experts, a.n, a.k, a.shared_n, a.shared_k, a.dual, a.tile_rows = b.max_tiles, experts, n, k, shared_n, shared_k, int(dual), b.tile_rows
+    up = lambda v, m: (v + m - 1) // m
+    if dual:
+        a.bank_section_row_tiles, a.bank_kb_total, a.rt_per_expert = experts * expert_pad // 128, up(k, 64), expert_pad // 128
+        a.shared_section_row_tiles, a.shared_kb_total = up(shared_n, 128), up(shared_k, 64)
+    else:
+        a.bank_kb_total, a.kb_per_expert, a.shared_kb_total = experts * expert_pad // 64, expert_pad // 64, up(shared_k, 64)
+    a.dtype = dtype_code_any(x.dtype)
+    N.check(N.lib().rf_moe_experts(C.byref(a), _stream()), "rf_moe_experts")
+    return out
+
+
 def moe_select(logits: torch.Tensor, k: int, *, bias: Optional[torch.Tensor] = None, score_fn: str = "sigmoid",
                norm_topk: bool = True, scale: float = 1.0, dense: bool = False):
     """Router top-k.  Returns ``(ids [T,k] int32, weights [T,k] fp32)`` and, with ``dense=True``, also the
