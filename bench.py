@@ -29,10 +29,11 @@ def parse_args(argv=None):
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="decode", choices=["decode", "pi05", "qwen3vl", "vabarax"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "pi05", "qwen3vl", "vabarax", "zulopel"],
                     help="decode: causal-LM decode throughput (headline); pi05: action-chunk latency; "
-                         "qwen3vl: multimodal prefill + decode; vabarax: latent-attention / HGRN2 decoder beside the "
-                         "hybrid K/V + Gated-DeltaNet decoder at equal size")
+                         "qwen3vl: multimodal prefill + decode; vabarax: latent-attention / HGRN2 decoder, zulopel: chunked "
+                         "attention / selective-scan decoder with routed experts, each beside the hybrid K/V + "
+                         "Gated-DeltaNet decoder at equal size")
     ap.add_argument("--model", default="qwen3-8b")
     ap.add_argument("--batch", type=int, default=64)
     ap.add_argument("--prompt-len", type=int, default=1024)
@@ -544,6 +545,13 @@ VABARAX_SIZES = {          # width, heads (of 128), latent rank, window, feed-fo
 }
 
 
+ZULOPEL_SIZES = {          # width, heads (of 128), K/V heads, chunk, scan channels, experts, top, groups, kept groups, expert and shared width, layers
+    "16e": (2048, 16, 4, 2048, 4096, 16, 2, 4, 2, 1024, 2048, 16),
+    "32e": (3072, 24, 6, 2048, 6144, 32, 4, 8, 4, 1024, 2048, 16),
+    "64e": (4096, 32, 8, 2048, 8192, 64, 6, 8, 4, 1408, 2816, 8),
+}
+
+
 def _serve(eng, vocab: int, batches, prompt_len: int, steps: int, warmup: int, total_prompts: int):
     """Device-timed prefill of ``total_prompts`` prompts and decode steps at every batch size of one engine."""
     import torch
@@ -595,34 +603,63 @@ def _serve(eng, vocab: int, batches, prompt_len: int, steps: int, warmup: int, t
 
 
 def run_vabarax(args) -> dict:
-    """Prefill and decode throughput of the Vabarax design at a few sizes, beside the closest decoder of this framework - the
-    hybrid of softmax attention (grouped K/V heads, SwiGLU) and Gated-DeltaNet layers - with the same width, heads, feed-forward
-    parameters, layer count, prompts and batch sizes.  Random weights, synthetic ids; a "step" is one decode step."""
+    """The Vabarax design; see :func:`_beside_hybrid`."""
+    from rhinoforge_b200.models.mixed import DenseMLP, HGRN2, LatentAttention, MixedConfig, MixedLayer
+    entries = {}
+    for name, (H, heads, rank, window, ff, side, layers) in VABARAX_SIZES.items():
+        att = MixedLayer(LatentAttention(heads, 128, 128, rank, 128 ** -0.5, window), DenseMLP(ff))
+        lin = MixedLayer(HGRN2(heads, 128, 128), DenseMLP(ff))
+        # a GLU of 2/3 of the width has the same feed-forward parameters
+        entries[name] = (lambda v, n=name, h=H, ls=(att, lin) * (layers // 2), p=side: MixedConfig("vabarax-" + n, v, h, 1e-6, ls, p),
+                         heads, heads // 4, 2 * ff // 3)
+    keys = ("width", "heads", "rank", "window", "ff", "side", "layers")
+    return _beside_hybrid(args, "vabarax", "Vabarax-8b-sized", entries, {k: dict(zip(keys, v)) for k, v in VABARAX_SIZES.items()})
+
+
+def run_zulopel(args) -> dict:
+    """The Zulopel design; see :func:`_beside_hybrid`.  The hybrid decoder's feed-forward is as wide as the experts that one token
+    uses, shared expert included."""
+    from rhinoforge_b200.models.mixed import GroupedAttention, Mamba1, MixedConfig, MixedLayer, MoE, Rotary, YarnScaling
+    entries = {}
+    for name, (H, heads, kv, chunk, inner, experts, top, groups, keep, ff, shared, layers) in ZULOPEL_SIZES.items():
+        moe = MoE(experts, top, ff, groups, keep, shared)
+        rot = Rotary(64, 5e5, YarnScaling(8.0, 8192, 32.0, 1.0))
+        att = MixedLayer(GroupedAttention(heads, kv, 128, 128, 128 ** -0.5, chunk, rot, True), moe)
+        scan = MixedLayer(Mamba1(inner, 16, H // 16, 4), moe)
+        entries[name] = (lambda v, n=name, h=H, ls=(scan, att) * (layers // 2): MixedConfig.zulopel("zulopel-" + n, v, h, 1e-6, ls, h ** 0.5),
+                         heads, kv, top * ff + shared)
+    keys = ("width", "heads", "kv_heads", "chunk", "scan_channels", "experts", "top", "groups", "keep", "ff", "shared_ff", "layers")
+    return _beside_hybrid(args, "zulopel", "Zulopel 64-expert", entries, {k: dict(zip(keys, v)) for k, v in ZULOPEL_SIZES.items()})
+
+
+def _beside_hybrid(args, design: str, headline: str, entries: dict, sizes: dict) -> dict:
+    """Prefill and decode throughput of a design with per-layer mixers at a few sizes, beside the closest decoder of this framework
+    - the hybrid of softmax attention (grouped K/V heads, SwiGLU) and Gated-DeltaNet layers - with the same width, heads, layer
+    count, prompts and batch sizes.  ``entries``: size name -> (config of a vocabulary size, heads, K/V heads, SwiGLU width of the
+    hybrid).  Random weights, synthetic ids; a "step" is one decode step."""
     import torch
     from rhinoforge_b200.models.decoder import DecoderConfig
-    from rhinoforge_b200.models.mixed import DenseMLP, HGRN2, LatentAttention, MixedConfig, MixedLayer, random_weights, weight_shapes
+    from rhinoforge_b200.models.mixed import random_weights, weight_shapes
     from rhinoforge_b200.runtime.engine import DecoderEngine, random_weight_getter
     from rhinoforge_b200.runtime.mixed_engine import MixedDecoderEngine
     if args.gpus != 1:
-        raise SystemExit("the vabarax workload runs on one GPU")
+        raise SystemExit(f"the {design} workload runs on one GPU")
     torch.cuda.set_device(0)
     batches = sorted({1, 8, args.batch})
     vocab, prompt, npre = 32768, args.prompt_len, 8
     max_seq = prompt + 2 * args.steps + args.warmup + 128
     res = {}
-    for name, (H, heads, rank, window, ff, side, layers) in VABARAX_SIZES.items():
-        att = MixedLayer(LatentAttention(heads, 128, 128, rank, 128 ** -0.5, window), DenseMLP(ff))
-        lin = MixedLayer(HGRN2(heads, 128, 128), DenseMLP(ff))
-        cfg = MixedConfig("vabarax-" + name, vocab, H, 1e-6, (att, lin) * (layers // 2), side)
+    for name, (make, heads, kv_heads, inter) in entries.items():
+        cfg = make(vocab)
+        H, layers = cfg.hidden_size, cfg.num_layers
         eng = MixedDecoderEngine(cfg, random_weights(cfg, device="cuda"), dtype=torch.bfloat16, max_batch=max(batches), max_seq_len=max_seq)
         r = {"params_m": round(sum(int(torch.Size(s).numel()) for _, s, _ in weight_shapes(cfg)) / 1e6), "ours": _serve(
             eng, vocab, batches, prompt, args.steps, args.warmup, npre), "cache_mb": round(eng.cache.nbytes() / 1e6)}
         eng.close()
         del eng
         torch.cuda.empty_cache()
-        # the closest existing decoder: a GLU of 2/3 of the width has the same feed-forward parameters
-        inter = (2 * ff // 3 + 127) // 128 * 128
-        like = DecoderConfig("hybrid-" + name, vocab, H, inter, layers, heads, heads // 4, 128, tie_embeddings=True, norm="rms_gemma",
+        inter = (inter + 127) // 128 * 128
+        like = DecoderConfig("hybrid-" + name, vocab, H, inter, layers, heads, kv_heads, 128, tie_embeddings=True, norm="rms_gemma",
                              attn_gate=True, model_type="qwen3_5", layer_types=("full_attention", "linear_attention") * (layers // 2),
                              gdn_heads_k=heads, gdn_heads_v=heads, gdn_dk=128, gdn_dv=128)
         try:
@@ -637,12 +674,11 @@ def run_vabarax(args) -> dict:
         res[name] = r
     big = list(res.values())[-1]["ours"]
     d = big["decode"][str(args.batch)]
-    return {"metric": "vabarax_decode_tokens_per_s", "value": d["tok_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
+    return {"metric": f"{design}_decode_tokens_per_s", "value": d["tok_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
             "warmup": max(args.warmup, 3), "ms_per_step": d["ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None,
             "dtype": "bf16", "data": "synthetic", "impl": "ours",
-            "config": {"model": "Vabarax-8b-sized random-init", "global_batch": args.batch, "seq_len": prompt, "parallelism": "tp1",
-                       "sizes": {k: dict(zip(("width", "heads", "rank", "window", "ff", "side", "layers"), v)) for k, v in VABARAX_SIZES.items()},
-                       "l2": "weights exceed L2"},
+            "config": {"model": f"{headline} random-init", "global_batch": args.batch, "seq_len": prompt, "parallelism": "tp1",
+                       "sizes": sizes, "l2": "weights exceed L2"},
             "clocks": d["clocks"], "e2e": {"value": big["e2e_tok_s"], "unit": "tokens/s", "h2d_bytes_per_step": 12 * args.batch,
                                            "d2h_bytes_per_step": 4 * args.batch},
             "gpu_launches": d["launches_per_step"] * args.steps, "by_size": res}
@@ -673,7 +709,7 @@ def main(argv=None) -> int:
         if int(os.environ.get("RANK", "0")) == 0:          # one line per job, also under torch.distributed.run
             print(json.dumps({"impl": "reference", "unavailable": REFERENCE_UNAVAILABLE}))
         return 0
-    out = {"decode": run, "pi05": run_pi05, "qwen3vl": run_qwen3vl, "vabarax": run_vabarax}[args.workload](args)
+    out = {"decode": run, "pi05": run_pi05, "qwen3vl": run_qwen3vl, "vabarax": run_vabarax, "zulopel": run_zulopel}[args.workload](args)
     if out is not None:
         print(json.dumps(out))
     try:

@@ -429,7 +429,7 @@ def random_weights(cfg: MixedConfig, *, seed: int = 0, dtype=torch.bfloat16, dev
             return (step + torch.log(-torch.expm1(-step))).to(dtype)
         t.normal_(0.0, 1.0, generator=g)
         if kind == "correction":
-            return (0.1 * t).to(dtype)
+            return (t * (0.25 / shape[0])).to(dtype)           # of the order of a softmax score
         if kind == "norm":
             return (1.0 + 0.1 * t).to(dtype)
         if kind == "linear":
