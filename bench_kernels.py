@@ -6,6 +6,7 @@
     python bench_kernels.py attn_decode --seqs 64 --len 1024 --heads 32 --kv-heads 8 --hd 128
     python bench_kernels.py gdn --seqs 1 --len 1024 --hk 16 --hv 32
     python bench_kernels.py mixed            # latent attention / HGRN2 / fp32 stream beside the like kernels at equal size
+    python bench_kernels.py routed           # chunked attention / selective scan / routed experts beside the like kernels
     python bench_kernels.py suite            # the shapes of one Qwen3-8B decode step and prefill chunk
 
 Every line is JSON: the achieved throughput and its fraction of the measured peaks in
@@ -381,6 +382,143 @@ def bench_mixed(hidden, heads, *, dim=128, vdim=128, rank=512, window=1024, batc
         bench_gdn(s_, l_, heads, heads, dtype=dtype, timer=time_cold_us, chunked=True)
 
 
+def bench_routed(hidden, heads, kv, inner, experts, top, ff, *, chunk=1024, groups=8, keep=4, states=16, batch=64, prefill=(4, 2048),
+                 dtype=torch.bfloat16) -> None:
+    """Kernels of decoders with chunked grouped attention, selective-scan layers and routed experts, each beside the like kernel of
+    the K/V and Gated-DeltaNet decoders at equal size."""
+    from rhinoforge_b200.ops import kernels as K
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
+    tag = dict(hidden=hidden)
+    rnd = lambda *sh: torch.randn(*sh, device="cuda", dtype=dtype)
+    f32 = lambda *sh: torch.randn(*sh, device="cuda")
+    S, Lp = prefill
+    T, hd = S * Lp, 128
+    starts, lens = i32([j * Lp for j in range(S)]), i32([Lp] * S)
+    seq, pos_p = i32([j for j in range(S) for _ in range(Lp)]), i32(list(range(Lp)) * S)
+    rows_p = lambda **kw: K.rows(pos_p, seq_of_row=seq, q_start=starts, q_len=lens, slot=i32(list(range(S))), **kw)
+    # ---- residual stream: the experts' rows added up
+    for n, r in ((batch, K.rows(i32([7] * batch))), (T, rows_p())):
+        x, yw, w16 = f32(n, hidden), f32(hidden), rnd(hidden)
+        yg, slots = rnd(n * (top + 1), hidden), torch.randperm(n * (top + 1), device="cuda").to(torch.int32).view(n, top + 1)
+        us = time_cold_us(lambda: K.stream_norm(x, r, dtype=dtype, eps=1e-6, y=yg, y_norm_w=yw, cast=True, y_slots=slots))
+        report("stream_norm (sum of picked rows, norm of it, add)", us, bytes_=n * hidden * (10 + 2 * (top + 1)), rows=n, picks=top + 1, **tag)
+        y1 = rnd(n, hidden)
+        us = time_cold_us(lambda: K.stream_norm(x, r, dtype=dtype, eps=1e-6, y=y1, y_norm_w=yw, cast=True))
+        report("stream_norm (norm of the output, add)", us, bytes_=n * hidden * 12, rows=n, **tag)
+        xx, out = rnd(n, hidden), rnd(n, hidden)
+        us = time_cold_us(lambda: K.rmsnorm(xx, w16, 1e-6, residual=y1, residual_out=xx, out=out))
+        report("like: rmsnorm with residual", us, bytes_=n * hidden * 8, rows=n, **tag)
+        del yg
+    # ---- attention
+    cos, sin = f32(4096, 32), f32(4096, 32)
+    qn, qn16 = f32(hd), rnd(hd)
+    for n, r_of, posn in ((batch, lambda **kw: K.rows(i32([chunk - 1] * batch), **kw), i32([chunk - 1] * batch)), (T, rows_p, pos_p)):
+        per = (max(Lp, chunk) + 15) // 16
+        nseq = batch if n == batch else S
+        pt = torch.randperm(nseq * per, device="cuda").to(torch.int32).view(nseq, per)
+        kp, vp = rnd(nseq * per, kv, 16, hd), rnd(nseq * per, kv, 16, hd)
+        x, first = rnd(n, (2 * heads + 2 * kv) * hd), rnd(n, kv * hd)
+        r = r_of(page_table=pt)
+        us = time_cold_us(lambda: K.qkv_insert(x, r, kp, vp, heads=heads, kv_heads=kv, hd=hd, eps=1e-6, q_norm=qn, k_norm=qn, cos=cos, sin=sin,
+                                               v_first=first, v_role="mix", v_lambda=0.5))
+        report("qkv_insert", us, bytes_=n * ((2 * heads + 4 * kv) * hd * 2 + kv * hd * 2), rows=n, heads=heads, kv_heads=kv, **tag)
+        x2 = rnd(n, (heads + 2 * kv) * hd)
+        us = time_cold_us(lambda: K.qk_norm_rope_kv(x2, heads, kv, hd, pos=posn.view(-1, 1), cos=cos, sin=sin, rot_dim=64, q_norm_w=qn16, k_norm_w=qn16,
+                                                    k_pool=kp, v_pool=vp, page_table=pt, seq_of_tok=None if n == batch else seq))
+        report("like: qk_norm_rope_kv", us, bytes_=n * (2 * heads + 4 * kv) * hd * 2, rows=n, **tag)
+        kw = dict(Hq=heads, Hkv=kv, hd=hd, scale=0.09, sink=f32(heads), gate=x[:, (heads + 2 * kv) * hd:])
+        q = x[:, :heads * hd]
+        if n == batch:
+            for b in (1, batch):
+                rb = K.rows(i32([chunk - 1] * b), page_table=pt[:b])
+                us = time_cold_us(lambda: K.attention_rows(q[:b], rb, kp, vp, max_kv=chunk, chunk=chunk, **kw))
+                report("attention by row (chunk, sink, gate)", us, bytes_=4.0 * b * chunk * kv * hd + 6.0 * b * heads * hd, rows=b, chunk=chunk, **tag)
+                bench_attn_decode(b, chunk, heads, kv, hd, dtype=dtype, timer=time_cold_us)
+        else:
+            out = rnd(n, heads * hd)
+            for ch in (chunk, Lp):
+                vis = sum(i % ch + 1 for i in range(Lp)) * S
+                us = time_cold_us(lambda: K.attention_prefill(q, out, q_start=starts, q_len=lens, kv_len=lens, max_q_len=Lp, k_pool=kp, v_pool=vp,
+                                                              page_table=pt, max_kv_len=Lp, chunk=ch, **kw))
+                report("attention prefill (chunk, sink, gate)", us, flops=4.0 * vis * heads * hd, rows=n, chunk=ch, **tag)
+            bench_attn_prefill(S, Lp, heads, kv, hd, dtype=dtype, timer=time_cold_us)
+            bench_attn_prefill(S * Lp // chunk, chunk, heads, kv, hd, dtype=dtype, timer=time_cold_us)
+        del kp, vp, x, x2
+    # ---- selective scan
+    rank = hidden // 16
+    a2, D, bias, w_dt = -f32(inner, states).abs(), f32(inner), f32(inner), rnd(inner, rank)
+    cw, cb = f32(4, inner), f32(inner)
+    for s_, l_ in ((1, 1), (batch, 1), (1, 4096), (S, Lp)):
+        n = s_ * l_
+        x, z, bc, dt = rnd(n, inner), rnd(n, inner), rnd(n, rank + 2 * states), rnd(n, inner)
+        state, cst = f32(s_, inner, states), rnd(s_, 3, inner)
+        rr = K.rows(i32([5] * n)) if l_ == 1 else K.rows(i32(list(range(l_)) * s_), q_start=i32([j * l_ for j in range(s_)]), q_len=i32([l_] * s_))
+        us = time_cold_us(lambda: K.conv_silu(x, cw, cb, cst, rr, max_q_len=l_))
+        report("conv_silu", us, bytes_=4.0 * n * inner + 12.0 * s_ * inner, seqs=s_, length=l_, channels=inner, **tag)
+        cw16, cst16 = rnd(inner, 4), rnd(s_, 3, inner)
+        us = time_cold_us(lambda: K.causal_conv1d(x, cw16, cst16, q_start=None if l_ == 1 else rr._keep[2], q_len=None if l_ == 1 else rr._keep[3], max_q_len=l_))
+        report("like: causal_conv1d", us, bytes_=4.0 * n * inner + 12.0 * s_ * inner, seqs=s_, length=l_, channels=inner, **tag)
+        if l_ == 1:
+            us = time_cold_us(lambda: K.mamba1(x, z, bc, a2, D, bias, state, rr, w_dt=w_dt))
+            report("mamba1 decode step (with step-size projection)", us, bytes_=8.0 * state.numel() + 6.0 * n * inner + 2.0 * w_dt.numel() + 4.0 * a2.numel(),
+                   rows=n, channels=inner, states=states, **tag)
+        else:
+            us = time_cold_us(lambda: K.mamba1(x, z, bc, a2, D, bias, state, rr, dt=dt))
+            report("mamba1 scan", us, bytes_=8.0 * n * inner + 2.0 * n * (rank + 2 * states), seqs=s_, length=l_, channels=inner, states=states,
+                   exponentials_per_us=round(n * inner * states / us), **tag)
+        bench_gdn(s_, l_, heads, heads, dtype=dtype, timer=time_cold_us, chunked=l_ > 1)
+        del x, z, bc, dt, state
+    # ---- routed experts
+    router, corr = rnd(experts, hidden) / hidden ** 0.5, f32(experts) * (0.1 / experts)
+    pad = (ff + 127) // 128 * 128
+    up = K.pack_weight(rnd(2 * experts * pad, hidden) / hidden ** 0.5, 2)
+    down = K.pack_weight(rnd(hidden, experts * pad) / ff ** 0.5)
+    for n in (1, 8, batch, 256, T):
+        x = rnd(n, hidden)
+        small = n <= 256
+        b = K.RoutedBatch(x, router, top, correction=corr, groups=groups, keep=keep, tile_rows=(16 if n * top <= 16 * experts else 32) if small else 128, scatter=small)
+        us = time_cold_us(b.route)
+        report("moe_router (logits, choice, plan)", us, bytes_=2.0 * (n + experts) * hidden, rows=n, experts=experts, top=top, **tag)
+        w16 = rnd((experts + 7) // 8 * 8, hidden)
+
+        def like():
+            ids, w = K.moe_select(K.gemm(x, w16)[:, :experts], top, score_fn="softmax")
+            K.moe_group(ids, w, experts)
+        report("like: gemm + moe_select + moe_group", time_cold_us(like), bytes_=2.0 * (n + experts) * hidden, rows=n, **tag)
+        b.route()
+        torch.cuda.synchronize()
+        used = int(b.ids.unique().numel())
+        e = dict(rows=n, experts=experts, used=used, ff=ff, **tag)
+        if small:
+            h = K.moe_experts(b, x, up, n=ff, k=hidden, experts=experts, expert_pad=pad, dual=True)
+            us = time_cold_us(lambda: K.moe_experts(b, x, up, n=ff, k=hidden, experts=experts, expert_pad=pad, dual=True))
+            report("experts: gate and up", us, bytes_=4.0 * used * ff * hidden + 2.0 * n * top * ff + 2.0 * n * hidden, **e)
+            us = time_cold_us(lambda: K.moe_experts(b, h, down, n=hidden, k=ff, experts=experts, expert_pad=pad, gathered=False, weighted=True))
+            report("experts: down", us, bytes_=2.0 * used * ff * hidden + 2.0 * n * top * (ff + hidden), **e)
+            # a dense GLU with as many weights as the experts that were used
+            bench_gemm(n, used * ff // 128 * 128, hidden, dual=True, packed=True, dtype=dtype)
+            bench_gemm(n, hidden, used * ff // 128 * 128, packed=True, dtype=dtype)
+        else:
+            us = time_cold_us(b.gather)
+            report("moe_gather", us, bytes_=2.0 * n * hidden * (top + 1), **e)
+            xg = b.gather()
+            tiles, pairs = b.tiles[3:], n * top
+            up_kw = dict(n=pad, k=hidden, bank_rows=experts * pad, bank_k=hidden, expert_rows=pad, dual=True, act="silu_mul", out=rnd(pairs, pad))
+            us = time_cold_us(lambda: K.moe_grouped_gemm(xg, up, tiles, **up_kw))
+            report("grouped GEMM: gate and up", us, flops=4.0 * pairs * ff * hidden, **e)
+            hg, yo = up_kw["out"], rnd(pairs, hidden)
+            us = time_cold_us(lambda: K.moe_grouped_gemm(hg, down, tiles, n=hidden, k=pad, bank_rows=hidden, bank_k=experts * pad, expert_k=pad,
+                                                         row_scale=b.slot_w[:pairs], out=yo))
+            report("grouped GEMM: down", us, flops=2.0 * pairs * ff * hidden, **e)
+            bench_gemm(pairs // 4, ff * 4, hidden, dual=True, packed=True, dtype=dtype)
+            bench_gemm(pairs // 4, hidden, ff * 4, packed=True, dtype=dtype)
+
+
+def routed() -> None:
+    bench_routed(2048, 16, 4, 4096, 16, 2, 1024, groups=4, keep=2)
+    bench_routed(4096, 32, 8, 8192, 64, 6, 1408)
+
+
 def mixed() -> None:
     bench_mixed(2048, 16)
     bench_mixed(4096, 32)
@@ -388,7 +526,7 @@ def mixed() -> None:
 
 def main() -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("what", choices=["gemm", "attn_prefill", "attn_decode", "gdn", "suite", "sweep", "heads", "mixed"])
+    ap.add_argument("what", choices=["gemm", "attn_prefill", "attn_decode", "gdn", "suite", "sweep", "heads", "mixed", "routed"])
     for name, d in (("m", 64), ("n", 4096), ("k", 4096), ("seqs", 4), ("len", 2048), ("heads", 32), ("kv-heads", 8),
                     ("hd", 128), ("hk", 16), ("hv", 32)):
         ap.add_argument(f"--{name}", type=int, default=d)
@@ -416,6 +554,8 @@ def main() -> int:
         heads()
     elif a.what == "mixed":
         mixed()
+    elif a.what == "routed":
+        routed()
     else:
         suite()
     return 0
