@@ -117,6 +117,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 
   if (warp == 0) {
     // ------------------------------------------------------------ TMA producer ----
+    // the warp reads 32 page numbers at a time, one lane issues the copies
+    constexpr int kPagesPerBlock = KVB / 16, kBlocksPerFetch = 32 / kPagesPerBlock;
     if (lane == 0) {
       mbar_arrive_expect_tx(&ctl->q_full, (uint32_t)G::kQBytes);
 #pragma unroll
@@ -124,28 +126,38 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 #pragma unroll
         for (int rg = 0; rg < kFaRows / 16; ++rg)
           tma_load_2d(qsm + c * (kFaRows * 128) + rg * kFaBox, &tmQ, &ctl->q_full, h * HD + c * 64, q_row0 + rg * 16);
-      int issued = 0;
+    }
+    {
+      int issued = 0, pages = 0;
       for (int j = 0; j < nblk; ++j) {
+        if (p.paged && j % kBlocksPerFetch == 0)
+          pages = p.page_table[(size_t)pt_row * p.pt_stride + min((kv_lo + j * KVB) / 16 + lane, p.pt_stride - 1)];
+        int block_pages[kPagesPerBlock];
+#pragma unroll
+        for (int w = 0; w < kPagesPerBlock; ++w) block_pages[w] = __shfl_sync(0xffffffffu, pages, (j % kBlocksPerFetch) * kPagesPerBlock + w);
+        int go = 1;
         const int s = j & 1;
         const uint32_t ph = (uint32_t)(j >> 1) & 1u;
-        if (!mbar_wait(&ctl->kv_empty[s], ph ^ 1u, kLocalWaitNs, 64)) {
-          report_status(p.status, kStatusTmaTimeout, kTagAttnPrefill, j);
-          ctl->abort_flag = 1;
-          break;
+        if (lane == 0) {
+          if (!mbar_wait(&ctl->kv_empty[s], ph ^ 1u, kLocalWaitNs, 64)) {
+            report_status(p.status, kStatusTmaTimeout, kTagAttnPrefill, j);
+            ctl->abort_flag = 1;
+          }
+          go = *abort_flag == 0;
         }
-        if (*abort_flag) break;
+        if (!__shfl_sync(0xffffffffu, go, 0)) break;
+        if (lane != 0) continue;
         const int t0 = kv_lo + j * KVB;
         uint8_t* ks = kvsm + (size_t)s * G::kStageBytes;
         uint8_t* vs = ks + G::kKBytes;
         mbar_arrive_expect_tx(&ctl->kv_full[s], (uint32_t)G::kStageBytes);
         // Whole blocks are always loaded: rows past the sequence end are other (finite) cache rows or the
         // zero fill beyond the tensor, and their probabilities are forced to zero.
-        for (int w = 0; w < KVB / 16; ++w) {
+#pragma unroll
+        for (int w = 0; w < kPagesPerBlock; ++w) {
           int row, col0;
           if (p.paged) {
-            const int pi = min((t0 >> 4) + w, p.pt_stride - 1);
-            const int page_id = p.page_table[(size_t)pt_row * p.pt_stride + pi];
-            row = (page_id * p.Hkv + kvh) * 16;
+            row = (block_pages[w] * p.Hkv + kvh) * 16;
             col0 = 0;
           } else {
             row = p.kv_start[seq] + t0 + w * 16;
@@ -159,7 +171,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         }
         issued = j + 1;
       }
-      if (*abort_flag) {   // let every copy that was issued land before the CTA can exit
+      if (lane == 0 && *abort_flag) {   // let every copy that was issued land before the CTA can exit
         mbar_wait(&ctl->q_full, 0, 20ull * 1000 * 1000);
         for (int j = max(0, issued - 2); j < issued; ++j)
           mbar_wait(&ctl->kv_full[j & 1], (uint32_t)(j >> 1) & 1u, 20ull * 1000 * 1000);

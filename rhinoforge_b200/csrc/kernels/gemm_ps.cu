@@ -313,16 +313,17 @@ gemm_ps_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       // 64-column round trips 30 % slower, a shared-memory transpose for full-line stores 35 % slower - long
       // instruction bursts of the epilogue warps delay the single MMA-issuing lane that shares their schedulers,
       // so the loop is kept short: scale / bias work and the activation switch are hoisted out of the element loop.
-      const bool affine = scale || bias || p.row_scale;   // per-element scale / bias work, hoisted out of the loop
+      const bool affine = scale || bias;                  // per-element scale / bias work, hoisted out of the loop
       // Output path without a residual, or with the residual already in place (out == residual, the decoder's
       // out-projection and down-projection): 64 finished columns of the warp's 32 rows are parked in a swizzled
       // staging tile and leave as ONE tiled bulk store (or bulk reduce-add, which makes the residual add an L2
       // operation) issued by lane 0 - whole 128-byte lines, asynchronous, no load or store instructions on the
       // epilogue warps (16-byte stores to 32 rows per instruction kept the store queue saturated: 537 MB on the
       // L1->L2 path for 67 MB of output).
-      const bool tma_out = p.tma_out != 0;
       uint8_t* stg = epi_stage + (size_t)(warp - 2) * kPsEpiBytes;
       const int row0 = pt.row0 + half * kPsBM + quarter * 32;
+      // grouped form: rows behind the expert's last one are another expert's, so only whole 32-row pieces leave this way
+      const bool tma_out = p.tma_out != 0 && (!p.grp || row0 + 32 <= M);
       auto chunk_begin = [&]() {                       // the previous bulk store has read the staging tile
         if (lane == 0) bulk_wait_read_all();
         __syncwarp();
@@ -343,12 +344,17 @@ gemm_ps_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
           g[j] = __uint_as_float(g16[j]);
           u[j] = DUAL ? __uint_as_float(u16[j]) : 0.f;
         }
+        if (p.row_scale) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j) {
+            g[j] *= rs;
+            if (DUAL) u[j] *= rs;
+          }
+        }
         if (affine) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const int n = n0 + j;
-            g[j] *= rs;
-            if (DUAL) u[j] *= rs;
             if (n < N) {
               if (scale) {
                 g[j] *= Num<T>::to_f(scale[n]);
@@ -518,9 +524,16 @@ template <typename T, bool DUAL>
 static int launch_ps_grouped(const RfMoeGroupedGemm* a, cudaStream_t stream) {
   auto kfn = gemm_ps_kernel<T, DUAL, 1>;
   RF_ALLOW_SMEM_PER_DEVICE(kfn, 227 * 1024);
-  CUtensorMap tmA;
+  CUtensorMap tmA, tmO;
   int rc = make_tmap_2d(&tmA, a->x, a->dtype, 2, a->K, a->max_rows, a->ldx, kPsBK, kPsBM, true);
   if (rc) return rc;
+  const bool tma_out = (a->ldo & 7) == 0 && (reinterpret_cast<uintptr_t>(a->out) & 15) == 0;
+  if (tma_out) {
+    rc = make_tmap_2d(&tmO, a->out, a->dtype, 2, a->N, a->max_rows, a->ldo, 64, 32, true);
+    if (rc) return rc;
+  } else {
+    tmO = tmA;
+  }
   const int bn = (!DUAL && a->N % 256 == 0) ? 256 : 128;
   GemmPsParams p = {};
   p.out = a->out; p.ldo = a->ldo;
@@ -531,13 +544,14 @@ static int launch_ps_grouped(const RfMoeGroupedGemm* a, cudaStream_t stream) {
   p.act = a->act; p.dual_offset = DUAL ? a->N : 0; p.dual_tiles = a->bank_section_row_tiles;
   p.tiles_m = 0; p.tiles_n = ceil_div(a->N, bn);
   p.band = 1;
+  p.tma_out = tma_out ? 1 : 0;
   p.grp = a->tiles; p.grp_rt_per_expert = a->rt_per_expert; p.grp_kb_per_expert = a->kb_per_expert;
   p.kb_total = a->bank_kb_total;
   const int stage_bytes = kPsATile + (DUAL ? 2 : 1) * bn * kPsBK * 2;
   const int ctl_bytes = (int)sizeof(GemmPsCtl) + 1024 + 4 * kPsEpiBytes;
   p.stages = std::min(kPsMaxStages, (227 * 1024 - ctl_bytes) / stage_bytes);
   const size_t smem = (size_t)p.stages * stage_bytes + ctl_bytes;
-  RF_CUDA_CHECK(::rf::launch_k(kfn, dim3(sm_count()), dim3(64 + 128), smem, stream, 1, tmA, tmA, p));
+  RF_CUDA_CHECK(::rf::launch_k(kfn, dim3(sm_count()), dim3(64 + 128), smem, stream, 1, tmA, tmO, p));
   ::rf::count_launch();
   return RF_OK;
 }

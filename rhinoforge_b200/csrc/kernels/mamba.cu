@@ -5,6 +5,7 @@
 // states, so that a warp reads and writes the states of eight channels as whole lines.
 #include "../common/dtype.cuh"
 #include "../common/host_util.h"
+#include "../common/mma.cuh"
 #include "../common/ptx.cuh"
 #include "../rf_api.h"
 
@@ -109,16 +110,22 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const RfConvSilu p, int 
 constexpr int kMbChannels = 64;       // channels per CTA (256 threads)
 constexpr int kMbRows = 8;            // rows staged in shared memory at a time
 
-// A CTA owns 64 channels of `seqs_per_cta` neighbouring sequences, whose rows are contiguous.  The step size of a row comes
-// from the step-size weights of these channels, kept in shared memory.
+// A CTA owns 64 channels of `seqs_per_cta` neighbouring sequences, whose rows are contiguous.  The step sizes of eight rows at a
+// time come from one small matrix product: 16-bit models run it on mma.sync (channels on the M axis, the rows on the N axis, eight
+// warps as four channel tiles times two halves of the rank, weights straight from L2 into the fragments), 32-bit ones keep the
+// weights of the channels in shared memory.
 template <typename T, int QPL>
 __global__ void __launch_bounds__(256) mamba_recurrent_kernel(const RfMamba1 p, int seqs_per_cta) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) uint8_t mb_raw[];
   constexpr int CH = kMbChannels, SP = 16 * QPL;                    // SP: states per channel in shared memory, zero padded
+  constexpr bool kMma = sizeof(T) == 2;
   const int rank_p = (p.rank + 31) & ~31, wp = rank_p + 8;
-  float* s_dt = reinterpret_cast<float*>(mb_raw);                   // [rows][rank_p]
-  float* s_b = s_dt + kMbRows * rank_p;                             // [rows][SP]
+  float* s_dt = reinterpret_cast<float*>(mb_raw);                   // 32 bits: [rows][rank_p] step-size inputs
+  T* s_di = reinterpret_cast<T*>(mb_raw);                           // 16 bits: [rows][wp], and behind them
+  float* s_pre = reinterpret_cast<float*>(s_di + kMbRows * wp);     // [2][rows][CH] halves of the products
+  const int head_floats = kMma ? kMbRows * wp / 2 + 2 * kMbRows * CH : kMbRows * rank_p;
+  float* s_b = s_dt + head_floats;                                  // [rows][SP]
   float* s_c = s_b + kMbRows * SP;
   float* s_x = s_c + kMbRows * SP;                                  // [rows][CH]
   float* s_z = s_x + kMbRows * CH;
@@ -126,14 +133,16 @@ __global__ void __launch_bounds__(256) mamba_recurrent_kernel(const RfMamba1 p, 
   const int tid = threadIdx.x, l = tid & 3, ci = tid >> 2, c0 = blockIdx.x * CH, c = c0 + ci;
   const bool live = c < p.inner;
   // the weights do not depend on the previous kernel
-  for (int i = tid; i < CH * (wp / 8); i += 256) {
-    const int r = i / (wp / 8), k = (i % (wp / 8)) * 8;
-    float f[8];
-    zero8(f);
-    if (c0 + r < p.inner && k < p.rank) load8(reinterpret_cast<const T*>(p.w_dt) + (size_t)(c0 + r) * p.rank + k, f);
-    store8(s_w + (size_t)r * wp + k, f);
+  if constexpr (!kMma) {
+    for (int i = tid; i < CH * (wp / 8); i += 256) {
+      const int r = i / (wp / 8), k = (i % (wp / 8)) * 8;
+      float f[8];
+      zero8(f);
+      if (c0 + r < p.inner && k < p.rank) load8(reinterpret_cast<const T*>(p.w_dt) + (size_t)(c0 + r) * p.rank + k, f);
+      store8(s_w + (size_t)r * wp + k, f);
+    }
   }
-  for (int i = tid; i < kMbRows * (rank_p + 2 * SP); i += 256) s_dt[i] = 0.f;
+  for (int i = tid; i < head_floats + kMbRows * 2 * SP; i += 256) s_dt[i] = 0.f;
   const int nq = p.states / 4;
   float4 A[QPL];
 #pragma unroll
@@ -162,7 +171,8 @@ __global__ void __launch_bounds__(256) mamba_recurrent_kernel(const RfMamba1 p, 
       const int r = i / (p.rank / 8), k = (i % (p.rank / 8)) * 8;
       float f[8];
       load8(reinterpret_cast<const T*>(p.bc) + (size_t)(r0 + r) * p.ld_bc + k, f);
-      store8(s_dt + r * rank_p + k, f);
+      if (kMma) store8(s_di + r * wp + k, f);
+      else store8(s_dt + r * rank_p + k, f);
     }
     for (int i = tid; i < nr * (p.states / 4); i += 256) {          // B and C: states / 8 pieces each
       const int r = i / (p.states / 4), k = (i % (p.states / 4)) * 8;
@@ -179,6 +189,27 @@ __global__ void __launch_bounds__(256) mamba_recurrent_kernel(const RfMamba1 p, 
       store8((zi ? s_z : s_x) + r * CH + k, f);
     }
     __syncthreads();
+    if constexpr (kMma) {
+      const int warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3, mt = warp & 3, half = warp >> 2;
+      float acc[4] = {0.f, 0.f, 0.f, 0.f};
+      const T* w0 = reinterpret_cast<const T*>(p.w_dt) + (size_t)(c0 + mt * 16 + g) * p.rank;
+      const bool in0 = c0 + mt * 16 + g < p.inner, in1 = c0 + mt * 16 + g + 8 < p.inner;
+      const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll 4
+      for (int kb = half; kb < rank_p / 32; kb += 2) {              // a lane's fragment: eight consecutive columns of both operands
+        const int k = kb * 32 + q * 8;
+        const uint4 a0 = in0 && k < p.rank ? *reinterpret_cast<const uint4*>(w0 + k) : zero;
+        const uint4 a1 = in1 && k < p.rank ? *reinterpret_cast<const uint4*>(w0 + (size_t)8 * p.rank + k) : zero;
+        const uint4 b = *reinterpret_cast<const uint4*>(s_di + g * wp + k);
+        const uint32_t lo[4] = {a0.x, a1.x, a0.y, a1.y}, hi[4] = {a0.z, a1.z, a0.w, a1.w};
+        MmaOp<T>::mma(acc, lo, b.x, b.y);
+        MmaOp<T>::mma(acc, hi, b.z, b.w);
+      }
+      float* o = s_pre + half * kMbRows * CH + mt * 16 + g;
+      o[(q * 2) * CH] = acc[0]; o[(q * 2 + 1) * CH] = acc[1];
+      o[(q * 2) * CH + 8] = acc[2]; o[(q * 2 + 1) * CH + 8] = acc[3];
+      __syncthreads();
+    }
     for (int r = 0; r < nr; ++r) {
       if (start) {
 #pragma unroll
@@ -187,17 +218,21 @@ __global__ void __launch_bounds__(256) mamba_recurrent_kernel(const RfMamba1 p, 
         start = false;
       }
       float dot = 0.f;
-      const T* wr = s_w + (size_t)ci * wp + l * 8;
-      const float* dr = s_dt + r * rank_p + l * 8;
-      for (int k = 0; k < rank_p; k += 32) {
-        float w8[8], d8[8];
-        load8(wr + k, w8);
-        load8(dr + k, d8);
+      if constexpr (kMma) {
+        dot = s_pre[r * CH + ci] + s_pre[(kMbRows + r) * CH + ci];
+      } else {
+        const T* wr = s_w + (size_t)ci * wp + l * 8;
+        const float* dr = s_dt + r * rank_p + l * 8;
+        for (int k = 0; k < rank_p; k += 32) {
+          float w8[8], d8[8];
+          load8(wr + k, w8);
+          load8(dr + k, d8);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) dot += w8[j] * d8[j];
+          for (int j = 0; j < 8; ++j) dot += w8[j] * d8[j];
+        }
+        dot += __shfl_xor_sync(0xffffffffu, dot, 1);
+        dot += __shfl_xor_sync(0xffffffffu, dot, 2);
       }
-      dot += __shfl_xor_sync(0xffffffffu, dot, 1);
-      dot += __shfl_xor_sync(0xffffffffu, dot, 2);
       const float dt = softplus_t<T>(dot + bias), x = s_x[r * CH + ci], dx = dt * x;
       float y = 0.f;
 #pragma unroll
@@ -366,7 +401,10 @@ static int launch_recurrent(const RfMamba1* a, cudaStream_t s) {
   // share the step-size weights of a channel tile between sequences once there are enough CTAs without it
   const int spc = std::max(1, std::min(8, seqs * tiles / (6 * sm_count())));
   const int rank_p = (a->rank + 31) & ~31;
-  const size_t smem = (size_t)kMbRows * (rank_p + 32 * QPL + 2 * kMbChannels) * sizeof(float) + (size_t)kMbChannels * (rank_p + 8) * sizeof(T);
+  const size_t head = sizeof(T) == 2 ? (size_t)kMbRows * ((rank_p + 8) * sizeof(T) + 2 * kMbChannels * sizeof(float))
+                                     : (size_t)kMbRows * rank_p * sizeof(float);
+  const size_t smem = head + (size_t)kMbRows * (32 * QPL + 2 * kMbChannels) * sizeof(float) +
+                      (sizeof(T) == 2 ? 0 : (size_t)kMbChannels * (rank_p + 8) * sizeof(T));
   RF_REQUIRE(smem <= 200 * 1024, "mamba: a step rank of %d does not fit in shared memory", a->rank);
   RF_ALLOW_SMEM_PER_DEVICE((mamba_recurrent_kernel<T, QPL>), 200 * 1024);
   RF_CUDA_CHECK(::rf::launch_k(mamba_recurrent_kernel<T, QPL>, dim3(tiles, ceil_div(seqs, spc)), dim3(256), smem, s, 1, *a, spc));

@@ -255,6 +255,99 @@ __global__ void __launch_bounds__(VPT == 4 ? 512 : 1024) stream_norm_reg_kernel(
   }
 }
 
+// The stream step behind a sublayer whose output is normalised (16-bit activations, no token shift): one CTA per row, a thread
+// holds NC groups of eight columns, so that every operand moves in 16-byte pieces; of several picked rows four are in flight at
+// a time.
+template <typename T, int NC>
+__global__ void __launch_bounds__(512) stream_out_kernel(const RfStreamNorm p) {
+  pdl_launch_dependents();
+  __shared__ float red[2][16];
+  const int H = p.H, nthr = blockDim.x, nw = nthr >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float inv_dim = 1.f / (float)p.dim;
+  auto col = [&](int k) { return (threadIdx.x + k * nthr) * 8; };
+  float w[NC][8];
+#pragma unroll
+  for (int k = 0; k < NC; ++k)
+    if (col(k) < H) load8(p.y_norm_w + col(k), w[k]);          // does not depend on the previous kernel
+  pdl_wait();
+  const int r = blockIdx.x, src = p.row_idx ? p.row_idx[r] : r;
+  const T* y = reinterpret_cast<const T*>(p.y);
+  float v[NC][8], a[NC][8];
+#pragma unroll
+  for (int k = 0; k < NC; ++k) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[k][j] = a[k][j] = 0.f;
+    if (col(k) >= H) continue;
+    if (p.x) load8(p.x + (size_t)src * H + col(k), v[k]);
+    else {
+      load8(reinterpret_cast<const T*>(p.table) + (size_t)p.ids[src] * H + col(k), v[k]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[k][j] *= p.embed_scale;
+    }
+  }
+  const int picks = p.y_picks > 0 ? p.y_picks : 1;
+  for (int j0 = 0; j0 < picks; j0 += 4) {
+    int row[4];
+    uint4 raw[4][NC];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) row[i] = j0 + i >= picks ? -1 : (p.y_picks > 0 ? p.y_slots[(size_t)src * picks + j0 + i] : src);
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int k = 0; k < NC; ++k) {
+        raw[i][k] = make_uint4(0u, 0u, 0u, 0u);                // zero bits are zero in both formats
+        if (row[i] >= 0 && col(k) < H) raw[i][k] = *reinterpret_cast<const uint4*>(y + (size_t)row[i] * H + col(k));
+      }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int k = 0; k < NC; ++k) {
+        const typename Num<T>::T2* t = reinterpret_cast<const typename Num<T>::T2*>(&raw[i][k]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float2 f = Num<T>::to_f2(t[j]);
+          a[k][2 * j] += f.x;
+          a[k][2 * j + 1] += f.y;
+        }
+      }
+  }
+  auto block_sum = [&](float s, int flip) -> float {
+    s = warp_sum(s);
+    if (lane == 0) red[flip][warp] = s;
+    __syncthreads();
+    return warp_sum(lane < nw ? red[flip][lane] : 0.f);
+  };
+  float s = 0.f;
+#pragma unroll
+  for (int k = 0; k < NC; ++k)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s += a[k][j] * a[k][j];
+  const float yr = rsqrtf(block_sum(s, 0) * inv_dim + p.eps);
+  s = 0.f;
+#pragma unroll
+  for (int k = 0; k < NC; ++k) {
+    if (col(k) >= H) continue;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      v[k][j] += a[k][j] * yr * w[k][j];
+      s += v[k][j] * v[k][j];
+    }
+    if (p.x_out) store8(p.x_out + (size_t)r * H + col(k), v[k]);
+    if (p.x_cast) store8(reinterpret_cast<T*>(p.x_cast) + (size_t)r * H + col(k), v[k]);
+  }
+  if (!p.norm_w) return;
+  const float xr = rsqrtf(block_sum(s, 1) * inv_dim + p.eps);
+#pragma unroll
+  for (int k = 0; k < NC; ++k) {
+    if (col(k) >= H) continue;
+    float n8[8];
+    load8(p.norm_w + col(k), n8);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) n8[j] *= v[k][j] * xr;
+    store8(reinterpret_cast<T*>(p.out) + (size_t)r * H + col(k), n8);
+  }
+}
+
 template <typename T>
 __global__ void token_gate_kernel(T* __restrict__ g, int64_t ldg, const T* __restrict__ table, int64_t ldt,
                                   const int32_t* __restrict__ ids, int col0, int rows, int cols) {
@@ -346,6 +439,19 @@ extern "C" int rf_stream_norm(const RfStreamNorm* args, rf_stream_t stream) {
   // halo of one row per CTA with the shift: walk several rows per CTA once that still fills the GPU
   const int rpc = (a->shift && a->rows.q_start) ? std::max(1, std::min(8, a->n_rows / (2 * sm_count()))) : 1;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const int groups = a->H / 8;
+  if (a->y && a->y_norm_w && !a->shift && a->dtype != kF32 && groups <= 1024) {
+    // decode rows: one group of columns per thread; many rows: two, so that several rows share an SM
+    const int nc = groups > 512 || (groups > 256 && a->n_rows > 4 * sm_count()) ? 2 : 1;
+    const dim3 block(std::max(32, round_up(ceil_div(groups, nc), 32)));
+#define RF_SO(T, NC) RF_CUDA_CHECK(::rf::launch_k(stream_out_kernel<T, NC>, dim3(a->n_rows), block, 0, s, 1, *a))
+#define RF_SO_T(T) if (nc == 1) { RF_SO(T, 1); } else { RF_SO(T, 2); }
+    if (a->dtype == kF16) { RF_SO_T(__half) } else { RF_SO_T(__nv_bfloat16) }
+#undef RF_SO_T
+#undef RF_SO
+    ::rf::count_launch();
+    return RF_OK;
+  }
   const int quads = a->H / 4;
   if (quads <= 2048) {
     // decode rows: as many threads as there are quads (one round trip); many rows: smaller CTAs, several per SM
