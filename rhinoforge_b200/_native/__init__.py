@@ -269,7 +269,8 @@ class RfMoeRouter(C.Structure):
                [(n, C.c_void_p) for n in ("w", "correction", "ids", "weights", "rank", "counters", "start", "tiles", "slot_of",
                                           "token_of_slot", "slot_w")] + \
                [(n, C.c_int32) for n in ("rows", "experts", "width", "k", "groups", "keep", "score_fn", "norm_topk")] + \
-               [("scale", C.c_float)] + [(n, C.c_int32) for n in ("tile_rows", "slot_ld", "has_shared", "shared_tiles", "scatter", "dtype")]
+               [("scale", C.c_float)] + [(n, C.c_int32) for n in ("tile_rows", "slot_ld", "has_shared", "shared_tiles", "scatter", "dtype")] + \
+               [("logits", C.c_void_p)]
 
 
 class RfMoeExperts(C.Structure):
@@ -319,6 +320,7 @@ def lib() -> C.CDLL:
         l.rf_mixed_status_ptr.restype = C.c_void_p
         l.rf_latent_attn_scratch_bytes.restype = C.c_uint64
         l.rf_attn_decode_scratch_bound.restype = C.c_uint64
+        l.rf_moe_router_scratch_bytes.restype = C.c_uint64
         l.rf_pack_weight_bytes.restype = C.c_uint64
         l.rf_pack_w4_bytes.restype = C.c_uint64
         l.rf_pack_w4_bytes.argtypes = [C.c_int64, C.c_int64, C.c_int32, C.c_int32]

@@ -1,5 +1,5 @@
-// Mixture of experts of the mixed-layer decoders: the router as one launch (logits in fp32, group-limited choice, weights, and
-// the plan of which expert gets which rows), the row gather of prefill-sized batches, and the expert GEMMs of small batches,
+// Mixture of experts of the mixed-layer decoders: the router (logits in fp32; group-limited choice, weights, and the plan of
+// which expert gets which rows), the row gather of prefill-sized batches, and the expert GEMMs of small batches,
 // whose work is reading the chosen experts' weights once.
 //
 // Sorted rows: the picks of an expert are neighbours; row k * T + t behind them belongs to the shared expert's token t.  A tile
@@ -15,41 +15,54 @@ namespace rf {
 
 constexpr int kRtLane = 8;            // experts per lane: up to 256
 
-struct BestPick { float v; int i; };
-__device__ __forceinline__ BestPick warp_argmax(BestPick b) {       // ties go to the lower index
+constexpr int kRtTokens = 32;         // tokens (warps) per CTA of the choice
+constexpr int kRtOneCta = 64;         // up to this many tokens one CTA chooses for all of them and plans in shared memory
+
+struct BestPick { uint32_t v; int i; };
+// floats in an order that unsigned comparison keeps
+__device__ __forceinline__ uint32_t ordered(float f) {
+  const uint32_t u = __float_as_uint(f);
+  return u ^ ((u >> 31) ? 0xffffffffu : 0x80000000u);
+}
+// largest of the lanes' values x[s] (index s * 32 + lane), ties to the lower index
+template <int S>
+__device__ __forceinline__ BestPick warp_argmax(const float (&x)[S], int lane) {
+  BestPick b = {0u, 0x7fffffff};
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const float ov = __shfl_xor_sync(0xffffffffu, b.v, o);
-    const int oi = __shfl_xor_sync(0xffffffffu, b.i, o);
-    if (ov > b.v || (ov == b.v && oi < b.i)) { b.v = ov; b.i = oi; }
+  for (int s = 0; s < S; ++s) {
+    const uint32_t v = ordered(x[s]);
+    if (v > b.v) { b.v = v; b.i = s * 32 + lane; }
   }
-  return b;
+  const uint32_t top = __reduce_max_sync(0xffffffffu, b.v);
+  return BestPick{top, (int)__reduce_min_sync(0xffffffffu, b.v == top ? (unsigned)b.i : 0x7fffffffu)};
 }
 
-// One warp routes one token.  sc[s]: this lane's logits (expert s * 32 + lane); keys: shared scratch of E floats.
-__device__ __forceinline__ void route_token(const RfMoeRouter& p, int t, int lane, float (&sc)[kRtLane], float* keys) {
+// One warp routes one token.  sc[s]: this lane's logits (expert s * 32 + lane); keys: shared scratch of E floats.  Lane j < k
+// leaves with the j-th expert and its weight.
+template <int S>
+__device__ __forceinline__ void route_token(const RfMoeRouter& p, int lane, float (&sc)[S], float* keys, int* my_id, float* my_w) {
   const int E = p.experts;
   float mx = -INFINITY;
 #pragma unroll
-  for (int s = 0; s < kRtLane; ++s) mx = fmaxf(mx, s * 32 + lane < E ? sc[s] : -INFINITY);
+  for (int s = 0; s < S; ++s) mx = fmaxf(mx, s * 32 + lane < E ? sc[s] : -INFINITY);
   if (p.score_fn == RF_MOE_SOFTMAX) {
     mx = warp_max(mx);
     float sum = 0.f;
 #pragma unroll
-    for (int s = 0; s < kRtLane; ++s) {
+    for (int s = 0; s < S; ++s) {
       sc[s] = s * 32 + lane < E ? expf(sc[s] - mx) : 0.f;
       sum += sc[s];
     }
     sum = warp_sum(sum);
 #pragma unroll
-    for (int s = 0; s < kRtLane; ++s) sc[s] /= sum;
+    for (int s = 0; s < S; ++s) sc[s] /= sum;
   } else {
 #pragma unroll
-    for (int s = 0; s < kRtLane; ++s) sc[s] = s * 32 + lane < E ? 1.f / (1.f + expf(-sc[s])) : 0.f;
+    for (int s = 0; s < S; ++s) sc[s] = s * 32 + lane < E ? 1.f / (1.f + expf(-sc[s])) : 0.f;
   }
-  float key[kRtLane];
+  float key[S];
 #pragma unroll
-  for (int s = 0; s < kRtLane; ++s) {
+  for (int s = 0; s < S; ++s) {
     const int e = s * 32 + lane;
     key[s] = e < E ? sc[s] + (p.correction ? p.correction[e] : 0.f) : -INFINITY;
   }
@@ -58,12 +71,12 @@ __device__ __forceinline__ void route_token(const RfMoeRouter& p, int t, int lan
     const int size = E / p.groups;
     __syncwarp();
 #pragma unroll
-    for (int s = 0; s < kRtLane; ++s)
+    for (int s = 0; s < S; ++s)
       if (s * 32 + lane < E) keys[s * 32 + lane] = key[s];
     __syncwarp();
-    float gs[kRtLane];
+    float gs[S];
 #pragma unroll
-    for (int s = 0; s < kRtLane; ++s) {
+    for (int s = 0; s < S; ++s) {
       const int g = s * 32 + lane;
       gs[s] = -INFINITY;
       if (g < p.groups)
@@ -71,233 +84,243 @@ __device__ __forceinline__ void route_token(const RfMoeRouter& p, int t, int lan
     }
     __syncwarp();
 #pragma unroll
-    for (int s = 0; s < kRtLane; ++s)
+    for (int s = 0; s < S; ++s)
       if (s * 32 + lane < p.groups) keys[s * 32 + lane] = 0.f;      // now: is this group kept?
     __syncwarp();
     for (int j = 0; j < p.keep; ++j) {
-      BestPick b = {-INFINITY, 0x7fffffff};
-#pragma unroll
-      for (int s = 0; s < kRtLane; ++s)
-        if (gs[s] > b.v) b = {gs[s], s * 32 + lane};
-      b = warp_argmax(b);
+      const BestPick b = warp_argmax<S>(gs, lane);
       if (b.i < p.groups && (b.i & 31) == lane) {
 #pragma unroll
-        for (int s = 0; s < kRtLane; ++s)
+        for (int s = 0; s < S; ++s)
           if (s == (b.i >> 5)) gs[s] = -INFINITY;
         keys[b.i] = 1.f;
       }
     }
     __syncwarp();
 #pragma unroll
-    for (int s = 0; s < kRtLane; ++s) {
+    for (int s = 0; s < S; ++s) {
       const int e = s * 32 + lane;
       if (e < E && keys[e / size] == 0.f) key[s] = -INFINITY;
     }
   }
-  float sum = 0.f, my_w = 0.f;
-  int my_id = -1;
+  float sum = 0.f;
+  *my_w = 0.f;
+  *my_id = -1;
   for (int j = 0; j < p.k; ++j) {
-    BestPick b = {-INFINITY, 0x7fffffff};
-#pragma unroll
-    for (int s = 0; s < kRtLane; ++s)
-      if (key[s] > b.v) b = {key[s], s * 32 + lane};
-    b = warp_argmax(b);
+    const BestPick b = warp_argmax<S>(key, lane);
     float w = 0.f;
     if (b.i < E && (b.i & 31) == lane) {
 #pragma unroll
-      for (int s = 0; s < kRtLane; ++s)
+      for (int s = 0; s < S; ++s)
         if (s == (b.i >> 5)) { w = sc[s]; key[s] = -INFINITY; }
     }
     w = __shfl_sync(0xffffffffu, w, b.i & 31);
     sum += w;
-    if (lane == j) { my_id = b.i < E ? b.i : -1; my_w = w; }
+    if (lane == j) { *my_id = b.i < E ? b.i : -1; *my_w = w; }
   }
-  const float mul = (p.norm_topk ? 1.f / (sum + 1e-20f) : 1.f) * p.scale;
-  if (lane < p.k) {
-    const size_t at = (size_t)t * p.k + lane;
-    p.ids[at] = my_id;
-    p.weights[at] = my_w * mul;
-    p.rank[at] = my_id >= 0 ? atomicAdd(&p.counters[my_id], 1) : -1;
-  }
+  *my_w *= (p.norm_topk ? 1.f / (sum + 1e-20f) : 1.f) * p.scale;
 }
 
-// Exclusive sums over the experts and the tile list; by the CTA whose ticket is the last (all of the router's results are
-// visible to it then).  Leaves the counters at zero for the next launch.
-__device__ __forceinline__ void router_plan(const RfMoeRouter& p) {
-  __shared__ int32_t rows_at[257], tiles_at[257], cnt[256];
+struct PlanSmem { int32_t cnt[256], rows_at[257], tiles_at[257]; };
+
+// Exclusive sums of the experts' counts (sm.cnt) and the tile list; all threads of the CTA.
+__device__ __forceinline__ void plan_tiles(const RfMoeRouter& p, PlanSmem& sm) {
   const int tid = threadIdx.x, E = p.experts, R = p.tile_rows;
-  for (int e = tid; e < E; e += blockDim.x) {
-    cnt[e] = __ldcg(p.counters + e);
-    p.counters[e] = 0;
-  }
-  __syncthreads();
   if (tid < 32) {
     int rows = 0, tiles = 0;
     for (int e0 = 0; e0 < E; e0 += 32) {
-      const int n = e0 + tid < E ? cnt[e0 + tid] : 0, nt = (n + R - 1) / R;
+      const int n = e0 + tid < E ? sm.cnt[e0 + tid] : 0, nt = (n + R - 1) / R;
       int ri = n, ti = nt;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
         const int ro = __shfl_up_sync(0xffffffffu, ri, o), to = __shfl_up_sync(0xffffffffu, ti, o);
         if (tid >= o) { ri += ro; ti += to; }
       }
-      if (e0 + tid < E) { rows_at[e0 + tid] = rows + ri - n; tiles_at[e0 + tid] = tiles + ti - nt; }
+      if (e0 + tid < E) { sm.rows_at[e0 + tid] = rows + ri - n; sm.tiles_at[e0 + tid] = tiles + ti - nt; }
       rows += __shfl_sync(0xffffffffu, ri, 31);
       tiles += __shfl_sync(0xffffffffu, ti, 31);
     }
-    if (tid == 0) { rows_at[E] = rows; tiles_at[E] = tiles; }
+    if (tid == 0) { sm.rows_at[E] = rows; sm.tiles_at[E] = tiles; }
   }
   __syncthreads();
   for (int e = tid; e < E; e += blockDim.x) {
-    const int r0 = rows_at[e], n = cnt[e];
+    const int r0 = sm.rows_at[e], n = sm.cnt[e];
     p.start[e] = r0;
     for (int i = 0; i * R < n; ++i)
-      reinterpret_cast<int4*>(p.tiles)[1 + tiles_at[e] + i] = make_int4(e, r0 + i * R, r0 + n, 0);
+      reinterpret_cast<int4*>(p.tiles)[1 + sm.tiles_at[e] + i] = make_int4(e, r0 + i * R, r0 + n, 0);
   }
   const int pairs = p.rows * p.k, shared = p.shared_tiles ? (p.rows + R - 1) / R : 0;
   for (int i = tid; i < shared; i += blockDim.x)
-    reinterpret_cast<int4*>(p.tiles)[1 + tiles_at[E] + i] = make_int4(E, pairs + i * R, pairs + p.rows, 0);
-  if (tid == 0) p.tiles[0] = p.tiles[3] = tiles_at[E] + shared;    // words 3.. are the list as rf_moe_grouped_gemm takes it
-  if (p.scatter) {
-    for (int i = tid; i < pairs; i += blockDim.x) {
-      const int e = __ldcg(p.ids + i), t = i / p.k;
-      const int slot = e >= 0 ? rows_at[e] + __ldcg(p.rank + i) : -1;
-      p.slot_of[(size_t)t * p.slot_ld + i % p.k] = slot;
-      if (slot >= 0) {
-        p.token_of_slot[slot] = t;
-        p.slot_w[slot] = __ldcg(p.weights + i);
-      }
+    reinterpret_cast<int4*>(p.tiles)[1 + sm.tiles_at[E] + i] = make_int4(E, pairs + i * R, pairs + p.rows, 0);
+  if (tid == 0) p.tiles[0] = p.tiles[3] = sm.tiles_at[E] + shared;   // words 3.. are the list as rf_moe_grouped_gemm takes it
+  if (p.scatter && p.has_shared)
+    for (int t = tid; t < p.rows; t += blockDim.x) {
+      p.slot_of[(size_t)t * p.slot_ld + p.k] = pairs + t;
+      p.token_of_slot[pairs + t] = t;
+      p.slot_w[pairs + t] = 1.f;
     }
-    if (p.has_shared)
-      for (int t = tid; t < p.rows; t += blockDim.x) {
-        p.slot_of[(size_t)t * p.slot_ld + p.k] = pairs + t;
-        p.token_of_slot[pairs + t] = t;
-        p.slot_w[pairs + t] = 1.f;
-      }
+}
+
+__device__ __forceinline__ void place_pick(const RfMoeRouter& p, const PlanSmem& sm, int i, int e, int rank, float w) {
+  const int t = i / p.k, slot = e >= 0 ? sm.rows_at[e] + rank : -1;
+  p.slot_of[(size_t)t * p.slot_ld + i % p.k] = slot;
+  if (slot >= 0) {
+    p.token_of_slot[slot] = t;
+    p.slot_w[slot] = w;
   }
 }
 
-__device__ __forceinline__ void router_ticket(const RfMoeRouter& p) {
+// Scores, choice and plan over the logits [splits][rows][experts] (partial sums, added in order).  One CTA: everything stays in
+// shared memory.  Several: a CTA counts its own picks, takes its places among the experts' rows with one atomic per expert, and
+// the last one to finish plans.
+template <int S>
+__global__ void __launch_bounds__(kRtTokens * 32) moe_choose_kernel(const RfMoeRouter p, int splits) {
+  pdl_prologue();
+  extern __shared__ __align__(16) float ch_sm[];          // [warps][E] keys, then the picks of one CTA's tokens
+  __shared__ PlanSmem sm;
+  __shared__ int32_t base[256];
   __shared__ int last;
+  const int E = p.experts, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const bool alone = gridDim.x == 1;
+  const int per_cta = alone ? kRtOneCta : kRtTokens, first = blockIdx.x * per_cta;
+  const int here = min(per_cta, p.rows - first);
+  float* keys = ch_sm + warp * E;
+  int32_t* s_id = reinterpret_cast<int32_t*>(ch_sm + kRtTokens * E);
+  int32_t* s_rank = s_id + per_cta * p.k;
+  float* s_w = reinterpret_cast<float*>(s_rank + per_cta * p.k);
+  for (int e = tid; e < E; e += blockDim.x) sm.cnt[e] = 0;
+  __syncthreads();
+  for (int t = warp; t < here; t += kRtTokens) {
+    float sc[S];
+#pragma unroll
+    for (int s = 0; s < S; ++s) {
+      const int e = s * 32 + lane;
+      sc[s] = 0.f;
+      if (e < E)
+        for (int z = 0; z < splits; ++z) sc[s] += p.logits[((size_t)z * p.rows + first + t) * E + e];
+    }
+    int id;
+    float w;
+    route_token<S>(p, lane, sc, keys, &id, &w);
+    if (lane < p.k) {
+      const int i = t * p.k + lane;
+      s_id[i] = id;
+      s_w[i] = w;
+      s_rank[i] = id >= 0 ? atomicAdd(&sm.cnt[id], 1) : -1;
+    }
+  }
+  __syncthreads();
+  if (!alone) {
+    for (int e = tid; e < E; e += blockDim.x) base[e] = sm.cnt[e] ? atomicAdd(p.counters + e, sm.cnt[e]) : 0;
+    __syncthreads();
+  }
+  for (int i = tid; i < here * p.k; i += blockDim.x) {
+    const size_t at = (size_t)first * p.k + i;
+    const int id = s_id[i];
+    p.ids[at] = id;
+    p.weights[at] = s_w[i];
+    p.rank[at] = alone || id < 0 ? s_rank[i] : base[id] + s_rank[i];
+  }
+  if (alone) {
+    plan_tiles(p, sm);
+    if (p.scatter)
+      for (int i = tid; i < here * p.k; i += blockDim.x) place_pick(p, sm, i, s_id[i], s_rank[i], s_w[i]);
+    return;
+  }
   __threadfence();
   __syncthreads();
-  if (threadIdx.x == 0) {
-    const int n = (int)(gridDim.x * gridDim.y * gridDim.z);
-    last = atomicAdd(p.counters + p.experts, 1) == n - 1;
-    if (last) p.counters[p.experts] = 0;
+  if (tid == 0) {
+    last = atomicAdd(p.counters + E, 1) == (int)gridDim.x - 1;
+    if (last) p.counters[E] = 0;
   }
   __syncthreads();
   if (!last) return;
   __threadfence();
-  router_plan(p);
+  for (int e = tid; e < E; e += blockDim.x) {             // the counters are left at zero for the next launch
+    sm.cnt[e] = __ldcg(p.counters + e);
+    p.counters[e] = 0;
+  }
+  __syncthreads();
+  plan_tiles(p, sm);
+  if (p.scatter)
+    for (int i = tid; i < p.rows * p.k; i += blockDim.x) place_pick(p, sm, i, __ldcg(p.ids + i), __ldcg(p.rank + i), __ldcg(p.weights + i));
 }
 
-// MT * 16 tokens per cluster.  Warps and cluster CTAs split the width; a lane's operand fragment is eight consecutive columns
-// (the order of the columns inside a product does not matter as long as both operands agree), so fragments come straight from
-// global memory as 16-byte loads.
-template <typename T, int MT>
-__global__ void __launch_bounds__(256) moe_router_kernel(const RfMoeRouter p) {
-  pdl_launch_dependents();
-  extern __shared__ __align__(16) float lg[];             // [16 * MT][E] logits, then one row of keys per warp
+// Logits in fp32: 16 * MT * TW tokens times 64 experts per CTA; TW warps along the tokens, the others and blockIdx.z split the
+// width.  A lane's operand fragment is eight consecutive columns (the order of the columns inside a product does not matter as
+// long as both operands agree), so fragments come straight from global memory as 16-byte loads.
+template <typename T, int MT, int TW>
+__global__ void __launch_bounds__(256, 2) moe_logits_kernel(const RfMoeRouter p) {
+  pdl_prologue();
+  constexpr int KW = 8 / TW, ROWS = 16 * MT * TW, LD = 68;
+  extern __shared__ __align__(16) float lg[];             // [KW][ROWS][LD]
   const int E = p.experts, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3;
-  const int splits = gridDim.z, rank = blockIdx.z, t0 = blockIdx.x * 16 * MT;
+  const int tw = warp % TW, kw = warp / TW, t0 = blockIdx.x * ROWS + tw * 16 * MT, e0 = blockIdx.y * 64;
   const T* x = reinterpret_cast<const T*>(p.x);
-  const T* w = reinterpret_cast<const T*>(p.w);
-  pdl_wait();
-  const int kb_n = (p.width + 31) / 32;
+  const T* w = reinterpret_cast<const T*>(p.w) + (size_t)(e0 + g) * p.width;
+  const int kb_n = (p.width + 31) / 32, step = KW * gridDim.z;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-  for (int e0 = 0; e0 < E; e0 += 64) {
-    float acc[MT][8][4];
+  float acc[MT][8][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[m][n][i] = 0.f;
+  for (int kb = blockIdx.z * KW + kw; kb < kb_n; kb += step) {
+    const int k = kb * 32 + q * 8;
+    const bool kin = k < p.width;
+    uint4 b[8], a[MT][2];
+#pragma unroll
+    for (int n = 0; n < 8; ++n) b[n] = kin && e0 + n * 8 + g < E ? *reinterpret_cast<const uint4*>(w + (size_t)(n * 8) * p.width + k) : zero;
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int n = 0; n < 8; ++n)
+      for (int h = 0; h < 2; ++h) {
+        const int t = t0 + m * 16 + h * 8 + g;
+        a[m][h] = kin && t < p.rows ? *reinterpret_cast<const uint4*>(x + (size_t)t * p.ldx + k) : zero;
+      }
 #pragma unroll
-        for (int i = 0; i < 4; ++i) acc[m][n][i] = 0.f;
-#pragma unroll 2
-    for (int kb = rank * 8 + warp; kb < kb_n; kb += 8 * splits) {
-      const int k = kb * 32 + q * 8;
-      const bool kin = k < p.width;
-      uint4 b[8], a[MT][2];
+    for (int m = 0; m < MT; ++m) {
+      const uint32_t a0[4] = {a[m][0].x, a[m][1].x, a[m][0].y, a[m][1].y}, a1[4] = {a[m][0].z, a[m][1].z, a[m][0].w, a[m][1].w};
 #pragma unroll
       for (int n = 0; n < 8; ++n) {
-        const int e = e0 + n * 8 + g;
-        b[n] = kin && e < E ? *reinterpret_cast<const uint4*>(w + (size_t)e * p.width + k) : zero;
+        MmaOp<T>::mma(acc[m][n], a0, b[n].x, b[n].y);
+        MmaOp<T>::mma(acc[m][n], a1, b[n].z, b[n].w);
       }
-#pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          const int t = t0 + m * 16 + h * 8 + g;
-          a[m][h] = kin && t < p.rows ? *reinterpret_cast<const uint4*>(x + (size_t)t * p.ldx + k) : zero;
-        }
-#pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        const uint32_t a0[4] = {a[m][0].x, a[m][1].x, a[m][0].y, a[m][1].y}, a1[4] = {a[m][0].z, a[m][1].z, a[m][0].w, a[m][1].w};
-#pragma unroll
-        for (int n = 0; n < 8; ++n) {
-          MmaOp<T>::mma(acc[m][n], a0, b[n].x, b[n].y);
-          MmaOp<T>::mma(acc[m][n], a1, b[n].z, b[n].w);
-        }
-      }
-    }
-    for (int v = 0; v < 8; ++v) {                          // the warps add in order: the same sum every time
-      if (warp == v) {
-#pragma unroll
-        for (int m = 0; m < MT; ++m)
-#pragma unroll
-          for (int n = 0; n < 8; ++n)
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-              const int e = e0 + n * 8 + q * 2 + (i & 1), r = m * 16 + g + (i >> 1) * 8;
-              if (e < E) lg[r * E + e] = (v ? lg[r * E + e] : 0.f) + acc[m][n][i];
-            }
-      }
-      __syncthreads();
     }
   }
-  if (splits > 1) cluster_sync_all();
-  float* keys = lg + 16 * MT * E + warp * E;
-  for (int r = rank + splits * warp; r < 16 * MT; r += splits * 8) {
-    if (t0 + r >= p.rows) break;
-    float sc[kRtLane];
 #pragma unroll
-    for (int s = 0; s < kRtLane; ++s) {
-      const int e = s * 32 + lane;
-      sc[s] = 0.f;
-      if (e < E) {
-        if (splits == 1) sc[s] = lg[r * E + e];
-        else
-          for (int z = 0; z < splits; ++z) sc[s] += ld_dsmem_f32(dsmem_addr(smem_u32(lg + r * E + e), (uint32_t)z));
-      }
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < 8; ++n) {
+      float* o = lg + ((size_t)kw * ROWS + tw * 16 * MT + m * 16 + g) * LD + n * 8 + q * 2;
+      *reinterpret_cast<float2*>(o) = make_float2(acc[m][n][0], acc[m][n][1]);
+      *reinterpret_cast<float2*>(o + 8 * LD) = make_float2(acc[m][n][2], acc[m][n][3]);
     }
-    route_token(p, t0 + r, lane, sc, keys);
+  __syncthreads();
+  for (int i = tid; i < ROWS * 64; i += 256) {
+    const int r = i >> 6, e = i & 63, t = blockIdx.x * ROWS + r;
+    if (t >= p.rows || e0 + e >= E) continue;
+    float s = 0.f;
+#pragma unroll
+    for (int z = 0; z < KW; ++z) s += lg[((size_t)z * ROWS + r) * LD + e];       // the warps' parts in order: the same sum every time
+    p.logits[((size_t)blockIdx.z * p.rows + t) * E + e0 + e] = s;
   }
-  if (splits > 1) cluster_sync_all();                      // nobody leaves while its logits are read
-  router_ticket(p);
 }
 
 // 32-bit models: one CTA per token, a warp per expert.
-__global__ void __launch_bounds__(256) moe_router_f32_kernel(const RfMoeRouter p) {
+__global__ void __launch_bounds__(256) moe_logits_f32_kernel(const RfMoeRouter p) {
   pdl_prologue();
-  extern __shared__ __align__(16) float lg[];
-  const int E = p.experts, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x;
   const float* x = reinterpret_cast<const float*>(p.x) + (size_t)t * p.ldx;
-  for (int e = warp; e < E; e += 8) {
+  for (int e = warp; e < p.experts; e += 8) {
     const float* w = reinterpret_cast<const float*>(p.w) + (size_t)e * p.width;
     float s = 0.f;
     for (int i = lane; i < p.width; i += 32) s += x[i] * w[i];
     s = warp_sum(s);
-    if (lane == 0) lg[e] = s;
+    if (lane == 0) p.logits[(size_t)t * p.experts + e] = s;
   }
-  __syncthreads();
-  if (warp == 0) {
-    float sc[kRtLane];
-#pragma unroll
-    for (int s = 0; s < kRtLane; ++s) sc[s] = s * 32 + lane < E ? lg[s * 32 + lane] : 0.f;
-    route_token(p, t, lane, sc, lg + E);
-  }
-  router_ticket(p);
 }
 
 // Prefill-sized batches: every token's row is copied to its sorted rows.
@@ -494,11 +517,30 @@ __global__ void __launch_bounds__(256) moe_f32_kernel(const RfMoeExperts p) {
     }
 }
 
-template <typename T, int MT>
-static int launch_router(const RfMoeRouter* a, int splits, cudaStream_t s) {
-  const size_t smem = (size_t)(16 * MT + 8) * a->experts * sizeof(float);
-  RF_ALLOW_SMEM_PER_DEVICE((moe_router_kernel<T, MT>), 128 * 1024);
-  RF_CUDA_CHECK(::rf::launch_k(moe_router_kernel<T, MT>, dim3(ceil_div(a->rows, 16 * MT), 1, splits), dim3(256), smem, s, splits, *a));
+// CTAs that share the width of one tile of tokens: about two 32-column blocks per warp, as long as the GPU has room
+static int router_splits(int rows, int experts, int width) {
+  if (rows > 1024) return 1;
+  const int tiles = ceil_div(rows, 16) * ceil_div(experts, 64);
+  return std::max(1, std::min({16, width / (32 * 8 * 2), 2 * sm_count() / tiles}));
+}
+
+template <typename T, int MT, int TW>
+static int launch_logits(const RfMoeRouter* a, int splits, cudaStream_t s) {
+  constexpr int ROWS = 16 * MT * TW;
+  const size_t smem = (size_t)(8 / TW) * ROWS * 68 * sizeof(float);
+  RF_ALLOW_SMEM_PER_DEVICE((moe_logits_kernel<T, MT, TW>), 80 * 1024);
+  RF_CUDA_CHECK(::rf::launch_k(moe_logits_kernel<T, MT, TW>, dim3(ceil_div(a->rows, ROWS), ceil_div(a->experts, 64), splits), dim3(256), smem, s, 1, *a));
+  ::rf::count_launch();
+  return RF_OK;
+}
+
+template <int S>
+static int launch_choose(const RfMoeRouter* a, int splits, cudaStream_t s) {
+  const bool alone = a->rows <= kRtOneCta;
+  const int per_cta = alone ? kRtOneCta : kRtTokens;
+  const size_t smem = ((size_t)kRtTokens * a->experts + 3 * per_cta * a->k) * sizeof(float);
+  RF_ALLOW_SMEM_PER_DEVICE(moe_choose_kernel<S>, 64 * 1024);
+  RF_CUDA_CHECK(::rf::launch_k(moe_choose_kernel<S>, dim3(alone ? 1 : ceil_div(a->rows, kRtTokens)), dim3(kRtTokens * 32), smem, s, 1, *a, splits));
   ::rf::count_launch();
   return RF_OK;
 }
@@ -540,19 +582,26 @@ extern "C" int rf_moe_router(const RfMoeRouter* a, rf_stream_t stream) {
   RF_SKIP_IF_REPLAYING();
   int rc = check_router(a);
   if (rc) return rc;
-  RF_REQUIRE(a->w, "moe_router: weights");
+  RF_REQUIRE(a->w && a->logits, "moe_router: weights and logits");
   if (a->rows == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  int splits = 1, rc2;
   if (a->dtype == kF32) {
-    RF_CUDA_CHECK(::rf::launch_k(moe_router_f32_kernel, dim3(a->rows), dim3(256), 2 * a->experts * sizeof(float), s, 1, *a));
+    RF_CUDA_CHECK(::rf::launch_k(moe_logits_f32_kernel, dim3(a->rows), dim3(256), 0, s, 1, *a));
     ::rf::count_launch();
-    return RF_OK;
+  } else {
+    const bool many = a->rows > 1024;
+    splits = router_splits(a->rows, a->experts, a->width);
+    if (a->dtype == kF16) rc2 = many ? launch_logits<__half, 2, 2>(a, 1, s) : launch_logits<__half, 1, 1>(a, splits, s);
+    else rc2 = many ? launch_logits<__nv_bfloat16, 2, 2>(a, 1, s) : launch_logits<__nv_bfloat16, 1, 1>(a, splits, s);
+    if (rc2) return rc2;
   }
-  // few tokens: the width is split over clusters of eight CTAs; many: 64 tokens share one pass over the router's weights
-  const bool many = a->rows > 1024;
-  const int tiles = ceil_div(a->rows, 16), splits = many || a->width < 512 ? 1 : (tiles > 32 ? 2 : (tiles > 16 ? 4 : 8));
-  if (a->dtype == kF16) return many ? launch_router<__half, 4>(a, 1, s) : launch_router<__half, 1>(a, splits, s);
-  return many ? launch_router<__nv_bfloat16, 4>(a, 1, s) : launch_router<__nv_bfloat16, 1>(a, splits, s);
+  return a->experts <= 64 ? launch_choose<2>(a, splits, s) : launch_choose<kRtLane>(a, splits, s);
+}
+
+extern "C" uint64_t rf_moe_router_scratch_bytes(int rows, int experts) {
+  // rows x splits stays below two waves of 16-row tiles unless there is one split only
+  return ((uint64_t)std::max(rows, 2 * sm_count() * 16 + 16)) * experts * sizeof(float);
 }
 
 extern "C" int rf_moe_gather(const RfMoeRouter* a, void* out, int64_t ldo, rf_stream_t stream) {

@@ -31,7 +31,7 @@ struct MixedStack {
   uint8_t* base = nullptr;
   uint64_t off_x[2] = {}, off_h = 0, off_cast = 0, off_wide = 0, off_mix = 0, off_y = 0, off_side = 0, off_qlat = 0, off_olat = 0,
            off_ctx = 0, off_kv = 0, off_kvmeta = 0, off_attn_ws = 0, off_head = 0, off_argmax = 0, off_sk_ws = 0, off_sk_flags = 0,
-           off_status = 0, off_vfirst = 0, off_conv = 0, off_bc = 0, off_dt = 0, off_moe = 0, off_xg = 0, off_hg = 0, off_yg = 0, total = 0;
+           off_status = 0, off_vfirst = 0, off_conv = 0, off_bc = 0, off_dt = 0, off_moe = 0, off_xg = 0, off_hg = 0, off_yg = 0, off_router = 0, total = 0;
   uint64_t attn_ws_bytes = 0, argmax_bytes = 0, sk_ws_bytes = 0, rows_ws_bytes = 0;
   int moe_tiles = 0;      // tile-list entries of any mixture-of-experts layer
   int lat_rows = 0;       // rows one latent-space attention launch takes
@@ -56,7 +56,7 @@ struct MixedStack {
     auto al = [](uint64_t v) { return (v + 1023) & ~uint64_t(1023); };
     const uint64_t T = (uint64_t)cfg.max_tokens, H = (uint64_t)cfg.hidden, e = esz();
     uint64_t wide = 8, mix = 8, lat = 0, rank = 0, kvw = 0, past = 0, heads = 0;
-    uint64_t vfirst = 0, inner = 0, bc = 0, picks = 0, hg = 0;
+    uint64_t vfirst = 0, inner = 0, bc = 0, picks = 0, experts = 0, hg = 0;
     rows_ws_bytes = 0; moe_tiles = 0;
     for (const RfMixedLayer& l : layers) {
       wide = std::max<uint64_t>(wide, std::max(l.in_dim, l.inter));
@@ -71,6 +71,7 @@ struct MixedStack {
       }
       if (l.experts > 0) {
         picks = std::max<uint64_t>(picks, l.top + 1);
+        experts = std::max<uint64_t>(experts, l.experts);
         hg = std::max<uint64_t>(hg, moe_ld(l));
         moe_tiles = std::max(moe_tiles, l.experts + (int)(T * (l.top + 1) / 16) + 2);
       }
@@ -114,6 +115,7 @@ struct MixedStack {
     off_dt = o; o += al(fp32() ? 0 : T * inner * e);
     // counters, start | tile list | ids, weights, rank | slot_of, token_of_slot, slot_w (one column more)
     off_moe = o; o += al(picks ? (6 * T * picks + 2 * kMoeExperts + 4 + 4ull * moe_tiles) * 4 : 0);
+    off_router = o; o += al(picks ? rf_moe_router_scratch_bytes(cfg.max_tokens, (int)experts) : 0);
     off_xg = o; o += al(fp32() || !picks ? 0 : T * (picks - 1) * H * e);
     off_hg = o; o += al(T * picks * hg * e);
     off_yg = o; o += al(T * picks * H * e);
@@ -407,6 +409,7 @@ static int experts(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f
   const int ldh = MixedStack::moe_ld(w), bank_rt = ceil_div(w.bank_inter, 128), kbH = ceil_div(H, 64);
   int32_t* m = s.at<int32_t>(s.off_moe);
   RfMoeRouter r = {};
+  r.logits = s.at<float>(s.off_router);
   r.x = h; r.ldx = H; r.w = w.router; r.correction = w.correction;
   r.counters = m; m += MixedStack::kMoeExperts;      // the same place whatever a layer's expert count: they are zero between launches
   r.start = m; m += MixedStack::kMoeExperts;

@@ -494,7 +494,7 @@ int rf_moe_combine(void* out, int64_t ldo, const void* y, int64_t ldy, const int
                    int dtype, rf_stream_t stream);
 
 
-// Router and expert plan in one launch.  logits = x w^T in fp32, scores = softmax (or sigmoid) over all experts, choice scores =
+// Router and expert plan, two launches.  logits = x w^T in fp32, scores = softmax (or sigmoid) over all experts, choice scores =
 // scores + correction; only experts of the `keep` best of `groups` equal groups (a group counts as much as its best expert) can be
 // chosen, the k largest choice scores are; weights are the chosen experts' scores, divided by their sum with norm_topk, times
 // scale.  Outputs: ids / weights [rows, k]; rank [rows, k] = the pick's place among its expert's picks; start [experts];
@@ -510,7 +510,9 @@ typedef struct RfMoeRouter {
   int32_t* slot_of; int32_t* token_of_slot; float* slot_w;
   int32_t rows, experts, width, k, groups, keep, score_fn, norm_topk; float scale;
   int32_t tile_rows, slot_ld, has_shared, shared_tiles, scatter, dtype;
+  float* logits;                       // scratch, rf_moe_router_scratch_bytes
 } RfMoeRouter;
+uint64_t rf_moe_router_scratch_bytes(int rows, int experts);
 int rf_moe_router(const RfMoeRouter* a, rf_stream_t stream);
 // Copies every row of x to the sorted rows of its picks (and writes slot_of, token_of_slot, slot_w).
 int rf_moe_gather(const RfMoeRouter* a, void* out, int64_t ldo, rf_stream_t stream);

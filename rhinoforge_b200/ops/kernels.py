@@ -764,6 +764,7 @@ class RoutedBatch:
         self.tiles = i32(4 * (self.max_tiles + 1))
         self.slot_of, self.token_of_slot = i32(T, k + shared), i32(T * (k + shared))
         self.slot_w = torch.zeros(T * (k + shared), dtype=torch.float32, device=x.device)
+        self.logits = torch.empty(N.lib().rf_moe_router_scratch_bytes(T, E), dtype=torch.uint8, device=x.device)
         a = self.args = N.RfMoeRouter()
         a.x, a.ldx, a.w, a.correction = x.data_ptr(), x.stride(0), w.data_ptr(), _ptr(correction)
         a.ids, a.weights, a.rank, a.counters, a.start, a.tiles, a.slot_of, a.token_of_slot, a.slot_w = (t.data_ptr() for t in (
@@ -771,7 +772,7 @@ class RoutedBatch:
         a.rows, a.experts, a.width, a.k, a.groups, a.keep = T, E, w.shape[1], k, groups, keep
         a.score_fn, a.norm_topk, a.scale = {"sigmoid": 0, "softmax": 1}[score_fn], int(norm_topk), scale
         a.tile_rows, a.slot_ld, a.has_shared, a.shared_tiles, a.scatter = tile_rows, k + shared, int(shared), int(shared and scatter), int(scatter)
-        a.dtype = dtype_code_any(x.dtype)
+        a.dtype, a.logits = dtype_code_any(x.dtype), self.logits.data_ptr()
 
     def route(self) -> "RoutedBatch":
         N.check(N.lib().rf_moe_router(C.byref(self.args), _stream()), "rf_moe_router")
@@ -785,7 +786,7 @@ class RoutedBatch:
 
 
 def moe_router(x: torch.Tensor, w: torch.Tensor, k: int, **kw) -> RoutedBatch:
-    """Logits (fp32), scores, group-limited choice, weights and the tile list of the expert GEMMs, in one launch."""
+    """Logits (fp32), scores, group-limited choice, weights and the tile list of the expert GEMMs."""
     return RoutedBatch(x, w, k, **kw).route()
 
 
