@@ -110,40 +110,143 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const RfConvSilu p, int 
 constexpr int kMbChannels = 64;       // channels per CTA (256 threads)
 constexpr int kMbRows = 8;            // rows staged in shared memory at a time
 
-// A CTA owns 64 channels of `seqs_per_cta` neighbouring sequences, whose rows are contiguous.  The step sizes of eight rows at a
-// time come from one small matrix product: 16-bit models run it on mma.sync (channels on the M axis, the rows on the N axis, eight
-// warps as four channel tiles times two halves of the rank, weights straight from L2 into the fragments), 32-bit ones keep the
-// weights of the channels in shared memory.
+// Shared memory of a CTA: operands of eight rows for its 64 channels, and what the step-size product needs (16-bit models: the
+// inputs of the rows and the two halves of the product; 32-bit models: inputs and the weights of the channels).
+template <typename T, int QPL>
+struct MbTile {
+  static constexpr int CH = kMbChannels, SP = 16 * QPL;             // SP: states per channel in shared memory, zero padded
+  static constexpr bool kMma = sizeof(T) == 2;
+  int rank_p, wp;
+  T* in;              // [rows][wp] step-size inputs
+  float* pre;         // [2][rows][CH] halves of the product (16 bits)
+  T* w;               // [CH][wp] (32 bits)
+  float* b; float* c; // [rows][SP]
+  float* x; float* z; // [rows][CH]; x is replaced by the result
+  __device__ __forceinline__ MbTile(uint8_t* raw, int rank) {
+    rank_p = (rank + 31) & ~31; wp = rank_p + 8;
+    in = reinterpret_cast<T*>(raw);
+    pre = reinterpret_cast<float*>(in + kMbRows * wp);
+    b = pre + (kMma ? 2 * kMbRows * CH : 0);
+    c = b + kMbRows * SP;
+    x = c + kMbRows * SP;
+    z = x + kMbRows * CH;
+    w = reinterpret_cast<T*>(z + kMbRows * CH);
+  }
+  static size_t bytes(int rank) {
+    const int rank_p = (rank + 31) & ~31, wp = rank_p + 8;
+    return (size_t)kMbRows * wp * sizeof(T) + ((size_t)(kMma ? 2 * kMbRows * CH : 0) + 2 * kMbRows * (SP + CH)) * sizeof(float) +
+           (kMma ? 0 : (size_t)CH * wp * sizeof(T));
+  }
+  // padding columns to zero, and in 32 bits the weights: nothing of this depends on the previous kernel
+  __device__ __forceinline__ void prepare(const RfMamba1& p, int c0) {
+    const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    for (int i = threadIdx.x; i < kMbRows * wp / 8; i += 256) store8(in + i * 8, zero);
+    for (int i = threadIdx.x; i < 2 * kMbRows * SP; i += 256) b[i] = 0.f;
+    if constexpr (!kMma) {
+      for (int i = threadIdx.x; i < CH * (wp / 8); i += 256) {
+        const int r = i / (wp / 8), k = (i % (wp / 8)) * 8;
+        float f[8];
+        zero8(f);
+        if (c0 + r < p.inner && k < p.rank) load8(reinterpret_cast<const T*>(p.w_dt) + (size_t)(c0 + r) * p.rank + k, f);
+        store8(w + (size_t)r * wp + k, f);
+      }
+    }
+  }
+  // operands of rows r0 .. r0 + nr - 1
+  __device__ __forceinline__ void stage(const RfMamba1& p, int c0, int r0, int nr) {
+    for (int i = threadIdx.x; i < nr * (p.rank / 8); i += 256) {
+      const int r = i / (p.rank / 8), k = (i % (p.rank / 8)) * 8;
+      *reinterpret_cast<Vec8<T>*>(in + r * wp + k) = *reinterpret_cast<const Vec8<T>*>(reinterpret_cast<const T*>(p.bc) + (size_t)(r0 + r) * p.ld_bc + k);
+    }
+    for (int i = threadIdx.x; i < nr * (p.states / 4); i += 256) {          // B and C: states / 8 pieces each
+      const int r = i / (p.states / 4), k = (i % (p.states / 4)) * 8;
+      const bool is_c = k >= p.states;
+      float f[8];
+      load8(reinterpret_cast<const T*>(p.bc) + (size_t)(r0 + r) * p.ld_bc + p.rank + k, f);
+      store8((is_c ? c : b) + r * SP + (is_c ? k - p.states : k), f);
+    }
+    for (int i = threadIdx.x; i < nr * (CH / 8) * 2; i += 256) {
+      const int zi = i & 1, r = (i >> 1) / (CH / 8), k = ((i >> 1) % (CH / 8)) * 8;
+      float f[8];
+      zero8(f);
+      if (c0 + k < p.inner) load8((zi ? reinterpret_cast<const T*>(p.z) + (size_t)(r0 + r) * p.ldz : reinterpret_cast<const T*>(p.x) + (size_t)(r0 + r) * p.ldx) + c0 + k, f);
+      store8((zi ? z : x) + r * CH + k, f);
+    }
+  }
+  // 16 bits: step sizes of the staged rows on mma.sync - channels on the M axis, rows on the N axis, eight warps as four channel
+  // tiles times two halves of the rank, weights straight from L2 into the fragments (a lane's eight consecutive columns)
+  __device__ __forceinline__ void project(const RfMamba1& p, int c0) {
+    if constexpr (kMma) {
+      const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3, mt = warp & 3, half = warp >> 2;
+      float acc[4] = {0.f, 0.f, 0.f, 0.f};
+      const T* w0 = reinterpret_cast<const T*>(p.w_dt) + (size_t)(c0 + mt * 16 + g) * p.rank;
+      const bool in0 = c0 + mt * 16 + g < p.inner, in1 = c0 + mt * 16 + g + 8 < p.inner;
+      const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll 4
+      for (int kb = half; kb < rank_p / 32; kb += 2) {
+        const int k = kb * 32 + q * 8;
+        const uint4 a0 = in0 && k < p.rank ? *reinterpret_cast<const uint4*>(w0 + k) : zero;
+        const uint4 a1 = in1 && k < p.rank ? *reinterpret_cast<const uint4*>(w0 + (size_t)8 * p.rank + k) : zero;
+        const uint4 bb = *reinterpret_cast<const uint4*>(in + g * wp + k);
+        const uint32_t lo[4] = {a0.x, a1.x, a0.y, a1.y}, hi[4] = {a0.z, a1.z, a0.w, a1.w};
+        MmaOp<T>::mma(acc, lo, bb.x, bb.y);
+        MmaOp<T>::mma(acc, hi, bb.z, bb.w);
+      }
+      float* o = pre + half * kMbRows * CH + mt * 16 + g;
+      o[(q * 2) * CH] = acc[0]; o[(q * 2 + 1) * CH] = acc[1];
+      o[(q * 2) * CH + 8] = acc[2]; o[(q * 2 + 1) * CH + 8] = acc[3];
+    }
+  }
+  // step-size product of staged row r and this thread's channel (all four lanes of the channel get it)
+  __device__ __forceinline__ float product(int r, int ci, int l) const {
+    if constexpr (kMma) return pre[r * CH + ci] + pre[(kMbRows + r) * CH + ci];
+    float dot = 0.f;
+    for (int k = l * 8; k < rank_p; k += 32) {
+      float w8[8], d8[8];
+      load8(w + (size_t)ci * wp + k, w8);
+      load8(in + r * wp + k, d8);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) dot += w8[j] * d8[j];
+    }
+    dot += __shfl_xor_sync(0xffffffffu, dot, 1);
+    return dot + __shfl_xor_sync(0xffffffffu, dot, 2);
+  }
+  // one token of one channel: new state, and the gated result in place of x
+  __device__ __forceinline__ void token(int r, int ci, int l, float bias, float D, const float4 (&A)[QPL], float4 (&S)[QPL]) {
+    const float dt = softplus_t<T>(product(r, ci, l) + bias), xv = x[r * CH + ci], dx = dt * xv;
+    float y = 0.f;
+#pragma unroll
+    for (int q = 0; q < QPL; ++q) {
+      const float4 B = *reinterpret_cast<const float4*>(b + r * SP + (l + 4 * q) * 4), C = *reinterpret_cast<const float4*>(c + r * SP + (l + 4 * q) * 4);
+      S[q].x = S[q].x * exp2_t<T>(dt * A[q].x) + dx * B.x; y += S[q].x * C.x;
+      S[q].y = S[q].y * exp2_t<T>(dt * A[q].y) + dx * B.y; y += S[q].y * C.y;
+      S[q].z = S[q].z * exp2_t<T>(dt * A[q].z) + dx * B.z; y += S[q].z * C.z;
+      S[q].w = S[q].w * exp2_t<T>(dt * A[q].w) + dx * B.w; y += S[q].w * C.w;
+    }
+    y += __shfl_xor_sync(0xffffffffu, y, 1);
+    y += __shfl_xor_sync(0xffffffffu, y, 2);
+    if (l == 0) x[r * CH + ci] = (y + D * xv) * silu_t<T>(z[r * CH + ci]);   // read by these four lanes only, all of them done
+  }
+  __device__ __forceinline__ void write(const RfMamba1& p, int c0, int r0, int nr) const {
+    for (int i = threadIdx.x; i < nr * (CH / 8); i += 256) {
+      const int r = i / (CH / 8), k = (i % (CH / 8)) * 8;
+      if (c0 + k >= p.inner) continue;
+      float f[8];
+      load8(x + r * CH + k, f);
+      store8(reinterpret_cast<T*>(p.out) + (size_t)(r0 + r) * p.ldo + c0 + k, f);
+    }
+  }
+};
+
+// Any portions: a CTA owns 64 channels of `seqs_per_cta` neighbouring sequences, whose rows are contiguous.
 template <typename T, int QPL>
 __global__ void __launch_bounds__(256) mamba_recurrent_kernel(const RfMamba1 p, int seqs_per_cta) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) uint8_t mb_raw[];
-  constexpr int CH = kMbChannels, SP = 16 * QPL;                    // SP: states per channel in shared memory, zero padded
-  constexpr bool kMma = sizeof(T) == 2;
-  const int rank_p = (p.rank + 31) & ~31, wp = rank_p + 8;
-  float* s_dt = reinterpret_cast<float*>(mb_raw);                   // 32 bits: [rows][rank_p] step-size inputs
-  T* s_di = reinterpret_cast<T*>(mb_raw);                           // 16 bits: [rows][wp], and behind them
-  float* s_pre = reinterpret_cast<float*>(s_di + kMbRows * wp);     // [2][rows][CH] halves of the products
-  const int head_floats = kMma ? kMbRows * wp / 2 + 2 * kMbRows * CH : kMbRows * rank_p;
-  float* s_b = s_dt + head_floats;                                  // [rows][SP]
-  float* s_c = s_b + kMbRows * SP;
-  float* s_x = s_c + kMbRows * SP;                                  // [rows][CH]
-  float* s_z = s_x + kMbRows * CH;
-  T* s_w = reinterpret_cast<T*>(s_z + kMbRows * CH);                // [CH][wp]
-  const int tid = threadIdx.x, l = tid & 3, ci = tid >> 2, c0 = blockIdx.x * CH, c = c0 + ci;
+  MbTile<T, QPL> tile(mb_raw, p.rank);
+  const int l = threadIdx.x & 3, ci = threadIdx.x >> 2, c0 = blockIdx.x * kMbChannels, c = c0 + ci, nq = p.states / 4;
   const bool live = c < p.inner;
-  // the weights do not depend on the previous kernel
-  if constexpr (!kMma) {
-    for (int i = tid; i < CH * (wp / 8); i += 256) {
-      const int r = i / (wp / 8), k = (i % (wp / 8)) * 8;
-      float f[8];
-      zero8(f);
-      if (c0 + r < p.inner && k < p.rank) load8(reinterpret_cast<const T*>(p.w_dt) + (size_t)(c0 + r) * p.rank + k, f);
-      store8(s_w + (size_t)r * wp + k, f);
-    }
-  }
-  for (int i = tid; i < head_floats + kMbRows * 2 * SP; i += 256) s_dt[i] = 0.f;
-  const int nq = p.states / 4;
+  tile.prepare(p, c0);
   float4 A[QPL];
 #pragma unroll
   for (int q = 0; q < QPL; ++q)
@@ -167,47 +270,10 @@ __global__ void __launch_bounds__(256) mamba_recurrent_kernel(const RfMamba1 p, 
   for (int r0 = row_begin; r0 < row_end; r0 += kMbRows) {
     const int nr = min(kMbRows, row_end - r0);
     __syncthreads();
-    for (int i = tid; i < nr * (p.rank / 8); i += 256) {
-      const int r = i / (p.rank / 8), k = (i % (p.rank / 8)) * 8;
-      float f[8];
-      load8(reinterpret_cast<const T*>(p.bc) + (size_t)(r0 + r) * p.ld_bc + k, f);
-      if (kMma) store8(s_di + r * wp + k, f);
-      else store8(s_dt + r * rank_p + k, f);
-    }
-    for (int i = tid; i < nr * (p.states / 4); i += 256) {          // B and C: states / 8 pieces each
-      const int r = i / (p.states / 4), k = (i % (p.states / 4)) * 8;
-      const bool is_c = k >= p.states;
-      float f[8];
-      load8(reinterpret_cast<const T*>(p.bc) + (size_t)(r0 + r) * p.ld_bc + p.rank + k, f);
-      store8((is_c ? s_c : s_b) + r * SP + (is_c ? k - p.states : k), f);
-    }
-    for (int i = tid; i < nr * (CH / 8) * 2; i += 256) {
-      const int zi = i & 1, r = (i >> 1) / (CH / 8), k = ((i >> 1) % (CH / 8)) * 8;
-      float f[8];
-      zero8(f);
-      if (c0 + k < p.inner) load8((zi ? reinterpret_cast<const T*>(p.z) + (size_t)(r0 + r) * p.ldz : reinterpret_cast<const T*>(p.x) + (size_t)(r0 + r) * p.ldx) + c0 + k, f);
-      store8((zi ? s_z : s_x) + r * CH + k, f);
-    }
+    tile.stage(p, c0, r0, nr);
     __syncthreads();
-    if constexpr (kMma) {
-      const int warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3, mt = warp & 3, half = warp >> 2;
-      float acc[4] = {0.f, 0.f, 0.f, 0.f};
-      const T* w0 = reinterpret_cast<const T*>(p.w_dt) + (size_t)(c0 + mt * 16 + g) * p.rank;
-      const bool in0 = c0 + mt * 16 + g < p.inner, in1 = c0 + mt * 16 + g + 8 < p.inner;
-      const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-#pragma unroll 4
-      for (int kb = half; kb < rank_p / 32; kb += 2) {              // a lane's fragment: eight consecutive columns of both operands
-        const int k = kb * 32 + q * 8;
-        const uint4 a0 = in0 && k < p.rank ? *reinterpret_cast<const uint4*>(w0 + k) : zero;
-        const uint4 a1 = in1 && k < p.rank ? *reinterpret_cast<const uint4*>(w0 + (size_t)8 * p.rank + k) : zero;
-        const uint4 b = *reinterpret_cast<const uint4*>(s_di + g * wp + k);
-        const uint32_t lo[4] = {a0.x, a1.x, a0.y, a1.y}, hi[4] = {a0.z, a1.z, a0.w, a1.w};
-        MmaOp<T>::mma(acc, lo, b.x, b.y);
-        MmaOp<T>::mma(acc, hi, b.z, b.w);
-      }
-      float* o = s_pre + half * kMbRows * CH + mt * 16 + g;
-      o[(q * 2) * CH] = acc[0]; o[(q * 2 + 1) * CH] = acc[1];
-      o[(q * 2) * CH + 8] = acc[2]; o[(q * 2 + 1) * CH + 8] = acc[3];
+    if (MbTile<T, QPL>::kMma) {
+      tile.project(p, c0);
       __syncthreads();
     }
     for (int r = 0; r < nr; ++r) {
@@ -217,35 +283,7 @@ __global__ void __launch_bounds__(256) mamba_recurrent_kernel(const RfMamba1 p, 
         if (seq + 1 < s1) load_state(seq + 1, next);
         start = false;
       }
-      float dot = 0.f;
-      if constexpr (kMma) {
-        dot = s_pre[r * CH + ci] + s_pre[(kMbRows + r) * CH + ci];
-      } else {
-        const T* wr = s_w + (size_t)ci * wp + l * 8;
-        const float* dr = s_dt + r * rank_p + l * 8;
-        for (int k = 0; k < rank_p; k += 32) {
-          float w8[8], d8[8];
-          load8(wr + k, w8);
-          load8(dr + k, d8);
-#pragma unroll
-          for (int j = 0; j < 8; ++j) dot += w8[j] * d8[j];
-        }
-        dot += __shfl_xor_sync(0xffffffffu, dot, 1);
-        dot += __shfl_xor_sync(0xffffffffu, dot, 2);
-      }
-      const float dt = softplus_t<T>(dot + bias), x = s_x[r * CH + ci], dx = dt * x;
-      float y = 0.f;
-#pragma unroll
-      for (int q = 0; q < QPL; ++q) {
-        const float4 B = *reinterpret_cast<const float4*>(s_b + r * SP + (l + 4 * q) * 4), C = *reinterpret_cast<const float4*>(s_c + r * SP + (l + 4 * q) * 4);
-        S[q].x = S[q].x * exp2_t<T>(dt * A[q].x) + dx * B.x; y += S[q].x * C.x;
-        S[q].y = S[q].y * exp2_t<T>(dt * A[q].y) + dx * B.y; y += S[q].y * C.y;
-        S[q].z = S[q].z * exp2_t<T>(dt * A[q].z) + dx * B.z; y += S[q].z * C.z;
-        S[q].w = S[q].w * exp2_t<T>(dt * A[q].w) + dx * B.w; y += S[q].w * C.w;
-      }
-      y += __shfl_xor_sync(0xffffffffu, y, 1);
-      y += __shfl_xor_sync(0xffffffffu, y, 2);
-      if (l == 0) s_x[r * CH + ci] = (y + D * x) * silu_t<T>(s_z[r * CH + ci]);     // read by these four lanes only, all of them done
+      tile.token(r, ci, l, bias, D, A, S);
       if (--left == 0) {
         float4* st = reinterpret_cast<float4*>(state_of(seq));
         if (live) {
@@ -258,14 +296,52 @@ __global__ void __launch_bounds__(256) mamba_recurrent_kernel(const RfMamba1 p, 
       }
     }
     __syncthreads();
-    for (int i = tid; i < nr * (CH / 8); i += 256) {
-      const int r = i / (CH / 8), k = (i % (CH / 8)) * 8;
-      if (c0 + k >= p.inner) continue;
-      float f[8];
-      load8(s_x + r * CH + k, f);
-      store8(reinterpret_cast<T*>(p.out) + (size_t)(r0 + r) * p.ldo + c0 + k, f);
+    tile.write(p, c0, r0, nr);
+  }
+}
+
+// Decode steps, one row per sequence: the states of SEQS sequences are all in flight before anything else happens.
+template <typename T, int QPL, int SEQS>
+__global__ void __launch_bounds__(256) mamba_decode_kernel(const RfMamba1 p) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) uint8_t mb_raw[];
+  MbTile<T, QPL> tile(mb_raw, p.rank);
+  const int l = threadIdx.x & 3, ci = threadIdx.x >> 2, c0 = blockIdx.x * kMbChannels, c = c0 + ci, nq = p.states / 4;
+  const bool live = c < p.inner;
+  tile.prepare(p, c0);
+  float4 A[QPL], S[SEQS][QPL];
+#pragma unroll
+  for (int q = 0; q < QPL; ++q)
+    A[q] = live && l + 4 * q < nq ? reinterpret_cast<const float4*>(p.a2 + (size_t)c * p.states)[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
+  const float bias = live ? p.dt_bias[c] : 0.f, D = live ? p.d[c] : 0.f;
+  pdl_wait();
+  const int s0 = blockIdx.y * SEQS, n = min(SEQS, p.rows.num_seqs - s0);
+  auto state_of = [&](int i) { return reinterpret_cast<float4*>(p.state + ((size_t)(p.rows.slot ? p.rows.slot[s0 + i] : s0 + i) * p.inner + c) * p.states); };
+#pragma unroll
+  for (int i = 0; i < SEQS; ++i) {
+    const bool use = live && i < n && p.rows.pos[min(s0 + i, p.rows.num_seqs - 1)] != 0;
+#pragma unroll
+    for (int q = 0; q < QPL; ++q) S[i][q] = use && l + 4 * q < nq ? state_of(i)[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  __syncthreads();
+  tile.stage(p, c0, s0, n);
+  __syncthreads();
+  if (MbTile<T, QPL>::kMma) {
+    tile.project(p, c0);
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < SEQS; ++i) {
+    if (i >= n) break;
+    tile.token(i, ci, l, bias, D, A, S[i]);
+    if (live) {
+#pragma unroll
+      for (int q = 0; q < QPL; ++q)
+        if (l + 4 * q < nq) state_of(i)[l + 4 * q] = S[i][q];
     }
   }
+  __syncthreads();
+  tile.write(p, c0, s0, n);
 }
 
 // ------------------------------------------------------------------------------------------------- scan ----
@@ -275,7 +351,7 @@ constexpr int kScanRows = 32;
 // next tile's while the current one is scanned), turns the step sizes and gates once per (row, channel), and the four lanes of a
 // channel run the recurrence, four rows at a time so that the sums over lanes cost three shuffles per four rows.
 template <typename T, int CH, int QPL>
-__global__ void __launch_bounds__(CH * 4) mamba_scan_kernel(const RfMamba1 p) {
+__global__ void __launch_bounds__(CH * 4, QPL == 1 ? 256 / CH : 1) mamba_scan_kernel(const RfMamba1 p) {
   pdl_prologue();
   extern __shared__ __align__(16) float sc_sm[];
   constexpr int SP = 16 * QPL, NT = CH * 4, TR = kScanRows;
@@ -398,14 +474,24 @@ static int check_mamba(const RfMamba1* a) {
 template <typename T, int QPL>
 static int launch_recurrent(const RfMamba1* a, cudaStream_t s) {
   const int tiles = ceil_div(a->inner, kMbChannels), seqs = a->rows.num_seqs;
-  // share the step-size weights of a channel tile between sequences once there are enough CTAs without it
-  const int spc = std::max(1, std::min(8, seqs * tiles / (6 * sm_count())));
-  const int rank_p = (a->rank + 31) & ~31;
-  const size_t head = sizeof(T) == 2 ? (size_t)kMbRows * ((rank_p + 8) * sizeof(T) + 2 * kMbChannels * sizeof(float))
-                                     : (size_t)kMbRows * rank_p * sizeof(float);
-  const size_t smem = head + (size_t)kMbRows * (32 * QPL + 2 * kMbChannels) * sizeof(float) +
-                      (sizeof(T) == 2 ? 0 : (size_t)kMbChannels * (rank_p + 8) * sizeof(T));
+  const size_t smem = MbTile<T, QPL>::bytes(a->rank);
   RF_REQUIRE(smem <= 200 * 1024, "mamba: a step rank of %d does not fit in shared memory", a->rank);
+  constexpr int SEQS = QPL == 1 ? 8 : (QPL == 2 ? 4 : 2);            // 32 registers of states
+  if (QPL <= 4 && !a->rows.q_start) {
+    constexpr int Q = QPL <= 4 ? QPL : 1;
+    // few channel tiles: fewer sequences per CTA, more CTAs
+    if (ceil_div(seqs, SEQS) * tiles >= sm_count() || SEQS == 2) {
+      RF_ALLOW_SMEM_PER_DEVICE((mamba_decode_kernel<T, Q, SEQS>), 200 * 1024);
+      RF_CUDA_CHECK(::rf::launch_k(mamba_decode_kernel<T, Q, SEQS>, dim3(tiles, ceil_div(seqs, SEQS)), dim3(256), smem, s, 1, *a));
+    } else {
+      RF_ALLOW_SMEM_PER_DEVICE((mamba_decode_kernel<T, Q, 2>), 200 * 1024);
+      RF_CUDA_CHECK(::rf::launch_k(mamba_decode_kernel<T, Q, 2>, dim3(tiles, ceil_div(seqs, 2)), dim3(256), smem, s, 1, *a));
+    }
+    ::rf::count_launch();
+    return RF_OK;
+  }
+  // share what a CTA reads for its channels between sequences once there are enough CTAs without that
+  const int spc = std::max(1, std::min(8, seqs * tiles / (6 * sm_count())));
   RF_ALLOW_SMEM_PER_DEVICE((mamba_recurrent_kernel<T, QPL>), 200 * 1024);
   RF_CUDA_CHECK(::rf::launch_k(mamba_recurrent_kernel<T, QPL>, dim3(tiles, ceil_div(seqs, spc)), dim3(256), smem, s, 1, *a, spc));
   ::rf::count_launch();

@@ -235,7 +235,7 @@ def test_convolution_carries_its_inputs(dtype, taps):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("form", ["recurrent", "scan"])
+@pytest.mark.parametrize("form", ["recurrent", "scan", "decode"])
 @pytest.mark.parametrize("inner,states,rank", [(8, 8, 8), (72, 16, 24), (136, 24, 8), (64, 40, 40), (40, 104, 16), (24, 256, 8), (4096, 16, 256)])
 def test_selective_scan_over_portions(dtype, form, inner, states, rank):
     small = inner < 1000
@@ -261,14 +261,20 @@ def test_selective_scan_over_portions(dtype, form, inner, states, rank):
         final.append(st)
     at = [0, 0, 0]
     for lens in ([1, 2, 0], [40, 1, 1], [2, 19, 1], [32, 14, 3]) if small else ([1, 1, 1], [5, 2, 1]):
+        if form == "decode":
+            lens = [1, 1, 1]
         live = [i for i in range(3) if lens[i]]
         d, _, _ = pack([lens[i] for i in live], [at[i] for i in live], [slots[i] for i in live])
+        if form == "decode":                                                       # single tokens: rows are sequences
+            d = dict(pos=d["pos"], slot=d["slot"])
         cut = lambda t: torch.cat([t[i][at[i]:at[i] + lens[i]] for i in live])
         bc = torch.cat([cut(ds), pad(cut(bs)), pad(cut(cs))], 1).cuda().contiguous()
-        kw = dict(w_dt=w_dt.cuda()) if form == "recurrent" else dict(dt=(cut(ds).double() @ w_dt.double().T).to(dtype).cuda())
+        kw = dict(w_dt=w_dt.cuda()) if form != "scan" else dict(dt=(cut(ds).double() @ w_dt.double().T).to(dtype).cuda())
         out = K().mamba1(cut(xs).cuda(), cut(zs).cuda(), bc, a2, D.cuda(), bias.cuda(), state, K().rows(**d), **kw)
         close(out, cut(want), dtype, 4.0)
         at = [a + m for a, m in zip(at, lens)]
+    if form == "decode":
+        return
     for i, s in enumerate(slots):
         close(state[s, :, :S], final[i], F32 if dtype == F32 else BF16, 2.0)
         assert not state[s, :, S:].any()
