@@ -300,29 +300,30 @@ __global__ void __launch_bounds__(256) mamba_recurrent_kernel(const RfMamba1 p, 
   }
 }
 
-// Decode steps, one row per sequence: the states of SEQS sequences are all in flight before anything else happens.
-template <typename T, int QPL, int SEQS>
-__global__ void __launch_bounds__(256) mamba_decode_kernel(const RfMamba1 p) {
+// Decode steps, one row per sequence, up to eight of them per CTA: the states of DEPTH sequences are in flight at any time.
+template <typename T, int QPL, int DEPTH>
+__global__ void __launch_bounds__(256) mamba_decode_kernel(const RfMamba1 p, int seqs_per_cta) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) uint8_t mb_raw[];
   MbTile<T, QPL> tile(mb_raw, p.rank);
   const int l = threadIdx.x & 3, ci = threadIdx.x >> 2, c0 = blockIdx.x * kMbChannels, c = c0 + ci, nq = p.states / 4;
   const bool live = c < p.inner;
   tile.prepare(p, c0);
-  float4 A[QPL], S[SEQS][QPL];
+  float4 A[QPL], S[DEPTH][QPL];
 #pragma unroll
   for (int q = 0; q < QPL; ++q)
     A[q] = live && l + 4 * q < nq ? reinterpret_cast<const float4*>(p.a2 + (size_t)c * p.states)[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
   const float bias = live ? p.dt_bias[c] : 0.f, D = live ? p.d[c] : 0.f;
   pdl_wait();
-  const int s0 = blockIdx.y * SEQS, n = min(SEQS, p.rows.num_seqs - s0);
+  const int s0 = blockIdx.y * seqs_per_cta, n = min(seqs_per_cta, p.rows.num_seqs - s0);
   auto state_of = [&](int i) { return reinterpret_cast<float4*>(p.state + ((size_t)(p.rows.slot ? p.rows.slot[s0 + i] : s0 + i) * p.inner + c) * p.states); };
-#pragma unroll
-  for (int i = 0; i < SEQS; ++i) {
+  auto fetch = [&](int i, float4 (&s)[QPL]) {
     const bool use = live && i < n && p.rows.pos[min(s0 + i, p.rows.num_seqs - 1)] != 0;
 #pragma unroll
-    for (int q = 0; q < QPL; ++q) S[i][q] = use && l + 4 * q < nq ? state_of(i)[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
+    for (int q = 0; q < QPL; ++q) s[q] = use && l + 4 * q < nq ? state_of(i)[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
+  };
+#pragma unroll
+  for (int i = 0; i < DEPTH; ++i) fetch(i, S[i]);
   __syncthreads();
   tile.stage(p, c0, s0, n);
   __syncthreads();
@@ -331,14 +332,16 @@ __global__ void __launch_bounds__(256) mamba_decode_kernel(const RfMamba1 p) {
     __syncthreads();
   }
 #pragma unroll
-  for (int i = 0; i < SEQS; ++i) {
+  for (int i = 0; i < kMbRows; ++i) {
     if (i >= n) break;
-    tile.token(i, ci, l, bias, D, A, S[i]);
+    float4 (&s)[QPL] = S[i % DEPTH];
+    tile.token(i, ci, l, bias, D, A, s);
     if (live) {
 #pragma unroll
       for (int q = 0; q < QPL; ++q)
-        if (l + 4 * q < nq) state_of(i)[l + 4 * q] = S[i][q];
+        if (l + 4 * q < nq) state_of(i)[l + 4 * q] = s[q];
     }
+    if (i + DEPTH < n) fetch(i + DEPTH, s);
   }
   __syncthreads();
   tile.write(p, c0, s0, n);
@@ -351,15 +354,15 @@ constexpr int kScanRows = 32;
 // next tile's while the current one is scanned), turns the step sizes and gates once per (row, channel), and the four lanes of a
 // channel run the recurrence, four rows at a time so that the sums over lanes cost three shuffles per four rows.
 template <typename T, int CH, int QPL>
-__global__ void __launch_bounds__(CH * 4, QPL == 1 ? 256 / CH : 1) mamba_scan_kernel(const RfMamba1 p) {
+__global__ void __launch_bounds__(CH * 4) mamba_scan_kernel(const RfMamba1 p) {
   pdl_prologue();
   extern __shared__ __align__(16) float sc_sm[];
-  constexpr int SP = 16 * QPL, NT = CH * 4, TR = kScanRows;
-  float* s_dt = sc_sm;                     // [TR][CH] step sizes
-  float* s_dx = s_dt + TR * CH;            // step size times input; then the result
-  float* s_d = s_dx + TR * CH;             // D times input
-  float* s_g = s_d + TR * CH;              // silu(z)
-  float* s_b = s_g + TR * CH;              // [TR][SP]
+  constexpr int SP = 16 * QPL, NT = CH * 4, TR = kScanRows, LD = CH + 8;   // LD: four rows of eight channels in different banks
+  float* s_dt = sc_sm;                     // [TR][LD] step sizes
+  float* s_dx = s_dt + TR * LD;            // step size times input; then the result
+  float* s_d = s_dx + TR * LD;             // D times input
+  float* s_g = s_d + TR * LD;              // silu(z)
+  float* s_b = s_g + TR * LD;              // [TR][SP]
   float* s_c = s_b + TR * SP;
   const int tid = threadIdx.x, l = tid & 3, ci = tid >> 2, c0 = blockIdx.x * CH, c = c0 + ci, seq = blockIdx.y;
   const int q0 = p.rows.q_start ? p.rows.q_start[seq] : seq, n = p.rows.q_len ? p.rows.q_len[seq] : 1;
@@ -409,10 +412,10 @@ __global__ void __launch_bounds__(CH * 4, QPL == 1 ? 256 / CH : 1) mamba_scan_ke
           g[2 * j] = silu_t<T>(z2.x); g[2 * j + 1] = silu_t<T>(z2.y);
         }
       }
-      store8(s_dt + lr * CH + lc, dt);     // rows behind the end: step size 0 leaves the state as it is
-      store8(s_dx + lr * CH + lc, dx);
-      store8(s_d + lr * CH + lc, dd);
-      store8(s_g + lr * CH + lc, g);
+      store8(s_dt + lr * LD + lc, dt);     // rows behind the end: step size 0 leaves the state as it is
+      store8(s_dx + lr * LD + lc, dx);
+      store8(s_d + lr * LD + lc, dd);
+      store8(s_g + lr * LD + lc, g);
     }
     for (int i = tid; i < TR * (p.states / 4); i += NT) {
       const int r = i / (p.states / 4), k = (i % (p.states / 4)) * 8;
@@ -428,7 +431,7 @@ __global__ void __launch_bounds__(CH * 4, QPL == 1 ? 256 / CH : 1) mamba_scan_ke
       float v[4];
 #pragma unroll
       for (int u = 0; u < 4; ++u) {
-        const float dt = s_dt[(t + u) * CH + ci], dx = s_dx[(t + u) * CH + ci];
+        const float dt = s_dt[(t + u) * LD + ci], dx = s_dx[(t + u) * LD + ci];
         v[u] = 0.f;
 #pragma unroll
         for (int q = 0; q < QPL; ++q) {
@@ -444,13 +447,13 @@ __global__ void __launch_bounds__(CH * 4, QPL == 1 ? 256 / CH : 1) mamba_scan_ke
       const float a0 = __shfl_xor_sync(0xffffffffu, hi ? v[0] : v[2], 2), a1 = __shfl_xor_sync(0xffffffffu, hi ? v[1] : v[3], 2);
       const float w0 = (hi ? v[2] : v[0]) + a0, w1 = (hi ? v[3] : v[1]) + a1;
       const float y = (odd ? w1 : w0) + __shfl_xor_sync(0xffffffffu, odd ? w0 : w1, 1);
-      const int at = (t + l) * CH + ci;
+      const int at = (t + l) * LD + ci;
       s_dx[at] = (y + s_d[at]) * s_g[at];
     }
     __syncthreads();
     if (lr < nr && in_c) {
       float f[8];
-      load8(s_dx + lr * CH + lc, f);
+      load8(s_dx + lr * LD + lc, f);
       store8(reinterpret_cast<T*>(p.out) + (size_t)(q0 + t0 + lr) * p.ldo + c0 + lc, f);
     }
   }
@@ -476,22 +479,15 @@ static int launch_recurrent(const RfMamba1* a, cudaStream_t s) {
   const int tiles = ceil_div(a->inner, kMbChannels), seqs = a->rows.num_seqs;
   const size_t smem = MbTile<T, QPL>::bytes(a->rank);
   RF_REQUIRE(smem <= 200 * 1024, "mamba: a step rank of %d does not fit in shared memory", a->rank);
-  constexpr int SEQS = QPL == 1 ? 8 : (QPL == 2 ? 4 : 2);            // 32 registers of states
+  // share what a CTA reads for its channels between sequences once there are enough CTAs without that
+  const int spc = std::max(1, std::min(kMbRows, seqs * tiles / (4 * sm_count())));
   if (QPL <= 4 && !a->rows.q_start) {
-    constexpr int Q = QPL <= 4 ? QPL : 1;
-    // few channel tiles: fewer sequences per CTA, more CTAs
-    if (ceil_div(seqs, SEQS) * tiles >= sm_count() || SEQS == 2) {
-      RF_ALLOW_SMEM_PER_DEVICE((mamba_decode_kernel<T, Q, SEQS>), 200 * 1024);
-      RF_CUDA_CHECK(::rf::launch_k(mamba_decode_kernel<T, Q, SEQS>, dim3(tiles, ceil_div(seqs, SEQS)), dim3(256), smem, s, 1, *a));
-    } else {
-      RF_ALLOW_SMEM_PER_DEVICE((mamba_decode_kernel<T, Q, 2>), 200 * 1024);
-      RF_CUDA_CHECK(::rf::launch_k(mamba_decode_kernel<T, Q, 2>, dim3(tiles, ceil_div(seqs, 2)), dim3(256), smem, s, 1, *a));
-    }
+    constexpr int Q = QPL <= 4 ? QPL : 1, DEPTH = QPL == 1 ? 4 : 2;
+    RF_ALLOW_SMEM_PER_DEVICE((mamba_decode_kernel<T, Q, DEPTH>), 200 * 1024);
+    RF_CUDA_CHECK(::rf::launch_k(mamba_decode_kernel<T, Q, DEPTH>, dim3(tiles, ceil_div(seqs, spc)), dim3(256), smem, s, 1, *a, spc));
     ::rf::count_launch();
     return RF_OK;
   }
-  // share what a CTA reads for its channels between sequences once there are enough CTAs without that
-  const int spc = std::max(1, std::min(8, seqs * tiles / (6 * sm_count())));
   RF_ALLOW_SMEM_PER_DEVICE((mamba_recurrent_kernel<T, QPL>), 200 * 1024);
   RF_CUDA_CHECK(::rf::launch_k(mamba_recurrent_kernel<T, QPL>, dim3(tiles, ceil_div(seqs, spc)), dim3(256), smem, s, 1, *a, spc));
   ::rf::count_launch();
@@ -502,12 +498,12 @@ template <typename T, int QPL>
 static int launch_scan(const RfMamba1* a, cudaStream_t s) {
   const int seqs = a->rows.num_seqs;
   const size_t per = (size_t)kScanRows * 32 * QPL * sizeof(float);
-  if (ceil_div(a->inner, 64) * seqs >= sm_count()) {
-    const size_t smem = (size_t)kScanRows * 64 * 4 * sizeof(float) + per;
+  if (ceil_div(a->inner, 64) * seqs >= 4 * sm_count()) {
+    const size_t smem = (size_t)kScanRows * (64 + 8) * 4 * sizeof(float) + per;
     RF_ALLOW_SMEM_PER_DEVICE((mamba_scan_kernel<T, 64, QPL>), 128 * 1024);
     RF_CUDA_CHECK(::rf::launch_k(mamba_scan_kernel<T, 64, QPL>, dim3(ceil_div(a->inner, 64), seqs), dim3(256), smem, s, 1, *a));
   } else {
-    const size_t smem = (size_t)kScanRows * 32 * 4 * sizeof(float) + per;
+    const size_t smem = (size_t)kScanRows * (32 + 8) * 4 * sizeof(float) + per;
     RF_ALLOW_SMEM_PER_DEVICE((mamba_scan_kernel<T, 32, QPL>), 128 * 1024);
     RF_CUDA_CHECK(::rf::launch_k(mamba_scan_kernel<T, 32, QPL>, dim3(ceil_div(a->inner, 32), seqs), dim3(128), smem, s, 1, *a));
   }
