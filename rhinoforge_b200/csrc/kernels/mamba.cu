@@ -350,34 +350,40 @@ __global__ void __launch_bounds__(256) mamba_decode_kernel(const RfMamba1 p, int
 // ------------------------------------------------------------------------------------------------- scan ----
 constexpr int kScanRows = 32;
 
-// A CTA owns CH channels of one sequence and walks it in tiles of 32 rows: one thread fetches eight channels of one row (the
-// next tile's while the current one is scanned), turns the step sizes and gates once per (row, channel), and the four lanes of a
-// channel run the recurrence, four rows at a time so that the sums over lanes cost three shuffles per four rows.
-template <typename T, int CH, int QPL>
-__global__ void __launch_bounds__(CH * 4) mamba_scan_kernel(const RfMamba1 p) {
+// A CTA owns CH channels of one sequence and walks it in tiles of 32 rows: a thread fetches CPL pieces of eight channels of one
+// row (the next tile's while the current one is scanned) and turns the step sizes and gates once per (row, channel).  Four lanes
+// run the recurrence of CPL channels, which share what is read of B and C - shared-memory bandwidth is what bounds this kernel -
+// and go four rows at a time, so that the sums over lanes cost three shuffles per four rows.
+template <typename T, int CH, int QPL, int CPL>
+__global__ void __launch_bounds__(CH * 4 / CPL) mamba_scan_kernel(const RfMamba1 p) {
   pdl_prologue();
   extern __shared__ __align__(16) float sc_sm[];
-  constexpr int SP = 16 * QPL, NT = CH * 4, TR = kScanRows, LD = CH + 8;   // LD: four rows of eight channels in different banks
-  float* s_dt = sc_sm;                     // [TR][LD] step sizes
-  float* s_dx = s_dt + TR * LD;            // step size times input; then the result
-  float* s_d = s_dx + TR * LD;             // D times input
-  float* s_g = s_d + TR * LD;              // silu(z)
-  float* s_b = s_g + TR * LD;              // [TR][SP]
+  constexpr int SP = 16 * QPL, NT = CH * 4 / CPL, TR = kScanRows, LD = CH + 8;   // LD: four rows of eight channels in different banks
+  float2* s_q = reinterpret_cast<float2*>(sc_sm);       // [TR][CH] step size, step size times input
+  float* s_d = reinterpret_cast<float*>(s_q + TR * CH); // [TR][LD] D times input; then the result
+  float* s_g = s_d + TR * LD;                           // silu(z)
+  float* s_b = s_g + TR * LD;                           // [TR][SP]
   float* s_c = s_b + TR * SP;
-  const int tid = threadIdx.x, l = tid & 3, ci = tid >> 2, c0 = blockIdx.x * CH, c = c0 + ci, seq = blockIdx.y;
+  const int tid = threadIdx.x, l = tid & 3, ci = tid >> 2, c0 = blockIdx.x * CH, seq = blockIdx.y;
   const int q0 = p.rows.q_start ? p.rows.q_start[seq] : seq, n = p.rows.q_len ? p.rows.q_len[seq] : 1;
   const int nq = p.states / 4;
-  const bool live = c < p.inner, fresh = p.rows.pos[q0] == 0;
+  const bool fresh = p.rows.pos[q0] == 0;
   for (int i = tid; i < TR * SP * 2; i += NT) s_b[i] = 0.f;
-  float4 A[QPL], S[QPL];
-  float* st = p.state + ((size_t)(p.rows.slot ? p.rows.slot[seq] : seq) * p.inner + (live ? c : 0)) * p.states;
+  float4 A[CPL][QPL], S[CPL][QPL];
+  float* st[CPL];
 #pragma unroll
-  for (int q = 0; q < QPL; ++q) {
-    const bool in = live && l + 4 * q < nq;
-    A[q] = in ? reinterpret_cast<const float4*>(p.a2 + (size_t)c * p.states)[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
-    S[q] = in && !fresh ? reinterpret_cast<const float4*>(st)[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int h = 0; h < CPL; ++h) {
+    const int c = c0 + ci + h * (CH / CPL);
+    const bool live = c < p.inner;
+    st[h] = p.state + ((size_t)(p.rows.slot ? p.rows.slot[seq] : seq) * p.inner + (live ? c : 0)) * p.states;
+#pragma unroll
+    for (int q = 0; q < QPL; ++q) {
+      const bool in = live && l + 4 * q < nq;
+      A[h][q] = in ? reinterpret_cast<const float4*>(p.a2 + (size_t)c * p.states)[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
+      S[h][q] = in && !fresh ? reinterpret_cast<const float4*>(st[h])[l + 4 * q] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
   }
-  // the thread's piece of a tile
+  // the thread's pieces of a tile: rows lr + u * TR / CPL
   const int lr = tid / (CH / 8), lc = (tid % (CH / 8)) * 8;
   const bool in_c = c0 + lc < p.inner;
   float bias[8], D[8];
@@ -387,35 +393,42 @@ __global__ void __launch_bounds__(CH * 4) mamba_scan_kernel(const RfMamba1 p) {
   const T* zp = reinterpret_cast<const T*>(p.z) + (size_t)q0 * p.ldz + c0 + lc;
   const T* dp = reinterpret_cast<const T*>(p.dt) + (size_t)q0 * p.ld_dt + c0 + lc;
   const T* bp = reinterpret_cast<const T*>(p.bc) + (size_t)q0 * p.ld_bc + p.rank;
-  Vec8<T> vx, vz, vd;
+  Vec8<T> vx[CPL], vz[CPL], vd[CPL];
   auto fetch = [&](int t0) {
-    if (t0 + lr < n && in_c) {
-      vx = *reinterpret_cast<const Vec8<T>*>(xp + (size_t)(t0 + lr) * p.ldx);
-      vz = *reinterpret_cast<const Vec8<T>*>(zp + (size_t)(t0 + lr) * p.ldz);
-      vd = *reinterpret_cast<const Vec8<T>*>(dp + (size_t)(t0 + lr) * p.ld_dt);
+#pragma unroll
+    for (int u = 0; u < CPL; ++u) {
+      const int t = t0 + lr + u * (TR / CPL);
+      if (t < n && in_c) {
+        vx[u] = *reinterpret_cast<const Vec8<T>*>(xp + (size_t)t * p.ldx);
+        vz[u] = *reinterpret_cast<const Vec8<T>*>(zp + (size_t)t * p.ldz);
+        vd[u] = *reinterpret_cast<const Vec8<T>*>(dp + (size_t)t * p.ld_dt);
+      }
     }
   };
   fetch(0);
   for (int t0 = 0; t0 < n; t0 += TR) {
     const int nr = min(TR, n - t0);
     __syncthreads();                       // the previous tile's results have left
-    {
-      float dt[8], dx[8], dd[8], g[8];
-      zero8(dt); zero8(dx); zero8(dd); zero8(g);
-      if (lr < nr && in_c) {
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const float2 x2 = Num<T>::to_f2(vx.v[j]), z2 = Num<T>::to_f2(vz.v[j]), d2 = Num<T>::to_f2(vd.v[j]);
-          dt[2 * j] = softplus_t<T>(d2.x + bias[2 * j]); dt[2 * j + 1] = softplus_t<T>(d2.y + bias[2 * j + 1]);
-          dx[2 * j] = dt[2 * j] * x2.x; dx[2 * j + 1] = dt[2 * j + 1] * x2.y;
+    for (int u = 0; u < CPL; ++u) {
+      const int r = lr + u * (TR / CPL);
+      float dd[8], g[8];
+      zero8(dd); zero8(g);
+      const bool in = r < nr && in_c;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        float4 dq = make_float4(0.f, 0.f, 0.f, 0.f);   // rows behind the end: step size 0 leaves the state as it is
+        if (in) {
+          const float2 x2 = Num<T>::to_f2(vx[u].v[j]), z2 = Num<T>::to_f2(vz[u].v[j]), d2 = Num<T>::to_f2(vd[u].v[j]);
+          dq.x = softplus_t<T>(d2.x + bias[2 * j]); dq.y = dq.x * x2.x;
+          dq.z = softplus_t<T>(d2.y + bias[2 * j + 1]); dq.w = dq.z * x2.y;
           dd[2 * j] = D[2 * j] * x2.x; dd[2 * j + 1] = D[2 * j + 1] * x2.y;
           g[2 * j] = silu_t<T>(z2.x); g[2 * j + 1] = silu_t<T>(z2.y);
         }
+        *reinterpret_cast<float4*>(s_q + r * CH + lc + 2 * j) = dq;
       }
-      store8(s_dt + lr * LD + lc, dt);     // rows behind the end: step size 0 leaves the state as it is
-      store8(s_dx + lr * LD + lc, dx);
-      store8(s_d + lr * LD + lc, dd);
-      store8(s_g + lr * LD + lc, g);
+      store8(s_d + r * LD + lc, dd);
+      store8(s_g + r * LD + lc, g);
     }
     for (int i = tid; i < TR * (p.states / 4); i += NT) {
       const int r = i / (p.states / 4), k = (i % (p.states / 4)) * 8;
@@ -428,39 +441,56 @@ __global__ void __launch_bounds__(CH * 4) mamba_scan_kernel(const RfMamba1 p) {
     __syncthreads();
     if (t0 + TR < n) fetch(t0 + TR);
     for (int t = 0; t < nr; t += 4) {
-      float v[4];
+      float v[CPL][4];
 #pragma unroll
       for (int u = 0; u < 4; ++u) {
-        const float dt = s_dt[(t + u) * LD + ci], dx = s_dx[(t + u) * LD + ci];
-        v[u] = 0.f;
+        float2 dq[CPL];
+#pragma unroll
+        for (int h = 0; h < CPL; ++h) {
+          dq[h] = s_q[(t + u) * CH + ci + h * (CH / CPL)];
+          v[h][u] = 0.f;
+        }
 #pragma unroll
         for (int q = 0; q < QPL; ++q) {
           const float4 B = *reinterpret_cast<const float4*>(s_b + (t + u) * SP + (l + 4 * q) * 4), C = *reinterpret_cast<const float4*>(s_c + (t + u) * SP + (l + 4 * q) * 4);
-          S[q].x = S[q].x * exp2_t<T>(dt * A[q].x) + dx * B.x; v[u] += S[q].x * C.x;
-          S[q].y = S[q].y * exp2_t<T>(dt * A[q].y) + dx * B.y; v[u] += S[q].y * C.y;
-          S[q].z = S[q].z * exp2_t<T>(dt * A[q].z) + dx * B.z; v[u] += S[q].z * C.z;
-          S[q].w = S[q].w * exp2_t<T>(dt * A[q].w) + dx * B.w; v[u] += S[q].w * C.w;
+#pragma unroll
+          for (int h = 0; h < CPL; ++h) {
+            float4& s = S[h][q];
+            const float dt = dq[h].x, dx = dq[h].y;
+            s.x = s.x * exp2_t<T>(dt * A[h][q].x) + dx * B.x; v[h][u] += s.x * C.x;
+            s.y = s.y * exp2_t<T>(dt * A[h][q].y) + dx * B.y; v[h][u] += s.y * C.y;
+            s.z = s.z * exp2_t<T>(dt * A[h][q].z) + dx * B.z; v[h][u] += s.z * C.z;
+            s.w = s.w * exp2_t<T>(dt * A[h][q].w) + dx * B.w; v[h][u] += s.w * C.w;
+          }
         }
       }
       // lane l ends with the sum of row t + l: swap halves with the lane two away, then with the neighbour
       const bool hi = l & 2, odd = l & 1;
-      const float a0 = __shfl_xor_sync(0xffffffffu, hi ? v[0] : v[2], 2), a1 = __shfl_xor_sync(0xffffffffu, hi ? v[1] : v[3], 2);
-      const float w0 = (hi ? v[2] : v[0]) + a0, w1 = (hi ? v[3] : v[1]) + a1;
-      const float y = (odd ? w1 : w0) + __shfl_xor_sync(0xffffffffu, odd ? w0 : w1, 1);
-      const int at = (t + l) * LD + ci;
-      s_dx[at] = (y + s_d[at]) * s_g[at];
+#pragma unroll
+      for (int h = 0; h < CPL; ++h) {
+        const float a0 = __shfl_xor_sync(0xffffffffu, hi ? v[h][0] : v[h][2], 2), a1 = __shfl_xor_sync(0xffffffffu, hi ? v[h][1] : v[h][3], 2);
+        const float w0 = (hi ? v[h][2] : v[h][0]) + a0, w1 = (hi ? v[h][3] : v[h][1]) + a1;
+        const float y = (odd ? w1 : w0) + __shfl_xor_sync(0xffffffffu, odd ? w0 : w1, 1);
+        const int at = (t + l) * LD + ci + h * (CH / CPL);
+        s_d[at] = (y + s_d[at]) * s_g[at];
+      }
     }
     __syncthreads();
-    if (lr < nr && in_c) {
+#pragma unroll
+    for (int u = 0; u < CPL; ++u) {
+      const int r = lr + u * (TR / CPL);
+      if (r >= nr || !in_c) continue;
       float f[8];
-      load8(s_dx + lr * LD + lc, f);
-      store8(reinterpret_cast<T*>(p.out) + (size_t)(q0 + t0 + lr) * p.ldo + c0 + lc, f);
+      load8(s_d + r * LD + lc, f);
+      store8(reinterpret_cast<T*>(p.out) + (size_t)(q0 + t0 + r) * p.ldo + c0 + lc, f);
     }
   }
-  if (live) {
+#pragma unroll
+  for (int h = 0; h < CPL; ++h) {
+    if (c0 + ci + h * (CH / CPL) >= p.inner) continue;
 #pragma unroll
     for (int q = 0; q < QPL; ++q)
-      if (l + 4 * q < nq) reinterpret_cast<float4*>(st)[l + 4 * q] = S[q];
+      if (l + 4 * q < nq) reinterpret_cast<float4*>(st[h])[l + 4 * q] = S[h][q];
   }
 }
 
@@ -494,21 +524,23 @@ static int launch_recurrent(const RfMamba1* a, cudaStream_t s) {
   return RF_OK;
 }
 
-template <typename T, int QPL>
-static int launch_scan(const RfMamba1* a, cudaStream_t s) {
-  const int seqs = a->rows.num_seqs;
-  const size_t per = (size_t)kScanRows * 32 * QPL * sizeof(float);
-  if (ceil_div(a->inner, 64) * seqs >= 4 * sm_count()) {
-    const size_t smem = (size_t)kScanRows * (64 + 8) * 4 * sizeof(float) + per;
-    RF_ALLOW_SMEM_PER_DEVICE((mamba_scan_kernel<T, 64, QPL>), 128 * 1024);
-    RF_CUDA_CHECK(::rf::launch_k(mamba_scan_kernel<T, 64, QPL>, dim3(ceil_div(a->inner, 64), seqs), dim3(256), smem, s, 1, *a));
-  } else {
-    const size_t smem = (size_t)kScanRows * (32 + 8) * 4 * sizeof(float) + per;
-    RF_ALLOW_SMEM_PER_DEVICE((mamba_scan_kernel<T, 32, QPL>), 128 * 1024);
-    RF_CUDA_CHECK(::rf::launch_k(mamba_scan_kernel<T, 32, QPL>, dim3(ceil_div(a->inner, 32), seqs), dim3(128), smem, s, 1, *a));
-  }
+template <typename T, int CH, int QPL, int CPL>
+static int launch_scan_t(const RfMamba1* a, cudaStream_t s) {
+  const size_t smem = (size_t)kScanRows * (2 * CH + 2 * (CH + 8) + 32 * QPL) * sizeof(float);
+  RF_ALLOW_SMEM_PER_DEVICE((mamba_scan_kernel<T, CH, QPL, CPL>), 128 * 1024);
+  RF_CUDA_CHECK(::rf::launch_k(mamba_scan_kernel<T, CH, QPL, CPL>, dim3(ceil_div(a->inner, CH), a->rows.num_seqs), dim3(CH * 4 / CPL), smem, s, 1, *a));
   ::rf::count_launch();
   return RF_OK;
+}
+
+template <typename T, int QPL>
+static int launch_scan(const RfMamba1* a, cudaStream_t s) {
+  constexpr int CPL = QPL <= 2 ? 2 : 1;              // wider states leave no registers for a second channel
+  const int seqs = a->rows.num_seqs;
+  if (ceil_div(a->inner, 64) * seqs >= 4 * sm_count()) return launch_scan_t<T, 64, QPL, CPL>(a, s);
+  // few sequences: latency counts, so more warps with one channel per four lanes
+  if (ceil_div(a->inner, 32) * seqs >= 3 * sm_count()) return launch_scan_t<T, 32, QPL, CPL>(a, s);
+  return launch_scan_t<T, 32, QPL, 1>(a, s);
 }
 
 }  // namespace rf
