@@ -26,7 +26,7 @@ HERE = Path(__file__).resolve().parent
 DEFAULT_CONFIG = HERE / "configs" / "qwen3_0_6b_full.toml"
 
 TARGETS = {name: f"{name}.py" for name in
-           ("causal_lm", "dinov3", "hy_embodied", "pi05", "qwen3_5_text", "qwen3_vl", "rhinovla", "vabarax", "wall_oss")}
+           ("causal_lm", "dinov3", "hy_embodied", "pi05", "qwen3_5_text", "qwen3_vl", "rhinovla", "vabarax", "wall_oss", "zulopel")}
 _PREFILL = ("chunk_size", "padding_rows", "padding_budget")
 EXECUTION_SUPPORT = {
     "causal_lm": {"prefill": _PREFILL},
@@ -37,6 +37,7 @@ EXECUTION_SUPPORT = {
     "qwen3_vl": {"prefill": _PREFILL, "vision": ("chunk_size",)},
     "rhinovla": None,
     "vabarax": {"prefill": _PREFILL},
+    "zulopel": {"prefill": _PREFILL},
     "wall_oss": {"prefill": _PREFILL, "vision": ("chunk_size",), "action": ("chunk_size",)},
 }
 DENIED_ENV = {"RPU_KERNEL_LIB_PATH", "LKN_MAX_BATCH_ENTRIES", "LKN_KD_BUF_MB", "LKN_INSTR_BUF_MB"}

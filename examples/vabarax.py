@@ -34,8 +34,8 @@ def load_config(path) -> dict:
     return config
 
 
-def main() -> int:
-    args = parse_args("vabarax.toml", __doc__)
+def main(default: str = "vabarax.toml", doc=__doc__) -> int:
+    args = parse_args(default, doc)
     config = load_config(args.config)
     if args.check_config:
         return ok(args.config, require_model(config))

@@ -129,6 +129,17 @@ def test_oracle_is_causal_and_respects_its_chunks():
     assert [oracle.first_visible(i, 4) for i in (0, 3, 4, 7, 8)] == [0, 0, 4, 4, 8]
 
 
+def test_example_configuration_is_checked():
+    import importlib.util
+    from pathlib import Path
+    root = Path(__file__).resolve().parents[1]
+    spec = importlib.util.spec_from_file_location("zulopel_example", root / "examples" / "zulopel.py")
+    mod = importlib.util.module_from_spec(spec)
+    spec.loader.exec_module(mod)
+    cfg = mod.load_config(root / "examples" / "configs" / "zulopel.toml")
+    assert cfg["model"]["checkpoint"] == "models/zulopel" and cfg["generation"]["slots"] == 2
+
+
 def test_groups_exclude_experts_even_when_every_choice_score_is_negative():
     s, corr = torch.tensor([0.4, 0.1, 0.3, 0.2]), torch.tensor([-1.0, -0.5, -2.0, -0.1])       # choice scores -0.6 -0.4 | -1.7 0.1
     assert oracle.choose(s, corr, 2, {"count": 2, "keep": 1}) == [3, 2]
