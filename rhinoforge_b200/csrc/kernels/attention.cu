@@ -564,7 +564,7 @@ struct DecodeSplitPlan {
 };
 static DecodeSplitPlan plan_decode_split(int num_seqs, int Hq, int Hkv, int hd, int max_kv_len, bool allow_split) {
   const int max_pages = std::max(1, (max_kv_len + 15) / 16);
-  const int ctas = num_seqs * Hkv * ceil_div(Hq / Hkv, 16);
+  const int ctas = num_seqs * Hkv;
   int splits = 1;
   // RF_ATTN_DECODE_CTAS_PER_SM (default 2; 1 for heads of 256): CTAs per SM the split aims at; RF_ATTN_DECODE_MIN_PAGES (default 8): fewest
   // pages a split may cover
