@@ -129,7 +129,7 @@ def expected(q, k, v, i, scale, sink, chunk, gate):
     return torch.stack(o) * torch.sigmoid(gate)
 
 
-SHAPES = [(8, 1, 64, 64, 64), (4, 4, 40, 64, 64), (20, 1, 128, 96, 128), (34, 2, 64, 64, 64), (4, 2, 256, 130, 256)]
+SHAPES = [(6, 1, 64, 64, 64), (4, 4, 40, 64, 64), (20, 1, 128, 96, 128), (34, 2, 64, 64, 64), (4, 2, 256, 130, 256)]
 
 
 @pytest.mark.parametrize("form", ["f32", "rows-bf16", "tensor", "prefill"])
@@ -167,10 +167,10 @@ def test_chunked_attention_with_sinks_and_gates(form, chunk, heads, kv, dim, vdi
 
 
 @pytest.mark.parametrize("form", ["f32", "tensor", "prefill"])
-@pytest.mark.parametrize("at", [0, 15, 16, 31, 63, 64, 95, 96])
+@pytest.mark.parametrize("at", [0, 15, 16, 31, 63, 64, 79, 80])
 def test_one_key_that_stands_out_is_seen_inside_its_chunk_only(form, at):
     """A key that every query likes, at page and chunk borders: the result is its value as long as it is visible."""
-    dtype, chunk, n = F32 if form == "f32" else BF16, 96, 130
+    dtype, chunk, n = F32 if form == "f32" else BF16, 80, 130
     pt, rnd = page_table(1, 9), gen(7)
     k, v, kp, vp = cached(rnd, [0], [n], 1, 64, 64, 64, dtype, pt, 9)
     like = torch.ones(64, dtype=torch.float64)
@@ -301,7 +301,7 @@ def test_scan_step_sizes_from_tiny_to_large():
 
 
 # ------------------------------------------------------------------------------------------------ experts
-ROUTERS = [(12, 3, 3, 2), (8, 1, 8, 1), (5, 5, 1, 1), (64, 6, 8, 3), (160, 8, 4, 4), (256, 32, 16, 9), (1, 1, 1, 1), (200, 4, 100, 2)]
+ROUTERS = [(15, 4, 5, 2), (8, 1, 8, 1), (5, 5, 1, 1), (64, 6, 8, 3), (160, 8, 4, 4), (256, 32, 16, 9), (1, 1, 1, 1), (200, 4, 100, 2)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -396,7 +396,7 @@ def test_expert_gemms_of_few_rows(dtype, E, k, ff, shared, H, T, tile):
 def test_invalid_sizes_are_refused_on_the_host():
     from rhinoforge_b200.api.errors import RPUBackendError
     x, w = torch.zeros(2, 64, device="cuda", dtype=BF16), torch.zeros(12, 64, device="cuda", dtype=BF16)
-    for kw in (dict(k=13), dict(k=3, groups=5), dict(k=5, groups=3, keep=1), dict(k=2, groups=3, keep=4)):
+    for kw in (dict(k=13), dict(k=4, groups=5), dict(k=5, groups=3, keep=1), dict(k=2, groups=3, keep=4)):
         with pytest.raises(RPUBackendError):
             K().moe_router(x, w, **kw)
     pool, pt = torch.zeros(1, 1, 16, 24, device="cuda"), page_table(1, 1)
