@@ -47,6 +47,7 @@ class RfGemm(C.Structure):
         ("ss_out", C.c_void_p), ("ss_in", C.c_void_p), ("ss_ld", C.c_int32), ("ss_dim", C.c_int32),
         ("ss_eps", C.c_float), ("streaming_only", C.c_int32),
         ("mul", C.c_void_p), ("mul_row", C.c_void_p), ("mul_ld", C.c_int64),
+        ("act_limit", C.c_float), ("act_alpha", C.c_float),
     ]
 
 
@@ -68,6 +69,7 @@ class RfMoeGroupedGemm(C.Structure):
         ("max_rows", C.c_int32), ("N", C.c_int32), ("K", C.c_int32), ("dual", C.c_int32), ("act", C.c_int32),
         ("bank_section_row_tiles", C.c_int32), ("bank_kb_total", C.c_int32),
         ("rt_per_expert", C.c_int32), ("kb_per_expert", C.c_int32), ("dtype", C.c_int32), ("status", C.c_void_p),
+        ("act_limit", C.c_float), ("act_alpha", C.c_float),
     ]
 
 
@@ -107,6 +109,7 @@ class RfAttn(C.Structure):
         ("ws", C.c_void_p), ("ws_bytes", C.c_uint64),
         ("status", C.c_void_p), ("dtype", C.c_int32),
         ("slot", C.c_void_p), ("chunk", C.c_int32), ("sink", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_int64),
+        ("gate_by_head", C.c_int32), ("keep_first", C.c_int32), ("slopes", C.c_void_p),
         ("seq_of_row", C.c_void_p), ("pos", C.c_void_p),
     ]
 
@@ -196,7 +199,8 @@ class RfStreamNorm(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("x", "table", "ids", "row_idx", "y", "y_norm_w", "x_out", "x_cast", "norm_w", "out",
                                           "shift", "shift_state")] + [("rows", RfRows)] + \
                [("n_rows", C.c_int32), ("H", C.c_int32), ("dim", C.c_int32), ("eps", C.c_float), ("dtype", C.c_int32),
-                ("embed_scale", C.c_float), ("y_slots", C.c_void_p), ("y_picks", C.c_int32)]
+                ("embed_scale", C.c_float), ("y_slots", C.c_void_p), ("y_picks", C.c_int32), ("y_mult", C.c_float),
+                ("table2", C.c_void_p), ("last_token", C.c_void_p), ("mul_prev", C.c_int64), ("mul_cur", C.c_int64), ("buckets", C.c_int32)]
 
 
 class RfHeadLinear(C.Structure):
@@ -222,12 +226,13 @@ class RfMixedConfig(C.Structure):
                                          "max_seq_len", "side_dim")] + \
                [("side_ld", C.c_int64), ("eps", C.c_float), ("weights_packed", C.c_int32), ("long_min", C.c_int32)] + \
                [(n, C.c_void_p) for n in ("embed", "side_table", "final_norm", "w_lm")] + \
-               [("embed_scale", C.c_float), ("norm_after", C.c_int32)]
+               [("embed_scale", C.c_float), ("norm_after", C.c_int32), ("residual_mult", C.c_float), ("logit_softcap", C.c_float),
+                ("pair_table", C.c_void_p), ("pair_mul_prev", C.c_int64), ("pair_mul_cur", C.c_int64), ("pair_buckets", C.c_int32)]
 
 
 class RfMixedState(C.Structure):
     _fields_ = [("latent_pool", C.c_void_p), ("k_pool", C.c_void_p), ("v_pool", C.c_void_p), ("pool_pages", C.c_int64),
-                ("rec_state", C.c_void_p), ("conv_state", C.c_void_p), ("shift_state", C.c_void_p)]
+                ("rec_state", C.c_void_p), ("conv_state", C.c_void_p), ("shift_state", C.c_void_p), ("last_token", C.c_void_p)]
 
 
 class RfMixedLayer(C.Structure):
@@ -238,18 +243,20 @@ class RfMixedLayer(C.Structure):
                                           "side_norm")] + \
                [(n, C.c_int32) for n in ("kv_heads", "dim_true", "tensor_core", "chunk", "gated", "rot_dims", "v_role")] + \
                [("v_lambda", C.c_float)] + [(n, C.c_void_p) for n in ("cos", "sin", "q_norm", "k_norm", "sink")] + \
+               [(n, C.c_int32) for n in ("keep_first", "norm_all", "gate_by_head", "conv_taps")] + [("slopes", C.c_void_p)] + \
                [(n, C.c_int32) for n in ("inner", "states", "dt_rank", "taps")] + \
                [(n, C.c_void_p) for n in ("conv_w", "conv_b", "a2", "d_skip", "dt_bias", "w_x", "w_dt", "w_dt_rows")] + \
                [(n, C.c_int32) for n in ("experts", "top", "groups", "keep", "score_fn", "norm_topk", "shared_inter", "bank_inter")] + \
                [("route_scale", C.c_float)] + [(n, C.c_void_p) for n in ("router", "correction", "shared_up", "shared_down")] + \
-               [("st", RfMixedState)]
+               [(n, C.c_float) for n in ("act_limit", "act_alpha", "shared_limit")] + [("shared_gate", C.c_int32), ("st", RfMixedState)]
 
 
 class RfQkvInsert(C.Structure):
     _fields_ = [("qkv", C.c_void_p), ("ld", C.c_int64), ("k_off", C.c_int32), ("v_off", C.c_int32)] + \
                [(n, C.c_void_p) for n in ("q_norm", "k_norm", "cos", "sin", "v_first", "k_pool", "v_pool")] + [("rows", RfRows)] + \
                [(n, C.c_int32) for n in ("n_rows", "heads", "kv_heads", "hd", "dim", "vdim", "rot_dims", "v_role")] + \
-               [("v_lambda", C.c_float), ("eps", C.c_float), ("dtype", C.c_int32)]
+               [("v_lambda", C.c_float), ("eps", C.c_float), ("dtype", C.c_int32), ("norm_all", C.c_int32), ("conv_w", C.c_void_p),
+                ("conv_state", C.c_void_p), ("q_out", C.c_void_p), ("taps", C.c_int32), ("max_q_len", C.c_int32)]
 
 
 class RfConvSilu(C.Structure):
@@ -270,7 +277,7 @@ class RfMoeRouter(C.Structure):
                                           "token_of_slot", "slot_w")] + \
                [(n, C.c_int32) for n in ("rows", "experts", "width", "k", "groups", "keep", "score_fn", "norm_topk")] + \
                [("scale", C.c_float)] + [(n, C.c_int32) for n in ("tile_rows", "slot_ld", "has_shared", "shared_tiles", "scatter", "dtype")] + \
-               [("logits", C.c_void_p)]
+               [("logits", C.c_void_p), ("shared_gate", C.c_int32)]
 
 
 class RfMoeExperts(C.Structure):
@@ -278,7 +285,8 @@ class RfMoeExperts(C.Structure):
                [(n, C.c_void_p) for n in ("tiles", "token_of_slot", "slot_w")] + \
                [(n, C.c_int32) for n in ("max_tiles", "experts", "n", "k", "shared_n", "shared_k", "dual", "tile_rows",
                                          "bank_section_row_tiles", "bank_kb_total", "rt_per_expert", "kb_per_expert",
-                                         "shared_section_row_tiles", "shared_kb_total", "dtype")]
+                                         "shared_section_row_tiles", "shared_kb_total", "dtype", "act")] + \
+               [(n, C.c_float) for n in ("act_limit", "act_alpha", "shared_limit")]
 
 
 class RfMixedForward(C.Structure):

@@ -12,6 +12,7 @@ BUILTIN_ADAPTERS = (
     ("Qwen3VLForConditionalGeneration", "rhinoforge_b200.adapters.qwen3_vl", "Qwen3VLAdapter"),
     ("Vabarax", "rhinoforge_b200.adapters.vabarax", "VabaraxAdapter"),
     ("Zulopel", "rhinoforge_b200.adapters.zulopel", "ZulopelAdapter"),
+    ("Kuzupel", "rhinoforge_b200.adapters.kuzupel", "KuzupelAdapter"),
 )
 
 __all__ = ["BUILTIN_ADAPTERS"]

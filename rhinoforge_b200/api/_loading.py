@@ -21,6 +21,7 @@ _ROUTES = {
     "Qwen3ForCausalLM": "use RPUModelForCausalLM.from_pretrained(...) and .to('rpu')",
     "Vabarax": "use RPUModelForCausalLM.from_pretrained(..., device='rpu')",
     "Zulopel": "use RPUModelForCausalLM.from_pretrained(..., device='rpu')",
+    "Kuzupel": "use RPUModelForCausalLM.from_pretrained(..., device='rpu')",
 }
 
 

@@ -91,6 +91,19 @@ __device__ __forceinline__ float relu2_f(float x) {
   return r * r;
 }
 
+// Gated unit with clipped operands: g sigmoid(alpha g) (u + 1) for g at most `limit` and u within +-limit.
+struct ActArgs { float limit, alpha; };
+__device__ __forceinline__ float clipped_glu_f(float g, float u, ActArgs a) {
+  g = fminf(g, a.limit);
+  u = fminf(fmaxf(u, -a.limit), a.limit);
+  return __fdividef(g, 1.0f + __expf(-a.alpha * g)) * (u + 1.f);
+}
+// limit * tanh(x / limit)
+__device__ __forceinline__ float soft_cap_f(float x, float limit) {
+  const float t = __fdividef(2.f, 1.f + __expf(__fdividef(-2.f * x, limit)));      // 1 + tanh
+  return limit * (t - 1.f);
+}
+
 enum Act : int32_t {
   kActNone = 0,
   kActSiluMul = 1,      // dual accumulator: silu(g) * u
@@ -99,9 +112,12 @@ enum Act : int32_t {
   kActGeluErf = 4,
   kActSilu = 5,
   kActRelu2 = 6,        // relu(g)^2
+  kActClippedGlu = 7,   // dual accumulator: clipped_glu_f (ActArgs)
+  kActSoftCap = 8,      // soft_cap_f (ActArgs.limit)
 };
+__host__ __device__ inline bool act_is_dual(int act) { return act == kActSiluMul || act == kActGeluTanhMul || act == kActClippedGlu; }
 
-__device__ __forceinline__ float apply_act(int act, float g, float u) {
+__device__ __forceinline__ float apply_act(int act, float g, float u, ActArgs a) {
   switch (act) {
     case kActSiluMul: return silu_f(g) * u;
     case kActGeluTanhMul: return gelu_tanh_f(g) * u;
@@ -109,6 +125,8 @@ __device__ __forceinline__ float apply_act(int act, float g, float u) {
     case kActGeluErf: return gelu_erf_f(g);
     case kActSilu: return silu_f(g);
     case kActRelu2: return relu2_f(g);
+    case kActClippedGlu: return clipped_glu_f(g, u, a);
+    case kActSoftCap: return soft_cap_f(g, a.limit);
     default: return g;
   }
 }
@@ -218,7 +236,7 @@ template <> __device__ __forceinline__ uint4 widen_e2m1x8<__nv_bfloat16>(uint32_
 
 // The same on N values with the activation switch outside the element loop.
 template <int N>
-__device__ __forceinline__ void apply_act_n(int act, const float (&g)[N], const float (&u)[N], float (&v)[N]) {
+__device__ __forceinline__ void apply_act_n(int act, const float (&g)[N], const float (&u)[N], float (&v)[N], ActArgs a) {
   switch (act) {
     case kActSiluMul:
 #pragma unroll
@@ -243,6 +261,14 @@ __device__ __forceinline__ void apply_act_n(int act, const float (&g)[N], const 
     case kActRelu2:
 #pragma unroll
       for (int j = 0; j < N; ++j) v[j] = relu2_f(g[j]);
+      break;
+    case kActClippedGlu:
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[j] = clipped_glu_f(g[j], u[j], a);
+      break;
+    case kActSoftCap:
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[j] = soft_cap_f(g[j], a.limit);
       break;
     default:
 #pragma unroll

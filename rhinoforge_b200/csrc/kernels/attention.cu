@@ -105,11 +105,15 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   const int owner = p.pos && p.seq_of_row ? p.seq_of_row[seq] : seq;
   const int pt_row = p.slot ? p.slot[owner] : owner;
   const int kvlen = p.pos ? p.pos[seq] + 1 : p.kv_len[seq];
-  const int kvlo = p.chunk > 0 && kvlen > 0 ? (kvlen - 1) / p.chunk * p.chunk : 0;
-  const int total_pages = (kvlen + 15) >> 4;
-  const int pg_begin = (kvlo >> 4) + split * p.pages_per_split;
+  int kvlo = p.chunk > 0 && kvlen > 0 ? (kvlen - 1) / p.chunk * p.chunk : 0;
+  if (p.window > 0) kvlo = max(kvlo, kvlen - p.window);
+  // pages in the order they are read: the ones of the kept first positions, then from the first visible position on
+  const int keep_pages = min((p.keep_first + 15) >> 4, kvlo >> 4), skipped = (kvlo >> 4) - keep_pages;
+  const int total_pages = ((kvlen + 15) >> 4) - skipped;
+  const int pg_begin = split * p.pages_per_split;
   const int pg_end = min(total_pages, pg_begin + p.pages_per_split);
   const int npg = max(0, pg_end - pg_begin);
+  auto page_at = [&](int i) { return i < keep_pages ? i : i + skipped; };
   const int iters = (npg + 3) >> 2;
   const int G = min(p.G - g_first, 16);          // query heads of this CTA
   const int head0 = kvh * p.G + g_first;
@@ -144,7 +148,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
         const int nvalid = min(4, npg - it * 4);
         mbar_arrive_expect_tx(&ctl->full[s], (uint32_t)(nvalid * kPageBytes));
         for (int w = 0; w < nvalid; ++w) {
-          const int pg = pg_begin + it * 4 + w;
+          const int pg = page_at(pg_begin + it * 4 + w);
           int row, col0;
           if (p.paged) {
             const int page_id = p.page_table[(size_t)pt_row * p.pt_stride + pg];
@@ -164,6 +168,11 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   } else {
     // query fragments of this kv head's group: row g = lane/4 (and g + 8)
     uint32_t qf[HD / 16][4];
+    float fall0 = 0.f, fall1 = 0.f;                // what the two rows' scores lose per token of distance
+    if (p.slopes) {
+      if ((lane >> 2) < G) fall0 = p.slopes[head0 + (lane >> 2)] * kLog2e;
+      if ((lane >> 2) + 8 < G) fall1 = p.slopes[head0 + (lane >> 2) + 8] * kLog2e;
+    }
     {
       const int g0 = lane >> 2, g1 = g0 + 8;
       const T* qbase = reinterpret_cast<const T*>(p.q) + (size_t)seq * p.ldq + (size_t)head0 * HD;
@@ -191,13 +200,14 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
         float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
         for (int ks = 0; ks < HD / 16; ++ks) qk_step<T>(s0, s1, qf[ks], kbase, ks, lane);
-        const int tok0 = (pg_begin + pgl) * 16 + (lane & 3) * 2;
+        const int tok0 = page_at(pg_begin + pgl) * 16 + (lane & 3) * 2;
         float x[2][4];
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int t0 = tok0 + (e & 1), t1 = tok0 + 8 + (e & 1);
-          x[0][e] = t0 < kvlen && t0 >= kvlo ? s0[e] * p.scale_log2 : -INFINITY;
-          x[1][e] = t1 < kvlen && t1 >= kvlo ? s1[e] * p.scale_log2 : -INFINITY;
+          const float fall = e < 2 ? fall0 : fall1;
+          x[0][e] = t0 < kvlen && (t0 >= kvlo || t0 < p.keep_first) ? s0[e] * p.scale_log2 - fall * (float)(kvlen - 1 - t0) : -INFINITY;
+          x[1][e] = t1 < kvlen && (t1 >= kvlo || t1 < p.keep_first) ? s1[e] * p.scale_log2 - fall * (float)(kvlen - 1 - t1) : -INFINITY;
         }
         const float mx0 = quad_max(fmaxf(fmaxf(x[0][0], x[0][1]), fmaxf(x[1][0], x[1][1])));
         const float mx1 = quad_max(fmaxf(fmaxf(x[0][2], x[0][3]), fmaxf(x[1][2], x[1][3])));
@@ -281,7 +291,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     float val = den > 0.f ? num / den : 0.f;
     if (p.splits == 1) {
       const size_t col_of_row = (size_t)head * HD + col;
-      if (p.gate) val *= sigmoid_fast(Num<T>::to_f(reinterpret_cast<const T*>(p.gate)[(size_t)seq * p.ld_gate + col_of_row]));
+      if (p.gate) val *= sigmoid_fast(Num<T>::to_f(reinterpret_cast<const T*>(p.gate)[(size_t)seq * p.ld_gate + (p.gate_by_head ? head : col_of_row)]));
       reinterpret_cast<T*>(p.out)[(size_t)seq * p.ldo + col_of_row] = Num<T>::from_f(val);
     } else {
       const size_t base = ((size_t)seq * p.Hq + head) * p.splits + split;
@@ -295,7 +305,7 @@ template <typename T>
 __global__ void attn_decode_combine_kernel(const float* __restrict__ ws_o,
                                            const float* __restrict__ ws_lse, T* __restrict__ out,
                                            int64_t ldo, int Hq, int hd, int splits, const float* __restrict__ sink,
-                                           const T* __restrict__ gate, int64_t ldg) {
+                                           const T* __restrict__ gate, int64_t ldg, int gate_by_head) {
   pdl_prologue();
   const int head = blockIdx.x, seq = blockIdx.y;
   const size_t base = ((size_t)seq * Hq + head) * splits;
@@ -312,7 +322,7 @@ __global__ void attn_decode_combine_kernel(const float* __restrict__ ws_o,
       if (sink) den += exp2f(sink[head] * kLog2e - M);
     }
     float val = den > 0.f ? num / den : 0.f;
-    if (gate) val *= sigmoid_fast(Num<T>::to_f(gate[(size_t)seq * ldg + (size_t)head * hd + col]));
+    if (gate) val *= sigmoid_fast(Num<T>::to_f(gate[(size_t)seq * ldg + (gate_by_head ? head : head * hd + col)]));
     out[(size_t)seq * ldo + (size_t)head * hd + col] = Num<T>::from_f(val);
   }
 }
@@ -534,8 +544,11 @@ static int fill_params(const RfAttn* a, AttnParams* p) {
   p->seg_q = a->seg_q; p->seg_k = a->seg_k;
   const float scale = a->scale > 0.f ? a->scale : 1.0f / sqrtf((float)a->hd);
   p->scale_log2 = scale * 1.4426950408889634f;
-  if (a->slot || a->chunk > 0 || a->pos) RF_REQUIRE(paged, "slots, chunks and attention by row need the paged pool");
+  if (a->slot || a->chunk > 0 || a->pos || a->keep_first > 0 || a->slopes)
+    RF_REQUIRE(paged, "slots, chunks, kept first positions, distance slopes and attention by row need the paged pool");
+  if (a->slopes || a->keep_first > 0) RF_REQUIRE(!a->mask && !a->seg_q, "distance slopes and kept first positions do not go with data-dependent masks");
   p->slot = a->slot; p->chunk = a->chunk; p->sink = a->sink; p->gate = a->gate; p->ld_gate = a->ld_gate;
+  p->gate_by_head = a->gate_by_head; p->keep_first = a->window > 0 || a->chunk > 0 ? std::max(a->keep_first, 0) : 0; p->slopes = a->slopes;
   p->seq_of_row = a->seq_of_row; p->pos = a->pos; p->g_tiles = ceil_div(p->G, 16);
   p->ws_o = nullptr; p->ws_lse = nullptr; p->splits = 1; p->pages_per_split = 1 << 28; p->stages = 2;
   p->status = a->status;
@@ -598,8 +611,10 @@ static int launch_decode(const RfAttn* a, AttnParams& p, cudaStream_t s) {
   auto kfn = attn_decode_kernel<T, HD>;
   RF_ALLOW_SMEM_PER_DEVICE(kfn, 200 * 1024);
   // split the KV range so that small batches still fill the machine
-  // a chunk may begin anywhere in a page: one page more than its own size
-  const int max_kv = a->chunk > 0 ? std::min(a->max_kv_len, a->chunk) + 15 : a->max_kv_len;
+  // a chunk or window may begin anywhere in a page: one page more than its own size; the kept first positions end anywhere
+  int max_kv = a->max_kv_len;
+  if (a->chunk > 0) max_kv = std::min(max_kv, a->chunk + 15 + p.keep_first + 15);
+  if (a->window > 0) max_kv = std::min(max_kv, a->window + 15 + p.keep_first + 15);
   const DecodeSplitPlan pl = plan_decode_split(a->num_seqs, a->Hq, a->Hkv, HD, max_kv, a->ws != nullptr);
   const int splits = pl.splits;
   if (splits > 1) {
@@ -620,7 +635,7 @@ static int launch_decode(const RfAttn* a, AttnParams& p, cudaStream_t s) {
   ::rf::count_launch();
   if (splits > 1) {
     dim3 g2(a->Hq, a->num_seqs);
-    RF_CUDA_CHECK(::rf::launch_k(attn_decode_combine_kernel<T>, dim3(g2), dim3(HD < 128 ? HD : 128), 0, s, 1, p.ws_o, p.ws_lse, (T*)a->out, a->ldo, a->Hq, HD, splits, a->sink, (const T*)a->gate, a->ld_gate));
+    RF_CUDA_CHECK(::rf::launch_k(attn_decode_combine_kernel<T>, dim3(g2), dim3(HD < 128 ? HD : 128), 0, s, 1, p.ws_o, p.ws_lse, (T*)a->out, a->ldo, a->Hq, HD, splits, a->sink, (const T*)a->gate, a->ld_gate, a->gate_by_head));
     RF_CUDA_CHECK(cudaGetLastError());
   ::rf::count_launch();
   }
@@ -682,8 +697,6 @@ extern "C" int rf_attn_decode(const RfAttn* a, rf_stream_t stream) {
   if (rc) return rc;
   RF_REQUIRE(a->num_seqs <= 65535, "decode attention: %d rows in one launch", a->num_seqs);
   RF_REQUIRE(a->max_kv_len > 0, "decode attention needs max_kv_len");
-  RF_REQUIRE(a->window <= 0, "decode attention has no sliding-window form (window=%d): every query would see the whole "
-             "context", a->window);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   RF_ATTN_DISPATCH(launch_decode)
 }
@@ -705,7 +718,8 @@ extern "C" int rf_attn_prefill(const RfAttn* a, rf_stream_t stream) {
   // tcgen05 kernel by default; RF_ATTN_TC=0 selects the mma.sync kernel (A/B timing)
   static const bool use_tc = [] { const char* e = getenv("RF_ATTN_TC"); return !(e && e[0] == '0'); }();
   if (use_tc) return rf::launch_prefill_tc(a, p, s);
-  RF_REQUIRE(!a->slot && a->chunk <= 0 && !a->sink && !a->gate, "slots, chunks, sinks and gates need the tcgen05 prefill kernel");
+  RF_REQUIRE(!a->slot && a->chunk <= 0 && !a->sink && !a->gate && a->keep_first <= 0 && !a->slopes,
+             "slots, chunks, sinks, gates, kept first positions and slopes need the tcgen05 prefill kernel");
   RF_ATTN_DISPATCH(launch_prefill)
 }
 

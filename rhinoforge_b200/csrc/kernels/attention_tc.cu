@@ -84,7 +84,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   if (p.window > 0) kv_lo = max(0, qpos0 + qt * kFaRows - p.window + 1);
   if (p.chunk > 0) kv_lo = max(kv_lo, (qpos0 + qt * kFaRows) / p.chunk * p.chunk);   // the first row's chunk
   kv_lo &= ~(KVB - 1);
-  const int nblk = kv_hi > kv_lo ? (kv_hi - kv_lo + KVB - 1) / KVB : 0;
+  // blocks of the kept first positions come first, then those from the first row's window or chunk on
+  const int keep_blk = min((p.keep_first + KVB - 1) / KVB, kv_lo / KVB);
+  const int nblk = kv_hi > kv_lo ? keep_blk + (kv_hi - kv_lo + KVB - 1) / KVB : 0;
+  auto block_start = [&](int j) { return j < keep_blk ? j * KVB : kv_lo + (j - keep_blk) * KVB; };
 
   if (tid == 0) {
     mbar_init(&ctl->q_full, 1);
@@ -131,7 +134,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       int issued = 0, pages = 0;
       for (int j = 0; j < nblk; ++j) {
         if (p.paged && j % kBlocksPerFetch == 0)
-          pages = p.page_table[(size_t)pt_row * p.pt_stride + min((kv_lo + j * KVB) / 16 + lane, p.pt_stride - 1)];
+          pages = p.page_table[(size_t)pt_row * p.pt_stride + min(block_start(j + lane / kPagesPerBlock) / 16 + lane % kPagesPerBlock, p.pt_stride - 1)];
         int block_pages[kPagesPerBlock];
 #pragma unroll
         for (int w = 0; w < kPagesPerBlock; ++w) block_pages[w] = __shfl_sync(0xffffffffu, pages, (j % kBlocksPerFetch) * kPagesPerBlock + w);
@@ -147,7 +150,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         }
         if (!__shfl_sync(0xffffffffu, go, 0)) break;
         if (lane != 0) continue;
-        const int t0 = kv_lo + j * KVB;
+        const int t0 = block_start(j);
         uint8_t* ks = kvsm + (size_t)s * G::kStageBytes;
         uint8_t* vs = ks + G::kKBytes;
         mbar_arrive_expect_tx(&ctl->kv_full[s], (uint32_t)G::kStageBytes);
@@ -237,11 +240,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     int lo_row = p.window > 0 ? qpos0 + qi - p.window + 1 : 0;
     if (p.chunk > 0) lo_row = max(lo_row, (qpos0 + qi) / p.chunk * p.chunk);
     const bool data_mask = mrow != nullptr || p.seg_q != nullptr;
+    const float fall = p.slopes ? p.slopes[h] * kLog2e : 0.f;
+    const float score_mul = p.slopes ? 1.f : p.scale_log2;
     for (int j = 0; j < nblk; ++j) {
       const int b = j & 1;
       if (!mbar_wait(&ctl->s_full[b], (uint32_t)(j >> 1) & 1u) || *abort_flag) { ok = false; break; }
       tc_fence_after_sync();
-      const int t0 = kv_lo + j * KVB;
+      const int t0 = block_start(j);
       const uint32_t s_addr = lane_base + (uint32_t)(b * KVB);
       // the whole row of S for this block: all loads in flight, one wait
       uint32_t sv[KVB];
@@ -254,12 +259,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       if (lane == 0) mbar_arrive(&ctl->s_empty[b]);
       // masking: interior blocks need none; edge blocks compare against the row's [lo, hi]; boolean
       // masks and segment ids (rare) take the per-element path
-      const bool edge = __any_sync(0xffffffffu, t0 < lo_row || t0 + KVB - 1 > hi_row) || data_mask;
+      const bool edge = __any_sync(0xffffffffu, (t0 < lo_row && t0 + KVB > p.keep_first) || t0 + KVB - 1 > hi_row) || data_mask;
+      if (p.slopes) {                                       // finished scores: scaled, less the fall over the distance
+        const float past = (float)(t0 - qpos0 - qi);
+#pragma unroll
+        for (int i = 0; i < KVB; ++i)
+          sv[i] = __float_as_uint(fmaf(fall, past + (float)i, __uint_as_float(sv[i]) * p.scale_log2));
+      }
       float mx = -INFINITY;
       if (!edge) {
 #pragma unroll
         for (int i = 0; i < KVB; ++i) {
-          const float v = __uint_as_float(sv[i]) * p.scale_log2;
+          const float v = __uint_as_float(sv[i]) * score_mul;
           sv[i] = __float_as_uint(v);
           mx = fmaxf(mx, v);
         }
@@ -277,7 +288,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           const int tk = t0 + i;
           const uint32_t word = reinterpret_cast<const uint32_t*>(&mv[i >> 4])[(i >> 2) & 3];
           const bool v = tk >= lo_row && tk <= hi_row && ((word >> ((i & 3) * 8)) & 0xffu) != 0;
-          const float x = v ? __uint_as_float(sv[i]) * p.scale_log2 : -INFINITY;
+          const float x = v ? __uint_as_float(sv[i]) * score_mul : -INFINITY;
           sv[i] = __float_as_uint(x);
           mx = fmaxf(mx, x);
         }
@@ -285,12 +296,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 #pragma unroll
         for (int i = 0; i < KVB; ++i) {
           const int tk = t0 + i;
-          bool v = tk >= lo_row && tk <= hi_row;
+          bool v = (tk >= lo_row || tk < p.keep_first) && tk <= hi_row;
           if (data_mask && v) {
             if (mrow) v = mrow[tk] != 0;
             if (p.seg_q && v) v = p.seg_k[kv0 + tk] == sq;
           }
-          const float x = v ? __uint_as_float(sv[i]) * p.scale_log2 : -INFINITY;
+          const float x = v ? __uint_as_float(sv[i]) * score_mul : -INFINITY;
           sv[i] = __float_as_uint(x);
           mx = fmaxf(mx, x);
         }
@@ -349,8 +360,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     tc_fence_after_sync();
     if (ok) {
       if (p.sink && l > 0.f) l += exp2f(p.sink[h] * kLog2e - m_ref);
-      const float inv = l > 0.f ? 1.f / l : 0.f;
-      const T* grow = p.gate ? reinterpret_cast<const T*>(p.gate) + (size_t)(p.q_start[seq] + qi) * p.ld_gate + (size_t)h * HD : nullptr;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      const T* grow = p.gate ? reinterpret_cast<const T*>(p.gate) + (size_t)(p.q_start[seq] + qi) * p.ld_gate + (p.gate_by_head ? h : h * HD) : nullptr;
+      if (p.gate_by_head && grow && qi < qlen) {
+        inv *= sigmoid_fast(Num<T>::to_f(grow[0]));
+        grow = nullptr;
+      }
       T* orow = reinterpret_cast<T*>(p.out) + (size_t)(p.q_start[seq] + qi) * p.ldo + (size_t)h * HD;
 #pragma unroll 1
       for (int c0 = 0; c0 < HD; c0 += 32) {

@@ -25,6 +25,8 @@ struct AttnParams {
   int32_t chunk;
   const float* sink;      // natural-log units
   const void* gate; int64_t ld_gate;
+  int32_t gate_by_head, keep_first;
+  const float* slopes;    // natural-log units per token of distance
   const int32_t* seq_of_row; const int32_t* pos;
   int32_t g_tiles;        // decode: CTAs that share one K/V head (16 query heads each)
 };

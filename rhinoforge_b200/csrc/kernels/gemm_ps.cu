@@ -43,6 +43,7 @@ struct GemmPsParams {
   const uint8_t* w_packed;
   int32_t* status;
   int M, N, k_blocks, bn, stages, act, dual_offset, dual_tiles;
+  ActArgs act_args;
   int tiles_m, tiles_n;   // tiles_m counts tiles of 128*MT rows
   int band;               // row tiles per band of the tile order
   int pf_blocks;          // k blocks prefetched into L2 ahead of the ring
@@ -367,7 +368,7 @@ gemm_ps_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             }
           }
         }
-        apply_act_n<16>(p.act, g, u, v);
+        apply_act_n<16>(p.act, g, u, v, p.act_args);
         if (tma_out) {
           // row `lane` of the warp's staging tile, 128-byte swizzled as the bulk store expects it
           const int ch = ((n0 - n_base) >> 3) & 7;
@@ -464,7 +465,7 @@ static int launch_ps(const RfGemm* g, int bn, cudaStream_t stream) {
   p.tma_out = tma_out ? (g->residual ? 2 : 1) : 0;
   p.M = g->M; p.N = g->N; p.k_blocks = ceil_div(g->K, kPsBK); p.bn = bn;
   p.kb_total = p.k_blocks;
-  p.act = g->act; p.dual_offset = g->dual_offset; p.dual_tiles = ceil_div(g->N, 128);
+  p.act = g->act; p.act_args = {g->act_limit, g->act_alpha}; p.dual_offset = g->dual_offset; p.dual_tiles = ceil_div(g->N, 128);
   p.tiles_m = ceil_div(g->M, kPsBM * MT); p.tiles_n = ceil_div(g->N, bn);
   const int stage_bytes = MT * kPsATile + (DUAL ? 2 : 1) * bn * kPsBK * 2;
   {
@@ -541,7 +542,7 @@ static int launch_ps_grouped(const RfMoeGroupedGemm* a, cudaStream_t stream) {
   p.w_packed = reinterpret_cast<const uint8_t*>(a->w);
   p.status = a->status;
   p.M = a->max_rows; p.N = a->N; p.k_blocks = ceil_div(a->K, kPsBK); p.bn = bn;
-  p.act = a->act; p.dual_offset = DUAL ? a->N : 0; p.dual_tiles = a->bank_section_row_tiles;
+  p.act = a->act; p.act_args = {a->act_limit, a->act_alpha}; p.dual_offset = DUAL ? a->N : 0; p.dual_tiles = a->bank_section_row_tiles;
   p.tiles_m = 0; p.tiles_n = ceil_div(a->N, bn);
   p.band = 1;
   p.tma_out = tma_out ? 1 : 0;
@@ -595,7 +596,7 @@ extern "C" int rf_moe_grouped_gemm(const RfMoeGroupedGemm* a, rf_stream_t stream
   RF_REQUIRE(a->dtype == 0 || a->dtype == 1, "moe_grouped_gemm dtype");
   RF_REQUIRE(a->bank_kb_total > 0 && a->rt_per_expert >= 0 && a->kb_per_expert >= 0, "moe_grouped_gemm bank geometry");
   RF_REQUIRE((reinterpret_cast<uintptr_t>(a->w) & 127) == 0, "packed expert bank must be 128-byte aligned");
-  if (a->dual) RF_REQUIRE(a->bank_section_row_tiles > 0 && (a->act == rf::kActSiluMul || a->act == rf::kActGeluTanhMul),
-                          "a GLU grouped GEMM needs the section size and a *_mul activation");
+  if (a->dual) RF_REQUIRE(a->bank_section_row_tiles > 0 && rf::act_is_dual(a->act), "a GLU grouped GEMM needs the section size and an activation of two operands");
+  if (a->act == rf::kActClippedGlu) RF_REQUIRE(a->act_limit > 0.f, "this activation needs a positive limit");
   return rf::launch_moe_grouped(a, static_cast<cudaStream_t>(stream));
 }

@@ -49,6 +49,7 @@ struct GemmSkParams {
   const uint8_t* w_packed;
   float* ws; uint32_t* flags; int32_t* status;
   int M, N, k_blocks, bn, stages, act, dual_offset, dual_tiles, tiles;
+  ActArgs act_args;
   long long units;
   int stage_off;             // shared-memory offset of the [token][128] staging rows
   int ctl_off;
@@ -333,7 +334,7 @@ gemm_sk_kernel(const __grid_constant__ CUtensorMap tmX, const GemmSkParams p) {
                 if (scale) { vg *= Num<T>::to_f(scale[n_feat]); if (DUAL) vu *= Num<T>::to_f(scale[p.dual_offset + n_feat]); }
                 if (use_bias) { vg += Num<T>::to_f(bias[n_feat]); if (DUAL) vu += Num<T>::to_f(bias[p.dual_offset + n_feat]); }
               }
-              v = apply_act(p.act, vg, vu);
+              v = apply_act(p.act, vg, vu, p.act_args);
               if (resid && !pub) v += Num<T>::to_f(resid[(size_t)tok * p.ldr + n_feat]);
             }
             if (pub_f32) reinterpret_cast<float*>(stage)[tok * kSkBM + r] = v;
@@ -487,7 +488,7 @@ static int launch_sk(const RfGemm* g, const SkPlan& pl, cudaStream_t stream) {
   p.bias = g->bias; p.scale = g->scale; p.row_scale = g->row_scale;
   p.w_packed = reinterpret_cast<const uint8_t*>(g->w);
   p.ws = g->ws; p.flags = g->sem; p.status = g->status;
-  p.M = g->M; p.N = g->N; p.k_blocks = pl.k_blocks; p.bn = pl.bn; p.stages = pl.stages; p.act = g->act;
+  p.M = g->M; p.N = g->N; p.k_blocks = pl.k_blocks; p.bn = pl.bn; p.stages = pl.stages; p.act = g->act; p.act_args = {g->act_limit, g->act_alpha};
   p.dual_offset = g->dual_offset; p.dual_tiles = pl.tiles; p.tiles = pl.tiles; p.units = pl.units;
   p.stage_off = pl.stage_off; p.ctl_off = pl.ctl_off; p.tmem_cols = pl.tmem_cols;
   p.ar_world = g->ar_world; p.ar_rank = g->ar_rank; p.ar_publish = g->ar_publish; p.ar_cnt_base = g->ar_cnt_base;

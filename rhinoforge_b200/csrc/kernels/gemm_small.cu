@@ -38,6 +38,7 @@ struct SmallParams {
   const void* scale;          // optional per-output-column factor, applied before the bias (16-bit weights only)
   const void* mul; const int32_t* mul_row; int64_t mul_ld;   // optional gate: result *= mul[mul_row[m] * mul_ld + n]
   int M, N, K, act, dual_offset, packed, kb_total, dual_tiles, splits;
+  ActArgs act_args;
 };
 
 __device__ __forceinline__ void sm_cp16(void* dst, const void* src, bool valid) {
@@ -224,7 +225,7 @@ gemm_small_kernel(const SmallParams p) {
         u1 += Num<T>::to_f(bias[p.dual_offset + n + 1]);
       }
     }
-    float v0 = apply_act(p.act, g0, u0), v1 = apply_act(p.act, g1, u1);
+    float v0 = apply_act(p.act, g0, u0, p.act_args), v1 = apply_act(p.act, g1, u1, p.act_args);
     if (p.mul) {
       const T* e = reinterpret_cast<const T*>(p.mul) + (size_t)p.mul_row[m] * p.mul_ld + n;
       v0 *= Num<T>::to_f(e[0]);
@@ -368,7 +369,7 @@ int gemm_small_run(const RfGemm* g, cudaStream_t s) {
   p.x = g->x; p.ldx = g->ldx; p.w = g->w; p.ldw = g->ldw; p.out = g->out; p.ldo = g->ldo;
   p.residual = g->residual; p.ldr = g->ldr; p.bias = g->bias; p.scale = g->scale;
   p.mul = g->mul; p.mul_row = g->mul_row; p.mul_ld = g->mul_ld;
-  p.M = g->M; p.N = g->N; p.K = g->K; p.act = g->act; p.dual_offset = g->dual_offset; p.packed = g->w_packed ? 1 : 0;
+  p.M = g->M; p.N = g->N; p.K = g->K; p.act = g->act; p.act_args = {g->act_limit, g->act_alpha}; p.dual_offset = g->dual_offset; p.packed = g->w_packed ? 1 : 0;
   p.kb_total = (g->K + 63) / 64;
   p.dual_tiles = dual ? (g->dual_offset + 127) / 128 : 0;    // the up section starts this many 128-row tiles after the gate section
   const int bm = g->M > 64 ? 128 : 64;

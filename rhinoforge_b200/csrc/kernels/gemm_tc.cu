@@ -42,6 +42,7 @@ struct GemmTcParams {
   float* ws; uint32_t* sem; int32_t* status;
   int M, N;
   int k_blocks, splits, bn, stages, act, dual_offset, tmem_cols, ctl_offset;
+  ActArgs act_args;
   int ar_world, ar_rank;
   void* const* ar_recv; uint32_t* const* ar_flags; uint32_t* ar_state;
   uint64_t ar_half_bytes;
@@ -444,7 +445,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
   // per-element epilogue math shared by both paths
   const bool affine = p.row_scale || scale || use_bias || use_rs;
   auto finish = [&](int tok, int n, float vg, float vu) -> float {
-    if (!affine) return apply_act(p.act, vg, vu);
+    if (!affine) return apply_act(p.act, vg, vu, p.act_args);
     if (use_rs) {
       const float rs = ss_rs[tok - blockIdx.y * bn];
       vg *= rs;
@@ -463,7 +464,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       vg += Num<T>::to_f(bias[n]);
       if (DUAL) vu += Num<T>::to_f(bias[p.dual_offset + n]);
     }
-    return apply_act(p.act, vg, vu);
+    return apply_act(p.act, vg, vu, p.act_args);
   };
   // Peer buffer addresses are read ONCE: the table lives in global memory and nothing tells the compiler
   // that the remote stores below cannot alias it, so a lookup per element would sit between every two stores.
@@ -1219,7 +1220,7 @@ static int launch_gemm(const RfGemm* g, const GemmPlan& pl, cudaStream_t stream)
   p.ws = g->ws; p.sem = g->sem; p.status = g->status;
   p.M = g->M; p.N = g->N;
   p.k_blocks = pl.k_blocks; p.splits = pl.splits; p.bn = pl.bn; p.stages = pl.stages; p.ctl_offset = pl.ctl_offset;
-  p.act = g->act; p.dual_offset = g->dual_offset; p.tmem_cols = pl.tmem_cols;
+  p.act = g->act; p.act_args = {g->act_limit, g->act_alpha}; p.dual_offset = g->dual_offset; p.tmem_cols = pl.tmem_cols;
   p.ar_world = g->ar_world; p.ar_rank = g->ar_rank;
   p.ar_recv = g->ar_recv; p.ar_flags = g->ar_flags; p.ar_state = g->ar_state;
   p.ar_half_bytes = g->ar_recv_bytes;
@@ -1286,8 +1287,8 @@ static int check_gemm(const RfGemm* g) {
     if (g->w_int8) RF_REQUIRE(g->scale != nullptr && g->K % 16 == 0, "int8 weights need a scale vector and K %% 16 == 0");
   }
   RF_REQUIRE(g->dtype == 0 || g->dtype == 1, "GEMM dtype must be fp16 or bf16");
-  const bool dual_act = g->act == kActSiluMul || g->act == kActGeluTanhMul;
-  RF_REQUIRE(dual_act == (g->dual_offset > 0), "dual_offset and a *_mul activation go together");
+  RF_REQUIRE(act_is_dual(g->act) == (g->dual_offset > 0), "dual_offset and an activation of two operands go together");
+  if (g->act == kActClippedGlu || g->act == kActSoftCap) RF_REQUIRE(g->act_limit > 0.f, "this activation needs a positive limit");
   if (g->ar_world > 1) {
     RF_REQUIRE(g->ar_world <= 8 && g->ar_rank >= 0 && g->ar_rank < g->ar_world, "bad ar rank/world");
     RF_REQUIRE(g->ar_recv && g->ar_flags && g->ar_state, "fused all-reduce needs recv/flags/state");

@@ -18,6 +18,7 @@ struct GemvParams {
   const void* residual; int64_t ldr;
   const void* bias; const void* scale; const float* row_scale;
   int M, N, K, act, dual_offset;
+  ActArgs act_args;
 };
 
 template <typename T, int MT, bool I8>
@@ -111,15 +112,15 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
     if (scale) { v0 *= Num<T>::to_f(scale[n0]); if (two) v1 *= Num<T>::to_f(scale[n1]); }
     if (bias) { v0 += Num<T>::to_f(bias[n0]); if (two) v1 += Num<T>::to_f(bias[n1]); }
     if (dual) {
-      float r = apply_act(p.act, v0, v1);
+      float r = apply_act(p.act, v0, v1, p.act_args);
       if (resid) r += Num<T>::to_f(resid[(size_t)m * p.ldr + n0]);
       out[(size_t)m * p.ldo + n0] = Num<T>::from_f(r);
     } else {
-      float r0 = apply_act(p.act, v0, 0.f);
+      float r0 = apply_act(p.act, v0, 0.f, p.act_args);
       if (resid) r0 += Num<T>::to_f(resid[(size_t)m * p.ldr + n0]);
       out[(size_t)m * p.ldo + n0] = Num<T>::from_f(r0);
       if (two) {
-        float r1 = apply_act(p.act, v1, 0.f);
+        float r1 = apply_act(p.act, v1, 0.f, p.act_args);
         if (resid) r1 += Num<T>::to_f(resid[(size_t)m * p.ldr + n1]);
         out[(size_t)m * p.ldo + n1] = Num<T>::from_f(r1);
       }
@@ -155,12 +156,11 @@ extern "C" int rf_gemv(const RfGemm* g, rf_stream_t stream) {
              "gemv K=%d / pitches must be multiples of %d", g->K, vec);
   RF_REQUIRE(!g->w_int8 || g->scale, "int8 weights need a scale vector");
   RF_REQUIRE(g->ar_world <= 1, "gemv has no fused all-reduce");
-  const bool dual_act = g->act == kActSiluMul || g->act == kActGeluTanhMul;
-  RF_REQUIRE(dual_act == (g->dual_offset > 0), "dual_offset and a *_mul activation go together");
+  RF_REQUIRE(act_is_dual(g->act) == (g->dual_offset > 0), "dual_offset and an activation of two operands go together");
   GemvParams p;
   p.x = g->x; p.ldx = g->ldx; p.w = g->w; p.ldw = g->ldw; p.out = g->out; p.ldo = g->ldo;
   p.residual = g->residual; p.ldr = g->ldr; p.bias = g->bias; p.scale = g->scale;
-  p.row_scale = g->row_scale; p.M = g->M; p.N = g->N; p.K = g->K; p.act = g->act;
+  p.row_scale = g->row_scale; p.M = g->M; p.N = g->N; p.K = g->K; p.act = g->act; p.act_args = {g->act_limit, g->act_alpha};
   p.dual_offset = g->dual_offset;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (g->dtype == 0)

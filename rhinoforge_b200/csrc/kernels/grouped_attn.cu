@@ -1,5 +1,5 @@
-// Grouped-head attention of the mixed-layer decoders: what happens between the input projection and the attention (per-head
-// norms, rotation, value mixing, insertion into the K/V pages; one launch), and a plain attention kernel for models served in
+// Grouped-head attention of the mixed-layer decoders: what happens between the input projection and the attention (causal
+// convolution, norms, rotation, value mixing, insertion into the K/V pages; one launch), and a plain attention kernel for models served in
 // 32 bits and for head sizes that the tensor-core kernels do not take.
 #include "../common/dtype.cuh"
 #include "../common/host_util.h"
@@ -8,34 +8,24 @@
 
 namespace rf {
 
-// A head of hd values is held by GL lanes, NC chunks of eight consecutive values each (hd <= 8 * GL * NC).  Groups are numbered
-// over (row, item), items of a row being its query heads, key heads and value heads.
-template <typename T, int GL, int NC>
-__global__ void __launch_bounds__(256) qkv_insert_kernel(const RfQkvInsert p) {
-  pdl_prologue();
-  extern __shared__ __align__(16) float rot_buf[];
-  constexpr int HPW = 32 / GL;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gl = lane % GL, sub = lane / GL;
-  const int items = p.heads + 2 * p.kv_heads;
-  const int64_t idx = ((int64_t)blockIdx.x * (blockDim.x >> 5) + warp) * HPW + sub;
-  const bool live = idx < (int64_t)p.n_rows * items;
-  const int row = live ? (int)(idx / items) : 0, item = live ? (int)(idx % items) : 0;
-  const bool is_q = item < p.heads, is_v = item >= p.heads + p.kv_heads;
-  const int head = is_q ? item : (is_v ? item - p.heads - p.kv_heads : item - p.heads);
-  const int hd = p.hd;
-  T* src = reinterpret_cast<T*>(p.qkv) + (size_t)row * p.ld + (is_q ? 0 : (is_v ? p.v_off : p.k_off)) + (size_t)head * hd;
-  const int pos = p.rows.pos[row];
-  float x[NC][8];
-#pragma unroll
-  for (int c = 0; c < NC; ++c) {
-    const int o = (gl + c * GL) * 8;
-    if (live && o < hd) load8(src + o, x[c]);
-    else {
-#pragma unroll
-      for (int j = 0; j < 8; ++j) x[c][j] = 0.f;
-    }
+// A head of hd values is held by GL lanes, NC chunks of eight consecutive values each (hd <= 8 * GL * NC).  The items of a row are
+// its query heads, key heads and value heads.
+struct HeadItem {
+  int row, item, head;
+  bool is_q, is_v, live;
+  __device__ __forceinline__ HeadItem(const RfQkvInsert& p, int row_, int item_, bool live_)
+      : row(row_), item(item_), is_q(item_ < p.heads), is_v(item_ >= p.heads + p.kv_heads), live(live_) {
+    head = is_q ? item : (is_v ? item - p.heads - p.kv_heads : item - p.heads);
   }
-  const float* nw = is_v ? nullptr : (is_q ? p.q_norm : p.k_norm);
+  template <typename T>
+  __device__ __forceinline__ T* source(const RfQkvInsert& p) const {
+    return reinterpret_cast<T*>(p.qkv) + (size_t)row * p.ld + (is_q ? 0 : (is_v ? p.v_off : p.k_off)) + (size_t)head * p.hd;
+  }
+};
+
+// 1 / rms of this group's head (all lanes of the warp).
+template <int GL, int NC>
+__device__ __forceinline__ float head_rstd(const RfQkvInsert& p, const float (&x)[NC][8]) {
   float ss = 0.f;
 #pragma unroll
   for (int c = 0; c < NC; ++c)
@@ -43,8 +33,16 @@ __global__ void __launch_bounds__(256) qkv_insert_kernel(const RfQkvInsert p) {
     for (int j = 0; j < 8; ++j) ss += x[c][j] * x[c][j];
 #pragma unroll
   for (int d = GL / 2; d >= 1; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+  return rsqrtf(ss / (float)p.dim + p.eps);
+}
+
+// Norm with `rstd`, rotation, value mixing and the store of one head; all lanes of the warp, buf: the group's scratch.
+template <typename T, int GL, int NC>
+__device__ __forceinline__ void finish_head(const RfQkvInsert& p, const HeadItem& it, float (&x)[NC][8], float rstd, int gl, float* buf) {
+  const int hd = p.hd, pos = p.rows.pos[it.row];
+  const float* nw = it.is_v ? nullptr : (it.is_q ? p.q_norm : p.k_norm);
   if (nw) {
-    const float rstd = rsqrtf(ss / (float)p.dim + p.eps);
+    if (p.norm_all) nw += (size_t)it.head * hd;
 #pragma unroll
     for (int c = 0; c < NC; ++c) {
       const int o = (gl + c * GL) * 8;
@@ -55,8 +53,8 @@ __global__ void __launch_bounds__(256) qkv_insert_kernel(const RfQkvInsert p) {
     }
   }
   if (p.rot_dims > 0) {                            // uniform over the grid
-    float* buf = rot_buf + (size_t)(warp * HPW + sub) * p.rot_dims;
     const int half = p.rot_dims >> 1;
+    __syncwarp();
 #pragma unroll
     for (int c = 0; c < NC; ++c) {
       const int o = (gl + c * GL) * 8;
@@ -65,7 +63,7 @@ __global__ void __launch_bounds__(256) qkv_insert_kernel(const RfQkvInsert p) {
         if (o + j < p.rot_dims) buf[o + j] = x[c][j];
     }
     __syncwarp();
-    if (live && !is_v) {
+    if (it.live && !it.is_v) {
       const float* cs = p.cos + (size_t)pos * half;
       const float* sn = p.sin + (size_t)pos * half;
 #pragma unroll
@@ -80,9 +78,9 @@ __global__ void __launch_bounds__(256) qkv_insert_kernel(const RfQkvInsert p) {
       }
     }
   }
-  if (!live) return;
-  if (is_v && p.v_role != RF_VMIX_NONE) {
-    T* first = reinterpret_cast<T*>(p.v_first) + (size_t)row * p.kv_heads * p.vdim + (size_t)head * p.vdim;
+  if (!it.live) return;
+  if (it.is_v && p.v_role != RF_VMIX_NONE) {
+    T* first = reinterpret_cast<T*>(p.v_first) + (size_t)it.row * p.kv_heads * p.vdim + (size_t)it.head * p.vdim;
 #pragma unroll
     for (int c = 0; c < NC; ++c) {
       const int o = (gl + c * GL) * 8;
@@ -94,18 +92,169 @@ __global__ void __launch_bounds__(256) qkv_insert_kernel(const RfQkvInsert p) {
       }
     }
   }
-  T* dst = src;
-  if (!is_q) {
-    const int seq = p.rows.seq_of_row ? p.rows.seq_of_row[row] : row;
+  T* dst;
+  if (it.is_q) {
+    dst = p.q_out ? reinterpret_cast<T*>(p.q_out) + ((size_t)it.row * p.heads + it.head) * hd : it.source<T>(p);
+  } else {
+    const int seq = p.rows.seq_of_row ? p.rows.seq_of_row[it.row] : it.row;
     const int slot = p.rows.slot ? p.rows.slot[seq] : seq;
     const int page = p.rows.page_table[(size_t)slot * p.rows.pt_stride + (pos >> 4)];
-    dst = reinterpret_cast<T*>(is_v ? p.v_pool : p.k_pool) + (((size_t)page * p.kv_heads + head) * 16 + (pos & 15)) * hd;
+    dst = reinterpret_cast<T*>(it.is_v ? p.v_pool : p.k_pool) + (((size_t)page * p.kv_heads + it.head) * 16 + (pos & 15)) * hd;
   }
 #pragma unroll
   for (int c = 0; c < NC; ++c) {
     const int o = (gl + c * GL) * 8;
     if (o < hd) store8(dst + o, x[c]);
   }
+}
+
+template <typename T, int GL, int NC>
+__device__ __forceinline__ void load_head(const T* src, bool live, int hd, int gl, float (&x)[NC][8]) {
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int o = (gl + c * GL) * 8;
+    if (live && o < hd) load8(src + o, x[c]);
+    else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[c][j] = 0.f;
+    }
+  }
+}
+
+// Groups are numbered over (row, item).
+template <typename T, int GL, int NC>
+__global__ void __launch_bounds__(256) qkv_insert_kernel(const RfQkvInsert p) {
+  pdl_prologue();
+  extern __shared__ __align__(16) float rot_buf[];
+  constexpr int HPW = 32 / GL;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gl = lane % GL, sub = lane / GL;
+  const int items = p.heads + 2 * p.kv_heads;
+  const int64_t idx = ((int64_t)blockIdx.x * (blockDim.x >> 5) + warp) * HPW + sub;
+  const bool live = idx < (int64_t)p.n_rows * items;
+  const HeadItem it(p, live ? (int)(idx / items) : 0, live ? (int)(idx % items) : 0, live);
+  float x[NC][8];
+  load_head<T, GL, NC>(it.source<T>(p), live, p.hd, gl, x);
+  finish_head<T, GL, NC>(p, it, x, head_rstd<GL, NC>(p, x), gl, rot_buf + (size_t)(warp * HPW + sub) * p.rot_dims);
+}
+
+// One norm over all query heads of a row and one over all key heads: a CTA per row, which is read twice.
+template <typename T, int GL, int NC>
+__global__ void __launch_bounds__(256) qkv_insert_row_kernel(const RfQkvInsert p) {
+  pdl_prologue();
+  extern __shared__ __align__(16) float rot_buf[];
+  __shared__ float red[2][8];
+  constexpr int HPW = 32 / GL;
+  const int warp = threadIdx.x >> 5, nw = blockDim.x >> 5, lane = threadIdx.x & 31, gl = lane % GL, sub = lane / GL;
+  const int row = blockIdx.x, items = p.heads + 2 * p.kv_heads, groups = nw * HPW, qn = p.heads * p.hd / 8, kn = p.kv_heads * p.hd / 8;
+  const T* src = reinterpret_cast<const T*>(p.qkv) + (size_t)row * p.ld;
+  float sq = 0.f, sk = 0.f;
+  for (int i = threadIdx.x; i < qn + kn; i += blockDim.x) {
+    float f[8], s = 0.f;
+    load8(i < qn ? src + i * 8 : src + p.k_off + (i - qn) * 8, f);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s += f[j] * f[j];
+    if (i < qn) sq += s;
+    else sk += s;
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+  __syncthreads();
+  sq = sk = 0.f;
+  for (int w = 0; w < nw; ++w) { sq += red[0][w]; sk += red[1][w]; }
+  const float rq = rsqrtf(sq / (float)(p.heads * p.dim) + p.eps), rk = rsqrtf(sk / (float)(p.kv_heads * p.dim) + p.eps);
+  for (int i0 = 0; i0 < items; i0 += groups) {
+    const int item = i0 + warp * HPW + sub;
+    const bool live = item < items;
+    const HeadItem it(p, row, live ? item : 0, live);
+    float x[NC][8];
+    load_head<T, GL, NC>(it.source<T>(p), live, p.hd, gl, x);
+    finish_head<T, GL, NC>(p, it, x, it.is_q ? rq : rk, gl, rot_buf + (size_t)(warp * HPW + sub) * p.rot_dims);
+  }
+}
+
+// With the convolution: a group walks `tile` neighbouring rows of one sequence for its head, the last inputs in registers
+// (TAPS = 0: any number of taps, every input read again for each of them).  The group of a sequence's first rows also replaces the
+// carried inputs; later tiles find theirs among the rows of this launch.
+template <typename T, int GL, int NC, int TAPS>
+__global__ void __launch_bounds__(256) qkv_conv_insert_kernel(const RfQkvInsert p, int tile) {
+  pdl_prologue();
+  extern __shared__ __align__(16) float rot_buf[];
+  constexpr int HPW = 32 / GL;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gl = lane % GL, sub = lane / GL;
+  const int items = p.heads + 2 * p.kv_heads, hd = p.hd, seq = blockIdx.z, past = (TAPS > 0 ? TAPS : p.taps) - 1;
+  const int q0 = p.rows.q_start ? p.rows.q_start[seq] : seq, n = p.rows.q_len ? p.rows.q_len[seq] : 1;
+  const int t0 = blockIdx.y * tile, t1 = min(n, t0 + tile);
+  if (t0 >= n) return;
+  const int item = (blockIdx.x * (blockDim.x >> 5) + warp) * HPW + sub;
+  const bool live = item < items, fresh = p.rows.pos[q0] == 0;
+  const size_t channels = (size_t)items * hd, at = (size_t)(live ? item : 0) * hd;
+  T* state = reinterpret_cast<T*>(p.conv_state) + (size_t)(p.rows.slot ? p.rows.slot[seq] : seq) * past * channels + at;
+  const T* src = reinterpret_cast<const T*>(p.qkv) + (size_t)q0 * p.ld + at;
+  const float* w = p.conv_w + at;
+  float* buf = rot_buf + (size_t)(warp * HPW + sub) * p.rot_dims;
+  // input at place i of this launch's rows; negative places are carried ones
+  auto input = [&](int i, float (&f)[NC][8]) {
+    if (i >= 0) load_head<T, GL, NC>(src + (size_t)i * p.ld, live, hd, gl, f);
+    else load_head<T, GL, NC>(state + (size_t)(past + i) * channels, live && !fresh, hd, gl, f);
+  };
+  auto finish = [&](int t, float (&x)[NC][8]) {
+    const HeadItem it(p, q0 + t, live ? item : 0, live);
+    finish_head<T, GL, NC>(p, it, x, head_rstd<GL, NC>(p, x), gl, buf);
+  };
+  if constexpr (TAPS > 0) {
+    float wt[TAPS][NC][8], win[TAPS][NC][8];
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) load_head<float, GL, NC>(w + k * channels, live, hd, gl, wt[k]);
+#pragma unroll
+    for (int k = 0; k < TAPS - 1; ++k) input(t0 - (TAPS - 1) + k, win[k]);
+    for (int t = t0; t < t1; ++t) {
+      float x[NC][8];
+      input(t, win[TAPS - 1]);
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          x[c][j] = 0.f;
+#pragma unroll
+          for (int k = 0; k < TAPS; ++k) x[c][j] += wt[k][c][j] * win[k][c][j];
+        }
+#pragma unroll
+      for (int k = 0; k < TAPS - 1; ++k)
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+#pragma unroll
+          for (int j = 0; j < 8; ++j) win[k][c][j] = win[k + 1][c][j];
+      finish(t, x);
+    }
+  } else {
+    for (int t = t0; t < t1; ++t) {
+      float x[NC][8], f[NC][8], v[NC][8];
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[c][j] = 0.f;
+      for (int k = 0; k <= past; ++k) {
+        load_head<float, GL, NC>(w + k * channels, live, hd, gl, f);
+        input(t - past + k, v);
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+#pragma unroll
+          for (int j = 0; j < 8; ++j) x[c][j] += f[c][j] * v[c][j];
+      }
+      finish(t, x);
+    }
+  }
+  if (blockIdx.y == 0 && live)
+    for (int i = 0; i < past; ++i) {             // ascending: row i comes from a later row of the old state, or from this launch
+      float v[NC][8];
+      input(n - past + i, v);
+#pragma unroll
+      for (int c = 0; c < NC; ++c) {
+        const int o = (gl + c * GL) * 8;
+        if (o < hd) store8(state + (size_t)i * channels + o, v[c]);
+      }
+    }
 }
 
 // One CTA per (row, query head): four warps walk the visible keys, lanes share the head dimension, everything in fp32.
@@ -119,20 +268,24 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const RfAttn p) {
   float* ml = ar_sm + hd * 5;
   const int seq = p.seq_of_row ? p.seq_of_row[row] : row, pt_row = p.slot ? p.slot[seq] : seq;
   const int pos = p.pos[row], kvh = h / (p.Hq / p.Hkv);
-  const int lo = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
+  int lo = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
+  if (p.window > 0) lo = max(lo, pos - p.window + 1);
+  const int keep = min(p.keep_first, lo);          // visible positions: [0, keep) and [lo, pos]
+  const float fall = p.slopes ? p.slopes[h] : 0.f;
   for (int i = threadIdx.x; i < hd; i += blockDim.x)
     q[i] = Num<T>::to_f(reinterpret_cast<const T*>(p.q)[(size_t)row * p.ldq + (size_t)h * hd + i]);
   for (int i = lane; i < hd; i += 32) acc[i] = 0.f;
   __syncthreads();
   float m = -INFINITY, l = 0.f;
-  for (int j = lo + warp; j <= pos; j += 4) {
+  for (int n = warp; n < keep + pos - lo + 1; n += 4) {
+    const int j = n < keep ? n : n - keep + lo;
     const int page = p.page_table[(size_t)pt_row * p.pt_stride + (j >> 4)];
     const size_t at = (((size_t)page * p.Hkv + kvh) * 16 + (j & 15)) * hd;
     const T* k = reinterpret_cast<const T*>(p.k_pool) + at;
     const T* v = reinterpret_cast<const T*>(p.v_pool) + at;
     float s = 0.f;
     for (int i = lane; i < hd; i += 32) s += q[i] * Num<T>::to_f(k[i]);
-    s = warp_sum(s) * p.scale;
+    s = warp_sum(s) * p.scale - fall * (float)(pos - j);
     const float mn = fmaxf(m, s), keep = expf(m - mn), w = expf(s - mn);
     l = l * keep + w;
     m = mn;
@@ -153,15 +306,43 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const RfAttn p) {
     for (int w = 0; w < 4; ++w) o += f[w] * ar_sm[hd * (1 + w) + i];
     o /= den;
     const size_t col = (size_t)h * hd + i;
-    if (p.gate) o *= 1.f / (1.f + expf(-Num<T>::to_f(reinterpret_cast<const T*>(p.gate)[(size_t)row * p.ld_gate + col])));
+    if (p.gate) o *= 1.f / (1.f + expf(-Num<T>::to_f(reinterpret_cast<const T*>(p.gate)[(size_t)row * p.ld_gate + (p.gate_by_head ? h : col)])));
     reinterpret_cast<T*>(p.out)[(size_t)row * p.ldo + col] = Num<T>::from_f(o);
   }
+}
+
+template <typename T, int GL, int NC, int TAPS>
+static int launch_qkv_conv(const RfQkvInsert* a, int warps, cudaStream_t s) {
+  const int per_block = warps * (32 / GL), tile = std::max(16, a->taps - 1);
+  const size_t smem = (size_t)per_block * a->rot_dims * sizeof(float);
+  RF_ALLOW_SMEM_PER_DEVICE((qkv_conv_insert_kernel<T, GL, NC, TAPS>), 64 * 1024);
+  const dim3 grid(ceil_div(a->heads + 2 * a->kv_heads, per_block), ceil_div(a->max_q_len, tile), a->rows.num_seqs);
+  RF_CUDA_CHECK(::rf::launch_k(qkv_conv_insert_kernel<T, GL, NC, TAPS>, grid, dim3(warps * 32), smem, s, 1, *a, tile));
+  ::rf::count_launch();
+  return RF_OK;
 }
 
 template <typename T, int GL, int NC>
 static int launch_qkv_insert(const RfQkvInsert* a, cudaStream_t s) {
   const int64_t groups = (int64_t)a->n_rows * (a->heads + 2 * a->kv_heads);
   const int warps = groups * GL / 32 < 8 * sm_count() ? 2 : 8, per_block = warps * (32 / GL);
+  if (a->taps > 0) {
+    if (NC > 1) return launch_qkv_conv<T, GL, NC, 0>(a, warps, s);
+    switch (a->taps) {
+      case 2: return launch_qkv_conv<T, GL, NC, NC == 1 ? 2 : 0>(a, warps, s);
+      case 3: return launch_qkv_conv<T, GL, NC, NC == 1 ? 3 : 0>(a, warps, s);
+      case 4: return launch_qkv_conv<T, GL, NC, NC == 1 ? 4 : 0>(a, warps, s);
+      default: return launch_qkv_conv<T, GL, NC, 0>(a, warps, s);
+    }
+  }
+  if (a->norm_all) {
+    const int threads = 256;
+    const size_t smem = (size_t)(threads / GL) * a->rot_dims * sizeof(float);
+    RF_ALLOW_SMEM_PER_DEVICE((qkv_insert_row_kernel<T, GL, NC>), 64 * 1024);
+    RF_CUDA_CHECK(::rf::launch_k(qkv_insert_row_kernel<T, GL, NC>, dim3(a->n_rows), dim3(threads), smem, s, 1, *a));
+    ::rf::count_launch();
+    return RF_OK;
+  }
   const size_t smem = (size_t)per_block * a->rot_dims * sizeof(float);
   RF_ALLOW_SMEM_PER_DEVICE((qkv_insert_kernel<T, GL, NC>), 64 * 1024);
   RF_CUDA_CHECK(::rf::launch_k(qkv_insert_kernel<T, GL, NC>, dim3((unsigned)((groups + per_block - 1) / per_block)), dim3(warps * 32),
@@ -195,6 +376,14 @@ extern "C" int rf_qkv_insert(const RfQkvInsert* a, rf_stream_t stream) {
              "qkv_insert: rotation of %d dimensions", a->rot_dims);
   RF_REQUIRE(a->v_role == RF_VMIX_NONE || a->v_first, "qkv_insert: value mixing needs the first values");
   RF_REQUIRE(a->dtype >= 0 && a->dtype <= 2, "qkv_insert: dtype %d", a->dtype);
+  if (a->taps > 0) {
+    RF_REQUIRE(a->conv_w && a->q_out && a->q_out != a->qkv && (a->taps == 1 || a->conv_state) && !a->norm_all,
+               "qkv_insert: the convolution needs weights, its state and an output for the queries, and per-head norms");
+    RF_REQUIRE(a->k_off == a->heads * a->hd && a->v_off == (a->heads + a->kv_heads) * a->hd, "qkv_insert: queries, keys and values are neighbours");
+    RF_REQUIRE(a->max_q_len >= 1 && a->rows.num_seqs <= 65535 && (int64_t)a->max_q_len <= 16ll * 65535, "qkv_insert: %d sequences of up to %d rows",
+               a->rows.num_seqs, a->max_q_len);
+    if (a->rows.num_seqs == 0) return RF_OK;
+  }
   if (a->n_rows == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (a->dtype == kF16) return dispatch_qkv_insert<__half>(a, s);
@@ -206,7 +395,7 @@ extern "C" int rf_attn_rows(const RfAttn* a, rf_stream_t stream) {
   RF_SKIP_IF_REPLAYING();
   RF_REQUIRE(a && a->q && a->out && a->k_pool && a->v_pool && a->page_table && a->pos, "attn_rows: missing buffers");
   RF_REQUIRE(a->hd > 0 && a->hd <= 2048 && a->Hkv > 0 && a->Hq % a->Hkv == 0, "attn_rows: heads");
-  RF_REQUIRE(a->window <= 0 && !a->mask && !a->seg_q && a->dtype >= 0 && a->dtype <= 2, "attn_rows: options");
+  RF_REQUIRE(a->keep_first >= 0 && !a->mask && !a->seg_q && a->dtype >= 0 && a->dtype <= 2, "attn_rows: options");
   RF_REQUIRE(a->num_seqs <= 65535, "attn_rows: %d rows in one launch", a->num_seqs);
   if (a->num_seqs == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);

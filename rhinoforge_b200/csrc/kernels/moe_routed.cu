@@ -45,7 +45,11 @@ __device__ __forceinline__ void route_token(const RfMoeRouter& p, int lane, floa
   float mx = -INFINITY;
 #pragma unroll
   for (int s = 0; s < S; ++s) mx = fmaxf(mx, s * 32 + lane < E ? sc[s] : -INFINITY);
-  if (p.score_fn == RF_MOE_SOFTMAX) {
+  if (p.score_fn == RF_MOE_CHOSEN) {
+#pragma unroll
+    for (int s = 0; s < S; ++s)
+      if (p.correction && s * 32 + lane < E) sc[s] += p.correction[s * 32 + lane];
+  } else if (p.score_fn == RF_MOE_SOFTMAX) {
     mx = warp_max(mx);
     float sum = 0.f;
 #pragma unroll
@@ -64,7 +68,7 @@ __device__ __forceinline__ void route_token(const RfMoeRouter& p, int lane, floa
 #pragma unroll
   for (int s = 0; s < S; ++s) {
     const int e = s * 32 + lane;
-    key[s] = e < E ? sc[s] + (p.correction ? p.correction[e] : 0.f) : -INFINITY;
+    key[s] = e < E ? sc[s] + (p.correction && p.score_fn != RF_MOE_CHOSEN ? p.correction[e] : 0.f) : -INFINITY;
   }
   if (p.keep < p.groups) {
     // a group counts as much as its best expert; experts outside the best groups cannot be chosen
@@ -118,6 +122,11 @@ __device__ __forceinline__ void route_token(const RfMoeRouter& p, int lane, floa
     sum += w;
     if (lane == j) { *my_id = b.i < E ? b.i : -1; *my_w = w; }
   }
+  if (p.score_fn == RF_MOE_CHOSEN) {                      // the first pick has the largest logit
+    const float top = __shfl_sync(0xffffffffu, *my_w, 0), e = lane < p.k ? expf(*my_w - top) : 0.f;
+    *my_w = e / warp_sum(e) * p.scale;
+    return;
+  }
   *my_w *= (p.norm_topk ? 1.f / (sum + 1e-20f) : 1.f) * p.scale;
 }
 
@@ -157,7 +166,7 @@ __device__ __forceinline__ void plan_tiles(const RfMoeRouter& p, PlanSmem& sm) {
     for (int t = tid; t < p.rows; t += blockDim.x) {
       p.slot_of[(size_t)t * p.slot_ld + p.k] = pairs + t;
       p.token_of_slot[pairs + t] = t;
-      p.slot_w[pairs + t] = 1.f;
+      if (!p.shared_gate) p.slot_w[pairs + t] = 1.f;
     }
 }
 
@@ -180,7 +189,7 @@ __global__ void __launch_bounds__(kRtTokens * 32) moe_choose_kernel(const RfMoeR
   __shared__ PlanSmem sm;
   __shared__ int32_t base[256];
   __shared__ int last;
-  const int E = p.experts, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int E = p.experts, columns = E + p.shared_gate, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const bool alone = gridDim.x == 1;
   const int per_cta = alone ? kRtOneCta : kRtTokens, first = blockIdx.x * per_cta;
   const int here = min(per_cta, p.rows - first);
@@ -197,7 +206,12 @@ __global__ void __launch_bounds__(kRtTokens * 32) moe_choose_kernel(const RfMoeR
       const int e = s * 32 + lane;
       sc[s] = 0.f;
       if (e < E)
-        for (int z = 0; z < splits; ++z) sc[s] += p.logits[((size_t)z * p.rows + first + t) * E + e];
+        for (int z = 0; z < splits; ++z) sc[s] += p.logits[((size_t)z * p.rows + first + t) * columns + e];
+    }
+    if (p.shared_gate && lane == 0) {
+      float v = 0.f;
+      for (int z = 0; z < splits; ++z) v += p.logits[((size_t)z * p.rows + first + t) * columns + E];
+      p.slot_w[(size_t)p.rows * p.k + first + t] = 1.f / (1.f + expf(-v));
     }
     int id;
     float w;
@@ -254,7 +268,7 @@ __global__ void __launch_bounds__(256, 2) moe_logits_kernel(const RfMoeRouter p)
   pdl_prologue();
   constexpr int KW = 8 / TW, ROWS = 16 * MT * TW, LD = 68;
   extern __shared__ __align__(16) float lg[];             // [KW][ROWS][LD]
-  const int E = p.experts, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3;
+  const int E = p.experts + p.shared_gate, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3;
   const int tw = warp % TW, kw = warp / TW, t0 = blockIdx.x * ROWS + tw * 16 * MT, e0 = blockIdx.y * 64;
   const T* x = reinterpret_cast<const T*>(p.x);
   const T* w = reinterpret_cast<const T*>(p.w) + (size_t)(e0 + g) * p.width;
@@ -314,12 +328,13 @@ __global__ void __launch_bounds__(256) moe_logits_f32_kernel(const RfMoeRouter p
   pdl_prologue();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x;
   const float* x = reinterpret_cast<const float*>(p.x) + (size_t)t * p.ldx;
-  for (int e = warp; e < p.experts; e += 8) {
+  const int columns = p.experts + p.shared_gate;
+  for (int e = warp; e < columns; e += 8) {
     const float* w = reinterpret_cast<const float*>(p.w) + (size_t)e * p.width;
     float s = 0.f;
     for (int i = lane; i < p.width; i += 32) s += x[i] * w[i];
     s = warp_sum(s);
-    if (lane == 0) p.logits[(size_t)t * p.experts + e] = s;
+    if (lane == 0) p.logits[(size_t)t * columns + e] = s;
   }
 }
 
@@ -342,7 +357,7 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const RfMoeRouter p, T*
   if (threadIdx.x == 32 && p.has_shared) {
     p.slot_of[(size_t)t * p.slot_ld + p.k] = pairs + t;
     p.token_of_slot[pairs + t] = t;
-    p.slot_w[pairs + t] = 1.f;
+    if (!p.shared_gate) p.slot_w[pairs + t] = 1.f;
   }
   __syncthreads();
   const T* x = reinterpret_cast<const T*>(p.x) + (size_t)t * p.ldx;
@@ -459,8 +474,18 @@ __global__ void __launch_bounds__(256, MT == 1 ? 2 : 1) moe_small_kernel(const R
       }
     }
     const float ws = p.slot_w ? p.slot_w[row0 + r] : 1.f;
+    if constexpr (DUAL) {
+      if (p.act == kActClippedGlu) {
+        const ActArgs a = {sh ? p.shared_limit : p.act_limit, p.act_alpha};
 #pragma unroll
-    for (int j = 0; j < 8; ++j) v[0][j] = (DUAL ? silu_f(v[0][j]) * v[D - 1][j] : v[0][j]) * ws;
+        for (int j = 0; j < 8; ++j) v[0][j] = clipped_glu_f(v[0][j], v[D - 1][j], a);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[0][j] = silu_f(v[0][j]) * v[D - 1][j];
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[0][j] *= ws;
     store8(reinterpret_cast<T*>(p.out) + (size_t)(row0 + r) * p.ldo + f0 + c, v[0]);
   }
 }
@@ -512,7 +537,11 @@ __global__ void __launch_bounds__(256) moe_f32_kernel(const RfMoeExperts p) {
       const int r = ty * 4 + i, n = n0 + tx * 4 + j;
       if (r >= rows || n >= N) continue;
       const float g = acc[0][i][j];
-      const float v = DUAL ? g / (1.f + expf(-g)) * acc[D - 1][i][j] : g;
+      float v = g;
+      if constexpr (DUAL) {
+        const float u = acc[D - 1][i][j], limit = sh ? p.shared_limit : p.act_limit, gc = fminf(g, limit);
+        v = p.act == kActClippedGlu ? gc / (1.f + expf(-p.act_alpha * gc)) * (fminf(fmaxf(u, -limit), limit) + 1.f) : g / (1.f + expf(-g)) * u;
+      }
       reinterpret_cast<float*>(p.out)[(size_t)(row0 + r) * p.ldo + n] = v * (p.slot_w ? p.slot_w[row0 + r] : 1.f);
     }
 }
@@ -529,7 +558,7 @@ static int launch_logits(const RfMoeRouter* a, int splits, cudaStream_t s) {
   constexpr int ROWS = 16 * MT * TW;
   const size_t smem = (size_t)(8 / TW) * ROWS * 68 * sizeof(float);
   RF_ALLOW_SMEM_PER_DEVICE((moe_logits_kernel<T, MT, TW>), 80 * 1024);
-  RF_CUDA_CHECK(::rf::launch_k(moe_logits_kernel<T, MT, TW>, dim3(ceil_div(a->rows, ROWS), ceil_div(a->experts, 64), splits), dim3(256), smem, s, 1, *a));
+  RF_CUDA_CHECK(::rf::launch_k(moe_logits_kernel<T, MT, TW>, dim3(ceil_div(a->rows, ROWS), ceil_div(a->experts + a->shared_gate, 64), splits), dim3(256), smem, s, 1, *a));
   ::rf::count_launch();
   return RF_OK;
 }
@@ -571,6 +600,8 @@ static int check_router(const RfMoeRouter* a) {
   RF_REQUIRE(a->width > 0 && a->width % 8 == 0 && a->ldx % 8 == 0 && a->tile_rows > 0 && a->slot_ld >= a->k + (a->has_shared ? 1 : 0),
              "moe_router: width %d, tile of %d rows", a->width, a->tile_rows);
   RF_REQUIRE(a->dtype >= 0 && a->dtype <= 2 && (int64_t)a->rows * (a->k + 1) < (1ll << 30), "moe_router: dtype %d", a->dtype);
+  RF_REQUIRE(a->score_fn >= RF_MOE_SIGMOID && a->score_fn <= RF_MOE_CHOSEN && (a->shared_gate == 0 || (a->shared_gate == 1 && a->has_shared)),
+             "moe_router: score function %d, gate of the shared expert %d", a->score_fn, a->shared_gate);
   return RF_OK;
 }
 
@@ -591,7 +622,7 @@ extern "C" int rf_moe_router(const RfMoeRouter* a, rf_stream_t stream) {
     ::rf::count_launch();
   } else {
     const bool many = a->rows > 1024;
-    splits = router_splits(a->rows, a->experts, a->width);
+    splits = router_splits(a->rows, a->experts + a->shared_gate, a->width);
     if (a->dtype == kF16) rc2 = many ? launch_logits<__half, 2, 2>(a, 1, s) : launch_logits<__half, 1, 1>(a, splits, s);
     else rc2 = many ? launch_logits<__nv_bfloat16, 2, 2>(a, 1, s) : launch_logits<__nv_bfloat16, 1, 1>(a, splits, s);
     if (rc2) return rc2;
@@ -624,6 +655,8 @@ extern "C" int rf_moe_experts(const RfMoeExperts* a, rf_stream_t stream) {
   RF_REQUIRE(a->n > 0 && a->k > 0 && a->n % 8 == 0 && a->k % 8 == 0 && a->ldx % 8 == 0 && a->ldo % 8 == 0, "moe_experts: %d x %d", a->n, a->k);
   RF_REQUIRE((a->shared_n > 0) == (a->w_shared != nullptr) && a->shared_n % 8 == 0 && a->shared_k % 8 == 0, "moe_experts: shared expert");
   RF_REQUIRE(a->dtype >= 0 && a->dtype <= 2, "moe_experts: dtype %d", a->dtype);
+  RF_REQUIRE(a->act == 0 || a->act == kActSiluMul || (a->act == kActClippedGlu && a->act_limit > 0.f && (!a->w_shared || a->shared_limit > 0.f)),
+             "moe_experts: activation %d", a->act);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (a->dtype == kF32) {
     RF_REQUIRE(a->tile_rows == 64, "moe_experts: 32-bit tiles have 64 rows");

@@ -46,6 +46,23 @@ __device__ __forceinline__ float4 pending4(const RfStreamNorm& p, const T* y, in
   return s;
 }
 __device__ __forceinline__ float4 mul4(float4 v, float f) { return make_float4(v.x * f, v.y * f, v.z * f, v.w * f); }
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+// Row of table2 for the token pair (previous token, token) that ends in row r.
+__device__ __forceinline__ int64_t pair_row(const RfStreamNorm& p, int r) {
+  const int seq = p.rows.seq_of_row ? p.rows.seq_of_row[r] : r, q0 = p.rows.q_start ? p.rows.q_start[seq] : r;
+  int64_t prev;
+  if (r > q0) prev = p.ids[r - 1];
+  else if (p.rows.pos[r] == 0) return p.buckets;
+  else prev = p.last_token[p.rows.slot ? p.rows.slot[seq] : seq];
+  return (prev * p.mul_prev + p.ids[r] * p.mul_cur) % p.buckets;
+}
+// The CTA of a sequence's first row, the only reader of the carried token, replaces it (all threads of the CTA, after pair_row).
+__device__ __forceinline__ void carry_token(const RfStreamNorm& p, int r) {
+  const int seq = p.rows.seq_of_row ? p.rows.seq_of_row[r] : r, q0 = p.rows.q_start ? p.rows.q_start[seq] : r;
+  if (r != q0) return;
+  __syncthreads();
+  if (threadIdx.x == 0) p.last_token[p.rows.slot ? p.rows.slot[seq] : seq] = p.ids[q0 + (p.rows.q_len ? p.rows.q_len[seq] : 1) - 1];
+}
 __device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
 
 // A CTA walks rows_per_cta neighbouring rows.  A thread always touches the same columns, so the shared copies of the
@@ -73,16 +90,19 @@ __global__ void stream_norm_kernel(const RfStreamNorm p, int rows_per_cta) {
     }
     const float* xr = p.x ? p.x + (size_t)src * H : nullptr;
     const T* er = p.x ? nullptr : table + (size_t)p.ids[src] * H;
+    const T* er2 = p.table2 ? reinterpret_cast<const T*>(p.table2) + (size_t)pair_row(p, src) * H : nullptr;
+    if (er2) carry_token(p, src);
     float s = 0.f;
     for (int i = c0; i < H; i += step) {
       float4 v = xr ? *reinterpret_cast<const float4*>(xr + i) : mul4(load4(er + i), p.embed_scale);
+      if (er2) v = add4(v, load4(er2 + i));
       if (y) {
         float4 a = pending4(p, y, src, i);
         if (p.y_norm_w) {
           const float4 w = *reinterpret_cast<const float4*>(p.y_norm_w + i);
           a.x *= yr * w.x; a.y *= yr * w.y; a.z *= yr * w.z; a.w *= yr * w.w;
         }
-        v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+        v = add4(v, mul4(a, p.y_mult));
       }
       *reinterpret_cast<float4*>(xs + i) = v;
       s += sq4(v);
@@ -175,10 +195,13 @@ __global__ void __launch_bounds__(VPT == 4 ? 512 : 1024) stream_norm_reg_kernel(
   float4 v[VPT], a[VPT];
   auto load = [&](int r) {
     const int src = p.row_idx ? p.row_idx[r] : r;
+    const T* second = p.table2 ? reinterpret_cast<const T*>(p.table2) + (size_t)pair_row(p, src) * H : nullptr;
+    if (second) carry_token(p, src);
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
       const bool in = col(k) < H;
       v[k] = !in ? zero : p.x ? *reinterpret_cast<const float4*>(p.x + (size_t)src * H + col(k)) : mul4(load4(table + (size_t)p.ids[src] * H + col(k)), p.embed_scale);
+      if (second && in) v[k] = add4(v[k], load4(second + col(k)));
       a[k] = y && in ? pending4(p, y, src, col(k)) : zero;
     }
   };
@@ -197,7 +220,7 @@ __global__ void __launch_bounds__(VPT == 4 ? 512 : 1024) stream_norm_reg_kernel(
       if (p.y_norm_w) {
         a[k].x *= yr * yw[k].x; a[k].y *= yr * yw[k].y; a[k].z *= yr * yw[k].z; a[k].w *= yr * yw[k].w;
       }
-      v[k].x += a[k].x; v[k].y += a[k].y; v[k].z += a[k].z; v[k].w += a[k].w;
+      v[k] = add4(v[k], mul4(a[k], p.y_mult));
       s += sq4(v[k]);
     }
     return p.norm_w ? rsqrtf(block_sum(s) * inv_dim + p.eps) : 1.f;
@@ -322,7 +345,7 @@ __global__ void __launch_bounds__(512) stream_out_kernel(const RfStreamNorm p) {
   for (int k = 0; k < NC; ++k)
 #pragma unroll
     for (int j = 0; j < 8; ++j) s += a[k][j] * a[k][j];
-  const float yr = rsqrtf(block_sum(s, 0) * inv_dim + p.eps);
+  const float yr = rsqrtf(block_sum(s, 0) * inv_dim + p.eps) * p.y_mult;
   s = 0.f;
 #pragma unroll
   for (int k = 0; k < NC; ++k) {
@@ -367,8 +390,11 @@ __global__ void token_gate_kernel(T* __restrict__ g, int64_t ldg, const T* __res
 // ------------------------------------------------------------------ fp32 GEMM ----
 constexpr int kFBM = 64, kFBN = 64, kFBK = 16;
 
-__device__ __forceinline__ float act_f32(int act, float v) {
+__device__ __forceinline__ float act_f32(int act, float v, float u, ActArgs a) {
   switch (act) {
+    case kActSiluMul: return v / (1.f + expf(-v)) * u;
+    case kActClippedGlu: v = fminf(v, a.limit); return v / (1.f + expf(-a.alpha * v)) * (fminf(fmaxf(u, -a.limit), a.limit) + 1.f);
+    case kActSoftCap: return a.limit * tanhf(v / a.limit);
     case kActRelu2: return relu2_f(v);
     case kActSilu: return v / (1.f + expf(-v));
     case kActGeluTanh: return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
@@ -377,30 +403,42 @@ __device__ __forceinline__ float act_f32(int act, float v) {
   }
 }
 
+// DUAL: a second block of weight rows, dual_offset rows below the first, feeds the activation's second operand.
+template <bool DUAL>
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ x, int64_t ldx, const float* __restrict__ w,
                                                        int64_t ldw, float* __restrict__ out, int64_t ldo, int M, int N,
-                                                       int K, int act) {
+                                                       int K, int act, int dual_offset, const float* __restrict__ row_scale, ActArgs args) {
   pdl_prologue();
-  __shared__ __align__(16) float sx[kFBK][kFBM + 4], sw[kFBK][kFBN + 4];
+  constexpr int D = DUAL ? 2 : 1;
+  __shared__ __align__(16) float sx[kFBK][kFBM + 4], sw[D][kFBK][kFBN + 4];
   const int n0 = blockIdx.x * kFBN, m0 = blockIdx.y * kFBM, tid = threadIdx.x;
   const int tx = tid % 16, ty = tid / 16, lr = tid / 4, lk = (tid % 4) * 4;
-  float acc[4][4] = {};
+  float acc[D][4][4] = {};
   for (int k0 = 0; k0 < K; k0 += kFBK) {
     const bool kin = k0 + lk < K;            // K is a multiple of 4
-    float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
     if (kin && m0 + lr < M) a = *reinterpret_cast<const float4*>(x + (size_t)(m0 + lr) * ldx + k0 + lk);
-    if (kin && n0 + lr < N) b = *reinterpret_cast<const float4*>(w + (size_t)(n0 + lr) * ldw + k0 + lk);
     sx[lk][lr] = a.x; sx[lk + 1][lr] = a.y; sx[lk + 2][lr] = a.z; sx[lk + 3][lr] = a.w;
-    sw[lk][lr] = b.x; sw[lk + 1][lr] = b.y; sw[lk + 2][lr] = b.z; sw[lk + 3][lr] = b.w;
+#pragma unroll
+    for (int d = 0; d < D; ++d) {
+      float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (kin && n0 + lr < N) b = *reinterpret_cast<const float4*>(w + (size_t)(n0 + lr + d * dual_offset) * ldw + k0 + lk);
+      sw[d][lk][lr] = b.x; sw[d][lk + 1][lr] = b.y; sw[d][lk + 2][lr] = b.z; sw[d][lk + 3][lr] = b.w;
+    }
     __syncthreads();
 #pragma unroll
     for (int k = 0; k < kFBK; ++k) {
-      const float4 av = *reinterpret_cast<const float4*>(&sx[k][ty * 4]), bv = *reinterpret_cast<const float4*>(&sw[k][tx * 4]);
-      const float am[4] = {av.x, av.y, av.z, av.w}, bn[4] = {bv.x, bv.y, bv.z, bv.w};
+      const float4 av = *reinterpret_cast<const float4*>(&sx[k][ty * 4]);
+      const float am[4] = {av.x, av.y, av.z, av.w};
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
+      for (int d = 0; d < D; ++d) {
+        const float4 bv = *reinterpret_cast<const float4*>(&sw[d][k][tx * 4]);
+        const float bn[4] = {bv.x, bv.y, bv.z, bv.w};
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(am[i], bn[j], acc[i][j]);
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) acc[d][i][j] = fmaf(am[i], bn[j], acc[d][i][j]);
+      }
     }
     __syncthreads();
   }
@@ -409,7 +447,9 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
-      if (m < M && n < N) out[(size_t)m * ldo + n] = act_f32(act, acc[i][j]);
+      if (m >= M || n >= N) continue;
+      const float rs = row_scale ? row_scale[m] : 1.f;
+      out[(size_t)m * ldo + n] = act_f32(act, acc[0][i][j] * rs, acc[D - 1][i][j] * rs, args);
     }
 }
 
@@ -427,6 +467,7 @@ extern "C" int rf_stream_norm(const RfStreamNorm* args, rf_stream_t stream) {
   RF_REQUIRE(args != nullptr, "stream_norm: null arguments");
   RfStreamNorm filled = *args;
   if (filled.embed_scale == 0.f) filled.embed_scale = 1.f;
+  if (filled.y_mult == 0.f) filled.y_mult = 1.f;
   const RfStreamNorm* a = &filled;
   RF_REQUIRE(a->y_picks <= 0 || (a->y && a->y_slots), "stream_norm: picked rows need y and y_slots");
   RF_REQUIRE(a && a->H > 0 && a->H % 8 == 0 && a->dim > 0 && a->dim <= a->H, "stream_norm: row length");
@@ -435,12 +476,14 @@ extern "C" int rf_stream_norm(const RfStreamNorm* args, rf_stream_t stream) {
   RF_REQUIRE(a->dtype >= 0 && a->dtype <= 2, "stream_norm: dtype %d", a->dtype);
   if (a->shift) RF_REQUIRE(a->norm_w && a->shift_state && a->rows.pos && !a->row_idx && a->x_out != a->x,
                            "stream_norm: the token shift needs a norm, its state, positions, all rows and separate streams");
+  if (a->table2) RF_REQUIRE(!a->x && !a->shift && !a->row_idx && a->rows.pos && a->last_token && a->buckets > 0 && a->mul_prev >= 0 && a->mul_cur >= 0,
+                            "stream_norm: token pairs need the embedding rows of all rows, positions, the carried tokens and no token shift");
   if (a->n_rows == 0) return RF_OK;
   // halo of one row per CTA with the shift: walk several rows per CTA once that still fills the GPU
   const int rpc = (a->shift && a->rows.q_start) ? std::max(1, std::min(8, a->n_rows / (2 * sm_count()))) : 1;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int groups = a->H / 8;
-  if (a->y && a->y_norm_w && !a->shift && a->dtype != kF32 && groups <= 1024) {
+  if (a->y && a->y_norm_w && !a->shift && !a->table2 && a->dtype != kF32 && groups <= 1024) {
     // decode rows: one group of columns per thread; many rows: two, so that several rows share an SM
     const int nc = groups > 512 || (groups > 256 && a->n_rows > 4 * sm_count()) ? 2 : 1;
     const dim3 block(std::max(32, round_up(ceil_div(groups, nc), 32)));
@@ -492,13 +535,19 @@ extern "C" int rf_gemm_f32(const RfGemm* g, rf_stream_t stream) {
   RF_SKIP_IF_REPLAYING();
   RF_REQUIRE(g && g->x && g->w && g->out && g->M >= 0 && g->N > 0 && g->K > 0, "gemm_f32 arguments");
   RF_REQUIRE(g->K % 4 == 0 && g->ldx % 4 == 0 && g->ldw % 4 == 0, "gemm_f32: K and the pitches must be multiples of 4");
-  RF_REQUIRE(!g->residual && !g->bias && !g->scale && !g->row_scale && g->dual_offset == 0 && !g->w_packed && g->ar_world <= 1,
-             "gemm_f32 has an activation epilogue only");
+  RF_REQUIRE(!g->residual && !g->bias && !g->scale && !g->w_packed && g->ar_world <= 1, "gemm_f32 has a row-scale and activation epilogue only");
+  RF_REQUIRE(act_is_dual(g->act) == (g->dual_offset > 0) && g->act != kActGeluTanhMul, "dual_offset and an activation of two operands go together");
+  if (g->act == kActClippedGlu || g->act == kActSoftCap) RF_REQUIRE(g->act_limit > 0.f, "this activation needs a positive limit");
   if (g->M == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  RF_CUDA_CHECK(::rf::launch_k(gemm_f32_kernel, dim3(ceil_div(g->N, kFBN), ceil_div(g->M, kFBM)), dim3(256), 0, s, 1,
-                               (const float*)g->x, g->ldx, (const float*)g->w, g->ldw, (float*)g->out, g->ldo, g->M, g->N,
-                               g->K, g->act));
+  const dim3 grid(ceil_div(g->N, kFBN), ceil_div(g->M, kFBM));
+  const ActArgs args = {g->act_limit, g->act_alpha};
+#define RF_F32(DUAL)                                                                                                                 \
+  RF_CUDA_CHECK(::rf::launch_k(gemm_f32_kernel<DUAL>, grid, dim3(256), 0, s, 1, (const float*)g->x, g->ldx, (const float*)g->w, g->ldw, \
+                               (float*)g->out, g->ldo, g->M, g->N, g->K, g->act, g->dual_offset, g->row_scale, args))
+  if (g->dual_offset > 0) RF_F32(true);
+  else RF_F32(false);
+#undef RF_F32
   ::rf::count_launch();
   return RF_OK;
 }

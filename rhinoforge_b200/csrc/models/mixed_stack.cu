@@ -31,7 +31,7 @@ struct MixedStack {
   uint8_t* base = nullptr;
   uint64_t off_x[2] = {}, off_h = 0, off_cast = 0, off_wide = 0, off_mix = 0, off_y = 0, off_side = 0, off_qlat = 0, off_olat = 0,
            off_ctx = 0, off_kv = 0, off_kvmeta = 0, off_attn_ws = 0, off_head = 0, off_argmax = 0, off_sk_ws = 0, off_sk_flags = 0,
-           off_status = 0, off_vfirst = 0, off_conv = 0, off_bc = 0, off_dt = 0, off_moe = 0, off_xg = 0, off_hg = 0, off_yg = 0, off_router = 0, total = 0;
+           off_status = 0, off_vfirst = 0, off_q = 0, off_conv = 0, off_bc = 0, off_dt = 0, off_moe = 0, off_xg = 0, off_hg = 0, off_yg = 0, off_router = 0, total = 0;
   uint64_t attn_ws_bytes = 0, argmax_bytes = 0, sk_ws_bytes = 0, rows_ws_bytes = 0;
   int moe_tiles = 0;      // tile-list entries of any mixture-of-experts layer
   int lat_rows = 0;       // rows one latent-space attention launch takes
@@ -56,13 +56,14 @@ struct MixedStack {
     auto al = [](uint64_t v) { return (v + 1023) & ~uint64_t(1023); };
     const uint64_t T = (uint64_t)cfg.max_tokens, H = (uint64_t)cfg.hidden, e = esz();
     uint64_t wide = 8, mix = 8, lat = 0, rank = 0, kvw = 0, past = 0, heads = 0;
-    uint64_t vfirst = 0, inner = 0, bc = 0, picks = 0, experts = 0, hg = 0;
+    uint64_t vfirst = 0, qout = 0, inner = 0, bc = 0, picks = 0, experts = 0, hg = 0;
     rows_ws_bytes = 0; moe_tiles = 0;
     for (const RfMixedLayer& l : layers) {
       wide = std::max<uint64_t>(wide, std::max(l.in_dim, l.inter));
       mix = std::max<uint64_t>(mix, (uint64_t)l.out_dim);
       if (l.mixer == RF_MIXER_ATTENTION) {
-        vfirst = std::max<uint64_t>(vfirst, (uint64_t)l.kv_heads * l.vdim);
+        vfirst = std::max<uint64_t>(vfirst, l.v_role != RF_VMIX_NONE ? (uint64_t)l.kv_heads * l.vdim : 0);
+        if (l.conv_taps > 0) qout = std::max<uint64_t>(qout, (uint64_t)l.heads * l.dim);
         if (l.tensor_core) rows_ws_bytes = std::max<uint64_t>(rows_ws_bytes, rf_attn_decode_scratch_bound(l.heads, l.kv_heads, l.dim));
       }
       if (l.mixer == RF_MIXER_MAMBA1) {
@@ -71,7 +72,7 @@ struct MixedStack {
       }
       if (l.experts > 0) {
         picks = std::max<uint64_t>(picks, l.top + 1);
-        experts = std::max<uint64_t>(experts, l.experts);
+        experts = std::max<uint64_t>(experts, l.experts + l.shared_gate);
         hg = std::max<uint64_t>(hg, moe_ld(l));
         moe_tiles = std::max(moe_tiles, l.experts + (int)(T * (l.top + 1) / 16) + 2);
       }
@@ -110,6 +111,7 @@ struct MixedStack {
     off_kv = o; o += al((uint64_t)ctx_rows * kvw * e);
     off_kvmeta = o; o += al((uint64_t)cfg.max_seqs * (2 * windows.size() + 1) * sizeof(int32_t));
     off_vfirst = o; o += al(T * vfirst * e);
+    off_q = o; o += al(T * qout * e);
     off_conv = o; o += al(T * inner * e);
     off_bc = o; o += al(T * bc * e);
     off_dt = o; o += al(fp32() ? 0 : T * inner * e);
@@ -156,6 +158,14 @@ static RfGemm gemm_args(const MixedStack& s, const void* x, int64_t ldx, const v
 static int linear(const MixedStack& s, const void* x, int64_t ldx, const void* w, void* out, int64_t ldo, int M, int N, int K,
                   int act, cudaStream_t st) {
   const RfGemm g = gemm_args(s, x, ldx, w, out, ldo, M, N, K, act);
+  return s.fp32() ? rf_gemm_f32(&g, st) : rf_gemm(&g, st);
+}
+
+// Gated pair: weight rows of the gates, then of the ups; out[M, N] = act(gate, up) with the activation's constants.
+static int linear_pair(const MixedStack& s, const void* x, int64_t ldx, const void* w, void* out, int64_t ldo, int M, int N, int K,
+                       int act, float limit, float alpha, cudaStream_t st) {
+  RfGemm g = gemm_args(s, x, ldx, w, out, ldo, M, N, K, act);
+  g.dual_offset = N; g.act_limit = limit; g.act_alpha = alpha;
   return s.fp32() ? rf_gemm_f32(&g, st) : rf_gemm(&g, st);
 }
 
@@ -317,6 +327,12 @@ static int hgrn2(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f, 
   return rc;
 }
 
+static int longest_portion(const RfMixedForward& f) {
+  int n = 1;
+  for (int i = 0; !f.decode && i < f.rows.num_seqs; ++i) n = std::max(n, (int)f.h_q_len[i]);
+  return n;
+}
+
 static int grouped_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f, const void* h, void* mix, cudaStream_t st) {
   const RfMixedConfig& c = s.cfg;
   const int T = f.tokens, H = c.hidden, hd = w.dim, QD = w.heads * hd, KD = w.kv_heads * hd;
@@ -329,22 +345,30 @@ static int grouped_attention(MixedStack& s, const RfMixedLayer& w, const RfMixed
   q.q_norm = w.q_norm; q.k_norm = w.k_norm; q.cos = w.cos; q.sin = w.sin;
   q.v_first = s.at(s.off_vfirst); q.k_pool = w.st.k_pool; q.v_pool = w.st.v_pool; q.rows = f.rows;
   q.n_rows = T; q.heads = w.heads; q.kv_heads = w.kv_heads; q.hd = hd; q.dim = w.dim_true; q.vdim = w.vdim_true;
-  q.rot_dims = w.rot_dims; q.v_role = w.v_role; q.v_lambda = w.v_lambda; q.eps = c.eps; q.dtype = c.dtype;
+  q.rot_dims = w.rot_dims; q.v_role = w.v_role; q.v_lambda = w.v_lambda; q.eps = c.eps; q.dtype = c.dtype; q.norm_all = w.norm_all;
+  uint8_t* queries = wide;
+  int64_t ldq = w.in_dim;
+  if (w.conv_taps > 0) {
+    queries = s.at<uint8_t>(s.off_q);
+    ldq = QD;
+    q.conv_w = w.conv_w; q.conv_state = w.st.conv_state; q.q_out = queries; q.taps = w.conv_taps; q.max_q_len = longest_portion(f);
+  }
   rc = rf_qkv_insert(&q, st);
   if (rc) return rc;
   RfAttn a = {};
-  a.q = wide; a.ldq = w.in_dim; a.out = mix; a.ldo = QD; a.q_rows_total = T;
+  a.q = queries; a.ldq = ldq; a.out = mix; a.ldo = QD; a.q_rows_total = T;
   a.k_pool = w.st.k_pool; a.v_pool = w.st.v_pool; a.pool_pages = w.st.pool_pages;
   a.page_table = f.rows.page_table; a.pt_stride = f.rows.pt_stride;
   a.Hq = w.heads; a.Hkv = w.kv_heads; a.hd = hd; a.scale = w.scale; a.chunk = w.chunk; a.sink = w.sink;
-  if (w.gated) { a.gate = wide + (size_t)(QD + 2 * KD) * e; a.ld_gate = w.in_dim; }
+  a.window = w.window; a.keep_first = w.keep_first; a.slopes = w.slopes;
+  if (w.gated) { a.gate = wide + (size_t)(QD + 2 * KD) * e; a.ld_gate = w.in_dim; a.gate_by_head = w.gate_by_head; }
   a.status = s.status(); a.dtype = c.dtype;
   // ---- decoded rows and short portions, by row (without a tensor-core form: every row)
   const int by_row = w.tensor_core ? f.short_rows : T;
   for (int r0 = 0; r0 < by_row; r0 += 32768) {
     RfAttn b = a;
     b.num_seqs = std::min(32768, by_row - r0);
-    b.q = wide + (size_t)r0 * w.in_dim * e; b.out = (uint8_t*)mix + (size_t)r0 * QD * e;
+    b.q = queries + (size_t)r0 * ldq * e; b.out = (uint8_t*)mix + (size_t)r0 * QD * e;
     if (a.gate) b.gate = (const uint8_t*)a.gate + (size_t)r0 * w.in_dim * e;
     b.pos = f.rows.pos + r0; b.seq_of_row = f.rows.seq_of_row ? f.rows.seq_of_row + r0 : nullptr;
     b.slot = f.rows.slot ? f.rows.slot + (b.seq_of_row ? 0 : r0) : nullptr;
@@ -373,9 +397,7 @@ static int mamba1(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f,
   if (rc) return rc;
   RfConvSilu cv = {};
   cv.x = wide; cv.ldx = w.in_dim; cv.y = conv; cv.ldy = w.inner; cv.w = w.conv_w; cv.bias = w.conv_b; cv.state = w.st.conv_state;
-  cv.rows = f.rows; cv.channels = w.inner; cv.taps = w.taps; cv.dtype = c.dtype; cv.max_q_len = 1;
-  if (!f.decode)
-    for (int i = 0; i < f.rows.num_seqs; ++i) cv.max_q_len = std::max(cv.max_q_len, (int)f.h_q_len[i]);
+  cv.rows = f.rows; cv.channels = w.inner; cv.taps = w.taps; cv.dtype = c.dtype; cv.max_q_len = longest_portion(f);
   rc = rf_conv_silu(&cv, st);
   if (rc) return rc;
   rc = linear(s, conv, w.inner, w.w_x, bc, BC, T, BC, w.inner, kActNone, st);
@@ -422,6 +444,8 @@ static int experts(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f
   r.slot_w = (float*)m;
   r.rows = T; r.experts = E; r.width = H; r.k = k; r.groups = w.groups; r.keep = w.keep; r.score_fn = w.score_fn;
   r.norm_topk = w.norm_topk; r.scale = w.route_scale; r.slot_ld = cols; r.has_shared = has_shared; r.dtype = c.dtype;
+  r.shared_gate = w.shared_gate;
+  const int act = w.act == RF_MIXED_ACT_CLIPPED_GLU ? kActClippedGlu : kActSiluMul;
   uint8_t* hg = s.at<uint8_t>(s.off_hg);
   uint8_t* yg = s.at<uint8_t>(s.off_yg);
   out->y = yg; out->slots = r.slot_of; out->picks = cols;
@@ -434,7 +458,7 @@ static int experts(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f
     x.tiles = r.tiles; x.experts = E; x.tile_rows = r.tile_rows; x.dtype = c.dtype;
     x.max_tiles = std::min(E, pairs) + pairs / r.tile_rows + (has_shared ? ceil_div(T, r.tile_rows) : 0);
     x.x = h; x.ldx = H; x.token_of_slot = r.token_of_slot; x.w = w.w_up; x.w_shared = w.shared_up; x.out = hg; x.ldo = ldh;
-    x.n = w.inter; x.k = H; x.dual = 1;
+    x.n = w.inter; x.k = H; x.dual = 1; x.act = act; x.act_limit = w.act_limit; x.act_alpha = w.act_alpha; x.shared_limit = w.shared_limit;
     x.bank_section_row_tiles = E * bank_rt; x.bank_kb_total = kbH; x.rt_per_expert = bank_rt;
     if (has_shared) { x.shared_n = w.shared_inter; x.shared_k = H; x.shared_section_row_tiles = ceil_div(w.shared_inter, 128); x.shared_kb_total = kbH; }
     rc = rf_moe_experts(&x, st);
@@ -453,7 +477,7 @@ static int experts(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f
   if (rc) return rc;
   RfMoeGroupedGemm g = {};
   g.x = xg; g.ldx = H; g.w = w.w_up; g.out = hg; g.ldo = ldh; g.tiles = r.tiles + 3; g.max_rows = pairs; g.N = w.bank_inter; g.K = H;
-  g.dual = 1; g.act = kActSiluMul; g.bank_section_row_tiles = E * bank_rt; g.bank_kb_total = kbH; g.rt_per_expert = bank_rt;
+  g.dual = 1; g.act = act; g.act_limit = w.act_limit; g.act_alpha = w.act_alpha; g.bank_section_row_tiles = E * bank_rt; g.bank_kb_total = kbH; g.rt_per_expert = bank_rt;
   g.dtype = c.dtype; g.status = s.status();
   rc = rf_moe_grouped_gemm(&g, st);
   if (rc) return rc;
@@ -462,11 +486,11 @@ static int experts(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f
   rc = rf_moe_grouped_gemm(&g, st);
   if (rc || !has_shared) return rc;
   uint8_t* hs = hg + (size_t)pairs * ldh * e;
-  RfGemm u = gemm_args(s, h, H, w.shared_up, hs, ldh, T, w.shared_inter, H, kActSiluMul);
-  u.dual_offset = w.shared_inter;
-  rc = rf_gemm(&u, st);
+  rc = linear_pair(s, h, H, w.shared_up, hs, ldh, T, w.shared_inter, H, act, w.shared_limit, w.act_alpha, st);
   if (rc) return rc;
-  return linear(s, hs, ldh, w.shared_down, yg + (size_t)pairs * H * e, H, T, H, w.shared_inter, kActNone, st);
+  RfGemm d = gemm_args(s, hs, ldh, w.shared_down, yg + (size_t)pairs * H * e, H, T, H, w.shared_inter, kActNone);
+  if (w.shared_gate) d.row_scale = r.slot_w + pairs;
+  return rf_gemm(&d, st);
 }
 
 static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
@@ -493,7 +517,11 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
   auto step = [&](const float* norm_w, const float* shift, float* shift_state, bool want_cast) -> int {
     RfStreamNorm a = {};
     a.x = cur < 0 ? nullptr : s.at<float>(s.off_x[cur]);
-    a.table = c.embed; a.ids = f.ids; a.embed_scale = c.embed_scale;
+    a.table = c.embed; a.ids = f.ids; a.embed_scale = c.embed_scale; a.y_mult = c.residual_mult;
+    if (cur < 0 && c.pair_table) {
+      a.table2 = c.pair_table; a.last_token = s.layers[0].st.last_token; a.buckets = c.pair_buckets;
+      a.mul_prev = c.pair_mul_prev; a.mul_cur = c.pair_mul_cur;
+    }
     a.y = pend.y; a.y_norm_w = pend.norm; a.y_slots = pend.slots; a.y_picks = pend.picks;
     const int nxt = cur < 0 ? 0 : cur ^ 1;
     a.x_out = s.at<float>(s.off_x[nxt]);
@@ -526,7 +554,9 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
         rc = experts(s, w, f, in, &pend, st);
       } else {
         void* wide = s.at(s.off_wide);
-        rc = linear(s, in, H, w.w_up, wide, w.inter, T, w.inter, H, kActRelu2, st);
+        rc = w.act == RF_MIXED_ACT_CLIPPED_GLU
+                 ? linear_pair(s, in, H, w.w_up, wide, w.inter, T, w.inter, H, kActClippedGlu, w.act_limit, w.act_alpha, st)
+                 : linear(s, in, H, w.w_up, wide, w.inter, T, w.inter, H, kActRelu2, st);
         if (rc) return rc;
         rc = linear(s, wide, w.inter, w.w_down, y, H, T, H, w.inter, kActNone, st);
         pend.y = y;
@@ -546,7 +576,7 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
     }
     if (f.taps) {
       RfStreamNorm a = {};
-      a.x = s.at<float>(s.off_x[cur]); a.y = pend.y; a.y_norm_w = pend.norm; a.y_slots = pend.slots; a.y_picks = pend.picks;
+      a.x = s.at<float>(s.off_x[cur]); a.y_mult = c.residual_mult; a.y = pend.y; a.y_norm_w = pend.norm; a.y_slots = pend.slots; a.y_picks = pend.picks;
       a.x_out = f.taps + (size_t)l * T * H;
       a.rows = f.rows; a.n_rows = T; a.H = H; a.dim = c.hidden_true; a.eps = c.eps; a.dtype = c.dtype;
       rc = rf_stream_norm(&a, st);
@@ -571,7 +601,8 @@ extern "C" int64_t rf_mixed_create(const RfMixedConfig* c) {
   if (!c || c->layers <= 0 || c->hidden <= 0 || c->hidden % 8 || c->hidden_true <= 0 || c->hidden_true > c->hidden || c->vocab <= 0 ||
       c->vocab_ld < c->vocab || c->vocab_ld % 8 || c->dtype < 0 || c->dtype > 2 || c->max_tokens <= 0 || c->max_seqs <= 0 ||
       c->max_seq_len <= 0 || c->side_dim < 0 || c->side_dim % 8 || !c->embed || !c->final_norm || !c->w_lm || c->long_min < 1 ||
-      (c->dtype == kF32 && c->weights_packed)) {
+      (c->dtype == kF32 && c->weights_packed) || c->logit_softcap < 0.f ||
+      (c->pair_table && (c->pair_buckets <= 0 || c->pair_mul_prev < 0 || c->pair_mul_cur < 0))) {
     fail(RF_ERR_BAD_ARG, "invalid mixed-stack config");
     return -1;
   }
@@ -594,13 +625,16 @@ extern "C" int rf_mixed_set_layer(int64_t h, int32_t layer, const RfMixedLayer* 
     RF_REQUIRE(w->out_dim == w->heads * w->vdim, "layer %d: output projection columns", layer);
   }
   RF_REQUIRE(w->norm1 && w->w_in && w->w_o && (!w->shift || w->st.shift_state), "layer %d: missing weights", layer);
-  if (w->inter > 0) RF_REQUIRE(w->norm2 && w->w_up && w->w_down && w->act == RF_MIXED_ACT_RELU2, "layer %d: feed-forward weights", layer);
+  if (w->inter > 0) RF_REQUIRE(w->norm2 && w->w_up && w->w_down && (w->act == RF_MIXED_ACT_RELU2 || (w->act == RF_MIXED_ACT_CLIPPED_GLU && w->act_limit > 0.f)),
+                                 "layer %d: feed-forward weights", layer);
+  if (s.cfg.pair_table) RF_REQUIRE(w->st.last_token && !w->shift, "layer %d: token pairs need the carried tokens and no token shift", layer);
   if (w->experts > 0) {
     RF_REQUIRE(w->inter > 0 && w->router && w->experts <= 256 && w->top > 0 && w->top <= 32 && w->groups > 0 && w->experts % w->groups == 0 &&
                    w->keep > 0 && w->keep <= w->groups && w->top <= w->experts / w->groups * w->keep,
                "layer %d: %d experts in %d groups, %d kept, %d chosen", layer, w->experts, w->groups, w->keep, w->top);
     RF_REQUIRE(w->bank_inter >= w->inter && w->bank_inter % (s.cfg.dtype == kF32 ? 8 : 128) == 0 && w->shared_inter >= 0 && w->shared_inter % 8 == 0 &&
-                   (w->shared_inter == 0 || (w->shared_up && w->shared_down)), "layer %d: expert widths", layer);
+                   (w->shared_inter == 0 || (w->shared_up && w->shared_down)) && (!w->shared_gate || w->shared_inter > 0) &&
+                   (w->act != RF_MIXED_ACT_CLIPPED_GLU || w->shared_inter == 0 || w->shared_limit > 0.f), "layer %d: expert widths", layer);
     RF_REQUIRE(s.cfg.dtype == kF32 || s.cfg.weights_packed, "layer %d: experts need tile-major weights", layer);
   }
   if (w->mixer == RF_MIXER_LATENT_ATTENTION) {
@@ -612,7 +646,9 @@ extern "C" int rf_mixed_set_layer(int64_t h, int32_t layer, const RfMixedLayer* 
   } else if (w->mixer == RF_MIXER_ATTENTION) {
     RF_REQUIRE(w->dim == w->vdim && w->kv_heads > 0 && w->heads % w->kv_heads == 0 && w->dim_true > 0 && w->dim_true <= w->dim &&
                    w->vdim_true > 0 && w->vdim_true <= w->vdim && w->st.k_pool && w->st.v_pool && w->st.pool_pages > 0, "layer %d: attention", layer);
-    RF_REQUIRE(w->in_dim >= ((w->gated ? 2 : 1) * w->heads + 2 * w->kv_heads) * w->dim, "layer %d: input projection rows", layer);
+    RF_REQUIRE(w->in_dim >= (w->heads + 2 * w->kv_heads) * w->dim + (w->gated ? w->heads * (w->gate_by_head ? 1 : w->dim) : 0), "layer %d: input projection rows", layer);
+    RF_REQUIRE(w->conv_taps >= 0 && (w->conv_taps == 0 || (w->conv_w && !w->norm_all && (w->conv_taps == 1 || w->st.conv_state))) && w->keep_first >= 0,
+               "layer %d: convolution of %d taps, %d kept positions", layer, w->conv_taps, w->keep_first);
     RF_REQUIRE(!w->tensor_core || (s.cfg.dtype != kF32 && (w->dim == 64 || w->dim == 128 || w->dim == 256) && w->scale > 0.f), "layer %d: heads", layer);
     RF_REQUIRE(w->rot_dims % 2 == 0 && w->rot_dims >= 0 && w->rot_dims <= w->dim_true && (w->rot_dims == 0 || (w->cos && w->sin)), "layer %d: rotation", layer);
   } else if (w->mixer == RF_MIXER_MAMBA1) {
@@ -691,13 +727,15 @@ extern "C" int rf_mixed_head(int64_t h, const int32_t* row_idx, int32_t rows, in
   RF_REQUIRE(rows > 0 && rows <= std::max(c.max_seqs, 64), "head rows %d (max %d)", rows, std::max(c.max_seqs, 64));
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   RfStreamNorm a = {};
-  a.x = s.at<float>(s.off_x[s.cur]); a.row_idx = row_idx;
+  a.x = s.at<float>(s.off_x[s.cur]); a.row_idx = row_idx; a.y_mult = c.residual_mult;
   a.y = s.tail.y; a.y_norm_w = s.tail.norm; a.y_slots = s.tail.slots; a.y_picks = s.tail.picks;
   a.norm_w = c.final_norm; a.out = s.at(s.off_head);
   a.n_rows = rows; a.H = c.hidden; a.dim = c.hidden_true; a.eps = c.eps; a.dtype = c.dtype;
   int rc = rf_stream_norm(&a, st);
   if (rc) return rc;
-  rc = linear(s, s.at(s.off_head), c.hidden, c.w_lm, logits, c.vocab_ld, rows, c.vocab_ld, c.hidden, kActNone, st);
+  RfGemm g = gemm_args(s, s.at(s.off_head), c.hidden, c.w_lm, logits, c.vocab_ld, rows, c.vocab_ld, c.hidden, c.logit_softcap > 0.f ? kActSoftCap : kActNone);
+  g.act_limit = c.logit_softcap;
+  rc = s.fp32() ? rf_gemm_f32(&g, st) : rf_gemm(&g, st);
   if (rc) return rc;
   if (out_ids)
     rc = rf_argmax(logits, rows, c.vocab, c.vocab_ld, out_ids, out_vals, 0, s.at(s.off_argmax), s.argmax_bytes, c.dtype, st);

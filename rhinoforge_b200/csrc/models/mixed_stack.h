@@ -1,8 +1,9 @@
 // Decoder stack whose layers differ: every layer names its own mixer (latent attention with a sliding window, HGRN2 linear
-// attention, grouped-head attention with chunks and sinks, a selective scan), sizes and feed-forward (dense or a mixture of
-// experts), and the stack adds what such designs share: an fp32 residual stream, norms in front of the sublayers or on their
-// outputs, a token shift in front of every mixer and a gated per-token side input behind every layer (both optional).  Activations are fp16 / bf16, or fp32
-// throughout (dtype 2).  Like rf_stack_* one handle owns the weight pointers and a static arena and enqueues the whole layer
+// attention, grouped-head attention with chunks or windows, sinks, distance slopes and convolved projections, a selective scan),
+// sizes and feed-forward (dense or a mixture of experts), and the stack adds what such designs share: an fp32 residual stream, an
+// embedding of token pairs, norms in front of the sublayers or on their outputs, a factor on those outputs, a token shift in front
+// of every mixer, a gated per-token side input behind every layer and a soft cap of the logits (all optional).  Activations are
+// fp16 / bf16, or fp32 throughout (dtype 2).  Like rf_stack_* one handle owns the weight pointers and a static arena and enqueues the whole layer
 // loop on a stream, so a decode step can be captured into a CUDA graph.
 #pragma once
 #include <stdint.h>
@@ -14,7 +15,7 @@ extern "C" {
 #endif
 
 enum RfMixerKind { RF_MIXER_LATENT_ATTENTION = 0, RF_MIXER_HGRN2 = 1, RF_MIXER_ATTENTION = 2, RF_MIXER_MAMBA1 = 3 };
-enum RfMixedAct { RF_MIXED_ACT_RELU2 = 0 };
+enum RfMixedAct { RF_MIXED_ACT_RELU2 = 0, RF_MIXED_ACT_CLIPPED_GLU = 1 };   // dense feed-forward; experts: 0 is silu(gate) * up
 
 typedef struct RfMixedConfig {
   int32_t layers;
@@ -33,6 +34,11 @@ typedef struct RfMixedConfig {
   const void* w_lm;              // [vocab_ld, hidden]
   float embed_scale;
   int32_t norm_after;            // 0: sublayers read the normalised stream; 1: they read the stream, norms act on their outputs
+  float residual_mult;           // factor of the sublayers' outputs (0 counts as 1)
+  float logit_softcap;           // logits <- cap * tanh(logits / cap) (0: none)
+  const void* pair_table;        // [pair_buckets + 1, hidden]: embedding of (previous token, token), see RfStreamNorm (null: none)
+  int64_t pair_mul_prev, pair_mul_cur;
+  int32_t pair_buckets;
 } RfMixedConfig;
 
 // Per-sequence memory of a layer; what a layer does not use is null.
@@ -41,17 +47,18 @@ typedef struct RfMixedState {
   void* k_pool; void* v_pool;           // [pages, kv_heads, 16, head size]
   int64_t pool_pages;
   float* rec_state;                     // HGRN2: [slots, heads, dim, vdim]; scan: [slots, inner, states]
-  void* conv_state;                     // [slots, taps - 1, inner]
+  void* conv_state;                     // [slots, taps - 1, inner] or [slots, taps - 1, (heads + 2 kv_heads) * dim]
   float* shift_state;                   // [slots, hidden]
+  int32_t* last_token;                  // [slots], one array for the whole stack
 } RfMixedState;
 
 // Padded sizes: per-head sizes and ranks are multiples of 8 / 16 with zero rows behind the true ones.
 typedef struct RfMixedLayer {
   int32_t mixer, heads, dim, vdim, vdim_true;
-  int32_t rank, rank_true, window;      // latent attention; window <= 0: unlimited
+  int32_t rank, rank_true, window;      // attention: window <= 0: unlimited
   int32_t expand_hd;                    // 64 / 128 / 256: portions expand K and V to heads of this size (== dim == vdim)
   int32_t inter;                        // 0: the layer has no feed-forward
-  int32_t act;                          // RfMixedAct
+  int32_t act;                          // RfMixedAct (clipped GLU: w_up holds gate rows, then up rows)
   float scale;
   int32_t in_dim;                       // rows of w_in: [q | latent], [q | f | v], [q | k | v | gate] or [x | z]
   int32_t out_dim;                      // columns of w_o
@@ -72,6 +79,11 @@ typedef struct RfMixedLayer {
   float v_lambda;
   const float* cos; const float* sin;   // [positions, rot_dims / 2]
   const float* q_norm; const float* k_norm; const float* sink;
+  int32_t keep_first;                   // with a window or chunk: first positions that stay visible
+  int32_t norm_all;                     // one norm over all query heads and one over all key heads (weights [heads, dim])
+  int32_t gate_by_head;                 // with `gated`: one gate number per head
+  int32_t conv_taps;                    // > 0: causal convolution of queries, keys and values (conv_w [taps, (heads + 2 kv_heads) * dim])
+  const float* slopes;                  // [heads]: what scores lose per token of distance
   // selective scan
   int32_t inner, states, dt_rank, taps;
   const float* conv_w; const float* conv_b; const float* a2; const float* d_skip; const float* dt_bias;
@@ -82,6 +94,8 @@ typedef struct RfMixedLayer {
   int32_t bank_inter;                   // inter padded to the bank's granularity (128 in 16 bits)
   float route_scale;
   const void* router; const float* correction; const void* shared_up; const void* shared_down;
+  float act_limit, act_alpha, shared_limit;   // constants of the clipped GLU
+  int32_t shared_gate;                  // the router holds one more row: the logit of the shared expert's weight
   RfMixedState st;
 } RfMixedLayer;
 

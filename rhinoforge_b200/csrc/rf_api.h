@@ -99,6 +99,7 @@ typedef struct RfGemm {
   // Gate by token (shapes for which rf_gemm_takes_mul returns 1): the activated result of row m, column n is multiplied by
   // mul[mul_row[m] * mul_ld + n] (same dtype), a slice of an embedding table.
   const void* mul; const int32_t* mul_row; int64_t mul_ld;
+  float act_limit, act_alpha;  // constants of the activations that have some (rf::ActArgs)
 } RfGemm;
 // bytes of the tile-major image of a [rows, K] weight with `sections` equal row sections
 uint64_t rf_pack_weight_bytes(int64_t rows, int64_t K, int32_t sections, int32_t elem_bytes);
@@ -256,6 +257,9 @@ typedef struct RfAttn {
   int32_t chunk;            // > 0: position i sees j only if i / chunk == j / chunk (positions count from the sequence's start)
   const float* sink;        // [Hq]: the softmax denominator also holds exp(sink[h])
   const void* gate; int64_t ld_gate;   // [rows, Hq * hd]: the result is multiplied by sigmoid(gate) before it is rounded
+  int32_t gate_by_head;     // 1: gate is [rows, Hq], one number per head
+  int32_t keep_first;       // with a window: the first keep_first positions of the sequence stay visible
+  const float* slopes;      // [Hq]: slopes[h] * (i - j) is taken off the scores of position i (paged forms)
   // rf_attn_decode by row: with `pos`, query row r is position pos[r] of sequence seq_of_row[r] (null: r) and sees everything
   // up to itself; kv_len is not used and num_seqs counts rows.
   const int32_t* seq_of_row; const int32_t* pos;
@@ -325,7 +329,10 @@ typedef struct RfRows {
 //   x_out = v (fp32), x_cast = v (activation dtype)
 //   h = v / rms(v) * norm_w;  with `shift`: out = h + (h_prev - h) * shift, h_prev the h of the sequence's previous token
 //   (carried over launches in shift_state[slot], zeros before the first token); without: out = h.
-// Embedding rows are multiplied by embed_scale (0 counts as 1).  With y_picks > 0 the outstanding output is the sum of y_picks rows of y, those
+// Embedding rows are multiplied by embed_scale (0 counts as 1); with table2 the row of the token pair (previous token, token) is
+// added to them: (previous * mul_prev + token * mul_cur) mod buckets, row `buckets` for a sequence's first token; last_token [slots]
+// carries every sequence's last token (not together with `shift`).  The outstanding output is multiplied by y_mult (0 counts as 1)
+// when it is added.  With y_picks > 0 the outstanding output is the sum of y_picks rows of y, those
 // that y_slots[row * y_picks ...] names (negative: none): the experts' results of a mixture of experts.
 // H is the (padded, multiple of 8) row length, dim the true one that the means run over.  x_out must not alias x when
 // `shift` is set.  row_idx (optional) selects the rows that are processed (not together with shift).
@@ -339,11 +346,13 @@ typedef struct RfStreamNorm {
   int32_t n_rows, H, dim; float eps; int32_t dtype;    // dtype 2: fp32 activations
   float embed_scale;
   const int32_t* y_slots; int32_t y_picks;
+  float y_mult;
+  const void* table2; int32_t* last_token; int64_t mul_prev, mul_cur; int32_t buckets;
 } RfStreamNorm;
 int rf_stream_norm(const RfStreamNorm* a, rf_stream_t stream);
 
 // out[M, N] = act(x[M, K] . w[N, K]^T) in true fp32 (row-major operands, no tensor cores): the linear layers of a model that
-// is served in 32 bits.  Uses x, w, out, their pitches, M, N, K and act of RfGemm.
+// is served in 32 bits.  Uses x, w, out, their pitches, M, N, K, row_scale, dual_offset and act (with its constants) of RfGemm.
 int rf_gemm_f32(const RfGemm* g, rf_stream_t stream);
 
 // g[r, c] *= table[ids[r] * ld_table + col0 + c] for c < cols (a gate multiplied by a per-token embedding slice)
@@ -402,10 +411,16 @@ typedef struct RfQkvInsert {
   void* v_first; void* k_pool; void* v_pool;
   RfRows rows;
   int32_t n_rows, heads, kv_heads, hd, dim, vdim, rot_dims, v_role; float v_lambda, eps; int32_t dtype;
+  int32_t norm_all;                    // 1: one RMSNorm over all query heads of a row and one over all key heads; q_norm [heads, hd],
+                                       // k_norm [kv_heads, hd] (per-head norms: [hd])
+  // Causal convolution per channel of queries, keys and values ahead of the norms: y[t] = sum_k w[k] x[t - (taps - 1) + k].  The last
+  // taps - 1 rows of [queries | keys | values] are carried in conv_state [slots, taps - 1, (heads + 2 kv_heads) * hd], oldest first.
+  // conv_w: [taps, (heads + 2 kv_heads) * hd].  The rows are read only, queries go to q_out [n_rows, heads * hd].
+  const float* conv_w; void* conv_state; void* q_out; int32_t taps, max_q_len;
 } RfQkvInsert;
 int rf_qkv_insert(const RfQkvInsert* a, rf_stream_t stream);
 // Attention by row on the CUDA cores in fp32, any head size up to 2048 and any scale: the by-row form of rf_attn_decode (pos,
-// seq_of_row, slot, chunk, sink, gate) for 32-bit models and heads the tensor-core kernels do not take.
+// seq_of_row, slot, chunk, window, sink, gate, slopes) for 32-bit models and heads the tensor-core kernels do not take.
 int rf_attn_rows(const RfAttn* a, rf_stream_t stream);
 
 // Causal convolution per channel over packed rows, silu applied: y[t] = silu(bias + sum_k w[k] x[t - (taps - 1) + k]).  The last
@@ -482,6 +497,7 @@ typedef struct RfMoeGroupedGemm {
   int32_t bank_kb_total;               // 64-column k blocks of one row tile of the bank image
   int32_t rt_per_expert, kb_per_expert;
   int32_t dtype; int32_t* status;
+  float act_limit, act_alpha;          // rf::ActArgs
 } RfMoeGroupedGemm;
 int rf_moe_grouped_gemm(const RfMoeGroupedGemm* a, rf_stream_t stream);
 // Bucket the picks by expert.  ids / w: [rows, k] (rf_moe_select).  Outputs (device): slot_of [rows*k] = sorted row
@@ -503,14 +519,17 @@ int rf_moe_combine(void* out, int64_t ldo, const void* y, int64_t ldy, const int
 // [rows * k, rows * k + rows)).  With `scatter` (few rows) also
 // what rf_moe_gather otherwise writes: slot_of [rows, slot_ld] (sorted row of every pick, then of the shared expert),
 // token_of_slot and slot_w.  counters: experts + 1 words, zero before the first launch and left zero.
-enum RfMoeScore { RF_MOE_SIGMOID = 0, RF_MOE_SOFTMAX = 1 };
+// RF_MOE_CHOSEN: the correction is a bias of the logits; the k largest logits are chosen and the weights are the softmax over the
+// chosen ones.  shared_gate: w has one more row behind the experts', sigmoid of its logit is the shared expert's weight (else 1).
+enum RfMoeScore { RF_MOE_SIGMOID = 0, RF_MOE_SOFTMAX = 1, RF_MOE_CHOSEN = 2 };
 typedef struct RfMoeRouter {
   const void* x; int64_t ldx; const void* w; const float* correction;
   int32_t* ids; float* weights; int32_t* rank; int32_t* counters; int32_t* start; int32_t* tiles;
   int32_t* slot_of; int32_t* token_of_slot; float* slot_w;
   int32_t rows, experts, width, k, groups, keep, score_fn, norm_topk; float scale;
   int32_t tile_rows, slot_ld, has_shared, shared_tiles, scatter, dtype;
-  float* logits;                       // scratch, rf_moe_router_scratch_bytes
+  float* logits;                       // scratch, rf_moe_router_scratch_bytes(rows, experts + shared_gate)
+  int32_t shared_gate;
 } RfMoeRouter;
 uint64_t rf_moe_router_scratch_bytes(int rows, int experts);
 int rf_moe_router(const RfMoeRouter* a, rf_stream_t stream);
@@ -526,6 +545,8 @@ typedef struct RfMoeExperts {
   const int32_t* tiles; const int32_t* token_of_slot; const float* slot_w;
   int32_t max_tiles, experts, n, k, shared_n, shared_k, dual, tile_rows;
   int32_t bank_section_row_tiles, bank_kb_total, rt_per_expert, kb_per_expert, shared_section_row_tiles, shared_kb_total, dtype;
+  int32_t act;                         // dual: rf::Act of two operands (0 counts as silu(g) u)
+  float act_limit, act_alpha, shared_limit;   // its constants; the shared expert has a limit of its own
 } RfMoeExperts;
 int rf_moe_experts(const RfMoeExperts* a, rf_stream_t stream);
 

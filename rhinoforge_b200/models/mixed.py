@@ -1,12 +1,13 @@
 """Decoders whose layers name their own mixer: configuration records and weight tables.
 
 A :class:`MixedConfig` is a list of layers, each with one mixer (:class:`LatentAttention`, :class:`HGRN2`,
-:class:`GroupedAttention`, :class:`Mamba1`) and an optional feed-forward (:class:`DenseMLP`, :class:`MoE`), over what the layers
-share: the width of an fp32 residual stream, RMSNorm epsilon, where the norms sit, and optionally a token shift in front of every
-mixer and a gated per-token side input behind every layer.  The native executor is ``csrc/models/mixed_stack.cu``, the engine
+:class:`GroupedAttention`, :class:`Mamba1`) and an optional feed-forward (:class:`DenseMLP`, :class:`ClippedGLU`, :class:`MoE`), over
+what the layers share: the width of an fp32 residual stream, RMSNorm epsilon, where the norms sit, and optionally an embedding of
+token pairs, a factor on the sublayers' outputs, a token shift in front of every mixer, a gated per-token side input behind every
+layer and a soft cap of the logits.  The native executor is ``csrc/models/mixed_stack.cu``, the engine
 :mod:`rhinoforge_b200.runtime.mixed_engine`.
 
-Readers of ``config.json``: :meth:`MixedConfig.from_vabarax`, :meth:`MixedConfig.from_zulopel`.
+Readers of ``config.json``: :meth:`MixedConfig.from_vabarax`, :meth:`MixedConfig.from_zulopel`, :meth:`MixedConfig.from_kuzupel`.
 """
 from __future__ import annotations
 
@@ -76,9 +77,15 @@ class Rotary:
 
 @dataclass(frozen=True)
 class GroupedAttention:
-    """Softmax attention with ``heads // kv_heads`` query heads per key / value head.  ``chunk``: positions see their own chunk of
-    this many positions only (None: everything before them).  ``sink``: one more learned term in every head's softmax denominator.
-    ``v_mix``: values are mixed with those of the first layer that says so.  ``gate``: sigmoid gate on the heads' outputs."""
+    """Softmax attention with ``heads // kv_heads`` query heads per key / value head.
+
+    What a position sees: ``chunk``, its own chunk of this many positions; ``window``, the last this many positions, its own
+    included, and then also the first ``keep_first`` ones (both None: everything before it).  ``distance_bias``: head h's scores
+    lose ``2^(-8 (h + 1) / heads)`` per token of distance.  ``sink``: one more learned term in every head's softmax denominator;
+    ``unit_sink``: that term is exp(0) in every head.  ``v_mix``: values are mixed with those of the first layer that says so.
+    ``qk_norm``: RMSNorm of every query and key head, or with ``norm_all`` one over all query heads and one over all key heads.
+    ``conv`` > 0: causal convolution of this many taps on the projected queries, keys and values.  ``gate``: sigmoid gate on the
+    heads' outputs, element by element, or with ``gate_by_head`` one number per head."""
     heads: int
     kv_heads: int
     dim: int
@@ -90,6 +97,19 @@ class GroupedAttention:
     qk_norm: bool = True
     sink: bool = True
     gate: bool = True
+    window: Optional[int] = None
+    keep_first: int = 0
+    distance_bias: bool = False
+    unit_sink: bool = False
+    norm_all: bool = False
+    conv: int = 0
+    gate_by_head: bool = False
+
+    def slopes(self) -> Optional[torch.Tensor]:
+        """float64 ``[heads]``: what the scores lose per token of distance."""
+        if not self.distance_bias:
+            return None
+        return torch.tensor([2.0 ** (-8.0 * (h + 1) / self.heads) for h in range(self.heads)], dtype=torch.float64)
 
 
 @dataclass(frozen=True)
@@ -108,27 +128,53 @@ class DenseMLP:
 
 
 @dataclass(frozen=True)
+class ClippedGLU:
+    """``down(g sigmoid(alpha g) (u + 1))`` with ``g = min(gate h, limit)`` and ``u = clamp(up h, -limit, limit)``."""
+    ff: int
+    limit: float
+    alpha: float = 1.702
+
+
+@dataclass(frozen=True)
 class MoE:
-    """``top`` of ``experts`` SwiGLU experts of width ``ff`` per token, chosen among the ``keep`` best of ``groups`` groups by
-    softmax score plus correction and weighted by normalised score; ``shared_ff`` > 0: one more expert that every token uses."""
+    """``top`` of ``experts`` gated experts of width ``ff`` per token; ``shared_ff`` > 0: one more expert that every token uses.
+
+    ``router`` "corrected": chosen among the ``keep`` best of ``groups`` groups by softmax score plus correction, weighted by
+    normalised score.  "chosen": the logits have a bias, the largest are chosen, weights are the softmax over the chosen ones.
+    ``limit``: experts are clipped (:class:`ClippedGLU`), the shared one with ``shared_limit``; None: SwiGLU.  ``shared_gate``: the
+    shared expert is weighted by a sigmoid of one number per token."""
     experts: int
     top: int
     ff: int
     groups: int = 1
     keep: int = 1
     shared_ff: int = 0
+    router: str = "corrected"
+    limit: Optional[float] = None
+    shared_limit: Optional[float] = None
+    alpha: float = 1.702
+    shared_gate: bool = False
+
+
+@dataclass(frozen=True)
+class TokenPairs:
+    """Embedding row of (previous token, token): ``(previous * mul_prev + token * mul_cur) % buckets``, row ``buckets`` for a
+    sequence's first token."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
 
 
 @dataclass(frozen=True)
 class MixedLayer:
     mixer: Union[LatentAttention, HGRN2, GroupedAttention, Mamba1]
-    mlp: Optional[Union[DenseMLP, MoE]] = None
+    mlp: Optional[Union[DenseMLP, ClippedGLU, MoE]] = None
 
 
-def _int(d: Mapping[str, Any], key: str, where: str) -> int:
+def _int(d: Mapping[str, Any], key: str, where: str, least: int = 1) -> int:
     v = d.get(key)
-    if isinstance(v, bool) or not isinstance(v, int) or v <= 0:
-        raise UnsupportedModelError(f"{where}: {key!r} must be a positive integer, got {v!r}")
+    if isinstance(v, bool) or not isinstance(v, int) or v < least:
+        raise UnsupportedModelError(f"{where}: {key!r} must be an integer of at least {least}, got {v!r}")
     return v
 
 
@@ -165,6 +211,9 @@ class MixedConfig:
     layer_scale: bool = False      # element-wise factors on the sublayers' outputs
     tied_head: bool = True
     embed_scale: float = 1.0
+    pairs: Optional[TokenPairs] = None     # embedding of token pairs, added to the tokens' own
+    residual_mult: float = 1.0             # factor of the sublayers' outputs
+    logit_softcap: Optional[float] = None  # logits <- cap * tanh(logits / cap)
     model_type: str = "vabarax"
     raw: Optional[Mapping[str, Any]] = field(default=None, compare=False, repr=False)
 
@@ -272,6 +321,72 @@ class MixedConfig:
         return {"architecture": "Zulopel", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.rms_eps},
                 "embedding": {"scale": self.embed_scale}, "layers": out}
 
+    @classmethod
+    def kuzupel(cls, name: str, vocab: int, width: int, eps: float, layers, *, pairs: Optional[TokenPairs] = None, embed_scale: float = 1.0,
+                residual_mult: float = 1.0, logit_softcap: Optional[float] = None, **kw) -> "MixedConfig":
+        """A decoder of the Kuzupel design: distance-biased and rotary window attention in any order, clipped gated feed-forwards or
+        mixtures of them, an embedding of token pairs, an untied head with a soft cap."""
+        return cls(name, vocab, width, eps, tuple(layers), 0, token_shift=False, tied_head=False, embed_scale=embed_scale, pairs=pairs,
+                   residual_mult=residual_mult, logit_softcap=logit_softcap, model_type="kuzupel", **kw)
+
+    @classmethod
+    def from_kuzupel(cls, c: Mapping[str, Any]) -> "MixedConfig":
+        """The mapping of a Kuzupel ``config.json``.  Keys that the reader does not know are refused rather than ignored."""
+        _known(c, ("architecture", "embedding", "layers", "logit_softcap", "norm", "residual_mult", "vocab", "width"), "Kuzupel")
+        if not isinstance(c.get("layers"), list) or not c["layers"]:
+            raise UnsupportedModelError("Kuzupel: 'layers' must be a non-empty list")
+        layers = []
+        for i, entry in enumerate(c["layers"]):
+            where = f"Kuzupel layer {i}"
+            if not isinstance(entry, Mapping):
+                raise UnsupportedModelError(f"{where}: must be a mapping")
+            _known(entry, ("type", "mixer", "mlp"), where)
+            read = {"attention": _kuzupel_biased, "attention_2": _kuzupel_rotary}.get(entry.get("type"))
+            if read is None:
+                raise UnsupportedModelError(f"{where}: mixer type {entry.get('type')!r} is not built")
+            mlp = None if entry.get("mlp") is None else _kuzupel_mlp(_map(entry, "mlp", where), where + " mlp")
+            layers.append(MixedLayer(read(_map(entry, "mixer", where), where), mlp))
+        norm, emb, pairs = _map(c, "norm", "Kuzupel"), c.get("embedding") or {}, None
+        _known(norm, ("eps",), "Kuzupel norm")
+        _known(emb, ("scale", "bigram"), "Kuzupel embedding")
+        if emb.get("bigram") is not None:
+            b, w = _map(emb, "bigram", "Kuzupel embedding"), "Kuzupel bigram"
+            _known(b, ("buckets", "mul_prev", "mul_cur"), w)
+            pairs = TokenPairs(_int(b, "buckets", w), _int(b, "mul_prev", w, 0), _int(b, "mul_cur", w, 0))
+        number = lambda d, key, default, where: default if d.get(key) is None else _float(d, key, where, True)
+        cap = c.get("logit_softcap")
+        return cls.kuzupel("kuzupel", _int(c, "vocab", "Kuzupel"), _int(c, "width", "Kuzupel"), _float(norm, "eps", "Kuzupel norm"), layers,
+                           pairs=pairs, embed_scale=number(emb, "scale", 1.0, "Kuzupel embedding"),
+                           residual_mult=number(c, "residual_mult", 1.0, "Kuzupel"),
+                           logit_softcap=None if cap is None else _float(c, "logit_softcap", "Kuzupel", True), raw=c)
+
+    def to_kuzupel(self) -> Dict[str, Any]:
+        """The inverse of :meth:`from_kuzupel`."""
+        out = []
+        for layer in self.layers:
+            m, f = layer.mixer, layer.mlp
+            d: Dict[str, Any] = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale}
+            if m.window is not None:
+                d["mask"] = {"size": m.window} if m.distance_bias else {"size": m.window, "keep_first": m.keep_first}
+            if not m.distance_bias:
+                d["conv"] = m.conv
+                if m.rot is not None:
+                    d["rot"] = {"dims": m.rot.dims, "base": m.rot.base}
+            mlp: Optional[Dict[str, Any]] = None
+            if isinstance(f, MoE):
+                mlp = {"kind": "moe", "expert": {"ff": f.ff, "limit": f.limit}, "router": {"experts": f.experts, "top": f.top}}
+                if f.shared_ff:
+                    mlp["shared"] = {"ff": f.shared_ff, "limit": f.shared_limit}
+            elif f is not None:
+                mlp = {"kind": "dense", "ff": f.ff, "limit": f.limit}
+            out.append({"type": "attention" if m.distance_bias else "attention_2", "mixer": d, "mlp": mlp})
+        emb: Dict[str, Any] = {"scale": self.embed_scale}
+        if self.pairs is not None:
+            emb["bigram"] = {"buckets": self.pairs.buckets, "mul_prev": self.pairs.mul_prev, "mul_cur": self.pairs.mul_cur}
+        top = {"architecture": "Kuzupel", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.rms_eps},
+               "embedding": emb, "residual_mult": self.residual_mult, "layers": out}
+        return top if self.logit_softcap is None else {**top, "logit_softcap": self.logit_softcap}
+
     def to_vabarax(self) -> Dict[str, Any]:
         """The inverse of :meth:`from_vabarax`."""
         out = []
@@ -331,11 +446,59 @@ def _zulopel_experts(f: Mapping[str, Any], where: str) -> MoE:
     return e
 
 
+def _kuzupel_sizes(m: Mapping[str, Any], where: str, keys, mask_keys) -> Dict[str, Any]:
+    _known(m, ("heads", "kv_heads", "dim", "vdim", "scale", "mask") + keys, where)
+    mask = m.get("mask") or {}
+    _known(mask, mask_keys, where + " mask")
+    a = {k: _int(m, k, where) for k in ("heads", "kv_heads", "dim", "vdim")}
+    if a["heads"] % a["kv_heads"]:
+        raise UnsupportedModelError(f"{where}: {a['heads']} heads do not share {a['kv_heads']} key / value heads evenly")
+    a.update(scale=_float(m, "scale", where), sink=False, window=_int(mask, "size", where + " mask") if mask else None)
+    return a
+
+
+def _kuzupel_biased(m: Mapping[str, Any], where: str) -> GroupedAttention:
+    return GroupedAttention(**_kuzupel_sizes(m, where, (), ("size",)), gate=False, distance_bias=True, norm_all=True)
+
+
+def _kuzupel_rotary(m: Mapping[str, Any], where: str) -> GroupedAttention:
+    a = _kuzupel_sizes(m, where, ("conv", "rot"), ("size", "keep_first"))
+    mask, rot = m.get("mask") or {}, None
+    if m.get("rot"):
+        r, w = _map(m, "rot", where), where + " rot"
+        _known(r, ("dims", "base"), w)
+        rot = Rotary(_int(r, "dims", w), _float(r, "base", w, True))
+        if rot.dims % 2 or rot.dims > a["dim"]:
+            raise UnsupportedModelError(f"{where}: rotation of {rot.dims} of {a['dim']} dimensions")
+    return GroupedAttention(**a, rot=rot, unit_sink=True, gate_by_head=True, conv=_int(m, "conv", where),
+                            keep_first=_int(mask, "keep_first", where + " mask", 0) if "keep_first" in mask else 0)
+
+
+def _kuzupel_mlp(f: Mapping[str, Any], where: str) -> Union[ClippedGLU, MoE]:
+    if f.get("kind") == "dense":
+        _known(f, ("kind", "ff", "limit"), where)
+        return ClippedGLU(_int(f, "ff", where), _float(f, "limit", where, True))
+    if f.get("kind") != "moe":
+        raise UnsupportedModelError(f"{where}: feed-forward kind {f.get('kind')!r} is not built")
+    _known(f, ("kind", "expert", "router", "shared"), where)
+    expert, r, shared = _map(f, "expert", where), _map(f, "router", where), f.get("shared") or {}
+    for d, keys, what in ((expert, ("ff", "limit"), " expert"), (r, ("experts", "top"), " router"), (shared, ("ff", "limit"), " shared")):
+        _known(d, keys, where + what)
+    e = MoE(_int(r, "experts", where), _int(r, "top", where), _int(expert, "ff", where), router="chosen",
+            limit=_float(expert, "limit", where + " expert", True), shared_ff=_int(shared, "ff", where + " shared") if shared else 0,
+            shared_limit=_float(shared, "limit", where + " shared", True) if shared else None, shared_gate=bool(shared))
+    if e.top > e.experts or e.experts > 256 or e.top > 32:
+        raise UnsupportedModelError(f"{where}: {e.top} of {e.experts} experts (the router takes up to 32 of 256)")
+    return e
+
+
 def weight_shapes(cfg: MixedConfig) -> Iterator[Tuple[str, Tuple[int, ...], str]]:
     """(tensor name, shape, kind) of a checkpoint; kind is 'linear', 'embed', 'norm', 'unit' (values in [0, 1)), 'bias', 'scale'
     (positive factors), 'log_a' (logarithms of decay rates), 'dt_bias' (step sizes before softplus) or 'correction'."""
     H, P = cfg.hidden_size, cfg.side_dim
     yield "embed", (cfg.vocab_size, H), "embed"
+    if cfg.pairs is not None:
+        yield "bigram", (cfg.pairs.buckets + 1, H), "embed"
     if P:
         yield "side.embed", (cfg.vocab_size, cfg.num_layers * P), "embed"
     for i, layer in enumerate(cfg.layers):
@@ -360,14 +523,17 @@ def weight_shapes(cfg: MixedConfig) -> Iterator[Tuple[str, Tuple[int, ...], str]
             yield p + "mix.k", (m.kv_heads * m.dim, H), "linear"
             yield p + "mix.v", (m.kv_heads * m.vdim, H), "linear"
             if m.qk_norm:
-                yield p + "mix.q.norm", (m.dim,), "norm"
-                yield p + "mix.k.norm", (m.dim,), "norm"
+                yield p + "mix.q.norm", (qd if m.norm_all else m.dim,), "norm"
+                yield p + "mix.k.norm", (m.kv_heads * m.dim if m.norm_all else m.dim,), "norm"
+            if m.conv:
+                for name, rows in (("q", qd), ("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim)):
+                    yield f"{p}mix.{name}.conv", (rows, m.conv), "linear"
             if m.v_mix:
                 yield p + "mix.vmix", (), "unit"
             if m.sink:
                 yield p + "mix.sink", (m.heads,), "bias"
             if m.gate:
-                yield p + "mix.g", (vd, H), "linear"
+                yield p + "mix.g", (m.heads if m.gate_by_head else vd, H), "linear"
         elif isinstance(m, LatentAttention):
             yield p + "mix.dkv", (m.kv_rank, H), "linear"
             yield p + "mix.dkv.norm", (m.kv_rank,), "norm"
@@ -389,8 +555,12 @@ def weight_shapes(cfg: MixedConfig) -> Iterator[Tuple[str, Tuple[int, ...], str]
                 yield f"{p}mlp.{e}.up", (ff, H), "linear"
                 yield f"{p}mlp.{e}.down", (H, ff), "linear"
             yield p + "mlp.router", (f.experts, H), "linear"
-            yield p + "mlp.correction", (f.experts,), "correction"
+            yield p + ("mlp.router.b" if f.router == "chosen" else "mlp.correction"), (f.experts,), "bias" if f.router == "chosen" else "correction"
+            if f.shared_gate:
+                yield p + "mlp.shared.sg", (1, H), "linear"
         elif layer.mlp is not None:
+            if isinstance(layer.mlp, ClippedGLU):
+                yield p + "mlp.gate", (layer.mlp.ff, H), "linear"
             yield p + "mlp.up", (layer.mlp.ff, H), "linear"
             yield p + "mlp.down", (H, layer.mlp.ff), "linear"
         if cfg.layer_scale:
@@ -440,5 +610,5 @@ def random_weights(cfg: MixedConfig, *, seed: int = 0, dtype=torch.bfloat16, dev
     return get
 
 
-__all__ = ["MixedConfig", "MixedLayer", "LatentAttention", "HGRN2", "GroupedAttention", "Mamba1", "Rotary", "YarnScaling", "DenseMLP", "MoE",
-           "weight_shapes", "random_weights"]
+__all__ = ["MixedConfig", "MixedLayer", "LatentAttention", "HGRN2", "GroupedAttention", "Mamba1", "Rotary", "YarnScaling", "DenseMLP",
+           "ClippedGLU", "MoE", "TokenPairs", "weight_shapes", "random_weights"]

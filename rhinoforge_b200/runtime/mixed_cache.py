@@ -1,9 +1,9 @@
 """Per-sequence state of decoders with per-layer mixers: paged latent rows or keys and values of the attention layers, fp32
-recurrent states and convolution inputs of the recurrent layers, and the token-shift rows of designs that have them.
+recurrent states, convolution inputs, and the token-shift rows and last tokens of designs that have them.
 
 Latent rows, keys and values live in 16-token pages addressed through the page table of :class:`PagedSequences`; a layer's pool
 is ``[pages, 16, rank]`` (latent) or ``[pages, kv_heads, 16, head size]`` and all layers share the page numbers.  Recurrent,
-convolution and shift state belong to the sequence SLOT: nothing has to be cleared when a slot is given to another request,
+convolution, shift and last-token state belong to the sequence SLOT: nothing has to be cleared when a slot is given to another request,
 because a row at position 0 starts from an empty state in every kernel.
 """
 from __future__ import annotations
@@ -48,7 +48,9 @@ class MixedCache(PagedSequences):
             if isinstance(m, LatentAttention):
                 latent = zeros(self.num_pages, PAGE_TOKENS, pad_to(m.kv_rank, 16))
             elif isinstance(m, GroupedAttention):
-                kv = zeros(2, self.num_pages, m.kv_heads, PAGE_TOKENS, head_layout(m, dtype)[0])
+                hd = head_layout(m, dtype)[0]
+                kv = zeros(2, self.num_pages, m.kv_heads, PAGE_TOKENS, hd)
+                conv = zeros(batch_size, m.conv - 1, (m.heads + 2 * m.kv_heads) * hd) if m.conv > 1 else None
             elif isinstance(m, HGRN2):
                 rec = zeros(batch_size, m.heads, pad_to(m.dim, 8), pad_to(m.vdim, 8), dt=torch.float32)
             elif isinstance(m, Mamba1):
@@ -59,6 +61,7 @@ class MixedCache(PagedSequences):
             self.recurrent.append(rec)
             self.conv.append(conv)
         self.shift = zeros(cfg.num_layers, batch_size, pad_to(cfg.hidden_size, 8), dt=torch.float32) if cfg.token_shift else None
+        self.last_token = zeros(batch_size, dt=torch.int32) if cfg.pairs is not None else None
 
     def layer_state(self, layer: int) -> N.RfMixedState:
         """Device addresses of one layer's memory; null where it has none."""
@@ -68,11 +71,12 @@ class MixedCache(PagedSequences):
         if self.kv[layer] is not None:
             st.k_pool, st.v_pool, st.pool_pages = self.kv[layer][0].data_ptr(), self.kv[layer][1].data_ptr(), self.num_pages
         st.shift_state = None if self.shift is None else self.shift[layer].data_ptr()
+        st.last_token = None if self.last_token is None else self.last_token.data_ptr()
         return st
 
     def state_tensors(self) -> List[torch.Tensor]:
         """Everything a step advances in place (pages are only ever written at new positions)."""
-        return [t for t in self.recurrent + self.conv + [self.shift] if t is not None]
+        return [t for t in self.recurrent + self.conv + [self.shift, self.last_token] if t is not None]
 
     def _tensors(self) -> List[torch.Tensor]:
         return [t for t in self.latent + self.kv if t is not None] + self.state_tensors()

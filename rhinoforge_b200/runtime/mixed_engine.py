@@ -18,7 +18,7 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from .. import _native as N
-from ..models.mixed import HGRN2, GroupedAttention, LatentAttention, Mamba1, MixedConfig, MoE
+from ..models.mixed import HGRN2, ClippedGLU, GroupedAttention, LatentAttention, Mamba1, MixedConfig, MoE
 from ..ops import kernels as K
 from ..parallel.tp import TPContext
 from .engine import DecoderEngine, WeightGetter
@@ -149,6 +149,11 @@ class MixedDecoderEngine(DecoderEngine):
         sc.embed, sc.final_norm, sc.w_lm = (t.data_ptr() for t in (self.embed, self.final_norm, lm))
         sc.side_table = None if self.side_table is None else self.side_table.data_ptr()
         sc.embed_scale, sc.norm_after = cfg.embed_scale, int(cfg.norm_after)
+        sc.residual_mult, sc.logit_softcap = cfg.residual_mult, cfg.logit_softcap or 0.0
+        if cfg.pairs is not None:
+            b = cfg.pairs
+            sc.pair_table = self._plain(_pad2(g("bigram"), b.buckets + 1, H)).data_ptr()
+            sc.pair_buckets, sc.pair_mul_prev, sc.pair_mul_cur = b.buckets, b.mul_prev, b.mul_cur
         h = lib.rf_mixed_create(C.byref(sc))
         if h < 0:
             N.check(-1, "rf_mixed_create")
@@ -169,6 +174,11 @@ class MixedDecoderEngine(DecoderEngine):
                 lw.norm2 = self._f32(norm("norm2", "ls2"), H).data_ptr()
             if isinstance(layer.mlp, MoE):
                 self._load_moe(lw, layer.mlp, g, p + "mlp.")
+            elif isinstance(layer.mlp, ClippedGLU):
+                f = layer.mlp
+                lw.inter, lw.act, lw.act_limit, lw.act_alpha = pad_to(f.ff, 8), 1, f.limit, f.alpha
+                lw.w_up = self._linear(torch.cat([_pad2(g(f"{p}mlp.{x}"), lw.inter, H) for x in ("gate", "up")], 0), 2).data_ptr()
+                lw.w_down = self._linear(_pad2(g(p + "mlp.down"), H, lw.inter)).data_ptr()
             elif layer.mlp is not None:
                 lw.inter, lw.act = pad_to(layer.mlp.ff, 8), 0
                 lw.w_up = self._linear(_pad2(g(p + "mlp.up"), lw.inter, H)).data_ptr()
@@ -215,18 +225,27 @@ class MixedDecoderEngine(DecoderEngine):
         hd, tensor_core = head_layout(m, self.dtype)
         lw.mixer, lw.dim, lw.vdim, lw.dim_true, lw.vdim_true = 2, hd, hd, m.dim, m.vdim
         lw.kv_heads, lw.tensor_core, lw.chunk, lw.scale = m.kv_heads, int(tensor_core), m.chunk or 0, m.scale
+        lw.window, lw.keep_first, lw.norm_all, lw.gate_by_head, lw.conv_taps = m.window or 0, m.keep_first, int(m.norm_all), int(m.gate_by_head), m.conv
         rows = lambda name, heads, true: _pad_heads(_pad2(g(p + name), heads * true, H), heads, true, hd)
         parts = [rows("q", m.heads, m.dim), rows("k", m.kv_heads, m.dim), rows("v", m.kv_heads, m.vdim)]
         if m.gate:
-            parts.append(rows("g", m.heads, m.vdim))
+            parts.append(_pad2(g(p + "g"), pad_to(m.heads, 8), H) if m.gate_by_head else rows("g", m.heads, m.vdim))
             lw.gated = 1
         w_in = torch.cat(parts, 0)
         lw.in_dim = w_in.shape[0]
         lw.w_in = self._linear(w_in).data_ptr()
         if m.qk_norm:
-            lw.q_norm, lw.k_norm = self._f32(g(p + "q.norm"), hd).data_ptr(), self._f32(g(p + "k.norm"), hd).data_ptr()
-        if m.sink:
-            lw.sink = self._f32(g(p + "sink"), m.heads).data_ptr()
+            heads = (m.heads, m.kv_heads) if m.norm_all else (1, 1)
+            lw.q_norm, lw.k_norm = (self._f32(_fill_heads(g(p + x).float(), n, m.dim, hd, 0.0), n * hd).data_ptr()
+                                    for x, n in zip(("q.norm", "k.norm"), heads))
+        if m.sink or m.unit_sink:
+            lw.sink = self._f32(g(p + "sink") if m.sink else torch.zeros(m.heads), m.heads).data_ptr()
+        if m.distance_bias:
+            lw.slopes = self._f32(m.slopes(), m.heads).data_ptr()
+        if m.conv:
+            taps = torch.cat([_pad_heads(g(f"{p}{x}.conv").float(), n, d, hd)
+                              for x, n, d in (("q", m.heads, m.dim), ("k", m.kv_heads, m.dim), ("v", m.kv_heads, m.vdim))], 0)
+            lw.conv_w = self._f32(taps.t().contiguous(), taps.numel()).data_ptr()
         if m.rot is not None:
             cos, sin = self._rotation(m.rot)
             lw.rot_dims, lw.cos, lw.sin = m.rot.dims, cos.data_ptr(), sin.data_ptr()
@@ -262,7 +281,9 @@ class MixedDecoderEngine(DecoderEngine):
         B = I if self.fp32 else pad_to(f.ff, 128)
         lw.inter, lw.bank_inter, lw.act = I, B, 0
         lw.experts, lw.top, lw.groups, lw.keep = f.experts, f.top, f.groups, f.keep
-        lw.score_fn, lw.norm_topk, lw.route_scale = 1, 1, 1.0
+        lw.score_fn, lw.norm_topk, lw.route_scale = {"corrected": 1, "chosen": 2}[f.router], 1, 1.0
+        if f.limit is not None:
+            lw.act, lw.act_limit, lw.act_alpha, lw.shared_limit = 1, f.limit, f.alpha, f.shared_limit or 0.0
         up = torch.zeros((2, f.experts, B, H), dtype=self.dtype, device=self.device)
         down = torch.zeros((f.experts, H, B), dtype=self.dtype, device=self.device)
         for e in range(f.experts):
@@ -273,8 +294,11 @@ class MixedDecoderEngine(DecoderEngine):
             down[e, :w.shape[0], :f.ff] = w
         lw.w_up = self._linear(up.view(2 * f.experts * B, H), 2).data_ptr()
         lw.w_down = self._linear(down.view(f.experts * H, B) if self.fp32 else down.transpose(0, 1).reshape(H, f.experts * B)).data_ptr()
-        lw.router = self._plain(_pad2(g(p + "router"), f.experts, H)).data_ptr()
-        lw.correction = self._f32(g(p + "correction"), f.experts).data_ptr()
+        router = _pad2(g(p + "router"), f.experts, H)
+        if f.shared_gate:
+            router, lw.shared_gate = torch.cat((router, _pad2(g(p + "shared.sg"), 1, H)), 0), 1
+        lw.router = self._plain(router).data_ptr()
+        lw.correction = self._f32(g(p + ("router.b" if f.router == "chosen" else "correction")), f.experts).data_ptr()
         if f.shared_ff:
             S = lw.shared_inter = pad_to(f.shared_ff, 8)
             gate_up = torch.cat((_pad2(g(p + "shared.gate"), S, H), _pad2(g(p + "shared.up"), S, H)), 0)
