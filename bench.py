@@ -29,11 +29,12 @@ def parse_args(argv=None):
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="decode", choices=["decode", "pi05", "qwen3vl", "vabarax", "zulopel"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "pi05", "qwen3vl", "vabarax", "zulopel", "kuzupel"],
                     help="decode: causal-LM decode throughput (headline); pi05: action-chunk latency; "
                          "qwen3vl: multimodal prefill + decode; vabarax: latent-attention / HGRN2 decoder, zulopel: chunked "
                          "attention / selective-scan decoder with routed experts, each beside the hybrid K/V + "
-                         "Gated-DeltaNet decoder at equal size")
+                         "Gated-DeltaNet decoder at equal size; kuzupel: window-attention decoder with clipped feed-forwards, "
+                         "beside a Zulopel decoder of attention layers")
     ap.add_argument("--model", default="qwen3-8b")
     ap.add_argument("--batch", type=int, default=64)
     ap.add_argument("--prompt-len", type=int, default=1024)
@@ -552,6 +553,14 @@ ZULOPEL_SIZES = {          # width, heads (of 128), K/V heads, chunk, scan chann
 }
 
 
+KUZUPEL_SIZES = {          # width, heads (of 128), K/V heads, window of the biased layers, of the rotary ones, kept tokens, dense feed-forward, experts, top,
+                           # expert and shared width, layers (half of each kind: biased + dense, rotary + experts)
+    "16e": (2048, 16, 4, 512, 2048, 64, 8192, 16, 2, 1024, 2048, 16),
+    "32e": (3072, 24, 6, 512, 2048, 64, 12288, 32, 4, 1024, 2048, 16),
+    "64e": (4096, 32, 8, 512, 2048, 64, 16384, 64, 6, 1408, 2816, 8),
+}
+
+
 def _serve(eng, vocab: int, batches, prompt_len: int, steps: int, warmup: int, total_prompts: int):
     """Device-timed prefill of ``total_prompts`` prompts and decode steps at every batch size of one engine."""
     import torch
@@ -603,7 +612,7 @@ def _serve(eng, vocab: int, batches, prompt_len: int, steps: int, warmup: int, t
 
 
 def run_vabarax(args) -> dict:
-    """The Vabarax design; see :func:`_beside_hybrid`."""
+    """The Vabarax design beside the hybrid decoder of softmax attention and Gated-DeltaNet layers; see :func:`_beside`."""
     from rhinoforge_b200.models.mixed import DenseMLP, HGRN2, LatentAttention, MixedConfig, MixedLayer
     entries = {}
     for name, (H, heads, rank, window, ff, side, layers) in VABARAX_SIZES.items():
@@ -611,14 +620,14 @@ def run_vabarax(args) -> dict:
         lin = MixedLayer(HGRN2(heads, 128, 128), DenseMLP(ff))
         # a GLU of 2/3 of the width has the same feed-forward parameters
         entries[name] = (lambda v, n=name, h=H, ls=(att, lin) * (layers // 2), p=side: MixedConfig("vabarax-" + n, v, h, 1e-6, ls, p),
-                         heads, heads // 4, 2 * ff // 3)
+                         lambda cfg, n=name, a=(heads, heads // 4, 2 * ff // 3): _hybrid(n, cfg, *a))
     keys = ("width", "heads", "rank", "window", "ff", "side", "layers")
-    return _beside_hybrid(args, "vabarax", "Vabarax-8b-sized", entries, {k: dict(zip(keys, v)) for k, v in VABARAX_SIZES.items()})
+    return _beside(args, "vabarax", "Vabarax-8b-sized", entries, {k: dict(zip(keys, v)) for k, v in VABARAX_SIZES.items()})
 
 
 def run_zulopel(args) -> dict:
-    """The Zulopel design; see :func:`_beside_hybrid`.  The hybrid decoder's feed-forward is as wide as the experts that one token
-    uses, shared expert included."""
+    """The Zulopel design beside the hybrid decoder of softmax attention and Gated-DeltaNet layers, whose feed-forward is as wide as
+    the experts that one token uses, shared expert included; see :func:`_beside`."""
     from rhinoforge_b200.models.mixed import GroupedAttention, Mamba1, MixedConfig, MixedLayer, MoE, Rotary, YarnScaling
     entries = {}
     for name, (H, heads, kv, chunk, inner, experts, top, groups, keep, ff, shared, layers) in ZULOPEL_SIZES.items():
@@ -627,19 +636,44 @@ def run_zulopel(args) -> dict:
         att = MixedLayer(GroupedAttention(heads, kv, 128, 128, 128 ** -0.5, chunk, rot, True), moe)
         scan = MixedLayer(Mamba1(inner, 16, H // 16, 4), moe)
         entries[name] = (lambda v, n=name, h=H, ls=(scan, att) * (layers // 2): MixedConfig.zulopel("zulopel-" + n, v, h, 1e-6, ls, h ** 0.5),
-                         heads, kv, top * ff + shared)
+                         lambda cfg, n=name, a=(heads, kv, top * ff + shared): _hybrid(n, cfg, *a))
     keys = ("width", "heads", "kv_heads", "chunk", "scan_channels", "experts", "top", "groups", "keep", "ff", "shared_ff", "layers")
-    return _beside_hybrid(args, "zulopel", "Zulopel 64-expert", entries, {k: dict(zip(keys, v)) for k, v in ZULOPEL_SIZES.items()})
+    return _beside(args, "zulopel", "Zulopel 64-expert", entries, {k: dict(zip(keys, v)) for k, v in ZULOPEL_SIZES.items()})
 
 
-def _beside_hybrid(args, design: str, headline: str, entries: dict, sizes: dict) -> dict:
-    """Prefill and decode throughput of a design with per-layer mixers at a few sizes, beside the closest decoder of this framework
-    - the hybrid of softmax attention (grouped K/V heads, SwiGLU) and Gated-DeltaNet layers - with the same width, heads, layer
-    count, prompts and batch sizes.  ``entries``: size name -> (config of a vocabulary size, heads, K/V heads, SwiGLU width of the
-    hybrid).  Random weights, synthetic ids; a "step" is one decode step."""
-    import torch
+def run_kuzupel(args) -> dict:
+    """The Kuzupel design beside a Zulopel decoder of attention layers with the same width, heads, experts and parameters (chunks of the
+    window's size; a dense feed-forward is a mixture of one expert there); see :func:`_beside`."""
+    from rhinoforge_b200.models.mixed import ClippedGLU, GroupedAttention, MixedConfig, MixedLayer, MoE, Rotary, TokenPairs
+    entries = {}
+    for name, (H, heads, kv, near, far, keep, dense, experts, top, ff, shared, layers) in KUZUPEL_SIZES.items():
+        head, rot = (heads, kv, 128, 128, 128 ** -0.5), Rotary(64, 5e5)
+        biased = MixedLayer(GroupedAttention(*head, sink=False, gate=False, window=near, distance_bias=True, norm_all=True), ClippedGLU(dense, 7.0))
+        rotary = MixedLayer(GroupedAttention(*head, rot=rot, sink=False, unit_sink=True, window=far, keep_first=keep, conv=4, gate_by_head=True),
+                            MoE(experts, top, ff, router="chosen", limit=7.0, shared_ff=shared, shared_limit=7.0, shared_gate=True))
+        like = (MixedLayer(GroupedAttention(*head, near, rot), MoE(1, 1, dense)), MixedLayer(GroupedAttention(*head, far, rot), MoE(experts, top, ff, 4, 4, shared)))
+        entries[name] = (lambda v, n=name, h=H, ls=(biased, rotary) * (layers // 2): MixedConfig.kuzupel(
+            "kuzupel-" + n, v, h, 1e-6, ls, pairs=TokenPairs(4 * v, 31, 7), residual_mult=0.5, logit_softcap=30.0),
+            lambda cfg, n=name, ls=like * (layers // 2): MixedConfig.zulopel("zulopel-" + n, cfg.vocab_size, cfg.hidden_size, 1e-6, ls))
+    keys = ("width", "heads", "kv_heads", "window_biased", "window_rotary", "keep_first", "dense_ff", "experts", "top", "ff", "shared_ff", "layers")
+    return _beside(args, "kuzupel", "Kuzupel 64-expert", entries, {k: dict(zip(keys, v)) for k, v in KUZUPEL_SIZES.items()})
+
+
+def _hybrid(name: str, cfg, heads: int, kv_heads: int, inter: int):
+    """The hybrid of softmax attention (grouped K/V heads, SwiGLU) and Gated-DeltaNet layers with a design's width and layer count."""
     from rhinoforge_b200.models.decoder import DecoderConfig
-    from rhinoforge_b200.models.mixed import random_weights, weight_shapes
+    return DecoderConfig("hybrid-" + name, cfg.vocab_size, cfg.hidden_size, (inter + 127) // 128 * 128, cfg.num_layers, heads, kv_heads, 128,
+                         tie_embeddings=True, norm="rms_gemma", attn_gate=True, model_type="qwen3_5",
+                         layer_types=("full_attention", "linear_attention") * (cfg.num_layers // 2),
+                         gdn_heads_k=heads, gdn_heads_v=heads, gdn_dk=128, gdn_dv=128)
+
+
+def _beside(args, design: str, headline: str, entries: dict, sizes: dict) -> dict:
+    """Prefill and decode throughput of a design with per-layer mixers at a few sizes, beside the closest decoder of this framework
+    with the same width, heads, layer count, prompts and batch sizes.  ``entries``: size name -> (config of a vocabulary size, config of
+    the closest decoder for that config).  Random weights, synthetic ids; a "step" is one decode step."""
+    import torch
+    from rhinoforge_b200.models.mixed import MixedConfig, random_weights, weight_shapes
     from rhinoforge_b200.runtime.engine import DecoderEngine, random_weight_getter
     from rhinoforge_b200.runtime.mixed_engine import MixedDecoderEngine
     if args.gpus != 1:
@@ -648,27 +682,30 @@ def _beside_hybrid(args, design: str, headline: str, entries: dict, sizes: dict)
     batches = sorted({1, 8, args.batch})
     vocab, prompt, npre = 32768, args.prompt_len, 8
     max_seq = prompt + 2 * args.steps + args.warmup + 128
-    res = {}
-    for name, (make, heads, kv_heads, inter) in entries.items():
-        cfg = make(vocab)
-        H, layers = cfg.hidden_size, cfg.num_layers
-        eng = MixedDecoderEngine(cfg, random_weights(cfg, device="cuda"), dtype=torch.bfloat16, max_batch=max(batches), max_seq_len=max_seq)
-        r = {"params_m": round(sum(int(torch.Size(s).numel()) for _, s, _ in weight_shapes(cfg)) / 1e6), "ours": _serve(
-            eng, vocab, batches, prompt, args.steps, args.warmup, npre), "cache_mb": round(eng.cache.nbytes() / 1e6)}
+
+    def serve(cfg):
+        kw = dict(dtype=torch.bfloat16, max_batch=max(batches), max_seq_len=max_seq)
+        if isinstance(cfg, MixedConfig):
+            eng = MixedDecoderEngine(cfg, random_weights(cfg, device="cuda"), **kw)
+        else:
+            eng = DecoderEngine(cfg, _hybrid_weights(cfg, random_weight_getter), **kw)
+        r = _serve(eng, vocab, batches, prompt, args.steps, args.warmup, npre)
+        cache = eng.cache.nbytes() if isinstance(cfg, MixedConfig) else 0
         eng.close()
-        del eng
+        return r, cache
+
+    res = {}
+    params = lambda cfg: round(sum(int(torch.Size(s).numel()) for _, s, _ in weight_shapes(cfg)) / 1e6)
+    for name, (make, closest) in entries.items():
+        cfg = make(vocab)
+        ours, cache = serve(cfg)
         torch.cuda.empty_cache()
-        inter = (inter + 127) // 128 * 128
-        like = DecoderConfig("hybrid-" + name, vocab, H, inter, layers, heads, kv_heads, 128, tie_embeddings=True, norm="rms_gemma",
-                             attn_gate=True, model_type="qwen3_5", layer_types=("full_attention", "linear_attention") * (layers // 2),
-                             gdn_heads_k=heads, gdn_heads_v=heads, gdn_dk=128, gdn_dv=128)
-        try:
-            eng = DecoderEngine(like, _hybrid_weights(like, random_weight_getter), dtype=torch.bfloat16, max_batch=max(batches), max_seq_len=max_seq)
-            r["closest"] = _serve(eng, vocab, batches, prompt, args.steps, args.warmup, npre)
-            eng.close()
-            del eng
-        finally:
-            torch.cuda.empty_cache()
+        r = {"params_m": params(cfg), "ours": ours, "cache_mb": round(cache / 1e6)}
+        like = closest(cfg)
+        if isinstance(like, MixedConfig):
+            r["closest_params_m"] = params(like)
+        r["closest"], _ = serve(like)
+        torch.cuda.empty_cache()
         r["ratio"] = {"prefill": r["ours"]["prefill_tok_s"] / r["closest"]["prefill_tok_s"],
                       **{f"decode_{b}": r["ours"]["decode"][str(b)]["tok_s"] / r["closest"]["decode"][str(b)]["tok_s"] for b in batches}}
         res[name] = r
@@ -709,7 +746,7 @@ def main(argv=None) -> int:
         if int(os.environ.get("RANK", "0")) == 0:          # one line per job, also under torch.distributed.run
             print(json.dumps({"impl": "reference", "unavailable": REFERENCE_UNAVAILABLE}))
         return 0
-    out = {"decode": run, "pi05": run_pi05, "qwen3vl": run_qwen3vl, "vabarax": run_vabarax, "zulopel": run_zulopel}[args.workload](args)
+    out = {"decode": run, "pi05": run_pi05, "qwen3vl": run_qwen3vl, "vabarax": run_vabarax, "zulopel": run_zulopel, "kuzupel": run_kuzupel}[args.workload](args)
     if out is not None:
         print(json.dumps(out))
     try:

@@ -7,6 +7,7 @@
     python bench_kernels.py gdn --seqs 1 --len 1024 --hk 16 --hv 32
     python bench_kernels.py mixed            # latent attention / HGRN2 / fp32 stream beside the like kernels at equal size
     python bench_kernels.py routed           # chunked attention / selective scan / routed experts beside the like kernels
+    python bench_kernels.py windowed         # window attention with slopes or kept tokens / clipped feed-forwards beside the like kernels
     python bench_kernels.py suite            # the shapes of one Qwen3-8B decode step and prefill chunk
 
 Every line is JSON: the achieved throughput and its fraction of the measured peaks in
@@ -514,6 +515,118 @@ def bench_routed(hidden, heads, kv, inner, experts, top, ff, *, chunk=1024, grou
             bench_gemm(pairs // 4, hidden, ff * 4, packed=True, dtype=dtype)
 
 
+def bench_windowed(hidden, heads, kv, dense, experts, top, ff, *, near=512, far=2048, keep=64, taps=4, batch=64, prefill=(4, 2048), vocab=32768,
+                   dtype=torch.bfloat16) -> None:
+    """Kernels of decoders with window attention (distance slopes and one norm over all heads; kept first tokens, convolved
+    projections and gates per head) and clipped feed-forwards, each beside the like kernel of the chunked-attention decoders at
+    equal size."""
+    from rhinoforge_b200.ops import kernels as K
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
+    tag = dict(hidden=hidden)
+    rnd = lambda *sh: torch.randn(*sh, device="cuda", dtype=dtype)
+    f32 = lambda *sh: torch.randn(*sh, device="cuda")
+    S, Lp = prefill
+    T, hd, clip = S * Lp, 128, dict(act="clipped_glu", limit=7.0, alpha=1.702)
+    starts, lens = i32([j * Lp for j in range(S)]), i32([Lp] * S)
+    seq, pos_p = i32([j for j in range(S) for _ in range(Lp)]), i32(list(range(Lp)) * S)
+    rows_p = lambda **kw: K.rows(pos_p, seq_of_row=seq, q_start=starts, q_len=lens, slot=i32(list(range(S))), **kw)
+    # ---- residual stream
+    table, pair = rnd(vocab, hidden), rnd(4 * vocab + 1, hidden)
+    for n, r in ((batch, K.rows(i32([7] * batch))), (T, rows_p())):
+        x, nw, yw = f32(n, hidden), f32(hidden), f32(hidden)
+        yg, slots = rnd(n * (top + 1), hidden), torch.randperm(n * (top + 1), device="cuda").to(torch.int32).view(n, top + 1)
+        y1, ids, last = rnd(n, hidden), torch.randint(0, vocab, (n,), device="cuda").to(torch.int32), i32([0] * n)
+        for what, y, sl, traffic in (("sum of picked rows", yg, slots, 2 * (top + 1)), ("one row", y1, None, 2)):
+            us = time_cold_us(lambda: K.stream_norm(x, r, dtype=dtype, eps=1e-6, norm_w=nw, y=y, y_slots=sl, y_mult=0.5))
+            report(f"stream_norm ({what}, factor, add, norm)", us, bytes_=n * hidden * (10 + traffic), rows=n, **tag)
+            us = time_cold_us(lambda: K.stream_norm(x, r, dtype=dtype, eps=1e-6, y=y, y_norm_w=yw, cast=True, y_slots=sl))
+            report(f"like: stream_norm ({what}, norm of it, add)", us, bytes_=n * hidden * (10 + traffic), rows=n, **tag)
+        us = time_cold_us(lambda: K.stream_norm(None, r, dtype=dtype, eps=1e-6, norm_w=nw, table=table, ids=ids, pairs=(pair, last, 31, 7)))
+        report("stream_norm (embedding and token pairs, norm)", us, bytes_=n * hidden * 10, rows=n, **tag)
+        us = time_cold_us(lambda: K.stream_norm(None, r, dtype=dtype, eps=1e-6, table=table, ids=ids, cast=True))
+        report("like: stream_norm (embedding)", us, bytes_=n * hidden * 8, rows=n, **tag)
+        del yg
+    del table, pair
+    # ---- attention
+    cos, sin = f32(4096, 32), f32(4096, 32)
+    qn, cols = f32(hd), (heads + 2 * kv) * hd
+    cw, slopes, ones = f32(taps, cols), torch.rand(heads, device="cuda"), torch.zeros(heads, device="cuda")
+    kw = dict(Hq=heads, Hkv=kv, hd=hd, scale=0.09)
+    for n, r_of in ((1, lambda **k: K.rows(i32([far - 1]), **k)), (batch, lambda **k: K.rows(i32([far - 1] * batch), **k)), (T, rows_p)):
+        per, nseq = (max(Lp, far) + 15) // 16, S if n == T else n
+        pt = torch.randperm(nseq * per, device="cuda").to(torch.int32).view(nseq, per)
+        kp, vp = rnd(nseq * per, kv, 16, hd), rnd(nseq * per, kv, 16, hd)
+        x, first, state = rnd(n, cols), rnd(n, kv * hd), rnd(nseq, taps - 1, cols)
+        r, moved = r_of(page_table=pt), n * (2 * heads + 4 * kv) * hd * 2
+        head = dict(heads=heads, kv_heads=kv, hd=hd, eps=1e-6)
+        qa, ka = f32(heads, hd), f32(kv, hd)
+        us = time_cold_us(lambda: K.qkv_insert(x, r, kp, vp, q_norm=qa, k_norm=ka, norm_all=True, **head))
+        report("qkv_insert (one norm over all heads)", us, bytes_=moved, rows=n, heads=heads, kv_heads=kv, **tag)
+        us = time_cold_us(lambda: K.qkv_insert(x, r, kp, vp, q_norm=qn, k_norm=qn, cos=cos, sin=sin, conv_w=cw, conv_state=state, max_q_len=1 if n != T else Lp, **head))
+        report("qkv_insert (convolution, norms, rotation)", us, bytes_=moved + 4.0 * nseq * (taps - 1) * cols + 4.0 * taps * cols, rows=n, **tag)
+        us = time_cold_us(lambda: K.qkv_insert(x, r, kp, vp, q_norm=qn, k_norm=qn, cos=cos, sin=sin, v_first=first, v_role="mix", v_lambda=0.5, **head))
+        report("like: qkv_insert (norms, rotation, value mixing)", us, bytes_=moved + n * kv * hd * 2, rows=n, **tag)
+        q, gate, gate1 = x[:, :heads * hd], rnd(n, heads * hd), rnd(n, (heads + 7) // 8 * 8)
+        forms = (("window and slopes", near, dict(window=near, slopes=slopes)),
+                 ("window, kept tokens, one in the denominator, gate per head", far, dict(window=far, keep_first=keep, sink=ones, gate=gate1, gate_by_head=True)),
+                 ("window over the kept tokens", near, dict(window=near, keep_first=keep, sink=ones, gate=gate1, gate_by_head=True)),
+                 ("like: chunk, sink, gate", near, dict(chunk=near, sink=ones, gate=gate)), ("like: chunk, sink, gate", far, dict(chunk=far, sink=ones, gate=gate)))
+        out = rnd(n, heads * hd)
+        for what, size, opt in forms:
+            seen = lambda i: i % size + 1 if "chunk" in opt else min(i + 1, size) + (min(keep, max(i + 1 - size, 0)) if "keep_first" in opt else 0)
+            if n == T:
+                us = time_cold_us(lambda: K.attention_prefill(q, out, q_start=starts, q_len=lens, kv_len=lens, max_q_len=Lp, k_pool=kp, v_pool=vp,
+                                                              page_table=pt, max_kv_len=Lp, **kw, **opt))
+                report(f"attention prefill ({what})", us, flops=4.0 * S * sum(seen(i) for i in range(Lp)) * heads * hd, rows=n, size=size, **tag)
+            else:
+                us = time_cold_us(lambda: K.attention_rows(q, r, kp, vp, max_kv=far, **kw, **opt))
+                report(f"attention by row ({what})", us, bytes_=4.0 * n * seen(far - 1) * kv * hd + 4.0 * n * heads * hd, rows=n, size=size, **tag)
+        del kp, vp, x, gate
+    # ---- feed-forward and head
+    wu, wd = K.pack_weight(rnd(2 * dense, hidden) / hidden ** 0.5, 2), K.pack_weight(rnd(vocab, hidden) / hidden ** 0.5)
+    for n in (1, 8, batch, T):
+        x = rnd(n, hidden)
+        shape = dict(flops=4.0 * n * dense * hidden, bytes_=4.0 * dense * hidden + 2.0 * n * (hidden + dense), rows=n, ff=dense, **tag)
+        report("GEMM pair, clipped", time_cold_us(lambda: K.gemm(x, wu, packed_shape=(2 * dense, hidden), dual=True, **clip)), **shape)
+        report("like: GEMM pair, silu", time_cold_us(lambda: K.gemm(x, wu, packed_shape=(2 * dense, hidden), dual=True, act="silu_mul")), **shape)
+        if n <= 64:
+            shape = dict(bytes_=2.0 * vocab * (hidden + n), rows=n, vocab=vocab, **tag)
+            report("head with soft cap", time_cold_us(lambda: K.gemm(x, wd, packed_shape=(vocab, hidden), act="soft_cap", limit=30.0)), **shape)
+            report("like: head", time_cold_us(lambda: K.gemm(x, wd, packed_shape=(vocab, hidden))), **shape)
+    del wu, wd
+    router, bias = rnd(experts + 1, hidden) / hidden ** 0.5, f32(experts) * 0.1
+    pad = (ff + 127) // 128 * 128
+    up = K.pack_weight(rnd(2 * experts * pad, hidden) / hidden ** 0.5, 2)
+    down = K.pack_weight(rnd(hidden, experts * pad) / ff ** 0.5)
+    for n in (1, 8, batch, T):
+        x = rnd(n, hidden)
+        small = n <= 256
+        plan = dict(tile_rows=(16 if n * top <= 16 * experts else 32) if small else 128, scatter=small, shared=True)
+        b = K.RoutedBatch(x, router, top, correction=bias, score_fn="chosen", shared_gate=True, **plan)
+        report("moe_router (biased logits, softmax over the chosen, shared weight)", time_cold_us(b.route), bytes_=2.0 * (n + experts) * hidden, rows=n, experts=experts, top=top, **tag)
+        like = K.RoutedBatch(x, router[:experts], top, correction=bias, **plan)
+        report("like: moe_router (softmax, correction)", time_cold_us(like.route), bytes_=2.0 * (n + experts) * hidden, rows=n, **tag)
+        b = K.RoutedBatch(x, router[:experts], top, correction=bias, score_fn="chosen", **dict(plan, shared=False)).route()
+        torch.cuda.synchronize()
+        used = int(b.ids.unique().numel())
+        e = dict(rows=n, experts=experts, used=used, ff=ff, **tag)
+        for what, opt in (("experts: gate and up, clipped", clip), ("like: experts: gate and up, silu", {})):
+            if small:
+                us = time_cold_us(lambda: K.moe_experts(b, x, up, n=ff, k=hidden, experts=experts, expert_pad=pad, dual=True, **opt))
+                report(what, us, bytes_=4.0 * used * ff * hidden + 2.0 * n * top * ff + 2.0 * n * hidden, **e)
+            else:
+                xg, out = b.gather(), rnd(n * top, pad)
+                opt = opt or dict(act="silu_mul")
+                us = time_cold_us(lambda: K.moe_grouped_gemm(xg, up, b.tiles[3:], n=pad, k=hidden, bank_rows=experts * pad, bank_k=hidden, expert_rows=pad,
+                                                             dual=True, out=out, **opt))
+                report(what + " (grouped)", us, flops=4.0 * n * top * ff * hidden, **e)
+
+
+def windowed() -> None:
+    bench_windowed(2048, 16, 4, 8192, 16, 2, 1024)
+    bench_windowed(4096, 32, 8, 16384, 64, 6, 1408)
+
+
 def routed() -> None:
     bench_routed(2048, 16, 4, 4096, 16, 2, 1024, groups=4, keep=2)
     bench_routed(4096, 32, 8, 8192, 64, 6, 1408)
@@ -526,7 +639,7 @@ def mixed() -> None:
 
 def main() -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("what", choices=["gemm", "attn_prefill", "attn_decode", "gdn", "suite", "sweep", "heads", "mixed", "routed"])
+    ap.add_argument("what", choices=["gemm", "attn_prefill", "attn_decode", "gdn", "suite", "sweep", "heads", "mixed", "routed", "windowed"])
     for name, d in (("m", 64), ("n", 4096), ("k", 4096), ("seqs", 4), ("len", 2048), ("heads", 32), ("kv-heads", 8),
                     ("hd", 128), ("hk", 16), ("hv", 32)):
         ap.add_argument(f"--{name}", type=int, default=d)
@@ -556,6 +669,8 @@ def main() -> int:
         mixed()
     elif a.what == "routed":
         routed()
+    elif a.what == "windowed":
+        windowed()
     else:
         suite()
     return 0

@@ -36,10 +36,17 @@ __device__ __forceinline__ float head_rstd(const RfQkvInsert& p, const float (&x
   return rsqrtf(ss / (float)p.dim + p.eps);
 }
 
-// Norm with `rstd`, rotation, value mixing and the store of one head; all lanes of the warp, buf: the group's scratch.
+// Page-table row of the sequence that owns a row.
+__device__ __forceinline__ int slot_of_row(const RfQkvInsert& p, int row) {
+  const int seq = p.rows.seq_of_row ? p.rows.seq_of_row[row] : row;
+  return p.rows.slot ? p.rows.slot[seq] : seq;
+}
+
+// Norm with `rstd`, rotation, value mixing and the store of one head at position pos; all lanes of the warp, buf: the group's scratch.
 template <typename T, int GL, int NC>
-__device__ __forceinline__ void finish_head(const RfQkvInsert& p, const HeadItem& it, float (&x)[NC][8], float rstd, int gl, float* buf) {
-  const int hd = p.hd, pos = p.rows.pos[it.row];
+__device__ __forceinline__ void finish_head(const RfQkvInsert& p, const HeadItem& it, int pos, int slot, float (&x)[NC][8], float rstd, int gl,
+                                            float* buf) {
+  const int hd = p.hd;
   const float* nw = it.is_v ? nullptr : (it.is_q ? p.q_norm : p.k_norm);
   if (nw) {
     if (p.norm_all) nw += (size_t)it.head * hd;
@@ -52,8 +59,23 @@ __device__ __forceinline__ void finish_head(const RfQkvInsert& p, const HeadItem
       }
     }
   }
-  if (p.rot_dims > 0) {                            // uniform over the grid
-    const int half = p.rot_dims >> 1;
+  const int half = p.rot_dims >> 1;                // uniform over the grid
+  if (NC == 1 && half > 0 && half % 8 == 0) {
+    // whole lanes turn with one another: dimensions of lane l with those of lane l + half / 8
+    const int hl = half >> 3, with = gl < hl ? gl + hl : (gl < 2 * hl ? gl - hl : gl), lane = threadIdx.x & 31;
+    const bool turns = it.live && !it.is_v && gl < 2 * hl;
+    const size_t at = (size_t)pos * half + (gl < hl ? gl : gl - hl) * 8;
+    float cs[8], sn[8];
+    if (turns) {
+      load8(p.cos + at, cs);
+      load8(p.sin + at, sn);
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const float other = __shfl_sync(0xffffffffu, x[0][j], lane - gl + with);
+      if (turns) x[0][j] = x[0][j] * cs[j] + (gl < hl ? -other : other) * sn[j];
+    }
+  } else if (half > 0) {
     __syncwarp();
 #pragma unroll
     for (int c = 0; c < NC; ++c) {
@@ -96,8 +118,6 @@ __device__ __forceinline__ void finish_head(const RfQkvInsert& p, const HeadItem
   if (it.is_q) {
     dst = p.q_out ? reinterpret_cast<T*>(p.q_out) + ((size_t)it.row * p.heads + it.head) * hd : it.source<T>(p);
   } else {
-    const int seq = p.rows.seq_of_row ? p.rows.seq_of_row[it.row] : it.row;
-    const int slot = p.rows.slot ? p.rows.slot[seq] : seq;
     const int page = p.rows.page_table[(size_t)slot * p.rows.pt_stride + (pos >> 4)];
     dst = reinterpret_cast<T*>(it.is_v ? p.v_pool : p.k_pool) + (((size_t)page * p.kv_heads + it.head) * 16 + (pos & 15)) * hd;
   }
@@ -134,7 +154,8 @@ __global__ void __launch_bounds__(256) qkv_insert_kernel(const RfQkvInsert p) {
   const HeadItem it(p, live ? (int)(idx / items) : 0, live ? (int)(idx % items) : 0, live);
   float x[NC][8];
   load_head<T, GL, NC>(it.source<T>(p), live, p.hd, gl, x);
-  finish_head<T, GL, NC>(p, it, x, head_rstd<GL, NC>(p, x), gl, rot_buf + (size_t)(warp * HPW + sub) * p.rot_dims);
+  finish_head<T, GL, NC>(p, it, p.rows.pos[it.row], slot_of_row(p, it.row), x, head_rstd<GL, NC>(p, x), gl,
+                         rot_buf + (size_t)(warp * HPW + sub) * p.rot_dims);
 }
 
 // One norm over all query heads of a row and one over all key heads: a CTA per row, which is read twice.
@@ -147,6 +168,7 @@ __global__ void __launch_bounds__(256) qkv_insert_row_kernel(const RfQkvInsert p
   const int warp = threadIdx.x >> 5, nw = blockDim.x >> 5, lane = threadIdx.x & 31, gl = lane % GL, sub = lane / GL;
   const int row = blockIdx.x, items = p.heads + 2 * p.kv_heads, groups = nw * HPW, qn = p.heads * p.hd / 8, kn = p.kv_heads * p.hd / 8;
   const T* src = reinterpret_cast<const T*>(p.qkv) + (size_t)row * p.ld;
+  const int pos = p.rows.pos[row], slot = slot_of_row(p, row);
   float sq = 0.f, sk = 0.f;
   for (int i = threadIdx.x; i < qn + kn; i += blockDim.x) {
     float f[8], s = 0.f;
@@ -169,15 +191,15 @@ __global__ void __launch_bounds__(256) qkv_insert_row_kernel(const RfQkvInsert p
     const HeadItem it(p, row, live ? item : 0, live);
     float x[NC][8];
     load_head<T, GL, NC>(it.source<T>(p), live, p.hd, gl, x);
-    finish_head<T, GL, NC>(p, it, x, it.is_q ? rq : rk, gl, rot_buf + (size_t)(warp * HPW + sub) * p.rot_dims);
+    finish_head<T, GL, NC>(p, it, pos, slot, x, it.is_q ? rq : rk, gl, rot_buf + (size_t)(warp * HPW + sub) * p.rot_dims);
   }
 }
 
-// With the convolution: a group walks `tile` neighbouring rows of one sequence for its head, the last inputs in registers
-// (TAPS = 0: any number of taps, every input read again for each of them).  The group of a sequence's first rows also replaces the
+// With the convolution: a group walks `tile` neighbouring rows of one sequence for its head, four at a time, the last inputs and the
+// next four rows in registers (TAPS = 0: any number of taps, every input read again for each of them).  The group of a sequence's first rows also replaces the
 // carried inputs; later tiles find theirs among the rows of this launch.
 template <typename T, int GL, int NC, int TAPS>
-__global__ void __launch_bounds__(256) qkv_conv_insert_kernel(const RfQkvInsert p, int tile) {
+__global__ void __launch_bounds__(128) qkv_conv_insert_kernel(const RfQkvInsert p, int tile) {
   pdl_prologue();
   extern __shared__ __align__(16) float rot_buf[];
   constexpr int HPW = 32 / GL;
@@ -187,45 +209,70 @@ __global__ void __launch_bounds__(256) qkv_conv_insert_kernel(const RfQkvInsert 
   const int t0 = blockIdx.y * tile, t1 = min(n, t0 + tile);
   if (t0 >= n) return;
   const int item = (blockIdx.x * (blockDim.x >> 5) + warp) * HPW + sub;
-  const bool live = item < items, fresh = p.rows.pos[q0] == 0;
+  const bool live = item < items;
+  const int pos0 = p.rows.pos[q0], slot = p.rows.slot ? p.rows.slot[seq] : seq;       // positions of a portion follow one another
   const size_t channels = (size_t)items * hd, at = (size_t)(live ? item : 0) * hd;
-  T* state = reinterpret_cast<T*>(p.conv_state) + (size_t)(p.rows.slot ? p.rows.slot[seq] : seq) * past * channels + at;
+  T* state = reinterpret_cast<T*>(p.conv_state) + (size_t)slot * past * channels + at;
   const T* src = reinterpret_cast<const T*>(p.qkv) + (size_t)q0 * p.ld + at;
   const float* w = p.conv_w + at;
   float* buf = rot_buf + (size_t)(warp * HPW + sub) * p.rot_dims;
   // input at place i of this launch's rows; negative places are carried ones
+  auto input_at = [&](int i) -> const T* {
+    return i >= 0 ? src + (size_t)i * p.ld : (pos0 > 0 ? state + (size_t)(past + i) * channels : nullptr);
+  };
   auto input = [&](int i, float (&f)[NC][8]) {
-    if (i >= 0) load_head<T, GL, NC>(src + (size_t)i * p.ld, live, hd, gl, f);
-    else load_head<T, GL, NC>(state + (size_t)(past + i) * channels, live && !fresh, hd, gl, f);
+    const T* q = input_at(i);
+    load_head<T, GL, NC>(q, live && q != nullptr, hd, gl, f);
   };
   auto finish = [&](int t, float (&x)[NC][8]) {
     const HeadItem it(p, q0 + t, live ? item : 0, live);
-    finish_head<T, GL, NC>(p, it, x, head_rstd<GL, NC>(p, x), gl, buf);
+    finish_head<T, GL, NC>(p, it, pos0 + t, slot, x, head_rstd<GL, NC>(p, x), gl, buf);
   };
-  if constexpr (TAPS > 0) {
-    float wt[TAPS][NC][8], win[TAPS][NC][8];
+  if constexpr (TAPS > 0 && NC == 1) {
+    constexpr int R = 4;
+    const bool mine = live && gl * 8 < hd;
+    Vec8<T> old[TAPS - 1], cur[R], nxt[R];
+    float wt[TAPS][1][8];
+    auto fetch = [&](int i, bool in) -> Vec8<T> {
+      const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      Vec8<T> v;
+      const T* q = in && mine ? input_at(i) : nullptr;
+      if (q) v = *reinterpret_cast<const Vec8<T>*>(q + gl * 8);
+      else store8(reinterpret_cast<T*>(&v), zero);
+      return v;
+    };
 #pragma unroll
-    for (int k = 0; k < TAPS; ++k) load_head<float, GL, NC>(w + k * channels, live, hd, gl, wt[k]);
+    for (int r = 0; r < R; ++r) nxt[r] = fetch(t0 + r, t0 + r < t1);
 #pragma unroll
-    for (int k = 0; k < TAPS - 1; ++k) input(t0 - (TAPS - 1) + k, win[k]);
-    for (int t = t0; t < t1; ++t) {
-      float x[NC][8];
-      input(t, win[TAPS - 1]);
+    for (int k = 0; k < TAPS - 1; ++k) old[k] = fetch(t0 - (TAPS - 1) + k, true);
 #pragma unroll
-      for (int c = 0; c < NC; ++c)
+    for (int k = 0; k < TAPS; ++k) load_head<float, GL, 1>(w + k * channels, live, hd, gl, wt[k]);
+    for (int t = t0; t < t1; t += R) {
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          x[c][j] = 0.f;
+      for (int r = 0; r < R; ++r) {
+        cur[r] = nxt[r];
+        nxt[r] = fetch(t + R + r, t + R + r < t1);
+      }
 #pragma unroll
-          for (int k = 0; k < TAPS; ++k) x[c][j] += wt[k][c][j] * win[k][c][j];
+      for (int r = 0; r < R; ++r) {
+        if (t + r >= t1) break;
+        float x[1][8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[0][j] = 0.f;
+#pragma unroll
+        for (int k = 0; k < TAPS; ++k) {
+          const int i = r - (TAPS - 1) + k;
+          const Vec8<T> v = i < 0 ? old[i < 0 ? TAPS - 1 + i : 0] : cur[i < 0 ? 0 : i];
+          float f[8];
+          load8(reinterpret_cast<const T*>(&v), f);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) x[0][j] += wt[k][0][j] * f[j];
         }
+        finish(t + r, x);
+      }
+      static_assert(TAPS - 1 <= R, "the last inputs lie in the rows just done");
 #pragma unroll
-      for (int k = 0; k < TAPS - 1; ++k)
-#pragma unroll
-        for (int c = 0; c < NC; ++c)
-#pragma unroll
-          for (int j = 0; j < 8; ++j) win[k][c][j] = win[k + 1][c][j];
-      finish(t, x);
+      for (int k = 0; k < TAPS - 1; ++k) old[k] = cur[R - (TAPS - 1) + k];
     }
   } else {
     for (int t = t0; t < t1; ++t) {
@@ -312,11 +359,12 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const RfAttn p) {
 }
 
 template <typename T, int GL, int NC, int TAPS>
-static int launch_qkv_conv(const RfQkvInsert* a, int warps, cudaStream_t s) {
-  const int per_block = warps * (32 / GL), tile = std::max(16, a->taps - 1);
+static int launch_qkv_conv(const RfQkvInsert* a, cudaStream_t s) {
+  const int items = a->heads + 2 * a->kv_heads, hpw = 32 / GL, warps = std::min(4, ceil_div(items, hpw)), per_block = warps * hpw;
+  const int tile = std::max(16, a->taps - 1);      // later tiles find their past in the rows of this launch
   const size_t smem = (size_t)per_block * a->rot_dims * sizeof(float);
   RF_ALLOW_SMEM_PER_DEVICE((qkv_conv_insert_kernel<T, GL, NC, TAPS>), 64 * 1024);
-  const dim3 grid(ceil_div(a->heads + 2 * a->kv_heads, per_block), ceil_div(a->max_q_len, tile), a->rows.num_seqs);
+  const dim3 grid(ceil_div(items, per_block), ceil_div(a->max_q_len, tile), a->rows.num_seqs);
   RF_CUDA_CHECK(::rf::launch_k(qkv_conv_insert_kernel<T, GL, NC, TAPS>, grid, dim3(warps * 32), smem, s, 1, *a, tile));
   ::rf::count_launch();
   return RF_OK;
@@ -327,12 +375,12 @@ static int launch_qkv_insert(const RfQkvInsert* a, cudaStream_t s) {
   const int64_t groups = (int64_t)a->n_rows * (a->heads + 2 * a->kv_heads);
   const int warps = groups * GL / 32 < 8 * sm_count() ? 2 : 8, per_block = warps * (32 / GL);
   if (a->taps > 0) {
-    if (NC > 1) return launch_qkv_conv<T, GL, NC, 0>(a, warps, s);
+    if (NC > 1) return launch_qkv_conv<T, GL, NC, 0>(a, s);
     switch (a->taps) {
-      case 2: return launch_qkv_conv<T, GL, NC, NC == 1 ? 2 : 0>(a, warps, s);
-      case 3: return launch_qkv_conv<T, GL, NC, NC == 1 ? 3 : 0>(a, warps, s);
-      case 4: return launch_qkv_conv<T, GL, NC, NC == 1 ? 4 : 0>(a, warps, s);
-      default: return launch_qkv_conv<T, GL, NC, 0>(a, warps, s);
+      case 2: return launch_qkv_conv<T, GL, NC, NC == 1 ? 2 : 0>(a, s);
+      case 3: return launch_qkv_conv<T, GL, NC, NC == 1 ? 3 : 0>(a, s);
+      case 4: return launch_qkv_conv<T, GL, NC, NC == 1 ? 4 : 0>(a, s);
+      default: return launch_qkv_conv<T, GL, NC, 0>(a, s);
     }
   }
   if (a->norm_all) {

@@ -278,9 +278,8 @@ __global__ void __launch_bounds__(VPT == 4 ? 512 : 1024) stream_norm_reg_kernel(
   }
 }
 
-// The stream step behind a sublayer whose output is normalised (16-bit activations, no token shift): one CTA per row, a thread
-// holds NC groups of eight columns, so that every operand moves in 16-byte pieces; of several picked rows four are in flight at
-// a time.
+// The stream step of 16-bit activations without a token shift: one CTA per row, a thread holds NC groups of eight columns, so that
+// every operand moves in 16-byte pieces; of several picked rows four are in flight at a time.
 template <typename T, int NC>
 __global__ void __launch_bounds__(512) stream_out_kernel(const RfStreamNorm p) {
   pdl_launch_dependents();
@@ -288,13 +287,16 @@ __global__ void __launch_bounds__(512) stream_out_kernel(const RfStreamNorm p) {
   const int H = p.H, nthr = blockDim.x, nw = nthr >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const float inv_dim = 1.f / (float)p.dim;
   auto col = [&](int k) { return (threadIdx.x + k * nthr) * 8; };
-  float w[NC][8];
+  float w[NC][8];                                              // the first norm's weights: they do not depend on the previous kernel
+  const float* first_w = p.y_norm_w ? p.y_norm_w : p.norm_w;
 #pragma unroll
   for (int k = 0; k < NC; ++k)
-    if (col(k) < H) load8(p.y_norm_w + col(k), w[k]);          // does not depend on the previous kernel
+    if (first_w && col(k) < H) load8(first_w + col(k), w[k]);
   pdl_wait();
   const int r = blockIdx.x, src = p.row_idx ? p.row_idx[r] : r;
   const T* y = reinterpret_cast<const T*>(p.y);
+  const T* second = p.table2 ? reinterpret_cast<const T*>(p.table2) + (size_t)pair_row(p, src) * H : nullptr;
+  if (second) carry_token(p, src);
   float v[NC][8], a[NC][8];
 #pragma unroll
   for (int k = 0; k < NC; ++k) {
@@ -306,9 +308,15 @@ __global__ void __launch_bounds__(512) stream_out_kernel(const RfStreamNorm p) {
       load8(reinterpret_cast<const T*>(p.table) + (size_t)p.ids[src] * H + col(k), v[k]);
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[k][j] *= p.embed_scale;
+      if (second) {
+        float f[8];
+        load8(second + col(k), f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[k][j] += f[j];
+      }
     }
   }
-  const int picks = p.y_picks > 0 ? p.y_picks : 1;
+  const int picks = !y ? 0 : p.y_picks > 0 ? p.y_picks : 1;
   for (int j0 = 0; j0 < picks; j0 += 4) {
     int row[4];
     uint4 raw[4][NC];
@@ -340,19 +348,24 @@ __global__ void __launch_bounds__(512) stream_out_kernel(const RfStreamNorm p) {
     __syncthreads();
     return warp_sum(lane < nw ? red[flip][lane] : 0.f);
   };
-  float s = 0.f;
+  float s = 0.f, yr = p.y_mult;
+  if (p.y_norm_w) {
 #pragma unroll
-  for (int k = 0; k < NC; ++k)
+    for (int k = 0; k < NC; ++k)
 #pragma unroll
-    for (int j = 0; j < 8; ++j) s += a[k][j] * a[k][j];
-  const float yr = rsqrtf(block_sum(s, 0) * inv_dim + p.eps) * p.y_mult;
+      for (int j = 0; j < 8; ++j) {
+        s += a[k][j] * a[k][j];
+        a[k][j] *= w[k][j];
+      }
+    yr *= rsqrtf(block_sum(s, 0) * inv_dim + p.eps);
+  }
   s = 0.f;
 #pragma unroll
   for (int k = 0; k < NC; ++k) {
     if (col(k) >= H) continue;
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-      v[k][j] += a[k][j] * yr * w[k][j];
+      v[k][j] += a[k][j] * yr;
       s += v[k][j] * v[k][j];
     }
     if (p.x_out) store8(p.x_out + (size_t)r * H + col(k), v[k]);
@@ -364,9 +377,9 @@ __global__ void __launch_bounds__(512) stream_out_kernel(const RfStreamNorm p) {
   for (int k = 0; k < NC; ++k) {
     if (col(k) >= H) continue;
     float n8[8];
-    load8(p.norm_w + col(k), n8);
+    if (p.y_norm_w) load8(p.norm_w + col(k), w[k]);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) n8[j] *= v[k][j] * xr;
+    for (int j = 0; j < 8; ++j) n8[j] = w[k][j] * v[k][j] * xr;
     store8(reinterpret_cast<T*>(p.out) + (size_t)r * H + col(k), n8);
   }
 }
@@ -483,7 +496,7 @@ extern "C" int rf_stream_norm(const RfStreamNorm* args, rf_stream_t stream) {
   const int rpc = (a->shift && a->rows.q_start) ? std::max(1, std::min(8, a->n_rows / (2 * sm_count()))) : 1;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int groups = a->H / 8;
-  if (a->y && a->y_norm_w && !a->shift && !a->table2 && a->dtype != kF32 && groups <= 1024) {
+  if (!a->shift && a->dtype != kF32 && groups <= 1024) {
     // decode rows: one group of columns per thread; many rows: two, so that several rows share an SM
     const int nc = groups > 512 || (groups > 256 && a->n_rows > 4 * sm_count()) ? 2 : 1;
     const dim3 block(std::max(32, round_up(ceil_div(groups, nc), 32)));

@@ -13,7 +13,8 @@ import torch
 
 from .. import _native as N
 
-ACT = {None: 0, "none": 0, "silu_mul": 1, "gelu_tanh_mul": 2, "gelu_tanh": 3, "gelu_erf": 4, "silu": 5, "relu2": 6}
+ACT = {None: 0, "none": 0, "silu_mul": 1, "gelu_tanh_mul": 2, "gelu_tanh": 3, "gelu_erf": 4, "silu": 5, "relu2": 6,
+       "clipped_glu": 7, "soft_cap": 8}
 ELT = {"add": 0, "mul": 1, "silu_mul": 2, "gelu_tanh_mul": 3, "axpy": 4, "gelu_tanh": 5, "gelu_erf": 6,
        "silu": 7, "scale": 8, "sigmoid_mul": 9, "mul_row": 10, "tanh": 11}
 
@@ -85,7 +86,7 @@ def gemm(x: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
          norm_eps: float = 1e-6, norm_gemma: bool = False, w_bits: int = 0, w_group: int = 0,
          w_fp4: bool = False, ss_out: Optional[torch.Tensor] = None, ss_in: Optional[torch.Tensor] = None,
          ss_dim: int = 0, ss_eps: float = 1e-6, mul: Optional[torch.Tensor] = None,
-         mul_row: Optional[torch.Tensor] = None) -> torch.Tensor:
+         mul_row: Optional[torch.Tensor] = None, limit: float = 0.0, alpha: float = 0.0) -> torch.Tensor:
     """``out = epilogue(x @ w.T)`` on the tcgen05 kernel (or the CUDA-core GEMV).
 
     ``dual=True``: ``w`` stacks ``[gate; up]`` (2N rows) and ``act`` is a ``*_mul``
@@ -105,6 +106,7 @@ def gemm(x: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
     is scaled per token by ``rsqrt(sum(ss_in[:, token]) / ss_dim + ss_eps)``: an RMSNorm of ``x`` whose weights were
     multiplied into the columns of ``w`` beforehand.
     ``mul`` / ``mul_row`` (few rows, small weights): row ``m`` of the activated result is multiplied by ``mul[mul_row[m], :N]``.
+    ``limit`` / ``alpha``: constants of ``act="clipped_glu"`` (``dual``) and ``"soft_cap"`` (``limit``).
     """
     M, K = x.shape
     if packed_shape is not None:          # ``w`` is the tile-major image made by pack_weight(); (rows, K) is its logical shape
@@ -129,6 +131,7 @@ def gemm(x: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
     g.dtype = dtype_code(x.dtype)
     g.act = ACT[act]
     g.dual_offset = Nn if dual else 0
+    g.act_limit, g.act_alpha = limit, alpha
     g.w_int8 = 1 if (w.dtype == torch.int8 or w_bits == 4) else 0
     if w_bits == 4:
         if packed_shape is None or w.dtype != torch.uint8:
@@ -414,14 +417,18 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, *, Hq: int, Hkv: int, 
                       mask: Optional[torch.Tensor] = None, seg_q: Optional[torch.Tensor] = None,
                       seg_k: Optional[torch.Tensor] = None, scale: float = 0.0,
                       status: Optional[torch.Tensor] = None, max_kv_len: int = 0, slot: Optional[torch.Tensor] = None, chunk: int = 0,
-                      sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_by_head: bool = False,
+                      keep_first: int = 0, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Flash-style attention over ``q`` rows [tokens, Hq*hd]; KV from the paged pool or from
     contiguous ``k``/``v`` [rows, Hkv*hd] (may be column slices of a packed qkv buffer).
     ``max_kv_len``: a host-side bound on ``kv_len`` (0: unknown); short contiguous problems (at most 64 query rows per
     sequence over at most 512 keys, heads of 64 / 128, causal / window masks only) then take the low-latency kernel.
     Paged form: ``slot`` names every sequence's page-table row, ``chunk`` limits every position to its own chunk, ``sink`` ``[Hq]``
-    adds ``exp(sink)`` to the softmax denominators, the result is multiplied by ``sigmoid(gate)``."""
+    adds ``exp(sink)`` to the softmax denominators, the result is multiplied by ``sigmoid(gate)`` (``gate_by_head``: ``[rows, Hq]``),
+    the first ``keep_first`` positions stay visible behind a window or chunk, ``slopes`` ``[Hq]`` times the distance is taken off the
+    scores."""
     a = N.RfAttn()
+    a.gate_by_head, a.keep_first, a.slopes = int(gate_by_head), keep_first, _ptr(slopes)
     a.q, a.ldq, a.out, a.ldo = q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0)
     a.q_rows_total = q.shape[0]
     a.num_seqs, a.Hq, a.Hkv, a.hd = q_len.numel(), Hq, Hkv, hd
@@ -473,11 +480,13 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, *, Hq: int, Hkv: int, h
 
 def attention_rows(q: torch.Tensor, r, k_pool: torch.Tensor, v_pool: torch.Tensor, *, Hq: int, Hkv: int, hd: int, scale: float, max_kv: int,
                    chunk: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, split: bool = True,
-                   tensor_core: bool = True) -> torch.Tensor:
+                   tensor_core: bool = True, window: int = 0, gate_by_head: bool = False, keep_first: int = 0,
+                   slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Every row of ``q [rows, Hq * hd]`` over the cached keys of its sequence up to its own position (``r``: :func:`rows`), with the
     options of :func:`attention_prefill`.  ``tensor_core=False``: the fp32 kernel for any head size and dtype."""
     out = torch.empty((q.shape[0], Hq * hd), dtype=q.dtype, device=q.device)
     a = N.RfAttn()
+    a.window, a.gate_by_head, a.keep_first, a.slopes = window, int(gate_by_head), keep_first, _ptr(slopes)
     a.q, a.ldq, a.out, a.ldo, a.q_rows_total, a.num_seqs = q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), q.shape[0], q.shape[0]
     a.Hq, a.Hkv, a.hd, a.scale, a.max_kv_len, a.chunk, a.sink = Hq, Hkv, hd, scale, max_kv, chunk, _ptr(sink)
     a.k_pool, a.v_pool, a.pool_pages = k_pool.data_ptr(), v_pool.data_ptr(), k_pool.shape[0]
@@ -606,11 +615,12 @@ def stream_norm(x: Optional[torch.Tensor], r, *, dtype: torch.dtype, eps: float,
                 table: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None,
                 y_norm_w: Optional[torch.Tensor] = None, shift: Optional[torch.Tensor] = None,
                 shift_state: Optional[torch.Tensor] = None, dim: Optional[int] = None, cast: bool = False, embed_scale: float = 1.0,
-                y_slots: Optional[torch.Tensor] = None):
+                y_slots: Optional[torch.Tensor] = None, y_mult: float = 1.0, pairs: Optional[tuple] = None):
     """One step of an fp32 residual stream: add the outstanding sublayer output ``y`` (RMS-normed with ``y_norm_w``), RMSNorm
     with ``norm_w``, mix with the previous token's normalised row (``shift``, state per slot).  Without ``x`` the stream starts
     from ``table[ids] * embed_scale``.  ``y_slots [rows, picks]``: the outstanding output is the sum of these rows of ``y`` (negative:
-    none).  Returns ``(x_out fp32, h or None, x in dtype or None)``."""
+    none).  ``y_mult``: factor of the outstanding output.  ``pairs = (table2 [buckets + 1, H], last_token [slots], mul_prev, mul_cur)``:
+    the row of (previous token, token) is added to the embedding.  Returns ``(x_out fp32, h or None, x in dtype or None)``."""
     H = (x if x is not None else table).shape[1]
     n = x.shape[0] if x is not None else ids.numel()
     dev = (x if x is not None else table).device
@@ -621,18 +631,23 @@ def stream_norm(x: Optional[torch.Tensor], r, *, dtype: torch.dtype, eps: float,
     a.x, a.table, a.ids, a.y, a.y_norm_w = _ptr(x), _ptr(table), _ptr(ids), _ptr(y), _ptr(y_norm_w)
     a.x_out, a.x_cast, a.norm_w, a.out, a.shift, a.shift_state = _ptr(x_out), _ptr(xc), _ptr(norm_w), _ptr(h), _ptr(shift), _ptr(shift_state)
     a.rows, a.n_rows, a.H, a.dim, a.eps, a.dtype = r, n, H, dim or H, eps, dtype_code_any(dtype)
-    a.embed_scale, a.y_slots, a.y_picks = embed_scale, _i32(y_slots), 0 if y_slots is None else y_slots.shape[1]
+    a.embed_scale, a.y_slots, a.y_picks, a.y_mult = embed_scale, _i32(y_slots), 0 if y_slots is None else y_slots.shape[1], y_mult
+    if pairs is not None:
+        a.table2, a.last_token, a.mul_prev, a.mul_cur, a.buckets = pairs[0].data_ptr(), _i32(pairs[1]), pairs[2], pairs[3], pairs[0].shape[0] - 1
     N.check(N.lib().rf_stream_norm(C.byref(a), _stream()), "rf_stream_norm")
     return x_out, h, xc
 
 
-def gemm_f32(x: torch.Tensor, w: torch.Tensor, act: Optional[str] = None) -> torch.Tensor:
-    """``act(x @ w.T)`` in true fp32."""
+def gemm_f32(x: torch.Tensor, w: torch.Tensor, act: Optional[str] = None, *, dual: bool = False, limit: float = 0.0, alpha: float = 0.0,
+             row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``act(x @ w.T)`` in true fp32; ``dual``: ``w`` stacks the two operands of the activation."""
     assert x.dtype == torch.float32 and w.dtype == torch.float32 and x.stride(1) == 1 and w.stride(1) == 1
-    out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32, device=x.device)
+    n = w.shape[0] // 2 if dual else w.shape[0]
+    out = torch.empty((x.shape[0], n), dtype=torch.float32, device=x.device)
     g = N.RfGemm()
     g.x, g.ldx, g.w, g.ldw, g.out, g.ldo = x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0)
-    g.M, g.N, g.K, g.dtype, g.act = x.shape[0], w.shape[0], x.shape[1], 2, ACT[act]
+    g.M, g.N, g.K, g.dtype, g.act = x.shape[0], n, x.shape[1], 2, ACT[act]
+    g.dual_offset, g.act_limit, g.act_alpha, g.row_scale = n if dual else 0, limit, alpha, _ptr(row_scale)
     N.check(N.lib().rf_gemm_f32(C.byref(g), _stream()), "rf_gemm_f32")
     return out
 
@@ -708,10 +723,19 @@ def hgrn2(x: torch.Tensor, f_bias: torch.Tensor, lower: torch.Tensor, norm_w: Op
 def qkv_insert(qkv: torch.Tensor, r, k_pool: torch.Tensor, v_pool: torch.Tensor, *, heads: int, kv_heads: int, hd: int, eps: float,
                dim: Optional[int] = None, vdim: Optional[int] = None, q_norm: Optional[torch.Tensor] = None,
                k_norm: Optional[torch.Tensor] = None, cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None,
-               v_first: Optional[torch.Tensor] = None, v_role: str = "none", v_lambda: float = 0.0) -> None:
+               v_first: Optional[torch.Tensor] = None, v_role: str = "none", v_lambda: float = 0.0, norm_all: bool = False,
+               conv_w: Optional[torch.Tensor] = None, conv_state: Optional[torch.Tensor] = None, max_q_len: int = 1) -> torch.Tensor:
     """Per-head norms, rotation, value mixing and page insertion of packed rows ``[q | k | v]`` (heads of ``hd`` values, ``dim`` /
-    ``vdim`` of them used); queries are replaced in place, keys and values go to the pools ``[pages, kv_heads, 16, hd]``."""
+    ``vdim`` of them used); queries are replaced in place, keys and values go to the pools ``[pages, kv_heads, 16, hd]``.
+    ``norm_all``: one norm over all query heads (weight ``[heads, hd]``) and one over all key heads.  ``conv_w [taps, columns]``: causal
+    convolution ahead of the norms with carried rows in ``conv_state [slots, taps - 1, columns]``.  Returns the queries (a tensor of
+    their own with the convolution)."""
     a = N.RfQkvInsert()
+    q = qkv[:, :heads * hd]
+    if conv_w is not None:
+        q = torch.empty((qkv.shape[0], heads * hd), dtype=qkv.dtype, device=qkv.device)
+        a.conv_w, a.conv_state, a.q_out, a.taps, a.max_q_len = conv_w.data_ptr(), _ptr(conv_state), q.data_ptr(), conv_w.shape[0], max_q_len
+    a.norm_all = int(norm_all)
     a.qkv, a.ld, a.k_off, a.v_off = qkv.data_ptr(), qkv.stride(0), heads * hd, (heads + kv_heads) * hd
     a.q_norm, a.k_norm, a.cos, a.sin, a.v_first = _ptr(q_norm), _ptr(k_norm), _ptr(cos), _ptr(sin), _ptr(v_first)
     a.k_pool, a.v_pool, a.rows, a.n_rows = k_pool.data_ptr(), v_pool.data_ptr(), r, qkv.shape[0]
@@ -719,6 +743,7 @@ def qkv_insert(qkv: torch.Tensor, r, k_pool: torch.Tensor, v_pool: torch.Tensor,
     a.rot_dims = 0 if cos is None else 2 * cos.shape[1]
     a.v_role, a.v_lambda, a.eps, a.dtype = {"none": 0, "first": 1, "mix": 2}[v_role], v_lambda, eps, dtype_code_any(qkv.dtype)
     N.check(N.lib().rf_qkv_insert(C.byref(a), _stream()), "rf_qkv_insert")
+    return q
 
 
 def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor], r, *, max_q_len: int = 1) -> torch.Tensor:
@@ -750,12 +775,14 @@ def mamba1(x: torch.Tensor, z: torch.Tensor, bc: torch.Tensor, a2: torch.Tensor,
 
 # ----------------------------------------------------------------------------- mixture of experts
 class RoutedBatch:
-    """Router of one batch and everything its expert GEMMs need (:func:`moe_router`)."""
+    """Router of one batch and everything its expert GEMMs need (:func:`moe_router`).  ``score_fn="chosen"``: ``correction`` is a bias
+    of the logits and the weights are the softmax over the chosen ones; ``shared_gate``: the last row of ``w`` gives the logit of the
+    shared expert's sigmoid weight."""
 
     def __init__(self, x: torch.Tensor, w: torch.Tensor, k: int, *, correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1,
                  score_fn: str = "softmax", norm_topk: bool = True, scale: float = 1.0, tile_rows: int = 16, shared: bool = False,
-                 scatter: bool = True):
-        T, E = x.shape[0], w.shape[0]
+                 scatter: bool = True, shared_gate: bool = False):
+        T, E = x.shape[0], w.shape[0] - int(shared_gate)
         i32 = lambda *sh: torch.zeros(sh, dtype=torch.int32, device=x.device)
         self.x, self.w, self.correction, self.tile_rows, self.k = x, w, correction, tile_rows, k
         self.ids, self.weights, self.rank = i32(T, k), torch.zeros((T, k), dtype=torch.float32, device=x.device), i32(T, k)
@@ -764,13 +791,14 @@ class RoutedBatch:
         self.tiles = i32(4 * (self.max_tiles + 1))
         self.slot_of, self.token_of_slot = i32(T, k + shared), i32(T * (k + shared))
         self.slot_w = torch.zeros(T * (k + shared), dtype=torch.float32, device=x.device)
-        self.logits = torch.empty(N.lib().rf_moe_router_scratch_bytes(T, E), dtype=torch.uint8, device=x.device)
+        self.logits = torch.empty(N.lib().rf_moe_router_scratch_bytes(T, E + int(shared_gate)), dtype=torch.uint8, device=x.device)
         a = self.args = N.RfMoeRouter()
         a.x, a.ldx, a.w, a.correction = x.data_ptr(), x.stride(0), w.data_ptr(), _ptr(correction)
         a.ids, a.weights, a.rank, a.counters, a.start, a.tiles, a.slot_of, a.token_of_slot, a.slot_w = (t.data_ptr() for t in (
             self.ids, self.weights, self.rank, self.counters, self.start, self.tiles, self.slot_of, self.token_of_slot, self.slot_w))
         a.rows, a.experts, a.width, a.k, a.groups, a.keep = T, E, w.shape[1], k, groups, keep
-        a.score_fn, a.norm_topk, a.scale = {"sigmoid": 0, "softmax": 1}[score_fn], int(norm_topk), scale
+        a.score_fn, a.norm_topk, a.scale = {"sigmoid": 0, "softmax": 1, "chosen": 2}[score_fn], int(norm_topk), scale
+        a.shared_gate = int(shared_gate)
         a.tile_rows, a.slot_ld, a.has_shared, a.shared_tiles, a.scatter = tile_rows, k + shared, int(shared), int(shared and scatter), int(scatter)
         a.dtype, a.logits = dtype_code_any(x.dtype), self.logits.data_ptr()
 
@@ -792,7 +820,7 @@ def moe_router(x: torch.Tensor, w: torch.Tensor, k: int, **kw) -> RoutedBatch:
 
 def moe_experts(b: RoutedBatch, x: torch.Tensor, bank: torch.Tensor, *, n: int, k: int, experts: int, expert_pad: int = 0, dual: bool = False,
                 gathered: bool = True, weighted: bool = False, shared: Optional[torch.Tensor] = None, shared_n: int = 0, shared_k: int = 0,
-                out_cols: int = 0) -> torch.Tensor:
+                out_cols: int = 0, act: str = "silu_mul", limit: float = 0.0, alpha: float = 0.0, shared_limit: float = 0.0) -> torch.Tensor:
     """Expert GEMMs of few rows over the tile list of a routed batch; ``bank`` (and ``shared``) as the mixed engine packs them,
     ``expert_pad`` the padded expert width inside 16-bit banks."""
     cols = max(out_cols, n, shared_n)
@@ -808,6 +836,7 @@ def moe_experts(b: RoutedBatch, x: torch.Tensor, bank: torch.Tensor, *, n: int, 
     else:
         a.bank_kb_total, a.kb_per_expert, a.shared_kb_total = experts * expert_pad // 64, expert_pad // 64, up(shared_k, 64)
     a.dtype = dtype_code_any(x.dtype)
+    a.act, a.act_limit, a.act_alpha, a.shared_limit = ACT[act], limit, alpha, shared_limit
     N.check(N.lib().rf_moe_experts(C.byref(a), _stream()), "rf_moe_experts")
     return out
 
@@ -858,7 +887,7 @@ def moe_group(ids: torch.Tensor, w: torch.Tensor, E: int):
 def moe_grouped_gemm(x: torch.Tensor, bank: torch.Tensor, tiles: torch.Tensor, *, n: int, k: int, bank_rows: int,
                      bank_k: int, expert_rows: int = 0, expert_k: int = 0, dual: bool = False, act: Optional[str] = None,
                      row_scale: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
-                     status: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     status: Optional[torch.Tensor] = None, limit: float = 0.0, alpha: float = 0.0) -> torch.Tensor:
     """``out[s] = act(x[s] @ W_e.T) * row_scale[s]`` for every sorted row ``s`` of every expert ``e`` (see
     :func:`moe_group`).  ``bank`` is the ``pack_weight`` image of the whole expert bank: ``bank_rows`` rows per section
     (GLU banks have two sections: gates, then ups) and ``bank_k`` columns.  Experts are ``expert_rows`` rows apart
@@ -874,7 +903,7 @@ def moe_grouped_gemm(x: torch.Tensor, bank: torch.Tensor, tiles: torch.Tensor, *
     a.bank_section_row_tiles = (bank_rows + 127) // 128
     a.bank_kb_total = (bank_k + 63) // 64
     a.rt_per_expert, a.kb_per_expert = expert_rows // 128, expert_k // 64
-    a.dtype, a.status = dtype_code(x.dtype), _ptr(status)
+    a.dtype, a.status, a.act_limit, a.act_alpha = dtype_code(x.dtype), _ptr(status), limit, alpha
     N.check(N.lib().rf_moe_grouped_gemm(C.byref(a), _stream()), "rf_moe_grouped_gemm")
     return out
 
