@@ -237,7 +237,7 @@ def test_windows_kept_tokens_slopes_and_gates(form, mask, heads, kv, dim, vdim, 
             one = attend(form, qq, d, pt, kp, vp, total, lens, split=False, **kw).view(n, heads, hd)[..., :vdim]
             close(one, got, dtype)
         got = got.double().cpu()
-        for i in range(0, n, 1 if n < 50 else 5):
+        for i in range(0, n, 9):
             s = seq[i]
             close(got[i], expected(q[i].double(), k[s].double(), v[s].double(), pos[i], scale, mask, biased, not biased, gate[i].double()), dtype)
 
