@@ -10,8 +10,8 @@
 //  * prefill: one CTA per (64 query rows, q head, sequence); causal,
 //    bidirectional, sliding-window, boolean 2-D mask and segment-id (block
 //    diagonal / packed images) masking; GQA by kv head = q head / group.
-//  * decode: one CTA per (KV split, kv head, sequence); the GQA group's query
-//    heads are the MMA rows, every consumer warp owns one page per stage, warps
+//  * decode: one CTA per (KV split, kv head, sequence), over the whole sequence,
+//    a chunk or a window with kept first tokens; the GQA group's query heads are the MMA rows, every consumer warp owns one page per stage, warps
 //    and splits are merged with log-sum-exp weights.
 //
 // Replaces llm_fp16_32b_prefill_flash_attn_univ_* and its vctxlen / minibatch

@@ -260,8 +260,8 @@ typedef struct RfAttn {
   int32_t gate_by_head;     // 1: gate is [rows, Hq], one number per head
   int32_t keep_first;       // with a window: the first keep_first positions of the sequence stay visible
   const float* slopes;      // [Hq]: slopes[h] * (i - j) is taken off the scores of position i (paged forms)
-  // rf_attn_decode by row: with `pos`, query row r is position pos[r] of sequence seq_of_row[r] (null: r) and sees everything
-  // up to itself; kv_len is not used and num_seqs counts rows.
+  // rf_attn_decode by row: with `pos`, query row r is position pos[r] of sequence seq_of_row[r] (null: r) and sees what its
+  // chunk or window leaves of everything up to itself; kv_len is not used and num_seqs counts rows.
   const int32_t* seq_of_row; const int32_t* pos;
 } RfAttn;
 int rf_attn_prefill(const RfAttn* a, rf_stream_t stream);
