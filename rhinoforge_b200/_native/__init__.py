@@ -109,7 +109,7 @@ class RfAttn(C.Structure):
         ("ws", C.c_void_p), ("ws_bytes", C.c_uint64),
         ("status", C.c_void_p), ("dtype", C.c_int32),
         ("slot", C.c_void_p), ("chunk", C.c_int32), ("sink", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_int64),
-        ("gate_by_head", C.c_int32), ("keep_first", C.c_int32), ("slopes", C.c_void_p),
+        ("gate_by_head", C.c_int32), ("keep_first", C.c_int32), ("slopes", C.c_void_p), ("rates", C.c_void_p),
         ("seq_of_row", C.c_void_p), ("pos", C.c_void_p),
     ]
 
@@ -200,7 +200,8 @@ class RfStreamNorm(C.Structure):
                                           "shift", "shift_state")] + [("rows", RfRows)] + \
                [("n_rows", C.c_int32), ("H", C.c_int32), ("dim", C.c_int32), ("eps", C.c_float), ("dtype", C.c_int32),
                 ("embed_scale", C.c_float), ("y_slots", C.c_void_p), ("y_picks", C.c_int32), ("y_mult", C.c_float),
-                ("table2", C.c_void_p), ("last_token", C.c_void_p), ("mul_prev", C.c_int64), ("mul_cur", C.c_int64), ("buckets", C.c_int32)]
+                ("table2", C.c_void_p), ("last_token", C.c_void_p), ("mul_prev", C.c_int64), ("mul_cur", C.c_int64), ("buckets", C.c_int32),
+                ("y_self", C.c_void_p), ("y_self_w", C.c_void_p), ("conv_w", C.c_void_p), ("conv_state", C.c_void_p), ("conv_taps", C.c_int32)]
 
 
 class RfHeadLinear(C.Structure):
@@ -208,10 +209,29 @@ class RfHeadLinear(C.Structure):
                 ("ys", C.c_int32), ("w", C.c_void_p)] + [(n, C.c_int32) for n in ("rows", "heads", "n", "k", "dtype")]
 
 
+class RfLatentInsert(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64), ("norm_w", C.c_void_p), ("pool", C.c_void_p), ("rows", RfRows)] + \
+               [(n, C.c_int32) for n in ("n_rows", "rank", "rank_true")] + [("eps", C.c_float), ("rot", C.c_int32), ("rot_pad", C.c_int32)] + \
+               [("cos", C.c_void_p), ("sin", C.c_void_p), ("q", C.c_void_p), ("ldq", C.c_int64), ("q_norm", C.c_void_p), ("q_rank", C.c_int32),
+                ("q_rank_true", C.c_int32)]
+
+
+class RfHeadRotate(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64), ("xs", C.c_int32), ("y", C.c_void_p), ("ldy", C.c_int64), ("ys", C.c_int32)] + \
+               [(n, C.c_void_p) for n in ("pos", "cos", "sin")] + [(n, C.c_int32) for n in ("rows", "heads", "dims", "dims_pad")]
+
+
+class RfDelta(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64), ("b", C.c_void_p), ("a", C.c_void_p), ("ld_ba", C.c_int64), ("gate", C.c_void_p),
+                ("ldg", C.c_int64)] + [(n, C.c_void_p) for n in ("rate", "dt_bias", "norm_w", "state", "out")] + [("ldo", C.c_int64), ("rows", RfRows)] + \
+               [(n, C.c_int32) for n in ("heads", "kv_heads", "dim", "dim_true", "vdim", "vdim_true")] + \
+               [("eps", C.c_float), ("dtype", C.c_int32), ("conv_w", C.c_void_p), ("conv_state", C.c_void_p), ("taps", C.c_int32)]
+
+
 class RfLatentAttn(C.Structure):
     _fields_ = [("q", C.c_void_p), ("o", C.c_void_p), ("pool", C.c_void_p), ("rows", RfRows)] + \
                [(n, C.c_int32) for n in ("n_rows", "heads", "rank", "window", "max_kv")] + \
-               [("scale", C.c_float), ("dtype", C.c_int32), ("ws", C.c_void_p), ("ws_bytes", C.c_uint64)]
+               [("scale", C.c_float), ("dtype", C.c_int32), ("ws", C.c_void_p), ("ws_bytes", C.c_uint64), ("vrank", C.c_int32)]
 
 
 class RfHgrn2(C.Structure):
@@ -227,28 +247,32 @@ class RfMixedConfig(C.Structure):
                [("side_ld", C.c_int64), ("eps", C.c_float), ("weights_packed", C.c_int32), ("long_min", C.c_int32)] + \
                [(n, C.c_void_p) for n in ("embed", "side_table", "final_norm", "w_lm")] + \
                [("embed_scale", C.c_float), ("norm_after", C.c_int32), ("residual_mult", C.c_float), ("logit_softcap", C.c_float),
-                ("pair_table", C.c_void_p), ("pair_mul_prev", C.c_int64), ("pair_mul_cur", C.c_int64), ("pair_buckets", C.c_int32)]
+                ("pair_table", C.c_void_p), ("pair_mul_prev", C.c_int64), ("pair_mul_cur", C.c_int64), ("pair_buckets", C.c_int32), ("input_taps", C.c_int32)]
 
 
 class RfMixedState(C.Structure):
     _fields_ = [("latent_pool", C.c_void_p), ("k_pool", C.c_void_p), ("v_pool", C.c_void_p), ("pool_pages", C.c_int64),
-                ("rec_state", C.c_void_p), ("conv_state", C.c_void_p), ("shift_state", C.c_void_p), ("last_token", C.c_void_p)]
+                ("rec_state", C.c_void_p), ("conv_state", C.c_void_p), ("shift_state", C.c_void_p), ("last_token", C.c_void_p),
+                ("input_state", C.c_void_p * 2)]
 
 
 class RfMixedLayer(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "vdim", "vdim_true", "rank", "rank_true", "window", "expand_hd",
                                          "inter", "act")] + [("scale", C.c_float), ("in_dim", C.c_int32), ("out_dim", C.c_int32)] + \
-               [(n, C.c_void_p) for n in ("norm1", "norm2", "shift", "w_in", "w_o", "w_up", "w_down", "latent_norm", "w_absorb",
-                                          "w_unabsorb", "w_expand", "f_bias", "lower", "head_norm", "side_gate", "side_proj",
-                                          "side_norm")] + \
+               [(n, C.c_void_p) for n in ("norm1", "norm2", "shift", "w_in", "w_o", "w_up", "w_down", "latent_norm", "w_absorb", "w_unabsorb",
+                                          "w_expand")] + \
+               [(n, C.c_int32) for n in ("plain", "q_rank", "q_rank_true", "rot", "rot_pad", "shares")] + [("w_uq", C.c_void_p), ("q_latent_norm", C.c_void_p)] + \
+               [(n, C.c_void_p) for n in ("f_bias", "lower", "head_norm", "side_gate", "side_proj", "side_norm")] + \
                [(n, C.c_int32) for n in ("kv_heads", "dim_true", "tensor_core", "chunk", "gated", "rot_dims", "v_role")] + \
                [("v_lambda", C.c_float)] + [(n, C.c_void_p) for n in ("cos", "sin", "q_norm", "k_norm", "sink")] + \
-               [(n, C.c_int32) for n in ("keep_first", "norm_all", "gate_by_head", "conv_taps")] + [("slopes", C.c_void_p)] + \
+               [(n, C.c_int32) for n in ("keep_first", "norm_all", "gate_by_head", "conv_taps")] + [("slopes", C.c_void_p), ("rates", C.c_void_p), ("growth", C.c_float), ("growth_every", C.c_int32)] + \
                [(n, C.c_int32) for n in ("inner", "states", "dt_rank", "taps")] + \
                [(n, C.c_void_p) for n in ("conv_w", "conv_b", "a2", "d_skip", "dt_bias", "w_x", "w_dt", "w_dt_rows")] + \
                [(n, C.c_int32) for n in ("experts", "top", "groups", "keep", "score_fn", "norm_topk", "shared_inter", "bank_inter")] + \
                [("route_scale", C.c_float)] + [(n, C.c_void_p) for n in ("router", "correction", "shared_up", "shared_down")] + \
-               [(n, C.c_float) for n in ("act_limit", "act_alpha", "shared_limit")] + [("shared_gate", C.c_int32), ("st", RfMixedState)]
+               [(n, C.c_float) for n in ("act_limit", "act_alpha", "shared_limit")] + \
+               [("identity", C.c_int32), ("norm1b", C.c_void_p), ("norm2b", C.c_void_p), ("input_conv", C.c_void_p * 2), ("rate", C.c_void_p),
+                ("shared_gate", C.c_int32), ("st", RfMixedState)]
 
 
 class RfQkvInsert(C.Structure):
@@ -256,12 +280,12 @@ class RfQkvInsert(C.Structure):
                [(n, C.c_void_p) for n in ("q_norm", "k_norm", "cos", "sin", "v_first", "k_pool", "v_pool")] + [("rows", RfRows)] + \
                [(n, C.c_int32) for n in ("n_rows", "heads", "kv_heads", "hd", "dim", "vdim", "rot_dims", "v_role")] + \
                [("v_lambda", C.c_float), ("eps", C.c_float), ("dtype", C.c_int32), ("norm_all", C.c_int32), ("conv_w", C.c_void_p),
-                ("conv_state", C.c_void_p), ("q_out", C.c_void_p), ("taps", C.c_int32), ("max_q_len", C.c_int32)]
+                ("conv_state", C.c_void_p), ("q_out", C.c_void_p), ("taps", C.c_int32), ("max_q_len", C.c_int32), ("growth", C.c_float), ("growth_every", C.c_int32)]
 
 
 class RfConvSilu(C.Structure):
     _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64), ("y", C.c_void_p), ("ldy", C.c_int64), ("w", C.c_void_p), ("bias", C.c_void_p),
-                ("state", C.c_void_p), ("rows", RfRows)] + [(n, C.c_int32) for n in ("max_q_len", "channels", "taps", "dtype")]
+                ("state", C.c_void_p), ("rows", RfRows)] + [(n, C.c_int32) for n in ("max_q_len", "channels", "taps", "dtype", "add", "ring")]
 
 
 class RfMamba1(C.Structure):
@@ -277,7 +301,7 @@ class RfMoeRouter(C.Structure):
                                           "token_of_slot", "slot_w")] + \
                [(n, C.c_int32) for n in ("rows", "experts", "width", "k", "groups", "keep", "score_fn", "norm_topk")] + \
                [("scale", C.c_float)] + [(n, C.c_int32) for n in ("tile_rows", "slot_ld", "has_shared", "shared_tiles", "scatter", "dtype")] + \
-               [("logits", C.c_void_p), ("shared_gate", C.c_int32)]
+               [("logits", C.c_void_p), ("shared_gate", C.c_int32), ("identity", C.c_int32), ("self_w", C.c_void_p)]
 
 
 class RfMoeExperts(C.Structure):

@@ -13,6 +13,7 @@ BUILTIN_ADAPTERS = (
     ("Vabarax", "rhinoforge_b200.adapters.vabarax", "VabaraxAdapter"),
     ("Zulopel", "rhinoforge_b200.adapters.zulopel", "ZulopelAdapter"),
     ("Kuzupel", "rhinoforge_b200.adapters.kuzupel", "KuzupelAdapter"),
+    ("Vasosun", "rhinoforge_b200.adapters.vasosun", "VasosunAdapter"),
 )
 
 __all__ = ["BUILTIN_ADAPTERS"]

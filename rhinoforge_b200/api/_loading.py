@@ -22,6 +22,7 @@ _ROUTES = {
     "Vabarax": "use RPUModelForCausalLM.from_pretrained(..., device='rpu')",
     "Zulopel": "use RPUModelForCausalLM.from_pretrained(..., device='rpu')",
     "Kuzupel": "use RPUModelForCausalLM.from_pretrained(..., device='rpu')",
+    "Vasosun": "use RPUModelForCausalLM.from_pretrained(..., device='rpu')",
 }
 
 

@@ -29,7 +29,7 @@ class RPUModelForCausalLM:
 
     _RESERVED_HF_KWARGS = frozenset({"torch_dtype", "dtype", "device_map", "device", "low_cpu_mem_usage", "tp_plan",
                                      "load_in_8bit", "load_in_4bit", "quantization_config"})
-    _SUPPORTED_BUILTIN_ARCHITECTURES = frozenset({"LlamaForCausalLM", "Qwen3ForCausalLM", "Vabarax", "Zulopel", "Kuzupel"})
+    _SUPPORTED_BUILTIN_ARCHITECTURES = frozenset({"LlamaForCausalLM", "Qwen3ForCausalLM", "Vabarax", "Zulopel", "Kuzupel", "Vasosun"})
     _CONFIG_KWARGS = frozenset({"cache_dir", "revision", "subfolder", "local_files_only", "token", "force_download",
                                 "proxies"})
     SUPPORTED_DTYPES = (torch.float16, torch.bfloat16)

@@ -170,8 +170,14 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     uint32_t qf[HD / 16][4];
     float fall0 = 0.f, fall1 = 0.f;                // what the two rows' scores lose per token of distance
     if (p.slopes) {
-      if ((lane >> 2) < G) fall0 = p.slopes[head0 + (lane >> 2)] * kLog2e;
-      if ((lane >> 2) + 8 < G) fall1 = p.slopes[head0 + (lane >> 2) + 8] * kLog2e;
+      const float unit = p.rates ? 1.f : kLog2e;   // with rates the logarithm is one to the base of two already
+      if ((lane >> 2) < G) fall0 = p.slopes[head0 + (lane >> 2)] * unit;
+      if ((lane >> 2) + 8 < G) fall1 = p.slopes[head0 + (lane >> 2) + 8] * unit;
+    }
+    float rate0 = 0.f, rate1 = 0.f;
+    if (p.rates) {
+      if ((lane >> 2) < G) rate0 = p.rates[head0 + (lane >> 2)];
+      if ((lane >> 2) + 8 < G) rate1 = p.rates[head0 + (lane >> 2) + 8];
     }
     {
       const int g0 = lane >> 2, g1 = g0 + 8;
@@ -206,8 +212,13 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
         for (int e = 0; e < 4; ++e) {
           const int t0 = tok0 + (e & 1), t1 = tok0 + 8 + (e & 1);
           const float fall = e < 2 ? fall0 : fall1;
-          x[0][e] = t0 < kvlen && (t0 >= kvlo || t0 < p.keep_first) ? s0[e] * p.scale_log2 - fall * (float)(kvlen - 1 - t0) : -INFINITY;
-          x[1][e] = t1 < kvlen && (t1 >= kvlo || t1 < p.keep_first) ? s1[e] * p.scale_log2 - fall * (float)(kvlen - 1 - t1) : -INFINITY;
+          float d0 = (float)(kvlen - 1 - t0), d1 = (float)(kvlen - 1 - t1);
+          if (p.rates) {
+            d0 = log2_distance(e < 2 ? rate0 : rate1, d0);
+            d1 = log2_distance(e < 2 ? rate0 : rate1, d1);
+          }
+          x[0][e] = t0 < kvlen && (t0 >= kvlo || t0 < p.keep_first) ? s0[e] * p.scale_log2 - fall * d0 : -INFINITY;
+          x[1][e] = t1 < kvlen && (t1 >= kvlo || t1 < p.keep_first) ? s1[e] * p.scale_log2 - fall * d1 : -INFINITY;
         }
         const float mx0 = quad_max(fmaxf(fmaxf(x[0][0], x[0][1]), fmaxf(x[1][0], x[1][1])));
         const float mx1 = quad_max(fmaxf(fmaxf(x[0][2], x[0][3]), fmaxf(x[1][2], x[1][3])));
@@ -546,9 +557,10 @@ static int fill_params(const RfAttn* a, AttnParams* p) {
   p->scale_log2 = scale * 1.4426950408889634f;
   if (a->slot || a->chunk > 0 || a->pos || a->keep_first > 0 || a->slopes)
     RF_REQUIRE(paged, "slots, chunks, kept first positions, distance slopes and attention by row need the paged pool");
+  RF_REQUIRE(!a->rates || a->slopes, "the rates of a logarithmic fall need its slopes");
   if (a->slopes || a->keep_first > 0) RF_REQUIRE(!a->mask && !a->seg_q, "distance slopes and kept first positions do not go with data-dependent masks");
   p->slot = a->slot; p->chunk = a->chunk; p->sink = a->sink; p->gate = a->gate; p->ld_gate = a->ld_gate;
-  p->gate_by_head = a->gate_by_head; p->keep_first = a->window > 0 || a->chunk > 0 ? std::max(a->keep_first, 0) : 0; p->slopes = a->slopes;
+  p->gate_by_head = a->gate_by_head; p->keep_first = a->window > 0 || a->chunk > 0 ? std::max(a->keep_first, 0) : 0; p->slopes = a->slopes; p->rates = a->rates;
   p->seq_of_row = a->seq_of_row; p->pos = a->pos; p->g_tiles = ceil_div(p->G, 16);
   p->ws_o = nullptr; p->ws_lse = nullptr; p->splits = 1; p->pages_per_split = 1 << 28; p->stages = 2;
   p->status = a->status;

@@ -240,7 +240,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     int lo_row = p.window > 0 ? qpos0 + qi - p.window + 1 : 0;
     if (p.chunk > 0) lo_row = max(lo_row, (qpos0 + qi) / p.chunk * p.chunk);
     const bool data_mask = mrow != nullptr || p.seg_q != nullptr;
-    const float fall = p.slopes ? p.slopes[h] * kLog2e : 0.f;
+    const float fall = p.slopes ? p.slopes[h] * (p.rates ? 1.f : kLog2e) : 0.f, rate = p.rates ? p.rates[h] : 0.f;
     const float score_mul = p.slopes ? 1.f : p.scale_log2;
     for (int j = 0; j < nblk; ++j) {
       const int b = j & 1;
@@ -260,7 +260,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       // masking: interior blocks need none; edge blocks compare against the row's [lo, hi]; boolean
       // masks and segment ids (rare) take the per-element path
       const bool edge = __any_sync(0xffffffffu, (t0 < lo_row && t0 + KVB > p.keep_first) || t0 + KVB - 1 > hi_row) || data_mask;
-      if (p.slopes) {                                       // finished scores: scaled, less the fall over the distance
+      if (p.rates) {                                        // finished scores: scaled, less the fall over the distance's logarithm
+        const float back = (float)(qpos0 + qi - t0);
+#pragma unroll
+        for (int i = 0; i < KVB; ++i)
+          sv[i] = __float_as_uint(fmaf(-fall, log2_distance(rate, back - (float)i), __uint_as_float(sv[i]) * p.scale_log2));
+      } else if (p.slopes) {                                // ... or over the distance
         const float past = (float)(t0 - qpos0 - qi);
 #pragma unroll
         for (int i = 0; i < KVB; ++i)

@@ -26,12 +26,19 @@ struct AttnParams {
   const float* sink;      // natural-log units
   const void* gate; int64_t ld_gate;
   int32_t gate_by_head, keep_first;
-  const float* slopes;    // natural-log units per token of distance
+  const float* slopes;    // natural-log units per token of distance, or per unit of ln(1 + rate * distance)
+  const float* rates;
   const int32_t* seq_of_row; const int32_t* pos;
   int32_t g_tiles;        // decode: CTAs that share one K/V head (16 query heads each)
 };
 
 constexpr float kLog2e = 1.4426950408889634f;
+// log2(1 + rate * distance); distances in front of a row (masked by the caller) may give anything
+__device__ __forceinline__ float log2_distance(float rate, float distance) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(fmaf(rate, distance, 1.f)));
+  return y;
+}
 __device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 
 

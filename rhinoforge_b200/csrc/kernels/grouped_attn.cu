@@ -59,6 +59,13 @@ __device__ __forceinline__ void finish_head(const RfQkvInsert& p, const HeadItem
       }
     }
   }
+  if (it.is_q && p.growth_every > 0) {             // queries grow with their position
+    const float f = 1.f + p.growth * logf((float)((pos + 1) / p.growth_every) + 1.f);
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[c][j] *= f;
+  }
   const int half = p.rot_dims >> 1;                // uniform over the grid
   if (NC == 1 && half > 0 && half % 8 == 0) {
     // whole lanes turn with one another: dimensions of lane l with those of lane l + half / 8
@@ -332,7 +339,8 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const RfAttn p) {
     const T* v = reinterpret_cast<const T*>(p.v_pool) + at;
     float s = 0.f;
     for (int i = lane; i < hd; i += 32) s += q[i] * Num<T>::to_f(k[i]);
-    s = warp_sum(s) * p.scale - fall * (float)(pos - j);
+    const float dist = (float)(pos - j);
+    s = warp_sum(s) * p.scale - fall * (p.rates ? logf(1.f + p.rates[h] * dist) : dist);
     const float mn = fmaxf(m, s), keep = expf(m - mn), w = expf(s - mn);
     l = l * keep + w;
     m = mn;
@@ -424,6 +432,7 @@ extern "C" int rf_qkv_insert(const RfQkvInsert* a, rf_stream_t stream) {
              "qkv_insert: rotation of %d dimensions", a->rot_dims);
   RF_REQUIRE(a->v_role == RF_VMIX_NONE || a->v_first, "qkv_insert: value mixing needs the first values");
   RF_REQUIRE(a->dtype >= 0 && a->dtype <= 2, "qkv_insert: dtype %d", a->dtype);
+  RF_REQUIRE(a->growth_every >= 0, "qkv_insert: growth of the queries");
   if (a->taps > 0) {
     RF_REQUIRE(a->conv_w && a->q_out && a->q_out != a->qkv && (a->taps == 1 || a->conv_state) && !a->norm_all,
                "qkv_insert: the convolution needs weights, its state and an output for the queries, and per-head norms");
@@ -444,6 +453,7 @@ extern "C" int rf_attn_rows(const RfAttn* a, rf_stream_t stream) {
   RF_REQUIRE(a && a->q && a->out && a->k_pool && a->v_pool && a->page_table && a->pos, "attn_rows: missing buffers");
   RF_REQUIRE(a->hd > 0 && a->hd <= 2048 && a->Hkv > 0 && a->Hq % a->Hkv == 0, "attn_rows: heads");
   RF_REQUIRE(a->keep_first >= 0 && !a->mask && !a->seg_q && a->dtype >= 0 && a->dtype <= 2, "attn_rows: options");
+  RF_REQUIRE(!a->rates || a->slopes, "attn_rows: the rates of a logarithmic fall need its slopes");
   RF_REQUIRE(a->num_seqs <= 65535, "attn_rows: %d rows in one launch", a->num_seqs);
   if (a->num_seqs == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);

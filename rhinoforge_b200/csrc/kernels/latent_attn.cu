@@ -15,30 +15,87 @@ __device__ __forceinline__ int row_seq(const RfRows& r, int row) { return r.seq_
 __device__ __forceinline__ int seq_slot(const RfRows& r, int seq) { return r.slot ? r.slot[seq] : seq; }
 
 // --------------------------------------------------------------- cache rows ----
-// One warp normalises one row and stores it at its position.
+// 1 / rms of n values of a row, eight per lane and step (all lanes of the warp); dim: what the mean runs over.
+template <typename T>
+__device__ __forceinline__ float row_rstd(const T* x, int n, int dim, float eps, int lane) {
+  float s = 0.f;
+  for (int i = lane * 8; i < n; i += 256) {
+    float f[8];
+    load8(x + i, f);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s += f[j] * f[j];
+  }
+  return rsqrtf(warp_sum(s) / (float)dim + eps);
+}
+template <typename T>
+__device__ __forceinline__ void scale_row(const T* x, T* y, const float* w, int n, float rstd, int lane) {
+  for (int i = lane * 8; i < n; i += 256) {
+    float f[8], g[8];
+    load8(x + i, f);
+    load8(w + i, g);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) f[j] *= rstd * g[j];
+    store8(y + i, f);
+  }
+}
+// Eight neighbouring values, from dimension c on, of `dims` rotated ones at one position.
+template <typename T>
+__device__ __forceinline__ void rotate8(const T* x, T* y, const float* cos, const float* sin, int pos, int c, int dims) {
+  float f[8];
+  load8(x + c, f);
+  const size_t at = (size_t)pos * (dims >> 1) + (c >> 1);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    if (c + 2 * i < dims) {
+      const float co = cos[at + i], si = sin[at + i], u = f[2 * i], v = f[2 * i + 1];
+      f[2 * i] = u * co - v * si;
+      f[2 * i + 1] = v * co + u * si;
+    } else {
+      f[2 * i] = f[2 * i + 1] = 0.f;
+    }
+  }
+  store8(y + c, f);
+}
+template <typename T>
+__device__ __forceinline__ void head_rotate_item(const RfHeadRotate& p, int64_t i) {
+  const int per = p.dims_pad / 8, c = (int)(i % per) * 8;
+  const int64_t rh = i / per;
+  if (rh >= (int64_t)p.rows * p.heads) return;
+  const int row = (int)(rh / p.heads), h = (int)(rh % p.heads);
+  rotate8(reinterpret_cast<const T*>(p.x) + (size_t)row * p.ldx + (size_t)h * p.xs, reinterpret_cast<T*>(p.y) + (size_t)row * p.ldy + (size_t)h * p.ys,
+          p.cos, p.sin, p.pos[row], c, p.dims);
+}
+
+// One warp normalises one row's latent and stores it at its position, together with the rotated part.
 template <typename T>
 __device__ __forceinline__ void latent_insert_row(const RfLatentInsert& p, int row, int lane) {
   const T* xr = reinterpret_cast<const T*>(p.x) + (size_t)row * p.ldx;
-  float s = 0.f;
-  for (int i = lane * 2; i < p.rank; i += 64) {
-    const float a = Num<T>::to_f(xr[i]), b = Num<T>::to_f(xr[i + 1]);
-    s += a * a + b * b;
-  }
   const int pos = p.rows.pos[row];
   const int page = p.rows.page_table[(size_t)seq_slot(p.rows, row_seq(p.rows, row)) * p.rows.pt_stride + (pos >> 4)];
-  const float rstd = rsqrtf(warp_sum(s) / (float)p.rank_true + p.eps);
-  T* dst = reinterpret_cast<T*>(p.pool) + ((size_t)page * 16 + (pos & 15)) * p.rank;
-  for (int i = lane * 2; i < p.rank; i += 64) {
-    dst[i] = Num<T>::from_f(Num<T>::to_f(xr[i]) * rstd * p.norm_w[i]);
-    dst[i + 1] = Num<T>::from_f(Num<T>::to_f(xr[i + 1]) * rstd * p.norm_w[i + 1]);
+  T* dst = reinterpret_cast<T*>(p.pool) + ((size_t)page * 16 + (pos & 15)) * (p.rank + p.rot_pad);
+  for (int c = lane * 8; c < p.rot_pad; c += 256) rotate8(xr + p.rank, dst + p.rank, p.cos, p.sin, pos, c, p.rot);
+  scale_row(xr, dst, p.norm_w, p.rank, row_rstd(xr, p.rank, p.rank_true, p.eps, lane), lane);
+}
+
+// A warp per row and part: the cached row (with x), the query latent (with q).
+template <typename T>
+__global__ void latent_insert_kernel(const RfLatentInsert p) {
+  pdl_prologue();
+  const int item = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31, parts = (p.x ? 1 : 0) + (p.q ? 1 : 0);
+  const int row = item / parts;
+  if (row >= p.n_rows) return;
+  if (p.x && item % parts == 0) {
+    latent_insert_row<T>(p, row, lane);
+  } else {
+    T* q = reinterpret_cast<T*>(p.q) + (size_t)row * p.ldq;
+    scale_row(q, q, p.q_norm, p.q_rank, row_rstd(q, p.q_rank, p.q_rank_true, p.eps, lane), lane);
   }
 }
 
 template <typename T>
-__global__ void latent_insert_kernel(const RfLatentInsert p) {
+__global__ void __launch_bounds__(256) head_rotate_kernel(const RfHeadRotate p) {
   pdl_prologue();
-  const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (row < p.n_rows) latent_insert_row<T>(p, row, threadIdx.x & 31);
+  head_rotate_item<T>(p, (int64_t)blockIdx.x * blockDim.x + threadIdx.x);
 }
 
 template <typename T>
@@ -105,12 +162,14 @@ template <int N> __device__ __forceinline__ void la_wait() { asm volatile("cp.as
 constexpr int kHmRows = 64, kHmK = 64, kHmLd = kHmK + 8, kHmStages = 4;
 
 template <typename T, int NT>
-__global__ void __launch_bounds__(128) head_linear_mma_kernel(const RfHeadLinear p, const RfLatentInsert ins, int row_tiles) {
+__global__ void __launch_bounds__(128) head_linear_mma_kernel(const RfHeadLinear p, const RfLatentInsert ins, const RfHeadRotate turn, int row_tiles) {
   pdl_launch_dependents();
-  if ((int)blockIdx.z >= row_tiles) {    // the grid's last planes insert latent rows, one per warp
+  if ((int)blockIdx.z >= row_tiles) {    // the grid's last planes insert latent rows, one per warp, then rotate, eight values per thread
     pdl_wait();
-    const int row = ((((int)blockIdx.z - row_tiles) * gridDim.y + blockIdx.y) * gridDim.x + blockIdx.x) * 4 + (threadIdx.x >> 5);
+    const int block = (((int)blockIdx.z - row_tiles) * gridDim.y + blockIdx.y) * gridDim.x + blockIdx.x, ins_blocks = (ins.n_rows + 3) / 4;
+    const int row = block * 4 + (threadIdx.x >> 5);
     if (row < ins.n_rows) latent_insert_row<T>(ins, row, threadIdx.x & 31);
+    if (block >= ins_blocks && turn.rows > 0) head_rotate_item<T>(turn, (int64_t)(block - ins_blocks) * 128 + threadIdx.x);
     return;
   }
   constexpr int BN = NT * 32;
@@ -190,16 +249,18 @@ __global__ void __launch_bounds__(128) head_linear_mma_kernel(const RfHeadLinear
 }
 
 template <typename T>
-static int launch_head_linear_mma(const RfHeadLinear* a, const RfLatentInsert* c, cudaStream_t s) {
+static int launch_head_linear_mma(const RfHeadLinear* a, const RfLatentInsert* c, const RfHeadRotate* t, cudaStream_t s) {
   const int rt = ceil_div(a->rows, kHmRows);
   const RfLatentInsert ins = c ? *c : RfLatentInsert{};
+  const RfHeadRotate turn = t ? *t : RfHeadRotate{};
+  const int extra = ceil_div(ins.n_rows, 4) + (int)(((int64_t)turn.rows * turn.heads * (turn.dims_pad / 8) + 127) / 128);
 #define RF_HM(NT)                                                                                                            \
   do {                                                                                                                       \
     constexpr size_t smem = (size_t)kHmStages * (kHmRows + NT * 32) * kHmLd * 2;                                              \
     const int gx = ceil_div(a->n, NT * 32);                                                                                  \
-    const dim3 grid(gx, a->heads, rt + ceil_div(ceil_div(ins.n_rows, 4), gx * a->heads));                                    \
+    const dim3 grid(gx, a->heads, rt + ceil_div(extra, gx * a->heads));                                                        \
     RF_ALLOW_SMEM_PER_DEVICE((head_linear_mma_kernel<T, NT>), smem);                                                         \
-    RF_CUDA_CHECK(::rf::launch_k(head_linear_mma_kernel<T, NT>, grid, dim3(128), smem, s, 1, *a, ins, rt)); \
+    RF_CUDA_CHECK(::rf::launch_k(head_linear_mma_kernel<T, NT>, grid, dim3(128), smem, s, 1, *a, ins, turn, rt)); \
   } while (0)
   if ((long)ceil_div(a->n, 64) * a->heads * rt < sm_count()) RF_HM(1);
   else RF_HM(2);
@@ -242,6 +303,7 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const RfLatentAttn p) 
 #pragma unroll
     for (int i = 0; i < RPL; ++i) acc[i] = acc[i] * corr + w * cv[i];
   }
+  const int vrank = p.vrank > 0 ? p.vrank : rank;
   float* sml = sm + 4 * rank;
 #pragma unroll
   for (int i = 0; i < RPL; ++i)
@@ -255,8 +317,8 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const RfLatentAttn p) 
     f[w] = sml[w] == -INFINITY ? 0.f : expf(sml[w] - mm);
     tot += f[w] * sml[4 + w];
   }
-  T* o = reinterpret_cast<T*>(p.o) + ((size_t)row * p.heads + h) * rank;
-  for (int i = threadIdx.x; i < rank; i += 128) {
+  T* o = reinterpret_cast<T*>(p.o) + ((size_t)row * p.heads + h) * vrank;
+  for (int i = threadIdx.x; i < vrank; i += 128) {
     float v = 0.f;
     for (int w = 0; w < 4; ++w) v += f[w] * sm[w * rank + i];
     o[i] = Num<T>::from_f(v / tot);
@@ -278,6 +340,8 @@ struct LatentSplit {
 
 template <int NT, int MT> struct LaGeom {
   static constexpr int W = NT >= 2 ? 16 : 8, KG = W / 2;            // warps; shares of the latent columns
+  static constexpr int steps = NT * 4, KS = (steps + KG - 1) / KG;  // k16 steps of all columns, of the largest share
+  static constexpr int out = NT * 64 > 512 ? 512 : NT * 64, NTW = (out / 8 + W - 1) / W;   // value columns at most, output tiles per warp
   static constexpr int M = 16 * MT, LD = NT * 64 + 8, LDS = kLaKeys + 4, LDP = kLaKeys + 8;
   static constexpr int c = 0;                                       // [2][64][LD] key blocks (the queries pass through here first)
   static constexpr int s = c + 2 * kLaKeys * LD * 2;                // [KG][M][LDS] partial scores
@@ -291,9 +355,9 @@ __global__ void __launch_bounds__(32 * LaGeom<NT, MT>::W, 1) latent_attn_mma_ker
   pdl_prologue();
   using L = LaGeom<NT, MT>;
   constexpr int M = L::M, ld = L::LD, LDS = L::LDS, LDP = L::LDP, RP = NT * 64;
-  constexpr int W = L::W, KG = L::KG, kThreads = 32 * W, KS = RP / KG / 16, NTW = RP / W / 8;   // k16 steps of a share, output tiles per warp
+  constexpr int W = L::W, KG = L::KG, kThreads = 32 * W, KS = L::KS, NTW = L::NTW;
   extern __shared__ __align__(16) uint8_t lsm[];
-  const int rank = p.rank;
+  const int rank = p.rank, vrank = p.vrank > 0 ? p.vrank : rank;
   T* sC = reinterpret_cast<T*>(lsm + L::c);
   float* sS = reinterpret_cast<float*>(lsm + L::s);
   T* sP = reinterpret_cast<T*>(lsm + L::p);
@@ -311,6 +375,8 @@ __global__ void __launch_bounds__(32 * LaGeom<NT, MT>::W, 1) latent_attn_mma_ker
   const T* q = reinterpret_cast<const T*>(p.q) + ((size_t)row * p.heads + h0) * rank;
   const int heads_here = min(M, p.heads - h0);
   const int kq = warp >> 1, key0 = (warp & 1) * 32;        // this warp's column share and key half for the scores
+  const int k0 = kq * L::steps / KG, kn = (kq + 1) * L::steps / KG - k0;
+  constexpr bool kEven = L::steps % KG == 0;
 
   for (int i = tid; i < M * (RP / 8); i += kThreads) {
     const int r = i / (RP / 8), c = (i % (RP / 8)) * 8;
@@ -326,7 +392,7 @@ __global__ void __launch_bounds__(32 * LaGeom<NT, MT>::W, 1) latent_attn_mma_ker
   for (int m = 0; m < MT; ++m)
 #pragma unroll
     for (int k = 0; k < KS; ++k)
-      ldsm_x4(smem_u32(sC + (m * 16 + (lane & 15)) * ld + kq * KS * 16 + k * 16 + (lane >> 4) * 8), qf[m][k][0], qf[m][k][1], qf[m][k][2], qf[m][k][3]);
+      if (kEven || k < kn) ldsm_x4(smem_u32(sC + (m * 16 + (lane & 15)) * ld + (k0 + k) * 16 + (lane >> 4) * 8), qf[m][k][0], qf[m][k][1], qf[m][k][2], qf[m][k][3]);
   __syncthreads();
   auto load_keys = [&](int b) {
     constexpr int TPR = kThreads / kLaKeys;                // threads per key row
@@ -357,8 +423,9 @@ __global__ void __launch_bounds__(32 * LaGeom<NT, MT>::W, 1) latent_attn_mma_ker
       for (int k = 0; k < KS; ++k)
 #pragma unroll
         for (int np = 0; np < 2; ++np) {                   // sixteen keys, one k16 step
+          if (!kEven && k >= kn) continue;
           uint32_t bf[4];
-          ldsm_x4(smem_u32(kc + (key0 + np * 16 + (lane >> 4) * 8 + (lane & 7)) * ld + kq * KS * 16 + k * 16 + ((lane >> 3) & 1) * 8), bf[0], bf[1], bf[2], bf[3]);
+          ldsm_x4(smem_u32(kc + (key0 + np * 16 + (lane >> 4) * 8 + (lane & 7)) * ld + (k0 + k) * 16 + ((lane >> 3) & 1) * 8), bf[0], bf[1], bf[2], bf[3]);
 #pragma unroll
           for (int m = 0; m < MT; ++m) {
             MmaOp<T>::mma(s[m][np * 2], qf[m][k], bf[0], bf[1]);
@@ -444,8 +511,8 @@ __global__ void __launch_bounds__(32 * LaGeom<NT, MT>::W, 1) latent_attn_mma_ker
                     a[m][hl][hk][2], a[m][hl][hk][3]);
 #pragma unroll
       for (int t = 0; t < NTW; ++t) {
-        const int c = (warp * NTW + t) * 8;
-        {
+        const int c = (warp + t * W) * 8;
+        if (c < vrank) {
           uint32_t bf[4];                                  // eight columns, 32 keys
           ldsm_x4_t(smem_u32(kc + (kk + lane) * ld + c), bf[0], bf[1], bf[2], bf[3]);
 #pragma unroll
@@ -472,11 +539,11 @@ __global__ void __launch_bounds__(32 * LaGeom<NT, MT>::W, 1) latent_attn_mma_ker
       const float inv = sp.splits == 1 ? 1.f / sL[r] : 1.f;
 #pragma unroll
       for (int t = 0; t < NTW; ++t) {
-        const int c = (warp * NTW + t) * 8 + q4 * 2;
-        if (c >= rank) continue;
+        const int c = (warp + t * W) * 8 + q4 * 2;
+        if (c >= vrank) continue;
         const float v0 = acc[m][t][half * 2] * inv, v1 = acc[m][t][half * 2 + 1] * inv;
-        if (sp.splits == 1) *reinterpret_cast<uint32_t*>(reinterpret_cast<T*>(p.o) + hr * rank + c) = MmaOp<T>::pack(v0, v1);
-        else *reinterpret_cast<float2*>(sp.o + (hr * sp.splits + split) * rank + c) = make_float2(v0, v1);
+        if (sp.splits == 1) *reinterpret_cast<uint32_t*>(reinterpret_cast<T*>(p.o) + hr * vrank + c) = MmaOp<T>::pack(v0, v1);
+        else *reinterpret_cast<float2*>(sp.o + (hr * sp.splits + split) * vrank + c) = make_float2(v0, v1);
       }
       if (sp.splits > 1 && warp == 0 && q4 == 0) {
         sp.ml[(hr * sp.splits + split) * 2] = sM[r];
@@ -540,21 +607,43 @@ static int check_rows(const RfRows* r) {
 }
 
 static int check_insert(const RfLatentInsert* c) {
-  RF_REQUIRE(c && c->x && c->norm_w && c->pool && c->rank > 0 && c->rank % 16 == 0 && c->rank_true > 0 && c->rank_true <= c->rank,
-             "latent_insert arguments");
+  RF_REQUIRE(c && (c->x || c->q), "latent_insert: neither latents nor query latents");
+  if (c->x) {
+    RF_REQUIRE(c->norm_w && c->pool && c->rank > 0 && c->rank % 16 == 0 && c->rank_true > 0 && c->rank_true <= c->rank && c->ldx % 8 == 0, "latent_insert arguments");
+    RF_REQUIRE(c->rot >= 0 && c->rot % 2 == 0 && c->rot_pad >= c->rot && c->rot_pad % 16 == 0 && (c->rot_pad == 0 || (c->rot > 0 && c->cos && c->sin)),
+               "latent_insert: rotated part of %d values", c->rot);
+  }
+  if (c->q) RF_REQUIRE(c->q_norm && c->q_rank > 0 && c->q_rank % 8 == 0 && c->ldq % 8 == 0 && c->q_rank_true > 0 && c->q_rank_true <= c->q_rank, "latent_insert: query latents");
   return check_rows(&c->rows);
 }
 
-extern "C" int rf_latent_insert(const void* x, int64_t ldx, const float* norm_w, void* pool, const RfRows* rows, int32_t n_rows,
-                                int32_t rank, int32_t rank_true, float eps, int32_t dtype, rf_stream_t stream) {
+extern "C" int rf_latent_insert(const RfLatentInsert* c, int32_t dtype, rf_stream_t stream) {
   RF_SKIP_IF_REPLAYING();
-  RF_REQUIRE(rows, "latent_insert: no rows");
-  const RfLatentInsert c = {x, ldx, norm_w, pool, *rows, n_rows, rank, rank_true, eps};
-  int rc = check_insert(&c);
+  int rc = check_insert(c);
   if (rc) return rc;
-  if (n_rows == 0) return RF_OK;
+  if (c->n_rows == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  RF_DISPATCH3(dtype, RF_CUDA_CHECK(::rf::launch_k(latent_insert_kernel<T>, dim3(ceil_div(n_rows, 4)), dim3(128), 0, s, 1, c)));
+  const int items = c->n_rows * ((c->x ? 1 : 0) + (c->q ? 1 : 0));
+  RF_DISPATCH3(dtype, RF_CUDA_CHECK(::rf::launch_k(latent_insert_kernel<T>, dim3(ceil_div(items, 4)), dim3(128), 0, s, 1, *c)));
+  ::rf::count_launch();
+  return RF_OK;
+}
+
+static int check_rotate(const RfHeadRotate* a) {
+  RF_REQUIRE(a && a->x && a->y && a->pos && a->cos && a->sin && a->heads > 0 && a->dims > 0 && a->dims % 2 == 0 && a->dims_pad >= a->dims && a->dims_pad % 8 == 0,
+             "head_rotate arguments");
+  RF_REQUIRE(a->ldx % 8 == 0 && a->xs % 8 == 0 && a->ldy % 8 == 0 && a->ys % 8 == 0, "head_rotate: pitches must be multiples of 8");
+  return RF_OK;
+}
+
+extern "C" int rf_head_rotate(const RfHeadRotate* a, int32_t dtype, rf_stream_t stream) {
+  RF_SKIP_IF_REPLAYING();
+  int rc = check_rotate(a);
+  if (rc) return rc;
+  if (a->rows == 0) return RF_OK;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const int64_t items = (int64_t)a->rows * a->heads * (a->dims_pad / 8);
+  RF_DISPATCH3(dtype, RF_CUDA_CHECK(::rf::launch_k(head_rotate_kernel<T>, dim3((unsigned)((items + 255) / 256)), dim3(256), 0, s, 1, *a)));
   ::rf::count_launch();
   return RF_OK;
 }
@@ -587,27 +676,30 @@ extern "C" int rf_head_linear(const RfHeadLinear* a, rf_stream_t stream) {
   if (rc) return rc;
   if (a->rows == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (a->dtype == kF16) return launch_head_linear_mma<__half>(a, nullptr, s);
-  if (a->dtype == kBF16) return launch_head_linear_mma<__nv_bfloat16>(a, nullptr, s);
+  if (a->dtype == kF16) return launch_head_linear_mma<__half>(a, nullptr, nullptr, s);
+  if (a->dtype == kBF16) return launch_head_linear_mma<__nv_bfloat16>(a, nullptr, nullptr, s);
   RF_DISPATCH3(a->dtype, RF_CUDA_CHECK(::rf::launch_k(head_linear_kernel<T>, dim3(ceil_div(a->n, kHlN), a->heads, ceil_div(a->rows, kHlRows)),
                                                       dim3(128), 0, s, 1, *a)));
   ::rf::count_launch();
   return RF_OK;
 }
 
-extern "C" int rf_latent_absorb(const RfHeadLinear* q, const RfLatentInsert* c, rf_stream_t stream) {
+extern "C" int rf_latent_absorb(const RfHeadLinear* q, const RfLatentInsert* c, const RfHeadRotate* t, rf_stream_t stream) {
   RF_SKIP_IF_REPLAYING();
-  int rc = check_insert(c);
-  if (rc) return rc;
   RF_REQUIRE(q != nullptr, "latent_absorb: no queries");
+  int rc = c ? check_insert(c) : RF_OK;
+  if (!rc && t) rc = check_rotate(t);
+  if (rc) return rc;
+  RF_REQUIRE(!c || (c->x && !c->q), "latent_absorb inserts cached rows only");
   if (q->dtype == kF32 || q->rows == 0) {
-    rc = rf_latent_insert(c->x, c->ldx, c->norm_w, c->pool, &c->rows, c->n_rows, c->rank, c->rank_true, c->eps, q->dtype, stream);
+    if (c) rc = rf_latent_insert(c, q->dtype, stream);
+    if (!rc && t) rc = rf_head_rotate(t, q->dtype, stream);
     return rc ? rc : rf_head_linear(q, stream);
   }
   rc = check_head_linear(q);
   if (rc) return rc;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  return q->dtype == kF16 ? launch_head_linear_mma<__half>(q, c, s) : launch_head_linear_mma<__nv_bfloat16>(q, c, s);
+  return q->dtype == kF16 ? launch_head_linear_mma<__half>(q, c, t, s) : launch_head_linear_mma<__nv_bfloat16>(q, c, t, s);
 }
 
 // Room for the largest split of any launch of at most `rows` rows.
@@ -625,6 +717,7 @@ template <typename T>
 static int launch_latent_attn_mma(const RfLatentAttn* a, cudaStream_t s) {
   LatentSplit sp = {};
   sp.splits = la_splits(a->n_rows, a->heads, a->max_kv);
+  const int vrank = a->vrank > 0 ? a->vrank : a->rank;
   const uint64_t slots = (uint64_t)a->n_rows * a->heads * sp.splits;
   if (sp.splits > 1 && (!a->ws || a->ws_bytes < slots * (a->rank + 2) * sizeof(float))) sp.splits = 1;
   sp.o = a->ws;
@@ -644,14 +737,17 @@ static int launch_latent_attn_mma(const RfLatentAttn* a, cudaStream_t s) {
   } while (0)
   if (a->rank <= 64) RF_LN(1);
   else if (a->rank <= 128) RF_LN(2);
+  else if (a->rank <= 192) RF_LN(3);
   else if (a->rank <= 256) RF_LN(4);
-  else RF_LN(8);
+  else if (a->rank <= 320) RF_LN(5);
+  else if (a->rank <= 512) RF_LN(8);
+  else RF_LN(9);
 #undef RF_LN
 #undef RF_LM
   ::rf::count_launch();
   if (sp.splits > 1) {
-    RF_CUDA_CHECK(::rf::launch_k(latent_combine_kernel<T>, dim3(a->n_rows * a->heads), dim3(std::min(128, round_up(a->rank / 4, 32))), 0, s, 1,
-                                 sp, (T*)a->o, a->rank));
+    RF_CUDA_CHECK(::rf::launch_k(latent_combine_kernel<T>, dim3(a->n_rows * a->heads), dim3(std::min(128, round_up(vrank / 4, 32))), 0, s, 1,
+                                 sp, (T*)a->o, vrank));
     ::rf::count_launch();
   }
   return RF_OK;
@@ -679,7 +775,9 @@ extern "C" int rf_latent_attn(const RfLatentAttn* a, rf_stream_t stream) {
   if (rc) return rc;
   if (a->n_rows == 0) return RF_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (a->rank <= 512 && a->dtype == kF16) return launch_latent_attn_mma<__half>(a, s);
-  if (a->rank <= 512 && a->dtype == kBF16) return launch_latent_attn_mma<__nv_bfloat16>(a, s);
+  RF_REQUIRE(a->vrank >= 0 && a->vrank % 16 == 0 && a->vrank <= a->rank, "latent_attn: %d value columns of %d", a->vrank, a->rank);
+  const bool mma = a->rank <= 576 && (a->vrank > 0 ? a->vrank : a->rank) <= 512;
+  if (mma && a->dtype == kF16) return launch_latent_attn_mma<__half>(a, s);
+  if (mma && a->dtype == kBF16) return launch_latent_attn_mma<__nv_bfloat16>(a, s);
   RF_DISPATCH3(a->dtype, return launch_latent_attn<T>(a, s));
 }

@@ -46,14 +46,15 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const RfConvSilu p, int 
   const int q0 = p.rows.q_start ? p.rows.q_start[seq] : seq, n = p.rows.q_len ? p.rows.q_len[seq] : 1;
   const int t0 = blockIdx.y * tile, t1 = min(n, t0 + tile), taps = TAPS > 0 ? TAPS : p.taps, past = taps - 1;
   if (c >= p.channels || t0 >= n) return;
-  const bool fresh = p.rows.pos[q0] == 0;
-  T* state = reinterpret_cast<T*>(p.state) + (size_t)(p.rows.slot ? p.rows.slot[seq] : seq) * past * p.channels + c;
+  T* state = reinterpret_cast<T*>(p.state) + (size_t)(p.rows.slot ? p.rows.slot[seq] : seq) * (p.ring ? taps : past) * p.channels + c;
+  const int pos0 = p.rows.pos[q0];
+  auto carried = [&](int i) -> T* { return state + (size_t)(p.ring ? (pos0 + i) % taps : past + i) * p.channels; };   // input at place i < 0
   const T* x = reinterpret_cast<const T*>(p.x) + (size_t)q0 * p.ldx + c;
   T* y = reinterpret_cast<T*>(p.y) + (size_t)q0 * p.ldy + c;
   // input at place i of this launch's rows; negative places are carried ones
   auto input = [&](int i, float (&f)[8]) {
     if (i >= 0) load8(x + (size_t)i * p.ldx, f);
-    else if (!fresh) load8(state + (size_t)(past + i) * p.channels, f);
+    else if (pos0 + i >= 0) load8(carried(i), f);
     else zero8(f);
   };
   float bias[8];
@@ -74,7 +75,7 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const RfConvSilu p, int 
         a[j] = bias[j];
 #pragma unroll
         for (int k = 0; k < TAPS; ++k) a[j] += w[k][j] * win[k][j];
-        a[j] = silu_t<T>(a[j]);
+        a[j] = p.add ? win[TAPS - 1][j] + a[j] : silu_t<T>(a[j]);
       }
       store8(y + (size_t)t * p.ldy, a);
 #pragma unroll
@@ -94,15 +95,17 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const RfConvSilu p, int 
         for (int j = 0; j < 8; ++j) a[j] += w[j] * v[j];
       }
 #pragma unroll
-      for (int j = 0; j < 8; ++j) a[j] = silu_t<T>(a[j]);
+      for (int j = 0; j < 8; ++j) a[j] = p.add ? v[j] + a[j] : silu_t<T>(a[j]);      // v: the row itself, the last tap's input
       store8(y + (size_t)t * p.ldy, a);
     }
   }
   if (blockIdx.y == 0)
     for (int i = 0; i < past; ++i) {             // ascending: row i comes from a later row of the old state, or from this launch
+      const int at = n - past + i;
+      if (p.ring && at < 0) continue;            // stays where it is
       float v[8];
-      input(n - past + i, v);
-      store8(state + (size_t)i * p.channels, v);
+      input(at, v);
+      store8(p.ring ? state + (size_t)((pos0 + at) % taps) * p.channels : state + (size_t)i * p.channels, v);
     }
 }
 

@@ -134,7 +134,7 @@ struct PlanSmem { int32_t cnt[256], rows_at[257], tiles_at[257]; };
 
 // Exclusive sums of the experts' counts (sm.cnt) and the tile list; all threads of the CTA.
 __device__ __forceinline__ void plan_tiles(const RfMoeRouter& p, PlanSmem& sm) {
-  const int tid = threadIdx.x, E = p.experts, R = p.tile_rows;
+  const int tid = threadIdx.x, E = p.experts - p.identity, R = p.tile_rows;
   if (tid < 32) {
     int rows = 0, tiles = 0;
     for (int e0 = 0; e0 < E; e0 += 32) {
@@ -189,7 +189,7 @@ __global__ void __launch_bounds__(kRtTokens * 32) moe_choose_kernel(const RfMoeR
   __shared__ PlanSmem sm;
   __shared__ int32_t base[256];
   __shared__ int last;
-  const int E = p.experts, columns = E + p.shared_gate, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int E = p.experts, real = E - p.identity, columns = E + p.shared_gate, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const bool alone = gridDim.x == 1;
   const int per_cta = alone ? kRtOneCta : kRtTokens, first = blockIdx.x * per_cta;
   const int here = min(per_cta, p.rows - first);
@@ -197,7 +197,7 @@ __global__ void __launch_bounds__(kRtTokens * 32) moe_choose_kernel(const RfMoeR
   int32_t* s_id = reinterpret_cast<int32_t*>(ch_sm + kRtTokens * E);
   int32_t* s_rank = s_id + per_cta * p.k;
   float* s_w = reinterpret_cast<float*>(s_rank + per_cta * p.k);
-  for (int e = tid; e < E; e += blockDim.x) sm.cnt[e] = 0;
+  for (int e = tid; e < real; e += blockDim.x) sm.cnt[e] = 0;
   __syncthreads();
   for (int t = warp; t < here; t += kRtTokens) {
     float sc[S];
@@ -216,6 +216,12 @@ __global__ void __launch_bounds__(kRtTokens * 32) moe_choose_kernel(const RfMoeR
     int id;
     float w;
     route_token<S>(p, lane, sc, keys, &id, &w);
+    if (p.identity > 0) {
+      const bool self = lane < p.k && id >= real;
+      const float sum = warp_sum(self ? w : 0.f);
+      if (lane == 0) p.self_w[first + t] = sum;
+      if (self) id = -1;
+    }
     if (lane < p.k) {
       const int i = t * p.k + lane;
       s_id[i] = id;
@@ -225,7 +231,7 @@ __global__ void __launch_bounds__(kRtTokens * 32) moe_choose_kernel(const RfMoeR
   }
   __syncthreads();
   if (!alone) {
-    for (int e = tid; e < E; e += blockDim.x) base[e] = sm.cnt[e] ? atomicAdd(p.counters + e, sm.cnt[e]) : 0;
+    for (int e = tid; e < real; e += blockDim.x) base[e] = sm.cnt[e] ? atomicAdd(p.counters + e, sm.cnt[e]) : 0;
     __syncthreads();
   }
   for (int i = tid; i < here * p.k; i += blockDim.x) {
@@ -244,13 +250,13 @@ __global__ void __launch_bounds__(kRtTokens * 32) moe_choose_kernel(const RfMoeR
   __threadfence();
   __syncthreads();
   if (tid == 0) {
-    last = atomicAdd(p.counters + E, 1) == (int)gridDim.x - 1;
-    if (last) p.counters[E] = 0;
+    last = atomicAdd(p.counters + real, 1) == (int)gridDim.x - 1;
+    if (last) p.counters[real] = 0;
   }
   __syncthreads();
   if (!last) return;
   __threadfence();
-  for (int e = tid; e < E; e += blockDim.x) {             // the counters are left at zero for the next launch
+  for (int e = tid; e < real; e += blockDim.x) {          // the counters are left at zero for the next launch
     sm.cnt[e] = __ldcg(p.counters + e);
     p.counters[e] = 0;
   }
@@ -483,6 +489,8 @@ __global__ void __launch_bounds__(256, MT == 1 ? 2 : 1) moe_small_kernel(const R
 #pragma unroll
         for (int j = 0; j < 8; ++j) v[0][j] = silu_f(v[0][j]) * v[D - 1][j];
       }
+    } else if (p.act != kActNone && !act_is_dual(p.act)) {
+      apply_act_n<8>(p.act, v[0], v[0], v[0], ActArgs{p.act_limit, p.act_alpha});
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j) v[0][j] *= ws;
@@ -541,6 +549,8 @@ __global__ void __launch_bounds__(256) moe_f32_kernel(const RfMoeExperts p) {
       if constexpr (DUAL) {
         const float u = acc[D - 1][i][j], limit = sh ? p.shared_limit : p.act_limit, gc = fminf(g, limit);
         v = p.act == kActClippedGlu ? gc / (1.f + expf(-p.act_alpha * gc)) * (fminf(fmaxf(u, -limit), limit) + 1.f) : g / (1.f + expf(-g)) * u;
+      } else if (p.act == kActGeluErf) {
+        v = gelu_erf_f(g);
       }
       reinterpret_cast<float*>(p.out)[(size_t)(row0 + r) * p.ldo + n] = v * (p.slot_w ? p.slot_w[row0 + r] : 1.f);
     }
@@ -602,6 +612,7 @@ static int check_router(const RfMoeRouter* a) {
   RF_REQUIRE(a->dtype >= 0 && a->dtype <= 2 && (int64_t)a->rows * (a->k + 1) < (1ll << 30), "moe_router: dtype %d", a->dtype);
   RF_REQUIRE(a->score_fn >= RF_MOE_SIGMOID && a->score_fn <= RF_MOE_CHOSEN && (a->shared_gate == 0 || (a->shared_gate == 1 && a->has_shared)),
              "moe_router: score function %d, gate of the shared expert %d", a->score_fn, a->shared_gate);
+  RF_REQUIRE(a->identity >= 0 && a->identity < a->experts && (a->identity == 0 || a->self_w), "moe_router: %d identity experts of %d", a->identity, a->experts);
   return RF_OK;
 }
 
@@ -655,7 +666,7 @@ extern "C" int rf_moe_experts(const RfMoeExperts* a, rf_stream_t stream) {
   RF_REQUIRE(a->n > 0 && a->k > 0 && a->n % 8 == 0 && a->k % 8 == 0 && a->ldx % 8 == 0 && a->ldo % 8 == 0, "moe_experts: %d x %d", a->n, a->k);
   RF_REQUIRE((a->shared_n > 0) == (a->w_shared != nullptr) && a->shared_n % 8 == 0 && a->shared_k % 8 == 0, "moe_experts: shared expert");
   RF_REQUIRE(a->dtype >= 0 && a->dtype <= 2, "moe_experts: dtype %d", a->dtype);
-  RF_REQUIRE(a->act == 0 || a->act == kActSiluMul || (a->act == kActClippedGlu && a->act_limit > 0.f && (!a->w_shared || a->shared_limit > 0.f)),
+  RF_REQUIRE(a->act == 0 || a->act == kActSiluMul || (a->act == kActGeluErf && !a->dual) || (a->act == kActClippedGlu && a->act_limit > 0.f && (!a->w_shared || a->shared_limit > 0.f)),
              "moe_experts: activation %d", a->act);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (a->dtype == kF32) {

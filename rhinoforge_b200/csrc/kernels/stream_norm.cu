@@ -35,6 +35,11 @@ template <typename T>
 __device__ __forceinline__ float4 pending4(const RfStreamNorm& p, const T* y, int src, int col) {
   if (p.y_picks <= 0) return load4(y + (size_t)src * p.H + col);
   float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (p.y_self_w) {
+    const float w = p.y_self_w[src];
+    const float4 v = load4(reinterpret_cast<const T*>(p.y_self) + (size_t)src * p.H + col);
+    s = make_float4(w * v.x, w * v.y, w * v.z, w * v.w);
+  }
   const int32_t* slots = p.y_slots + (size_t)src * p.y_picks;
 #pragma unroll 4
   for (int j = 0; j < p.y_picks; ++j) {
@@ -278,9 +283,40 @@ __global__ void __launch_bounds__(VPT == 4 ? 512 : 1024) stream_norm_reg_kernel(
   }
 }
 
+// Input convolution of eight columns of a decode row: h <- h + conv(h), carried rows read and moved up by one.
+template <typename T>
+__device__ __forceinline__ void input_conv8(const RfStreamNorm& p, int r, int col, float (&h)[8]) {
+  const int past = p.conv_taps - 1;
+  T* state = reinterpret_cast<T*>(p.conv_state) + (size_t)(p.rows.slot ? p.rows.slot[r] : r) * past * p.H + col;
+  const bool fresh = p.rows.pos[r] == 0;
+  float w[8], f[8], s[8];
+  load8(p.conv_w + (size_t)past * p.H + col, w);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    h[j] = Num<T>::to_f(Num<T>::from_f(h[j]));     // rows enter the convolution as they are carried
+    s[j] = w[j] * h[j];
+  }
+#pragma unroll 4
+  for (int k = 0; k < past; ++k) {
+    load8(p.conv_w + (size_t)k * p.H + col, w);
+    if (fresh) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] = 0.f;
+    } else {
+      load8(state + (size_t)k * p.H, f);
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s[j] += w[j] * f[j];
+    if (k > 0) store8(state + (size_t)(k - 1) * p.H, f);
+  }
+  if (past > 0) store8(state + (size_t)(past - 1) * p.H, h);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) h[j] += s[j];
+}
+
 // The stream step of 16-bit activations without a token shift: one CTA per row, a thread holds NC groups of eight columns, so that
 // every operand moves in 16-byte pieces; of several picked rows four are in flight at a time.
-template <typename T, int NC>
+template <typename T, int NC, bool CONV>
 __global__ void __launch_bounds__(512) stream_out_kernel(const RfStreamNorm p) {
   pdl_launch_dependents();
   __shared__ float red[2][16];
@@ -342,6 +378,17 @@ __global__ void __launch_bounds__(512) stream_out_kernel(const RfStreamNorm p) {
         }
       }
   }
+  if (p.y_self_w) {
+    const float sw = p.y_self_w[src];
+#pragma unroll
+    for (int k = 0; k < NC; ++k) {
+      if (col(k) >= H) continue;
+      float f[8];
+      load8(reinterpret_cast<const T*>(p.y_self) + (size_t)src * H + col(k), f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a[k][j] += sw * f[j];
+    }
+  }
   auto block_sum = [&](float s, int flip) -> float {
     s = warp_sum(s);
     if (lane == 0) red[flip][warp] = s;
@@ -380,6 +427,7 @@ __global__ void __launch_bounds__(512) stream_out_kernel(const RfStreamNorm p) {
     if (p.y_norm_w) load8(p.norm_w + col(k), w[k]);
 #pragma unroll
     for (int j = 0; j < 8; ++j) n8[j] = w[k][j] * v[k][j] * xr;
+    if constexpr (CONV) input_conv8<T>(p, r, col(k), n8);
     store8(reinterpret_cast<T*>(p.out) + (size_t)r * H + col(k), n8);
   }
 }
@@ -491,6 +539,9 @@ extern "C" int rf_stream_norm(const RfStreamNorm* args, rf_stream_t stream) {
                            "stream_norm: the token shift needs a norm, its state, positions, all rows and separate streams");
   if (a->table2) RF_REQUIRE(!a->x && !a->shift && !a->row_idx && a->rows.pos && a->last_token && a->buckets > 0 && a->mul_prev >= 0 && a->mul_cur >= 0,
                             "stream_norm: token pairs need the embedding rows of all rows, positions, the carried tokens and no token shift");
+  RF_REQUIRE(!a->y_self_w || (a->y_self && a->y_picks > 0), "stream_norm: the identity part belongs to picked rows");
+  if (a->conv_w) RF_REQUIRE(a->conv_taps >= 1 && (a->conv_taps == 1 || a->conv_state) && a->norm_w && a->rows.pos && !a->rows.q_start && !a->shift &&
+                                !a->row_idx && a->dtype != kF32 && a->H / 8 <= 1024, "stream_norm: the input convolution takes decode rows in 16 bits");
   if (a->n_rows == 0) return RF_OK;
   // halo of one row per CTA with the shift: walk several rows per CTA once that still fills the GPU
   const int rpc = (a->shift && a->rows.q_start) ? std::max(1, std::min(8, a->n_rows / (2 * sm_count()))) : 1;
@@ -500,10 +551,12 @@ extern "C" int rf_stream_norm(const RfStreamNorm* args, rf_stream_t stream) {
     // decode rows: one group of columns per thread; many rows: two, so that several rows share an SM
     const int nc = groups > 512 || (groups > 256 && a->n_rows > 4 * sm_count()) ? 2 : 1;
     const dim3 block(std::max(32, round_up(ceil_div(groups, nc), 32)));
-#define RF_SO(T, NC) RF_CUDA_CHECK(::rf::launch_k(stream_out_kernel<T, NC>, dim3(a->n_rows), block, 0, s, 1, *a))
-#define RF_SO_T(T) if (nc == 1) { RF_SO(T, 1); } else { RF_SO(T, 2); }
+#define RF_SO(T, NC, CV) RF_CUDA_CHECK(::rf::launch_k(stream_out_kernel<T, NC, CV>, dim3(a->n_rows), block, 0, s, 1, *a))
+#define RF_SO_C(T, NC) if (a->conv_w) { RF_SO(T, NC, true); } else { RF_SO(T, NC, false); }
+#define RF_SO_T(T) if (nc == 1) { RF_SO_C(T, 1) } else { RF_SO_C(T, 2) }
     if (a->dtype == kF16) { RF_SO_T(__half) } else { RF_SO_T(__nv_bfloat16) }
 #undef RF_SO_T
+#undef RF_SO_C
 #undef RF_SO
     ::rf::count_launch();
     return RF_OK;

@@ -31,14 +31,14 @@ struct MixedStack {
   uint8_t* base = nullptr;
   uint64_t off_x[2] = {}, off_h = 0, off_cast = 0, off_wide = 0, off_mix = 0, off_y = 0, off_side = 0, off_qlat = 0, off_olat = 0,
            off_ctx = 0, off_kv = 0, off_kvmeta = 0, off_attn_ws = 0, off_head = 0, off_argmax = 0, off_sk_ws = 0, off_sk_flags = 0,
-           off_status = 0, off_vfirst = 0, off_q = 0, off_conv = 0, off_bc = 0, off_dt = 0, off_moe = 0, off_xg = 0, off_hg = 0, off_yg = 0, off_router = 0, total = 0;
+           off_status = 0, off_vfirst = 0, off_q = 0, off_conv = 0, off_bc = 0, off_dt = 0, off_moe = 0, off_xg = 0, off_hg = 0, off_yg = 0, off_router = 0, off_self = 0, total = 0;
   uint64_t attn_ws_bytes = 0, argmax_bytes = 0, sk_ws_bytes = 0, rows_ws_bytes = 0;
   int moe_tiles = 0;      // tile-list entries of any mixture-of-experts layer
   int lat_rows = 0;       // rows one latent-space attention launch takes
   int ctx_rows = 0;       // rows of expanded keys / values one group of portions takes
   int cur = 0;            // which stream buffer holds the last forward's rows
   // the sublayer output that is still to be added behind the last layer
-  struct Pending { const void* y = nullptr; const float* norm = nullptr; const int32_t* slots = nullptr; int picks = 0; } tail;
+  struct Pending { const void* y = nullptr; const float* norm = nullptr; const int32_t* slots = nullptr; int picks = 0; const void* self = nullptr; const float* self_w = nullptr; } tail;
   const int32_t* full_len = nullptr;      // device: cached tokens, new ones included, of every prefill-sized sequence
   int max_full = 0, max_long_q = 0;
   bool planned = false;
@@ -49,6 +49,7 @@ struct MixedStack {
   size_t esz() const { return cfg.dtype == kF32 ? 4 : 2; }
   bool fp32() const { return cfg.dtype == kF32; }
   template <typename P = void> P* at(uint64_t off) const { return reinterpret_cast<P*>(base + off); }
+  static int delta_channels(const RfMixedLayer& l) { return 2 * l.kv_heads * l.dim + l.heads * l.vdim; }
   static int moe_ld(const RfMixedLayer& l) { return std::max(l.bank_inter, l.shared_inter); }
   int32_t* status() const { return base ? at<int32_t>(off_status) : nullptr; }
 
@@ -66,19 +67,21 @@ struct MixedStack {
         if (l.conv_taps > 0) qout = std::max<uint64_t>(qout, (uint64_t)l.heads * l.dim);
         if (l.tensor_core) rows_ws_bytes = std::max<uint64_t>(rows_ws_bytes, rf_attn_decode_scratch_bound(l.heads, l.kv_heads, l.dim));
       }
+      if (l.mixer == RF_MIXER_DELTA) inner = std::max<uint64_t>(inner, delta_channels(l));
       if (l.mixer == RF_MIXER_MAMBA1) {
         inner = std::max<uint64_t>(inner, l.inner);
         bc = std::max<uint64_t>(bc, l.dt_rank + 2 * l.states);
       }
       if (l.experts > 0) {
         picks = std::max<uint64_t>(picks, l.top + 1);
-        experts = std::max<uint64_t>(experts, l.experts + l.shared_gate);
+        experts = std::max<uint64_t>(experts, l.experts + l.identity + l.shared_gate);
         hg = std::max<uint64_t>(hg, moe_ld(l));
         moe_tiles = std::max(moe_tiles, l.experts + (int)(T * (l.top + 1) / 16) + 2);
       }
       if (l.mixer != RF_MIXER_LATENT_ATTENTION) continue;
-      lat = std::max<uint64_t>(lat, (uint64_t)l.heads * l.rank);
-      rank = std::max<uint64_t>(rank, l.rank);
+      lat = std::max<uint64_t>(lat, (uint64_t)l.heads * (l.rank + l.rot_pad));
+      rank = std::max<uint64_t>(rank, l.rank + l.rot_pad);
+      if (l.q_rank > 0) qout = std::max<uint64_t>(qout, (uint64_t)l.heads * l.dim);
       heads = std::max<uint64_t>(heads, l.heads);
       if (l.expand_hd > 0) {
         kvw = std::max<uint64_t>(kvw, 2ull * l.heads * l.expand_hd);
@@ -118,6 +121,7 @@ struct MixedStack {
     // counters, start | tile list | ids, weights, rank | slot_of, token_of_slot, slot_w (one column more)
     off_moe = o; o += al(picks ? (6 * T * picks + 2 * kMoeExperts + 4 + 4ull * moe_tiles) * 4 : 0);
     off_router = o; o += al(picks ? rf_moe_router_scratch_bytes(cfg.max_tokens, (int)experts) : 0);
+    off_self = o; o += al(picks ? T * sizeof(float) : 0);
     off_xg = o; o += al(fp32() || !picks ? 0 : T * (picks - 1) * H * e);
     off_hg = o; o += al(T * picks * hg * e);
     off_yg = o; o += al(T * picks * H * e);
@@ -195,26 +199,46 @@ static RfRows sub_rows(const RfRows& r, int seq0, int num_seqs) {
 
 static int latent_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f, const void* h, void* mix, cudaStream_t st) {
   const RfMixedConfig& c = s.cfg;
-  const int T = f.tokens, H = c.hidden, QD = w.heads * w.dim, VD = w.heads * w.vdim;
+  const int T = f.tokens, H = c.hidden, QD = w.heads * w.dim, VD = w.heads * w.vdim, R = w.rank + w.rot_pad;
   const size_t e = s.esz();
   uint8_t* wide = s.at<uint8_t>(s.off_wide);
   int rc = linear(s, h, H, w.w_in, wide, w.in_dim, T, w.in_dim, H, kActNone, st);
   if (rc) return rc;
-  RfLatentInsert ins = {wide + (size_t)QD * e, w.in_dim, w.latent_norm, w.st.latent_pool, f.rows, T, w.rank, w.rank_true, c.eps};
+  RfLatentInsert ins = {};
+  ins.norm_w = w.latent_norm; ins.pool = w.st.latent_pool; ins.rows = f.rows; ins.n_rows = T; ins.rank = w.rank; ins.rank_true = w.rank_true; ins.eps = c.eps;
+  ins.rot = w.rot; ins.rot_pad = w.rot_pad; ins.cos = w.cos; ins.sin = w.sin;
+  if (!w.shares) { ins.x = wide + (size_t)(w.q_rank > 0 ? w.q_rank : QD) * e; ins.ldx = w.in_dim; }
+  uint8_t* queries = wide;
+  int64_t ldq = w.in_dim;
+  bool inserted = false;
+  if (w.q_rank > 0) {
+    ins.q = wide; ins.ldq = w.in_dim; ins.q_norm = w.q_latent_norm; ins.q_rank = w.q_rank; ins.q_rank_true = w.q_rank_true;
+    rc = rf_latent_insert(&ins, c.dtype, st);
+    if (rc) return rc;
+    inserted = true;
+    queries = s.at<uint8_t>(s.off_q);
+    ldq = QD;
+    rc = linear(s, wide, w.in_dim, w.w_uq, queries, QD, T, QD, w.q_rank, kActNone, st);
+    if (rc) return rc;
+  }
+  RfHeadRotate turn = {};               // the rotated part of the queries; rows are filled in below
+  turn.ldx = ldq; turn.xs = w.dim; turn.cos = w.cos; turn.sin = w.sin; turn.heads = w.heads; turn.dims = w.rot;
   // ---- decode rows and short portions (and everything without an expanded form): in the latent space
   const bool expand = w.expand_hd > 0 && f.short_seqs < f.rows.num_seqs;
   const int lat_total = expand ? f.short_rows : T;
-  if (lat_total == 0) {
-    rc = rf_latent_insert(ins.x, ins.ldx, ins.norm_w, ins.pool, &ins.rows, T, w.rank, w.rank_true, c.eps, c.dtype, st);
+  if (lat_total == 0 && !inserted) {
+    rc = rf_latent_insert(&ins, c.dtype, st);
     if (rc) return rc;
   }
   for (int r0 = 0; r0 < lat_total; r0 += s.lat_rows) {
     const int n = std::min(s.lat_rows, lat_total - r0);
     RfHeadLinear q = {};
-    q.x = wide + (size_t)r0 * w.in_dim * e; q.ldx = w.in_dim; q.xs = w.dim;
-    q.y = s.at(s.off_qlat); q.ldy = (int64_t)w.heads * w.rank; q.ys = w.rank;
-    q.w = w.w_absorb; q.rows = n; q.heads = w.heads; q.n = w.rank; q.k = w.dim; q.dtype = c.dtype;
-    rc = r0 == 0 ? rf_latent_absorb(&q, &ins, st) : rf_head_linear(&q, st);      // every row is cached before the first attends
+    q.x = queries + (size_t)r0 * ldq * e; q.ldx = ldq; q.xs = w.dim;
+    q.y = s.at(s.off_qlat); q.ldy = (int64_t)w.heads * R; q.ys = R;
+    q.w = w.w_absorb; q.rows = n; q.heads = w.heads; q.n = w.rank; q.k = w.plain; q.dtype = c.dtype;
+    turn.x = (const uint8_t*)q.x + (size_t)w.plain * e; turn.y = (uint8_t*)q.y + (size_t)w.rank * e; turn.ldy = q.ldy; turn.ys = R;
+    turn.pos = f.rows.pos + r0; turn.rows = n; turn.dims_pad = w.rot_pad;
+    rc = rf_latent_absorb(&q, r0 == 0 && !inserted ? &ins : nullptr, w.rot > 0 ? &turn : nullptr, st);      // every row is cached before the first attends
     if (rc) return rc;
     RfLatentAttn a = {};
     a.q = s.at(s.off_qlat); a.o = s.at(s.off_olat); a.pool = w.st.latent_pool;
@@ -222,7 +246,7 @@ static int latent_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedF
     if (a.rows.seq_of_row) a.rows.seq_of_row += r0;
     else if (a.rows.slot) a.rows.slot += r0;
     else RF_REQUIRE(r0 == 0, "mixed stack: %d decode rows need slots", lat_total);
-    a.n_rows = n; a.heads = w.heads; a.rank = w.rank; a.window = w.window; a.scale = w.scale; a.dtype = c.dtype;
+    a.n_rows = n; a.heads = w.heads; a.rank = R; a.vrank = w.rank; a.window = w.window; a.scale = w.scale; a.dtype = c.dtype;
     a.max_kv = w.window > 0 ? std::min(w.window, f.max_kv) : f.max_kv;
     a.ws = s.at<float>(s.off_attn_ws); a.ws_bytes = s.attn_ws_bytes;
     rc = rf_latent_attn(&a, st);
@@ -235,6 +259,12 @@ static int latent_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedF
     if (rc) return rc;
   }
   if (!expand) return RF_OK;
+  if (w.rot > 0) {                      // their queries turn in place
+    turn.x = queries + ((size_t)lat_total * ldq + w.plain) * e; turn.y = (void*)turn.x; turn.ldy = ldq; turn.ys = w.dim;
+    turn.pos = f.rows.pos + lat_total; turn.rows = T - lat_total; turn.dims_pad = (w.rot + 7) / 8 * 8;
+    rc = rf_head_rotate(&turn, c.dtype, st);
+    if (rc) return rc;
+  }
   // ---- prefill-sized portions: keys and values of the visible rows, group by group so that the buffers stay bounded
   const WindowPlan* plan = nullptr;
   for (const WindowPlan& p : s.windows)
@@ -247,12 +277,12 @@ static int latent_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedF
     void* ctx = s.at(s.off_ctx);
     uint8_t* kv = s.at<uint8_t>(s.off_kv);
     const int KD = w.heads * w.expand_hd, KV = 2 * KD;
-    rc = rf_latent_gather(w.st.latent_pool, ctx, &g, kv_start, kv_len, w.rank, grp.max_len, c.dtype, st);
+    rc = rf_latent_gather(w.st.latent_pool, ctx, &g, kv_start, kv_len, R, grp.max_len, c.dtype, st);
     if (rc) return rc;
-    rc = linear(s, ctx, w.rank, w.w_expand, kv, KV, grp.total, KV, w.rank, kActNone, st);
+    rc = linear(s, ctx, R, w.w_expand, kv, KV, grp.total, KV, R, kActNone, st);
     if (rc) return rc;
     RfAttn a = {};
-    a.q = wide; a.ldq = w.in_dim; a.out = mix; a.ldo = VD; a.q_rows_total = T;     // q_start holds rows of the whole batch
+    a.q = queries; a.ldq = ldq; a.out = mix; a.ldo = VD; a.q_rows_total = T;     // q_start holds rows of the whole batch
     a.k = kv; a.v = kv + (size_t)KD * e; a.ldk = KV; a.ldv = KV; a.kv_rows_total = grp.total;
     a.num_seqs = grp.seqs; a.Hq = w.heads; a.Hkv = w.heads; a.hd = w.expand_hd;
     a.q_start = g.q_start; a.q_len = g.q_len; a.kv_start = kv_start; a.kv_len = kv_len;
@@ -346,6 +376,7 @@ static int grouped_attention(MixedStack& s, const RfMixedLayer& w, const RfMixed
   q.v_first = s.at(s.off_vfirst); q.k_pool = w.st.k_pool; q.v_pool = w.st.v_pool; q.rows = f.rows;
   q.n_rows = T; q.heads = w.heads; q.kv_heads = w.kv_heads; q.hd = hd; q.dim = w.dim_true; q.vdim = w.vdim_true;
   q.rot_dims = w.rot_dims; q.v_role = w.v_role; q.v_lambda = w.v_lambda; q.eps = c.eps; q.dtype = c.dtype; q.norm_all = w.norm_all;
+  q.growth = w.growth; q.growth_every = w.growth_every;
   uint8_t* queries = wide;
   int64_t ldq = w.in_dim;
   if (w.conv_taps > 0) {
@@ -360,7 +391,7 @@ static int grouped_attention(MixedStack& s, const RfMixedLayer& w, const RfMixed
   a.k_pool = w.st.k_pool; a.v_pool = w.st.v_pool; a.pool_pages = w.st.pool_pages;
   a.page_table = f.rows.page_table; a.pt_stride = f.rows.pt_stride;
   a.Hq = w.heads; a.Hkv = w.kv_heads; a.hd = hd; a.scale = w.scale; a.chunk = w.chunk; a.sink = w.sink;
-  a.window = w.window; a.keep_first = w.keep_first; a.slopes = w.slopes;
+  a.window = w.window; a.keep_first = w.keep_first; a.slopes = w.slopes; a.rates = w.rates;
   if (w.gated) { a.gate = wide + (size_t)(QD + 2 * KD) * e; a.ld_gate = w.in_dim; a.gate_by_head = w.gate_by_head; }
   a.status = s.status(); a.dtype = c.dtype;
   // ---- decoded rows and short portions, by row (without a tensor-core form: every row)
@@ -423,6 +454,31 @@ static int mamba1(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f,
   return rc;
 }
 
+static int delta(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f, const void* h, void* mix, cudaStream_t st) {
+  const RfMixedConfig& c = s.cfg;
+  const int T = f.tokens, H = c.hidden, CH = MixedStack::delta_channels(w), VD = w.heads * w.vdim;
+  const size_t e = s.esz();
+  uint8_t* wide = s.at<uint8_t>(s.off_wide);
+  int rc = linear(s, h, H, w.w_in, wide, w.in_dim, T, w.in_dim, H, kActNone, st);
+  if (rc) return rc;
+  RfDelta a = {};
+  a.x = wide; a.ldx = w.in_dim; a.gate = wide + (size_t)CH * e; a.ldg = w.in_dim;
+  a.b = wide + (size_t)(CH + VD) * e; a.a = wide + (size_t)(CH + VD + (w.heads + 7) / 8 * 8) * e; a.ld_ba = w.in_dim;
+  a.rate = w.rate; a.dt_bias = w.dt_bias; a.norm_w = w.head_norm; a.state = w.st.rec_state; a.out = mix; a.ldo = VD; a.rows = f.rows;
+  a.heads = w.heads; a.kv_heads = w.kv_heads; a.dim = w.dim; a.dim_true = w.dim_true; a.vdim = w.vdim; a.vdim_true = w.vdim_true; a.eps = c.eps; a.dtype = c.dtype;
+  if (f.decode) {
+    a.conv_w = w.conv_w; a.conv_state = w.st.conv_state; a.taps = w.taps;
+    return rf_delta_recurrent(&a, st);
+  }
+  RfConvSilu cv = {};
+  cv.x = wide; cv.ldx = w.in_dim; cv.y = s.at(s.off_conv); cv.ldy = CH; cv.w = w.conv_w; cv.state = w.st.conv_state; cv.rows = f.rows;
+  cv.channels = CH; cv.taps = w.taps; cv.dtype = c.dtype; cv.max_q_len = longest_portion(f); cv.ring = 1;
+  rc = rf_conv_silu(&cv, st);
+  if (rc) return rc;
+  a.x = cv.y; a.ldx = CH;
+  return rf_delta_recurrent(&a, st);
+}
+
 // The experts' results stay where they are, one row per pick; the next stream step adds them up (see RfStreamNorm.y_slots).
 static int experts(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f, const void* h, MixedStack::Pending* out, cudaStream_t st) {
   const RfMixedConfig& c = s.cfg;
@@ -432,7 +488,7 @@ static int experts(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f
   int32_t* m = s.at<int32_t>(s.off_moe);
   RfMoeRouter r = {};
   r.logits = s.at<float>(s.off_router);
-  r.x = h; r.ldx = H; r.w = w.router; r.correction = w.correction;
+  r.x = h; r.ldx = H; r.w = w.router; r.correction = w.correction; r.identity = w.identity; r.self_w = s.at<float>(s.off_self);
   r.counters = m; m += MixedStack::kMoeExperts;      // the same place whatever a layer's expert count: they are zero between launches
   r.start = m; m += MixedStack::kMoeExperts;
   r.tiles = m; m += 4 + 4 * s.moe_tiles;
@@ -442,13 +498,15 @@ static int experts(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f
   r.slot_of = m; m += T * cols;
   r.token_of_slot = m; m += T * cols;
   r.slot_w = (float*)m;
-  r.rows = T; r.experts = E; r.width = H; r.k = k; r.groups = w.groups; r.keep = w.keep; r.score_fn = w.score_fn;
+  r.rows = T; r.experts = E + w.identity; r.width = H; r.k = k; r.groups = w.groups; r.keep = w.keep; r.score_fn = w.score_fn;
   r.norm_topk = w.norm_topk; r.scale = w.route_scale; r.slot_ld = cols; r.has_shared = has_shared; r.dtype = c.dtype;
   r.shared_gate = w.shared_gate;
-  const int act = w.act == RF_MIXED_ACT_CLIPPED_GLU ? kActClippedGlu : kActSiluMul;
+  const int act = w.act == RF_MIXED_ACT_CLIPPED_GLU ? kActClippedGlu : w.act == RF_MIXED_ACT_GELU ? kActGeluErf : kActSiluMul;
+  const int dual = act_is_dual(act);
   uint8_t* hg = s.at<uint8_t>(s.off_hg);
   uint8_t* yg = s.at<uint8_t>(s.off_yg);
   out->y = yg; out->slots = r.slot_of; out->picks = cols;
+  if (w.identity > 0) { out->self = h; out->self_w = r.self_w; }
   if (s.fp32() || T <= MixedStack::kMoeSmallRows) {
     r.tile_rows = s.fp32() ? 64 : (pairs <= 16 * E ? 16 : 32);
     r.shared_tiles = has_shared; r.scatter = 1;
@@ -458,13 +516,13 @@ static int experts(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f
     x.tiles = r.tiles; x.experts = E; x.tile_rows = r.tile_rows; x.dtype = c.dtype;
     x.max_tiles = std::min(E, pairs) + pairs / r.tile_rows + (has_shared ? ceil_div(T, r.tile_rows) : 0);
     x.x = h; x.ldx = H; x.token_of_slot = r.token_of_slot; x.w = w.w_up; x.w_shared = w.shared_up; x.out = hg; x.ldo = ldh;
-    x.n = w.inter; x.k = H; x.dual = 1; x.act = act; x.act_limit = w.act_limit; x.act_alpha = w.act_alpha; x.shared_limit = w.shared_limit;
+    x.n = w.inter; x.k = H; x.dual = dual; x.act = act; x.act_limit = w.act_limit; x.act_alpha = w.act_alpha; x.shared_limit = w.shared_limit;
     x.bank_section_row_tiles = E * bank_rt; x.bank_kb_total = kbH; x.rt_per_expert = bank_rt;
     if (has_shared) { x.shared_n = w.shared_inter; x.shared_k = H; x.shared_section_row_tiles = ceil_div(w.shared_inter, 128); x.shared_kb_total = kbH; }
     rc = rf_moe_experts(&x, st);
     if (rc) return rc;
     x.x = hg; x.ldx = ldh; x.token_of_slot = nullptr; x.slot_w = r.slot_w; x.w = w.w_down; x.w_shared = w.shared_down; x.out = yg; x.ldo = H;
-    x.n = H; x.k = w.inter; x.dual = 0;
+    x.n = H; x.k = w.inter; x.dual = 0; x.act = kActNone;
     x.bank_section_row_tiles = 0; x.bank_kb_total = E * w.bank_inter / 64; x.rt_per_expert = 0; x.kb_per_expert = w.bank_inter / 64;
     if (has_shared) { x.shared_n = H; x.shared_k = w.shared_inter; x.shared_section_row_tiles = 0; x.shared_kb_total = ceil_div(w.shared_inter, 64); }
     return rf_moe_experts(&x, st);
@@ -477,7 +535,7 @@ static int experts(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f
   if (rc) return rc;
   RfMoeGroupedGemm g = {};
   g.x = xg; g.ldx = H; g.w = w.w_up; g.out = hg; g.ldo = ldh; g.tiles = r.tiles + 3; g.max_rows = pairs; g.N = w.bank_inter; g.K = H;
-  g.dual = 1; g.act = act; g.act_limit = w.act_limit; g.act_alpha = w.act_alpha; g.bank_section_row_tiles = E * bank_rt; g.bank_kb_total = kbH; g.rt_per_expert = bank_rt;
+  g.dual = dual; g.act = act; g.act_limit = w.act_limit; g.act_alpha = w.act_alpha; g.bank_section_row_tiles = E * bank_rt; g.bank_kb_total = kbH; g.rt_per_expert = bank_rt;
   g.dtype = c.dtype; g.status = s.status();
   rc = rf_moe_grouped_gemm(&g, st);
   if (rc) return rc;
@@ -514,7 +572,7 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
   int cur = -1;                       // stream buffer in use; -1: still the embedding
   MixedStack::Pending pend;           // sublayer output that the next stream_norm adds
   // stream step: adds the pending output, optionally writes the 16-bit copy and / or the normalised rows
-  auto step = [&](const float* norm_w, const float* shift, float* shift_state, bool want_cast) -> int {
+  auto step = [&](const float* norm_w, const float* shift, float* shift_state, bool want_cast, const float* conv_w = nullptr, void* conv_state = nullptr) -> int {
     RfStreamNorm a = {};
     a.x = cur < 0 ? nullptr : s.at<float>(s.off_x[cur]);
     a.table = c.embed; a.ids = f.ids; a.embed_scale = c.embed_scale; a.y_mult = c.residual_mult;
@@ -522,7 +580,7 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
       a.table2 = c.pair_table; a.last_token = s.layers[0].st.last_token; a.buckets = c.pair_buckets;
       a.mul_prev = c.pair_mul_prev; a.mul_cur = c.pair_mul_cur;
     }
-    a.y = pend.y; a.y_norm_w = pend.norm; a.y_slots = pend.slots; a.y_picks = pend.picks;
+    a.y = pend.y; a.y_norm_w = pend.norm; a.y_slots = pend.slots; a.y_picks = pend.picks; a.y_self = pend.self; a.y_self_w = pend.self_w;
     const int nxt = cur < 0 ? 0 : cur ^ 1;
     a.x_out = s.at<float>(s.off_x[nxt]);
     a.x_cast = want_cast ? cast : nullptr;
@@ -530,39 +588,51 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
     a.rows = f.rows; a.n_rows = T; a.H = H; a.dim = c.hidden_true; a.eps = c.eps; a.dtype = c.dtype;
     cur = nxt;
     pend = {};
-    return rf_stream_norm(&a, st);
+    if (!conv_w) return rf_stream_norm(&a, st);
+    if (f.decode && !s.fp32()) {
+      a.conv_w = conv_w; a.conv_state = conv_state; a.conv_taps = c.input_taps;
+      return rf_stream_norm(&a, st);
+    }
+    a.out = cast;                       // portions: the rows are written, then convolved
+    int rc = rf_stream_norm(&a, st);
+    if (rc) return rc;
+    RfConvSilu cv = {};
+    cv.x = cast; cv.ldx = H; cv.y = h; cv.ldy = H; cv.w = conv_w; cv.state = conv_state; cv.rows = f.rows;
+    cv.channels = H; cv.taps = c.input_taps; cv.dtype = c.dtype; cv.max_q_len = longest_portion(f); cv.add = 1;
+    return rf_conv_silu(&cv, st);
   };
   for (int l = 0; l < c.layers; ++l) {
     const RfMixedLayer& w = s.layers[l];
-    rc = c.norm_after ? step(nullptr, nullptr, nullptr, true) : step(w.norm1, w.shift, w.st.shift_state, false);
+    rc = c.norm_after ? step(nullptr, nullptr, nullptr, true) : step(w.norm1, w.shift, w.st.shift_state, false, w.input_conv[0], w.st.input_state[0]);
     if (rc) return rc;
     const void* in = c.norm_after ? cast : h;
     switch (w.mixer) {
       case RF_MIXER_LATENT_ATTENTION: rc = latent_attention(s, w, f, in, mix, st); break;
       case RF_MIXER_HGRN2: rc = hgrn2(s, w, f, in, mix, st); break;
+      case RF_MIXER_DELTA: rc = delta(s, w, f, in, mix, st); break;
       case RF_MIXER_ATTENTION: rc = grouped_attention(s, w, f, in, mix, st); break;
       default: rc = mamba1(s, w, f, in, mix, st);
     }
     if (rc) return rc;
     rc = linear(s, mix, w.out_dim, w.w_o, y, H, T, H, w.out_dim, kActNone, st);
     if (rc) return rc;
-    pend.y = y; pend.norm = c.norm_after ? w.norm1 : nullptr;
+    pend.y = y; pend.norm = c.norm_after ? w.norm1 : w.norm1b;
     if (w.inter > 0) {
-      rc = c.norm_after ? step(nullptr, nullptr, nullptr, true) : step(w.norm2, nullptr, nullptr, false);
+      rc = c.norm_after ? step(nullptr, nullptr, nullptr, true) : step(w.norm2, nullptr, nullptr, false, w.input_conv[1], w.st.input_state[1]);
       if (rc) return rc;
       if (w.experts > 0) {
         rc = experts(s, w, f, in, &pend, st);
       } else {
         void* wide = s.at(s.off_wide);
-        rc = w.act == RF_MIXED_ACT_CLIPPED_GLU
-                 ? linear_pair(s, in, H, w.w_up, wide, w.inter, T, w.inter, H, kActClippedGlu, w.act_limit, w.act_alpha, st)
+        rc = w.act != RF_MIXED_ACT_RELU2
+                 ? linear_pair(s, in, H, w.w_up, wide, w.inter, T, w.inter, H, w.act == RF_MIXED_ACT_SWIGLU ? kActSiluMul : kActClippedGlu, w.act_limit, w.act_alpha, st)
                  : linear(s, in, H, w.w_up, wide, w.inter, T, w.inter, H, kActRelu2, st);
         if (rc) return rc;
         rc = linear(s, wide, w.inter, w.w_down, y, H, T, H, w.inter, kActNone, st);
         pend.y = y;
       }
       if (rc) return rc;
-      pend.norm = c.norm_after ? w.norm2 : nullptr;
+      pend.norm = c.norm_after ? w.norm2 : w.norm2b;
     }
     if (c.side_dim > 0) {
       rc = step(nullptr, nullptr, nullptr, true);
@@ -577,6 +647,7 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
     if (f.taps) {
       RfStreamNorm a = {};
       a.x = s.at<float>(s.off_x[cur]); a.y_mult = c.residual_mult; a.y = pend.y; a.y_norm_w = pend.norm; a.y_slots = pend.slots; a.y_picks = pend.picks;
+      a.y_self = pend.self; a.y_self_w = pend.self_w;
       a.x_out = f.taps + (size_t)l * T * H;
       a.rows = f.rows; a.n_rows = T; a.H = H; a.dim = c.hidden_true; a.eps = c.eps; a.dtype = c.dtype;
       rc = rf_stream_norm(&a, st);
@@ -601,7 +672,7 @@ extern "C" int64_t rf_mixed_create(const RfMixedConfig* c) {
   if (!c || c->layers <= 0 || c->hidden <= 0 || c->hidden % 8 || c->hidden_true <= 0 || c->hidden_true > c->hidden || c->vocab <= 0 ||
       c->vocab_ld < c->vocab || c->vocab_ld % 8 || c->dtype < 0 || c->dtype > 2 || c->max_tokens <= 0 || c->max_seqs <= 0 ||
       c->max_seq_len <= 0 || c->side_dim < 0 || c->side_dim % 8 || !c->embed || !c->final_norm || !c->w_lm || c->long_min < 1 ||
-      (c->dtype == kF32 && c->weights_packed) || c->logit_softcap < 0.f ||
+      (c->dtype == kF32 && c->weights_packed) || c->logit_softcap < 0.f || c->input_taps < 0 || (c->input_taps > 0 && c->norm_after) ||
       (c->pair_table && (c->pair_buckets <= 0 || c->pair_mul_prev < 0 || c->pair_mul_cur < 0))) {
     fail(RF_ERR_BAD_ARG, "invalid mixed-stack config");
     return -1;
@@ -620,17 +691,22 @@ extern "C" int rf_mixed_set_layer(int64_t h, int32_t layer, const RfMixedLayer* 
   RF_GET_MIXED(h);
   RF_REQUIRE(w && layer >= 0 && layer < s.cfg.layers, "layer index %d out of range", layer);
   RF_REQUIRE(w->in_dim % 8 == 0 && w->out_dim > 0 && w->out_dim % 8 == 0 && w->inter >= 0 && w->inter % 8 == 0, "layer %d: projection and feed-forward sizes", layer);
+  if (s.cfg.input_taps > 0)
+    RF_REQUIRE(w->input_conv[0] && !w->shift && (w->inter == 0 || w->input_conv[1]) && (s.cfg.input_taps == 1 || (w->st.input_state[0] && w->st.input_state[1])),
+               "layer %d: input convolutions", layer);
   if (w->mixer != RF_MIXER_MAMBA1) {
     RF_REQUIRE(w->heads > 0 && w->dim > 0 && w->dim % 8 == 0 && w->vdim > 0 && w->vdim % 8 == 0, "layer %d: head sizes", layer);
     RF_REQUIRE(w->out_dim == w->heads * w->vdim, "layer %d: output projection columns", layer);
   }
   RF_REQUIRE(w->norm1 && w->w_in && w->w_o && (!w->shift || w->st.shift_state), "layer %d: missing weights", layer);
-  if (w->inter > 0) RF_REQUIRE(w->norm2 && w->w_up && w->w_down && (w->act == RF_MIXED_ACT_RELU2 || (w->act == RF_MIXED_ACT_CLIPPED_GLU && w->act_limit > 0.f)),
+  if (w->inter > 0) RF_REQUIRE(w->norm2 && w->w_up && w->w_down && (w->act == RF_MIXED_ACT_RELU2 || w->act == RF_MIXED_ACT_SWIGLU ||
+                                  (w->act == RF_MIXED_ACT_CLIPPED_GLU && w->act_limit > 0.f) || (w->act == RF_MIXED_ACT_GELU && w->experts > 0 && w->shared_inter == 0)),
                                  "layer %d: feed-forward weights", layer);
   if (s.cfg.pair_table) RF_REQUIRE(w->st.last_token && !w->shift, "layer %d: token pairs need the carried tokens and no token shift", layer);
   if (w->experts > 0) {
-    RF_REQUIRE(w->inter > 0 && w->router && w->experts <= 256 && w->top > 0 && w->top <= 32 && w->groups > 0 && w->experts % w->groups == 0 &&
-                   w->keep > 0 && w->keep <= w->groups && w->top <= w->experts / w->groups * w->keep,
+    const int routed = w->experts + w->identity;
+    RF_REQUIRE(w->inter > 0 && w->router && w->identity >= 0 && routed <= 256 && w->top > 0 && w->top <= 32 && w->groups > 0 && routed % w->groups == 0 &&
+                   w->keep > 0 && w->keep <= w->groups && w->top <= routed / w->groups * w->keep,
                "layer %d: %d experts in %d groups, %d kept, %d chosen", layer, w->experts, w->groups, w->keep, w->top);
     RF_REQUIRE(w->bank_inter >= w->inter && w->bank_inter % (s.cfg.dtype == kF32 ? 8 : 128) == 0 && w->shared_inter >= 0 && w->shared_inter % 8 == 0 &&
                    (w->shared_inter == 0 || (w->shared_up && w->shared_down)) && (!w->shared_gate || w->shared_inter > 0) &&
@@ -638,9 +714,13 @@ extern "C" int rf_mixed_set_layer(int64_t h, int32_t layer, const RfMixedLayer* 
     RF_REQUIRE(s.cfg.dtype == kF32 || s.cfg.weights_packed, "layer %d: experts need tile-major weights", layer);
   }
   if (w->mixer == RF_MIXER_LATENT_ATTENTION) {
-    RF_REQUIRE(w->rank > 0 && w->rank % 16 == 0 && w->rank_true > 0 && w->latent_norm && w->w_absorb && w->w_unabsorb && w->st.latent_pool,
+    RF_REQUIRE(w->rank > 0 && w->rank % 16 == 0 && w->rank_true > 0 && (w->latent_norm || w->shares) && w->w_absorb && w->w_unabsorb && w->st.latent_pool,
                "layer %d: latent-attention weights", layer);
-    RF_REQUIRE(w->in_dim >= w->heads * w->dim + w->rank, "layer %d: input projection rows", layer);
+    RF_REQUIRE(w->q_rank % 8 == 0 && (w->q_rank == 0 || (w->w_uq && w->q_latent_norm && w->q_rank_true > 0 && w->q_rank_true <= w->q_rank)) && (!w->shares || w->q_rank > 0),
+               "layer %d: query latent", layer);
+    RF_REQUIRE(w->plain > 0 && w->plain % 8 == 0 && w->rot >= 0 && w->rot % 2 == 0 && w->rot_pad >= w->rot && w->rot_pad % 16 == 0 &&
+                   w->plain + (w->rot + 7) / 8 * 8 <= w->dim && (w->rot == 0 || (w->cos && w->sin)), "layer %d: rotated part", layer);
+    RF_REQUIRE(w->in_dim >= (w->q_rank > 0 ? w->q_rank : w->heads * w->dim) + (w->shares ? 0 : w->rank + w->rot_pad), "layer %d: input projection rows", layer);
     RF_REQUIRE(w->expand_hd == 0 || (w->w_expand && w->dim == w->expand_hd && w->vdim == w->expand_hd && s.cfg.dtype != kF32),
                "layer %d: expanded heads", layer);
   } else if (w->mixer == RF_MIXER_ATTENTION) {
@@ -651,6 +731,10 @@ extern "C" int rf_mixed_set_layer(int64_t h, int32_t layer, const RfMixedLayer* 
                "layer %d: convolution of %d taps, %d kept positions", layer, w->conv_taps, w->keep_first);
     RF_REQUIRE(!w->tensor_core || (s.cfg.dtype != kF32 && (w->dim == 64 || w->dim == 128 || w->dim == 256) && w->scale > 0.f), "layer %d: heads", layer);
     RF_REQUIRE(w->rot_dims % 2 == 0 && w->rot_dims >= 0 && w->rot_dims <= w->dim_true && (w->rot_dims == 0 || (w->cos && w->sin)), "layer %d: rotation", layer);
+  } else if (w->mixer == RF_MIXER_DELTA) {
+    RF_REQUIRE(w->kv_heads > 0 && w->heads % w->kv_heads == 0 && w->dim_true > 0 && w->dim_true <= w->dim && w->vdim_true > 0 && w->vdim_true <= w->vdim &&
+                   w->taps > 0 && w->in_dim >= MixedStack::delta_channels(*w) + w->heads * w->vdim + 2 * ((w->heads + 7) / 8 * 8), "layer %d: delta-rule sizes", layer);
+    RF_REQUIRE(w->conv_w && w->rate && w->dt_bias && w->head_norm && w->st.rec_state && w->st.conv_state, "layer %d: delta-rule weights", layer);
   } else if (w->mixer == RF_MIXER_MAMBA1) {
     RF_REQUIRE(w->inner > 0 && w->inner % 8 == 0 && w->states > 0 && w->states % 8 == 0 && w->states <= 256 && w->dt_rank > 0 && w->dt_rank % 8 == 0 &&
                    w->taps > 0 && w->in_dim == 2 * w->inner && w->out_dim == w->inner, "layer %d: scan sizes", layer);
@@ -728,7 +812,7 @@ extern "C" int rf_mixed_head(int64_t h, const int32_t* row_idx, int32_t rows, in
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   RfStreamNorm a = {};
   a.x = s.at<float>(s.off_x[s.cur]); a.row_idx = row_idx; a.y_mult = c.residual_mult;
-  a.y = s.tail.y; a.y_norm_w = s.tail.norm; a.y_slots = s.tail.slots; a.y_picks = s.tail.picks;
+  a.y = s.tail.y; a.y_norm_w = s.tail.norm; a.y_slots = s.tail.slots; a.y_picks = s.tail.picks; a.y_self = s.tail.self; a.y_self_w = s.tail.self_w;
   a.norm_w = c.final_norm; a.out = s.at(s.off_head);
   a.n_rows = rows; a.H = c.hidden; a.dim = c.hidden_true; a.eps = c.eps; a.dtype = c.dtype;
   int rc = rf_stream_norm(&a, st);
@@ -747,5 +831,6 @@ extern "C" void rf_mixed_struct_sizes(int32_t* out) {
   out[3] = (int32_t)sizeof(RfRows); out[4] = (int32_t)sizeof(RfStreamNorm); out[5] = (int32_t)sizeof(RfLatentAttn);
   out[6] = (int32_t)sizeof(RfHgrn2); out[7] = (int32_t)sizeof(RfHeadLinear); out[8] = (int32_t)sizeof(RfMixedState);
   out[9] = (int32_t)sizeof(RfAttn); out[10] = (int32_t)sizeof(RfQkvInsert); out[11] = (int32_t)sizeof(RfConvSilu);
+  out[15] = (int32_t)sizeof(RfLatentInsert); out[16] = (int32_t)sizeof(RfHeadRotate); out[17] = (int32_t)sizeof(RfDelta);
   out[12] = (int32_t)sizeof(RfMamba1); out[13] = (int32_t)sizeof(RfMoeRouter); out[14] = (int32_t)sizeof(RfMoeExperts);
 }

@@ -260,6 +260,7 @@ typedef struct RfAttn {
   int32_t gate_by_head;     // 1: gate is [rows, Hq], one number per head
   int32_t keep_first;       // with a window: the first keep_first positions of the sequence stay visible
   const float* slopes;      // [Hq]: slopes[h] * (i - j) is taken off the scores of position i (paged forms)
+  const float* rates;       // [Hq], with slopes: slopes[h] * ln(1 + rates[h] * (i - j)) instead
   // rf_attn_decode by row: with `pos`, query row r is position pos[r] of sequence seq_of_row[r] (null: r) and sees what its
   // chunk or window leaves of everything up to itself; kv_len is not used and num_seqs counts rows.
   const int32_t* seq_of_row; const int32_t* pos;
@@ -334,6 +335,10 @@ typedef struct RfRows {
 // carries every sequence's last token (not together with `shift`).  The outstanding output is multiplied by y_mult (0 counts as 1)
 // when it is added.  With y_picks > 0 the outstanding output is the sum of y_picks rows of y, those
 // that y_slots[row * y_picks ...] names (negative: none): the experts' results of a mixture of experts.
+// y_self_w [rows] adds y_self_w[row] * y_self[row] to that sum (experts whose output is their input).
+// With conv_w (decode rows only: every row is a sequence of its own) the normalised row, rounded to the activation dtype, goes through
+// the input convolution before it is written: out = h + sum_k conv_w[k] h[t - (taps - 1) + k], the last taps - 1 rows h carried in
+// conv_state [slots, taps - 1, H], oldest first (portions: rf_conv_silu with `add` behind this step, same state).
 // H is the (padded, multiple of 8) row length, dim the true one that the means run over.  x_out must not alias x when
 // `shift` is set.  row_idx (optional) selects the rows that are processed (not together with shift).
 typedef struct RfStreamNorm {
@@ -348,6 +353,8 @@ typedef struct RfStreamNorm {
   const int32_t* y_slots; int32_t y_picks;
   float y_mult;
   const void* table2; int32_t* last_token; int64_t mul_prev, mul_cur; int32_t buckets;
+  const void* y_self; const float* y_self_w;
+  const float* conv_w; void* conv_state; int32_t conv_taps;
 } RfStreamNorm;
 int rf_stream_norm(const RfStreamNorm* a, rf_stream_t stream);
 
@@ -369,17 +376,31 @@ typedef struct RfHeadLinear {
 } RfHeadLinear;
 int rf_head_linear(const RfHeadLinear* a, rf_stream_t stream);
 
-// Latent-attention cache: one row of `rank` (padded to a multiple of 16) values per token, pool [pages, 16, rank].
-// rf_latent_insert: c = x / rms(x) * norm_w (mean over the true rank), stored at the row's position.
-int rf_latent_insert(const void* x, int64_t ldx, const float* norm_w, void* pool, const RfRows* rows, int32_t n_rows,
-                     int32_t rank, int32_t rank_true, float eps, int32_t dtype, rf_stream_t stream);
-// The insertion above together with the per-head map of the queries into the latent space (one launch in 16 bits): what a
-// decode step does between the input projection and the attention.
+// Latent-attention cache: one row of `rank` (padded to a multiple of 16) values per token, pool [pages, 16, rank], or, with a
+// rotated key part that all heads share, [pages, 16, rank + rot_pad] (rot values behind the latent, padded to a multiple of 16).
+// rf_latent_insert: c = x / rms(x) * norm_w (mean over the true rank), stored at the row's position; x holds the rotated part at
+// column `rank`, turned by the row's position on the way (RfHeadRotate).  With q also the rows' query latents (their own norm, in
+// place).  x null: the query latents alone (a layer that attends over another layer's cache).
 typedef struct RfLatentInsert {
   const void* x; int64_t ldx; const float* norm_w; void* pool; RfRows rows;
   int32_t n_rows, rank, rank_true; float eps;
+  int32_t rot, rot_pad; const float* cos; const float* sin;
+  void* q; int64_t ldq; const float* q_norm; int32_t q_rank, q_rank_true;
 } RfLatentInsert;
-int rf_latent_absorb(const RfHeadLinear* q, const RfLatentInsert* c, rf_stream_t stream);
+int rf_latent_insert(const RfLatentInsert* c, int32_t dtype, rf_stream_t stream);
+// Rotation of `dims` values of every head in neighbouring pairs: (u, v) of pair i at position p becomes (u c - v s, v c + u s) with
+// c, s = cos / sin[p, i] (tables [positions, dims / 2]).  Head h of row r starts at x + r * ldx + h * xs (to y likewise, possibly in
+// place); values from dims to dims_pad (a multiple of 8) are written as zeros.
+typedef struct RfHeadRotate {
+  const void* x; int64_t ldx; int32_t xs;
+  void* y; int64_t ldy; int32_t ys;
+  const int32_t* pos; const float* cos; const float* sin;
+  int32_t rows, heads, dims, dims_pad;
+} RfHeadRotate;
+int rf_head_rotate(const RfHeadRotate* a, int32_t dtype, rf_stream_t stream);
+// The per-head map of the queries into the latent space together with the insertion and / or the rotation above (either may be
+// null; one launch in 16 bits): what a decode step does between the query projection and the attention.
+int rf_latent_absorb(const RfHeadLinear* q, const RfLatentInsert* c, const RfHeadRotate* t, rf_stream_t stream);
 // Dense copies of the latents that sequences can see: the last kv_len[s] cached rows of sequence s, its own new rows (already
 // inserted) included, to rows [kv_start[s], kv_start[s] + kv_len[s]) of out.  max_len: host bound of kv_len.
 int rf_latent_gather(const void* pool, void* out, const RfRows* rows, const int32_t* kv_start, const int32_t* kv_len, int32_t rank,
@@ -388,11 +409,13 @@ int rf_latent_gather(const void* pool, void* out, const RfRows* rows, const int3
 // Attention in the latent space (keys and values folded into the queries and the output): every row attends from its own
 // position to the window before it, score = (q[r, h] . c[j]) * scale, o[r, h] = sum_j softmax(score)_j c[j].
 // q, o: [rows, heads, rank] dense.  window <= 0: no lower bound.  max_kv: host bound of the keys one row sees.
+// With vrank > 0 only the first vrank of the rank cached columns are values (the others are a rotated key part): o is [rows, heads, vrank].
 typedef struct RfLatentAttn {
   const void* q; void* o; const void* pool;
   RfRows rows;
   int32_t n_rows, heads, rank, window, max_kv; float scale; int32_t dtype;
   float* ws; uint64_t ws_bytes;      // split partials, optional
+  int32_t vrank;
 } RfLatentAttn;
 int rf_latent_attn(const RfLatentAttn* a, rf_stream_t stream);
 uint64_t rf_latent_attn_scratch_bytes(int rows, int heads, int rank, int max_kv);
@@ -417,6 +440,7 @@ typedef struct RfQkvInsert {
   // taps - 1 rows of [queries | keys | values] are carried in conv_state [slots, taps - 1, (heads + 2 kv_heads) * hd], oldest first.
   // conv_w: [taps, (heads + 2 kv_heads) * hd].  The rows are read only, queries go to q_out [n_rows, heads * hd].
   const float* conv_w; void* conv_state; void* q_out; int32_t taps, max_q_len;
+  float growth; int32_t growth_every;  // every > 0: queries of position p times 1 + growth * ln(floor((p + 1) / every) + 1)
 } RfQkvInsert;
 int rf_qkv_insert(const RfQkvInsert* a, rf_stream_t stream);
 // Attention by row on the CUDA cores in fp32, any head size up to 2048 and any scale: the by-row form of rf_attn_decode (pos,
@@ -425,11 +449,13 @@ int rf_attn_rows(const RfAttn* a, rf_stream_t stream);
 
 // Causal convolution per channel over packed rows, silu applied: y[t] = silu(bias + sum_k w[k] x[t - (taps - 1) + k]).  The last
 // taps - 1 inputs of every sequence are carried in state [slots, taps - 1, channels], oldest first.  w: [taps, channels] fp32.
+// `add`: y[t] = x[t] + the sum, without silu.  `ring`: state is [slots, taps, channels], the input of position p in row p mod taps.
 typedef struct RfConvSilu {
   const void* x; int64_t ldx; void* y; int64_t ldy;
   const float* w; const float* bias; void* state;
   RfRows rows;
   int32_t max_q_len, channels, taps, dtype;
+  int32_t add, ring;
 } RfConvSilu;
 int rf_conv_silu(const RfConvSilu* a, rf_stream_t stream);
 
@@ -447,6 +473,20 @@ typedef struct RfMamba1 {
 } RfMamba1;
 int rf_mamba1_recurrent(const RfMamba1* a, rf_stream_t stream);
 int rf_mamba1_scan(const RfMamba1* a, rf_stream_t stream);
+
+// Gated delta rule with an output norm and gate (see kernels/delta_rule.cu).  Rows of x hold [q: kv_heads * dim | k: kv_heads * dim |
+// v: heads * vdim] behind the short convolution and silu; head h uses query / key head h / (heads / kv_heads).  rate [heads] = exp(A_log);
+// state fp32 [slots, heads, dim, vdim]; padding dimensions of q, k and v are zero.  b, a: [rows, >= heads]; gate [rows, heads * vdim].
+// With conv_w (decode steps of the recurrent form) x are the projections: conv_w [taps, channels] and the ring of rf_conv_silu.
+typedef struct RfDelta {
+  const void* x; int64_t ldx; const void* b; const void* a; int64_t ld_ba; const void* gate; int64_t ldg;
+  const float* rate; const float* dt_bias; const float* norm_w;
+  float* state; void* out; int64_t ldo;
+  RfRows rows;
+  int32_t heads, kv_heads, dim, dim_true, vdim, vdim_true; float eps; int32_t dtype;
+  const float* conv_w; void* conv_state; int32_t taps;
+} RfDelta;
+int rf_delta_recurrent(const RfDelta* a, rf_stream_t stream);
 
 // HGRN2 linear attention (what a gate takes from the state it gives to the new value), over packed input rows [q | f | v]:
 //   q = silu(q), f = lower + (1 - lower) * sigmoid(f + f_bias), S = diag(f) S + (1 - f) v^T, o = S^T q,
@@ -520,7 +560,8 @@ int rf_moe_combine(void* out, int64_t ldo, const void* y, int64_t ldy, const int
 // what rf_moe_gather otherwise writes: slot_of [rows, slot_ld] (sorted row of every pick, then of the shared expert),
 // token_of_slot and slot_w.  counters: experts + 1 words, zero before the first launch and left zero.
 // RF_MOE_CHOSEN: the correction is a bias of the logits; the k largest logits are chosen and the weights are the softmax over the
-// chosen ones.  shared_gate: w has one more row behind the experts', sigmoid of its logit is the shared expert's weight (else 1).
+// chosen ones.  identity: the last this many experts have no weights, their output is their input; picks of them get no row, their
+// weights are added up in self_w [rows].  shared_gate: w has one more row behind the experts', sigmoid of its logit is the shared expert's weight (else 1).
 enum RfMoeScore { RF_MOE_SIGMOID = 0, RF_MOE_SOFTMAX = 1, RF_MOE_CHOSEN = 2 };
 typedef struct RfMoeRouter {
   const void* x; int64_t ldx; const void* w; const float* correction;
@@ -530,6 +571,7 @@ typedef struct RfMoeRouter {
   int32_t tile_rows, slot_ld, has_shared, shared_tiles, scatter, dtype;
   float* logits;                       // scratch, rf_moe_router_scratch_bytes(rows, experts + shared_gate)
   int32_t shared_gate;
+  int32_t identity; float* self_w;
 } RfMoeRouter;
 uint64_t rf_moe_router_scratch_bytes(int rows, int experts);
 int rf_moe_router(const RfMoeRouter* a, rf_stream_t stream);
@@ -545,7 +587,7 @@ typedef struct RfMoeExperts {
   const int32_t* tiles; const int32_t* token_of_slot; const float* slot_w;
   int32_t max_tiles, experts, n, k, shared_n, shared_k, dual, tile_rows;
   int32_t bank_section_row_tiles, bank_kb_total, rt_per_expert, kb_per_expert, shared_section_row_tiles, shared_kb_total, dtype;
-  int32_t act;                         // dual: rf::Act of two operands (0 counts as silu(g) u)
+  int32_t act;                         // dual: rf::Act of two operands (0 counts as silu(g) u); else of one operand (two-operand ones count as none)
   float act_limit, act_alpha, shared_limit;   // its constants; the shared expert has a limit of its own
 } RfMoeExperts;
 int rf_moe_experts(const RfMoeExperts* a, rf_stream_t stream);

@@ -1,13 +1,14 @@
 """Decoders whose layers name their own mixer: configuration records and weight tables.
 
 A :class:`MixedConfig` is a list of layers, each with one mixer (:class:`LatentAttention`, :class:`HGRN2`,
-:class:`GroupedAttention`, :class:`Mamba1`) and an optional feed-forward (:class:`DenseMLP`, :class:`ClippedGLU`, :class:`MoE`), over
-what the layers share: the width of an fp32 residual stream, RMSNorm epsilon, where the norms sit, and optionally an embedding of
-token pairs, a factor on the sublayers' outputs, a token shift in front of every mixer, a gated per-token side input behind every
-layer and a soft cap of the logits.  The native executor is ``csrc/models/mixed_stack.cu``, the engine
+:class:`GroupedAttention`, :class:`Mamba1`, :class:`DeltaRule`) and an optional feed-forward (:class:`DenseMLP`, :class:`GatedMLP`,
+:class:`ClippedGLU`, :class:`MoE`), over what the layers share: the width of an fp32 residual stream, RMSNorm epsilon, where the norms
+sit, and optionally an embedding of token pairs, a factor on the sublayers' outputs, a token shift in front of every mixer, a
+convolution in front of every sublayer, a gated per-token side input behind every layer and a soft cap of the logits.  The native executor is ``csrc/models/mixed_stack.cu``, the engine
 :mod:`rhinoforge_b200.runtime.mixed_engine`.
 
-Readers of ``config.json``: :meth:`MixedConfig.from_vabarax`, :meth:`MixedConfig.from_zulopel`, :meth:`MixedConfig.from_kuzupel`.
+Readers of ``config.json``: :meth:`MixedConfig.from_vabarax`, :meth:`MixedConfig.from_zulopel`, :meth:`MixedConfig.from_kuzupel`,
+:meth:`MixedConfig.from_vasosun`.
 """
 from __future__ import annotations
 
@@ -23,13 +24,18 @@ from ..runtime.errors import UnsupportedModelError
 @dataclass(frozen=True)
 class LatentAttention:
     """Attention over one cached latent row per token; keys and values of a head are linear maps of it.  ``window``: how many
-    positions a query sees, its own included (None: all of them)."""
+    positions a query sees, its own included (None: all of them).  ``q_rank`` > 0: queries go through a normalised latent of this size.
+    ``rot``: every query head has ``rot.dims`` more dimensions, rotated in neighbouring pairs, against one rotated key part per token that
+    all heads share and that is cached behind the latent.  ``kv_from``: the layer whose cache this one attends over (None: its own)."""
     heads: int
     dim: int
     vdim: int
     kv_rank: int
     scale: float
     window: Optional[int] = None
+    q_rank: int = 0
+    rot: Optional["Rotary"] = None
+    kv_from: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -52,7 +58,8 @@ class YarnScaling:
 
 @dataclass(frozen=True)
 class Rotary:
-    """Rotation of the first ``dims`` dimensions of a head, dimension i paired with i + dims / 2."""
+    """Rotation of ``dims`` dimensions of a head: the first ones, dimension i paired with i + dims / 2 (:class:`GroupedAttention`), or a
+    part of their own, dimension 2 i paired with 2 i + 1 (:class:`LatentAttention`)."""
     dims: int
     base: float
     scaling: Optional[YarnScaling] = None
@@ -85,7 +92,9 @@ class GroupedAttention:
     ``unit_sink``: that term is exp(0) in every head.  ``v_mix``: values are mixed with those of the first layer that says so.
     ``qk_norm``: RMSNorm of every query and key head, or with ``norm_all`` one over all query heads and one over all key heads.
     ``conv`` > 0: causal convolution of this many taps on the projected queries, keys and values.  ``gate``: sigmoid gate on the
-    heads' outputs, element by element, or with ``gate_by_head`` one number per head."""
+    heads' outputs, element by element, or with ``gate_by_head`` one number per head.  ``log_bias``: head h's scores lose
+    ``r1[h] ln(1 + r2[h] distance)`` with learned r1 and r2.  ``growth_every`` > 0: queries of position p are multiplied by
+    ``1 + growth ln(floor((p + 1) / growth_every) + 1)``."""
     heads: int
     kv_heads: int
     dim: int
@@ -104,6 +113,9 @@ class GroupedAttention:
     norm_all: bool = False
     conv: int = 0
     gate_by_head: bool = False
+    log_bias: bool = False
+    growth: float = 0.0
+    growth_every: int = 0
 
     def slopes(self) -> Optional[torch.Tensor]:
         """float64 ``[heads]``: what the scores lose per token of distance."""
@@ -119,6 +131,23 @@ class Mamba1:
     state: int
     dt_rank: int
     conv: int
+
+
+@dataclass(frozen=True)
+class DeltaRule:
+    """Gated delta rule (state ``[heads, dim, vdim]``) over ``kv_heads`` query / key heads, behind a causal convolution of ``conv`` taps
+    with silu on queries, keys and values; the outputs are normalised per head and gated."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+
+
+@dataclass(frozen=True)
+class GatedMLP:
+    """``down(silu(gate h) * up h)``."""
+    ff: int
 
 
 @dataclass(frozen=True)
@@ -142,7 +171,9 @@ class MoE:
     ``router`` "corrected": chosen among the ``keep`` best of ``groups`` groups by softmax score plus correction, weighted by
     normalised score.  "chosen": the logits have a bias, the largest are chosen, weights are the softmax over the chosen ones.
     ``limit``: experts are clipped (:class:`ClippedGLU`), the shared one with ``shared_limit``; None: SwiGLU.  ``shared_gate``: the
-    shared expert is weighted by a sigmoid of one number per token."""
+    shared expert is weighted by a sigmoid of one number per token.  ``gated`` False: experts are ``down(gelu(up h))``.  ``identity``: this
+    many more experts behind the others whose output is their input.  ``renormalise`` False: the weights of "corrected" stay the
+    chosen experts' scores."""
     experts: int
     top: int
     ff: int
@@ -154,6 +185,9 @@ class MoE:
     shared_limit: Optional[float] = None
     alpha: float = 1.702
     shared_gate: bool = False
+    gated: bool = True
+    identity: int = 0
+    renormalise: bool = True
 
 
 @dataclass(frozen=True)
@@ -167,8 +201,8 @@ class TokenPairs:
 
 @dataclass(frozen=True)
 class MixedLayer:
-    mixer: Union[LatentAttention, HGRN2, GroupedAttention, Mamba1]
-    mlp: Optional[Union[DenseMLP, ClippedGLU, MoE]] = None
+    mixer: Union[LatentAttention, HGRN2, GroupedAttention, Mamba1, DeltaRule]
+    mlp: Optional[Union[DenseMLP, GatedMLP, ClippedGLU, MoE]] = None
 
 
 def _int(d: Mapping[str, Any], key: str, where: str, least: int = 1) -> int:
@@ -208,6 +242,9 @@ class MixedConfig:
     side_dim: int = 0              # width of the per-token side input behind every layer (0: none)
     token_shift: bool = True       # mix every token's normalised row with the one before, in front of every mixer
     norm_after: bool = False       # norms on the sublayers' outputs instead of their inputs
+    norm_both: bool = False        # norms on the sublayers' outputs as well as on their inputs
+    scalar_norms: bool = False     # the norms around the sublayers and the last one have one weight for all coordinates
+    input_taps: int = 0            # > 0: h + convolution of this many taps over h in front of every sublayer
     layer_scale: bool = False      # element-wise factors on the sublayers' outputs
     tied_head: bool = True
     embed_scale: float = 1.0
@@ -346,17 +383,13 @@ class MixedConfig:
                 raise UnsupportedModelError(f"{where}: mixer type {entry.get('type')!r} is not built")
             mlp = None if entry.get("mlp") is None else _kuzupel_mlp(_map(entry, "mlp", where), where + " mlp")
             layers.append(MixedLayer(read(_map(entry, "mixer", where), where), mlp))
-        norm, emb, pairs = _map(c, "norm", "Kuzupel"), c.get("embedding") or {}, None
+        norm, emb = _map(c, "norm", "Kuzupel"), c.get("embedding") or {}
         _known(norm, ("eps",), "Kuzupel norm")
         _known(emb, ("scale", "bigram"), "Kuzupel embedding")
-        if emb.get("bigram") is not None:
-            b, w = _map(emb, "bigram", "Kuzupel embedding"), "Kuzupel bigram"
-            _known(b, ("buckets", "mul_prev", "mul_cur"), w)
-            pairs = TokenPairs(_int(b, "buckets", w), _int(b, "mul_prev", w, 0), _int(b, "mul_cur", w, 0))
         number = lambda d, key, default, where: default if d.get(key) is None else _float(d, key, where, True)
         cap = c.get("logit_softcap")
         return cls.kuzupel("kuzupel", _int(c, "vocab", "Kuzupel"), _int(c, "width", "Kuzupel"), _float(norm, "eps", "Kuzupel norm"), layers,
-                           pairs=pairs, embed_scale=number(emb, "scale", 1.0, "Kuzupel embedding"),
+                           pairs=_token_pairs(emb, "Kuzupel"), embed_scale=number(emb, "scale", 1.0, "Kuzupel embedding"),
                            residual_mult=number(c, "residual_mult", 1.0, "Kuzupel"),
                            logit_softcap=None if cap is None else _float(c, "logit_softcap", "Kuzupel", True), raw=c)
 
@@ -387,6 +420,89 @@ class MixedConfig:
                "embedding": emb, "residual_mult": self.residual_mult, "layers": out}
         return top if self.logit_softcap is None else {**top, "logit_softcap": self.logit_softcap}
 
+    @classmethod
+    def vasosun(cls, name: str, vocab: int, width: int, eps: float, layers, *, input_taps: int = 0, pairs: Optional[TokenPairs] = None,
+                logit_softcap: Optional[float] = None, **kw) -> "MixedConfig":
+        """A decoder of the Vasosun design: delta-rule, window-attention and latent-attention layers in any order, SwiGLU feed-forwards
+        or mixtures with identity experts, scalar norms on both sides of the sublayers, a convolution in front of each."""
+        cfg = cls(name, vocab, width, eps, tuple(layers), 0, token_shift=False, norm_both=True, scalar_norms=True, input_taps=input_taps,
+                  tied_head=False, pairs=pairs, logit_softcap=logit_softcap, model_type="vasosun", **kw)
+        for i, m in enumerate(layer.mixer for layer in cfg.layers):
+            if getattr(m, "kv_from", None) is None:
+                continue
+            of = cfg.layers[m.kv_from].mixer if 0 <= m.kv_from < i else None
+            if not isinstance(of, LatentAttention) or of.kv_from is not None or (of.kv_rank, of.rot) != (m.kv_rank, m.rot):
+                raise UnsupportedModelError(f"{name} layer {i}: layer {m.kv_from} has no cache of its own with the same latent and rotation")
+        return cfg
+
+    @classmethod
+    def from_vasosun(cls, c: Mapping[str, Any]) -> "MixedConfig":
+        """The mapping of a Vasosun ``config.json``.  Keys that the reader does not know are refused rather than ignored."""
+        _known(c, ("architecture", "canon", "embedding", "layers", "logit_softcap", "norm", "vocab", "width"), "Vasosun")
+        if not isinstance(c.get("layers"), list) or not c["layers"]:
+            raise UnsupportedModelError("Vasosun: 'layers' must be a non-empty list")
+        layers = []
+        for i, entry in enumerate(c["layers"]):
+            where = f"Vasosun layer {i}"
+            if not isinstance(entry, Mapping):
+                raise UnsupportedModelError(f"{where}: must be a mapping")
+            _known(entry, ("type", "mixer", "mlp"), where)
+            read = {"attention": _vasosun_window, "latent_attention": _vasosun_latent, "delta": _vasosun_delta}.get(entry.get("type"))
+            if read is None:
+                raise UnsupportedModelError(f"{where}: mixer type {entry.get('type')!r} is not built")
+            mlp = None if entry.get("mlp") is None else _vasosun_mlp(_map(entry, "mlp", where), where + " mlp")
+            layers.append(MixedLayer(read(_map(entry, "mixer", where), where), mlp))
+        norm, taps = _map(c, "norm", "Vasosun"), 0
+        _known(norm, ("eps",), "Vasosun norm")
+        if c.get("canon") is not None:
+            _known(_map(c, "canon", "Vasosun"), ("taps",), "Vasosun canon")
+            taps = _int(c["canon"], "taps", "Vasosun canon")
+        emb = c.get("embedding") or {}
+        _known(emb, ("bigram",), "Vasosun embedding")
+        return cls.vasosun("vasosun", _int(c, "vocab", "Vasosun"), _int(c, "width", "Vasosun"), _float(norm, "eps", "Vasosun norm"), layers,
+                           input_taps=taps, pairs=_token_pairs(emb, "Vasosun"),
+                           logit_softcap=None if c.get("logit_softcap") is None else _float(c, "logit_softcap", "Vasosun", True), raw=c)
+
+    def to_vasosun(self) -> Dict[str, Any]:
+        """The inverse of :meth:`from_vasosun`."""
+        out = []
+        for layer in self.layers:
+            m, f = layer.mixer, layer.mlp
+            d: Dict[str, Any] = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim}
+            if isinstance(m, DeltaRule):
+                kind = "delta"
+                d.update(kv_heads=m.kv_heads, conv=m.conv)
+            elif isinstance(m, GroupedAttention):
+                kind = "attention"
+                d.update(kv_heads=m.kv_heads, scale=m.scale)
+                if m.window is not None:
+                    d["mask"] = {"size": m.window}
+                if m.growth_every:
+                    d["q_temp"] = {"coef": m.growth, "every": m.growth_every}
+            else:
+                kind = "latent_attention"
+                d.update(kv_rank=m.kv_rank, q_rank=m.q_rank, rot_dim=m.rot.dims, scale=m.scale, rot={"dims": m.rot.dims, "base": m.rot.base})
+                if m.rot.scaling is not None:
+                    y = m.rot.scaling
+                    d["rot"]["scaling"] = {"factor": y.factor, "original": y.original, "fast": y.fast, "slow": y.slow}
+                if m.kv_from is not None:
+                    d["kv_from"] = m.kv_from
+            mlp: Optional[Dict[str, Any]] = None
+            if isinstance(f, MoE):
+                mlp = {"kind": "moe", "expert": {"ff": f.ff}, "router": {"experts": f.experts, "identity": f.identity, "top": f.top}}
+            elif f is not None:
+                mlp = {"kind": "dense", "ff": f.ff}
+            out.append({"type": kind, "mixer": d, "mlp": mlp})
+        top: Dict[str, Any] = {"architecture": "Vasosun", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.rms_eps},
+                               "embedding": {}, "layers": out}
+        if self.pairs is not None:
+            top["embedding"]["bigram"] = {"buckets": self.pairs.buckets, "mul_prev": self.pairs.mul_prev, "mul_cur": self.pairs.mul_cur}
+        if self.input_taps:
+            top["canon"] = {"taps": self.input_taps}
+        if self.logit_softcap is not None:
+            top["logit_softcap"] = self.logit_softcap
+        return top
+
     def to_vabarax(self) -> Dict[str, Any]:
         """The inverse of :meth:`from_vabarax`."""
         out = []
@@ -403,6 +519,22 @@ class MixedConfig:
                 "token_side": {"dim": self.side_dim}, "layers": out}
 
 
+def _token_pairs(emb: Mapping[str, Any], design: str) -> Optional[TokenPairs]:
+    if emb.get("bigram") is None:
+        return None
+    b, w = _map(emb, "bigram", design + " embedding"), design + " bigram"
+    _known(b, ("buckets", "mul_prev", "mul_cur"), w)
+    return TokenPairs(_int(b, "buckets", w), _int(b, "mul_prev", w, 0), _int(b, "mul_cur", w, 0))
+
+
+def _yarn(r: Mapping[str, Any], where: str) -> Optional[YarnScaling]:
+    if not r.get("scaling"):
+        return None
+    sc, w = _map(r, "scaling", where), where + " scaling"
+    _known(sc, ("factor", "original", "fast", "slow"), w)
+    return YarnScaling(*(_float(sc, k, w, True) for k in ("factor", "original", "fast", "slow")))
+
+
 def _zulopel_attention(m: Mapping[str, Any], where: str) -> GroupedAttention:
     _known(m, ("heads", "kv_heads", "dim", "vdim", "scale", "mask", "rot", "v_mix"), where)
     mask, rot = m.get("mask") or {}, None
@@ -410,13 +542,7 @@ def _zulopel_attention(m: Mapping[str, Any], where: str) -> GroupedAttention:
     if m.get("rot"):
         r, w = _map(m, "rot", where), where + " rot"
         _known(r, ("dims", "base", "scaling"), w)
-        yarn = None
-        if r.get("scaling"):
-            sc, ws = _map(r, "scaling", w), w + " scaling"
-            _known(sc, ("factor", "original", "fast", "slow"), ws)
-            yarn = YarnScaling(_float(sc, "factor", ws, True), _float(sc, "original", ws, True), _float(sc, "fast", ws, True),
-                               _float(sc, "slow", ws, True))
-        rot = Rotary(_int(r, "dims", w), _float(r, "base", w, True), yarn)
+        rot = Rotary(_int(r, "dims", w), _float(r, "base", w, True), _yarn(r, w))
     a = GroupedAttention(_int(m, "heads", where), _int(m, "kv_heads", where), _int(m, "dim", where), _int(m, "vdim", where),
                          _float(m, "scale", where), _int(mask, "size", where + " mask") if mask else None, rot, bool(m.get("v_mix", False)))
     if a.heads % a.kv_heads:
@@ -492,10 +618,65 @@ def _kuzupel_mlp(f: Mapping[str, Any], where: str) -> Union[ClippedGLU, MoE]:
     return e
 
 
+def _shares(a: Mapping[str, int], where: str) -> None:
+    if a["heads"] % a["kv_heads"]:
+        raise UnsupportedModelError(f"{where}: {a['heads']} heads do not share {a['kv_heads']} key / value heads evenly")
+
+
+def _vasosun_window(m: Mapping[str, Any], where: str) -> GroupedAttention:
+    _known(m, ("heads", "kv_heads", "dim", "vdim", "scale", "mask", "q_temp"), where)
+    mask, t = m.get("mask") or {}, m.get("q_temp") or {}
+    _known(mask, ("size",), where + " mask")
+    _known(t, ("coef", "every"), where + " q_temp")
+    a = {k: _int(m, k, where) for k in ("heads", "kv_heads", "dim", "vdim")}
+    _shares(a, where)
+    return GroupedAttention(**a, scale=_float(m, "scale", where), qk_norm=False, sink=False, gate=False, log_bias=True,
+                            window=_int(mask, "size", where + " mask") if mask else None,
+                            growth=_float(t, "coef", where + " q_temp") if t else 0.0, growth_every=_int(t, "every", where + " q_temp") if t else 0)
+
+
+def _vasosun_latent(m: Mapping[str, Any], where: str) -> LatentAttention:
+    _known(m, ("heads", "dim", "vdim", "kv_rank", "q_rank", "rot_dim", "rot", "scale", "kv_from"), where)
+    a = {k: _int(m, k, where) for k in ("heads", "dim", "vdim", "kv_rank", "q_rank")}
+    r, w = _map(m, "rot", where), where + " rot"
+    _known(r, ("dims", "base", "scaling"), w)
+    rot = Rotary(_int(r, "dims", w), _float(r, "base", w, True), _yarn(r, w))
+    if rot.dims % 2 or rot.dims != _int(m, "rot_dim", where):
+        raise UnsupportedModelError(f"{where}: rotation of {rot.dims} of {m['rot_dim']} rotated dimensions")
+    return LatentAttention(**a, scale=_float(m, "scale", where), rot=rot, kv_from=None if m.get("kv_from") is None else _int(m, "kv_from", where, 0))
+
+
+def _vasosun_delta(m: Mapping[str, Any], where: str) -> DeltaRule:
+    _known(m, ("heads", "kv_heads", "dim", "vdim", "conv"), where)
+    a = {k: _int(m, k, where) for k in ("heads", "kv_heads", "dim", "vdim", "conv")}
+    _shares(a, where)
+    if a["dim"] > 256 or a["vdim"] > 512:
+        raise UnsupportedModelError(f"{where}: the delta rule takes states of up to 256 x 512, got {a['dim']} x {a['vdim']}")
+    return DeltaRule(**a)
+
+
+def _vasosun_mlp(f: Mapping[str, Any], where: str) -> Union[GatedMLP, MoE]:
+    if f.get("kind") == "dense":
+        _known(f, ("kind", "ff"), where)
+        return GatedMLP(_int(f, "ff", where))
+    if f.get("kind") != "moe":
+        raise UnsupportedModelError(f"{where}: feed-forward kind {f.get('kind')!r} is not built")
+    _known(f, ("kind", "expert", "router"), where)
+    expert, r = _map(f, "expert", where), _map(f, "router", where)
+    _known(expert, ("ff",), where + " expert")
+    _known(r, ("experts", "identity", "top"), where + " router")
+    e = MoE(_int(r, "experts", where), _int(r, "top", where), _int(expert, "ff", where), gated=False, renormalise=False,
+            identity=_int(r, "identity", where, 0) if r.get("identity") is not None else 0)
+    if e.top > e.experts + e.identity or e.experts + e.identity > 256 or e.top > 32:
+        raise UnsupportedModelError(f"{where}: {e.top} of {e.experts} + {e.identity} experts (the router takes up to 32 of 256)")
+    return e
+
+
 def weight_shapes(cfg: MixedConfig) -> Iterator[Tuple[str, Tuple[int, ...], str]]:
     """(tensor name, shape, kind) of a checkpoint; kind is 'linear', 'embed', 'norm', 'unit' (values in [0, 1)), 'bias', 'scale'
     (positive factors), 'log_a' (logarithms of decay rates), 'dt_bias' (step sizes before softplus) or 'correction'."""
     H, P = cfg.hidden_size, cfg.side_dim
+    around = () if cfg.scalar_norms else (H,)
     yield "embed", (cfg.vocab_size, H), "embed"
     if cfg.pairs is not None:
         yield "bigram", (cfg.pairs.buckets + 1, H), "embed"
@@ -503,7 +684,11 @@ def weight_shapes(cfg: MixedConfig) -> Iterator[Tuple[str, Tuple[int, ...], str]
         yield "side.embed", (cfg.vocab_size, cfg.num_layers * P), "embed"
     for i, layer in enumerate(cfg.layers):
         p, m = f"l{i}.", layer.mixer
-        yield p + "norm1", (H,), "norm"
+        yield p + "norm1", around, "norm"
+        if cfg.norm_both:
+            yield p + "norm1b", around, "norm"
+        if cfg.input_taps:
+            yield p + "canon1", (H, cfg.input_taps), "linear"
         if cfg.token_shift:
             yield p + "shift", (H,), "unit"
         if isinstance(m, Mamba1):
@@ -516,6 +701,22 @@ def weight_shapes(cfg: MixedConfig) -> Iterator[Tuple[str, Tuple[int, ...], str]
             yield p + "mix.A_log", (m.inner, m.state), "log_a"
             yield p + "mix.D", (m.inner,), "norm"
             vd = m.inner
+        elif isinstance(m, DeltaRule):
+            vd = m.heads * m.vdim
+            for name, rows in (("q", m.kv_heads * m.dim), ("k", m.kv_heads * m.dim), ("v", vd)):
+                yield f"{p}mix.{name}", (rows, H), "linear"
+                yield f"{p}mix.{name}.conv", (rows, m.conv), "linear"
+            yield p + "mix.g", (vd, H), "linear"
+            yield p + "mix.b", (m.heads, H), "linear"
+            yield p + "mix.a", (m.heads, H), "linear"
+            yield p + "mix.A_log", (m.heads,), "log_a"
+            yield p + "mix.dt_bias", (m.heads,), "dt_bias"
+            yield p + "mix.norm", (m.vdim,), "norm"
+        elif getattr(m, "q_rank", 0):
+            qd, vd = m.heads * (m.dim + (m.rot.dims if m.rot else 0)), m.heads * m.vdim
+            yield p + "mix.dq", (m.q_rank, H), "linear"
+            yield p + "mix.dq.norm", (m.q_rank,), "norm"
+            yield p + "mix.uq", (qd, m.q_rank), "linear"
         else:
             qd, vd = m.heads * m.dim, m.heads * m.vdim
             yield p + "mix.q", (qd, H), "linear"
@@ -532,12 +733,16 @@ def weight_shapes(cfg: MixedConfig) -> Iterator[Tuple[str, Tuple[int, ...], str]
                 yield p + "mix.vmix", (), "unit"
             if m.sink:
                 yield p + "mix.sink", (m.heads,), "bias"
+            if m.log_bias:
+                yield p + "mix.r1", (m.heads,), "scale"
+                yield p + "mix.r2", (m.heads,), "scale"
             if m.gate:
                 yield p + "mix.g", (m.heads if m.gate_by_head else vd, H), "linear"
         elif isinstance(m, LatentAttention):
-            yield p + "mix.dkv", (m.kv_rank, H), "linear"
-            yield p + "mix.dkv.norm", (m.kv_rank,), "norm"
-            yield p + "mix.uk", (qd, m.kv_rank), "linear"
+            if m.kv_from is None:
+                yield p + "mix.dkv", (m.kv_rank + (m.rot.dims if m.rot else 0), H), "linear"
+                yield p + "mix.dkv.norm", (m.kv_rank,), "norm"
+            yield p + "mix.uk", (m.heads * m.dim, m.kv_rank), "linear"
             yield p + "mix.uv", (vd, m.kv_rank), "linear"
         elif isinstance(m, HGRN2):
             yield p + "mix.f", (qd, H), "linear"
@@ -547,19 +752,24 @@ def weight_shapes(cfg: MixedConfig) -> Iterator[Tuple[str, Tuple[int, ...], str]
             yield p + "mix.norm", (m.vdim,), "norm"
         yield p + "mix.o", (H, vd), "linear"
         if layer.mlp is not None:
-            yield p + "norm2", (H,), "norm"
+            yield p + "norm2", around, "norm"
+            if cfg.norm_both:
+                yield p + "norm2b", around, "norm"
+            if cfg.input_taps:
+                yield p + "canon2", (H, cfg.input_taps), "linear"
         if isinstance(layer.mlp, MoE):
             f = layer.mlp
             for e, ff in [(f"e{j}", f.ff) for j in range(f.experts)] + ([("shared", f.shared_ff)] if f.shared_ff else []):
-                yield f"{p}mlp.{e}.gate", (ff, H), "linear"
+                if f.gated:
+                    yield f"{p}mlp.{e}.gate", (ff, H), "linear"
                 yield f"{p}mlp.{e}.up", (ff, H), "linear"
                 yield f"{p}mlp.{e}.down", (H, ff), "linear"
-            yield p + "mlp.router", (f.experts, H), "linear"
-            yield p + ("mlp.router.b" if f.router == "chosen" else "mlp.correction"), (f.experts,), "bias" if f.router == "chosen" else "correction"
+            yield p + "mlp.router", (f.experts + f.identity, H), "linear"
+            yield p + ("mlp.router.b" if f.router == "chosen" else "mlp.correction"), (f.experts + f.identity,), "bias" if f.router == "chosen" else "correction"
             if f.shared_gate:
                 yield p + "mlp.shared.sg", (1, H), "linear"
         elif layer.mlp is not None:
-            if isinstance(layer.mlp, ClippedGLU):
+            if isinstance(layer.mlp, (ClippedGLU, GatedMLP)):
                 yield p + "mlp.gate", (layer.mlp.ff, H), "linear"
             yield p + "mlp.up", (layer.mlp.ff, H), "linear"
             yield p + "mlp.down", (H, layer.mlp.ff), "linear"
@@ -571,7 +781,7 @@ def weight_shapes(cfg: MixedConfig) -> Iterator[Tuple[str, Tuple[int, ...], str]
             yield p + "side.gate", (P, H), "linear"
             yield p + "side.proj", (H, P), "linear"
             yield p + "side.norm", (H,), "norm"
-    yield "final.norm", (H,), "norm"
+    yield "final.norm", around, "norm"
     if not cfg.tied_head:
         yield "head", (cfg.vocab_size, H), "linear"
 
@@ -610,5 +820,5 @@ def random_weights(cfg: MixedConfig, *, seed: int = 0, dtype=torch.bfloat16, dev
     return get
 
 
-__all__ = ["MixedConfig", "MixedLayer", "LatentAttention", "HGRN2", "GroupedAttention", "Mamba1", "Rotary", "YarnScaling", "DenseMLP",
-           "ClippedGLU", "MoE", "TokenPairs", "weight_shapes", "random_weights"]
+__all__ = ["MixedConfig", "MixedLayer", "LatentAttention", "HGRN2", "GroupedAttention", "Mamba1", "DeltaRule", "Rotary", "YarnScaling", "DenseMLP",
+           "GatedMLP", "ClippedGLU", "MoE", "TokenPairs", "weight_shapes", "random_weights"]

@@ -673,11 +673,21 @@ def head_linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def latent_insert(x: torch.Tensor, norm_w: torch.Tensor, pool: torch.Tensor, r, eps: float, rank: Optional[int] = None) -> None:
-    """RMS-normed latent rows into the paged pool ``[pages, 16, rank_padded]``."""
-    N.check(N.lib().rf_latent_insert(C.c_void_p(x.data_ptr()), C.c_int64(x.stride(0)), C.c_void_p(norm_w.data_ptr()),
-                                     C.c_void_p(pool.data_ptr()), C.byref(r), x.shape[0], pool.shape[2], rank or pool.shape[2],
-                                     C.c_float(eps), dtype_code_any(x.dtype), _stream()), "rf_latent_insert")
+def latent_insert(x: Optional[torch.Tensor], norm_w: Optional[torch.Tensor], pool: Optional[torch.Tensor], r, eps: float, rank: Optional[int] = None,
+                  cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None, q: Optional[torch.Tensor] = None,
+                  q_norm: Optional[torch.Tensor] = None, q_rank: Optional[int] = None) -> None:
+    """RMS-normed latent rows into the paged pool ``[pages, 16, columns]``.  With ``cos`` / ``sin [positions, dims / 2]`` the rotated part that
+    lies behind the latent (``norm_w`` tells the latent's columns) is turned and cached too; ``q``: query latents, normalised in place."""
+    c = N.RfLatentInsert()
+    c.rows, c.n_rows, c.eps = r, (x if x is not None else q).shape[0], eps
+    if x is not None:
+        c.x, c.ldx, c.norm_w, c.pool, c.rank = x.data_ptr(), x.stride(0), norm_w.data_ptr(), pool.data_ptr(), norm_w.numel()
+        c.rank_true, c.rot_pad = rank or c.rank, pool.shape[2] - c.rank
+        if cos is not None:
+            c.rot, c.cos, c.sin = 2 * cos.shape[1], cos.data_ptr(), sin.data_ptr()
+    if q is not None:
+        c.q, c.ldq, c.q_norm, c.q_rank, c.q_rank_true = q.data_ptr(), q.stride(0), q_norm.data_ptr(), q_norm.numel(), q_rank or q_norm.numel()
+    N.check(N.lib().rf_latent_insert(C.byref(c), dtype_code_any((x if x is not None else q).dtype), _stream()), "rf_latent_insert")
 
 
 def latent_gather(pool: torch.Tensor, r, kv_start: torch.Tensor, kv_len: torch.Tensor, total: int, max_len: int) -> torch.Tensor:
@@ -689,13 +699,14 @@ def latent_gather(pool: torch.Tensor, r, kv_start: torch.Tensor, kv_len: torch.T
     return out
 
 
-def latent_attention(q: torch.Tensor, pool: torch.Tensor, r, *, window: int, scale: float, max_kv: int) -> torch.Tensor:
-    """Attention of ``q [rows, heads, rank]`` over the cached latent rows (keys and values both) -> ``[rows, heads, rank]``."""
+def latent_attention(q: torch.Tensor, pool: torch.Tensor, r, *, window: int, scale: float, max_kv: int, vrank: int = 0) -> torch.Tensor:
+    """Attention of ``q [rows, heads, rank]`` over the cached latent rows (keys and values both) -> ``[rows, heads, rank]``; ``vrank`` > 0:
+    the first this many columns are the values."""
     R, Hh, rank = q.shape
     assert q.is_contiguous() and pool.shape[2] == rank
-    o = torch.empty_like(q)
+    o = torch.empty((R, Hh, vrank or rank), dtype=q.dtype, device=q.device)
     a = N.RfLatentAttn()
-    a.q, a.o, a.pool, a.rows = q.data_ptr(), o.data_ptr(), pool.data_ptr(), r
+    a.q, a.o, a.pool, a.rows, a.vrank = q.data_ptr(), o.data_ptr(), pool.data_ptr(), r, vrank
     a.n_rows, a.heads, a.rank, a.window, a.max_kv, a.scale, a.dtype = R, Hh, rank, window, max_kv, scale, dtype_code_any(q.dtype)
     need = N.lib().rf_latent_attn_scratch_bytes(R, Hh, rank, max_kv)
     if need:

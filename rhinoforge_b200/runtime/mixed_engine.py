@@ -18,12 +18,12 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from .. import _native as N
-from ..models.mixed import HGRN2, ClippedGLU, GroupedAttention, LatentAttention, Mamba1, MixedConfig, MoE
+from ..models.mixed import HGRN2, ClippedGLU, DeltaRule, GatedMLP, GroupedAttention, LatentAttention, Mamba1, MixedConfig, MoE
 from ..ops import kernels as K
 from ..parallel.tp import TPContext
 from .engine import DecoderEngine, WeightGetter
 from .errors import RPUBackendError
-from .mixed_cache import MixedCache, head_layout, pad_to
+from .mixed_cache import MixedCache, delta_layout, head_layout, latent_layout, pad_to
 
 
 def _pad2(w: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
@@ -136,7 +136,9 @@ class MixedDecoderEngine(DecoderEngine):
                 wide[:, :, :cfg.side_dim] = side
                 side = wide
             self.side_table = self._plain(side.reshape(V, L * P))
-        self.final_norm = self._f32(g("final.norm"), H)
+        # norms with one weight for all coordinates are spread over the row
+        weight = lambda name: g(name).reshape(-1).expand(cfg.hidden_size) if cfg.scalar_norms else g(name)
+        self.final_norm = self._f32(weight("final.norm"), H)
         lm = self._linear(_pad2(self.embed if cfg.tied_head else g("head"), self.vocab_ld, H))
         self._rotations: Dict[object, tuple] = {}
         self._v_mixing = False                  # has a value-mixing layer been loaded already?
@@ -154,6 +156,7 @@ class MixedDecoderEngine(DecoderEngine):
             b = cfg.pairs
             sc.pair_table = self._plain(_pad2(g("bigram"), b.buckets + 1, H)).data_ptr()
             sc.pair_buckets, sc.pair_mul_prev, sc.pair_mul_cur = b.buckets, b.mul_prev, b.mul_cur
+        sc.input_taps = cfg.input_taps
         h = lib.rf_mixed_create(C.byref(sc))
         if h < 0:
             N.check(-1, "rf_mixed_create")
@@ -163,20 +166,30 @@ class MixedDecoderEngine(DecoderEngine):
             lw = N.RfMixedLayer()
             lw.heads = getattr(m, "heads", 0)
             # layer scales act on the normalised outputs: one factor with the norm's weight
-            norm = lambda name, scale: g(p + name).float() * g(p + scale).float() if cfg.layer_scale else g(p + name)
+            norm = lambda name, scale: g(p + name).float() * g(p + scale).float() if cfg.layer_scale else weight(p + name)
             lw.norm1 = self._f32(norm("norm1", "ls1"), H).data_ptr()
             if cfg.token_shift:
                 lw.shift = self._f32(g(p + "shift"), H).data_ptr()
-            load = {LatentAttention: self._load_latent, HGRN2: self._load_hgrn2, GroupedAttention: self._load_grouped, Mamba1: self._load_mamba1}
+            sublayers = 1 if layer.mlp is None else 2
+            if cfg.norm_both:
+                for n in range(sublayers):
+                    setattr(lw, f"norm{n + 1}b", self._f32(weight(f"{p}norm{n + 1}b"), H).data_ptr())
+            if cfg.input_taps:
+                for n in range(sublayers):
+                    taps = _pad2(g(f"{p}canon{n + 1}").t().float(), cfg.input_taps, H)
+                    lw.input_conv[n] = self._f32(taps, taps.numel()).data_ptr()
+            load = {DeltaRule: self._load_delta, LatentAttention: self._load_latent, HGRN2: self._load_hgrn2, GroupedAttention: self._load_grouped, Mamba1: self._load_mamba1}
             load[type(m)](lw, m, g, p + "mix.")
             lw.st = self.cache.layer_state(i)
             if layer.mlp is not None:
                 lw.norm2 = self._f32(norm("norm2", "ls2"), H).data_ptr()
             if isinstance(layer.mlp, MoE):
                 self._load_moe(lw, layer.mlp, g, p + "mlp.")
-            elif isinstance(layer.mlp, ClippedGLU):
+            elif isinstance(layer.mlp, (ClippedGLU, GatedMLP)):
                 f = layer.mlp
-                lw.inter, lw.act, lw.act_limit, lw.act_alpha = pad_to(f.ff, 8), 1, f.limit, f.alpha
+                lw.inter, lw.act = pad_to(f.ff, 8), 2
+                if isinstance(f, ClippedGLU):
+                    lw.act, lw.act_limit, lw.act_alpha = 1, f.limit, f.alpha
                 lw.w_up = self._linear(torch.cat([_pad2(g(f"{p}mlp.{x}"), lw.inter, H) for x in ("gate", "up")], 0), 2).data_ptr()
                 lw.w_down = self._linear(_pad2(g(p + "mlp.down"), H, lw.inter)).data_ptr()
             elif layer.mlp is not None:
@@ -191,25 +204,48 @@ class MixedDecoderEngine(DecoderEngine):
         torch.cuda.empty_cache()
 
     def _load_latent(self, lw, m: LatentAttention, g, p: str) -> None:
-        H, R = self.H, pad_to(m.kv_rank, 16)
-        big = max(m.dim, m.vdim)
+        H = self.H
+        R, P = latent_layout(m)
+        rot, plain = m.rot.dims if m.rot is not None else 0, pad_to(m.dim, 8)
+        key = plain + pad_to(rot, 8)                          # a head: plain dimensions, then rotated ones
+        big = max(key, m.vdim)
         # heads of the tcgen05 prefill attention; without one (fp32, very wide heads) every row attends in the latent space
         hd = next((x for x in (64, 128, 256) if big <= x), 0) if not self.fp32 and m.scale > 0 else 0
-        D, VD = hd or pad_to(m.dim, 8), hd or pad_to(m.vdim, 8)
+        D, VD = hd or key, hd or pad_to(m.vdim, 8)
         lw.mixer, lw.dim, lw.vdim, lw.vdim_true = 0, D, VD, m.vdim
         lw.rank, lw.rank_true, lw.window, lw.scale, lw.expand_hd = R, m.kv_rank, m.window or 0, m.scale, hd
-        q = _pad_heads(_pad2(g(p + "q"), m.heads * m.dim, H), m.heads, m.dim, D)
-        dkv = _pad2(g(p + "dkv"), R, H)
-        w_in = torch.cat((q, dkv), 0)
+        lw.plain, lw.rot, lw.rot_pad, lw.shares = plain, rot, P, int(m.kv_from is not None)
+        QR = lw.q_rank = pad_to(m.q_rank, 8)
+        q = g(p + ("uq" if QR else "q"))
+        q = _pad2(q, q.shape[0], QR or H).view(m.heads, m.dim + rot, QR or H)
+        heads = q.new_zeros((m.heads, D, QR or H))
+        heads[:, :m.dim], heads[:, plain:plain + rot] = q[:, :m.dim], q[:, m.dim:]
+        q = heads.view(m.heads * D, QR or H)
+        if QR:
+            lw.q_rank_true, lw.q_latent_norm, lw.w_uq = m.q_rank, self._f32(g(p + "dq.norm"), QR).data_ptr(), self._linear(q).data_ptr()
+            q = _pad2(g(p + "dq"), QR, H)
+        parts = [q]
+        if m.kv_from is None:
+            dkv = g(p + "dkv")
+            parts += [_pad2(dkv[:m.kv_rank], R, H)] + ([_pad2(dkv[m.kv_rank:], P, H)] if rot else [])
+            lw.latent_norm = self._f32(g(p + "dkv.norm"), R).data_ptr()
+        w_in = torch.cat(parts, 0)
         lw.in_dim = w_in.shape[0]
         lw.w_in = self._linear(w_in).data_ptr()
-        lw.latent_norm = self._f32(g(p + "dkv.norm"), R).data_ptr()
-        uk = _pad_heads(_pad2(g(p + "uk"), m.heads * m.dim, R), m.heads, m.dim, D)
+        if rot:
+            cos, sin = self._rotation(m.rot)
+            lw.cos, lw.sin = cos.data_ptr(), sin.data_ptr()
+        uk = _pad_heads(_pad2(g(p + "uk"), m.heads * m.dim, R), m.heads, m.dim, plain)
         uv = _pad_heads(_pad2(g(p + "uv"), m.heads * m.vdim, R), m.heads, m.vdim, VD)
-        lw.w_absorb = self._plain(uk.view(m.heads, D, R).transpose(1, 2)).data_ptr()
+        lw.w_absorb = self._plain(uk.view(m.heads, plain, R).transpose(1, 2)).data_ptr()
         lw.w_unabsorb = self._plain(uv).data_ptr()
         if hd:
-            lw.w_expand = self._linear(torch.cat((uk, uv), 0)).data_ptr()
+            # keys of a head are a map of the latent and a copy of the rotated part, values a map of the latent
+            expand = uk.new_zeros((2, m.heads, hd, R + P))
+            expand[0, :, :plain, :R], expand[1, :, :, :R] = uk.view(m.heads, plain, R), uv.view(m.heads, hd, R)
+            for i in range(rot):
+                expand[0, :, plain + i, R + i] = 1.0
+            lw.w_expand = self._linear(expand.view(2 * m.heads * hd, R + P)).data_ptr()
         o = g(p + "o")
         o = _pad_heads(o.t().contiguous(), m.heads, m.vdim, VD).t()
         lw.w_o, lw.out_dim = self._linear(_pad2(o, H, m.heads * VD)).data_ptr(), m.heads * VD
@@ -242,6 +278,9 @@ class MixedDecoderEngine(DecoderEngine):
             lw.sink = self._f32(g(p + "sink") if m.sink else torch.zeros(m.heads), m.heads).data_ptr()
         if m.distance_bias:
             lw.slopes = self._f32(m.slopes(), m.heads).data_ptr()
+        if m.log_bias:
+            lw.slopes, lw.rates = self._f32(g(p + "r1"), m.heads).data_ptr(), self._f32(g(p + "r2"), m.heads).data_ptr()
+        lw.growth, lw.growth_every = m.growth, m.growth_every
         if m.conv:
             taps = torch.cat([_pad_heads(g(f"{p}{x}.conv").float(), n, d, hd)
                               for x, n, d in (("q", m.heads, m.dim), ("k", m.kv_heads, m.dim), ("v", m.kv_heads, m.vdim))], 0)
@@ -255,6 +294,22 @@ class MixedDecoderEngine(DecoderEngine):
             self._v_mixing = True
         o = _pad_heads(g(p + "o").t().contiguous(), m.heads, m.vdim, hd).t()
         lw.w_o, lw.out_dim = self._linear(_pad2(o, H, m.heads * hd)).data_ptr(), m.heads * hd
+
+    def _load_delta(self, lw, m: DeltaRule, g, p: str) -> None:
+        H = self.H
+        D, V = delta_layout(m, self.dtype)
+        lw.mixer, lw.dim, lw.vdim, lw.dim_true, lw.vdim_true, lw.kv_heads, lw.taps = 4, D, V, m.dim, m.vdim, m.kv_heads, m.conv
+        parts = (("q", m.kv_heads, m.dim, D), ("k", m.kv_heads, m.dim, D), ("v", m.heads, m.vdim, V), ("g", m.heads, m.vdim, V))
+        w_in = [_pad_heads(_pad2(g(p + x), n * true, H), n, true, padded) for x, n, true, padded in parts]
+        w_in += [_pad2(g(p + x), pad_to(m.heads, 8), H) for x in ("b", "a")]
+        w_in = torch.cat(w_in, 0)
+        lw.w_in, lw.in_dim = self._linear(w_in).data_ptr(), w_in.shape[0]
+        taps = torch.cat([_pad_heads(g(f"{p}{x}.conv").float(), n, true, padded) for x, n, true, padded in parts[:3]], 0)
+        lw.conv_w = self._f32(taps.t().contiguous(), taps.numel()).data_ptr()
+        lw.rate = self._f32(g(p + "A_log").double().exp(), m.heads).data_ptr()
+        lw.dt_bias, lw.head_norm = self._f32(g(p + "dt_bias"), m.heads).data_ptr(), self._f32(g(p + "norm"), V).data_ptr()
+        o = _pad_heads(g(p + "o").t().contiguous(), m.heads, m.vdim, V).t()
+        lw.w_o, lw.out_dim = self._linear(_pad2(o, H, m.heads * V)).data_ptr(), m.heads * V
 
     def _load_mamba1(self, lw, m: Mamba1, g, p: str) -> None:
         H, I, S, R = self.H, pad_to(m.inner, 8), pad_to(m.state, 8), pad_to(m.dt_rank, 8)
@@ -281,24 +336,28 @@ class MixedDecoderEngine(DecoderEngine):
         B = I if self.fp32 else pad_to(f.ff, 128)
         lw.inter, lw.bank_inter, lw.act = I, B, 0
         lw.experts, lw.top, lw.groups, lw.keep = f.experts, f.top, f.groups, f.keep
-        lw.score_fn, lw.norm_topk, lw.route_scale = {"corrected": 1, "chosen": 2}[f.router], 1, 1.0
+        lw.score_fn, lw.norm_topk, lw.route_scale = {"corrected": 1, "chosen": 2}[f.router], int(f.renormalise), 1.0
+        lw.identity = f.identity
         if f.limit is not None:
             lw.act, lw.act_limit, lw.act_alpha, lw.shared_limit = 1, f.limit, f.alpha, f.shared_limit or 0.0
-        up = torch.zeros((2, f.experts, B, H), dtype=self.dtype, device=self.device)
+        if not f.gated:
+            lw.act = 3
+        names = ("gate", "up") if f.gated else ("up",)
+        up = torch.zeros((len(names), f.experts, B, H), dtype=self.dtype, device=self.device)
         down = torch.zeros((f.experts, H, B), dtype=self.dtype, device=self.device)
         for e in range(f.experts):
-            for i, name in enumerate(("gate", "up")):
+            for i, name in enumerate(names):
                 w = g(f"{p}e{e}.{name}")
                 up[i, e, :f.ff, :w.shape[1]] = w
             w = g(f"{p}e{e}.down")
             down[e, :w.shape[0], :f.ff] = w
-        lw.w_up = self._linear(up.view(2 * f.experts * B, H), 2).data_ptr()
+        lw.w_up = self._linear(up.view(len(names) * f.experts * B, H), len(names)).data_ptr()
         lw.w_down = self._linear(down.view(f.experts * H, B) if self.fp32 else down.transpose(0, 1).reshape(H, f.experts * B)).data_ptr()
-        router = _pad2(g(p + "router"), f.experts, H)
+        router = _pad2(g(p + "router"), f.experts + f.identity, H)
         if f.shared_gate:
             router, lw.shared_gate = torch.cat((router, _pad2(g(p + "shared.sg"), 1, H)), 0), 1
         lw.router = self._plain(router).data_ptr()
-        lw.correction = self._f32(g(p + ("router.b" if f.router == "chosen" else "correction")), f.experts).data_ptr()
+        lw.correction = self._f32(g(p + ("router.b" if f.router == "chosen" else "correction")), f.experts + f.identity).data_ptr()
         if f.shared_ff:
             S = lw.shared_inter = pad_to(f.shared_ff, 8)
             gate_up = torch.cat((_pad2(g(p + "shared.gate"), S, H), _pad2(g(p + "shared.up"), S, H)), 0)

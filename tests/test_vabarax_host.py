@@ -205,10 +205,11 @@ def test_native_argument_blocks_have_the_same_size_on_both_sides():
     from rhinoforge_b200 import _native as N
     if not N.available():
         pytest.skip("native library is not built")
-    sizes = (C.c_int32 * 15)()
+    sizes = (C.c_int32 * 18)()
     N.lib().rf_mixed_struct_sizes(sizes)
     ours = (N.RfMixedConfig, N.RfMixedLayer, N.RfMixedForward, N.RfRows, N.RfStreamNorm, N.RfLatentAttn, N.RfHgrn2, N.RfHeadLinear,
-            N.RfMixedState, N.RfAttn, N.RfQkvInsert, N.RfConvSilu, N.RfMamba1, N.RfMoeRouter, N.RfMoeExperts)
+            N.RfMixedState, N.RfAttn, N.RfQkvInsert, N.RfConvSilu, N.RfMamba1, N.RfMoeRouter, N.RfMoeExperts, N.RfLatentInsert,
+            N.RfHeadRotate, N.RfDelta)
     assert list(sizes) == [C.sizeof(x) for x in ours]
 
 
