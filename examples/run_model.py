@@ -26,13 +26,14 @@ HERE = Path(__file__).resolve().parent
 DEFAULT_CONFIG = HERE / "configs" / "qwen3_0_6b_full.toml"
 
 TARGETS = {name: f"{name}.py" for name in
-           ("causal_lm", "dinov3", "hy_embodied", "kuzupel", "pi05", "qwen3_5_text", "qwen3_vl", "rhinovla", "vabarax", "wall_oss", "zulopel")}
+           ("causal_lm", "dinov3", "hy_embodied", "kuzupel", "pi05", "qwen3_5_text", "qwen3_vl", "rhinovla", "vabarax", "vasosun", "wall_oss", "zulopel")}
 _PREFILL = ("chunk_size", "padding_rows", "padding_budget")
 EXECUTION_SUPPORT = {
     "causal_lm": {"prefill": _PREFILL},
     "dinov3": {"vision": ("chunk_size",)},
     "hy_embodied": {},
     "kuzupel": {"prefill": _PREFILL},
+    "vasosun": {"prefill": _PREFILL},
     "pi05": {"prefill": _PREFILL, "vision": ("chunk_size",), "action": ("chunk_size",)},
     "qwen3_5_text": {"prefill": _PREFILL},
     "qwen3_vl": {"prefill": _PREFILL, "vision": ("chunk_size",)},

@@ -476,7 +476,17 @@ static int delta(MixedStack& s, const RfMixedLayer& w, const RfMixedForward& f, 
   rc = rf_conv_silu(&cv, st);
   if (rc) return rc;
   a.x = cv.y; a.ldx = CH;
-  return rf_delta_recurrent(&a, st);
+  const int n_rec = rf_delta_chunked_supported(w.dim, w.vdim, c.dtype) ? f.short_seqs : f.rows.num_seqs;
+  if (n_rec > 0) {
+    a.rows = sub_rows(f.rows, 0, n_rec);
+    rc = rf_delta_recurrent(&a, st);
+    if (rc) return rc;
+  }
+  if (n_rec < f.rows.num_seqs) {
+    a.rows = sub_rows(f.rows, n_rec, f.rows.num_seqs - n_rec);
+    rc = rf_delta_chunked(&a, f.short_rows, T - f.short_rows, st);
+  }
+  return rc;
 }
 
 // The experts' results stay where they are, one row per pick; the next stream step adds them up (see RfStreamNorm.y_slots).
@@ -589,7 +599,7 @@ static int forward(MixedStack& s, const RfMixedForward& f, cudaStream_t st) {
     cur = nxt;
     pend = {};
     if (!conv_w) return rf_stream_norm(&a, st);
-    if (f.decode && !s.fp32()) {
+    if (f.decode && !s.fp32() && H <= 8192) {
       a.conv_w = conv_w; a.conv_state = conv_state; a.conv_taps = c.input_taps;
       return rf_stream_norm(&a, st);
     }

@@ -487,6 +487,10 @@ typedef struct RfDelta {
   const float* conv_w; void* conv_state; int32_t taps;
 } RfDelta;
 int rf_delta_recurrent(const RfDelta* a, rf_stream_t stream);
+// Same contract, 64 tokens at a time (prefill-sized portions; 16-bit activations, dim 64 / 128, vdim a multiple of 32).  The
+// sequences' rows are [row0, row0 + rows).
+int rf_delta_chunked(const RfDelta* a, int row0, int rows, rf_stream_t stream);
+int rf_delta_chunked_supported(int dim, int vdim, int dtype);
 
 // HGRN2 linear attention (what a gate takes from the state it gives to the new value), over packed input rows [q | f | v]:
 //   q = silu(q), f = lower + (1 - lower) * sigmoid(f + f_bias), S = diag(f) S + (1 - f) v^T, o = S^T q,

@@ -418,17 +418,18 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, *, Hq: int, Hkv: int, 
                       seg_k: Optional[torch.Tensor] = None, scale: float = 0.0,
                       status: Optional[torch.Tensor] = None, max_kv_len: int = 0, slot: Optional[torch.Tensor] = None, chunk: int = 0,
                       sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_by_head: bool = False,
-                      keep_first: int = 0, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      keep_first: int = 0, slopes: Optional[torch.Tensor] = None, rates: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Flash-style attention over ``q`` rows [tokens, Hq*hd]; KV from the paged pool or from
     contiguous ``k``/``v`` [rows, Hkv*hd] (may be column slices of a packed qkv buffer).
     ``max_kv_len``: a host-side bound on ``kv_len`` (0: unknown); short contiguous problems (at most 64 query rows per
     sequence over at most 512 keys, heads of 64 / 128, causal / window masks only) then take the low-latency kernel.
     Paged form: ``slot`` names every sequence's page-table row, ``chunk`` limits every position to its own chunk, ``sink`` ``[Hq]``
     adds ``exp(sink)`` to the softmax denominators, the result is multiplied by ``sigmoid(gate)`` (``gate_by_head``: ``[rows, Hq]``),
-    the first ``keep_first`` positions stay visible behind a window or chunk, ``slopes`` ``[Hq]`` times the distance is taken off the
-    scores."""
+    the first ``keep_first`` positions stay visible behind a window or chunk, ``slopes`` ``[Hq]`` times the distance, or with ``rates``
+    ``[Hq]`` times ``ln(1 + rate * distance)``, is taken off the scores."""
     a = N.RfAttn()
     a.gate_by_head, a.keep_first, a.slopes = int(gate_by_head), keep_first, _ptr(slopes)
+    a.rates = _ptr(rates)
     a.q, a.ldq, a.out, a.ldo = q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0)
     a.q_rows_total = q.shape[0]
     a.num_seqs, a.Hq, a.Hkv, a.hd = q_len.numel(), Hq, Hkv, hd
@@ -481,12 +482,13 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, *, Hq: int, Hkv: int, h
 def attention_rows(q: torch.Tensor, r, k_pool: torch.Tensor, v_pool: torch.Tensor, *, Hq: int, Hkv: int, hd: int, scale: float, max_kv: int,
                    chunk: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, split: bool = True,
                    tensor_core: bool = True, window: int = 0, gate_by_head: bool = False, keep_first: int = 0,
-                   slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   slopes: Optional[torch.Tensor] = None, rates: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Every row of ``q [rows, Hq * hd]`` over the cached keys of its sequence up to its own position (``r``: :func:`rows`), with the
     options of :func:`attention_prefill`.  ``tensor_core=False``: the fp32 kernel for any head size and dtype."""
     out = torch.empty((q.shape[0], Hq * hd), dtype=q.dtype, device=q.device)
     a = N.RfAttn()
     a.window, a.gate_by_head, a.keep_first, a.slopes = window, int(gate_by_head), keep_first, _ptr(slopes)
+    a.rates = _ptr(rates)
     a.q, a.ldq, a.out, a.ldo, a.q_rows_total, a.num_seqs = q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), q.shape[0], q.shape[0]
     a.Hq, a.Hkv, a.hd, a.scale, a.max_kv_len, a.chunk, a.sink = Hq, Hkv, hd, scale, max_kv, chunk, _ptr(sink)
     a.k_pool, a.v_pool, a.pool_pages = k_pool.data_ptr(), v_pool.data_ptr(), k_pool.shape[0]
@@ -615,12 +617,14 @@ def stream_norm(x: Optional[torch.Tensor], r, *, dtype: torch.dtype, eps: float,
                 table: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None,
                 y_norm_w: Optional[torch.Tensor] = None, shift: Optional[torch.Tensor] = None,
                 shift_state: Optional[torch.Tensor] = None, dim: Optional[int] = None, cast: bool = False, embed_scale: float = 1.0,
-                y_slots: Optional[torch.Tensor] = None, y_mult: float = 1.0, pairs: Optional[tuple] = None):
+                y_slots: Optional[torch.Tensor] = None, y_mult: float = 1.0, pairs: Optional[tuple] = None, y_self: Optional[tuple] = None,
+                conv: Optional[tuple] = None):
     """One step of an fp32 residual stream: add the outstanding sublayer output ``y`` (RMS-normed with ``y_norm_w``), RMSNorm
     with ``norm_w``, mix with the previous token's normalised row (``shift``, state per slot).  Without ``x`` the stream starts
     from ``table[ids] * embed_scale``.  ``y_slots [rows, picks]``: the outstanding output is the sum of these rows of ``y`` (negative:
     none).  ``y_mult``: factor of the outstanding output.  ``pairs = (table2 [buckets + 1, H], last_token [slots], mul_prev, mul_cur)``:
-    the row of (previous token, token) is added to the embedding.  Returns ``(x_out fp32, h or None, x in dtype or None)``."""
+    the row of (previous token, token) is added to the embedding.  ``y_self = (rows, weights)``: weight times row is part of the picked
+    sum.  ``conv = (w [taps, H], state [slots, taps - 1, H])``: input convolution of decode rows behind the norm.  Returns ``(x_out fp32, h or None, x in dtype or None)``."""
     H = (x if x is not None else table).shape[1]
     n = x.shape[0] if x is not None else ids.numel()
     dev = (x if x is not None else table).device
@@ -632,6 +636,10 @@ def stream_norm(x: Optional[torch.Tensor], r, *, dtype: torch.dtype, eps: float,
     a.x_out, a.x_cast, a.norm_w, a.out, a.shift, a.shift_state = _ptr(x_out), _ptr(xc), _ptr(norm_w), _ptr(h), _ptr(shift), _ptr(shift_state)
     a.rows, a.n_rows, a.H, a.dim, a.eps, a.dtype = r, n, H, dim or H, eps, dtype_code_any(dtype)
     a.embed_scale, a.y_slots, a.y_picks, a.y_mult = embed_scale, _i32(y_slots), 0 if y_slots is None else y_slots.shape[1], y_mult
+    if y_self is not None:
+        a.y_self, a.y_self_w = y_self[0].data_ptr(), y_self[1].data_ptr()
+    if conv is not None:
+        a.conv_w, a.conv_state, a.conv_taps = conv[0].data_ptr(), _ptr(conv[1]), conv[0].shape[0]
     if pairs is not None:
         a.table2, a.last_token, a.mul_prev, a.mul_cur, a.buckets = pairs[0].data_ptr(), _i32(pairs[1]), pairs[2], pairs[3], pairs[0].shape[0] - 1
     N.check(N.lib().rf_stream_norm(C.byref(a), _stream()), "rf_stream_norm")
@@ -735,18 +743,19 @@ def qkv_insert(qkv: torch.Tensor, r, k_pool: torch.Tensor, v_pool: torch.Tensor,
                dim: Optional[int] = None, vdim: Optional[int] = None, q_norm: Optional[torch.Tensor] = None,
                k_norm: Optional[torch.Tensor] = None, cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None,
                v_first: Optional[torch.Tensor] = None, v_role: str = "none", v_lambda: float = 0.0, norm_all: bool = False,
-               conv_w: Optional[torch.Tensor] = None, conv_state: Optional[torch.Tensor] = None, max_q_len: int = 1) -> torch.Tensor:
+               conv_w: Optional[torch.Tensor] = None, conv_state: Optional[torch.Tensor] = None, max_q_len: int = 1,
+               growth: float = 0.0, growth_every: int = 0) -> torch.Tensor:
     """Per-head norms, rotation, value mixing and page insertion of packed rows ``[q | k | v]`` (heads of ``hd`` values, ``dim`` /
     ``vdim`` of them used); queries are replaced in place, keys and values go to the pools ``[pages, kv_heads, 16, hd]``.
     ``norm_all``: one norm over all query heads (weight ``[heads, hd]``) and one over all key heads.  ``conv_w [taps, columns]``: causal
     convolution ahead of the norms with carried rows in ``conv_state [slots, taps - 1, columns]``.  Returns the queries (a tensor of
-    their own with the convolution)."""
+    their own with the convolution).  ``growth_every`` > 0: queries grow by ``growth`` times a logarithm of their position."""
     a = N.RfQkvInsert()
     q = qkv[:, :heads * hd]
     if conv_w is not None:
         q = torch.empty((qkv.shape[0], heads * hd), dtype=qkv.dtype, device=qkv.device)
         a.conv_w, a.conv_state, a.q_out, a.taps, a.max_q_len = conv_w.data_ptr(), _ptr(conv_state), q.data_ptr(), conv_w.shape[0], max_q_len
-    a.norm_all = int(norm_all)
+    a.norm_all, a.growth, a.growth_every = int(norm_all), growth, growth_every
     a.qkv, a.ld, a.k_off, a.v_off = qkv.data_ptr(), qkv.stride(0), heads * hd, (heads + kv_heads) * hd
     a.q_norm, a.k_norm, a.cos, a.sin, a.v_first = _ptr(q_norm), _ptr(k_norm), _ptr(cos), _ptr(sin), _ptr(v_first)
     a.k_pool, a.v_pool, a.rows, a.n_rows = k_pool.data_ptr(), v_pool.data_ptr(), r, qkv.shape[0]
@@ -757,14 +766,51 @@ def qkv_insert(qkv: torch.Tensor, r, k_pool: torch.Tensor, v_pool: torch.Tensor,
     return q
 
 
-def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor], r, *, max_q_len: int = 1) -> torch.Tensor:
+def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor], r, *, max_q_len: int = 1,
+              add: bool = False, ring: bool = False) -> torch.Tensor:
     """Causal convolution per channel and silu over packed rows; ``w`` fp32 ``[taps, channels]``, ``state [slots, taps - 1, channels]``
-    holds the last inputs and is replaced."""
+    holds the last inputs and is replaced.  ``add``: the input plus the convolution, no silu; ``ring``: ``state [slots, taps, channels]`` by
+    position."""
     y = torch.empty((x.shape[0], w.shape[1]), dtype=x.dtype, device=x.device)
     a = N.RfConvSilu()
     a.x, a.ldx, a.y, a.ldy, a.w, a.bias, a.state = x.data_ptr(), x.stride(0), y.data_ptr(), y.stride(0), w.data_ptr(), _ptr(bias), _ptr(state)
     a.rows, a.max_q_len, a.channels, a.taps, a.dtype = r, max_q_len, w.shape[1], w.shape[0], dtype_code_any(x.dtype)
+    a.add, a.ring = int(add), int(ring)
     N.check(N.lib().rf_conv_silu(C.byref(a), _stream()), "rf_conv_silu")
+    return y
+
+
+def delta_rule(x: torch.Tensor, b: torch.Tensor, a: torch.Tensor, gate: torch.Tensor, rate: torch.Tensor, dt_bias: torch.Tensor, norm_w: torch.Tensor,
+               state: torch.Tensor, r, *, kv_heads: int, eps: float, dim: Optional[int] = None, vdim: Optional[int] = None,
+               conv: Optional[tuple] = None, chunked: bool = False) -> torch.Tensor:
+    """Gated delta rule over packed rows ``x = [q | k | v]`` with the fp32 ``state [slots, heads, dim, vdim]`` updated in place, output norm
+    and gate included.  ``dim`` / ``vdim``: true sizes of padded heads.  ``conv = (w [taps, channels], ring [slots, taps, channels])``: ``x`` are
+    projections of decode rows and the short convolution runs inside.  ``chunked``: 64 tokens at a time on the tensor cores."""
+    _, Hh, D, V = state.shape
+    out = torch.empty((x.shape[0], Hh * V), dtype=x.dtype, device=x.device)
+    p = N.RfDelta()
+    p.x, p.ldx, p.b, p.a, p.ld_ba, p.gate, p.ldg = x.data_ptr(), x.stride(0), b.data_ptr(), a.data_ptr(), b.stride(0), gate.data_ptr(), gate.stride(0)
+    p.rate, p.dt_bias, p.norm_w, p.state, p.out = (t.data_ptr() for t in (rate, dt_bias, norm_w, state, out))
+    p.ldo = Hh * V
+    p.rows, p.heads, p.kv_heads, p.dim, p.dim_true, p.vdim, p.vdim_true, p.eps, p.dtype = r, Hh, kv_heads, D, dim or D, V, vdim or V, eps, dtype_code_any(x.dtype)
+    if conv is not None:
+        p.conv_w, p.conv_state, p.taps = conv[0].data_ptr(), conv[1].data_ptr(), conv[0].shape[0]
+    if chunked:
+        N.check(N.lib().rf_delta_chunked(C.byref(p), 0, x.shape[0], _stream()), "rf_delta_chunked")
+    else:
+        N.check(N.lib().rf_delta_recurrent(C.byref(p), _stream()), "rf_delta_recurrent")
+    return out
+
+
+def head_rotate(x: torch.Tensor, pos: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Rotation of ``x [rows, heads, dims]`` (a view whose last dim is contiguous and padded in memory to a multiple of 8) in neighbouring
+    pairs, tables ``[positions, dims / 2]``; in place without ``out``."""
+    y = x if out is None else out
+    a = N.RfHeadRotate()
+    a.x, a.ldx, a.xs, a.y, a.ldy, a.ys = x.data_ptr(), x.stride(0), x.stride(1), y.data_ptr(), y.stride(0), y.stride(1)
+    a.pos, a.cos, a.sin, a.rows, a.heads, a.dims = _i32(pos), cos.data_ptr(), sin.data_ptr(), x.shape[0], x.shape[1], 2 * cos.shape[1]
+    a.dims_pad = (a.dims + 7) // 8 * 8
+    N.check(N.lib().rf_head_rotate(C.byref(a), dtype_code_any(x.dtype), _stream()), "rf_head_rotate")
     return y
 
 
@@ -787,12 +833,13 @@ def mamba1(x: torch.Tensor, z: torch.Tensor, bc: torch.Tensor, a2: torch.Tensor,
 # ----------------------------------------------------------------------------- mixture of experts
 class RoutedBatch:
     """Router of one batch and everything its expert GEMMs need (:func:`moe_router`).  ``score_fn="chosen"``: ``correction`` is a bias
-    of the logits and the weights are the softmax over the chosen ones; ``shared_gate``: the last row of ``w`` gives the logit of the
+    of the logits and the weights are the softmax over the chosen ones; ``identity``: the last this many experts return their input,
+    ``self_w`` are their weights by token; ``shared_gate``: the last row of ``w`` gives the logit of the
     shared expert's sigmoid weight."""
 
     def __init__(self, x: torch.Tensor, w: torch.Tensor, k: int, *, correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1,
                  score_fn: str = "softmax", norm_topk: bool = True, scale: float = 1.0, tile_rows: int = 16, shared: bool = False,
-                 scatter: bool = True, shared_gate: bool = False):
+                 scatter: bool = True, shared_gate: bool = False, identity: int = 0):
         T, E = x.shape[0], w.shape[0] - int(shared_gate)
         i32 = lambda *sh: torch.zeros(sh, dtype=torch.int32, device=x.device)
         self.x, self.w, self.correction, self.tile_rows, self.k = x, w, correction, tile_rows, k
@@ -809,7 +856,9 @@ class RoutedBatch:
             self.ids, self.weights, self.rank, self.counters, self.start, self.tiles, self.slot_of, self.token_of_slot, self.slot_w))
         a.rows, a.experts, a.width, a.k, a.groups, a.keep = T, E, w.shape[1], k, groups, keep
         a.score_fn, a.norm_topk, a.scale = {"sigmoid": 0, "softmax": 1, "chosen": 2}[score_fn], int(norm_topk), scale
-        a.shared_gate = int(shared_gate)
+        a.shared_gate, a.identity = int(shared_gate), identity
+        self.self_w = torch.zeros(T, dtype=torch.float32, device=x.device)
+        a.self_w = self.self_w.data_ptr()
         a.tile_rows, a.slot_ld, a.has_shared, a.shared_tiles, a.scatter = tile_rows, k + shared, int(shared), int(shared and scatter), int(scatter)
         a.dtype, a.logits = dtype_code_any(x.dtype), self.logits.data_ptr()
 
@@ -831,9 +880,11 @@ def moe_router(x: torch.Tensor, w: torch.Tensor, k: int, **kw) -> RoutedBatch:
 
 def moe_experts(b: RoutedBatch, x: torch.Tensor, bank: torch.Tensor, *, n: int, k: int, experts: int, expert_pad: int = 0, dual: bool = False,
                 gathered: bool = True, weighted: bool = False, shared: Optional[torch.Tensor] = None, shared_n: int = 0, shared_k: int = 0,
-                out_cols: int = 0, act: str = "silu_mul", limit: float = 0.0, alpha: float = 0.0, shared_limit: float = 0.0) -> torch.Tensor:
+                out_cols: int = 0, act: str = "silu_mul", limit: float = 0.0, alpha: float = 0.0, shared_limit: float = 0.0,
+                stacked: bool = False) -> torch.Tensor:
     """Expert GEMMs of few rows over the tile list of a routed batch; ``bank`` (and ``shared``) as the mixed engine packs them,
-    ``expert_pad`` the padded expert width inside 16-bit banks."""
+    ``expert_pad`` the padded expert width inside 16-bit banks; ``stacked``: a bank of single-operand up projections (experts along the
+    rows)."""
     cols = max(out_cols, n, shared_n)
     out = torch.zeros((b.slot_w.numel(), cols), dtype=x.dtype, device=x.device)
     a = N.RfMoeExperts()
@@ -844,6 +895,8 @@ def moe_experts(b: RoutedBatch, x: torch.Tensor, bank: torch.Tensor, *, n: int, 
     if dual:
         a.bank_section_row_tiles, a.bank_kb_total, a.rt_per_expert = experts * expert_pad // 128, up(k, 64), expert_pad // 128
         a.shared_section_row_tiles, a.shared_kb_total = up(shared_n, 128), up(shared_k, 64)
+    elif stacked:
+        a.bank_kb_total, a.rt_per_expert = up(k, 64), expert_pad // 128
     else:
         a.bank_kb_total, a.kb_per_expert, a.shared_kb_total = experts * expert_pad // 64, expert_pad // 64, up(shared_k, 64)
     a.dtype = dtype_code_any(x.dtype)
