@@ -29,12 +29,13 @@ def parse_args(argv=None):
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="decode", choices=["decode", "pi05", "qwen3vl", "vabarax", "zulopel", "kuzupel"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "pi05", "qwen3vl", "vabarax", "zulopel", "kuzupel", "vasosun"],
                     help="decode: causal-LM decode throughput (headline); pi05: action-chunk latency; "
                          "qwen3vl: multimodal prefill + decode; vabarax: latent-attention / HGRN2 decoder, zulopel: chunked "
                          "attention / selective-scan decoder with routed experts, each beside the hybrid K/V + "
                          "Gated-DeltaNet decoder at equal size; kuzupel: window-attention decoder with clipped feed-forwards, "
-                         "beside a Zulopel decoder of attention layers")
+                         "beside a Zulopel decoder of attention layers; vasosun: delta-rule / window / latent-attention decoder, "
+                         "beside a Zulopel decoder of scan and attention layers")
     ap.add_argument("--model", default="qwen3-8b")
     ap.add_argument("--batch", type=int, default=64)
     ap.add_argument("--prompt-len", type=int, default=1024)
@@ -561,6 +562,14 @@ KUZUPEL_SIZES = {          # width, heads (of 128), K/V heads, window of the bia
 }
 
 
+VASOSUN_SIZES = {          # width, heads (of 128), K/V heads, window, latent, query latent, rotated part, dense feed-forward, experts, identities, top,
+                           # expert width, layers (a delta-rule, a window and two latent layers in four, the second over the first one's cache)
+    "16e": (2048, 16, 4, 512, 512, 768, 64, 5632, 16, 4, 2, 1536, 16),
+    "32e": (3072, 24, 6, 512, 512, 1024, 64, 8192, 32, 8, 4, 1536, 16),
+    "64e": (4096, 32, 8, 512, 512, 1536, 64, 11008, 64, 16, 6, 2112, 8),
+}
+
+
 def _serve(eng, vocab: int, batches, prompt_len: int, steps: int, warmup: int, total_prompts: int):
     """Device-timed prefill of ``total_prompts`` prompts and decode steps at every batch size of one engine."""
     import torch
@@ -659,6 +668,30 @@ def run_kuzupel(args) -> dict:
     return _beside(args, "kuzupel", "Kuzupel 64-expert", entries, {k: dict(zip(keys, v)) for k, v in KUZUPEL_SIZES.items()})
 
 
+def run_vasosun(args) -> dict:
+    """The Vasosun design beside a Zulopel decoder with the same width, heads and experts (gated ones of two thirds of the width have
+    the same parameters; a dense feed-forward is a mixture of one expert there), a scan for the delta rule and chunked attention for
+    the three attention layers in four; see :func:`_beside`."""
+    from rhinoforge_b200.models.mixed import (DeltaRule, GatedMLP, GroupedAttention, LatentAttention, Mamba1, MixedConfig, MixedLayer, MoE, Rotary,
+                                              TokenPairs, YarnScaling)
+    entries = {}
+    for name, (H, heads, kv, near, rank, q_rank, turn, dense, experts, identity, top, ff, layers) in VASOSUN_SIZES.items():
+        rot, moe = Rotary(turn, 1e6, YarnScaling(8.0, 8192, 32.0, 1.0)), MoE(experts, top, ff, gated=False, identity=identity, renormalise=False)
+        latent = lambda i, of=None: LatentAttention(heads, 128, 128, rank, (128 + turn) ** -0.5, q_rank=q_rank, rot=rot, kv_from=of)
+        quad = lambda i: (MixedLayer(DeltaRule(heads, heads // 2, 128, 128, 4), GatedMLP(dense)),
+                          MixedLayer(GroupedAttention(heads, kv, 128, 128, 128 ** -0.5, qk_norm=False, sink=False, gate=False, log_bias=True, window=near,
+                                                      growth=0.1, growth_every=8192), moe),
+                          MixedLayer(latent(i), moe), MixedLayer(latent(i, i + 2), moe))
+        head, wide = (heads, kv, 128, 128, 128 ** -0.5), MoE(experts, top, 2 * ff // 3, 4, 4)
+        like = (MixedLayer(Mamba1(2 * H, 16, H // 16, 4), MoE(1, 1, dense)), MixedLayer(GroupedAttention(*head, near, Rotary(64, 5e5)), wide)) + \
+               (MixedLayer(GroupedAttention(*head, None, Rotary(64, 5e5)), wide),) * 2
+        entries[name] = (lambda v, n=name, h=H, ls=tuple(x for i in range(0, layers, 4) for x in quad(i)): MixedConfig.vasosun(
+            "vasosun-" + n, v, h, 1e-6, ls, input_taps=4, pairs=TokenPairs(4 * v, 31, 7), logit_softcap=30.0),
+            lambda cfg, n=name, ls=like * (layers // 4): MixedConfig.zulopel("zulopel-" + n, cfg.vocab_size, cfg.hidden_size, 1e-6, ls))
+    keys = ("width", "heads", "kv_heads", "window", "kv_rank", "q_rank", "rot", "dense_ff", "experts", "identity", "top", "ff", "layers")
+    return _beside(args, "vasosun", "Vasosun 64-expert", entries, {k: dict(zip(keys, v)) for k, v in VASOSUN_SIZES.items()})
+
+
 def _hybrid(name: str, cfg, heads: int, kv_heads: int, inter: int):
     """The hybrid of softmax attention (grouped K/V heads, SwiGLU) and Gated-DeltaNet layers with a design's width and layer count."""
     from rhinoforge_b200.models.decoder import DecoderConfig
@@ -746,7 +779,8 @@ def main(argv=None) -> int:
         if int(os.environ.get("RANK", "0")) == 0:          # one line per job, also under torch.distributed.run
             print(json.dumps({"impl": "reference", "unavailable": REFERENCE_UNAVAILABLE}))
         return 0
-    out = {"decode": run, "pi05": run_pi05, "qwen3vl": run_qwen3vl, "vabarax": run_vabarax, "zulopel": run_zulopel, "kuzupel": run_kuzupel}[args.workload](args)
+    out = {"decode": run, "pi05": run_pi05, "qwen3vl": run_qwen3vl, "vabarax": run_vabarax, "zulopel": run_zulopel, "kuzupel": run_kuzupel,
+           "vasosun": run_vasosun}[args.workload](args)
     if out is not None:
         print(json.dumps(out))
     try:

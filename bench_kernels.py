@@ -622,6 +622,176 @@ def bench_windowed(hidden, heads, kv, dense, experts, top, ff, *, near=512, far=
                 report(what + " (grouped)", us, flops=4.0 * n * top * ff * hidden, **e)
 
 
+def bench_stated(hidden, heads, kv, experts, identity, top, ff, *, rank=512, q_rank=1536, dim=128, turn=64, near=512, far=2048, taps=4, batch=64,
+                 prefill=(4, 2048), dtype=torch.bfloat16) -> None:
+    """Kernels of decoders with input convolutions, delta-rule layers, window attention with a logarithmic fall, latent attention with a
+    rotated key part, and identity experts, each beside the like kernel of the other decoders at equal size."""
+    from rhinoforge_b200.ops import kernels as K
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
+    tag = dict(hidden=hidden)
+    rnd = lambda *sh: torch.randn(*sh, device="cuda", dtype=dtype)
+    f32 = lambda *sh: torch.randn(*sh, device="cuda")
+    S, Lp = prefill
+    T, hd = S * Lp, 128
+    starts, lens = i32([j * Lp for j in range(S)]), i32([Lp] * S)
+    seq, pos_p = i32([j for j in range(S) for _ in range(Lp)]), i32(list(range(Lp)) * S)
+    rows_p = lambda **kw: K.rows(pos_p, seq_of_row=seq, q_start=starts, q_len=lens, slot=i32(list(range(S))), **kw)
+    # ---- residual stream
+    nw, yw, cw = f32(hidden), f32(hidden), f32(taps, hidden)
+    for n, r in ((batch, K.rows(i32([7] * batch))), (T, rows_p())):
+        x, own, sw = f32(n, hidden), rnd(n, hidden), f32(n)
+        yg, slots = rnd(n * top, hidden), torch.randperm(n * top, device="cuda").to(torch.int32).view(n, top)
+        y1, state = rnd(n, hidden), rnd(max(n, S), taps - 1, hidden)
+        conv = dict(conv=(cw, state)) if n == batch else {}
+        carried = 4 * (taps - 1) if n == batch else 0
+        us = time_cold_us(lambda: K.stream_norm(x, r, dtype=dtype, eps=1e-6, norm_w=nw, y=yg, y_norm_w=yw, y_slots=slots, y_self=(own, sw), **conv))
+        report("stream_norm (picked rows and identity, norm of it, add, norm" + (", convolution)" if conv else ")"), us,
+               bytes_=n * hidden * (12 + 2 * top + carried), rows=n, **tag)
+        us = time_cold_us(lambda: K.stream_norm(x, r, dtype=dtype, eps=1e-6, norm_w=nw, y=y1, y_norm_w=yw, **conv))
+        report("stream_norm (norm of the output, add, norm" + (", convolution)" if conv else ")"), us, bytes_=n * hidden * (12 + carried), rows=n, **tag)
+        us = time_cold_us(lambda: K.stream_norm(x, r, dtype=dtype, eps=1e-6, y=yg, y_norm_w=yw, cast=True, y_slots=slots))
+        report("like: stream_norm (picked rows, norm of it, add)", us, bytes_=n * hidden * (10 + 2 * top), rows=n, **tag)
+        us = time_cold_us(lambda: K.stream_norm(x, r, dtype=dtype, eps=1e-6, y=y1, y_norm_w=yw, cast=True))
+        report("like: stream_norm (norm of the output, add)", us, bytes_=n * hidden * 12, rows=n, **tag)
+        if n == T:
+            us = time_cold_us(lambda: K.conv_silu(own, cw, None, state, r, max_q_len=Lp, add=True))
+            report("input convolution", us, bytes_=4.0 * n * hidden, rows=n, **tag)
+            us = time_cold_us(lambda: K.conv_silu(own, cw, nw, state, r, max_q_len=Lp))
+            report("like: conv_silu", us, bytes_=4.0 * n * hidden, rows=n, **tag)
+        del yg
+    # ---- delta rule
+    ch = heads // 2 * 2 * hd + heads * hd
+    rate, dt, hw, taps_w = f32(heads).abs(), f32(heads), f32(hd), f32(taps, ch)
+    for s_, l_ in ((1, 1), (batch, 1), (1, 4096), (S, Lp), (1, 15)):
+        n = s_ * l_
+        x, gates, z = rnd(n, ch), rnd(n, 2 * heads), rnd(n, heads * hd)
+        state, ring = f32(s_, heads, hd, hd), rnd(s_, taps, ch)
+        rr = K.rows(i32([5] * n)) if l_ == 1 else K.rows(i32(list(range(l_)) * s_), q_start=i32([j * l_ for j in range(s_)]), q_len=i32([l_] * s_))
+        kw = dict(kv_heads=heads // 2, eps=1e-6)
+        bytes_ = 8.0 * state.numel() + 2.0 * n * (ch + 2 * heads * hd)
+        e = dict(seqs=s_, length=l_, heads=heads, **tag)
+        if l_ > 1:
+            us = time_cold_us(lambda: K.conv_silu(x, taps_w, None, ring, rr, max_q_len=l_, ring=True))
+            report("short convolution", us, bytes_=4.0 * n * ch, **e)
+            us = time_cold_us(lambda: K.delta_rule(x, gates, gates[:, heads:], z, rate, dt, hw, state, rr, chunked=l_ >= 16, **kw))
+            report("delta rule, chunks and output norm" if l_ >= 16 else "delta rule, short portion", us, bytes_=bytes_, flops=6.0 * n * heads * hd * hd, **e)
+        else:
+            us = time_cold_us(lambda: K.delta_rule(x, gates, gates[:, heads:], z, rate, dt, hw, state, rr, conv=(taps_w, ring), **kw))
+            report("delta rule, decode step (convolution, norm, gate)", us, bytes_=bytes_ + 2.0 * s_ * taps * ch, **e)
+        bench_gdn(s_, l_, heads // 2, heads, dtype=dtype, timer=time_cold_us, chunked=l_ >= 16)
+        xg, cst, c16 = rnd(n, ch), rnd(s_, 3, ch), rnd(ch, 4)
+        qs, ql = (None, None) if l_ == 1 else (rr._keep[2], rr._keep[3])
+        report("like: causal_conv1d", time_cold_us(lambda: K.causal_conv1d(xg, c16, cst, q_start=qs, q_len=ql, max_q_len=l_)), bytes_=4.0 * n * ch, **e)
+        zz, w16 = rnd(n, heads * hd), rnd(hd)
+        report("like: rmsnorm_gated", time_cold_us(lambda: K.rmsnorm_gated(z, zz, w16, heads, 1e-6)), bytes_=6.0 * n * heads * hd, **e)
+    # ---- window attention
+    r1, r2, slopes = torch.rand(heads, device="cuda"), torch.rand(heads, device="cuda"), torch.rand(heads, device="cuda")
+    cols = (heads + 2 * kv) * hd
+    qn, cos, sin = f32(hd), f32(4096, 32), f32(4096, 32)
+    for n, r_of in ((1, lambda **k: K.rows(i32([far - 1]), **k)), (batch, lambda **k: K.rows(i32([far - 1] * batch), **k)), (T, rows_p)):
+        per, nseq = (max(Lp, far) + 15) // 16, S if n == T else n
+        pt = torch.randperm(nseq * per, device="cuda").to(torch.int32).view(nseq, per)
+        kp, vp = rnd(nseq * per, kv, 16, hd), rnd(nseq * per, kv, 16, hd)
+        x, r, moved = rnd(n, cols), r_of(page_table=pt), n * (2 * heads + 4 * kv) * hd * 2
+        head = dict(heads=heads, kv_heads=kv, hd=hd, eps=1e-6)
+        report("qkv_insert (growth)", time_cold_us(lambda: K.qkv_insert(x, r, kp, vp, growth=0.1, growth_every=64, **head)), bytes_=moved, rows=n, **tag)
+        report("like: qkv_insert (norms, rotation)", time_cold_us(lambda: K.qkv_insert(x, r, kp, vp, q_norm=qn, k_norm=qn, cos=cos, sin=sin, **head)), bytes_=moved, rows=n, **tag)
+        q, out = x[:, :heads * hd], rnd(n, heads * hd)
+        for what, opt in (("window and logarithmic fall", dict(slopes=r1, rates=r2)), ("like: window and slopes", dict(slopes=slopes))):
+            opt = dict(Hq=heads, Hkv=kv, hd=hd, scale=0.09, window=near, **opt)
+            if n == T:
+                us = time_cold_us(lambda: K.attention_prefill(q, out, q_start=starts, q_len=lens, kv_len=lens, max_q_len=Lp, k_pool=kp, v_pool=vp,
+                                                              page_table=pt, max_kv_len=Lp, **opt))
+                report(f"attention prefill ({what})", us, flops=4.0 * S * sum(min(i + 1, near) for i in range(Lp)) * heads * hd, rows=n, **tag)
+            else:
+                us = time_cold_us(lambda: K.attention_rows(q, r, kp, vp, max_kv=far, **opt))
+                report(f"attention by row ({what})", us, bytes_=4.0 * n * near * kv * hd + 4.0 * n * heads * hd, rows=n, **tag)
+        del kp, vp, x
+    # ---- latent attention
+    key, wide = dim + turn, rank + turn
+    ct, st = f32(4096, turn // 2), f32(4096, turn // 2)
+    lw, qw = f32(rank), f32(q_rank)
+    wa, wu = rnd(heads, rank, dim) / dim ** 0.5, rnd(heads, hd, rank) / rank ** 0.5
+    for b in (1, batch):
+        pages = (far + 15) // 16
+        pt = torch.randperm(b * pages, device="cuda").to(torch.int32).view(b, pages)
+        r = K.rows(i32([far - 1] * b), page_table=pt)
+        pool, xin = rnd(b * pages, 16, wide), rnd(b, q_rank + wide)
+        us = time_cold_us(lambda: K.latent_insert(xin[:, q_rank:], lw, pool, r, 1e-6, cos=ct, sin=st, q=xin, q_norm=qw))
+        report("latent_insert (latent, rotated part, query latent)", us, bytes_=4.0 * b * (wide + q_rank), rows=b, **tag)
+        q = rnd(b, heads, key)
+        for w_, x_, what in ((wa, q[..., :dim], "query -> latent"), (wu, rnd(b, heads, rank), "latent -> value")):
+            report(f"head_linear ({what})", time_cold_us(lambda: K.head_linear(x_, w_)), bytes_=2.0 * (w_.numel() + b * heads * (w_.shape[1] + w_.shape[2])), rows=b, **tag)
+        ql = rnd(b, heads, wide)
+        us = time_cold_us(lambda: K.latent_attention(ql, pool, r, window=0, scale=0.05, max_kv=far, vrank=rank))
+        report("latent_attn decode (rotated part)", us, bytes_=2.0 * b * (far * wide + 2 * heads * rank), flops=2.0 * b * heads * far * (wide + rank), rows=b, keys=far, **tag)
+        pl, qp = rnd(b * pages, 16, rank), rnd(b, heads, rank)
+        us = time_cold_us(lambda: K.latent_attention(qp, pl, r, window=0, scale=0.05, max_kv=far))
+        report("like: latent_attn decode", us, bytes_=2.0 * b * (far * rank + 2 * heads * rank), flops=4.0 * b * heads * far * rank, rows=b, keys=far, **tag)
+    pages = (Lp + 15) // 16
+    pt = torch.randperm(S * pages, device="cuda").to(torch.int32).view(S, pages)
+    pool, r, xin = rnd(S * pages, 16, wide), rows_p(page_table=pt), rnd(T, q_rank + wide)
+    us = time_cold_us(lambda: K.latent_insert(xin[:, q_rank:], lw, pool, r, 1e-6, cos=ct, sin=st, q=xin, q_norm=qw))
+    report("latent_insert (latent, rotated part, query latent)", us, bytes_=4.0 * T * (wide + q_rank), rows=T, **tag)
+    pl, xl = rnd(S * pages, 16, rank), rnd(T, rank)
+    report("like: latent_insert", time_cold_us(lambda: K.latent_insert(xl, lw, pl, r, 1e-6)), bytes_=4.0 * T * rank, rows=T, **tag)
+    report("latent_gather", time_cold_us(lambda: K.latent_gather(pool, r, starts, lens, T, Lp)), bytes_=4.0 * T * wide, rows=T, **tag)
+    report("like: latent_gather", time_cold_us(lambda: K.latent_gather(pl, r, starts, lens, T, Lp)), bytes_=4.0 * T * rank, rows=T, **tag)
+    hk, hv = K.latent_heads(key, hd)
+    q = rnd(T, heads * hk)
+    qv = q.view(T, heads, hk)[..., dim:dim + turn]
+    report("head_rotate", time_cold_us(lambda: K.head_rotate(qv, pos_p, ct, st)), bytes_=4.0 * T * heads * turn, rows=T, **tag)
+    kv_, oo = rnd(T, heads * (hk + hv)), rnd(T, heads * hv)
+    vis = S * Lp * (Lp + 1) // 2
+    att = dict(Hq=heads, Hkv=heads, q_start=starts, q_len=lens, kv_len=lens, max_q_len=Lp, kv_start=starts, causal=True, scale=0.05)
+    us = time_cold_us(lambda: K.attention_prefill(q, oo, hd=hk, vd=hv, k=kv_[:, :heads * hk], v=kv_[:, heads * hk:], **att))
+    report("attention over expanded keys (rotated part)", us, flops=2.0 * vis * heads * (key + hd), rows=T, **tag)
+    q1, kv1 = rnd(T, heads * hd), rnd(T, 2 * heads * hd)
+    us = time_cold_us(lambda: K.attention_prefill(q1, oo[:, :heads * hd].contiguous(), hd=hd, k=kv1[:, :heads * hd], v=kv1[:, heads * hd:], **att))
+    report("like: attention over expanded keys", us, flops=4.0 * vis * heads * hd, rows=T, **tag)
+    del q, kv_, oo, q1, kv1, pool, pl, xin, xl
+    # ---- experts
+    routed = experts + identity
+    router, bias = rnd(routed, hidden) / hidden ** 0.5, f32(routed) * (0.25 / routed)
+    pad, like_ff = (ff + 127) // 128 * 128, 2 * ff // 3 // 8 * 8
+    like_pad = (like_ff + 127) // 128 * 128
+    up, down = K.pack_weight(rnd(experts * pad, hidden) / hidden ** 0.5), K.pack_weight(rnd(hidden, experts * pad) / ff ** 0.5)
+    like_up = K.pack_weight(rnd(2 * experts * like_pad, hidden) / hidden ** 0.5, 2)
+    for n in (1, 8, batch, 256, T):
+        x = rnd(n, hidden)
+        small = n <= 256
+        plan = dict(tile_rows=(16 if n * top <= 16 * experts else 32) if small else 128, scatter=small)
+        b = K.RoutedBatch(x, router, top, correction=bias, norm_topk=False, identity=identity, **plan)
+        report("moe_router (identity experts)", time_cold_us(b.route), bytes_=2.0 * (n + routed) * hidden, rows=n, experts=routed, top=top, **tag)
+        like = K.RoutedBatch(x, router[:experts], top, correction=bias[:experts].contiguous(), **plan)
+        report("like: moe_router", time_cold_us(like.route), bytes_=2.0 * (n + experts) * hidden, rows=n, **tag)
+        like.route()
+        torch.cuda.synchronize()
+        used = int(like.ids.unique().numel())
+        e = dict(rows=n, experts=experts, used=used, ff=ff, **tag)
+        if small:
+            h = K.moe_experts(like, x, up, n=ff, k=hidden, experts=experts, expert_pad=pad, act="gelu_erf", stacked=True)
+            us = time_cold_us(lambda: K.moe_experts(like, x, up, n=ff, k=hidden, experts=experts, expert_pad=pad, act="gelu_erf", stacked=True))
+            report("experts: up, gelu", us, bytes_=2.0 * used * ff * hidden + 2.0 * n * top * ff + 2.0 * n * hidden, **e)
+            us = time_cold_us(lambda: K.moe_experts(like, x, like_up, n=like_ff, k=hidden, experts=experts, expert_pad=like_pad, dual=True))
+            report("like: experts: gate and up, silu", us, bytes_=4.0 * used * like_ff * hidden + 2.0 * n * top * like_ff + 2.0 * n * hidden, **e)
+            us = time_cold_us(lambda: K.moe_experts(like, h, down, n=hidden, k=ff, experts=experts, expert_pad=pad, gathered=False, weighted=True))
+            report("experts: down", us, bytes_=2.0 * used * ff * hidden + 2.0 * n * top * (ff + hidden), **e)
+        else:
+            xg, out, like_out = like.gather(), rnd(n * top, pad), rnd(n * top, like_pad)
+            us = time_cold_us(lambda: K.moe_grouped_gemm(xg, up, like.tiles[3:], n=pad, k=hidden, bank_rows=experts * pad, bank_k=hidden, expert_rows=pad,
+                                                         act="gelu_erf", out=out))
+            report("experts: up, gelu (grouped)", us, flops=2.0 * n * top * ff * hidden, **e)
+            us = time_cold_us(lambda: K.moe_grouped_gemm(xg, like_up, like.tiles[3:], n=like_pad, k=hidden, bank_rows=experts * like_pad, bank_k=hidden,
+                                                         expert_rows=like_pad, dual=True, act="silu_mul", out=like_out))
+            report("like: experts: gate and up, silu (grouped)", us, flops=4.0 * n * top * like_ff * hidden, **e)
+
+
+def stated() -> None:
+    bench_stated(2048, 16, 4, 16, 4, 2, 1536, q_rank=768)
+    bench_stated(4096, 32, 8, 64, 16, 6, 2112)
+
+
 def windowed() -> None:
     bench_windowed(2048, 16, 4, 8192, 16, 2, 1024)
     bench_windowed(4096, 32, 8, 16384, 64, 6, 1408)
@@ -639,7 +809,7 @@ def mixed() -> None:
 
 def main() -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("what", choices=["gemm", "attn_prefill", "attn_decode", "gdn", "suite", "sweep", "heads", "mixed", "routed", "windowed"])
+    ap.add_argument("what", choices=["gemm", "attn_prefill", "attn_decode", "gdn", "suite", "sweep", "heads", "mixed", "routed", "windowed", "stated"])
     for name, d in (("m", 64), ("n", 4096), ("k", 4096), ("seqs", 4), ("len", 2048), ("heads", 32), ("kv-heads", 8),
                     ("hd", 128), ("hk", 16), ("hv", 32)):
         ap.add_argument(f"--{name}", type=int, default=d)
@@ -669,6 +839,8 @@ def main() -> int:
         mixed()
     elif a.what == "routed":
         routed()
+    elif a.what == "stated":
+        stated()
     elif a.what == "windowed":
         windowed()
     else:

@@ -110,7 +110,7 @@ class RfAttn(C.Structure):
         ("status", C.c_void_p), ("dtype", C.c_int32),
         ("slot", C.c_void_p), ("chunk", C.c_int32), ("sink", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_int64),
         ("gate_by_head", C.c_int32), ("keep_first", C.c_int32), ("slopes", C.c_void_p), ("rates", C.c_void_p),
-        ("seq_of_row", C.c_void_p), ("pos", C.c_void_p),
+        ("seq_of_row", C.c_void_p), ("pos", C.c_void_p), ("vd", C.c_int32),
     ]
 
 

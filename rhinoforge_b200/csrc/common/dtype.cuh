@@ -82,8 +82,13 @@ __device__ __forceinline__ float gelu_tanh_f(float x) {
   float u = k0 * (x + k1 * x * x * x);
   return 0.5f * x * (1.0f + tanh_approx_f(u));
 }
+// x Phi(x) with the error function by Abramowitz and Stegun, Handbook of Mathematical Functions, 7.1.26 (absolute error 1.5e-7): half of
+// erfc(|x| / sqrt 2) is a polynomial in t times exp(-x^2 / 2), and is used as it is on the negative side, where 1 + erf would cancel.
 __device__ __forceinline__ float gelu_erf_f(float x) {
-  return 0.5f * x * (1.0f + erff(x * 0.7071067811865476f));
+  const float z = fabsf(x) * 0.7071067811865476f, t = __fdividef(1.f, fmaf(0.3275911f, z, 1.f));
+  const float poly = t * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.061405429f, -1.453152027f), 1.421413741f), -0.284496736f), 0.254829592f);
+  const float half_erfc = 0.5f * poly * __expf(-z * z);
+  return x * (x < 0.f ? half_erfc : 1.f - half_erfc);
 }
 
 __device__ __forceinline__ float relu2_f(float x) {

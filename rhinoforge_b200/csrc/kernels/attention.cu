@@ -538,7 +538,9 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 // ----------------------------------------------------------------- host -----
 static int fill_params(const RfAttn* a, AttnParams* p) {
   RF_REQUIRE(a && a->q && a->out, "attention needs q and out");
-  RF_REQUIRE(a->hd == 64 || a->hd == 128 || a->hd == 256, "attention head_dim %d (64/128/256; pad others)", a->hd);
+  const bool split_sizes = a->hd == 192 && a->vd == 128 && !a->k_pool;      // key heads larger than value heads: tcgen05 prefill over rows
+  RF_REQUIRE(split_sizes || ((a->hd == 64 || a->hd == 128 || a->hd == 256) && (a->vd == 0 || a->vd == a->hd)),
+             "attention head_dim %d, values %d (64/128/256, or 192 and 128; pad others)", a->hd, a->vd);
   RF_REQUIRE(a->Hkv > 0 && a->Hq % a->Hkv == 0, "attention heads %d / kv heads %d", a->Hq, a->Hkv);
   RF_REQUIRE((a->kv_len || a->pos) && a->num_seqs > 0, "attention needs kv_len and sequences");
   RF_REQUIRE(a->dtype == 0 || a->dtype == 1, "attention dtype");
@@ -729,7 +731,7 @@ extern "C" int rf_attn_prefill(const RfAttn* a, rf_stream_t stream) {
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   // tcgen05 kernel by default; RF_ATTN_TC=0 selects the mma.sync kernel (A/B timing)
   static const bool use_tc = [] { const char* e = getenv("RF_ATTN_TC"); return !(e && e[0] == '0'); }();
-  if (use_tc) return rf::launch_prefill_tc(a, p, s);
+  if (use_tc || a->hd == 192) return rf::launch_prefill_tc(a, p, s);
   RF_REQUIRE(!a->slot && a->chunk <= 0 && !a->sink && !a->gate && a->keep_first <= 0 && !a->slopes,
              "slots, chunks, sinks, gates, kept first positions and slopes need the tcgen05 prefill kernel");
   RF_ATTN_DISPATCH(launch_prefill)

@@ -34,26 +34,27 @@ struct alignas(8) FaCtl {
   int32_t abort_flag;
 };
 
-template <int HD> struct FaGeom {
-  static constexpr int J = HD / 64;                      // 64-column chunks of the head dimension
+// HD: size of a query / key head, VD: of a value head
+template <int HD, int VD> struct FaGeom {
+  static constexpr int J = HD / 64, JV = VD / 64;        // 64-column chunks of the heads
   static constexpr int KVB = 64;                         // kv tokens per block: small enough for TWO CTAs per SM
                                                          // (HD <= 128), whose softmax and MMA phases interleave
   static constexpr int PC = KVB / 64;                    // 64-token chunks of P
   static constexpr int kQBytes = J * kFaRows * 128;
-  static constexpr int kKBytes = J * KVB * 128;          // K (and V) of one stage
-  static constexpr int kStageBytes = 2 * kKBytes;
+  static constexpr int kKBytes = J * KVB * 128;          // K of one stage, V behind it
+  static constexpr int kStageBytes = kKBytes + JV * KVB * 128;
   static constexpr int kPBytes = PC * kFaRows * 128;
   static constexpr int kSmem = kQBytes + 2 * kStageBytes + kPBytes;
-  static constexpr int kTmemCols = HD == 256 ? 512 : 256; // 2 x KVB (S) + HD (O), rounded up to a power of two
+  static constexpr int kTmemCols = VD == 256 ? 512 : 256; // 2 x KVB (S) + VD (O), rounded up to a power of two
   static constexpr int kOCol = 2 * KVB;
 };
 
-template <typename T, int HD>
+template <typename T, int HD, int VD>
 __global__ void __launch_bounds__(kFaThreads)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, const AttnParams p) {
-  using G = FaGeom<HD>;
-  constexpr int J = G::J, KVB = G::KVB;
+  using G = FaGeom<HD, VD>;
+  constexpr int J = G::J, JV = G::JV, KVB = G::KVB;
   // No alignment slack: two CTAs of the HD <= 128 configuration fill the SM's shared memory to within 2 KB.
   // The swizzled tiles need a 1024-byte aligned base, which the runtime provides when the kernel has no
   // static shared memory; a misaligned base is reported instead of being used.
@@ -158,18 +159,19 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         // zero fill beyond the tensor, and their probabilities are forced to zero.
 #pragma unroll
         for (int w = 0; w < kPagesPerBlock; ++w) {
-          int row, col0;
+          int row, colk, colv;
           if (p.paged) {
             row = (block_pages[w] * p.Hkv + kvh) * 16;
-            col0 = 0;
+            colk = colv = 0;
           } else {
             row = p.kv_start[seq] + t0 + w * 16;
-            col0 = kvh * HD;
+            colk = kvh * HD;
+            colv = kvh * VD;
           }
 #pragma unroll
           for (int c = 0; c < J; ++c) {
-            tma_load_2d(ks + c * (KVB * 128) + w * kFaBox, &tmK, &ctl->kv_full[s], col0 + c * 64, row);
-            tma_load_2d(vs + c * (KVB * 128) + w * kFaBox, &tmV, &ctl->kv_full[s], col0 + c * 64, row);
+            tma_load_2d(ks + c * (KVB * 128) + w * kFaBox, &tmK, &ctl->kv_full[s], colk + c * 64, row);
+            if (c < JV) tma_load_2d(vs + c * (KVB * 128) + w * kFaBox, &tmV, &ctl->kv_full[s], colv + c * 64, row);
           }
         }
         issued = j + 1;
@@ -184,7 +186,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     // ------------------------------------------------------------- MMA issuer ----
     if (lane == 0 && nblk > 0) {
       const uint32_t idesc_qk = umma_idesc_f16(kFaRows, KVB, Num<T>::kFmt, 0);
-      const uint32_t idesc_pv = umma_idesc_f16(kFaRows, HD, Num<T>::kFmt, 1);
+      const uint32_t idesc_pv = umma_idesc_f16(kFaRows, VD, Num<T>::kFmt, 1);
       const uint32_t q_addr = smem_u32(qsm), p_addr = smem_u32(psm);
       bool ok = mbar_wait(&ctl->q_full, 0, kLocalWaitNs, 32);
       auto issue_qk = [&](int j) -> bool {
@@ -320,7 +322,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         const float alpha = (m_ref == -INFINITY) ? 0.f : exp2f(m_ref - m_new);
         if (j > 0) {
 #pragma unroll 1
-          for (int c0 = 0; c0 < HD; c0 += 32) {
+          for (int c0 = 0; c0 < VD; c0 += 32) {
             uint32_t ov[32];
             tmem_ld32(lane_base + (uint32_t)(G::kOCol + c0), ov);
             tmem_ld_wait();
@@ -366,14 +368,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     if (ok) {
       if (p.sink && l > 0.f) l += exp2f(p.sink[h] * kLog2e - m_ref);
       float inv = l > 0.f ? 1.f / l : 0.f;
-      const T* grow = p.gate ? reinterpret_cast<const T*>(p.gate) + (size_t)(p.q_start[seq] + qi) * p.ld_gate + (p.gate_by_head ? h : h * HD) : nullptr;
+      const T* grow = p.gate ? reinterpret_cast<const T*>(p.gate) + (size_t)(p.q_start[seq] + qi) * p.ld_gate + (p.gate_by_head ? h : h * VD) : nullptr;
       if (p.gate_by_head && grow && qi < qlen) {
         inv *= sigmoid_fast(Num<T>::to_f(grow[0]));
         grow = nullptr;
       }
-      T* orow = reinterpret_cast<T*>(p.out) + (size_t)(p.q_start[seq] + qi) * p.ldo + (size_t)h * HD;
+      T* orow = reinterpret_cast<T*>(p.out) + (size_t)(p.q_start[seq] + qi) * p.ldo + (size_t)h * VD;
 #pragma unroll 1
-      for (int c0 = 0; c0 < HD; c0 += 32) {
+      for (int c0 = 0; c0 < VD; c0 += 32) {
         uint32_t ov[32];
         if (nblk > 0) {
           tmem_ld32(lane_base + (uint32_t)(G::kOCol + c0), ov);
@@ -406,9 +408,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   if (warp == 1) tmem_dealloc(tmem_base, (uint32_t)G::kTmemCols);
 }
 
-template <typename T, int HD>
+template <typename T, int HD, int VD = HD>
 static int launch_prefill_tc_t(const RfAttn* a, const AttnParams& p, cudaStream_t s) {
-  using G = FaGeom<HD>;
+  using G = FaGeom<HD, VD>;
   CUtensorMap tmQ, tmK, tmV;
   int rc;
   if (a->k_pool) {
@@ -419,13 +421,13 @@ static int launch_prefill_tc_t(const RfAttn* a, const AttnParams& p, cudaStream_
   } else {
     rc = make_tmap_2d(&tmK, a->k, a->dtype, 2, (uint64_t)a->Hkv * a->hd, a->kv_rows_total, a->ldk, 64, 16, true);
     if (rc) return rc;
-    rc = make_tmap_2d(&tmV, a->v, a->dtype, 2, (uint64_t)a->Hkv * a->hd, a->kv_rows_total, a->ldv, 64, 16, true);
+    rc = make_tmap_2d(&tmV, a->v, a->dtype, 2, (uint64_t)a->Hkv * VD, a->kv_rows_total, a->ldv, 64, 16, true);
   }
   if (rc) return rc;
   rc = make_tmap_2d(&tmQ, a->q, a->dtype, 2, (uint64_t)a->Hq * a->hd, a->q_rows_total, a->ldq, 64, 16, true);
   if (rc) return rc;
   const size_t smem = (size_t)G::kSmem + sizeof(FaCtl);
-  auto kfn = attn_prefill_tc_kernel<T, HD>;
+  auto kfn = attn_prefill_tc_kernel<T, HD, VD>;
   RF_ALLOW_SMEM_PER_DEVICE(kfn, 227 * 1024);
   dim3 grid(ceil_div(a->max_q_len, kFaRows), a->Hq, a->num_seqs);
   RF_CUDA_CHECK(::rf::launch_k(kfn, grid, dim3(kFaThreads), smem, s, 1, tmQ, tmK, tmV, p));
@@ -440,10 +442,12 @@ int launch_prefill_tc(const RfAttn* a, const AttnParams& p, cudaStream_t s) {
   if (a->dtype == 0) {
     if (a->hd == 64) return launch_prefill_tc_t<__half, 64>(a, p, s);
     if (a->hd == 128) return launch_prefill_tc_t<__half, 128>(a, p, s);
+    if (a->hd == 192) return launch_prefill_tc_t<__half, 192, 128>(a, p, s);
     return launch_prefill_tc_t<__half, 256>(a, p, s);
   }
   if (a->hd == 64) return launch_prefill_tc_t<__nv_bfloat16, 64>(a, p, s);
   if (a->hd == 128) return launch_prefill_tc_t<__nv_bfloat16, 128>(a, p, s);
+  if (a->hd == 192) return launch_prefill_tc_t<__nv_bfloat16, 192, 128>(a, p, s);
   return launch_prefill_tc_t<__nv_bfloat16, 256>(a, p, s);
 }
 

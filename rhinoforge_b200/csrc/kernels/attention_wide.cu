@@ -244,7 +244,7 @@ using namespace rf;
 bool rf_attn_tiny_eligible(const RfAttn* a) {
   static const bool on = [] { const char* e = getenv("RF_ATTN_TINY"); return !(e && e[0] == '0'); }();
   if (!on || !a || a->k_pool || !a->k || !a->v || a->mask || a->seg_q || a->seg_k || a->chunk > 0 || a->sink || a->gate) return false;
-  if (a->hd != 64 && a->hd != 128) return false;
+  if ((a->hd != 64 && a->hd != 128) || (a->vd != 0 && a->vd != a->hd)) return false;
   if (a->ldq % 8 || a->ldk % 8 || a->ldv % 8 || a->ldo % 2) return false;
   const int max_q = a->q_len ? a->max_q_len : 1;
   return max_q > 0 && max_q <= 64 && a->max_kv_len > 0 && a->max_kv_len <= 512;

@@ -21,8 +21,8 @@ constexpr int kDrRows = 4;            // ... times 4 groups of state rows
 
 // One CTA per (head, sequence).  Warps lie side by side over blocks of 32 state columns (`col_blocks`) and over row blocks; a
 // thread holds RPT rows of four columns in registers, rows interleaved over the row groups.
-template <typename T, int RPT, bool CONV>
-__global__ void __launch_bounds__(512) delta_recurrent_kernel(const RfDelta p, int col_blocks, int row_blocks) {
+template <typename T, int RPT, bool CONV, int PER_SM>
+__global__ void __launch_bounds__(512, PER_SM) delta_recurrent_kernel(const RfDelta p, int col_blocks, int row_blocks) {
   pdl_prologue();
   extern __shared__ __align__(16) float dsm[];
   const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -46,6 +46,7 @@ __global__ void __launch_bounds__(512) delta_recurrent_kernel(const RfDelta p, i
     st[r] = live && pos0 > 0 && row < D ? *reinterpret_cast<const float4*>(S + (size_t)row * V + col) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
   const float rate = p.rate[h], dt_bias = p.dt_bias[h], q_scale = rsqrtf((float)p.dim_true);
+  const int now = CONV ? pos0 % p.taps : 0;            // ring row of the current token
   for (int t = 0; t < n; ++t) {
     const size_t row = (size_t)(q0 + t);
     const T* x = reinterpret_cast<const T*>(p.x) + row * p.ldx;
@@ -58,9 +59,12 @@ __global__ void __launch_bounds__(512) delta_recurrent_kernel(const RfDelta p, i
         const int taps = p.taps, channels = vo + p.heads * V;
         T* ring = reinterpret_cast<T*>(p.conv_state) + (size_t)slot * taps * channels + c;
         float s = f * p.conv_w[(size_t)(taps - 1) * channels + c];
-        for (int k = 1; k < taps; ++k)
-          if (pos0 - k >= 0) s += Num<T>::to_f(ring[(size_t)((pos0 - k) % taps) * channels]) * p.conv_w[(size_t)(taps - 1 - k) * channels + c];
-        ring[(size_t)(pos0 % taps) * channels] = x[c];
+#pragma unroll 3
+        for (int k = 1; k < taps; ++k) {
+          const int at = now - k + (now < k ? taps : 0);
+          if (pos0 >= k) s += Num<T>::to_f(ring[(size_t)at * channels]) * p.conv_w[(size_t)(taps - 1 - k) * channels + c];
+        }
+        ring[(size_t)now * channels] = x[c];
         f = s * sigmoid_f(s);
       }
       dsm[i] = f;
@@ -147,8 +151,12 @@ template <typename T, int RPT>
 static int launch_delta_recurrent(const RfDelta* a, int col_blocks, int row_blocks, cudaStream_t s) {
   const size_t smem = ((size_t)2 * a->dim + a->vdim + 2 * row_blocks * a->vdim + 16) * sizeof(float);
   const dim3 grid(a->heads, a->rows.num_seqs), block(32 * col_blocks * row_blocks);
-  if (a->conv_w) RF_CUDA_CHECK(::rf::launch_k(delta_recurrent_kernel<T, RPT, true>, grid, block, smem, s, 1, *a, col_blocks, row_blocks));
-  else RF_CUDA_CHECK(::rf::launch_k(delta_recurrent_kernel<T, RPT, false>, grid, block, smem, s, 1, *a, col_blocks, row_blocks));
+  constexpr int kMany = RPT <= 8 ? 2 : 1;                // decode steps with more heads than SMs: two CTAs overlap their phases
+#define RF_DR(CONV, PER_SM) RF_CUDA_CHECK(::rf::launch_k(delta_recurrent_kernel<T, RPT, CONV, PER_SM>, grid, block, smem, s, 1, *a, col_blocks, row_blocks))
+  if (!a->conv_w) RF_DR(false, 1);
+  else if (a->heads * a->rows.num_seqs > sm_count()) RF_DR(true, kMany);
+  else RF_DR(true, 1);
+#undef RF_DR
   ::rf::count_launch();
   return RF_OK;
 }

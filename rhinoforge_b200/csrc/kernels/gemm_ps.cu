@@ -53,6 +53,7 @@ struct GemmPsParams {
   const int32_t* grp;
   int grp_rt_per_expert;  // row tiles of the weight image between two experts (projection whose N axis is split by expert)
   int grp_kb_per_expert;  // k blocks of the weight image between two experts (projection whose K axis is split by expert)
+  int n_blocks;           // 128-row weight tiles of one matrix: a 256-wide column tile may end in the middle
   int kb_total;           // k blocks of a row tile of the whole weight image (stride between row tiles)
 };
 
@@ -152,12 +153,11 @@ gemm_ps_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       const int nsub = bn / 128;
       auto load_w = [&](const PsTile& t, int kb, int s) {
         uint8_t* sb = smem + (size_t)s * stage_bytes + kAStage;
-        const int rt0 = t.tn * nsub + t.rt_add;
 #pragma unroll
         for (int wt = 0; wt < kW; ++wt)
-          for (int sub = 0; sub < nsub; ++sub)
+          for (int sub = 0; sub < nsub; ++sub)             // behind the last weight tile: that tile once more, never stored
             bulk_load_1d(sb + wt * b_bytes + sub * kPsBlock,
-                         p.w_packed + ((size_t)(rt0 + sub + wt * p.dual_tiles) * p.kb_total + t.kb_add + kb) * kPsBlock,
+                         p.w_packed + ((size_t)(min(t.tn * nsub + sub, p.n_blocks - 1) + t.rt_add + wt * p.dual_tiles) * p.kb_total + t.kb_add + kb) * kPsBlock,
                          kPsBlock, &ctl->full[s]);
       };
       auto load_x = [&](const PsTile& t, int kb, int s) {
@@ -464,7 +464,7 @@ static int launch_ps(const RfGemm* g, int bn, cudaStream_t stream) {
   p.status = g->status;
   p.tma_out = tma_out ? (g->residual ? 2 : 1) : 0;
   p.M = g->M; p.N = g->N; p.k_blocks = ceil_div(g->K, kPsBK); p.bn = bn;
-  p.kb_total = p.k_blocks;
+  p.kb_total = p.k_blocks; p.n_blocks = ceil_div(g->N, 128);
   p.act = g->act; p.act_args = {g->act_limit, g->act_alpha}; p.dual_offset = g->dual_offset; p.dual_tiles = ceil_div(g->N, 128);
   p.tiles_m = ceil_div(g->M, kPsBM * MT); p.tiles_n = ceil_div(g->N, bn);
   const int stage_bytes = MT * kPsATile + (DUAL ? 2 : 1) * bn * kPsBK * 2;
@@ -535,7 +535,7 @@ static int launch_ps_grouped(const RfMoeGroupedGemm* a, cudaStream_t stream) {
   } else {
     tmO = tmA;
   }
-  const int bn = (!DUAL && a->N % 256 == 0) ? 256 : 128;
+  const int bn = !DUAL && (a->N % 256 == 0 || a->N >= 1024) ? 256 : 128;
   GemmPsParams p = {};
   p.out = a->out; p.ldo = a->ldo;
   p.row_scale = a->row_scale;
@@ -547,7 +547,7 @@ static int launch_ps_grouped(const RfMoeGroupedGemm* a, cudaStream_t stream) {
   p.band = 1;
   p.tma_out = tma_out ? 1 : 0;
   p.grp = a->tiles; p.grp_rt_per_expert = a->rt_per_expert; p.grp_kb_per_expert = a->kb_per_expert;
-  p.kb_total = a->bank_kb_total;
+  p.kb_total = a->bank_kb_total; p.n_blocks = ceil_div(a->N, 128);
   const int stage_bytes = kPsATile + (DUAL ? 2 : 1) * bn * kPsBK * 2;
   const int ctl_bytes = (int)sizeof(GemmPsCtl) + 1024 + 4 * kPsEpiBytes;
   p.stages = std::min(kPsMaxStages, (227 * 1024 - ctl_bytes) / stage_bytes);

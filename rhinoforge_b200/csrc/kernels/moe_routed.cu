@@ -550,7 +550,7 @@ __global__ void __launch_bounds__(256) moe_f32_kernel(const RfMoeExperts p) {
         const float u = acc[D - 1][i][j], limit = sh ? p.shared_limit : p.act_limit, gc = fminf(g, limit);
         v = p.act == kActClippedGlu ? gc / (1.f + expf(-p.act_alpha * gc)) * (fminf(fmaxf(u, -limit), limit) + 1.f) : g / (1.f + expf(-g)) * u;
       } else if (p.act == kActGeluErf) {
-        v = gelu_erf_f(g);
+        v = 0.5f * g * (1.f + erff(g * 0.7071067811865476f));
       }
       reinterpret_cast<float*>(p.out)[(size_t)(row0 + r) * p.ldo + n] = v * (p.slot_w ? p.slot_w[row0 + r] : 1.f);
     }
@@ -597,8 +597,14 @@ static int launch_small(const RfMoeExperts* a, cudaStream_t s) {
 
 template <typename T>
 static int dispatch_small(const RfMoeExperts* a, cudaStream_t s) {
-  if (a->tile_rows <= 16) return a->dual ? launch_small<T, 1, true, 8, 4>(a, s) : launch_small<T, 1, false, 4, 8>(a, s);
-  return a->dual ? launch_small<T, 2, true, 8, 4>(a, s) : launch_small<T, 2, false, 4, 8>(a, s);
+  // one operand: CTAs of 128 features, or of 32 where those would not fill the GPU
+  const bool narrow = (long)ceil_div(std::max(a->n, a->shared_n), 128) * a->max_tiles < 2 * sm_count();
+  if (a->tile_rows <= 16) {
+    if (a->dual) return launch_small<T, 1, true, 8, 4>(a, s);
+    return narrow ? launch_small<T, 1, false, 8, 4>(a, s) : launch_small<T, 1, false, 4, 8>(a, s);
+  }
+  if (a->dual) return launch_small<T, 2, true, 8, 4>(a, s);
+  return narrow ? launch_small<T, 2, false, 8, 4>(a, s) : launch_small<T, 2, false, 4, 8>(a, s);
 }
 
 static int check_router(const RfMoeRouter* a) {
@@ -638,7 +644,8 @@ extern "C" int rf_moe_router(const RfMoeRouter* a, rf_stream_t stream) {
     else rc2 = many ? launch_logits<__nv_bfloat16, 2, 2>(a, 1, s) : launch_logits<__nv_bfloat16, 1, 1>(a, splits, s);
     if (rc2) return rc2;
   }
-  return a->experts <= 64 ? launch_choose<2>(a, splits, s) : launch_choose<kRtLane>(a, splits, s);
+  if (a->experts <= 64) return launch_choose<2>(a, splits, s);
+  return a->experts <= 128 ? launch_choose<4>(a, splits, s) : launch_choose<kRtLane>(a, splits, s);
 }
 
 extern "C" uint64_t rf_moe_router_scratch_bytes(int rows, int experts) {

@@ -84,7 +84,7 @@ struct MixedStack {
       if (l.q_rank > 0) qout = std::max<uint64_t>(qout, (uint64_t)l.heads * l.dim);
       heads = std::max<uint64_t>(heads, l.heads);
       if (l.expand_hd > 0) {
-        kvw = std::max<uint64_t>(kvw, 2ull * l.heads * l.expand_hd);
+        kvw = std::max<uint64_t>(kvw, (uint64_t)l.heads * (l.expand_hd + l.vdim));
         past = std::max<uint64_t>(past, l.window > 0 ? l.window - 1 : cfg.max_seq_len);
       }
     }
@@ -276,7 +276,7 @@ static int latent_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedF
     const int32_t* kv_len = plan->kv_len + grp.seq0;
     void* ctx = s.at(s.off_ctx);
     uint8_t* kv = s.at<uint8_t>(s.off_kv);
-    const int KD = w.heads * w.expand_hd, KV = 2 * KD;
+    const int KD = w.heads * w.expand_hd, KV = KD + VD;
     rc = rf_latent_gather(w.st.latent_pool, ctx, &g, kv_start, kv_len, R, grp.max_len, c.dtype, st);
     if (rc) return rc;
     rc = linear(s, ctx, R, w.w_expand, kv, KV, grp.total, KV, R, kActNone, st);
@@ -284,7 +284,7 @@ static int latent_attention(MixedStack& s, const RfMixedLayer& w, const RfMixedF
     RfAttn a = {};
     a.q = queries; a.ldq = ldq; a.out = mix; a.ldo = VD; a.q_rows_total = T;     // q_start holds rows of the whole batch
     a.k = kv; a.v = kv + (size_t)KD * e; a.ldk = KV; a.ldv = KV; a.kv_rows_total = grp.total;
-    a.num_seqs = grp.seqs; a.Hq = w.heads; a.Hkv = w.heads; a.hd = w.expand_hd;
+    a.num_seqs = grp.seqs; a.Hq = w.heads; a.Hkv = w.heads; a.hd = w.expand_hd; a.vd = w.vdim;
     a.q_start = g.q_start; a.q_len = g.q_len; a.kv_start = kv_start; a.kv_len = kv_len;
     a.max_q_len = grp.max_q; a.max_kv_len = grp.max_len; a.causal = 1; a.window = w.window > 0 ? w.window : 0;
     a.scale = w.scale; a.status = s.status(); a.dtype = c.dtype;
@@ -731,7 +731,7 @@ extern "C" int rf_mixed_set_layer(int64_t h, int32_t layer, const RfMixedLayer* 
     RF_REQUIRE(w->plain > 0 && w->plain % 8 == 0 && w->rot >= 0 && w->rot % 2 == 0 && w->rot_pad >= w->rot && w->rot_pad % 16 == 0 &&
                    w->plain + (w->rot + 7) / 8 * 8 <= w->dim && (w->rot == 0 || (w->cos && w->sin)), "layer %d: rotated part", layer);
     RF_REQUIRE(w->in_dim >= (w->q_rank > 0 ? w->q_rank : w->heads * w->dim) + (w->shares ? 0 : w->rank + w->rot_pad), "layer %d: input projection rows", layer);
-    RF_REQUIRE(w->expand_hd == 0 || (w->w_expand && w->dim == w->expand_hd && w->vdim == w->expand_hd && s.cfg.dtype != kF32),
+    RF_REQUIRE(w->expand_hd == 0 || (w->w_expand && w->dim == w->expand_hd && (w->vdim == w->expand_hd || (w->expand_hd == 192 && w->vdim == 128)) && s.cfg.dtype != kF32),
                "layer %d: expanded heads", layer);
   } else if (w->mixer == RF_MIXER_ATTENTION) {
     RF_REQUIRE(w->dim == w->vdim && w->kv_heads > 0 && w->heads % w->kv_heads == 0 && w->dim_true > 0 && w->dim_true <= w->dim &&

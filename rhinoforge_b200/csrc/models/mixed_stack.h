@@ -60,7 +60,7 @@ typedef struct RfMixedState {
 typedef struct RfMixedLayer {
   int32_t mixer, heads, dim, vdim, vdim_true;
   int32_t rank, rank_true, window;      // attention: window <= 0: unlimited
-  int32_t expand_hd;                    // 64 / 128 / 256: portions expand K and V to heads of this size (== dim == vdim)
+  int32_t expand_hd;                    // 64 / 128 / 256: portions expand K and V to heads of this size (== dim == vdim), or 192: values of 128
   int32_t inter;                        // 0: the layer has no feed-forward
   int32_t act;                          // RfMixedAct (clipped GLU: w_up holds gate rows, then up rows)
   float scale;
@@ -72,7 +72,7 @@ typedef struct RfMixedLayer {
   const float* latent_norm;
   const void* w_absorb;                 // [heads, rank, plain]: query -> latent space
   const void* w_unabsorb;               // [heads, vdim, rank]: latent space -> value
-  const void* w_expand;                 // [2 * heads * expand_hd, rank + rot_pad]: keys of all heads (the rotated part copied), then values
+  const void* w_expand;                 // [heads * (expand_hd + vdim), rank + rot_pad]: keys of all heads (the rotated part copied), then values
   int32_t plain;                        // unrotated dimensions of a query head (multiple of 8); the rotated ones lie behind them
   int32_t q_rank, q_rank_true;          // > 0: queries go through a latent of this size
   int32_t rot, rot_pad;                 // rotated key part that all heads share: size and columns in the cache

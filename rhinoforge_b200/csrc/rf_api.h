@@ -264,6 +264,7 @@ typedef struct RfAttn {
   // rf_attn_decode by row: with `pos`, query row r is position pos[r] of sequence seq_of_row[r] (null: r) and sees what its
   // chunk or window leaves of everything up to itself; kv_len is not used and num_seqs counts rows.
   const int32_t* seq_of_row; const int32_t* pos;
+  int32_t vd;               // size of a value head (0: hd); contiguous rows with hd = 192 take 128, out is [rows, Hq * vd]
 } RfAttn;
 int rf_attn_prefill(const RfAttn* a, rf_stream_t stream);
 int rf_attn_decode(const RfAttn* a, rf_stream_t stream);

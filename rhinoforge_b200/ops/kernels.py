@@ -418,7 +418,7 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, *, Hq: int, Hkv: int, 
                       seg_k: Optional[torch.Tensor] = None, scale: float = 0.0,
                       status: Optional[torch.Tensor] = None, max_kv_len: int = 0, slot: Optional[torch.Tensor] = None, chunk: int = 0,
                       sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_by_head: bool = False,
-                      keep_first: int = 0, slopes: Optional[torch.Tensor] = None, rates: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      keep_first: int = 0, slopes: Optional[torch.Tensor] = None, rates: Optional[torch.Tensor] = None, vd: int = 0) -> torch.Tensor:
     """Flash-style attention over ``q`` rows [tokens, Hq*hd]; KV from the paged pool or from
     contiguous ``k``/``v`` [rows, Hkv*hd] (may be column slices of a packed qkv buffer).
     ``max_kv_len``: a host-side bound on ``kv_len`` (0: unknown); short contiguous problems (at most 64 query rows per
@@ -426,13 +426,14 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, *, Hq: int, Hkv: int, 
     Paged form: ``slot`` names every sequence's page-table row, ``chunk`` limits every position to its own chunk, ``sink`` ``[Hq]``
     adds ``exp(sink)`` to the softmax denominators, the result is multiplied by ``sigmoid(gate)`` (``gate_by_head``: ``[rows, Hq]``),
     the first ``keep_first`` positions stay visible behind a window or chunk, ``slopes`` ``[Hq]`` times the distance, or with ``rates``
-    ``[Hq]`` times ``ln(1 + rate * distance)``, is taken off the scores."""
+    ``[Hq]`` times ``ln(1 + rate * distance)``, is taken off the scores.  ``vd``: size of the value heads, 128 beside key heads of 192
+    (contiguous form)."""
     a = N.RfAttn()
     a.gate_by_head, a.keep_first, a.slopes = int(gate_by_head), keep_first, _ptr(slopes)
     a.rates = _ptr(rates)
     a.q, a.ldq, a.out, a.ldo = q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0)
     a.q_rows_total = q.shape[0]
-    a.num_seqs, a.Hq, a.Hkv, a.hd = q_len.numel(), Hq, Hkv, hd
+    a.num_seqs, a.Hq, a.Hkv, a.hd, a.vd = q_len.numel(), Hq, Hkv, hd, vd
     if k_pool is not None:
         a.k_pool, a.v_pool, a.pool_pages = k_pool.data_ptr(), v_pool.data_ptr(), k_pool.shape[0]
         a.page_table, a.pt_stride = _i32(page_table), page_table.stride(0)
@@ -705,6 +706,11 @@ def latent_gather(pool: torch.Tensor, r, kv_start: torch.Tensor, kv_len: torch.T
                                      C.c_void_p(_i32(kv_len)), pool.shape[2], max_len, dtype_code_any(pool.dtype), _stream()),
             "rf_latent_gather")
     return out
+
+
+def latent_heads(key: int, value: int):
+    """Head sizes ``(keys, values)`` in which the tcgen05 prefill attention takes expanded latent heads; ``(0, 0)``: it does not."""
+    return next(((a, b) for a, b in ((64, 64), (128, 128), (192, 128), (256, 256)) if key <= a and value <= b), (0, 0))
 
 
 def latent_attention(q: torch.Tensor, pool: torch.Tensor, r, *, window: int, scale: float, max_kv: int, vrank: int = 0) -> torch.Tensor:

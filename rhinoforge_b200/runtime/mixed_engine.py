@@ -208,10 +208,9 @@ class MixedDecoderEngine(DecoderEngine):
         R, P = latent_layout(m)
         rot, plain = m.rot.dims if m.rot is not None else 0, pad_to(m.dim, 8)
         key = plain + pad_to(rot, 8)                          # a head: plain dimensions, then rotated ones
-        big = max(key, m.vdim)
         # heads of the tcgen05 prefill attention; without one (fp32, very wide heads) every row attends in the latent space
-        hd = next((x for x in (64, 128, 256) if big <= x), 0) if not self.fp32 and m.scale > 0 else 0
-        D, VD = hd or key, hd or pad_to(m.vdim, 8)
+        hd, hv = K.latent_heads(key, m.vdim) if not self.fp32 and m.scale > 0 else (0, 0)
+        D, VD = hd or key, hv or pad_to(m.vdim, 8)
         lw.mixer, lw.dim, lw.vdim, lw.vdim_true = 0, D, VD, m.vdim
         lw.rank, lw.rank_true, lw.window, lw.scale, lw.expand_hd = R, m.kv_rank, m.window or 0, m.scale, hd
         lw.plain, lw.rot, lw.rot_pad, lw.shares = plain, rot, P, int(m.kv_from is not None)
@@ -241,11 +240,11 @@ class MixedDecoderEngine(DecoderEngine):
         lw.w_unabsorb = self._plain(uv).data_ptr()
         if hd:
             # keys of a head are a map of the latent and a copy of the rotated part, values a map of the latent
-            expand = uk.new_zeros((2, m.heads, hd, R + P))
-            expand[0, :, :plain, :R], expand[1, :, :, :R] = uk.view(m.heads, plain, R), uv.view(m.heads, hd, R)
+            keys = uk.new_zeros((m.heads, hd, R + P))
+            keys[:, :plain, :R] = uk.view(m.heads, plain, R)
             for i in range(rot):
-                expand[0, :, plain + i, R + i] = 1.0
-            lw.w_expand = self._linear(expand.view(2 * m.heads * hd, R + P)).data_ptr()
+                keys[:, plain + i, R + i] = 1.0
+            lw.w_expand = self._linear(torch.cat((keys.view(m.heads * hd, R + P), _pad2(uv, m.heads * hv, R + P)), 0)).data_ptr()
         o = g(p + "o")
         o = _pad_heads(o.t().contiguous(), m.heads, m.vdim, VD).t()
         lw.w_o, lw.out_dim = self._linear(_pad2(o, H, m.heads * VD)).data_ptr(), m.heads * VD

@@ -173,6 +173,26 @@ def test_cached_rows_hold_the_latent_and_the_rotated_part(dtype, rank, rot):
     assert torch.equal(pool, before)
 
 
+@pytest.mark.parametrize("dtype", [BF16, F16])
+@pytest.mark.parametrize("size", [0, 70])
+def test_prefill_attention_with_keys_wider_than_values(dtype, size):
+    """Keys of 192 and values of 128 as column blocks of one buffer, ragged sequences with cached rows ahead of the portion."""
+    lens, total, heads, rnd = [130, 1, 64, 40], [200, 33, 64, 41], 3, gen(10)
+    q, kv = rnd(sum(lens), heads * 192).to("cuda", dtype), rnd(sum(total), heads * (192 + 128)).to("cuda", dtype)
+    starts, kv_starts = [sum(lens[:i]) for i in range(4)], [sum(total[:i]) for i in range(4)]
+    out, status = torch.zeros(sum(lens), heads * 128, dtype=dtype, device="cuda"), torch.zeros(8, dtype=torch.int32, device="cuda")
+    K().attention_prefill(q, out, Hq=heads, Hkv=heads, hd=192, vd=128, q_start=i32(*starts), q_len=i32(*lens), kv_len=i32(*total), max_q_len=130,
+                          kv_start=i32(*kv_starts), k=kv[:, :heads * 192], v=kv[:, heads * 192:], window=size, scale=0.1, status=status)
+    assert int(status[0]) == 0
+    kk, vv = (t.double().cpu().view(sum(total), heads, -1) for t in (kv[:, :heads * 192], kv[:, heads * 192:]))
+    for s, (n, t) in enumerate(zip(lens, total)):
+        for i in range(0, n, 7):
+            at, lo = t - n + i, max(0, t - n + i - size + 1) if size else 0
+            rows = slice(kv_starts[s] + lo, kv_starts[s] + at + 1)
+            p = torch.softmax(torch.einsum("hd,jhd->hj", q[starts[s] + i].double().cpu().view(heads, 192), kk[rows]) * 0.1, -1)
+            close(out[starts[s] + i].view(heads, 128), torch.einsum("hj,jhd->hd", p, vv[rows]), dtype)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads", [1, 17, 40])
 @pytest.mark.parametrize("rank,vrank", [(48, 32), (128, 64), (176, 160), (192, 128), (320, 256), (512, 448), (576, 512), (640, 512)])
