@@ -402,6 +402,16 @@ def test_single_operand_experts(dtype, E, identity, k, ff, H, T, tile):
         close(got[t], want, dtype, 2.0)
 
 
+@pytest.mark.parametrize("M", [4, 200, 700])
+def test_exact_gelu_of_the_gemms_keeps_its_small_values(M):
+    """The negative side, where one plus the error function cancels: relative error down to where results vanish."""
+    x = torch.linspace(-5.0, 5.0, M * 64).view(M, 64).to("cuda", BF16)
+    w = torch.eye(64).repeat(4, 1).to("cuda", BF16)
+    got = K().gemm(x, K().pack_weight(w), packed_shape=(256, 64), act="gelu_erf").double().cpu()
+    want = (x.double().cpu() * 0.5 * torch.erfc(-x.double().cpu() / math.sqrt(2.0))).repeat(1, 4)
+    torch.testing.assert_close(got, want, rtol=2e-2, atol=2e-7)
+
+
 def test_invalid_options_are_refused_on_the_host():
     from rhinoforge_b200.api.errors import RPUBackendError
     pt = page_table(1, 1)
